@@ -86,7 +86,7 @@ class Model:
 
     @property
     def portable(self) -> bool:
-        return not hasattr(self.model, "fused_linears")
+        return not hasattr(self.model, "forward_paged")
 
     def _generator(self):
         if self._gen is None:

@@ -24,6 +24,14 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-ffp-contract=off", "-pthread"]   # no FMA contraction: byte-exact quantisers
 
 
+# sources (csrc/*.cu) that a product entry point can be built from alone, for a checkout where nothing is compiled yet
+COMPONENTS = {
+    "hybrid": ("attention_tc", "gemm_2sm", "gemm_tcgen05", "gemv", "latent_attn", "postnorm", "ssm"),
+    "decoder": ("attention", "attention_tc", "decode_mega", "elementwise", "gemm_2sm", "gemm_tcgen05", "gemv",
+                "grouped_gemm", "moe_quant"),
+}
+
+
 def _nvcc() -> str:
     for c in (os.environ.get("NVCC"), shutil.which("nvcc"), "/usr/local/cuda/bin/nvcc"):
         if c and os.path.exists(c):
@@ -131,6 +139,26 @@ def build_native(force: bool = False, verbose: bool = False) -> dict:
         print("\n".join(log))
     out["log"] = "\n".join(log)
     return out
+
+
+def build_component(name: str) -> str:
+    """Compile and link ``lib/libpmetal_b200_<name>.so`` from the sources of one component (objects are shared with the full
+    build); returns its path."""
+    os.makedirs(OBJDIR, exist_ok=True)
+    write_abi_header()
+    headers = glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
+    nvcc, log, jobs, objs = _nvcc(), [], [], []
+    for stem in COMPONENTS[name]:
+        src, obj = os.path.join(CSRC, stem + ".cu"), os.path.join(OBJDIR, stem + ".o")
+        objs.append(obj)
+        if _stale(obj, [src] + headers):
+            jobs.append([nvcc] + NVCC_FLAGS + ["-c", src, "-o", obj])
+    so = os.path.join(LIBDIR, f"libpmetal_b200_{name}.so")
+    with ThreadPoolExecutor(max_workers=min(8, max(len(jobs), 1))) as ex:
+        list(ex.map(lambda c: _run(c, log), jobs))
+    if jobs or _stale(so, objs):
+        _run([nvcc, "-shared", "-o", so] + objs + ["-gencode", "arch=compute_100a,code=sm_100a"], log)
+    return so
 
 
 if __name__ == "__main__":

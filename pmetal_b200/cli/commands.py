@@ -346,6 +346,9 @@ def _load_for_inference(a):
     if getattr(a, "minimal", False):
         a.backend = "minimal"
     lora = getattr(a, "lora", None)
+    refused = [f for f in ("lora", "fp8", "adapter", "draft_model", "ep") if getattr(a, f, None)]
+    if not hasattr(model, "fused_linears") and (refused or getattr(a, "tp", 1) > 1):
+        raise SystemExit(f"error: {args.model_type} models take no --" + (refused or ["tp"])[0].replace("_", "-"))
     if lora:
         from ..lora import apply_lora
         from ..lora.adapter import load_adapter, load_adapter_config
@@ -476,6 +479,11 @@ def _paged_cache_options(a, model, num_blocks: int) -> dict:
     import torch
     from ..models.kv_cache import BLOCK, select_cache_mode
     cfg = model.cfg
+    if getattr(model, "slotted_cache", False):
+        if a.kv_quant or a.kv_k_bits or a.kv_v_bits or a.kv_turboquant or a.kv_turboquant_preset or a.kv_quant_preset or a.kv_window:
+            print(f"note: {cfg.model_type} keeps latents and states in the model's type; the --kv-* options have no effect",
+                  file=sys.stderr)
+        return {}
     weight_bytes = sum(p.numel() * p.element_size() for p in model.parameters())
     kv16 = 2 * cfg.num_hidden_layers * num_blocks * BLOCK * cfg.num_key_value_heads * cfg.head_dim * 2
     dev = model.embed_tokens.device

@@ -15,6 +15,7 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
+#include "elem.cuh"
 #include "host_util.cuh"
 
 #include "pdl.cuh"
@@ -53,9 +54,28 @@ struct GemvParams {
   float am_scale, am_offset;
   int qblock;                    // elements per absmax block (multiple of 32)
   int fp4;
+  const float* bias;             // [N_w] fp32 or null, added before the gate
+  int clamped;                   // gate of the SWIGLU variants: 0 silu(g) * u, 1 the clamped unit of elem.cuh
+  float glu_limit, glu_beta, glu_shift;
+  float* y_f32;                  // [M, ldy] instead of y
 };
 
 __device__ __forceinline__ float gv_silu(float v) { return v / (1.f + __expf(-v)); }
+
+// Output element n (and its up half v2) from the accumulated sums: scale, bias, gate, residual.
+template <bool SWIGLU>
+__device__ __forceinline__ void gv_finish(const GemvParams& p, int m, int n, float v, float v2) {
+  v *= p.alpha;
+  if (p.bias) v += p.bias[n];
+  if (SWIGLU) {
+    v2 *= p.alpha;
+    if (p.bias) v2 += p.bias[n + p.N];
+    v = p.clamped ? clamped_glu(v, v2, p.glu_limit, p.glu_beta, p.glu_shift) : gv_silu(v) * v2;
+  }
+  if (p.residual) v += __bfloat162float(p.residual[static_cast<long long>(m) * p.ldr + n]);
+  if (p.y_f32) p.y_f32[static_cast<long long>(m) * p.ldy + n] = v;
+  else p.y[static_cast<long long>(m) * p.ldy + n] = __float2bfloat16(v);
+}
 
 // MR rows of x, C output columns per warp at a time, KU 16-byte weight loads in flight per column and lane.
 template <int MR, int C, int KU, bool SWIGLU>
@@ -228,10 +248,7 @@ __global__ void __launch_bounds__(kGvThreads) gemv_kernel(const GemvParams p) {
           v += lora(n);
           if (SWIGLU) v2 += lora(n + p.N);
         }
-        v *= p.alpha;
-        if (SWIGLU) v = gv_silu(v) * (v2 * p.alpha);
-        if (p.residual) v += __bfloat162float(p.residual[static_cast<long long>(m) * p.ldr + n]);
-        p.y[static_cast<long long>(m) * p.ldy + n] = __float2bfloat16(v);
+        gv_finish<SWIGLU>(p, m, n, v, v2);
       }
     }
   }
@@ -337,10 +354,7 @@ __device__ __forceinline__ void gv_tile_epilogue(const GemvParams& p, const floa
         v += gv_lora(p, m, n);
         if (SWIGLU) v2 += gv_lora(p, m, n + p.N);
       }
-      v *= p.alpha;
-      if (SWIGLU) v = gv_silu(v) * (v2 * p.alpha);
-      if (p.residual) v += __bfloat162float(p.residual[static_cast<long long>(m) * p.ldr + n]);
-      p.y[static_cast<long long>(m) * p.ldy + n] = __float2bfloat16(v);
+      gv_finish<SWIGLU>(p, m, n, v, v2);
     }
   }
 }
@@ -559,11 +573,13 @@ static int launch_gemv(const GemvParams& p, cudaStream_t st) {
 
 using namespace pm;
 
-// Returns 0, a negative argument error, or a CUDA error code. K % 8 == 0, row strides % 8 == 0, M <= 16,
-// M * cols-per-warp <= 32.
-extern "C" int pm_gemv(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps, const void* residual,
-                       int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha, const void* t, int ldt,
-                       const float* lora_b, int r, const int* seg_end, cudaStream_t st) {
+// As pm_gemv with the epilogue of models that have biases and clamped gated units: bias [N_w] fp32 (nullable) is added to
+// the scaled products; with swiglu and clamped != 0 the pair becomes min(g, limit) * sigmoid(beta min(g, limit)) *
+// (clamp(u, -limit, limit) + shift); out_f32 != 0: y is fp32.
+extern "C" int pm_gemv_ex(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps,
+                          const void* residual, int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha,
+                          const void* t, int ldt, const float* lora_b, int r, const int* seg_end, const float* bias,
+                          int clamped, float limit, float beta, float shift, int out_f32, cudaStream_t st) {
   if (M < 1 || M > 16 || N < 1 || K < 8 || (K % 8) || (ldx % 8) || (ldw % 8)) return -1;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return -2;
   if (norm_w && (reinterpret_cast<uintptr_t>(norm_w) & 15)) return -2;
@@ -574,6 +590,8 @@ extern "C" int pm_gemv(const void* x, int ldx, const void* w, int ldw, const voi
   p.norm_w = static_cast<const __nv_bfloat16*>(norm_w); p.eps = eps;
   p.residual = static_cast<const __nv_bfloat16*>(residual); p.ldr = ldr;
   p.y = static_cast<__nv_bfloat16*>(y); p.ldy = ldy;
+  if (out_f32) p.y_f32 = static_cast<float*>(y);
+  p.bias = bias; p.clamped = clamped; p.glu_limit = limit; p.glu_beta = beta; p.glu_shift = shift;
   p.M = M; p.N = N; p.K = K; p.swiglu = swiglu; p.alpha = alpha;
   p.t = static_cast<const __nv_bfloat16*>(t); p.ldt = ldt; p.lora_b = lora_b; p.r = r;
   for (int i = 0; i < 4; ++i) p.seg_end[i] = seg_end ? seg_end[i] : 0x7fffffff;
@@ -601,6 +619,15 @@ extern "C" int pm_gemv(const void* x, int ldx, const void* w, int ldw, const voi
   if (M <= 4) return wide ? launch_gemv<4, 4, 4, false>(p, st) : launch_gemv<4, 1, 8, false>(p, st);
   if (M <= 8) return wide ? launch_gemv<8, 2, 4, false>(p, st) : launch_gemv<8, 1, 8, false>(p, st);
   return wide ? launch_gemv<16, 2, 2, false>(p, st) : launch_gemv<16, 1, 4, false>(p, st);
+}
+
+// Returns 0, a negative argument error, or a CUDA error code. K % 8 == 0, row strides % 8 == 0, M <= 16,
+// M * cols-per-warp <= 32.
+extern "C" int pm_gemv(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps, const void* residual,
+                       int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha, const void* t, int ldt,
+                       const float* lora_b, int r, const int* seg_end, cudaStream_t st) {
+  return pm_gemv_ex(x, ldx, w, ldw, norm_w, eps, residual, ldr, y, ldy, M, N, K, swiglu, alpha, t, ldt, lora_b, r, seg_end,
+                    nullptr, 0, 0.f, 0.f, 0.f, 0, st);
 }
 
 // 4-bit weights: qdata holds N_w * K / 2 bytes (two codes per byte, first element in the high nibble), absmax one fp32

@@ -1,0 +1,652 @@
+// Multi-head latent attention over a paged cache. Per token and layer the cache holds one row [c: R | k_r: D_r | 0 ..]
+// (W = R + D_r rounded up to 16 columns): the normed latent and one rotated key part shared by all heads. With per-head
+// up-projections W_uk (D_n x R) and W_uv (D_v x R), head h scores  (q_n . W_uk c + q_r . k_r) * scale  and reads out
+// W_uv (sum_j p_j c_j).
+//
+// Short portions (decode) move W_uk to the query side: q_l = W_uk^T q_n once per token and head, then every head attends
+// to the cached rows themselves (keys: all W columns, values: the first R), so a step streams the cache once for all
+// heads:
+//   latent_prep_kernel      norm of the latent, rotation of k_r and of the queries' rotated part, cache append
+//   latent_absorb_kernel    [q_l | q_r | 0] rows of width W
+//   latent_attn_mma_kernel  bf16, split over key pages: 16 or 32 (token, head) rows share each 64-key page in shared
+//                           memory; S by mma.sync with the keys cut over the warps, P V with the columns cut over the warps
+//   latent_attn_row_kernel  any type and size, one (token, head) row per CTA (fp32 models)
+//   latent_up_kernel        joins the splits and applies W_uv
+// Longer portions expand keys and values of the visible rows with one GEMM and run the flash-attention kernels of
+// attention_tc.cu; latent_gather_kernel / latent_assemble_kernel lay out their operands (128 channels per head, zero
+// padded).
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <math_constants.h>
+#include <stdint.h>
+#include "elem.cuh"
+#include "host_util.cuh"
+#include "mma_sync.cuh"
+#include "pmetal_b200.h"
+
+namespace pm {
+
+constexpr int kPage = 64;
+
+// One CTA per token. qd [tokens, ld]: H heads of [D_n | D_r], then (own != 0) the down-projection [R | D_r].
+template <typename T>
+__global__ void latent_prep_kernel(T* __restrict__ qd, long long ld, const float* __restrict__ norm_w, float eps,
+                                   const float* __restrict__ cs, const float* __restrict__ sn, int H, int dn, int dr, int rank,
+                                   int own, T* __restrict__ cache, int W, const long long* __restrict__ slots) {
+  const long long t = blockIdx.x;
+  T* row = qd + t * ld;
+  const int half = dr / 2;
+  const float* c = cs + t * half;
+  const float* s = sn + t * half;
+  for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
+    const int h = i / half, j = i - h * half;
+    T* p = row + h * (dn + dr) + dn + 2 * j;
+    const float a = to_f(p[0]), b = to_f(p[1]);
+    put(p, a * c[j] - b * s[j]);
+    put(p + 1, b * c[j] + a * s[j]);
+  }
+  if (!own) return;
+  const T* d = row + H * (dn + dr);
+  T* dst = cache + slots[t] * W;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
+    const float v = to_f(d[i]);
+    ss = fmaf(v, v, ss);
+  }
+  const float r = 1.f / sqrtf(block_sum(ss) / static_cast<float>(rank) + eps);
+  for (int i = threadIdx.x; i < rank; i += blockDim.x) put(dst + i, to_f(d[i]) * r * norm_w[i]);
+  for (int j = threadIdx.x; j < half; j += blockDim.x) {
+    const float a = to_f(d[rank + 2 * j]), b = to_f(d[rank + 2 * j + 1]);
+    put(dst + rank + 2 * j, a * c[j] - b * s[j]);
+    put(dst + rank + 2 * j + 1, b * c[j] + a * s[j]);
+  }
+}
+
+// grid (column tiles of 128, H, token groups of kAbsTok per sequence, sequences folded into z). The CTA computes 128
+// columns of q_l for up to kAbsTok tokens of one head; the last column tile copies the rotated part and zeroes the rest.
+constexpr int kAbsTok = 8;
+template <typename T>
+__global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict__ qd, long long ld, const T* __restrict__ wuk,
+                                                            int H, int dn, int dr, int rank, int W,
+                                                            const int* __restrict__ q_start, const int* __restrict__ c_start,
+                                                            const int* __restrict__ q_lens, int tok_tiles,
+                                                            T* __restrict__ out) {
+  extern __shared__ float abs_q[];           // [kAbsTok][dn]
+  const int h = blockIdx.y, seq = blockIdx.z / tok_tiles, t0 = (blockIdx.z % tok_tiles) * kAbsTok;
+  const int len = q_lens[seq];
+  if (t0 >= len) return;
+  const int n_tok = min(kAbsTok, len - t0);
+  const long long q0 = q_start[seq] + t0, o0 = c_start[seq] + t0;
+  if (blockIdx.x == gridDim.x - 1) {
+    const int tail = W - rank;
+    for (int i = threadIdx.x; i < n_tok * tail; i += 128) {
+      const int t = i / tail, j = i - t * tail;
+      put(out + ((o0 + t) * H + h) * W + rank + j, j < dr ? to_f(qd[(q0 + t) * ld + h * (dn + dr) + dn + j]) : 0.f);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < kAbsTok * dn; i += 128) {
+    const int t = i / dn, j = i - t * dn;
+    abs_q[i] = t < n_tok ? to_f(qd[(q0 + t) * ld + h * (dn + dr) + j]) : 0.f;
+  }
+  __syncthreads();
+  const int c = blockIdx.x * 128 + threadIdx.x;
+  if (c >= rank) return;
+  float acc[kAbsTok];
+#pragma unroll
+  for (int t = 0; t < kAbsTok; ++t) acc[t] = 0.f;
+  const T* w = wuk + static_cast<long long>(h) * dn * rank + c;
+#pragma unroll 8
+  for (int j = 0; j < dn; ++j) {
+    const float wv = to_f(w[static_cast<long long>(j) * rank]);
+#pragma unroll
+    for (int t = 0; t < kAbsTok; ++t) acc[t] = fmaf(abs_q[t * dn + j], wv, acc[t]);
+  }
+#pragma unroll
+  for (int t = 0; t < kAbsTok; ++t)
+    if (t < n_tok) put(out + ((o0 + t) * H + h) * W + c, acc[t]);
+}
+
+struct LatentParams {
+  const void* q;             // [compact tokens, H, W]
+  const void* cache;         // [pages, 64, W]
+  const int* block_table;
+  const int* seq_lens;
+  const int* c_start;        // first row of each sequence in the compact buffers (q, part_o, part_ml)
+  const int* q_lens;
+  float* part_o;             // [split][compact tokens * H][rank], not normalised
+  float* part_ml;            // [split][compact tokens * H][2]: maximum (log2 domain), sum
+  int max_blocks, H, W, rank, n_split, row_tiles;
+  long long rows;            // compact tokens * H
+  float scale_log2;          // scale * log2(e)
+};
+
+// One (token, head) row per CTA, all keys, any type. grid (rows of the longest portion, sequences).
+template <typename T>
+__global__ void __launch_bounds__(128) latent_attn_row_kernel(const LatentParams p) {
+  extern __shared__ float lr_smem[];
+  float* sq = lr_smem;               // [W]
+  float* so = sq + p.W;              // [rank]
+  float* ss = so + p.rank;           // [64]
+  const int seq = blockIdx.y, len = p.q_lens[seq], r = blockIdx.x;
+  if (r >= len * p.H) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long row = static_cast<long long>(p.c_start[seq]) * p.H + r;
+  const int n_keys = p.seq_lens[seq] - len + r / p.H + 1;
+  const T* q = static_cast<const T*>(p.q) + row * p.W;
+  for (int i = threadIdx.x; i < p.W; i += 128) sq[i] = to_f(q[i]) * p.scale_log2;
+  for (int i = threadIdx.x; i < p.rank; i += 128) so[i] = 0.f;
+  float m = -CUDART_INF_F, l = 0.f;
+  for (int j0 = 0; j0 < n_keys; j0 += kPage) {
+    const int n = min(kPage, n_keys - j0);
+    const T* page = static_cast<const T*>(p.cache) +
+                    static_cast<long long>(p.block_table[static_cast<long long>(seq) * p.max_blocks + j0 / kPage]) * kPage * p.W;
+    __syncthreads();
+    for (int k = warp; k < n; k += 4) {
+      float v = 0.f;
+      for (int i = lane; i < p.W; i += 32) v = fmaf(sq[i], to_f(page[static_cast<long long>(k) * p.W + i]), v);
+      v = warp_sum(v);
+      if (lane == 0) ss[k] = v;
+    }
+    __syncthreads();
+    const float a = lane < n ? ss[lane] : -CUDART_INF_F, b = lane + 32 < n ? ss[lane + 32] : -CUDART_INF_F;
+    float mx = fmaxf(a, b);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float m_new = fmaxf(m, mx);
+    const float corr = exp2f(m - m_new), pa = exp2f(a - m_new), pb = exp2f(b - m_new);
+    l = l * corr + warp_sum(pa + pb);
+    m = m_new;
+    __syncthreads();
+    if (warp == 0) {
+      ss[lane] = pa;
+      ss[lane + 32] = pb;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < p.rank; i += 128) {
+      float o = so[i] * corr;
+#pragma unroll 4
+      for (int k = 0; k < n; ++k) o = fmaf(ss[k], to_f(page[static_cast<long long>(k) * p.W + i]), o);
+      so[i] = o;
+    }
+  }
+  for (int i = threadIdx.x; i < p.rank; i += 128) p.part_o[row * p.rank + i] = so[i];
+  if (threadIdx.x == 0) {
+    p.part_ml[row * 2] = m;
+    p.part_ml[row * 2 + 1] = l;
+  }
+}
+
+// 8 warps. MT: 16-row tiles of (token, head) rows; NT: 8-column tiles of the latent per warp.
+template <int MT, int NT>
+__global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams p) {
+  extern __shared__ __align__(16) uint8_t lm_smem[];
+  constexpr int RT = 16 * MT;
+  constexpr int kLdS = kPage + 4, kLdP = kPage + 8;
+  const int ld = p.W + 8;
+  __nv_bfloat16* sKV = reinterpret_cast<__nv_bfloat16*>(lm_smem);           // [2][64][ld]
+  __nv_bfloat16* sQ = sKV + 2 * kPage * ld;                                  // [RT][ld]
+  __nv_bfloat16* sP = sQ + RT * ld;                                          // [RT][kLdP]
+  float* sS = reinterpret_cast<float*>(sP + RT * kLdP);                      // [RT][kLdS]
+  float* sCorr = sS + RT * kLdS;                                             // [RT]
+  const int seq = blockIdx.x / p.row_tiles, row0 = (blockIdx.x % p.row_tiles) * RT, split = blockIdx.y;
+  const int len = p.q_lens[seq], n_rows = len * p.H;
+  if (row0 >= n_rows) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, t4 = lane & 3;
+  const int prior = p.seq_lens[seq] - len;
+  const int last_row = min(row0 + RT, n_rows) - 1;
+  const int n_keys = prior + last_row / p.H + 1;                             // keys the last row of the tile sees
+  const int n_blocks = (n_keys + kPage - 1) / kPage;
+  const int per = (n_blocks + p.n_split - 1) / p.n_split;
+  const int b0 = split * per, b1 = min(n_blocks, b0 + per);
+  const long long base_row = static_cast<long long>(p.c_start[seq]) * p.H + row0;
+  const long long part_base = split * p.rows + base_row;
+  if (b0 >= b1) {
+    for (int i = threadIdx.x; i < RT && row0 + i < n_rows; i += 256) {
+      p.part_ml[(part_base + i) * 2] = -CUDART_INF_F;
+      p.part_ml[(part_base + i) * 2 + 1] = 0.f;
+    }
+    return;
+  }
+  const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.cache);
+  const int* bt = p.block_table + static_cast<long long>(seq) * p.max_blocks;
+  const int chunks = p.W / 8;
+  auto load_page = [&](int b, int buf) {
+    const __nv_bfloat16* src = cache + static_cast<long long>(bt[b]) * kPage * p.W;
+    __nv_bfloat16* dst = sKV + buf * kPage * ld;
+    const int valid = n_keys - b * kPage;
+    for (int i = threadIdx.x; i < kPage * chunks; i += 256) {
+      const int r = i / chunks, c = (i - r * chunks) * 8;
+      ms_cp16(ms_addr(dst + r * ld + c), src + static_cast<long long>(r) * p.W + c, r < valid);
+    }
+    ms_commit();
+  };
+  {
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + base_row * p.W;
+    for (int i = threadIdx.x; i < RT * chunks; i += 256) {
+      const int r = i / chunks, c = (i - r * chunks) * 8;
+      const bool ok = row0 + r < n_rows;
+      ms_cp16(ms_addr(sQ + r * ld + c), q + static_cast<long long>(ok ? r : 0) * p.W + c, ok);
+    }
+  }
+  load_page(b0, 0);
+  float acc[MT][NT][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
+  // softmax rows of this warp: RT / 8 consecutive rows
+  constexpr int kRows = RT / 8;
+  float m_run[kRows], l_run[kRows];
+#pragma unroll
+  for (int i = 0; i < kRows; ++i) { m_run[i] = -CUDART_INF_F; l_run[i] = 0.f; }
+  const uint32_t aQ = ms_addr(sQ), aP = ms_addr(sP);
+  const int n8 = (p.rank + 7) / 8;
+
+  for (int b = b0; b < b1; ++b) {
+    const int buf = (b - b0) & 1;
+    if (b + 1 < b1) {
+      load_page(b + 1, buf ^ 1);
+      ms_wait<1>();
+    } else {
+      ms_wait<0>();
+    }
+    __syncthreads();
+    const uint32_t aK = ms_addr(sKV + buf * kPage * ld);
+    // scores: warp w owns keys 8 w .. 8 w + 7 of the page
+    float s[MT][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[i][e] = 0.f;
+#pragma unroll 4
+    for (int k = 0; k < p.W; k += 16) {
+      uint32_t fb0, fb1;
+      ms_ldsm2(aK + static_cast<uint32_t>(((warp * 8 + (lane & 7)) * ld + k + ((lane >> 3) & 1) * 8) * 2), fb0, fb1);
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        uint32_t fa[4];
+        ms_ldsm4(ms_a_at(aQ, ld, i * 16, k, lane), fa);
+        ms_mma(s[i], fa, fb0, fb1);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf)
+        *reinterpret_cast<float2*>(sS + (i * 16 + g4 + 8 * hf) * kLdS + warp * 8 + 2 * t4) =
+            make_float2(s[i][2 * hf], s[i][2 * hf + 1]);
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kRows; ++i) {
+      const int r = warp * kRows + i, lim = prior + (row0 + r) / p.H;        // last key this row sees
+      const float2 v = *reinterpret_cast<const float2*>(sS + r * kLdS + 2 * lane);
+      const int j = b * kPage + 2 * lane;
+      const float x0 = j <= lim ? v.x * p.scale_log2 : -CUDART_INF_F, x1 = j + 1 <= lim ? v.y * p.scale_log2 : -CUDART_INF_F;
+      float mx = fmaxf(x0, x1);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float m_new = fmaxf(m_run[i], mx), m_use = m_new == -CUDART_INF_F ? 0.f : m_new;
+      const float corr = exp2f(m_run[i] - m_use), e0 = exp2f(x0 - m_use), e1 = exp2f(x1 - m_use);
+      l_run[i] = l_run[i] * corr + warp_sum(e0 + e1);
+      m_run[i] = m_new;
+      *reinterpret_cast<uint32_t*>(sP + r * kLdP + 2 * lane) = pack_bf16(e0, e1);
+      if (lane == 0) sCorr[r] = corr;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < MT; ++i) {
+      const float c0 = sCorr[i * 16 + g4], c1 = sCorr[i * 16 + g4 + 8];
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        acc[i][j][0] *= c0; acc[i][j][1] *= c0;
+        acc[i][j][2] *= c1; acc[i][j][3] *= c1;
+      }
+    }
+#pragma unroll
+    for (int kk = 0; kk < kPage; kk += 16) {
+      uint32_t fp[MT][4];
+#pragma unroll
+      for (int i = 0; i < MT; ++i) ms_ldsm4(ms_a_at(aP, kLdP, i * 16, kk, lane), fp[i]);
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const int tile = warp + 8 * j;
+        if (tile < n8) {
+          uint32_t fb0, fb1;
+          ms_ldsm2_t(aK + static_cast<uint32_t>(((kk + (lane & 15)) * ld + tile * 8) * 2), fb0, fb1);
+#pragma unroll
+          for (int i = 0; i < MT; ++i) ms_mma(acc[i][j], fp[i], fb0, fb1);
+        }
+      }
+    }
+    __syncthreads();                  // the page buffer, scores and probabilities may be overwritten
+  }
+#pragma unroll
+  for (int i = 0; i < kRows; ++i) {
+    const int r = warp * kRows + i;
+    if (lane == 0 && row0 + r < n_rows) {
+      p.part_ml[(part_base + r) * 2] = m_run[i];
+      p.part_ml[(part_base + r) * 2 + 1] = l_run[i];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = i * 16 + g4 + ((e & 2) ? 8 : 0), c = (warp + 8 * j) * 8 + 2 * t4 + (e & 1);
+        if (row0 + r < n_rows && c < p.rank) p.part_o[(part_base + r) * p.rank + c] = acc[i][j][e];
+      }
+}
+
+// out[token, h, v] = W_uv[h, v, :] . (joined splits of row (token, h)). grid (H, token groups per sequence folded with
+// the sequences); a CTA joins up to kUpTok rows of one head and shares the weight rows between them.
+constexpr int kUpTok = 4;
+template <typename T>
+__global__ void __launch_bounds__(256) latent_up_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                        const T* __restrict__ wuv, const int* __restrict__ q_start,
+                                                        const int* __restrict__ c_start, const int* __restrict__ q_lens,
+                                                        int tok_tiles, int H, int dv, int rank, int n_split, long long rows,
+                                                        T* __restrict__ out, long long ldo) {
+  extern __shared__ float up_o[];            // [kUpTok][rank]
+  __shared__ float coef[kUpTok][64];
+  const int h = blockIdx.x, seq = blockIdx.y / tok_tiles, t0 = (blockIdx.y % tok_tiles) * kUpTok;
+  const int len = q_lens[seq];
+  if (t0 >= len) return;
+  const int n_tok = min(kUpTok, len - t0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long q0 = q_start[seq] + t0, c0 = c_start[seq] + t0;
+  if (warp < n_tok) {                        // n_split <= 64: two splits per lane
+    const long long row = (c0 + warp) * H + h;
+    float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
+    if (lane < n_split) { m0 = part_ml[(lane * rows + row) * 2]; l0 = part_ml[(lane * rows + row) * 2 + 1]; }
+    if (lane + 32 < n_split) { m1 = part_ml[((lane + 32) * rows + row) * 2]; l1 = part_ml[((lane + 32) * rows + row) * 2 + 1]; }
+    float mx = fmaxf(m0, m1);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float e0 = l0 > 0.f ? exp2f(m0 - mx) : 0.f, e1 = l1 > 0.f ? exp2f(m1 - mx) : 0.f;
+    const float inv = 1.f / warp_sum(e0 * l0 + e1 * l1);
+    coef[warp][lane] = e0 * inv;
+    coef[warp][lane + 32] = e1 * inv;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < kUpTok * rank; i += 256) {
+    const int t = i / rank, c = i - t * rank;
+    float v = 0.f;
+    if (t < n_tok) {
+      const long long row = (c0 + t) * H + h;
+      for (int s = 0; s < n_split; ++s) {
+        const float w = coef[t][s];
+        if (w != 0.f) v = fmaf(w, part_o[(s * rows + row) * rank + c], v);
+      }
+    }
+    up_o[i] = v;
+  }
+  __syncthreads();
+  for (int r = warp; r < dv; r += 8) {
+    const T* w = wuv + (static_cast<long long>(h) * dv + r) * rank;
+    float acc[kUpTok];
+#pragma unroll
+    for (int t = 0; t < kUpTok; ++t) acc[t] = 0.f;
+#pragma unroll 4
+    for (int c = lane; c < rank; c += 32) {
+      const float wv = to_f(w[c]);
+#pragma unroll
+      for (int t = 0; t < kUpTok; ++t) acc[t] = fmaf(wv, up_o[t * rank + c], acc[t]);
+    }
+#pragma unroll
+    for (int t = 0; t < kUpTok; ++t) acc[t] = warp_sum(acc[t]);
+    if (lane < n_tok) {
+      float v = acc[0];
+#pragma unroll
+      for (int t = 1; t < kUpTok; ++t)
+        if (lane == t) v = acc[t];
+      put(out + (q0 + lane) * ldo + h * dv + r, v);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------- expanded keys and values
+// lat [n, R8] (R8 >= rank, zero padded) = latents of one sequence's first n positions, read through its block table row.
+__global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ table, int n, int W,
+                                     int rank, int r8, __nv_bfloat16* __restrict__ lat) {
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < static_cast<long long>(n) * r8;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int j = static_cast<int>(i / r8), c = static_cast<int>(i - static_cast<long long>(j) * r8);
+    const __nv_bfloat16* src = cache + (static_cast<long long>(table[j / kPage]) * kPage + j % kPage) * W;
+    lat[i] = c < rank ? src[c] : __float2bfloat16(0.f);
+  }
+}
+__global__ void latent_gather8_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ table, int n, int W,
+                                      int rank, __nv_bfloat16* __restrict__ lat) {
+  const int per = rank / 8;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < static_cast<long long>(n) * per;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int j = static_cast<int>(i / per), c = static_cast<int>(i - static_cast<long long>(j) * per) * 8;
+    const __nv_bfloat16* src = cache + (static_cast<long long>(table[j / kPage]) * kPage + j % kPage) * W;
+    *reinterpret_cast<uint4*>(lat + static_cast<long long>(j) * rank + c) = *reinterpret_cast<const uint4*>(src + c);
+  }
+}
+
+// Query / key / value operands of the 128-channel attention kernels, zero padded. kv [n, ldkv]: H heads of D_n key
+// channels, then H heads of D_v value channels. blockIdx.y: 0 = queries (n_q rows of qd), 1 = keys, 2 = values.
+// A thread writes 8 channels.
+__global__ void latent_assemble_kernel(const __nv_bfloat16* __restrict__ qd, long long ldq, int n_q,
+                                       const __nv_bfloat16* __restrict__ kv, long long ldkv, int n,
+                                       const __nv_bfloat16* __restrict__ cache, const int* __restrict__ table, int W, int rank,
+                                       int H, int dn, int dr, int dv, __nv_bfloat16* __restrict__ q128,
+                                       __nv_bfloat16* __restrict__ k128, __nv_bfloat16* __restrict__ v128) {
+  const int what = blockIdx.y;
+  const long long rows = static_cast<long long>(what == 0 ? n_q : n) * H;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < rows * 16;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i >> 4;
+    const int c0 = static_cast<int>(i & 15) * 8, h = static_cast<int>(r % H);
+    const long long t = r / H;
+    __nv_bfloat16* dst = (what == 0 ? q128 : (what == 1 ? k128 : v128)) + r * 128 + c0;
+    const __nv_bfloat16 *a, *b = nullptr;      // channels [0, na) from a, [na, nb) from b
+    int na, nb;
+    if (what == 0) {
+      a = qd + t * ldq + h * (dn + dr);
+      na = nb = dn + dr;
+    } else if (what == 1) {
+      a = kv + t * ldkv + h * dn;
+      b = cache + (static_cast<long long>(table[t / kPage]) * kPage + t % kPage) * W + rank;
+      na = dn;
+      nb = dn + dr;
+    } else {
+      a = kv + t * ldkv + static_cast<long long>(H) * dn + h * dv;
+      na = nb = dv;
+    }
+    uint32_t w[4];
+    const bool from_a = c0 + 8 <= na, from_b = b && c0 >= na && c0 + 8 <= nb;
+    const __nv_bfloat16* src = from_a ? a + c0 : b + (c0 - na);
+    if ((from_a || from_b) && !(reinterpret_cast<uintptr_t>(src) & 15)) {
+      *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
+      continue;
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float v[2];
+#pragma unroll
+      for (int f = 0; f < 2; ++f) {
+        const int c = c0 + 2 * e + f;
+        v[f] = c < na ? __bfloat162float(a[c]) : (c < nb ? __bfloat162float(b[c - na]) : 0.f);
+      }
+      w[e] = pack_bf16(v[0], v[1]);
+    }
+    *reinterpret_cast<uint4*>(dst) = make_uint4(w[0], w[1], w[2], w[3]);
+  }
+}
+
+// Rows of [n, H, 128] back to [n, H * dv] (row stride ldo).
+__global__ void latent_take_kernel(const __nv_bfloat16* __restrict__ o128, int n, int H, int dv, __nv_bfloat16* __restrict__ out,
+                                   long long ldo) {
+  const long long total = static_cast<long long>(n) * H * dv;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int c = static_cast<int>(i % dv);
+    const long long r = i / dv;
+    out[(r / H) * ldo + (r % H) * dv + c] = o128[r * 128 + c];
+  }
+}
+
+static size_t latent_mma_smem(int mt, int W) {
+  const size_t rt = 16 * mt, ld = W + 8;
+  return (2 * kPage * ld + rt * ld + rt * (kPage + 8)) * 2 + (rt * (kPage + 4) + rt) * 4;
+}
+static int latent_mma_tiles(int H, int W) {      // 16-row tiles per CTA, 0: not covered
+  if (H > 16 && latent_mma_smem(2, W) <= 220 * 1024) return 2;
+  return latent_mma_smem(1, W) <= 220 * 1024 ? 1 : 0;
+}
+
+template <int MT, int NT>
+static int latent_mma_launch(const LatentParams& p, dim3 grid, size_t smem, cudaStream_t st) {
+  static DeviceMax configured;
+  if (smem > configured.get()) {
+    const cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                               static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured.set(smem);
+  }
+  latent_attn_mma_kernel<MT, NT><<<grid, 256, smem, st>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace pm
+
+using namespace pm;
+
+// qd [n, ld]: the queries' rotated parts are turned in place; with cache != null the down-projection behind the queries is
+// normed / rotated and written to row slots[t] of cache [.., W]. cs / sn [n, dr / 2].
+extern "C" int pm_latent_prep(void* qd, int f32, long long ld, const float* norm_w, float eps, const float* cs,
+                              const float* sn, int n, int H, int dn, int dr, int rank, void* cache, int W,
+                              const long long* slots, cudaStream_t st) {
+  if (n < 0 || H < 1 || dn < 0 || dr < 0 || (dr & 1) || rank < 1 || W < rank + dr) return -1;
+  if (ld < static_cast<long long>(H) * (dn + dr) + (cache ? rank + dr : 0)) return -2;
+  if (n == 0) return 0;
+  const int own = cache != nullptr;
+  if (f32)
+    latent_prep_kernel<float><<<n, 128, 0, st>>>(static_cast<float*>(qd), ld, norm_w, eps, cs, sn, H, dn, dr, rank, own,
+                                                 static_cast<float*>(cache), W, slots);
+  else
+    latent_prep_kernel<__nv_bfloat16><<<n, 128, 0, st>>>(static_cast<__nv_bfloat16*>(qd), ld, norm_w, eps, cs, sn, H, dn, dr,
+                                                         rank, own, static_cast<__nv_bfloat16*>(cache), W, slots);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Whether the tensor-core kernel covers H heads over rows of W columns with `rank` value columns.
+extern "C" int pm_latent_mma_supported(int H, int W, int rank) {
+  return W % 16 == 0 && rank <= 512 && latent_mma_tiles(H, W) > 0;
+}
+
+// Attention of short portions in the latent space. qd as pm_latent_prep leaves it, wuk [H * dn, rank], wuv [H * dv, rank],
+// cache [pages, 64, W]. Sequence i covers rows q_start[i] .. of qd and out and rows c_start[i] .. of the work buffers
+// q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32, part_ml [n_split, n_tok * H, 2] fp32 (n_tok: tokens of the
+// listed sequences). out [.., ldo]: H * dv columns. max_q: longest of q_lens.
+// n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
+extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void* wuk, const void* wuv, const void* cache,
+                              const int* block_table, const int* seq_lens, const int* q_start, const int* c_start,
+                              const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr, int dv, int rank, int W,
+                              int n_split, float scale, void* q_lat, float* part_o, float* part_ml, void* out,
+                              long long ldo, cudaStream_t st) {
+  if (H < 1 || rank < 1 || W < rank + dr || dv < 1 || n_split < 1 || n_split > 64 || ldo < static_cast<long long>(H) * dv)
+    return -1;
+  if (n_seq < 1 || max_q < 1) return 0;
+  const bool mma = !f32 && pm_latent_mma_supported(H, W, rank);
+  if (!mma && n_split != 1) return -2;
+  const size_t sm_abs = static_cast<size_t>(kAbsTok) * dn * 4, sm_row = (static_cast<size_t>(W) + rank + kPage) * 4,
+               sm_up = static_cast<size_t>(kUpTok) * rank * 4;
+  if (sm_abs > 48 * 1024 || (!mma && sm_row > 48 * 1024) || sm_up > 46 * 1024) return -3;
+  const int abs_tiles = (max_q + kAbsTok - 1) / kAbsTok, up_tiles = (max_q + kUpTok - 1) / kUpTok;
+  if (static_cast<long long>(abs_tiles) * n_seq > 65535 || static_cast<long long>(up_tiles) * n_seq > 65535) return -4;
+  const dim3 g_abs((rank + 127) / 128 + 1, H, abs_tiles * n_seq);
+  if (f32)
+    latent_absorb_kernel<float><<<g_abs, 128, sm_abs, st>>>(static_cast<const float*>(qd), ld, static_cast<const float*>(wuk),
+                                                            H, dn, dr, rank, W, q_start, c_start, q_lens, abs_tiles,
+                                                            static_cast<float*>(q_lat));
+  else
+    latent_absorb_kernel<__nv_bfloat16><<<g_abs, 128, sm_abs, st>>>(
+        static_cast<const __nv_bfloat16*>(qd), ld, static_cast<const __nv_bfloat16*>(wuk), H, dn, dr, rank, W, q_start,
+        c_start, q_lens, abs_tiles, static_cast<__nv_bfloat16*>(q_lat));
+  cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) return static_cast<int>(e);
+  LatentParams p{};
+  p.q = q_lat; p.cache = cache; p.block_table = block_table; p.seq_lens = seq_lens; p.c_start = c_start; p.q_lens = q_lens;
+  p.part_o = part_o; p.part_ml = part_ml; p.max_blocks = max_blocks; p.H = H; p.W = W; p.rank = rank; p.n_split = n_split;
+  p.rows = static_cast<long long>(n_tok) * H;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  if (mma) {
+    const int mt = latent_mma_tiles(H, W), rt = 16 * mt, n8 = (rank + 7) / 8, nt = (n8 + 7) / 8;
+    p.row_tiles = (max_q * H + rt - 1) / rt;
+    const dim3 grid(p.row_tiles * n_seq, n_split);
+    const size_t smem = latent_mma_smem(mt, W);
+    int rc;
+    if (mt == 1)
+      rc = nt <= 1 ? latent_mma_launch<1, 1>(p, grid, smem, st) : nt <= 2 ? latent_mma_launch<1, 2>(p, grid, smem, st)
+         : nt <= 4 ? latent_mma_launch<1, 4>(p, grid, smem, st) : latent_mma_launch<1, 8>(p, grid, smem, st);
+    else
+      rc = nt <= 1 ? latent_mma_launch<2, 1>(p, grid, smem, st) : nt <= 2 ? latent_mma_launch<2, 2>(p, grid, smem, st)
+         : nt <= 4 ? latent_mma_launch<2, 4>(p, grid, smem, st) : latent_mma_launch<2, 8>(p, grid, smem, st);
+    if (rc) return rc;
+  } else {
+    const dim3 grid(max_q * H, n_seq);
+    if (f32) latent_attn_row_kernel<float><<<grid, 128, sm_row, st>>>(p);
+    else latent_attn_row_kernel<__nv_bfloat16><<<grid, 128, sm_row, st>>>(p);
+    e = cudaGetLastError();
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  const dim3 g_up(H, up_tiles * n_seq);
+  if (f32)
+    latent_up_kernel<float><<<g_up, 256, sm_up, st>>>(part_o, part_ml, static_cast<const float*>(wuv), q_start, c_start,
+                                                      q_lens, up_tiles, H, dv, rank, n_split, p.rows, static_cast<float*>(out), ldo);
+  else
+    latent_up_kernel<__nv_bfloat16><<<g_up, 256, sm_up, st>>>(part_o, part_ml, static_cast<const __nv_bfloat16*>(wuv), q_start,
+                                                              c_start, q_lens, up_tiles, H, dv, rank, n_split, p.rows,
+                                                              static_cast<__nv_bfloat16*>(out), ldo);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// lat [n, r8] bf16 = latents of positions 0 .. n - 1 of the sequence whose block table row is `table` (zero padded).
+extern "C" int pm_latent_gather(const void* cache, const int* table, int n, int W, int rank, int r8, void* lat,
+                                cudaStream_t st) {
+  if (n < 0 || rank < 1 || r8 < rank || W < rank) return -1;
+  if (n == 0) return 0;
+  const bool vec = rank == r8 && rank % 8 == 0 && W % 8 == 0;
+  long long grid = (static_cast<long long>(n) * (vec ? rank / 8 : r8) + 255) / 256;
+  if (grid > num_sms() * 16) grid = num_sms() * 16;
+  if (vec)
+    latent_gather8_kernel<<<static_cast<int>(grid), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(cache), table, n, W, rank,
+                                                                  static_cast<__nv_bfloat16*>(lat));
+  else
+    latent_gather_kernel<<<static_cast<int>(grid), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(cache), table, n, W, rank,
+                                                                 r8, static_cast<__nv_bfloat16*>(lat));
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Operands [.., H, 128] bf16 of the flash-attention kernels for n_q queries and n keys of one sequence; dn + dr <= 128,
+// dv <= 128. qd: the first query row; kv [n, ldkv] = [keys: H * dn | values: H * dv].
+extern "C" int pm_latent_assemble(const void* qd, long long ldq, int n_q, const void* kv, long long ldkv, int n,
+                                  const void* cache, const int* table, int W, int rank, int H, int dn, int dr, int dv,
+                                  void* q128, void* k128, void* v128, cudaStream_t st) {
+  if (n_q < 1 || n < 1 || H < 1 || dn + dr > 128 || dv > 128 || W < rank + dr) return -1;
+  long long grid = (static_cast<long long>(n > n_q ? n : n_q) * H * 16 + 255) / 256;
+  if (grid > num_sms() * 16) grid = num_sms() * 16;
+  latent_assemble_kernel<<<dim3(static_cast<int>(grid), 3), 256, 0, st>>>(
+      static_cast<const __nv_bfloat16*>(qd), ldq, n_q, static_cast<const __nv_bfloat16*>(kv), ldkv, n,
+      static_cast<const __nv_bfloat16*>(cache), table, W, rank, H, dn, dr, dv, static_cast<__nv_bfloat16*>(q128),
+      static_cast<__nv_bfloat16*>(k128), static_cast<__nv_bfloat16*>(v128));
+  return static_cast<int>(cudaGetLastError());
+}
+
+// out [n, ldo] (H * dv columns) = the first dv channels of every head of o128 [n, H, 128].
+extern "C" int pm_latent_take(const void* o128, int n, int H, int dv, void* out, long long ldo, cudaStream_t st) {
+  if (n < 1 || H < 1 || dv < 1 || dv > 128) return -1;
+  long long grid = (static_cast<long long>(n) * H * dv + 255) / 256;
+  if (grid > num_sms() * 16) grid = num_sms() * 16;
+  latent_take_kernel<<<static_cast<int>(grid), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(o128), n, H, dv,
+                                                             static_cast<__nv_bfloat16*>(out), ldo);
+  return static_cast<int>(cudaGetLastError());
+}

@@ -170,6 +170,13 @@ int pm_gemm_bf16(const void* A, int a_mn, int lda, int a_rows, const void* B, in
     ws_cnt, long long ws_cnt_len, int* status, cudaStream_t stream);
 
 // ---------------------------------------------------------------- gemv.cu
+// As pm_gemv with the epilogue of models that have biases and clamped gated units: bias [N_w] fp32 (nullable) is added to
+// the scaled products; with swiglu and clamped != 0 the pair becomes min(g, limit) * sigmoid(beta min(g, limit)) *
+// (clamp(u, -limit, limit) + shift); out_f32 != 0: y is fp32.
+int pm_gemv_ex(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps, const void* residual,
+    int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha, const void* t, int ldt, const float*
+    lora_b, int r, const int* seg_end, const float* bias, int clamped, float limit, float beta, float shift, int
+    out_f32, cudaStream_t st);
 // Returns 0, a negative argument error, or a CUDA error code. K % 8 == 0, row strides % 8 == 0, M <= 16,
 // M * cols-per-warp <= 32.
 int pm_gemv(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps, const void* residual,
@@ -194,6 +201,33 @@ int pm_grouped_gemm(int mode, const void* a, int lda, const void* b, int ldb, vo
 // bn (32, 64, 128) is the token tile: experts with more rows take several passes over their weights.
 int pm_grouped_gemm_skinny(const void* x, int ldx, int rows, const void* w, int ldw, void* y, int ldy, const int*
     off, int E, int N, int K, int bn, int swiglu, float alpha, int* status, cudaStream_t stream);
+
+// ---------------------------------------------------------------- latent_attn.cu
+// qd [n, ld]: the queries' rotated parts are turned in place; with cache != null the down-projection behind the queries is
+// normed / rotated and written to row slots[t] of cache [.., W]. cs / sn [n, dr / 2].
+int pm_latent_prep(void* qd, int f32, long long ld, const float* norm_w, float eps, const float* cs, const float*
+    sn, int n, int H, int dn, int dr, int rank, void* cache, int W, const long long* slots, cudaStream_t st);
+// Whether the tensor-core kernel covers H heads over rows of W columns with `rank` value columns.
+int pm_latent_mma_supported(int H, int W, int rank);
+// Attention of short portions in the latent space. qd as pm_latent_prep leaves it, wuk [H * dn, rank], wuv [H * dv, rank],
+// cache [pages, 64, W]. Sequence i covers rows q_start[i] .. of qd and out and rows c_start[i] .. of the work buffers
+// q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32, part_ml [n_split, n_tok * H, 2] fp32 (n_tok: tokens of the
+// listed sequences). out [.., ldo]: H * dv columns. max_q: longest of q_lens.
+// n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
+int pm_latent_attn(const void* qd, int f32, long long ld, const void* wuk, const void* wuv, const void* cache,
+    const int* block_table, const int* seq_lens, const int* q_start, const int* c_start, const int* q_lens, int
+    n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr, int dv, int rank, int W, int n_split, float
+    scale, void* q_lat, float* part_o, float* part_ml, void* out, long long ldo, cudaStream_t st);
+// lat [n, r8] bf16 = latents of positions 0 .. n - 1 of the sequence whose block table row is `table` (zero padded).
+int pm_latent_gather(const void* cache, const int* table, int n, int W, int rank, int r8, void* lat, cudaStream_t
+    st);
+// Operands [.., H, 128] bf16 of the flash-attention kernels for n_q queries and n keys of one sequence; dn + dr <= 128,
+// dv <= 128. qd: the first query row; kv [n, ldkv] = [keys: H * dn | values: H * dv].
+int pm_latent_assemble(const void* qd, long long ldq, int n_q, const void* kv, long long ldkv, int n, const void*
+    cache, const int* table, int W, int rank, int H, int dn, int dr, int dv, void* q128, void* k128, void* v128,
+    cudaStream_t st);
+// out [n, ldo] (H * dv columns) = the first dv channels of every head of o128 [n, H, 128].
+int pm_latent_take(const void* o128, int n, int H, int dv, void* out, long long ldo, cudaStream_t st);
 
 // ---------------------------------------------------------------- mhc.cu
 // x [T, n, C] bf16; either phi [n C, n^2 + 2n] fp32 (dot products formed here) or raw [T, ld_raw] fp32 = x . phi computed by
@@ -250,6 +284,22 @@ int pm_gguf_dequant_bf16(const void* src, void* dst, long long n, int type, cuda
 int pm_fp8_quant(const void* x, void* q, float* scales, long long n, cudaStream_t st);
 int pm_fp8_dequant(const void* q, const float* scales, void* y, long long n, cudaStream_t st);
 
+// ---------------------------------------------------------------- postnorm.cu
+// xf [n, width] fp32 = table[ids] * scale, xc the same in the table's type (nullable). f32: the table is fp32, else bf16.
+int pm_embed_scale(const long long* ids, const void* table, int f32, float scale, int n, int width, float* xf,
+    void* xc, cudaStream_t st);
+// of / oc [n, width] (fp32 / compute type, each nullable) = LN(alpha * x + y + bias) * w + b for the n rows listed in
+// `rows` (nullable: row i). y [.., ldy] and bias are nullable; without y the row is x itself. of may be x when rows is
+// null.
+int pm_post_layernorm(const float* x, const void* y, int f32, long long ldy, const float* bias, float alpha, const
+    float* w, const float* b, float eps, int n, int width, const long long* rows, float* of, void* oc, cudaStream_t
+    st);
+// gu [n, ld]: gate columns [0, ff), up columns [ff, 2 ff); bias fp32 [2 ff] or null -> out [n, ff].
+int pm_clamped_glu(const void* gu, int f32, long long ld, const float* bias, int n, int ff, float limit, float
+    beta, float shift, void* out, cudaStream_t st);
+// cos / sin [n, half] fp32 of pos * freq (freq fp64 [half] on the device).
+int pm_rope_table_f64(const int* pos, const double* freq, int n, int half, float* cs, float* sn, cudaStream_t st);
+
 // ---------------------------------------------------------------- sampling.cu
 int pm_sample(const void* logits, int is_bf16, long long ld, int rows, int vocab, const int* counts, const int*
     count_rows, const float* temperature, const int* top_k, const float* top_p, const float* min_p, const float*
@@ -259,6 +309,28 @@ int pm_spec_verify(const float* target, const float* draft, const int* tokens, i
     temperature, const unsigned long long* seeds, unsigned long long step, int* n_accepted, int* next_token,
     cudaStream_t st);
 int pm_count_tokens(int* counts, const int* count_rows, const int* tokens, int rows, int vocab, cudaStream_t st);
+
+// ---------------------------------------------------------------- ssm.cu
+// Token-by-token recurrence with the convolution inside. u [tokens, ldu]; conv_w [taps][conv], conv_b, dt_bias, a_log,
+// dskip fp32; ring [slots][taps][conv] in u's type; state [slots][H][N][P4] fp32, read and written; y [tokens, H P].
+// Sequence i covers tokens q_start[i] .. + q_lens[i] - 1 and ends at position seq_lens[i] - 1.
+int pm_ssm_scan(const void* u, int f32, long long ldu, const float* conv_w, const float* conv_b, const float*
+    dt_bias, const float* a_log, const float* dskip, const void* ring, float* state, const int* slots, const int*
+    q_start, const int* q_lens, const int* seq_lens, int n_seq, int H, int P, int N, int G, int taps, void* y,
+    cudaStream_t st);
+// Whether pm_ssm_chunk covers a state of N rows.
+int pm_ssm_chunk_supported(int N);
+// The same for longer portions of bf16 models: act [tokens, conv] bf16 and dt [tokens, H] fp32 are work buffers that the
+// first kernel fills, max_q is the longest of q_lens.
+int pm_ssm_chunk(const void* u, long long ldu, const float* conv_w, const float* conv_b, const float* dt_bias,
+    const float* a_log, const float* dskip, const void* ring, float* state, const int* slots, const int* q_start,
+    const int* q_lens, const int* seq_lens, int n_seq, int max_q, int H, int P, int N, int G, int taps, void* act,
+    float* dt, void* y, cudaStream_t st);
+// out [tokens, H P] = RMS norm over `parts` equal parts of y * silu(z) (z: the first H P columns of u), times w; the last
+// taps - 1 convolution inputs of every sequence go to the ring. seq_of / pos [tokens]: sequence index and position.
+int pm_ssm_gate_norm(const void* y, const void* u, int f32, long long ldu, const float* w, float eps, int parts,
+    void* out, void* ring, const int* slots, const int* seq_of, const int* pos, const int* seq_lens, int n_tok, int
+    H, int P, int N, int G, int taps, cudaStream_t st);
 
 // ---------------------------------------------------------------- tp_fused.cu
 // mode 0: x_ptrs[r] = rank r's X shard [rows_per_rank, K] (ldx), w = W_loc [N, K] (ldw), out = Y [M, ldd].

@@ -1,0 +1,211 @@
+// Pieces of decoders whose residual stream is kept in fp32 and normalised after each sum:
+//   * token embedding times a factor, written as the fp32 stream and as the compute-type copy the projections read
+//   * residual sum + layer norm:  x <- LN(alpha * x + y (+ bias)) * w + b, statistics in fp32 over the row held in
+//     shared memory (the variance is the mean of squared deviations, taken in a second pass)
+//   * clamped gated unit:  g = min(g, limit), u = clamp(u, -limit, limit), out = g * sigmoid(beta g) * (u + shift)
+//   * rotation table whose angles are formed and reduced in fp64, so that far positions keep fp32-accurate angles
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+#include "elem.cuh"
+#include "host_util.cuh"
+#include "pmetal_b200.h"
+
+namespace pm {
+
+template <typename T, int V>
+__global__ void embed_scale_kernel(const long long* __restrict__ ids, const T* __restrict__ table, float scale, int width,
+                                   float* __restrict__ xf, T* __restrict__ xc) {
+  const long long t = blockIdx.x;
+  const T* src = table + ids[t] * static_cast<long long>(width);
+  for (int k = threadIdx.x * V; k < width; k += blockDim.x * V) {
+    float v[V];
+    load_vec<V>(src + k, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] *= scale;
+    store_vec<V>(xf + t * width + k, v);
+    if (xc) store_vec<V>(xc + t * width + k, v);
+  }
+}
+
+// One CTA per output row; `rows` (nullable) picks the input row. Outputs are nullable.
+template <typename T, int V>
+__global__ void post_layernorm_kernel(const float* x, const T* __restrict__ y, long long ldy,
+                                      const float* __restrict__ bias, float alpha, const float* __restrict__ w,
+                                      const float* __restrict__ b, float eps, int width, const long long* __restrict__ rows,
+                                      float* of, T* __restrict__ oc) {
+  extern __shared__ float row_buf[];
+  const long long o = blockIdx.x, r = rows ? rows[o] : o;
+  float sum = 0.f;
+  for (int k = threadIdx.x * V; k < width; k += blockDim.x * V) {
+    float v[V];
+    load_vec<V>(x + r * width + k, v);
+    if (y) {
+      float s[V];
+      load_vec<V>(y + r * ldy + k, s);
+      if (bias) {
+        float c[V];
+        load_vec<V>(bias + k, c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s[e] += c[e];
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = fmaf(alpha, v[e], s[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      row_buf[k + e] = v[e];
+      sum += v[e];
+    }
+  }
+  const float mean = block_sum(sum) / static_cast<float>(width);
+  float dev = 0.f;
+  for (int k = threadIdx.x * V; k < width; k += blockDim.x * V)
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float d = row_buf[k + e] - mean;
+      dev = fmaf(d, d, dev);
+    }
+  const float rstd = 1.f / sqrtf(block_sum(dev) / static_cast<float>(width) + eps);
+  for (int k = threadIdx.x * V; k < width; k += blockDim.x * V) {
+    float v[V], ww[V], bb[V];
+    load_vec<V>(w + k, ww);
+    load_vec<V>(b + k, bb);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = fmaf((row_buf[k + e] - mean) * rstd, ww[e], bb[e]);
+    if (of) store_vec<V>(of + o * width + k, v);
+    if (oc) store_vec<V>(oc + o * width + k, v);
+  }
+}
+
+template <typename T, int V>
+__global__ void clamped_glu_kernel(const T* __restrict__ gu, long long ld, const float* __restrict__ bias, int ff,
+                                   float limit, float beta, float shift, T* __restrict__ out, long long n_vec) {
+  const int per_row = ff / V;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n_vec;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long t = i / per_row;
+    const int k = static_cast<int>(i - t * per_row) * V;
+    float g[V], u[V];
+    load_vec<V>(gu + t * ld + k, g);
+    load_vec<V>(gu + t * ld + ff + k, u);
+    if (bias) {
+      float a[V], c[V];
+      load_vec<V>(bias + k, a);
+      load_vec<V>(bias + ff + k, c);
+#pragma unroll
+      for (int e = 0; e < V; ++e) { g[e] += a[e]; u[e] += c[e]; }
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) g[e] = clamped_glu(g[e], u[e], limit, beta, shift);
+    store_vec<V>(out + t * ff + k, g);
+  }
+}
+
+__global__ void rope_table_f64_kernel(const int* __restrict__ pos, const double* __restrict__ freq, int n, int half,
+                                      float* __restrict__ cs, float* __restrict__ sn) {
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n * half; i += gridDim.x * blockDim.x) {
+    const int t = i / half, j = i - t * half;
+    const double two_pi = 6.283185307179586476925286766559;
+    double a = static_cast<double>(pos[t]) * freq[j];
+    a -= rint(a / two_pi) * two_pi;
+    float s, c;
+    sincosf(static_cast<float>(a), &s, &c);
+    cs[i] = c;
+    sn[i] = s;
+  }
+}
+
+static int row_threads(int width, int v) {
+  const int want = (width / v + 31) / 32 * 32;
+  return want < 32 ? 32 : (want > 256 ? 256 : want);
+}
+
+template <typename T>
+static int embed_launch(const long long* ids, const void* table, float scale, int n, int width, float* xf, void* xc,
+                        cudaStream_t st) {
+  const T* tab = static_cast<const T*>(table);
+  T* out = static_cast<T*>(xc);
+  if (width % 4 == 0) embed_scale_kernel<T, 4><<<n, row_threads(width, 4), 0, st>>>(ids, tab, scale, width, xf, out);
+  else embed_scale_kernel<T, 1><<<n, row_threads(width, 1), 0, st>>>(ids, tab, scale, width, xf, out);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int V>
+static int postnorm_launch(const float* x, const void* y, long long ldy, const float* bias, float alpha, const float* w,
+                           const float* b, float eps, int n, int width, const long long* rows, float* of, void* oc,
+                           cudaStream_t st) {
+  const size_t smem = static_cast<size_t>(width) * sizeof(float);
+  static DeviceMax configured;
+  if (smem > 40 * 1024 && smem > configured.get()) {
+    const cudaError_t e = cudaFuncSetAttribute(post_layernorm_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                               200 * 1024);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured.set(200 * 1024);
+  }
+  post_layernorm_kernel<T, V><<<n, row_threads(width, V), smem, st>>>(x, static_cast<const T*>(y), ldy, bias, alpha, w, b,
+                                                                      eps, width, rows, of, static_cast<T*>(oc));
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+static int glu_launch(const void* gu, long long ld, const float* bias, int n, int ff, float limit, float beta, float shift,
+                      void* out, cudaStream_t st) {
+  const bool vec = ff % 4 == 0 && ld % 4 == 0;
+  const long long n_vec = static_cast<long long>(n) * (vec ? ff / 4 : ff);
+  long long grid = (n_vec + 255) / 256;
+  if (grid > num_sms() * 16) grid = num_sms() * 16;
+  const T* src = static_cast<const T*>(gu);
+  if (vec) clamped_glu_kernel<T, 4><<<static_cast<int>(grid), 256, 0, st>>>(src, ld, bias, ff, limit, beta, shift, static_cast<T*>(out), n_vec);
+  else clamped_glu_kernel<T, 1><<<static_cast<int>(grid), 256, 0, st>>>(src, ld, bias, ff, limit, beta, shift, static_cast<T*>(out), n_vec);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace pm
+
+using namespace pm;
+
+// xf [n, width] fp32 = table[ids] * scale, xc the same in the table's type (nullable). f32: the table is fp32, else bf16.
+extern "C" int pm_embed_scale(const long long* ids, const void* table, int f32, float scale, int n, int width, float* xf,
+                              void* xc, cudaStream_t st) {
+  if (n < 0 || width < 1) return -1;
+  if (n == 0) return 0;
+  return f32 ? embed_launch<float>(ids, table, scale, n, width, xf, xc, st)
+             : embed_launch<__nv_bfloat16>(ids, table, scale, n, width, xf, xc, st);
+}
+
+// of / oc [n, width] (fp32 / compute type, each nullable) = LN(alpha * x + y + bias) * w + b for the n rows listed in
+// `rows` (nullable: row i). y [.., ldy] and bias are nullable; without y the row is x itself. of may be x when rows is
+// null.
+extern "C" int pm_post_layernorm(const float* x, const void* y, int f32, long long ldy, const float* bias, float alpha,
+                                 const float* w, const float* b, float eps, int n, int width, const long long* rows,
+                                 float* of, void* oc, cudaStream_t st) {
+  if (n < 0 || width < 1 || static_cast<size_t>(width) * 4 > 200 * 1024 || (rows && of == x)) return -1;
+  if (n == 0) return 0;
+  const bool vec = width % 4 == 0 && ldy % 4 == 0;
+  if (f32)
+    return vec ? postnorm_launch<float, 4>(x, y, ldy, bias, alpha, w, b, eps, n, width, rows, of, oc, st)
+               : postnorm_launch<float, 1>(x, y, ldy, bias, alpha, w, b, eps, n, width, rows, of, oc, st);
+  return vec ? postnorm_launch<__nv_bfloat16, 4>(x, y, ldy, bias, alpha, w, b, eps, n, width, rows, of, oc, st)
+             : postnorm_launch<__nv_bfloat16, 1>(x, y, ldy, bias, alpha, w, b, eps, n, width, rows, of, oc, st);
+}
+
+// gu [n, ld]: gate columns [0, ff), up columns [ff, 2 ff); bias fp32 [2 ff] or null -> out [n, ff].
+extern "C" int pm_clamped_glu(const void* gu, int f32, long long ld, const float* bias, int n, int ff, float limit,
+                              float beta, float shift, void* out, cudaStream_t st) {
+  if (n < 0 || ff < 1 || ld < 2ll * ff) return -1;
+  if (n == 0) return 0;
+  return f32 ? glu_launch<float>(gu, ld, bias, n, ff, limit, beta, shift, out, st)
+             : glu_launch<__nv_bfloat16>(gu, ld, bias, n, ff, limit, beta, shift, out, st);
+}
+
+// cos / sin [n, half] fp32 of pos * freq (freq fp64 [half] on the device).
+extern "C" int pm_rope_table_f64(const int* pos, const double* freq, int n, int half, float* cs, float* sn,
+                                 cudaStream_t st) {
+  if (n < 0 || half < 1) return -1;
+  if (n == 0) return 0;
+  int grid = (n * half + 255) / 256;
+  if (grid > num_sms() * 8) grid = num_sms() * 8;
+  rope_table_f64_kernel<<<grid, 256, 0, st>>>(pos, freq, n, half, cs, sn);
+  return static_cast<int>(cudaGetLastError());
+}

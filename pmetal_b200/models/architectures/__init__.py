@@ -2,8 +2,9 @@
 
 Mirrors the reference's dispatcher (crates/pmetal-models/src/dispatcher.rs:90-160: ``from_model_type`` then
 ``from_architectures``). The families with hand-written kernels (Qwen3, Qwen3-MoE, Llama, Qwen2, Mistral) resolve to
-``models.decoder.DecoderLM``; every other decoder resolves to the portable ``GenericDecoderLM``; hybrids, encoders and
-encoder-decoders have their own classes."""
+``models.decoder.DecoderLM``; the config-driven attention / recurrent stacks that run on the paged state cache (Duvivik)
+to ``models.hybrid_decoder.HybridDecoderLM``; every other decoder resolves to the portable ``GenericDecoderLM``; other
+hybrids, encoders and encoder-decoders have their own classes."""
 from __future__ import annotations
 
 import json
@@ -15,6 +16,8 @@ GENERIC_DECODER = {"mixtral", "gemma", "gemma2", "gemma3", "gemma3_text", "phi",
                    "command_r", "command-r", "granite", "granitemoe", "granite_moe", "olmo2", "gpt_oss", "gptoss", "gpt-oss",
                    "llama4", "llama4_text", "deepseek", "deepseek2", "deepseek_v2", "deepseek_v3", "qwen3_next", "qwen3_5",
                    "qwen3.5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text"}
+HYBRID_DECODER = {"duvivik"}
+PAGED_FAMILIES = ("fast", "hybrid")       # served from the paged caches by the generator and the batching engine
 OTHER = {"nemotron_h": "nemotron_h", "nemotronh": "nemotron_h", "nemotron-h": "nemotron_h", "bert": "bert", "roberta": "bert",
          "distilbert": "bert", "xlm-roberta": "bert", "xlm_roberta": "bert", "t5": "t5", "clip": "clip", "whisper": "whisper",
          "flux": "flux", "flux-1": "flux", "flux.1": "flux", "pixtral": "pixtral", "qwen2_vl": "qwen2_vl", "mllama": "mllama",
@@ -22,8 +25,10 @@ OTHER = {"nemotron_h": "nemotron_h", "nemotronh": "nemotron_h", "nemotron-h": "n
 
 
 def family_of(config: dict) -> Optional[str]:
-    """``fast`` | ``generic`` | one of the names in ``OTHER`` | None for an unknown architecture."""
+    """``fast`` | ``hybrid`` | ``generic`` | one of the names in ``OTHER`` | None for an unknown architecture."""
     mt = str(config.get("model_type", "")).lower()
+    if str(config.get("architecture", mt)).lower() in HYBRID_DECODER:
+        return "hybrid"
     if mt in ("gemma4", "gemma4_text"):
         return "gemma4"
     if "text_config" in config and mt not in OTHER:
@@ -56,6 +61,9 @@ def build_model(config: dict, dtype=None, device=None):
         from ..config import ModelArgs
         from ..decoder import DecoderLM
         return DecoderLM(ModelArgs.from_dict(config), dtype=dtype or torch.float32, device=device)
+    if fam == "hybrid":
+        from ..hybrid_decoder import HybridArgs, HybridDecoderLM
+        return HybridDecoderLM(HybridArgs.from_dict(config), dtype=dtype or torch.float32, device=device)
     if fam == "generic":
         from .generic import GenericDecoderLM
         m = GenericDecoderLM.from_hf_config(config)

@@ -388,12 +388,13 @@ class DecoderLM(nn.Module):
     # ------------------------------------------------------------------ cached (paged) forward
     @torch.no_grad()
     def forward_paged(self, input_ids: torch.Tensor, cache, meta, all_logits: bool = False,
-                      return_hidden: bool = False) -> torch.Tensor:
+                      return_hidden: bool = False, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Forward over the new tokens of several sequences with a paged KV cache.
 
         ``input_ids`` [total_q] are the new tokens in ``meta`` order; keys/values are appended to ``cache`` and
         attention reads the block table directly. Returns logits for the last new token of every sequence
-        ([n_seq, V]) or for every new token ([total_q, V], speculative verification)."""
+        ([n_seq, V]), for every new token ([total_q, V], speculative verification) or for the token rows listed in ``rows``
+        (int64, single-rank models)."""
         cfg = self.cfg
         ch = getattr(self, "step_channel", None)
         if ch is not None and ch.leader and not ch.muted:
@@ -457,10 +458,14 @@ class DecoderLM(nn.Module):
             h = at.o_proj(o, x)
             n2 = ops.rms_norm(h, layer.post_attention_layernorm, cfg.rms_norm_eps)
             x = layer.mlp(n2, h)
-        if not all_logits:
+        if rows is not None:
+            x = x[rows]
+        elif not all_logits:
             last = (meta.q_start + meta.q_lens - 1).long()
             x = x[last]               # RMSNorm is per row, so selecting rows first is equivalent
         head = self.head_weight()
+        if x.shape[0] == 0:
+            return x.new_empty(0, x.shape[1] if return_hidden else head.shape[0])
         if (skinny and not return_hidden and x.shape[0] <= GEMV_MAX_ROWS and cfg.final_logit_softcap <= 0
                 and head.dtype == torch.bfloat16 and not head.requires_grad):
             from ..ops import native as nat

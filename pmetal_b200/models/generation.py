@@ -65,10 +65,14 @@ class GraphedDecoder:
 
     def __init__(self, model, cache: PagedKVCache, pad_block: Optional[int] = None):
         self.model, self.cache, self.device = model, cache, cache.device
+        self.state_slots = getattr(cache, "slot_of", None)      # caches with a state slot per sequence
         self.graphs = {}
         self.channel = getattr(model, "step_channel", None)
         if pad_block is not None:           # a rank that follows another rank's scheduler uses that rank's scratch block
             self.pad_block = pad_block
+            return
+        if cache.scratch_block is not None:
+            self.pad_block = cache.scratch_block
             return
         if self.PAD_SEQ not in cache.seqs:
             cache.add_sequence(self.PAD_SEQ)
@@ -94,18 +98,21 @@ class GraphedDecoder:
 
     def _capture(self, key, nb: int, mb: int):
         dev = self.device
+        n32 = 2 * nb + nb * mb + (nb if self.state_slots is not None else 0)
         st = {
             "h64": torch.zeros(2 * nb, dtype=torch.int64).pin_memory(),              # slots | tokens
-            "h32": torch.zeros(2 * nb + nb * mb, dtype=torch.int32).pin_memory(),    # positions | seq_lens | table
+            "h32": torch.zeros(n32, dtype=torch.int32).pin_memory(),                 # positions | seq_lens | table (| state slots)
             "d64": torch.zeros(2 * nb, dtype=torch.int64, device=dev),
-            "d32": torch.zeros(2 * nb + nb * mb, dtype=torch.int32, device=dev),
+            "d32": torch.zeros(n32, dtype=torch.int32, device=dev),
         }
         d64, d32 = st["d64"], st["d32"]
-        st["meta"] = BatchMeta(list(range(nb)), d32[2 * nb:].view(nb, mb), d32[nb:2 * nb],
-                               torch.arange(nb, dtype=torch.int32, device=dev), torch.ones(nb, dtype=torch.int32, device=dev),
-                               d64[:nb], d32[:nb], nb, 1, mb * BLOCK)
+        first = torch.arange(nb, dtype=torch.int32, device=dev)
+        st["meta"] = BatchMeta(list(range(nb)), d32[2 * nb:2 * nb + nb * mb].view(nb, mb), d32[nb:2 * nb], first,
+                               torch.ones(nb, dtype=torch.int32, device=dev), d64[:nb], d32[:nb], nb, 1, mb * BLOCK)
+        if self.state_slots is not None:
+            st["meta"].state_slots, st["meta"].seq_of = d32[2 * nb + nb * mb:], first
         st["tokens"] = d64[nb:]
-        self._fill(st, nb, mb, [], [], [], [], [])
+        self._fill(st, nb, mb, [], [], [], [], [], [])
         self._copy(st)
         # warm-up outside capture (lazy initialisations), then capture
         side = torch.cuda.Stream()
@@ -122,11 +129,11 @@ class GraphedDecoder:
         self.graphs[key] = st
         return st
 
-    def _fill(self, st, nb, mb, slots, pos, lens, tables, tokens):
+    def _fill(self, st, nb, mb, slots, pos, lens, tables, tokens, states):
         """Write one step's metadata into the pinned host buffers (numpy views; no tensor constructions)."""
         if "n64" not in st:
             st["n64"], st["n32"] = st["h64"].numpy(), st["h32"].numpy()
-            st["rows"] = [None] * nb               # (first block, block count) last written per row
+            st["rows"] = [None] * nb               # block list last written per row
             st["n32"][2 * nb:] = self.pad_block
         a64, a32 = st["n64"], st["n32"]
         n = len(slots)
@@ -138,14 +145,17 @@ class GraphedDecoder:
         a32[n:nb] = 0
         a32[nb:nb + n] = lens
         a32[nb + n:2 * nb] = 1
-        tab = a32[2 * nb:].reshape(nb, mb)
+        tab = a32[2 * nb:2 * nb + nb * mb].reshape(nb, mb)
+        if self.state_slots is not None:
+            sl = a32[2 * nb + nb * mb:]
+            sl[:n] = states
+            sl[n:] = self.cache.scratch_slot
         rows = st["rows"]
         for i in range(nb):
             bl = tables[i] if i < n else None
-            sig = None if bl is None else (bl[0], len(bl), bl[-1], sum(1 for b in bl if b < 0) if self.cache.window > 0 else 0)
-            if rows[i] == sig:
+            if rows[i] == bl and bl is not None:     # blocks are recycled: only the whole list says that nothing changed
                 continue
-            rows[i] = sig
+            rows[i] = None if bl is None else list(bl)
             if bl is None:
                 tab[i, :] = self.pad_block
             else:
@@ -175,7 +185,8 @@ class GraphedDecoder:
         nb, mb = _bucket(n), _bucket(max(len(t) for t in tables), 8)
         st = self._state(nb, mb)
         toks = tokens.tolist() if isinstance(tokens, torch.Tensor) else list(tokens)
-        self._fill(st, nb, mb, slots, pos, lens, tables, toks)
+        states = [self.state_slots[sid] for sid in seq_ids] if self.state_slots is not None else []
+        self._fill(st, nb, mb, slots, pos, lens, tables, toks, states)
         if self.channel is not None and self.channel.leader:
             self.channel.publish_graph(nb, mb, n, self.pad_block, st["h64"], st["h32"])
         self._copy(st)
@@ -206,11 +217,44 @@ class Generator:
         self.cache.add_sequence(sid)
         return sid
 
+    def check_tokens(self, ids: Sequence[int]) -> None:
+        """Token ids index the embedding on the device: they are checked on the host."""
+        if ids and not (0 <= min(ids) and max(ids) < self.model.cfg.vocab_size):
+            raise ValueError(f"token ids must lie in [0, {self.model.cfg.vocab_size})")
+
     # ------------------------------------------------------------------ prefill / decode primitives
+    @torch.no_grad()
+    def step(self, seq_ids: Sequence[int], tokens: Sequence[Sequence[int]],
+             want: Optional[Sequence[Sequence[int]]] = None) -> torch.Tensor:
+        """One batch in which sequence ``seq_ids[i]`` gets ``tokens[i]``: portions of prompts beside single decoded tokens.
+        Returns the logits at the places ``want[i]`` among the new tokens (default: the last one of every sequence), in
+        that order. A step of single tokens runs as a decode step (captured graphs)."""
+        flat = [t for ts in tokens for t in ts]
+        self.check_tokens(flat)
+        counts = [len(ts) for ts in tokens]
+        if min(counts) < 1:
+            raise ValueError("every sequence of a step needs at least one token")
+        if want is not None and any(not 0 <= k < n for w, n in zip(want, counts) for k in w):
+            raise ValueError("a wanted place lies outside its portion")
+        if max(counts) == 1:
+            logits = self.decode_step(seq_ids, torch.tensor(flat, dtype=torch.int64, device=self.device))
+            if want is None:
+                return logits
+            return logits[torch.tensor([i for i, w in enumerate(want) for _ in w], dtype=torch.int64, device=self.device)]
+        meta = self.cache.prepare(seq_ids, counts)
+        ids = torch.tensor(flat, dtype=torch.int64, device=self.device)
+        rows = None
+        if want is not None:
+            start = meta.host[3]
+            rows = torch.tensor([start[i] + k for i, w in enumerate(want) for k in w], dtype=torch.int64, device=self.device)
+        return self.model.forward_paged(ids, self.cache, meta, rows=rows)
+
     @torch.no_grad()
     def prefill(self, seq_ids: Sequence[int], prompts: Sequence[Sequence[int]], chunk: int = PREFILL_CHUNK):
         """Feed whole prompts (chunked); returns logits of each prompt's last token [n, V]."""
         n = len(seq_ids)
+        for p in prompts:
+            self.check_tokens(p)
         offs = [0] * n
         last_logits = [None] * n
         while True:
@@ -246,7 +290,8 @@ class Generator:
     def _decode_step(self, seq_ids: Sequence[int], tokens: torch.Tensor) -> torch.Tensor:
         if self.cuda_graphs:
             from ..ops import functional as ops
-            if ops.native_enabled(self.model.embed_tokens) and self.model.cfg.head_dim == 128:
+            if ops.native_enabled(self.model.embed_tokens) and (getattr(self.model, "graph_decode", False)
+                                                                or self.model.cfg.head_dim == 128):
                 if self._graphed is None:
                     self._graphed = GraphedDecoder(self.model, self.cache)
                 return self._graphed.step(seq_ids, tokens)

@@ -1,0 +1,302 @@
+"""Config-driven serving decoder for stacks that mix attention and recurrent layers (Duvivik).
+
+Each layer has a token mixer (``mixers.MIXERS``) and optionally a feed-forward; both sublayers read the stream itself and
+the norm comes after the sum: x <- LN(alpha * x + sublayer(x)). The stream, norms, rotation angles, softmax and recurrent
+states are fp32; projections and their activations run in the model's type (bf16 on the sm_100a kernels, or fp32
+throughout with full-precision matrix products).
+
+``forward_paged`` has the interface of ``DecoderLM.forward_paged``: the new tokens of several sequences in one batch, their
+cache a ``StateCache``, so the generator, the CUDA-graph decoder, the continuous-batching engine and the sampler serve it
+as they serve the other models. There is no CPU path: the model can be built, loaded and saved anywhere, and runs on a
+GPU."""
+from __future__ import annotations
+
+import copy
+import json
+import os
+from dataclasses import dataclass, field
+from typing import Dict, List, Optional
+
+import torch
+import torch.nn as nn
+
+from ..ops import functional as ops
+from .kv_cache import BLOCK
+from .mixers import MIXERS, RotationFreqs, StepContext, frozen
+from .state_cache import StateCache
+
+GLU_BETA, GLU_SHIFT = 1.702, 1.0          # gate slope and the offset of the up half in the clamped gated unit
+
+ARCHITECTURES = {"duvivik"}
+
+
+@dataclass
+class HybridArgs:
+    vocab_size: int
+    hidden_size: int
+    layers: List[dict]                    # {"type", "mixer", "mlp"} per layer, as in the configuration file
+    embed_scale: float = 1.0
+    residual_alpha: float = 1.0
+    norm_eps: float = 1e-5
+    model_type: str = "duvivik"
+    bos_token_id: Optional[int] = None
+    eos_token_id: Optional[int] = None
+    raw: dict = field(default_factory=dict, repr=False)
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layers)
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "HybridArgs":
+        name = str(d.get("architecture", d.get("model_type", ""))).lower()
+        if name not in ARCHITECTURES:
+            raise ValueError(f"unknown hybrid architecture {name!r}")
+        layers = [dict(l, mlp=l.get("mlp")) for l in d["layers"]]
+        for i, l in enumerate(layers):
+            kind = MIXERS.get(l["type"])
+            if kind is None:
+                raise ValueError(f"layer {i}: unknown mixer {l['type']!r} (known: {', '.join(sorted(MIXERS))})")
+            missing = [k for k in kind.KEYS if k not in l["mixer"]]
+            if missing:
+                raise ValueError(f"layer {i}: mixer entry lacks {', '.join(missing)}")
+            kind.check(l["mixer"], i, layers)
+            mlp = l["mlp"]
+            if mlp is not None and mlp.get("kind") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        eos = d.get("eos_token_id")
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
+                   embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+                   residual_alpha=float(d.get("postln_alpha", 1.0)), norm_eps=float(d["norm"]["eps"]), model_type=name,
+                   bos_token_id=d.get("bos_token_id"), eos_token_id=eos[0] if isinstance(eos, list) else eos,
+                   raw=copy.deepcopy(d))
+
+    @classmethod
+    def from_pretrained(cls, model_dir: str) -> "HybridArgs":
+        with open(os.path.join(model_dir, "config.json"), "r", encoding="utf-8") as fh:
+            return cls.from_dict(json.load(fh))
+
+    def to_hf_dict(self) -> dict:
+        return copy.deepcopy(self.raw)
+
+
+def _stack(width: int, vocab: int, ff: int, attn: dict, ssm: dict, pattern: str, limit: float = 7.0) -> dict:
+    """Configuration dict: one letter per layer, A = latent attention with its own latents, a = reading those of the latest
+    A, m = state-space layer without feed-forward, M = with one."""
+    layers, src = [], None
+    for i, ch in enumerate(pattern):
+        mlp = {"kind": "dense", "ff": ff, "limit": limit} if ch in "AaM" else None
+        if ch in "Aa":
+            m = dict(attn)
+            if ch == "A":
+                src = i
+            else:
+                m["kv_from"] = src
+            layers.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+        else:
+            layers.append({"type": "mamba2", "mixer": dict(ssm), "mlp": mlp})
+    return {"architecture": "Duvivik", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "postln_alpha": 2.0,
+            "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def _attn(heads, dim, rot, vdim, rank):
+    return {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "scale": (dim + rot) ** -0.5,
+            "rot": {"base": 10000.0, "dims": rot}}
+
+
+def _ssm(heads, vdim, state, groups, conv=4, norm_groups=1):
+    return {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": norm_groups}
+
+
+# random-weight models for smoke runs and measurements (``random:<name>``)
+PRESETS: Dict[str, dict] = {
+    "duvivik-tiny": _stack(64, 512, 96, _attn(4, 16, 8, 24, 40), _ssm(4, 24, 16, 2, norm_groups=2), "AmaM"),
+    "duvivik-1b": _stack(2048, 65536, 6144, _attn(32, 64, 64, 128, 512), _ssm(64, 64, 128, 8, norm_groups=8), "Ammmammm" * 2),
+    "duvivik-4b": _stack(2560, 65536, 9728, _attn(32, 96, 32, 128, 512), _ssm(80, 64, 128, 8, norm_groups=8), "Ammmammm" * 4),
+}
+
+
+class ClampedMLP(nn.Module):
+    """Gated feed-forward with clamped inputs and biases on all projections."""
+
+    def __init__(self, m: dict, width: int, dtype, device):
+        super().__init__()
+        self.ff, self.limit, self.width = m["ff"], float(m["limit"]), width
+        up8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        self.w_gu = frozen(torch.zeros(up8(2 * self.ff), width, dtype=dtype, device=device))
+        self.b_gu = frozen(torch.zeros(2 * self.ff, device=device))
+        self.w_down = frozen(torch.zeros(up8(width), self.ff, dtype=dtype, device=device))
+        self.b_down = frozen(torch.zeros(width, device=device))
+
+    def named_weights(self):
+        f, w = self.ff, self.width
+        yield "gate", (f, w), lambda t: self.w_gu[:f].copy_(t), lambda: self.w_gu[:f]
+        yield "gate.b", (f,), lambda t: self.b_gu[:f].copy_(t), lambda: self.b_gu[:f]
+        yield "up", (f, w), lambda t: self.w_gu[f:2 * f].copy_(t), lambda: self.w_gu[f:2 * f]
+        yield "up.b", (f,), lambda t: self.b_gu[f:].copy_(t), lambda: self.b_gu[f:]
+        yield "down", (w, f), lambda t: self.w_down[:w].copy_(t), lambda: self.w_down[:w]
+        yield "down.b", (w,), self.b_down.copy_, lambda: self.b_down
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        """Without the down-projection's bias, which the caller adds in fp32 with the residual."""
+        from ..ops import native as nat
+        glu = (self.limit, GLU_BETA, GLU_SHIFT)
+        if x.dtype == torch.bfloat16 and ops.gemv_fits(*x.shape) and x.stride(0) % 8 == 0:
+            a = nat.gemv_ex(x, self.w_gu, self.b_gu, glu, n=self.ff)
+        else:
+            a = nat.clamped_glu(ops.project(x, self.w_gu), self.ff, *glu, bias=self.b_gu)
+        return ops.project(a, self.w_down)
+
+
+class HybridLayer(nn.Module):
+    def __init__(self, spec: dict, cfg: HybridArgs, index: int, dtype, device):
+        super().__init__()
+        self.cfg = cfg
+        self.mixer = MIXERS[spec["type"]](spec["mixer"], cfg, index, dtype, device)
+        self.mlp = ClampedMLP(spec["mlp"], cfg.hidden_size, dtype, device) if spec["mlp"] is not None else None
+        vec = lambda: frozen(torch.zeros(cfg.hidden_size, device=device))      # noqa: E731
+        self.norm1_w, self.norm1_b = vec(), vec()
+        if self.mlp is not None:
+            self.norm2_w, self.norm2_b = vec(), vec()
+
+    def named_weights(self):
+        vecs = [("norm1", self.norm1_w), ("norm1.b", self.norm1_b)]
+        if self.mlp is not None:
+            vecs += [("norm2", self.norm2_w), ("norm2.b", self.norm2_b)]
+        for name, p in vecs:
+            yield name, (self.cfg.hidden_size,), p.copy_, (lambda p=p: p)
+        for pre, mod in (("mix.", self.mixer), ("mlp.", self.mlp)):
+            if mod is not None:
+                for name, *rest in mod.named_weights():
+                    yield (pre + name, *rest)
+
+    def forward(self, xf, xc, cache, ctx):
+        """(fp32 stream, compute-type copy) -> the same after the layer."""
+        from ..ops import native as nat
+        cfg = self.cfg
+        y = self.mixer(xc, cache, ctx)
+        xf, xc = nat.post_layernorm(xf, y, self.norm1_w, self.norm1_b, cfg.norm_eps, cfg.residual_alpha)
+        if self.mlp is not None:
+            y = self.mlp(xc)
+            xf, xc = nat.post_layernorm(xf, y, self.norm2_w, self.norm2_b, cfg.norm_eps, cfg.residual_alpha,
+                                        bias=self.mlp.b_down)
+        return xf, xc
+
+
+class HybridDecoderLM(nn.Module):
+    graph_decode = True         # single-token steps can be captured (generation.GraphedDecoder)
+    mixed_batches = True        # the scheduler puts prompt portions and decoded tokens into one step
+    slotted_cache = True        # ``new_cache`` takes the number of live sequences
+
+    def __init__(self, cfg: HybridArgs, dtype=torch.float32, device=None):
+        super().__init__()
+        if dtype not in (torch.float32, torch.bfloat16):
+            raise ValueError("the hybrid decoder runs in bf16 or fp32")
+        self.cfg, self.dtype = cfg, dtype
+        self.embed_tokens = frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
+        self.layers = nn.ModuleList([HybridLayer(s, cfg, i, dtype, device) for i, s in enumerate(cfg.layers)])
+        self.norm_w = frozen(torch.zeros(cfg.hidden_size, device=device))
+        self.norm_b = frozen(torch.zeros(cfg.hidden_size, device=device))
+        self.head = frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
+        self._freqs = RotationFreqs()
+
+    # ------------------------------------------------------------------ weights
+    def named_weights(self):
+        """(checkpoint name, shape, setter, getter) of every tensor."""
+        c = self.cfg
+        yield "embed", (c.vocab_size, c.hidden_size), self.embed_tokens.copy_, lambda: self.embed_tokens
+        for i, layer in enumerate(self.layers):
+            for name, *rest in layer.named_weights():
+                yield (f"l{i}.{name}", *rest)
+        yield "final.norm", (c.hidden_size,), self.norm_w.copy_, lambda: self.norm_w
+        yield "final.norm.b", (c.hidden_size,), self.norm_b.copy_, lambda: self.norm_b
+        yield "head", (c.vocab_size, c.hidden_size), self.head.copy_, lambda: self.head
+
+    @torch.no_grad()
+    def load_hf_state_dict(self, sd: Dict[str, torch.Tensor], strict: bool = True) -> List[str]:
+        """Copy checkpoint tensors into place; returns the names that were not used."""
+        used = set()
+        for name, shape, put, _ in self.named_weights():
+            t = sd.get(name)
+            if t is None:
+                if strict:
+                    raise KeyError(f"missing weight {name}")
+                continue
+            if tuple(t.shape) != tuple(shape):
+                raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {tuple(shape)}")
+            put(t)
+            used.add(name)
+        return [k for k in sd if k not in used]
+
+    def hf_state_dict(self, merged: bool = False) -> Dict[str, torch.Tensor]:
+        """Checkpoint names -> tensors, in bf16 as the design's files store them."""
+        return {name: get().detach().to(torch.bfloat16).contiguous() for name, _, _, get in self.named_weights()}
+
+    @torch.no_grad()
+    def init_weights(self, std: float = 0.02, seed: int = 0, device=None) -> "HybridDecoderLM":
+        """Random model: N(0, std) matrices, unit norms, decays and step sizes spread over their usual ranges. Drawn on
+        ``device`` (CPU unless given: the values then do not depend on the model's device)."""
+        g = torch.Generator(device=device or "cpu").manual_seed(seed)
+        for name, shape, put, _ in self.named_weights():
+            leaf = name.split(".", 1)[1] if name[0] == "l" and name[1].isdigit() else name
+            rnd = lambda: torch.empty(shape, device=device or "cpu")      # noqa: E731
+            if leaf.endswith(".A_log"):
+                put(rnd().uniform_(1.0, 16.0, generator=g).log_())
+            elif leaf.endswith(".dt_bias"):
+                put(rnd().uniform_(-4.6, -2.3, generator=g))
+            elif leaf.endswith(".D") or leaf.endswith("norm") or leaf in ("norm1", "norm2"):
+                put(torch.ones(shape, device=device or "cpu"))
+            elif leaf.endswith(".conv"):
+                put(rnd().uniform_(-0.5, 0.5, generator=g))
+            elif leaf.endswith(".b"):
+                put(torch.zeros(shape, device=device or "cpu"))
+            else:
+                put(rnd().normal_(0.0, std, generator=g))
+        return self
+
+    def num_parameters(self, trainable_only: bool = False) -> int:
+        return 0 if trainable_only else sum(p.numel() for p in self.parameters())
+
+    # ------------------------------------------------------------------ cache / forward
+    def new_cache(self, num_blocks: int, dtype=None, device=None, max_seqs: int = 64, quant=None, window: int = 0,
+                  sink: int = 0) -> StateCache:
+        if quant or window:
+            raise ValueError("the latent / state cache has no quantised or windowed variant")
+        p = self.embed_tokens
+        return StateCache([l.mixer.cache_spec() for l in self.layers], num_blocks, max_seqs, dtype or p.dtype,
+                          device or p.device)
+
+    @torch.no_grad()
+    def forward(self, input_ids: torch.Tensor) -> torch.Tensor:
+        """Logits of whole sequences [T] or [B, L] -> [.., vocab] on a cache of their own."""
+        seqs = input_ids[None] if input_ids.dim() == 1 else input_ids
+        B, L = seqs.shape
+        cache = self.new_cache(B * -(-L // BLOCK), max_seqs=B)
+        for i in range(B):
+            cache.add_sequence(i)
+        out = self.forward_paged(seqs.reshape(-1), cache, cache.prepare(list(range(B)), [L] * B), all_logits=True)
+        return out.view(*input_ids.shape, -1)
+
+    @torch.no_grad()
+    def forward_paged(self, input_ids: torch.Tensor, cache: StateCache, meta, all_logits: bool = False,
+                      return_hidden: bool = False, rows: Optional[torch.Tensor] = None, on_layer=None) -> torch.Tensor:
+        """Logits (fp32) of the last new token of every sequence, of every new token (``all_logits``) or of the token rows
+        listed in ``rows`` (int64). ``on_layer(i, stream)`` sees the fp32 stream after every layer."""
+        from ..ops import native as nat
+        if not self.embed_tokens.is_cuda or not nat.available():
+            raise RuntimeError("the hybrid decoder runs on a CUDA device with the native kernel library "
+                               f"({nat.load_error() or 'no CUDA device'})")
+        cfg = self.cfg
+        ctx = StepContext(meta, self._freqs)
+        xf, xc = nat.embed_scale(input_ids, self.embed_tokens, cfg.embed_scale)
+        for i, layer in enumerate(self.layers):
+            xf, xc = layer(xf, xc, cache, ctx)
+            if on_layer is not None:
+                on_layer(i, xf)
+        if rows is None and not all_logits:
+            rows = (meta.q_start + meta.q_lens - 1).long()
+        if rows is not None and rows.shape[0] == 0:
+            return torch.empty(0, cfg.vocab_size, dtype=torch.float32, device=xf.device)
+        _, h = nat.post_layernorm(xf, None, self.norm_w, self.norm_b, cfg.norm_eps, rows=rows, want_stream=False,
+                                  dtype=self.dtype)
+        return h if return_hidden else ops.project_f32(h, self.head, cfg.vocab_size)

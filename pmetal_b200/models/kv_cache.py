@@ -48,6 +48,8 @@ class BatchMeta:
     max_q: int = 1
     max_kv: int = 0
     host: Optional[tuple] = None    # host copies (slots, positions, seq_lens, q_start, q_lens, block table) when known
+    state_slots: Optional[torch.Tensor] = None   # [n_seq] int32: row of each sequence in per-sequence state pools
+    seq_of: Optional[torch.Tensor] = None        # [total_q] int32: index of each token's sequence in this batch
 
 
 GROUP = 64      # channels per quantisation scale of the int8 cache
@@ -87,46 +89,30 @@ def select_cache_mode(weight_bytes: int, fp16_kv_bytes: int, device_bytes: Optio
     return CacheMode("standard", 16, group_size, "auto_fp16")
 
 
-class PagedKVCache:
-    def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, num_blocks: int, dtype=torch.bfloat16,
-                 device="cuda", quant: Optional[str] = None, window: int = 0, sink: int = 0):
-        self.num_layers, self.hkv, self.d, self.num_blocks = num_layers, num_kv_heads, head_dim, num_blocks
-        self.device = torch.device(device)
-        if quant not in (None, "int8", "tq4"):
-            raise ValueError("the paged cache stores bf16, int8 or rotated 4-bit codes; other widths use the portable "
-                             "QuantKVCache")
-        if quant == "int8" and head_dim % GROUP:
-            raise ValueError(f"int8 cache needs head_dim to be a multiple of {GROUP}")
-        if quant == "tq4" and head_dim != 128:
-            raise ValueError("the rotated 4-bit cache is built for head_dim 128")
-        self.quant, self.window, self.sink = quant, int(window), int(sink)
-        shape = (num_blocks, BLOCK, num_kv_heads, head_dim // 2 if quant == "tq4" else head_dim)
-        store = torch.int8 if quant == "int8" else (torch.uint8 if quant == "tq4" else dtype)
-        self.tq = None
-        if quant == "tq4":
-            # random signed Hadamard rotation + 16-level Lloyd-Max code book of the unit normal (models/turboquant.py)
-            from .turboquant import TurboQuant
-            self.tq = TurboQuant(head_dim, 4, qjl=False, seed=0, device=device)
-            self.tq_lut = [float(x) for x in self.tq.centroids.tolist()]
-        self.compute_dtype = dtype
-        self.k = [torch.zeros(shape, dtype=store, device=device) for _ in range(num_layers)]
-        self.v = [torch.zeros(shape, dtype=store, device=device) for _ in range(num_layers)]
-        self.k_scale = self.v_scale = None
-        if quant in ("int8", "tq4"):
-            sshape = (num_blocks, BLOCK, num_kv_heads, head_dim // GROUP)
-            self.k_scale = [torch.ones(sshape, dtype=torch.float32, device=device) for _ in range(num_layers)]
-            self.v_scale = [torch.ones(sshape, dtype=torch.float32, device=device) for _ in range(num_layers)]
+class PagedBlocks:
+    """Block allocator and per-sequence block tables of a paged cache. What a block holds is up to the subclass, which
+    says how to copy one (``_copy_block``)."""
+
+    quant: Optional[str] = None
+    window = 0
+    sink = 0
+    can_truncate = True                   # a sequence may drop its latest tokens (no state that has already absorbed them)
+    scratch_block: Optional[int] = None   # block outside the pool that padding rows of a captured step may write to
+
+    def __init__(self, num_blocks: int, device):
+        self.num_blocks, self.device = num_blocks, torch.device(device)
         self.free: List[int] = list(range(num_blocks - 1, -1, -1))
         self.ref = [0] * num_blocks
         self.seqs: Dict[int, SeqState] = {}
 
-    # ------------------------------------------------------------------ allocation
-    @classmethod
-    def blocks_for_budget(cls, bytes_budget: int, num_layers: int, num_kv_heads: int, head_dim: int,
-                          elem_size: int = 2) -> int:
-        per_block = 2 * num_layers * BLOCK * num_kv_heads * head_dim * elem_size
-        return max(int(bytes_budget // per_block), 1)
+    def _copy_block(self, dst: int, src: int) -> None:
+        raise NotImplementedError
 
+    def can_admit(self) -> bool:
+        """Whether one more sequence may be added (beyond the blocks it will need)."""
+        return True
+
+    # ------------------------------------------------------------------ allocation
     def num_free(self) -> int:
         return len(self.free)
 
@@ -176,12 +162,7 @@ class PagedKVCache:
             b = st.blocks[bi]
             if self.ref[b] > 1:          # copy-on-write of a shared, partially filled block
                 nb = self._take()
-                for l in range(self.num_layers):
-                    self.k[l][nb].copy_(self.k[l][b])
-                    self.v[l][nb].copy_(self.v[l][b])
-                    if self.k_scale is not None:
-                        self.k_scale[l][nb].copy_(self.k_scale[l][b])
-                        self.v_scale[l][nb].copy_(self.v_scale[l][b])
+                self._copy_block(nb, b)
                 self._release(b)
                 st.blocks[bi] = b = nb
             stop = min(end, (bi + 1) * BLOCK)
@@ -247,6 +228,51 @@ class PagedKVCache:
 
     def live_blocks(self, seq_id: int) -> int:
         return sum(1 for b in self.seqs[seq_id].blocks if b >= 0)
+
+
+class PagedKVCache(PagedBlocks):
+    def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, num_blocks: int, dtype=torch.bfloat16,
+                 device="cuda", quant: Optional[str] = None, window: int = 0, sink: int = 0):
+        super().__init__(num_blocks, device)
+        self.num_layers, self.hkv, self.d = num_layers, num_kv_heads, head_dim
+        if quant not in (None, "int8", "tq4"):
+            raise ValueError("the paged cache stores bf16, int8 or rotated 4-bit codes; other widths use the portable "
+                             "QuantKVCache")
+        if quant == "int8" and head_dim % GROUP:
+            raise ValueError(f"int8 cache needs head_dim to be a multiple of {GROUP}")
+        if quant == "tq4" and head_dim != 128:
+            raise ValueError("the rotated 4-bit cache is built for head_dim 128")
+        self.quant, self.window, self.sink = quant, int(window), int(sink)
+        shape = (num_blocks, BLOCK, num_kv_heads, head_dim // 2 if quant == "tq4" else head_dim)
+        store = torch.int8 if quant == "int8" else (torch.uint8 if quant == "tq4" else dtype)
+        self.tq = None
+        if quant == "tq4":
+            # random signed Hadamard rotation + 16-level Lloyd-Max code book of the unit normal (models/turboquant.py)
+            from .turboquant import TurboQuant
+            self.tq = TurboQuant(head_dim, 4, qjl=False, seed=0, device=device)
+            self.tq_lut = [float(x) for x in self.tq.centroids.tolist()]
+        self.compute_dtype = dtype
+        self.k = [torch.zeros(shape, dtype=store, device=device) for _ in range(num_layers)]
+        self.v = [torch.zeros(shape, dtype=store, device=device) for _ in range(num_layers)]
+        self.k_scale = self.v_scale = None
+        if quant in ("int8", "tq4"):
+            sshape = (num_blocks, BLOCK, num_kv_heads, head_dim // GROUP)
+            self.k_scale = [torch.ones(sshape, dtype=torch.float32, device=device) for _ in range(num_layers)]
+            self.v_scale = [torch.ones(sshape, dtype=torch.float32, device=device) for _ in range(num_layers)]
+
+    def _copy_block(self, dst: int, src: int) -> None:
+        for l in range(self.num_layers):
+            self.k[l][dst].copy_(self.k[l][src])
+            self.v[l][dst].copy_(self.v[l][src])
+            if self.k_scale is not None:
+                self.k_scale[l][dst].copy_(self.k_scale[l][src])
+                self.v_scale[l][dst].copy_(self.v_scale[l][src])
+
+    @classmethod
+    def blocks_for_budget(cls, bytes_budget: int, num_layers: int, num_kv_heads: int, head_dim: int,
+                          elem_size: int = 2) -> int:
+        per_block = 2 * num_layers * BLOCK * num_kv_heads * head_dim * elem_size
+        return max(int(bytes_budget // per_block), 1)
 
     # ------------------------------------------------------------------ device-side append / attention
     def append(self, layer: int, k: torch.Tensor, v: torch.Tensor, slots: torch.Tensor) -> None:

@@ -11,7 +11,7 @@ from __future__ import annotations
 
 import json
 import os
-from typing import Dict, Optional, Tuple
+from typing import Dict, Optional
 
 import torch
 
@@ -57,12 +57,17 @@ def read_state_dict(model_dir: str) -> Dict[str, torch.Tensor]:
 
 
 def load_pretrained(model: str, dtype: torch.dtype = torch.bfloat16, device="cpu", seed: int = 0,
-                    strict: bool = False, experts_dir: Optional[str] = None) -> Tuple[DecoderLM, ModelArgs, Optional[str]]:
-    """Returns (model, args, model_dir or None). With ``experts_dir`` (written by ``pack-experts``) the routed experts are
+                    strict: bool = False, experts_dir: Optional[str] = None):
+    """Returns (model, args, model_dir or None); the class follows the configuration: ``DecoderLM`` with ``ModelArgs``, or
+    ``HybridDecoderLM`` with ``HybridArgs``. With ``experts_dir`` (written by ``pack-experts``) the routed experts are
     not read from the checkpoint: they are served from that directory on demand (models/expert_store.py)."""
     path = resolve_model_path(model)
     if path.startswith("random:"):
         name = path.split(":", 1)[1]
+        from . import hybrid_decoder as hd
+        if name in hd.PRESETS:
+            args = hd.HybridArgs.from_dict(hd.PRESETS[name])
+            return hd.HybridDecoderLM(args, dtype, device).init_weights(0.02, seed).eval(), args, None
         args = preset(name)
         m = DecoderLM(args).init_weights(0.02, seed)
         return _cast(m, dtype, device), args, None
@@ -70,7 +75,16 @@ def load_pretrained(model: str, dtype: torch.dtype = torch.bfloat16, device="cpu
         from ..gguf.loader import load_gguf_model
         m, args = load_gguf_model(path)
         return _cast(m, dtype, device), args, os.path.dirname(path)
-    args = ModelArgs.from_pretrained(path)
+    with open(os.path.join(path, "config.json"), "r", encoding="utf-8") as fh:
+        config = json.load(fh)
+    from .architectures import family_of
+    if family_of(config) == "hybrid":
+        from .hybrid_decoder import HybridArgs, HybridDecoderLM
+        args = HybridArgs.from_dict(config)
+        m = HybridDecoderLM(args, dtype, device)
+        m.load_hf_state_dict(read_state_dict(path), strict=True)      # every tensor of the design is needed
+        return m.eval(), args, path
+    args = ModelArgs.from_dict(config)
     m = DecoderLM(args)
     sd = read_state_dict(path)
     sd = {k: v for k, v in sd.items() if not k.endswith("rotary_emb.inv_freq")}

@@ -1,0 +1,223 @@
+"""Token mixers of the config-driven serving decoder (``hybrid_decoder.py``).
+
+A mixer is built from its entry in the configuration, says what it keeps in the cache (``cache_spec``), reads its weights
+through ``take(name, shape)`` and runs on the new tokens of a step: ``forward(x, cache, ctx)`` with x [tokens, width] in
+the compute type returns [tokens, width]. ``MIXERS`` maps the configuration's ``type`` to the class; a new kind of mixer
+is one more entry.
+
+``Mamba2Mixer``          selective state space with one decay per head (csrc/ssm.cu)
+``LatentAttentionMixer`` multi-head latent attention on cached latents, its own or an earlier layer's (csrc/latent_attn.cu)
+"""
+from __future__ import annotations
+
+from typing import Callable, Dict, Optional
+
+import torch
+import torch.nn as nn
+
+from ..ops import functional as ops
+from .state_cache import CacheSpec, SeqGroup, split_groups
+
+# portions up to this many tokens take the decode kernels (state-space scan, attention in the latent space)
+SHORT = 16
+
+
+def pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
+    """Zero rows behind a weight so that products can be stored in 16-byte pieces."""
+    n = -w.shape[0] % multiple
+    return torch.cat([w, w.new_zeros(n, w.shape[1])]) if n else w
+
+
+def frozen(t: torch.Tensor) -> nn.Parameter:
+    return nn.Parameter(t.contiguous(), requires_grad=False)
+
+
+class StepContext:
+    """What the layers of one forward share: batch metadata, rotation tables, the split into short and long portions."""
+
+    def __init__(self, meta, freqs: "RotationFreqs"):
+        self.meta, self.freqs = meta, freqs
+        self._rope: Dict[tuple, tuple] = {}
+        self._groups: Dict[int, tuple] = {}
+        self._zeros: Optional[torch.Tensor] = None
+
+    def rope(self, base: float, dims: int):
+        key = (base, dims)
+        if key not in self._rope:
+            from ..ops import native as nat
+            self._rope[key] = nat.rope_table_f64(self.meta.positions, self.freqs.get(base, dims, self.meta.positions.device))
+        return self._rope[key]
+
+    def groups(self, limit: int):
+        if limit not in self._groups:
+            self._groups[limit] = split_groups(self.meta, limit)
+        return self._groups[limit]
+
+    def zeros(self, n: int) -> torch.Tensor:
+        if self._zeros is None or self._zeros.shape[0] < n:
+            self._zeros = torch.zeros(n, dtype=torch.int32, device=self.meta.positions.device)
+        return self._zeros
+
+
+class RotationFreqs:
+    """base^(-2 i / dims) in fp64, one device tensor per (base, dims)."""
+
+    def __init__(self):
+        self._t: Dict[tuple, torch.Tensor] = {}
+
+    def get(self, base: float, dims: int, device) -> torch.Tensor:
+        key = (base, dims, str(device))
+        if key not in self._t:
+            i = torch.arange(0, dims, 2, dtype=torch.float64)
+            self._t[key] = torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / dims).to(device)
+        return self._t[key]
+
+
+Take = Callable[..., torch.Tensor]
+
+
+class Mamba2Mixer(nn.Module):
+    """[z | x | B | C | dt] projection, causal convolution + silu on (x, B, C), recurrence, gate before a norm in
+    ``norm_groups`` equal parts, output projection."""
+
+    KEYS = ("heads", "vdim", "state", "groups", "conv", "norm_groups")
+
+    @classmethod
+    def check(cls, m: dict, index: int, layers) -> None:
+        if m["heads"] % m["groups"]:
+            raise ValueError(f"layer {index}: {m['heads']} heads do not divide into {m['groups']} groups")
+        if m["heads"] * m["vdim"] % m["norm_groups"]:
+            raise ValueError(f"layer {index}: inner width does not divide into {m['norm_groups']} norm parts")
+
+    def __init__(self, m: dict, cfg, index: int, dtype, device):
+        super().__init__()
+        self.dims = (m["heads"], m["vdim"], m["state"], m["groups"], m["conv"])
+        self.H, self.P, self.N, self.G, self.taps = self.dims
+        self.parts, self.eps, self.index = m["norm_groups"], cfg.norm_eps, index
+        self.inner = self.H * self.P
+        self.conv_dim = self.inner + 2 * self.G * self.N
+        self.width, self.dtype = cfg.hidden_size, dtype
+        kw = dict(device=device)
+        n_in = self.inner + self.conv_dim + self.H
+        self.w_in = frozen(torch.zeros(-(-n_in // 8) * 8, self.width, dtype=dtype, **kw))
+        self.conv_w = frozen(torch.zeros(self.taps, self.conv_dim, **kw))          # [taps][channel]
+        self.conv_b = frozen(torch.zeros(self.conv_dim, **kw))
+        self.dt_bias, self.a_log, self.dskip = (frozen(torch.zeros(self.H, **kw)) for _ in range(3))
+        self.norm_w = frozen(torch.zeros(self.inner, **kw))
+        self.w_o = frozen(torch.zeros(-(-self.width // 8) * 8, self.inner, dtype=dtype, **kw))
+
+    def cache_spec(self) -> CacheSpec:
+        p4 = -(-self.P // 4) * 4
+        return CacheSpec(slots={"conv": ((self.taps, self.conv_dim), None), "state": ((self.H, self.N, p4), torch.float32)})
+
+    def named_weights(self):
+        """(checkpoint suffix, shape, setter, getter)."""
+        n_in = self.inner + self.conv_dim + self.H
+        yield "in", (n_in, self.width), lambda t: self.w_in[:n_in].copy_(t), lambda: self.w_in[:n_in]
+        yield "conv", (self.conv_dim, self.taps), lambda t: self.conv_w.copy_(t.t()), lambda: self.conv_w.t()
+        yield "conv.b", (self.conv_dim,), self.conv_b.copy_, lambda: self.conv_b
+        yield "dt_bias", (self.H,), self.dt_bias.copy_, lambda: self.dt_bias
+        yield "A_log", (self.H,), self.a_log.copy_, lambda: self.a_log
+        yield "D", (self.H,), self.dskip.copy_, lambda: self.dskip
+        yield "norm", (self.inner,), self.norm_w.copy_, lambda: self.norm_w
+        yield "o", (self.width, self.inner), lambda t: self.w_o[:self.width].copy_(t), lambda: self.w_o[:self.width]
+
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext) -> torch.Tensor:
+        from ..ops import native as nat
+        store = cache.slots[self.index]
+        u = ops.project(x, self.w_in)
+        y = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
+        args = (u, self.conv_w, self.conv_b, self.dt_bias, self.a_log, self.dskip, store["conv"], store["state"])
+        tensor_cores = x.dtype == torch.bfloat16 and nat.ssm_chunk_supported(self.N)
+        short, long = ctx.groups(SHORT if tensor_cores else 1 << 30)
+        if short is not None:
+            nat.ssm_scan(*args, short, self.dims, y)
+        if long is not None:
+            nat.ssm_chunk(*args, long, self.dims, y)
+        g = nat.ssm_gate_norm(y, u, self.norm_w, self.eps, self.parts, store["conv"], ctx.meta, self.dims)
+        return ops.project(g, self.w_o)
+
+
+class LatentAttentionMixer(nn.Module):
+    """Causal attention whose cache is one latent and one rotated key part per token. ``kv_from`` makes the layer read an
+    earlier layer's rows with its own up-projections."""
+
+    KEYS = ("heads", "dim", "rot_dim", "vdim", "kv_rank", "rot", "scale")
+
+    @classmethod
+    def check(cls, m: dict, index: int, layers) -> None:
+        if m["rot_dim"] % 2:
+            raise ValueError(f"layer {index}: rot_dim must be even")
+        if m["rot"]["dims"] != m["rot_dim"]:
+            raise ValueError(f"layer {index}: rot.dims must equal rot_dim")
+        src = m.get("kv_from")
+        if src is None:
+            return
+        if not 0 <= src < index or layers[src]["type"] != "latent_attention" or layers[src]["mixer"].get("kv_from") is not None:
+            raise ValueError(f"layer {index}: kv_from must name an earlier latent attention layer with its own latents")
+        o = layers[src]["mixer"]
+        if any(o[k] != m[k] for k in ("kv_rank", "rot_dim", "rot")):
+            raise ValueError(f"layer {index}: kv_rank, rot_dim and rotation must equal layer {src}'s")
+
+    def __init__(self, m: dict, cfg, index: int, dtype, device):
+        super().__init__()
+        H, dn, dr, dv, r = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        self.row = -(-(r + dr) // 16) * 16
+        self.dims = (H, dn, dr, dv, r, self.row)
+        self.base, self.scale, self.eps = float(m["rot"]["base"]), float(m["scale"]), cfg.norm_eps
+        src = m.get("kv_from")
+        self.own, self.source, self.index = src is None, index if src is None else src, index
+        self.width = cfg.hidden_size
+        self.n_q, self.n_d, self.n_k, self.n_v = H * (dn + dr), (r + dr) if src is None else 0, H * dn, H * dv
+        kw = dict(dtype=dtype, device=device)
+        up8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        self.w_q = frozen(torch.zeros(up8(self.n_q + self.n_d), self.width, **kw))       # queries, then the down-projection
+        self.w_ukv = frozen(torch.zeros(up8(self.n_k + self.n_v), r, **kw))              # keys of all heads, then values
+        self.w_o = frozen(torch.zeros(up8(self.width), self.n_v, **kw))
+        self.norm_w = frozen(torch.zeros(r, device=device)) if self.own else None
+        self._ukv8: Optional[torch.Tensor] = None
+        self.expand = dtype == torch.bfloat16 and dn + dr <= 128 and dv <= 128
+
+    def cache_spec(self) -> CacheSpec:
+        return CacheSpec(page_width=self.row if self.own else 0)
+
+    def named_weights(self):
+        q, d, k, v = self.n_q, self.n_d, self.n_k, self.n_v
+        r = self.dims[4]
+        yield "q", (q, self.width), lambda t: self.w_q[:q].copy_(t), lambda: self.w_q[:q]
+        if self.own:
+            yield "dkv", (d, self.width), lambda t: self.w_q[q:q + d].copy_(t), lambda: self.w_q[q:q + d]
+            yield "dkv.norm", (r,), self.norm_w.copy_, lambda: self.norm_w
+        yield "uk", (k, r), lambda t: self.w_ukv[:k].copy_(t), lambda: self.w_ukv[:k]
+        yield "uv", (v, r), lambda t: self.w_ukv[k:k + v].copy_(t), lambda: self.w_ukv[k:k + v]
+        yield "o", (self.width, v), lambda t: self.w_o[:self.width].copy_(t), lambda: self.w_o[:self.width]
+
+    def _expand_weight(self) -> torch.Tensor:
+        """[keys; values] up-projection with its rank padded to 16-byte rows (the weight itself when it is already)."""
+        r = self.dims[4]
+        if r % 8 == 0:
+            return self.w_ukv
+        if self._ukv8 is None or self._ukv8.device != self.w_ukv.device:
+            self._ukv8 = torch.nn.functional.pad(self.w_ukv, (0, -r % 8)).contiguous()
+        return self._ukv8
+
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext) -> torch.Tensor:
+        from ..ops import native as nat
+        H, dn, dr, dv, r, W = self.dims
+        pages = cache.pages[self.source]
+        qd = ops.project(x, self.w_q)
+        cos, sin = ctx.rope(self.base, dr) if dr else (None, None)
+        nat.latent_prep(qd, self.norm_w, self.eps, cos, sin, self.dims, pages if self.own else None, ctx.meta.slots)
+        o = torch.empty(x.shape[0], H * dv, dtype=x.dtype, device=x.device)
+        short, long = ctx.groups(SHORT if self.expand else 1 << 30)
+        if short is not None:
+            nat.latent_attn(qd, self.w_ukv, self.w_ukv[self.n_k:], pages, short, self.dims, self.scale, o)
+        if long is not None:
+            w = self._expand_weight()
+            for i, q0, n, n_keys in long.host:
+                nat.latent_expand_attn(qd[q0:q0 + n], w, pages, ctx.meta.block_table[i], n_keys, self.dims, self.scale,
+                                       o[q0:q0 + n], ctx.zeros(n))
+        return ops.project(o, self.w_o)
+
+
+MIXERS = {"mamba2": Mamba2Mixer, "latent_attention": LatentAttentionMixer}

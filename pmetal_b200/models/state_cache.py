@@ -1,0 +1,146 @@
+"""Cache of decoders that mix attention over a paged cache with recurrent layers.
+
+Two kinds of storage on one sequence table:
+
+* *pages*: per layer that asks for them a pool ``[num_blocks + 1, 64, width]`` addressed through the block tables of
+  ``PagedBlocks`` (rows of any width: the latent attention layers keep one row per token for all heads);
+* *slots*: per recurrent layer named tensors ``[max_seqs + 1, ...]``; a sequence owns one slot index in all of them from
+  ``add_sequence`` to ``free_sequence``. A slot is never cleared: the kernels start from zeros when a sequence's first
+  token of a step is its position 0.
+
+The last block and the last slot lie outside the pools; padding rows of captured decode steps write there. A recurrent
+state has absorbed every token it saw, so a sequence with slots cannot be cut back (``can_truncate``); ``fork`` copies the
+slot and shares the pages.
+
+``split_groups`` divides a step's sequences into short and long portions, which run on different kernels."""
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+from typing import Dict, List, Optional, Sequence, Tuple
+
+import torch
+
+from .kv_cache import BLOCK, BatchMeta, PagedBlocks
+
+
+@dataclass
+class CacheSpec:
+    """What one layer keeps per token (``page_width`` columns) and per sequence (``slots``: name -> (shape, dtype), a
+    dtype of None is the model's)."""
+    page_width: int = 0
+    slots: Dict[str, Tuple[Tuple[int, ...], Optional[torch.dtype]]] = field(default_factory=dict)
+
+
+class StateCache(PagedBlocks):
+    def __init__(self, specs: Sequence[CacheSpec], num_blocks: int, max_seqs: int, dtype=torch.bfloat16, device="cuda"):
+        super().__init__(num_blocks, device)
+        self.max_seqs = max_seqs
+        self.scratch_block, self.scratch_slot = num_blocks, max_seqs
+        self.pages: Dict[int, torch.Tensor] = {}
+        self.slots: Dict[int, Dict[str, torch.Tensor]] = {}
+        for i, s in enumerate(specs):
+            if s.page_width:
+                self.pages[i] = torch.zeros(num_blocks + 1, BLOCK, s.page_width, dtype=dtype, device=device)
+            if s.slots:
+                self.slots[i] = {n: torch.zeros(max_seqs + 1, *shape, dtype=dt or dtype, device=device)
+                                 for n, (shape, dt) in s.slots.items()}
+        self.can_truncate = not self.slots
+        self.free_slots: List[int] = list(range(max_seqs - 1, -1, -1))
+        self.slot_of: Dict[int, int] = {}
+
+    def _copy_block(self, dst: int, src: int) -> None:
+        for t in self.pages.values():
+            t[dst].copy_(t[src])
+
+    def nbytes(self) -> int:
+        ts = list(self.pages.values()) + [t for d in self.slots.values() for t in d.values()]
+        return sum(t.numel() * t.element_size() for t in ts)
+
+    # ------------------------------------------------------------------ sequences
+    def can_admit(self) -> bool:
+        return bool(self.free_slots)
+
+    def add_sequence(self, seq_id: int) -> None:
+        if not self.free_slots:
+            raise MemoryError(f"all {self.max_seqs} state slots are in use")
+        super().add_sequence(seq_id)
+        self.slot_of[seq_id] = self.free_slots.pop()
+
+    def free_sequence(self, seq_id: int) -> None:
+        super().free_sequence(seq_id)
+        self.free_slots.append(self.slot_of.pop(seq_id))
+
+    def fork(self, src_id: int, dst_id: int) -> None:
+        if not self.free_slots:
+            raise MemoryError(f"all {self.max_seqs} state slots are in use")
+        super().fork(src_id, dst_id)
+        a, b = self.slot_of[src_id], self.free_slots.pop()
+        self.slot_of[dst_id] = b
+        for d in self.slots.values():
+            for t in d.values():
+                t[b].copy_(t[a])
+
+    def truncate(self, seq_id: int, new_len: int) -> None:
+        if new_len not in (0, self.seqs[seq_id].length) and not self.can_truncate:
+            raise ValueError("a recurrent state cannot drop tokens it has absorbed")
+        super().truncate(seq_id, new_len)
+
+    # ------------------------------------------------------------------ batch metadata
+    def prepare(self, seq_ids: Sequence[int], new_tokens: Sequence[int]) -> BatchMeta:
+        meta = super().prepare(seq_ids, new_tokens)
+        dev = self.device
+        meta.state_slots = torch.tensor([self.slot_of[s] for s in seq_ids], dtype=torch.int32).to(dev, non_blocking=True)
+        meta.seq_of = torch.repeat_interleave(torch.arange(len(seq_ids), dtype=torch.int32),
+                                              torch.tensor(list(new_tokens))).to(dev, non_blocking=True)
+        return meta
+
+
+@dataclass
+class SeqGroup:
+    """Some sequences of a step, as the kernels take them. ``q_start`` points into the step's token rows, ``c_start`` into
+    rows counted over the group alone."""
+    n: int
+    n_tok: int
+    max_q: int
+    max_kv: int
+    block_table: torch.Tensor
+    seq_lens: torch.Tensor
+    q_start: torch.Tensor
+    q_lens: torch.Tensor
+    c_start: torch.Tensor
+    state_slots: Optional[torch.Tensor]
+    host: List[Tuple[int, int, int, int]] = field(default_factory=list)     # (batch index, q_start, q_len, seq_len)
+
+
+def split_groups(meta: BatchMeta, limit: int) -> Tuple[Optional[SeqGroup], Optional[SeqGroup]]:
+    """(sequences with at most ``limit`` new tokens, the others); None for an empty side. A step whose lengths are not
+    known on the host (a captured one) has one token per sequence."""
+    if meta.host is None:
+        if meta.max_q != 1:
+            raise ValueError("a step without host metadata must bring one token per sequence")
+        n = meta.q_lens.shape[0]
+        return SeqGroup(n, n, 1, meta.max_kv, meta.block_table, meta.seq_lens, meta.q_start, meta.q_lens, meta.q_start,
+                        meta.state_slots), None
+    _, _, seq_lens, q_start, q_lens, _ = meta.host
+    sides = ([i for i, q in enumerate(q_lens) if q <= limit], [i for i, q in enumerate(q_lens) if q > limit])
+    out = []
+    for ix in sides:
+        if not ix:
+            out.append(None)
+            continue
+        c, c_start = 0, []
+        for i in ix:
+            c_start.append(c)
+            c += q_lens[i]
+        host = [(i, q_start[i], q_lens[i], seq_lens[i]) for i in ix]
+        mq, mk = max(q_lens[i] for i in ix), max(seq_lens[i] for i in ix)
+        if len(ix) == len(q_lens):
+            out.append(SeqGroup(len(ix), c, mq, mk, meta.block_table, meta.seq_lens, meta.q_start, meta.q_lens,
+                                meta.q_start, meta.state_slots, host))
+            continue
+        dev = meta.q_lens.device
+        sel = torch.tensor(ix, dtype=torch.int64).to(dev, non_blocking=True)
+        cs = torch.tensor(c_start, dtype=torch.int32).to(dev, non_blocking=True)
+        out.append(SeqGroup(len(ix), c, mq, mk, meta.block_table[sel], meta.seq_lens[sel], meta.q_start[sel],
+                            meta.q_lens[sel], cs, meta.state_slots[sel] if meta.state_slots is not None else None, host))
+    return out[0], out[1]

@@ -630,3 +630,31 @@ def token_logprobs(hidden: torch.Tensor, weight: torch.Tensor, tokens: torch.Ten
         lp = torch.log_softmax(lg, -1).gather(-1, t.clamp(min=0)[:, None])[:, 0]
         out.append(torch.where(t >= 0, lp, torch.zeros_like(lp)))
     return torch.cat(out)
+
+
+# ------------------------------------------------------------------------------------------- serving projections
+GEMV_ROWS = 16          # rows up to which a projection runs on the mat-vec kernel instead of tensor-core tiles
+
+
+def gemv_fits(rows: int, k: int) -> bool:
+    """Whether the mat-vec kernel can stage ``rows`` rows of ``k`` bf16 values."""
+    return rows <= GEMV_ROWS and k % 8 == 0 and (4 if rows <= 4 else 8 if rows <= 8 else 16) * k * 2 <= 200 * 1024
+
+
+def project(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x [M, K] w^T for serving (no autograd), w [N, K]: bf16 on the mat-vec kernel (a few rows) or the tensor-core GEMM;
+    fp32 and shapes that cannot be copied in 16-byte pieces on the vendor GEMM, fp32 in full precision."""
+    if x.dtype != torch.bfloat16 or w.shape[1] % 8 or w.shape[0] % 8 or x.stride(0) % 8 or not use_native(x):
+        return F.linear(x, w)
+    nat = _native()
+    return nat.gemv_ex(x, w) if gemv_fits(x.shape[0], x.shape[1]) else nat.gemm(x, w)
+
+
+def project_f32(x: torch.Tensor, w: torch.Tensor, n: int) -> torch.Tensor:
+    """First ``n`` columns of x w^T as fp32 (read-out)."""
+    if x.dtype != torch.bfloat16 or w.shape[1] % 8 or x.stride(0) % 8 or not use_native(x):
+        return F.linear(x, w[:n]).float()
+    nat = _native()
+    if gemv_fits(x.shape[0], x.shape[1]):
+        return nat.gemv_ex(x, w, out_f32=True, n=n)
+    return nat.gemm_f32(x, w)[:, :n]

@@ -49,15 +49,25 @@ def _load():
     except OSError as e:  # pragma: no cover
         _ERR = str(e)
         return
-    for name in dir(_LIB):
-        pass
     for fn in ("pm_gemm_bf16", "pm_gemm_bf16_2sm", "pm_rmsnorm_fwd", "pm_rmsnorm_bwd", "pm_rope_table", "pm_qknorm_rope_fwd",
                "pm_qknorm_rope_bwd", "pm_swiglu_fwd", "pm_swiglu_bwd", "pm_ce_fwd_bwd", "pm_sumsq", "pm_adamw_flat",
                "pm_attn_delta", "pm_attn_fwd", "pm_attn_bwd", "pm_f32_to_bf16", "pm_paged_attn", "pm_kv_append", "pm_attn_fwd_tc", "pm_attn_bwd_tc", "pm_dequant_4bit", "pm_sample", "pm_spec_verify", "pm_count_tokens",
                "pm_moe_route", "pm_moe_gather", "pm_moe_combine", "pm_gguf_dequant_bf16", "pm_fp8_quant", "pm_fp8_dequant",
                "pm_kd_fwd_bwd", "pm_merge_fused", "pm_dot_norms", "pm_attn_fwd_tc_rect", "pm_attn_fwd_tc_rect_v1", "pm_gemv",
                "pm_qknorm_rope_cache"):
-        getattr(_LIB, fn).restype = c_int
+        if hasattr(_LIB, fn):               # a partial library (``require``) holds some of them
+            getattr(_LIB, fn).restype = c_int
+
+
+def require(component: str) -> None:
+    """Make sure that the kernels of ``component`` can be loaded: the full library when it has been built, else a library
+    of just that component's sources, compiled now (``build.COMPONENTS``)."""
+    global LIB_PATH, _ERR
+    if _LIB is not None or os.path.exists(LIB_PATH):
+        return
+    from ..build import build_component
+    LIB_PATH = build_component(component)
+    _ERR = None
 
 
 def available() -> bool:
@@ -1078,6 +1088,20 @@ def gemv(x, w, norm_w=None, eps: float = 1e-6, residual=None, swiglu: bool = Fal
     return y
 
 
+def gemv_ex(x, w, bias=None, glu=None, out_f32: bool = False, n: Optional[int] = None):
+    """x [M <= 16, K] bf16, w [>= n, K] bf16 -> [M, n]: products plus ``bias`` (fp32). ``glu`` = (limit, beta, shift): w
+    stacks gate rows above up rows and the result is the clamped gated unit, n = rows / 2. ``out_f32``: fp32 result."""
+    M, K = x.shape
+    N = n if n is not None else (w.shape[0] // 2 if glu else w.shape[0])
+    y = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
+    lim, beta, shift = glu if glu else (0.0, 0.0, 0.0)
+    _chk(lib().pm_gemv_ex(_p(x), c_int(x.stride(0)), _p(w), c_int(w.stride(0)), _p(None), c_float(0.0), _p(None), c_int(0),
+                          _p(y), c_int(N), c_int(M), c_int(N), c_int(K), c_int(1 if glu else 0), c_float(1.0), _p(None),
+                          c_int(0), _p(None), c_int(0), (c_int * 4)(*([0x7FFFFFFF] * 4)), _p(bias), c_int(1 if glu else 0),
+                          c_float(lim), c_float(beta), c_float(shift), c_int(int(out_f32)), _stream()), "pm_gemv_ex")
+    return y
+
+
 def gemv_q4(x, q, norm_w=None, eps: float = 1e-6, residual=None, swiglu: bool = False, alpha: float = 1.0, t=None,
             lora_b=None, r: int = 0, seg_sizes: Sequence[int] = ()):
     """As ``gemv`` with the weight given as a 4-bit ``QuantizedTensor`` (nf4 / fp4) of shape [N_w, K]: the codes are
@@ -1147,3 +1171,152 @@ def decode_scratch(M: int, H: int, hq: int, hkv: int, I: int, n_split: int, devi
                 part_ml=torch.empty(n_split, M, hq, 2, dtype=torch.float32, device=device),
                 counters=torch.zeros(M * hkv, dtype=torch.int32, device=device),
                 bar=torch.zeros(2, dtype=torch.int32, device=device), n_split=n_split)
+
+
+# ------------------------------------------------------------------------------------------- fp32-stream decoders
+def _is_f32(t: torch.Tensor) -> c_int:
+    if t.dtype not in (torch.float32, torch.bfloat16):
+        raise TypeError(f"fp32 or bf16 expected, got {t.dtype}")
+    return c_int(int(t.dtype == torch.float32))
+
+
+def embed_scale(ids, table, scale: float):
+    """(fp32 stream [n, width], the same in the table's type) = table[ids] * scale."""
+    n, width = ids.shape[0], table.shape[1]
+    xf = torch.empty(n, width, dtype=torch.float32, device=table.device)
+    xc = xf if table.dtype == torch.float32 else torch.empty(n, width, dtype=table.dtype, device=table.device)
+    _chk(lib().pm_embed_scale(_p(ids), _p(table), _is_f32(table), c_float(scale), c_int(n), c_int(width), _p(xf),
+                              _p(None if xc is xf else xc), _stream()), "pm_embed_scale")
+    return xf, xc
+
+
+def post_layernorm(x, y, w, b, eps: float, alpha: float = 1.0, bias=None, rows=None, want_stream: bool = True, dtype=None):
+    """LN(alpha * x + y + bias) * w + b on the fp32 stream x [n, width] -> (fp32 result or None, result in ``dtype``).
+    y (compute type, any row stride) and bias (fp32) may be None; ``rows`` (int64) picks rows of x and y."""
+    dtype = dtype or (y.dtype if y is not None else x.dtype)
+    n, width = (rows.shape[0] if rows is not None else x.shape[0]), x.shape[1]
+    single = dtype == torch.float32
+    of = torch.empty(n, width, dtype=torch.float32, device=x.device) if (want_stream or single) else None
+    oc = None if single else torch.empty(n, width, dtype=dtype, device=x.device)
+    if y is not None and (y.dtype != dtype or y.stride(1) != 1):
+        raise ValueError("y must have the compute type and contiguous rows")
+    _chk(lib().pm_post_layernorm(_p(x), _p(y), c_int(int(single)), c_ll(y.stride(0) if y is not None else 0), _p(bias),
+                                 c_float(alpha), _p(w), _p(b), c_float(eps), c_int(n), c_int(width), _p(rows), _p(of),
+                                 _p(oc), _stream()), "pm_post_layernorm")
+    return of, (of if single else oc)
+
+
+def clamped_glu(gu, ff: int, limit: float, beta: float, shift: float, bias=None):
+    """gu [n, >= 2 ff] (gate columns, then up columns), bias fp32 [2 ff] or None -> [n, ff]."""
+    out = torch.empty(gu.shape[0], ff, dtype=gu.dtype, device=gu.device)
+    _chk(lib().pm_clamped_glu(_p(gu), _is_f32(gu), c_ll(gu.stride(0)), _p(bias), c_int(gu.shape[0]), c_int(ff),
+                              c_float(limit), c_float(beta), c_float(shift), _p(out), _stream()), "pm_clamped_glu")
+    return out
+
+
+def rope_table_f64(positions, freq):
+    """cos / sin [n, half] fp32 of positions (int32) times freq (fp64 [half]), angles formed and reduced in fp64."""
+    n, half = positions.shape[0], freq.shape[0]
+    cs = torch.empty(n, half, dtype=torch.float32, device=positions.device)
+    sn = torch.empty_like(cs)
+    _chk(lib().pm_rope_table_f64(_p(positions), _p(freq), c_int(n), c_int(half), _p(cs), _p(sn), _stream()),
+         "pm_rope_table_f64")
+    return cs, sn
+
+
+# ------------------------------------------------------------------------------------------- state-space layers
+def ssm_scan(u, conv_w, conv_b, dt_bias, a_log, dskip, ring, state, group, dims, y) -> None:
+    """Recurrence token by token for the sequences of ``group`` (models/state_cache.SeqGroup); ``dims`` = (heads, channels
+    per head, state rows, groups, taps). Writes the rows of y [tokens, heads * channels]; layouts in csrc/ssm.cu."""
+    H, P, N, G, taps = dims
+    _chk(lib().pm_ssm_scan(_p(u), _is_f32(u), c_ll(u.stride(0)), _p(conv_w), _p(conv_b), _p(dt_bias), _p(a_log), _p(dskip),
+                           _p(ring), _p(state), _p(group.state_slots), _p(group.q_start), _p(group.q_lens),
+                           _p(group.seq_lens), c_int(group.n), c_int(H), c_int(P), c_int(N), c_int(G), c_int(taps), _p(y),
+                           _stream()), "pm_ssm_scan")
+
+
+def ssm_chunk_supported(n_state: int) -> bool:
+    return n_state <= 128
+
+
+def ssm_chunk(u, conv_w, conv_b, dt_bias, a_log, dskip, ring, state, group, dims, y) -> None:
+    """As ``ssm_scan`` for longer portions of bf16 models: convolution for all tokens, then the recurrence in blocks of 64
+    tokens on the tensor cores."""
+    global LAUNCHES
+    H, P, N, G, taps = dims
+    T = u.shape[0]
+    act = torch.empty(T, H * P + 2 * G * N, dtype=torch.bfloat16, device=u.device)
+    dt = torch.empty(T, H, dtype=torch.float32, device=u.device)
+    _chk(lib().pm_ssm_chunk(_p(u), c_ll(u.stride(0)), _p(conv_w), _p(conv_b), _p(dt_bias), _p(a_log), _p(dskip), _p(ring),
+                            _p(state), _p(group.state_slots), _p(group.q_start), _p(group.q_lens), _p(group.seq_lens),
+                            c_int(group.n), c_int(group.max_q), c_int(H), c_int(P), c_int(N), c_int(G), c_int(taps),
+                            _p(act), _p(dt), _p(y), _stream()), "pm_ssm_chunk")
+    LAUNCHES += 1          # two kernels
+
+
+def ssm_gate_norm(y, u, w, eps: float, parts: int, ring, meta, dims):
+    """RMS norm in ``parts`` equal parts of y * silu(first columns of u), times w; updates the convolution ring."""
+    H, P, N, G, taps = dims
+    out = torch.empty_like(y)
+    _chk(lib().pm_ssm_gate_norm(_p(y), _p(u), _is_f32(u), c_ll(u.stride(0)), _p(w), c_float(eps), c_int(parts), _p(out),
+                                _p(ring), _p(meta.state_slots), _p(meta.seq_of), _p(meta.positions), _p(meta.seq_lens),
+                                c_int(y.shape[0]), c_int(H), c_int(P), c_int(N), c_int(G), c_int(taps), _stream()),
+         "pm_ssm_gate_norm")
+    return out
+
+
+# ------------------------------------------------------------------------------------------- latent attention
+def latent_prep(qd, norm_w, eps: float, cos, sin, dims, pages, slots) -> None:
+    """Rotates the queries in place; with ``pages`` the latent and rotated key of every token go to its cache row. ``dims`` =
+    (heads, unrotated, rotated, value channels, rank, row width)."""
+    H, dn, dr, _, rank, W = dims
+    _chk(lib().pm_latent_prep(_p(qd), _is_f32(qd), c_ll(qd.stride(0)), _p(norm_w), c_float(eps), _p(cos), _p(sin),
+                              c_int(qd.shape[0]), c_int(H), c_int(dn), c_int(dr), c_int(rank), _p(pages), c_int(W),
+                              _p(slots), _stream()), "pm_latent_prep")
+
+
+def latent_mma_supported(H: int, W: int, rank: int) -> bool:
+    return bool(lib().pm_latent_mma_supported(c_int(H), c_int(W), c_int(rank)))
+
+
+def latent_attn(qd, wuk, wuv, pages, group, dims, scale: float, out) -> None:
+    """Attention in the latent space for the sequences of ``group``: rows of out [tokens, >= heads * value channels]."""
+    global LAUNCHES
+    H, dn, dr, dv, rank, W = dims
+    n_split = 1
+    if qd.dtype == torch.bfloat16 and latent_mma_supported(H, W, rank):
+        tile = 32 if H > 16 else 16
+        ctas = group.n * -(-group.max_q * H // tile)
+        n_blocks = -(-group.max_kv // 64)
+        n_split = max(1, min(sm_count() // max(ctas, 1), n_blocks, 64))
+    dev = qd.device
+    q_lat = torch.empty(group.n_tok, H, W, dtype=qd.dtype, device=dev)
+    po = torch.empty(n_split, group.n_tok * H, rank, dtype=torch.float32, device=dev)
+    pml = torch.empty(n_split, group.n_tok * H, 2, dtype=torch.float32, device=dev)
+    _chk(lib().pm_latent_attn(_p(qd), _is_f32(qd), c_ll(qd.stride(0)), _p(wuk), _p(wuv), _p(pages), _p(group.block_table),
+                              _p(group.seq_lens), _p(group.q_start), _p(group.c_start), _p(group.q_lens), c_int(group.n),
+                              c_int(group.block_table.shape[1]), c_int(group.n_tok), c_int(group.max_q), c_int(H), c_int(dn),
+                              c_int(dr), c_int(dv), c_int(rank), c_int(W), c_int(n_split), c_float(scale), _p(q_lat), _p(po),
+                              _p(pml), _p(out), c_ll(out.stride(0)), _stream()), "pm_latent_attn")
+    LAUNCHES += 2          # three kernels
+
+
+def latent_expand_attn(qd, wukv, pages, table_row, n_keys: int, dims, scale: float, out, zeros) -> None:
+    """Attention of one sequence's new tokens (rows of qd / out) over its ``n_keys`` positions with keys and values expanded
+    from the latents: one GEMM, then the flash-attention kernel. ``zeros``: int32 zeros, at least as many as new tokens."""
+    H, dn, dr, dv, rank, W = dims
+    n_q, dev = qd.shape[0], qd.device
+    r8 = wukv.shape[1]
+    lat = torch.empty(n_keys, r8, dtype=torch.bfloat16, device=dev)
+    _chk(lib().pm_latent_gather(_p(pages), _p(table_row), c_int(n_keys), c_int(W), c_int(rank), c_int(r8), _p(lat),
+                                _stream()), "pm_latent_gather")
+    kv = gemm(lat, wukv)
+    q128 = torch.empty(n_q, H, 128, dtype=torch.bfloat16, device=dev)
+    k128 = torch.empty(n_keys, H, 128, dtype=torch.bfloat16, device=dev)
+    v128 = torch.empty(n_keys, H, 128, dtype=torch.bfloat16, device=dev)
+    _chk(lib().pm_latent_assemble(_p(qd), c_ll(qd.stride(0)), c_int(n_q), _p(kv), c_ll(kv.stride(0)), c_int(n_keys),
+                                  _p(pages), _p(table_row), c_int(W), c_int(rank), c_int(H), c_int(dn), c_int(dr),
+                                  c_int(dv), _p(q128), _p(k128), _p(v128), _stream()), "pm_latent_assemble")
+    o, _ = attn_fwd_rect(q128, k128, v128, zeros[:n_q], scale, n_keys - n_q)
+    _chk(lib().pm_latent_take(_p(o), c_int(n_q), c_int(H), c_int(dv), _p(out), c_ll(out.stride(0)), _stream()),
+         "pm_latent_take")

@@ -102,13 +102,19 @@ class EngineStats:
 class ContinuousBatchEngine:
     def __init__(self, model, eos_ids: Sequence[int] = (), max_slots: int = 64, num_blocks: int = 8192,
                  prefill_chunk: int = PREFILL_CHUNK, prefix_cache: bool = True, max_queue: int = 1024,
-                 cache_options: Optional[dict] = None, adapters=None):
+                 cache_options: Optional[dict] = None, adapters=None, mixed_batches: Optional[bool] = None):
         self.model = model
+        # one step per tick for the prompt portion and all decoded tokens together, instead of two model calls
+        self.mixed = getattr(model, "mixed_batches", False) if mixed_batches is None else bool(mixed_batches)
         self.adapters = adapters        # lora.batched.AdapterSet: every request picks an adapter (or none) by name
         opts = dict(cache_options or {})
+        if getattr(model, "slotted_cache", False):
+            opts["max_seqs"] = max_slots
         self.gen = Generator(model, cache=model.new_cache(num_blocks, **opts)) if opts else Generator(model, num_blocks=num_blocks)
         if opts.get("window"):
             prefix_cache = False      # a rotating cache recycles prompt blocks: there is no stable prefix to share
+        if not self.gen.cache.can_truncate:
+            prefix_cache = False      # a recurrent state belongs to the whole prefix it has read, not to a part of it
         if adapters is not None:
             self.gen.cuda_graphs = False      # the adapter of every row changes from step to step
             prefix_cache = False              # cached keys/values depend on the adapter that produced them
@@ -135,6 +141,7 @@ class ContinuousBatchEngine:
             if self.adapters is None:
                 raise KeyError(f"no adapters are loaded (request asked for {req.adapter!r})")
             self.adapters.index(req.adapter)         # raises KeyError for an unknown name
+        self.gen.check_tokens(req.prompt)
         with self._lock:
             if len(self.queue) >= self.max_queue:
                 raise RuntimeError("queue full")
@@ -161,7 +168,7 @@ class ContinuousBatchEngine:
         return (len(req.prompt) + req.params.max_tokens + BLOCK - 1) // BLOCK + 1
 
     def _admit(self) -> None:
-        while self.queue and len(self.slots) < self.max_slots:
+        while self.queue and len(self.slots) < self.max_slots and self.cache.can_admit():
             req = self.queue[0]
             need = self._blocks_needed(req)
             reserved = sum(self._blocks_needed(s.req) - (self.cache.length(s.seq) // BLOCK) for s in self.slots)
@@ -314,6 +321,8 @@ class ContinuousBatchEngine:
         if not self.slots:
             return False
         pre = next((s for s in self.slots if s.state == "prefill"), None)
+        if self.mixed and pre is not None and self.adapters is None:
+            return self._mixed_tick(pre)
         if pre is not None:
             t0 = time.perf_counter()
             req = pre.req
@@ -343,6 +352,33 @@ class ContinuousBatchEngine:
                 self._emit(s, ids[j], lps[j] if lps else None)
             self.stats.decode_steps += 1
             self.stats.decode_seconds += time.perf_counter() - t0
+        return True
+
+    def _mixed_tick(self, pre: _Slot) -> bool:
+        """The next portion of one prompt and one token of every decoding slot as a single batch."""
+        t0 = time.perf_counter()
+        req = pre.req
+        dec = [s for s in self.slots if s.state == "decode" and s.last_token >= 0]
+        take = min(self.prefill_chunk, len(req.prompt) - pre.prefill_pos)
+        portion = req.prompt[pre.prefill_pos:pre.prefill_pos + take]
+        done = pre.prefill_pos + take == len(req.prompt)
+        logits = self.gen.step([pre.seq] + [s.seq for s in dec], [portion] + [[s.last_token] for s in dec],
+                               [[take - 1] if done else []] + [[0]] * len(dec))
+        pre.prefill_pos += take
+        slots = list(dec)
+        if done:
+            if self.prefix is not None:
+                self.prefix.insert(pre.seq, req.prompt)
+            pre.state = "decode"
+            slots = [pre] + slots
+        if slots:
+            ids, lps = self._sample(logits, slots)
+            for j, s in enumerate(slots):
+                self._emit(s, ids[j], lps[j] if lps else None)
+        dt = time.perf_counter() - t0
+        self.stats.prefill_seconds += dt
+        if dec:
+            self.stats.decode_steps += 1
         return True
 
     # ------------------------------------------------------------------ background pump

@@ -74,7 +74,7 @@ def _portable_model_dir(model: str) -> Optional[str]:
     llama / qwen2 / qwen3 / qwen3-moe / mistral family of the hand-written kernels), else None."""
     import json as _json
 
-    from ..models.architectures import family_of
+    from ..models.architectures import PAGED_FAMILIES, family_of
     from ..models.loader import resolve_model_path
     try:
         path = resolve_model_path(model)
@@ -85,7 +85,7 @@ def _portable_model_dir(model: str) -> Optional[str]:
         return None
     with open(cfg_path, "r", encoding="utf-8") as fh:
         fam = family_of(_json.load(fh))
-    return path if fam not in (None, "fast") else None
+    return path if fam is not None and fam not in PAGED_FAMILIES else None
 
 
 def _run_portable_training(job: "TrainingJobConfig", model_dir: str, dev, dtype, out_dir: str, phase, callbacks, t_start) -> dict:
@@ -261,6 +261,8 @@ def run_training(job: TrainingJobConfig, phase_cb: Optional[Callable[[str], None
             return summary
         phase("loading_model")
         model, margs, model_dir = load_pretrained(job.model, dtype, dev, seed=tcfg.seed)
+        if not hasattr(model, "fused_linears"):
+            raise ValueError(f"{margs.model_type} models are served, not trained")
         max_seq = tcfg.max_seq_len if tcfg.max_seq_len and tcfg.max_seq_len != 8192 else min(
             margs.max_position_embeddings, 8192)
         # ---- tokenizer + dataset
