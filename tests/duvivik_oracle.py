@@ -1,9 +1,33 @@
 """Plain, slow statement of the Duvivik decoder on whole sequences (PyTorch, CPU, fp32 or fp64), one function per
 mechanism. It shares no code with the package: the tests compare the product path with it. ``p`` maps checkpoint names to
-tensors, ``cfg`` is the parsed configuration; sequences are [T, width] with positions 0 .. T - 1."""
+tensors, ``cfg`` is the parsed configuration; sequences are [T, width] with positions 0 .. T - 1.
+
+``low`` marks every value that a bf16 model may hold in bf16 (projection inputs and outputs, convolution outputs, cached
+latents, attention outputs). It is the identity; inside ``rounding()`` it rounds to bf16, which shows how much of a
+difference such rounding alone explains."""
+import contextlib
 import math
 
 import torch
+
+_ROUND = [False]
+
+
+def low(x):
+    return x.to(torch.bfloat16).to(x.dtype) if _ROUND[0] else x
+
+
+@contextlib.contextmanager
+def rounding():
+    _ROUND[0] = True
+    try:
+        yield
+    finally:
+        _ROUND[0] = False
+
+
+def linear(x, w):
+    return low(low(x) @ w.t())
 
 
 def layer_norm(x, w, b, eps):
@@ -42,7 +66,7 @@ def causal_conv(x, w, b):
             if src >= 0:
                 acc = acc + w[:, j] * x[src]
         out[t] = acc
-    return out * torch.sigmoid(out)
+    return low(out * torch.sigmoid(out))
 
 
 def ssd_recurrence(x, B, C, dt, A_log, D, S=None):
@@ -67,7 +91,7 @@ def gated_group_norm(y, z, w, groups, eps):
 
 def mamba2(h, p, pre, m, eps):
     inner, gn = m["heads"] * m["vdim"], m["groups"] * m["state"]
-    u = h @ p[pre + "in"].t()
+    u = linear(h, p[pre + "in"])
     z, xbc, dt = u[:, :inner], u[:, inner:2 * inner + 2 * gn], u[:, 2 * inner + 2 * gn:]
     assert dt.shape[1] == m["heads"]
     xbc = causal_conv(xbc, p[pre + "conv"], p[pre + "conv.b"])
@@ -78,36 +102,36 @@ def mamba2(h, p, pre, m, eps):
     v = dt + p[pre + "dt_bias"]
     dt = torch.logaddexp(v, torch.zeros_like(v))
     y, _ = ssd_recurrence(x, B, C, dt, p[pre + "A_log"], p[pre + "D"])
-    y = gated_group_norm(y.reshape(T, inner), z, p[pre + "norm"], m["norm_groups"], eps)
-    return y @ p[pre + "o"].t()
+    y = gated_group_norm(low(y.reshape(T, inner)), z, p[pre + "norm"], m["norm_groups"], eps)
+    return linear(y, p[pre + "o"])
 
 
 def latent_kv(h, p, pre, m, eps):
     """What a layer with its own down-projection leaves for itself and for the layers that read it."""
-    u = h @ p[pre + "dkv"].t()
+    u = linear(h, p[pre + "dkv"])
     r = m["kv_rank"]
     c = rms(u[:, :r], eps) * p[pre + "dkv.norm"]
-    return c, rotate_pairs(u[:, r:], m["rot"]["base"])
+    return low(c), low(rotate_pairs(u[:, r:], m["rot"]["base"]))
 
 
 def latent_attention(h, p, pre, m, c, kr):
     T, H, dn, dr, dv = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"]
-    q = (h @ p[pre + "q"].t()).reshape(T, H, dn + dr)
-    qr = rotate_pairs(q[..., dn:], m["rot"]["base"])
-    k = (c @ p[pre + "uk"].t()).reshape(T, H, dn)
-    v = (c @ p[pre + "uv"].t()).reshape(T, H, dv)
+    q = linear(h, p[pre + "q"]).reshape(T, H, dn + dr)
+    qr = low(rotate_pairs(q[..., dn:], m["rot"]["base"]))
+    k = linear(c, p[pre + "uk"]).reshape(T, H, dn)
+    v = linear(c, p[pre + "uv"]).reshape(T, H, dv)
     out = torch.zeros(T, H, dv, dtype=h.dtype)
     for i in range(T):
         for hd in range(H):
             s = (k[:i + 1, hd] @ q[i, hd, :dn] + kr[:i + 1] @ qr[i, hd]) * m["scale"]
             out[i, hd] = torch.softmax(s, 0) @ v[:i + 1, hd]
-    return out.reshape(T, H * dv) @ p[pre + "o"].t()
+    return linear(out.reshape(T, H * dv), p[pre + "o"])
 
 
 def clamped_glu(h, p, pre, limit):
-    g = torch.minimum(h @ p[pre + "gate"].t() + p[pre + "gate.b"], torch.tensor(limit, dtype=h.dtype))
-    u = (h @ p[pre + "up"].t() + p[pre + "up.b"]).clamp(-limit, limit)
-    return (g * torch.sigmoid(1.702 * g) * (u + 1)) @ p[pre + "down"].t() + p[pre + "down.b"]
+    g = torch.minimum(linear(h, p[pre + "gate"]) + p[pre + "gate.b"], torch.tensor(limit, dtype=h.dtype))
+    u = (linear(h, p[pre + "up"]) + p[pre + "up.b"]).clamp(-limit, limit)
+    return linear(g * torch.sigmoid(1.702 * g) * (u + 1), p[pre + "down"]) + p[pre + "down.b"]
 
 
 def forward(tokens, p, cfg):
@@ -130,4 +154,4 @@ def forward(tokens, p, cfg):
             x = layer_norm(alpha * x + y, p[f"l{i}.norm2"], p[f"l{i}.norm2.b"], eps)
         stream.append(x)
     x = layer_norm(x, p["final.norm"], p["final.norm.b"], eps)
-    return x @ p["head"].t(), torch.stack(stream)
+    return low(x) @ p["head"].t(), torch.stack(stream)
