@@ -8,6 +8,8 @@ Config (the reference's LoRA SFT benchmark re-stated for one NVSwitch box): 28 l
 LoRA r=16 alpha=32 on all seven projections; synthetic documents with lengths uniform in [64, 2048]
 packed to 4096 tokens with per-document causal masking; 4 packs per GPU per step; data parallel over N GPUs.
 
+    python bench.py --serve-hybrid [PRESET ...]     (serving of the hybrid decoder, its own report)
+
 Prints one JSON line on rank 0. ``value`` is whole-job tokens/s over K device-timed steps (CUDA events,
 max over ranks); ``e2e`` is the same step driven through the public training-loop API with the batch
 copied from pinned host memory and the loss read back every step.
@@ -148,7 +150,19 @@ def main() -> None:
     ap.add_argument("--profile-step", action="store_true",
                     help="after the warm-up, run one extra (untimed) step under the profiler and print per-kernel device "
                          "times to stderr")
+    ap.add_argument("--serve-hybrid", nargs="*", metavar="PRESET", default=None,
+                    help="instead of the headline benchmark: prefill / decode throughput and kernel times of the hybrid "
+                         "decoder presets (default duvivik-1b duvivik-4b) beside the dense decoder of equal size")
     args = ap.parse_args()
+    if args.serve_hybrid is not None:
+        from pmetal_b200.bench.hybrid_serve import report
+        sampler = ClockSampler(0)
+        sampler.start()
+        t0 = time.time()
+        res = report(args.serve_hybrid or ["duvivik-1b", "duvivik-4b"])
+        res["clocks"] = sampler.stop(t0, time.time())
+        print(json.dumps(res))
+        return
     if args.impl == "reference":
         reference_arm(args)
         return

@@ -1,0 +1,234 @@
+"""Serving throughput of the hybrid decoder beside the dense fast decoder at equal size, and its kernels beside the like
+kernels of the existing models (``bench.py --serve-hybrid``). Random weights; device time by CUDA events."""
+from __future__ import annotations
+
+import statistics
+from typing import Callable, Dict, List
+
+import torch
+
+from ..models import hybrid_decoder as hd
+from ..models.config import ModelArgs
+from ..models.decoder import DecoderLM
+from ..models.generation import Generator
+from ..models.kv_cache import BLOCK, PagedKVCache
+from ..models.state_cache import CacheSpec, StateCache, split_groups
+from ..ops import native as nat
+from .kernels import peaks
+
+# dense models of the fast path with about the same width, depth of weights and parameter count
+DENSE = {
+    "duvivik-1b": dict(hidden_size=2048, intermediate_size=6144, num_hidden_layers=12, num_attention_heads=16,
+                       num_key_value_heads=8),
+    "duvivik-4b": dict(hidden_size=2560, intermediate_size=9728, num_hidden_layers=19, num_attention_heads=32,
+                       num_key_value_heads=8),
+}
+
+
+def build(name: str, kind: str):
+    args = hd.HybridArgs.from_dict(hd.PRESETS[name])
+    if kind == "hybrid":
+        return hd.HybridDecoderLM(args, torch.bfloat16, "cuda").init_weights(0.02, 0, "cuda").eval()
+    cfg = ModelArgs(vocab_size=args.vocab_size, head_dim=128, tie_word_embeddings=False, **DENSE[name])
+    m = DecoderLM(cfg, torch.bfloat16, "cuda").init_weights_on_device().eval()
+    for p in m.parameters():
+        p.requires_grad_(False)
+    return m
+
+
+def event_ms(fn: Callable[[], None], iters: int) -> float:
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(iters):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / iters
+
+
+def throughput(model, context: int = 1024, prompt: int = 4096, batches=(1, 16, 64), steps: int = 48) -> Dict[str, dict]:
+    """Prefill of one long prompt and of four prompts together; decode of several batch sizes from ``context`` tokens, token
+    ids read back every step."""
+    V = model.cfg.vocab_size
+    g = torch.Generator().manual_seed(0)
+    kw = {"max_seqs": max(batches)} if getattr(model, "slotted_cache", False) else {}
+    gen = Generator(model, cache=model.new_cache(max(batches) * (-(-(context + steps + 16) // BLOCK) + 1) + 4 * prompt // BLOCK, **kw))
+    out = {}
+    for n_seq in (1, 4):
+        prompts = [torch.randint(0, V, (prompt // n_seq,), generator=g).tolist() for _ in range(n_seq)]
+
+        def run():
+            seqs = [gen.new_seq() for _ in prompts]
+            gen.prefill(seqs, prompts, chunk=prompt)
+            for s in seqs:
+                gen.cache.free_sequence(s)
+        for _ in range(3):
+            run()
+        ms = event_ms(run, 5)
+        out[f"prefill_{n_seq}x{prompt // n_seq}"] = {"ms": round(ms, 3), "tokens_per_s": round(prompt / ms * 1e3)}
+    for n in batches:
+        seqs = [gen.new_seq() for _ in range(n)]
+        ids = gen.prefill(seqs, [torch.randint(0, V, (context,), generator=g).tolist() for _ in range(n)]).argmax(-1)
+
+        def step():
+            nonlocal ids
+            ids = gen.decode_step(seqs, ids).argmax(-1)
+            ids.tolist()
+        for _ in range(8):
+            step()
+        ms = event_ms(step, steps)
+        out[f"decode_b{n}"] = {"ms": round(ms, 4), "tokens_per_s": round(n / ms * 1e3, 1)}
+        for s in seqs:
+            gen.cache.free_sequence(s)
+    nat.check_status()
+    return out
+
+
+def graph_us(fn: Callable[[], None], iters: int = 15) -> float:
+    """Median device time of one captured call with a cold L2 (256 MB written before every replay)."""
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    side = torch.cuda.Stream()
+    side.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(side):
+        for _ in range(2):
+            fn()
+    torch.cuda.current_stream().wait_stream(side)
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        fn()
+    ts = []
+    for _ in range(iters + 3):
+        flush.zero_()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        g.replay()
+        b.record()
+        torch.cuda.synchronize()
+        ts.append(a.elapsed_time(b) * 1e3)
+    return statistics.median(ts[3:])
+
+
+def _bf(*shape, scale=1.0):
+    return (torch.randn(*shape, device="cuda") * scale).to(torch.bfloat16)
+
+
+def _group(cache, n_seq: int, prior: int, new: int):
+    """Batch in which ``n_seq`` sequences with ``prior`` cached tokens bring ``new`` each."""
+    for i in range(n_seq):
+        cache.add_sequence(i)
+        if prior:
+            cache.reserve(i, prior)
+    meta = cache.prepare(list(range(n_seq)), [new] * n_seq)
+    return meta, (split_groups(meta, 1 << 30)[0] if isinstance(cache, StateCache) else None)
+
+
+def kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096) -> List[dict]:
+    """Every kernel of the hybrid layers at the sizes of preset ``name`` and, behind it, the like kernel of the other
+    models: bytes and operations that the computation needs, device time, fraction of the slower of the two bounds."""
+    cfg = hd.HybridArgs.from_dict(hd.PRESETS[name])
+    W = cfg.hidden_size
+    at = next(l["mixer"] for l in cfg.layers if l["type"] == "latent_attention")
+    sm = next(l["mixer"] for l in cfg.layers if l["type"] == "mamba2")
+    ff = next(l["mlp"]["ff"] for l in cfg.layers if l["mlp"])
+    H, dn, dr, dv, r = at["heads"], at["dim"], at["rot_dim"], at["vdim"], at["kv_rank"]
+    row = -(-(r + dr) // 16) * 16
+    S = (sm["heads"], sm["vdim"], sm["state"], sm["groups"], sm["conv"])
+    SH, P, N, G, taps = S
+    inner, conv = SH * P, SH * P + 2 * G * N
+    pk, out = peaks(), []
+
+    def case(label, fn, nbytes=0, flops=0):
+        us = graph_us(fn)
+        bound = max(nbytes / pk["hbm_gbs"] / 1e3, flops / pk["bf16_tflops"] / 1e6)
+        out.append({"kernel": label, "us": round(us, 2), "bound_us": round(bound, 2), "of_measured_peak": round(bound / us, 3)})
+
+    f = lambda *s: torch.randn(*s, device="cuda")      # noqa: E731
+    n_in = -(-(inner + conv + SH) // 8) * 8
+    for mode, n_seq, prior, new in (("decode", batch, ctx - 1, 1), ("prefill", 1, 0, prompt)):
+        T = n_seq * new
+        tag = f"{mode} T={T} "
+        # state-space recurrence (with its convolution) | gated delta rule scan
+        c = StateCache([CacheSpec(slots={"conv": ((taps, conv), None), "state": ((SH, N, P), torch.float32)})],
+                       n_seq * (prior + new) // BLOCK + n_seq + 1, n_seq, torch.bfloat16, "cuda")
+        meta, grp = _group(c, n_seq, prior, new)
+        u, y = _bf(T, n_in), torch.empty(T, inner, dtype=torch.bfloat16, device="cuda")
+        vec = (f(taps, conv), f(conv), f(SH) - 3, f(SH), f(SH))
+        fn = nat.ssm_scan if mode == "decode" else nat.ssm_chunk
+        state_b = 2 * n_seq * SH * N * P * 4
+        # products of the blocked form: scores and their use in the block, state in and out
+        blk = 2 * T * SH * (64 * (N + P) / 2 + 2 * N * P) if mode == "prefill" else 0
+        case(tag + "ssm recurrence", lambda: fn(u, *vec, c.slots[0]["conv"], c.slots[0]["state"], grp, S, y),
+             T * (conv + inner + SH) * 2 + state_b, blk)
+        gh = SH * N * P // (128 * 128)
+        q, k, v = f(n_seq, new, gh, 128), f(n_seq, new, gh, 128), f(n_seq, new, gh, 128)
+        gt, st = torch.rand(n_seq, new, gh, device="cuda"), f(n_seq, gh, 128, 128)
+        yy = torch.empty_like(v)
+        call = lambda: nat._chk(nat.lib().pm_gdn_scan(*[nat._p(t) for t in (q, k, v, gt, gt, st, yy)], nat.c_int(n_seq),      # noqa: E731
+                                                      nat.c_int(new), nat.c_int(gh), nat.c_int(128), nat.c_int(128),
+                                                      nat._stream()), "pm_gdn_scan")
+        case(tag + "  | gated delta rule scan", call, 4 * T * gh * 128 * 4 + 2 * n_seq * gh * 128 * 128 * 4,
+             2 * T * gh * (64 * 128 + 2 * 128 * 128) if mode == "prefill" else 0)
+        # row kernels | rms norm, swiglu
+        nw = f(inner)
+        case(tag + "ssm gate + norm", lambda: nat.ssm_gate_norm(y, u, nw, 1e-5, sm["norm_groups"], c.slots[0]["conv"], meta, S),
+             3 * T * inner * 2)
+        x, yo, lw, lb = f(T, W), _bf(T, W), f(W), f(W)
+        case(tag + "residual sum + layer norm", lambda: nat.post_layernorm(x, yo, lw, lb, 1e-5, 2.0), T * W * (4 + 2 + 4 + 2))
+        xb, rw = _bf(T, W), _bf(W)
+        case(tag + "  | residual sum + rms norm", lambda: nat.rmsnorm_fwd(xb, rw, 1e-6, yo), 4 * T * W * 2)
+        wgu, bgu = _bf(2 * ff, W, scale=W ** -0.5), f(2 * ff)
+        if mode == "decode":
+            case(tag + "gate/up mat-vec, clamped", lambda: nat.gemv_ex(xb, wgu, bgu, (7.0, 1.702, 1.0), n=ff), 2 * ff * W * 2)
+            case(tag + "  | gate/up mat-vec, swiglu", lambda: nat.gemv(xb, wgu, swiglu=True), 2 * ff * W * 2)
+        else:
+            gu = _bf(T, 2 * ff)
+            case(tag + "clamped gated unit", lambda: nat.clamped_glu(gu, ff, 7.0, 1.702, 1.0, bgu), 3 * T * ff * 2)
+            case(tag + "  | swiglu", lambda: nat.swiglu_fwd(gu), 3 * T * ff * 2)
+        # attention | paged attention of the dense decoder at 16 / 8 heads of 128
+        c2 = StateCache([CacheSpec(page_width=row)], n_seq * (prior + new) // BLOCK + n_seq + 1, n_seq, torch.bfloat16, "cuda")
+        meta, grp = _group(c2, n_seq, prior, new)
+        c2.pages[0].normal_()
+        dims = (H, dn, dr, dv, r, row)
+        qd, wukv = _bf(T, H * (dn + dr) + r + dr), _bf(H * (dn + dv), r, scale=r ** -0.5)
+        cs, sn = f(T, dr // 2), f(T, dr // 2)
+        o = torch.empty(T, H * dv, dtype=torch.bfloat16, device="cuda")
+        case(tag + "latent norm + rotation + append", lambda: nat.latent_prep(qd, nw[:r], 1e-5, cs, sn, dims, c2.pages[0], meta.slots),
+             T * 2 * (2 * H * dr + 2 * (r + dr)))
+        pairs = n_seq * (new * prior + new * (new + 1) // 2)
+        if mode == "decode":
+            case(tag + f"latent attention, {ctx} keys", lambda: nat.latent_attn(qd, wukv, wukv[H * dn:], c2.pages[0], grp, dims, 0.1, o),
+                 n_seq * ctx * row * 2 + wukv.numel() * 2, pairs * H * 2 * (2 * r + dr))
+        else:
+            z = torch.zeros(T, dtype=torch.int32, device="cuda")
+            case(tag + "latent attention, expanded", lambda: nat.latent_expand_attn(qd, wukv, c2.pages[0], meta.block_table[0], T, dims, 0.1, o, z),
+                 0, pairs * H * 2 * (dn + dr + dv) + 2 * T * wukv.numel())
+        c3 = PagedKVCache(1, 8, 128, n_seq * (prior + new) // BLOCK + n_seq + 1, device="cuda")
+        meta3, _ = _group(c3, n_seq, prior, new)
+        c3.k[0].normal_()
+        c3.v[0].normal_()
+        q3 = _bf(T, 16, 128)
+        case(tag + "  | paged attention", lambda: nat.paged_attn(q3, c3.k[0], c3.v[0], meta3, 0.09),
+             n_seq * (prior + new) * 8 * 128 * 4, pairs * 16 * 4 * 128)
+        del c, c2, c3
+        torch.cuda.empty_cache()
+    nat.check_status()
+    return out
+
+
+def report(names: List[str], kernels: bool = True) -> dict:
+    """Throughput of every named preset beside the dense decoder of its size, and the kernel cases of the first."""
+    res = {"what": "hybrid decoder beside the dense decoder of equal size", "dtype": "bf16", "data": "synthetic",
+           "device": torch.cuda.get_device_name(), "peaks": peaks(), "models": {}}
+    for n in names:
+        row = {}
+        for kind in ("hybrid", "dense"):
+            m = build(n, kind)
+            row[kind] = {"parameters": sum(p.numel() for p in m.parameters()), **throughput(m)}
+            del m
+            torch.cuda.empty_cache()
+        res["models"][n] = row
+    if kernels:
+        res["kernels"] = {names[0]: kernel_cases(names[0])}
+    return res
