@@ -363,8 +363,8 @@ template <bool SWIGLU>
 __global__ void __launch_bounds__(kTcThreads) gemv_tc_kernel(const GemvParams p) {
   extern __shared__ __align__(16) uint8_t gv_smem[];
   const int K = p.K, lds = K + kTcPad;
-  __nv_bfloat16* sx = reinterpret_cast<__nv_bfloat16*>(gv_smem);                      // [16][lds]
-  float* red = reinterpret_cast<float*>(gv_smem + static_cast<size_t>(16) * lds * 2);   // [warps][2][128]
+  __nv_bfloat16* sx = reinterpret_cast<__nv_bfloat16*>(gv_smem);                      // [8 or 16][lds]
+  float* red = reinterpret_cast<float*>(gv_smem + static_cast<size_t>(p.M > 8 ? 16 : 8) * lds * 2);   // [warps][2][128]
   __shared__ float s_rstd[16];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane & 3, col = lane >> 2;
@@ -538,14 +538,19 @@ static int launch_gemv_q4(const GemvParams& p, cudaStream_t st) {
   return static_cast<int>(launch_pdl(gemv_q4_tc_kernel<SWIGLU>, dim3(grid), dim3(kTcThreads), smem, st, p));
 }
 
+constexpr int kTcSmemMax = 224 * 1024;
+static size_t gv_tc_smem(int M, int K) {
+  return static_cast<size_t>(M > 8 ? 16 : 8) * (K + kTcPad) * 2 + kTcWarps * 2 * 128 * sizeof(float);
+}
+
 template <bool SWIGLU>
 static int launch_gemv_tc(const GemvParams& p, cudaStream_t st) {
-  const size_t smem = static_cast<size_t>(16) * (p.K + kTcPad) * 2 + kTcWarps * 2 * 128 * sizeof(float);
+  const size_t smem = gv_tc_smem(p.M, p.K);
   static DeviceMax configured;
   if (smem > 40 * 1024 && smem > configured.get()) {
-    cudaError_t e = cudaFuncSetAttribute(gemv_tc_kernel<SWIGLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(gemv_tc_kernel<SWIGLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmemMax);
     if (e != cudaSuccess) return static_cast<int>(e);
-    configured.set(200 * 1024);
+    configured.set(kTcSmemMax);
   }
   const int n_tiles = (p.N + 7) / 8;
   const int grid = n_tiles < num_sms() * 2 ? n_tiles : num_sms() * 2;      // each CTA stages x once and loops over its tiles
@@ -606,7 +611,7 @@ extern "C" int pm_gemv_ex(const void* x, int ldx, const void* w, int ldw, const 
     const char* e = getenv("PMETAL_GEMV_TC");
     use_tc = e ? atoi(e) : 1;
   }
-  if (use_tc && (K % 32) == 0 && static_cast<size_t>(16) * (K + kTcPad) * 2 + 8192 <= 200 * 1024)
+  if (use_tc && (K % 32) == 0 && gv_tc_smem(M, K) <= kTcSmemMax)
     return swiglu ? launch_gemv_tc<true>(p, st) : launch_gemv_tc<false>(p, st);
   // wide outputs: several columns per warp; narrow outputs: one column per warp (so that every SM gets work) with a
   // deeper load pipeline instead

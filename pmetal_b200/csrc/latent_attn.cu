@@ -9,7 +9,8 @@
 //   latent_prep_kernel      norm of the latent, rotation of k_r and of the queries' rotated part, cache append
 //   latent_absorb_kernel    [q_l | q_r | 0] rows of width W
 //   latent_attn_mma_kernel  bf16, split over key pages: 16 or 32 (token, head) rows share each 64-key page in shared
-//                           memory; S by mma.sync with the keys cut over the warps, P V with the columns cut over the warps
+//                           memory; S by mma.sync with keys and rows (or columns) cut over 16 warps, P V with the columns
+//                           cut over the warps
 //   latent_attn_row_kernel  any type and size, one (token, head) row per CTA (fp32 models)
 //   latent_up_kernel        joins the splits and applies W_uv
 // Longer portions expand keys and values of the visible rows with one GEMM and run the flash-attention kernels of
@@ -27,6 +28,26 @@
 namespace pm {
 
 constexpr int kPage = 64;
+
+// One element, or two neighbours at an even offset.
+template <int V>
+__device__ __forceinline__ void load_pair(const float* p, float (&v)[V]) {
+  if constexpr (V == 2) {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    v[0] = f.x; v[1] = f.y;
+  } else {
+    v[0] = p[0];
+  }
+}
+template <int V>
+__device__ __forceinline__ void load_pair(const __nv_bfloat16* p, float (&v)[V]) {
+  if constexpr (V == 2) {
+    const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+    v[0] = f.x; v[1] = f.y;
+  } else {
+    v[0] = to_f(p[0]);
+  }
+}
 
 // One CTA per token. qd [tokens, ld]: H heads of [D_n | D_r], then (own != 0) the down-projection [R | D_r].
 template <typename T>
@@ -62,49 +83,52 @@ __global__ void latent_prep_kernel(T* __restrict__ qd, long long ld, const float
   }
 }
 
-// grid (column tiles of 128, H, token groups of kAbsTok per sequence, sequences folded into z). The CTA computes 128
-// columns of q_l for up to kAbsTok tokens of one head; the last column tile copies the rotated part and zeroes the rest.
+// grid (column tiles of 128 plus one, H, groups of kAbsTok tokens), 128 / V threads. The CTA computes 128 columns of q_l for
+// kAbsTok tokens of one head (compact token i is row rows[i] of qd); the last column tile copies the rotated part and zeroes
+// the rest.
 constexpr int kAbsTok = 8;
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict__ qd, long long ld, const T* __restrict__ wuk,
-                                                            int H, int dn, int dr, int rank, int W,
-                                                            const int* __restrict__ q_start, const int* __restrict__ c_start,
-                                                            const int* __restrict__ q_lens, int tok_tiles,
-                                                            T* __restrict__ out) {
-  extern __shared__ float abs_q[];           // [kAbsTok][dn]
-  const int h = blockIdx.y, seq = blockIdx.z / tok_tiles, t0 = (blockIdx.z % tok_tiles) * kAbsTok;
-  const int len = q_lens[seq];
-  if (t0 >= len) return;
-  const int n_tok = min(kAbsTok, len - t0);
-  const long long q0 = q_start[seq] + t0, o0 = c_start[seq] + t0;
+                                                            int H, int dn, int dr, int rank, int W, const int* __restrict__ rows,
+                                                            int n, T* __restrict__ out) {
+  extern __shared__ __align__(16) float abs_q[];           // [kAbsTok][dn]
+  const int h = blockIdx.y, t0 = blockIdx.z * kAbsTok, n_tok = min(kAbsTok, n - t0);
   if (blockIdx.x == gridDim.x - 1) {
     const int tail = W - rank;
-    for (int i = threadIdx.x; i < n_tok * tail; i += 128) {
+    for (int i = threadIdx.x; i < n_tok * tail; i += blockDim.x) {
       const int t = i / tail, j = i - t * tail;
-      put(out + ((o0 + t) * H + h) * W + rank + j, j < dr ? to_f(qd[(q0 + t) * ld + h * (dn + dr) + dn + j]) : 0.f);
+      put(out + (static_cast<long long>(t0 + t) * H + h) * W + rank + j,
+          j < dr ? to_f(qd[rows[t0 + t] * ld + h * (dn + dr) + dn + j]) : 0.f);
     }
     return;
   }
-  for (int i = threadIdx.x; i < kAbsTok * dn; i += 128) {
-    const int t = i / dn, j = i - t * dn;
-    abs_q[i] = t < n_tok ? to_f(qd[(q0 + t) * ld + h * (dn + dr) + j]) : 0.f;
+  for (int t = 0; t < kAbsTok; ++t) {
+    const T* q = qd + (t < n_tok ? rows[t0 + t] : 0) * ld + h * (dn + dr);
+    for (int j = threadIdx.x; j < dn; j += blockDim.x) abs_q[t * dn + j] = t < n_tok ? to_f(q[j]) : 0.f;
   }
   __syncthreads();
-  const int c = blockIdx.x * 128 + threadIdx.x;
+  const int c = blockIdx.x * 128 + threadIdx.x * V;
   if (c >= rank) return;
-  float acc[kAbsTok];
+  float acc[kAbsTok][V];
 #pragma unroll
-  for (int t = 0; t < kAbsTok; ++t) acc[t] = 0.f;
+  for (int t = 0; t < kAbsTok; ++t)
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[t][e] = 0.f;
   const T* w = wuk + static_cast<long long>(h) * dn * rank + c;
-#pragma unroll 8
+#pragma unroll 16
   for (int j = 0; j < dn; ++j) {
-    const float wv = to_f(w[static_cast<long long>(j) * rank]);
+    float wv[V];
+    load_pair<V>(w + static_cast<long long>(j) * rank, wv);
 #pragma unroll
-    for (int t = 0; t < kAbsTok; ++t) acc[t] = fmaf(abs_q[t * dn + j], wv, acc[t]);
+    for (int t = 0; t < kAbsTok; ++t)
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[t][e] = fmaf(abs_q[t * dn + j], wv[e], acc[t][e]);
   }
 #pragma unroll
   for (int t = 0; t < kAbsTok; ++t)
-    if (t < n_tok) put(out + ((o0 + t) * H + h) * W + c, acc[t]);
+    if (t < n_tok)
+#pragma unroll
+      for (int e = 0; e < V; ++e) put(out + (static_cast<long long>(t0 + t) * H + h) * W + c + e, acc[t][e]);
 }
 
 struct LatentParams {
@@ -124,7 +148,7 @@ struct LatentParams {
 // One (token, head) row per CTA, all keys, any type. grid (rows of the longest portion, sequences).
 template <typename T>
 __global__ void __launch_bounds__(128) latent_attn_row_kernel(const LatentParams p) {
-  extern __shared__ float lr_smem[];
+  extern __shared__ __align__(16) float lr_smem[];
   float* sq = lr_smem;               // [W]
   float* so = sq + p.W;              // [rank]
   float* ss = so + p.rank;           // [64]
@@ -177,9 +201,10 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const LatentParams
   }
 }
 
-// 8 warps. MT: 16-row tiles of (token, head) rows; NT: 8-column tiles of the latent per warp.
+// 16 warps. MT: 16-row tiles of (token, head) rows; NT: 8-column tiles of the latent per warp.
+constexpr int kMmaThreads = 512;
 template <int MT, int NT>
-__global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams p) {
+__global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const LatentParams p) {
   extern __shared__ __align__(16) uint8_t lm_smem[];
   constexpr int RT = 16 * MT;
   constexpr int kLdS = kPage + 4, kLdP = kPage + 8;
@@ -187,8 +212,8 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
   __nv_bfloat16* sKV = reinterpret_cast<__nv_bfloat16*>(lm_smem);           // [2][64][ld]
   __nv_bfloat16* sQ = sKV + 2 * kPage * ld;                                  // [RT][ld]
   __nv_bfloat16* sP = sQ + RT * ld;                                          // [RT][kLdP]
-  float* sS = reinterpret_cast<float*>(sP + RT * kLdP);                      // [RT][kLdS]
-  float* sCorr = sS + RT * kLdS;                                             // [RT]
+  float* sS = reinterpret_cast<float*>(sP + RT * kLdP);                      // [32][kLdS]
+  float* sCorr = sS + 32 * kLdS;                                             // [RT]
   const int seq = blockIdx.x / p.row_tiles, row0 = (blockIdx.x % p.row_tiles) * RT, split = blockIdx.y;
   const int len = p.q_lens[seq], n_rows = len * p.H;
   if (row0 >= n_rows) return;
@@ -202,7 +227,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
   const long long base_row = static_cast<long long>(p.c_start[seq]) * p.H + row0;
   const long long part_base = split * p.rows + base_row;
   if (b0 >= b1) {
-    for (int i = threadIdx.x; i < RT && row0 + i < n_rows; i += 256) {
+    for (int i = threadIdx.x; i < RT && row0 + i < n_rows; i += kMmaThreads) {
       p.part_ml[(part_base + i) * 2] = -CUDART_INF_F;
       p.part_ml[(part_base + i) * 2 + 1] = 0.f;
     }
@@ -215,18 +240,22 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
     const __nv_bfloat16* src = cache + static_cast<long long>(bt[b]) * kPage * p.W;
     __nv_bfloat16* dst = sKV + buf * kPage * ld;
     const int valid = n_keys - b * kPage;
-    for (int i = threadIdx.x; i < kPage * chunks; i += 256) {
-      const int r = i / chunks, c = (i - r * chunks) * 8;
-      ms_cp16(ms_addr(dst + r * ld + c), src + static_cast<long long>(r) * p.W + c, r < valid);
+#pragma unroll
+    for (int i = 0; i < kPage / 16; ++i) {
+      const int r = warp + 16 * i;
+      for (int c = lane; c < chunks; c += 32)
+        ms_cp16(ms_addr(dst + r * ld + c * 8), src + static_cast<long long>(r) * p.W + c * 8, r < valid);
     }
     ms_commit();
   };
   {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + base_row * p.W;
-    for (int i = threadIdx.x; i < RT * chunks; i += 256) {
-      const int r = i / chunks, c = (i - r * chunks) * 8;
+#pragma unroll
+    for (int i = 0; i < MT; ++i) {
+      const int r = warp + 16 * i;
       const bool ok = row0 + r < n_rows;
-      ms_cp16(ms_addr(sQ + r * ld + c), q + static_cast<long long>(ok ? r : 0) * p.W + c, ok);
+      for (int c = lane; c < chunks; c += 32)
+        ms_cp16(ms_addr(sQ + r * ld + c * 8), q + static_cast<long long>(ok ? r : 0) * p.W + c * 8, ok);
     }
   }
   load_page(b0, 0);
@@ -237,13 +266,17 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
     for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
-  // softmax rows of this warp: RT / 8 consecutive rows
-  constexpr int kRows = RT / 8;
-  float m_run[kRows], l_run[kRows];
+  // softmax rows of this warp: MT consecutive rows
+  float m_run[MT], l_run[MT];
 #pragma unroll
-  for (int i = 0; i < kRows; ++i) { m_run[i] = -CUDART_INF_F; l_run[i] = 0.f; }
+  for (int i = 0; i < MT; ++i) { m_run[i] = -CUDART_INF_F; l_run[i] = 0.f; }
   const uint32_t aQ = ms_addr(sQ), aP = ms_addr(sP);
   const int n8 = (p.rank + 7) / 8;
+  // scores: warp w owns keys 8 (w % 8) .. + 7 of the page, and with w / 8 one of two row tiles (MT = 2) or one half of
+  // the columns, whose products the softmax adds (MT = 1)
+  const int kt = warp & 7, half = warp >> 3;
+  const int steps = p.W / 16, k0 = MT == 2 ? 0 : half * (steps / 2) * 16, k1 = MT == 2 || half == 1 ? p.W : (steps / 2) * 16;
+  const int q_row = MT == 2 ? half * 16 : 0;
 
   for (int b = b0; b < b1; ++b) {
     const int buf = (b - b0) & 1;
@@ -255,34 +288,42 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
     }
     __syncthreads();
     const uint32_t aK = ms_addr(sKV + buf * kPage * ld);
-    // scores: warp w owns keys 8 w .. 8 w + 7 of the page
-    float s[MT][4];
+    float s[2][4];
 #pragma unroll
-    for (int i = 0; i < MT; ++i)
+    for (int i = 0; i < 2; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[i][e] = 0.f;
-#pragma unroll 4
-    for (int k = 0; k < p.W; k += 16) {
-      uint32_t fb0, fb1;
-      ms_ldsm2(aK + static_cast<uint32_t>(((warp * 8 + (lane & 7)) * ld + k + ((lane >> 3) & 1) * 8) * 2), fb0, fb1);
-#pragma unroll
-      for (int i = 0; i < MT; ++i) {
-        uint32_t fa[4];
-        ms_ldsm4(ms_a_at(aQ, ld, i * 16, k, lane), fa);
-        ms_mma(s[i], fa, fb0, fb1);
-      }
+    const uint32_t k_at = aK + static_cast<uint32_t>(((kt * 8 + (lane & 7)) * ld + (lane >> 3) * 8) * 2);
+    int k = k0;
+#pragma unroll 2
+    for (; k + 32 <= k1; k += 32) {          // two steps with independent sums
+      uint32_t fb[4], fa0[4], fa1[4];
+      ms_ldsm4(k_at + k * 2, fb);
+      ms_ldsm4(ms_a_at(aQ, ld, q_row, k, lane), fa0);
+      ms_ldsm4(ms_a_at(aQ, ld, q_row, k + 16, lane), fa1);
+      ms_mma(s[0], fa0, fb[0], fb[1]);
+      ms_mma(s[1], fa1, fb[2], fb[3]);
+    }
+    if (k < k1) {
+      uint32_t fb0, fb1, fa[4];
+      ms_ldsm2(aK + static_cast<uint32_t>(((kt * 8 + (lane & 7)) * ld + k + ((lane >> 3) & 1) * 8) * 2), fb0, fb1);
+      ms_ldsm4(ms_a_at(aQ, ld, q_row, k, lane), fa);
+      ms_mma(s[0], fa, fb0, fb1);
     }
 #pragma unroll
-    for (int i = 0; i < MT; ++i)
-#pragma unroll
-      for (int hf = 0; hf < 2; ++hf)
-        *reinterpret_cast<float2*>(sS + (i * 16 + g4 + 8 * hf) * kLdS + warp * 8 + 2 * t4) =
-            make_float2(s[i][2 * hf], s[i][2 * hf + 1]);
+    for (int hf = 0; hf < 2; ++hf)           // MT = 1: the two halves lie in rows 0 .. 15 and 16 .. 31
+      *reinterpret_cast<float2*>(sS + (half * 16 + g4 + 8 * hf) * kLdS + kt * 8 + 2 * t4) =
+          make_float2(s[0][2 * hf] + s[1][2 * hf], s[0][2 * hf + 1] + s[1][2 * hf + 1]);
     __syncthreads();
 #pragma unroll
-    for (int i = 0; i < kRows; ++i) {
-      const int r = warp * kRows + i, lim = prior + (row0 + r) / p.H;        // last key this row sees
-      const float2 v = *reinterpret_cast<const float2*>(sS + r * kLdS + 2 * lane);
+    for (int i = 0; i < MT; ++i) {
+      const int r = warp * MT + i, lim = prior + (row0 + r) / p.H;           // last key this row sees
+      float2 v = *reinterpret_cast<const float2*>(sS + r * kLdS + 2 * lane);
+      if (MT == 1) {
+        const float2 w = *reinterpret_cast<const float2*>(sS + (16 + r) * kLdS + 2 * lane);
+        v.x += w.x;
+        v.y += w.y;
+      }
       const int j = b * kPage + 2 * lane;
       const float x0 = j <= lim ? v.x * p.scale_log2 : -CUDART_INF_F, x1 = j + 1 <= lim ? v.y * p.scale_log2 : -CUDART_INF_F;
       float mx = fmaxf(x0, x1);
@@ -290,7 +331,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
       for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       const float m_new = fmaxf(m_run[i], mx), m_use = m_new == -CUDART_INF_F ? 0.f : m_new;
       const float corr = exp2f(m_run[i] - m_use), e0 = exp2f(x0 - m_use), e1 = exp2f(x1 - m_use);
-      l_run[i] = l_run[i] * corr + warp_sum(e0 + e1);
+      l_run[i] = l_run[i] * corr + e0 + e1;  // this lane's keys; the lanes meet at the end
       m_run[i] = m_new;
       *reinterpret_cast<uint32_t*>(sP + r * kLdP + 2 * lane) = pack_bf16(e0, e1);
       if (lane == 0) sCorr[r] = corr;
@@ -312,7 +353,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
       for (int i = 0; i < MT; ++i) ms_ldsm4(ms_a_at(aP, kLdP, i * 16, kk, lane), fp[i]);
 #pragma unroll
       for (int j = 0; j < NT; ++j) {
-        const int tile = warp + 8 * j;
+        const int tile = warp + 16 * j;
         if (tile < n8) {
           uint32_t fb0, fb1;
           ms_ldsm2_t(aK + static_cast<uint32_t>(((kk + (lane & 15)) * ld + tile * 8) * 2), fb0, fb1);
@@ -324,11 +365,12 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
     __syncthreads();                  // the page buffer, scores and probabilities may be overwritten
   }
 #pragma unroll
-  for (int i = 0; i < kRows; ++i) {
-    const int r = warp * kRows + i;
+  for (int i = 0; i < MT; ++i) {
+    const int r = warp * MT + i;
+    const float l = warp_sum(l_run[i]);
     if (lane == 0 && row0 + r < n_rows) {
       p.part_ml[(part_base + r) * 2] = m_run[i];
-      p.part_ml[(part_base + r) * 2 + 1] = l_run[i];
+      p.part_ml[(part_base + r) * 2 + 1] = l;
     }
   }
 #pragma unroll
@@ -336,33 +378,36 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
 #pragma unroll
     for (int j = 0; j < NT; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = i * 16 + g4 + ((e & 2) ? 8 : 0), c = (warp + 8 * j) * 8 + 2 * t4 + (e & 1);
-        if (row0 + r < n_rows && c < p.rank) p.part_o[(part_base + r) * p.rank + c] = acc[i][j][e];
+      for (int hf = 0; hf < 2; ++hf) {
+        const int r = i * 16 + g4 + 8 * hf, c = (warp + 16 * j) * 8 + 2 * t4;
+        if (row0 + r >= n_rows || c >= p.rank) continue;
+        float* dst = p.part_o + (part_base + r) * p.rank + c;
+        if (p.rank % 2 == 0) {
+          *reinterpret_cast<float2*>(dst) = make_float2(acc[i][j][2 * hf], acc[i][j][2 * hf + 1]);
+        } else {
+          dst[0] = acc[i][j][2 * hf];
+          if (c + 1 < p.rank) dst[1] = acc[i][j][2 * hf + 1];
+        }
       }
 }
 
-// out[token, h, v] = W_uv[h, v, :] . (joined splits of row (token, h)). grid (H, token groups per sequence folded with
-// the sequences); a CTA joins up to kUpTok rows of one head and shares the weight rows between them.
+// out[rows[i], h, v] = W_uv[h, v, :] . (joined splits of row (i, h)). grid (H, groups of kUpTok tokens, chunks of value
+// channels); a CTA joins the rows of its tokens and shares the weight rows between them. V: elements per weight load.
 constexpr int kUpTok = 4;
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(256) latent_up_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                                        const T* __restrict__ wuv, const int* __restrict__ q_start,
-                                                        const int* __restrict__ c_start, const int* __restrict__ q_lens,
-                                                        int tok_tiles, int H, int dv, int rank, int n_split, long long rows,
-                                                        T* __restrict__ out, long long ldo) {
-  extern __shared__ float up_o[];            // [kUpTok][rank]
+                                                        const T* __restrict__ wuv, const int* __restrict__ rows, int n, int H,
+                                                        int dv, int rank, int n_split, T* __restrict__ out, long long ldo) {
+  extern __shared__ __align__(16) float up_o[];            // [kUpTok][rank]
   __shared__ float coef[kUpTok][64];
-  const int h = blockIdx.x, seq = blockIdx.y / tok_tiles, t0 = (blockIdx.y % tok_tiles) * kUpTok;
-  const int len = q_lens[seq];
-  if (t0 >= len) return;
-  const int n_tok = min(kUpTok, len - t0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long q0 = q_start[seq] + t0, c0 = c_start[seq] + t0;
+  const int h = blockIdx.x, t0 = blockIdx.y * kUpTok, n_tok = min(kUpTok, n - t0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long part_rows = static_cast<long long>(n) * H;
   if (warp < n_tok) {                        // n_split <= 64: two splits per lane
-    const long long row = (c0 + warp) * H + h;
+    const float* ml = part_ml + (static_cast<long long>(t0 + warp) * H + h) * 2;
     float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
-    if (lane < n_split) { m0 = part_ml[(lane * rows + row) * 2]; l0 = part_ml[(lane * rows + row) * 2 + 1]; }
-    if (lane + 32 < n_split) { m1 = part_ml[((lane + 32) * rows + row) * 2]; l1 = part_ml[((lane + 32) * rows + row) * 2 + 1]; }
+    if (lane < n_split) { m0 = ml[lane * part_rows * 2]; l0 = ml[lane * part_rows * 2 + 1]; }
+    if (lane + 32 < n_split) { m1 = ml[(lane + 32) * part_rows * 2]; l1 = ml[(lane + 32) * part_rows * 2 + 1]; }
     float mx = fmaxf(m0, m1);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -372,29 +417,45 @@ __global__ void __launch_bounds__(256) latent_up_kernel(const float* __restrict_
     coef[warp][lane + 32] = e1 * inv;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < kUpTok * rank; i += 256) {
+  constexpr int JV = V >= 4 ? 4 : 1;
+  for (int i = threadIdx.x * JV; i < kUpTok * rank; i += 256 * JV) {
     const int t = i / rank, c = i - t * rank;
-    float v = 0.f;
+    float v[JV];
+#pragma unroll
+    for (int e = 0; e < JV; ++e) v[e] = 0.f;
     if (t < n_tok) {
-      const long long row = (c0 + t) * H + h;
-      for (int s = 0; s < n_split; ++s) {
+      const float* src = part_o + (static_cast<long long>(t0 + t) * H + h) * rank + c;
+#pragma unroll 4
+      for (int s = 0; s < n_split; ++s) {    // an empty split left its rows unwritten
         const float w = coef[t][s];
-        if (w != 0.f) v = fmaf(w, part_o[(s * rows + row) * rank + c], v);
+        float x[JV];
+#pragma unroll
+        for (int e = 0; e < JV; ++e) x[e] = 0.f;
+        if (w != 0.f) load_vec<JV>(src + s * part_rows * rank, x);
+#pragma unroll
+        for (int e = 0; e < JV; ++e) v[e] = fmaf(w, x[e], v[e]);
       }
     }
-    up_o[i] = v;
+    store_vec<JV>(up_o + i, v);
   }
   __syncthreads();
-  for (int r = warp; r < dv; r += 8) {
+  const int per = (dv + gridDim.z - 1) / gridDim.z, r1 = min(dv, (static_cast<int>(blockIdx.z) + 1) * per);
+  for (int r = blockIdx.z * per + warp; r < r1; r += 8) {
     const T* w = wuv + (static_cast<long long>(h) * dv + r) * rank;
     float acc[kUpTok];
 #pragma unroll
     for (int t = 0; t < kUpTok; ++t) acc[t] = 0.f;
-#pragma unroll 4
-    for (int c = lane; c < rank; c += 32) {
-      const float wv = to_f(w[c]);
+#pragma unroll 2
+    for (int c = lane * V; c < rank; c += 32 * V) {
+      float wv[V];
+      load_vec<V>(w + c, wv);
 #pragma unroll
-      for (int t = 0; t < kUpTok; ++t) acc[t] = fmaf(wv, up_o[t * rank + c], acc[t]);
+      for (int t = 0; t < kUpTok; ++t) {
+        float x[V];
+        load_vec<V>(up_o + t * rank + c, x);
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[t] = fmaf(wv[e], x[e], acc[t]);
+      }
     }
 #pragma unroll
     for (int t = 0; t < kUpTok; ++t) acc[t] = warp_sum(acc[t]);
@@ -403,7 +464,7 @@ __global__ void __launch_bounds__(256) latent_up_kernel(const float* __restrict_
 #pragma unroll
       for (int t = 1; t < kUpTok; ++t)
         if (lane == t) v = acc[t];
-      put(out + (q0 + lane) * ldo + h * dv + r, v);
+      put(out + rows[t0 + lane] * ldo + h * dv + r, v);
     }
   }
 }
@@ -432,20 +493,22 @@ __global__ void latent_gather8_kernel(const __nv_bfloat16* __restrict__ cache, c
 
 // Query / key / value operands of the 128-channel attention kernels, zero padded. kv [n, ldkv]: H heads of D_n key
 // channels, then H heads of D_v value channels. blockIdx.y: 0 = queries (n_q rows of qd), 1 = keys, 2 = values.
-// A thread writes 8 channels.
+// A thread writes 8 channels. Operands without a destination are left out.
 __global__ void latent_assemble_kernel(const __nv_bfloat16* __restrict__ qd, long long ldq, int n_q,
                                        const __nv_bfloat16* __restrict__ kv, long long ldkv, int n,
                                        const __nv_bfloat16* __restrict__ cache, const int* __restrict__ table, int W, int rank,
                                        int H, int dn, int dr, int dv, __nv_bfloat16* __restrict__ q128,
                                        __nv_bfloat16* __restrict__ k128, __nv_bfloat16* __restrict__ v128) {
   const int what = blockIdx.y;
+  __nv_bfloat16* to = what == 0 ? q128 : (what == 1 ? k128 : v128);
+  if (!to) return;
   const long long rows = static_cast<long long>(what == 0 ? n_q : n) * H;
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < rows * 16;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
     const long long r = i >> 4;
     const int c0 = static_cast<int>(i & 15) * 8, h = static_cast<int>(r % H);
     const long long t = r / H;
-    __nv_bfloat16* dst = (what == 0 ? q128 : (what == 1 ? k128 : v128)) + r * 128 + c0;
+    __nv_bfloat16* dst = to + r * 128 + c0;
     const __nv_bfloat16 *a, *b = nullptr;      // channels [0, na) from a, [na, nb) from b
     int na, nb;
     if (what == 0) {
@@ -495,7 +558,7 @@ __global__ void latent_take_kernel(const __nv_bfloat16* __restrict__ o128, int n
 
 static size_t latent_mma_smem(int mt, int W) {
   const size_t rt = 16 * mt, ld = W + 8;
-  return (2 * kPage * ld + rt * ld + rt * (kPage + 8)) * 2 + (rt * (kPage + 4) + rt) * 4;
+  return (2 * kPage * ld + rt * ld + rt * (kPage + 8)) * 2 + (32 * (kPage + 4) + rt) * 4;
 }
 static int latent_mma_tiles(int H, int W) {      // 16-row tiles per CTA, 0: not covered
   if (H > 16 && latent_mma_smem(2, W) <= 220 * 1024) return 2;
@@ -511,7 +574,29 @@ static int latent_mma_launch(const LatentParams& p, dim3 grid, size_t smem, cuda
     if (e != cudaSuccess) return static_cast<int>(e);
     configured.set(smem);
   }
-  latent_attn_mma_kernel<MT, NT><<<grid, 256, smem, st>>>(p);
+  latent_attn_mma_kernel<MT, NT><<<grid, kMmaThreads, smem, st>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+static int latent_absorb_launch(const void* qd, long long ld, const void* wuk, int H, int dn, int dr, int rank, int W,
+                                const int* rows, int n, int tiles, size_t smem, void* out, cudaStream_t st) {
+  const dim3 grid((rank + 127) / 128 + 1, H, tiles);
+  const T *q = static_cast<const T*>(qd), *w = static_cast<const T*>(wuk);
+  if (rank % 2 == 0) latent_absorb_kernel<T, 2><<<grid, 64, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out));
+  else latent_absorb_kernel<T, 1><<<grid, 128, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out));
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+static int latent_up_launch(const float* part_o, const float* part_ml, const void* wuv, const int* rows, int n, int H, int dv,
+                            int rank, int n_split, dim3 grid, size_t smem, void* out, long long ldo, cudaStream_t st) {
+  const T* w = static_cast<const T*>(wuv);
+  T* o = static_cast<T*>(out);
+  // whole 16-byte pieces need aligned weight rows (the value weights may lie behind the keys' in one allocation)
+  const int v = rank % 8 == 0 && !(reinterpret_cast<uintptr_t>(w) & 15) ? 8 : 1;
+  if (v == 8) latent_up_kernel<T, 8><<<grid, 256, smem, st>>>(part_o, part_ml, w, rows, n, H, dv, rank, n_split, o, ldo);
+  else latent_up_kernel<T, 1><<<grid, 256, smem, st>>>(part_o, part_ml, w, rows, n, H, dv, rank, n_split, o, ldo);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -543,70 +628,59 @@ extern "C" int pm_latent_mma_supported(int H, int W, int rank) {
 }
 
 // Attention of short portions in the latent space. qd as pm_latent_prep leaves it, wuk [H * dn, rank], wuv [H * dv, rank],
-// cache [pages, 64, W]. Sequence i covers rows q_start[i] .. of qd and out and rows c_start[i] .. of the work buffers
-// q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32, part_ml [n_split, n_tok * H, 2] fp32 (n_tok: tokens of the
-// listed sequences). out [.., ldo]: H * dv columns. max_q: longest of q_lens.
-// n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
+// cache [pages, 64, W]. The n_tok tokens of the listed sequences are counted through: sequence i covers compact tokens
+// c_start[i] .. of the work buffers q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32 and part_ml [n_split,
+// n_tok * H, 2] fp32, and compact token j is row tok_rows[j] of qd and out. out [.., ldo]: H * dv columns. max_q: longest of
+// q_lens. n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
 extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void* wuk, const void* wuv, const void* cache,
-                              const int* block_table, const int* seq_lens, const int* q_start, const int* c_start,
-                              const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr, int dv, int rank, int W,
-                              int n_split, float scale, void* q_lat, float* part_o, float* part_ml, void* out,
-                              long long ldo, cudaStream_t st) {
+                              const int* block_table, const int* seq_lens, const int* c_start, const int* q_lens,
+                              const int* tok_rows, int n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr,
+                              int dv, int rank, int W, int n_split, float scale, void* q_lat, float* part_o, float* part_ml,
+                              void* out, long long ldo, cudaStream_t st) {
   if (H < 1 || rank < 1 || W < rank + dr || dv < 1 || n_split < 1 || n_split > 64 || ldo < static_cast<long long>(H) * dv)
     return -1;
-  if (n_seq < 1 || max_q < 1) return 0;
+  if (n_seq < 1 || max_q < 1 || n_tok < 1) return 0;
   const bool mma = !f32 && pm_latent_mma_supported(H, W, rank);
   if (!mma && n_split != 1) return -2;
   const size_t sm_abs = static_cast<size_t>(kAbsTok) * dn * 4, sm_row = (static_cast<size_t>(W) + rank + kPage) * 4,
                sm_up = static_cast<size_t>(kUpTok) * rank * 4;
   if (sm_abs > 48 * 1024 || (!mma && sm_row > 48 * 1024) || sm_up > 46 * 1024) return -3;
-  const int abs_tiles = (max_q + kAbsTok - 1) / kAbsTok, up_tiles = (max_q + kUpTok - 1) / kUpTok;
-  if (static_cast<long long>(abs_tiles) * n_seq > 65535 || static_cast<long long>(up_tiles) * n_seq > 65535) return -4;
-  const dim3 g_abs((rank + 127) / 128 + 1, H, abs_tiles * n_seq);
-  if (f32)
-    latent_absorb_kernel<float><<<g_abs, 128, sm_abs, st>>>(static_cast<const float*>(qd), ld, static_cast<const float*>(wuk),
-                                                            H, dn, dr, rank, W, q_start, c_start, q_lens, abs_tiles,
-                                                            static_cast<float*>(q_lat));
-  else
-    latent_absorb_kernel<__nv_bfloat16><<<g_abs, 128, sm_abs, st>>>(
-        static_cast<const __nv_bfloat16*>(qd), ld, static_cast<const __nv_bfloat16*>(wuk), H, dn, dr, rank, W, q_start,
-        c_start, q_lens, abs_tiles, static_cast<__nv_bfloat16*>(q_lat));
-  cudaError_t e = cudaGetLastError();
-  if (e != cudaSuccess) return static_cast<int>(e);
+  const int abs_tiles = (n_tok + kAbsTok - 1) / kAbsTok, up_tiles = (n_tok + kUpTok - 1) / kUpTok;
+  if (abs_tiles > 65535 || up_tiles > 65535) return -4;
+  int rc = f32 ? latent_absorb_launch<float>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, st)
+               : latent_absorb_launch<__nv_bfloat16>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, st);
+  if (rc) return rc;
   LatentParams p{};
   p.q = q_lat; p.cache = cache; p.block_table = block_table; p.seq_lens = seq_lens; p.c_start = c_start; p.q_lens = q_lens;
   p.part_o = part_o; p.part_ml = part_ml; p.max_blocks = max_blocks; p.H = H; p.W = W; p.rank = rank; p.n_split = n_split;
   p.rows = static_cast<long long>(n_tok) * H;
   p.scale_log2 = scale * 1.4426950408889634f;
   if (mma) {
-    const int mt = latent_mma_tiles(H, W), rt = 16 * mt, n8 = (rank + 7) / 8, nt = (n8 + 7) / 8;
+    const int mt = latent_mma_tiles(H, W), rt = 16 * mt, nt = (rank + 127) / 128;
     p.row_tiles = (max_q * H + rt - 1) / rt;
     const dim3 grid(p.row_tiles * n_seq, n_split);
     const size_t smem = latent_mma_smem(mt, W);
-    int rc;
     if (mt == 1)
       rc = nt <= 1 ? latent_mma_launch<1, 1>(p, grid, smem, st) : nt <= 2 ? latent_mma_launch<1, 2>(p, grid, smem, st)
-         : nt <= 4 ? latent_mma_launch<1, 4>(p, grid, smem, st) : latent_mma_launch<1, 8>(p, grid, smem, st);
+                                                                          : latent_mma_launch<1, 4>(p, grid, smem, st);
     else
       rc = nt <= 1 ? latent_mma_launch<2, 1>(p, grid, smem, st) : nt <= 2 ? latent_mma_launch<2, 2>(p, grid, smem, st)
-         : nt <= 4 ? latent_mma_launch<2, 4>(p, grid, smem, st) : latent_mma_launch<2, 8>(p, grid, smem, st);
+                                                                          : latent_mma_launch<2, 4>(p, grid, smem, st);
     if (rc) return rc;
   } else {
     const dim3 grid(max_q * H, n_seq);
     if (f32) latent_attn_row_kernel<float><<<grid, 128, sm_row, st>>>(p);
     else latent_attn_row_kernel<__nv_bfloat16><<<grid, 128, sm_row, st>>>(p);
-    e = cudaGetLastError();
+    const cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  const dim3 g_up(H, up_tiles * n_seq);
-  if (f32)
-    latent_up_kernel<float><<<g_up, 256, sm_up, st>>>(part_o, part_ml, static_cast<const float*>(wuv), q_start, c_start,
-                                                      q_lens, up_tiles, H, dv, rank, n_split, p.rows, static_cast<float*>(out), ldo);
-  else
-    latent_up_kernel<__nv_bfloat16><<<g_up, 256, sm_up, st>>>(part_o, part_ml, static_cast<const __nv_bfloat16*>(wuv), q_start,
-                                                              c_start, q_lens, up_tiles, H, dv, rank, n_split, p.rows,
-                                                              static_cast<__nv_bfloat16*>(out), ldo);
-  return static_cast<int>(cudaGetLastError());
+  // few heads and tokens: the value channels are cut so that the launch still fills the machine
+  int cut = (2 * num_sms() + H * up_tiles - 1) / (H * up_tiles);
+  const int most = (dv + 7) / 8;
+  if (cut > most) cut = most;
+  const dim3 g_up(H, up_tiles, cut);
+  return f32 ? latent_up_launch<float>(part_o, part_ml, wuv, tok_rows, n_tok, H, dv, rank, n_split, g_up, sm_up, out, ldo, st)
+             : latent_up_launch<__nv_bfloat16>(part_o, part_ml, wuv, tok_rows, n_tok, H, dv, rank, n_split, g_up, sm_up, out, ldo, st);
 }
 
 // lat [n, r8] bf16 = latents of positions 0 .. n - 1 of the sequence whose block table row is `table` (zero padded).

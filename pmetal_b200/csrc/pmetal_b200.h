@@ -210,12 +210,12 @@ int pm_latent_prep(void* qd, int f32, long long ld, const float* norm_w, float e
 // Whether the tensor-core kernel covers H heads over rows of W columns with `rank` value columns.
 int pm_latent_mma_supported(int H, int W, int rank);
 // Attention of short portions in the latent space. qd as pm_latent_prep leaves it, wuk [H * dn, rank], wuv [H * dv, rank],
-// cache [pages, 64, W]. Sequence i covers rows q_start[i] .. of qd and out and rows c_start[i] .. of the work buffers
-// q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32, part_ml [n_split, n_tok * H, 2] fp32 (n_tok: tokens of the
-// listed sequences). out [.., ldo]: H * dv columns. max_q: longest of q_lens.
-// n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
+// cache [pages, 64, W]. The n_tok tokens of the listed sequences are counted through: sequence i covers compact tokens
+// c_start[i] .. of the work buffers q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32 and part_ml [n_split,
+// n_tok * H, 2] fp32, and compact token j is row tok_rows[j] of qd and out. out [.., ldo]: H * dv columns. max_q: longest of
+// q_lens. n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
 int pm_latent_attn(const void* qd, int f32, long long ld, const void* wuk, const void* wuv, const void* cache,
-    const int* block_table, const int* seq_lens, const int* q_start, const int* c_start, const int* q_lens, int
+    const int* block_table, const int* seq_lens, const int* c_start, const int* q_lens, const int* tok_rows, int
     n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr, int dv, int rank, int W, int n_split, float
     scale, void* q_lat, float* part_o, float* part_ml, void* out, long long ldo, cudaStream_t st);
 // lat [n, r8] bf16 = latents of positions 0 .. n - 1 of the sequence whose block table row is `table` (zero padded).
@@ -320,12 +320,13 @@ int pm_ssm_scan(const void* u, int f32, long long ldu, const float* conv_w, cons
     cudaStream_t st);
 // Whether pm_ssm_chunk covers a state of N rows.
 int pm_ssm_chunk_supported(int N);
-// The same for longer portions of bf16 models: act [tokens, conv] bf16 and dt [tokens, H] fp32 are work buffers that the
-// first kernel fills, max_q is the longest of q_lens.
+// The same for longer portions of bf16 models: act [tokens, conv] bf16, dt [tokens, H], seg_state [n_seq][max_seg][H][N][P4]
+// and seg_decay [n_seq][max_seg][H] fp32 are work buffers, max_q is the longest of q_lens. A portion is cut into at most
+// max_seg segments that run in parallel (fewer when sequences and heads fill the machine by themselves).
 int pm_ssm_chunk(const void* u, long long ldu, const float* conv_w, const float* conv_b, const float* dt_bias,
     const float* a_log, const float* dskip, const void* ring, float* state, const int* slots, const int* q_start,
     const int* q_lens, const int* seq_lens, int n_seq, int max_q, int H, int P, int N, int G, int taps, void* act,
-    float* dt, void* y, cudaStream_t st);
+    float* dt, float* seg_state, float* seg_decay, int max_seg, void* y, cudaStream_t st);
 // out [tokens, H P] = RMS norm over `parts` equal parts of y * silu(z) (z: the first H P columns of u), times w; the last
 // taps - 1 convolution inputs of every sequence go to the ring. seq_of / pos [tokens]: sequence index and position.
 int pm_ssm_gate_norm(const void* y, const void* u, int f32, long long ldu, const float* w, float eps, int parts,

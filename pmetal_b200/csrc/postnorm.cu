@@ -34,7 +34,7 @@ __global__ void post_layernorm_kernel(const float* x, const T* __restrict__ y, l
                                       const float* __restrict__ bias, float alpha, const float* __restrict__ w,
                                       const float* __restrict__ b, float eps, int width, const long long* __restrict__ rows,
                                       float* of, T* __restrict__ oc) {
-  extern __shared__ float row_buf[];
+  extern __shared__ __align__(16) float row_buf[];
   const long long o = blockIdx.x, r = rows ? rows[o] : o;
   float sum = 0.f;
   for (int k = threadIdx.x * V; k < width; k += blockDim.x * V) {

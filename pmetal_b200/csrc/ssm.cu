@@ -12,7 +12,9 @@
 //   ssm_scan_kernel   any number of tokens, one after the other, convolution included; one CTA per (sequence, head,
 //                     slice of P), the state in registers. Decode, short portions, fp32 models.
 //   ssm_conv_kernel   convolution + silu and softplus of the step sizes for all tokens of longer portions.
-//   ssd_chunk_kernel  the recurrence of longer portions in blocks of 64 tokens on the tensor cores:
+//   ssd_segment_kernel / ssd_chunk_kernel  the recurrence of longer portions in blocks of 64 tokens on the tensor cores,
+//                     segments of several blocks in parallel (the first kernel sums what each segment adds to the state,
+//                     the second starts every segment from the decayed sum of the earlier ones):
 //                     y_i = sum_{j <= i} (C_i.B_j) exp(a_i - a_j) dt_j x_j + exp(a_i) S^T C_i + D x_i (a: running sum of
 //                     the log decays), S <- exp(a_63) S + sum_j exp(a_63 - a_j) dt_j B_j x_j^T. x, B and C are bf16
 //                     activations; every fp32 factor (decayed scores, state, decayed B) enters the products as the sum
@@ -69,7 +71,7 @@ constexpr int kScanThreads = 256;
 // E: state rows per thread (float4 each).
 template <typename T, int E>
 __global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const ScanParams<T> p) {
-  extern __shared__ float scan_smem[];
+  extern __shared__ __align__(16) float scan_smem[];
   const SsmDims& d = p.d;
   const int seq = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * p.pw;
   const int len = p.q_lens[seq];
@@ -108,12 +110,19 @@ __global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const ScanParams
       float v = 0.f;
       if (c >= 0) {
         v = p.conv_b[c];
-        for (int j = 0; j < d.taps; ++j) {
-          const int back = d.taps - 1 - j, src = pos - back;
-          if (src < 0) continue;
-          const float in = t >= back ? to_f(row[d.inner + c - static_cast<long long>(back) * p.ldu])
-                                     : to_f(p.ring[(slot * d.taps + src % d.taps) * d.conv + c]);
-          v = fmaf(p.conv_w[static_cast<long long>(j) * d.conv + c], in, v);
+        for (int j0 = 0; j0 < d.taps; j0 += 4) {           // four independent loads at a time
+          float w[4], in[4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int j = j0 + k, back = d.taps - 1 - j, src = pos - back;
+            const bool ok = j < d.taps && src >= 0;
+            const T* at = t >= back ? row + d.inner + c - static_cast<long long>(back) * p.ldu
+                                    : p.ring + (slot * d.taps + (ok ? src % d.taps : 0)) * d.conv + c;
+            w[k] = ok ? p.conv_w[static_cast<long long>(j) * d.conv + c] : 0.f;
+            in[k] = ok ? to_f(*at) : 0.f;
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k) v = fmaf(w[k], in[k], v);
         }
         v = silu_f(v);
       }
@@ -174,8 +183,8 @@ struct ConvParams {
 };
 
 // grid (tiles of 8 tokens, sequences, channel tiles + 1): a thread owns V channels of 8 consecutive tokens; the last
-// channel tile computes the step sizes.
-template <int V>
+// channel tile computes the step sizes. TAPS = 0: any number of taps.
+template <int V, int TAPS>
 __global__ void __launch_bounds__(128) ssm_conv_kernel(const ConvParams p) {
   const SsmDims& d = p.d;
   const int seq = blockIdx.y, len = p.q_lens[seq], t0 = blockIdx.x * kConvTokens;
@@ -198,19 +207,46 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const ConvParams p) {
   for (int t = 0; t < kConvTokens; ++t)
 #pragma unroll
     for (int e = 0; e < V; ++e) acc[t][e] = b[e];
-  for (int j = 0; j < d.taps; ++j) {
-    const int back = d.taps - 1 - j;
-    float w[V];
-    load_vec<V>(p.conv_w + static_cast<long long>(j) * d.conv + c, w);
+  auto input = [&](int t, float (&in)[V]) {               // input of token t0 + t (t may be negative), zeros before the start
+    const int src = start + t0 + t;
+    if (src < 0) {
 #pragma unroll
-    for (int t = 0; t < kConvTokens; ++t) {
-      const int src = start + t0 + t - back;
-      if (t >= n_tok || src < 0) continue;
+      for (int e = 0; e < V; ++e) in[e] = 0.f;
+    } else if (t0 + t >= 0) {
+      load_vec<V>(p.u + static_cast<long long>(q0 + t0 + t) * p.ldu + d.inner + c, in);
+    } else {
+      load_vec<V>(p.ring + (slot * d.taps + src % d.taps) * d.conv + c, in);
+    }
+  };
+  if (TAPS > 0) {
+    float w[TAPS > 0 ? TAPS : 1][V];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load_vec<V>(p.conv_w + static_cast<long long>(j) * d.conv + c, w[j]);
+#pragma unroll
+    for (int r = 1 - TAPS; r < kConvTokens; ++r) {
+      if (r >= n_tok) break;
       float in[V];
-      if (t0 + t >= back) load_vec<V>(p.u + static_cast<long long>(q0 + t0 + t - back) * p.ldu + d.inner + c, in);
-      else load_vec<V>(p.ring + (slot * d.taps + src % d.taps) * d.conv + c, in);
+      input(r, in);
 #pragma unroll
-      for (int e = 0; e < V; ++e) acc[t][e] = fmaf(w[e], in[e], acc[t][e]);
+      for (int j = 0; j < TAPS; ++j) {
+        const int t = r + TAPS - 1 - j;                    // row r is tap j of token t
+        if (t >= 0 && t < kConvTokens)
+#pragma unroll
+          for (int e = 0; e < V; ++e) acc[t][e] = fmaf(w[j][e], in[e], acc[t][e]);
+      }
+    }
+  } else {
+    for (int j = 0; j < d.taps; ++j) {
+      float w[V];
+      load_vec<V>(p.conv_w + static_cast<long long>(j) * d.conv + c, w);
+#pragma unroll
+      for (int t = 0; t < kConvTokens; ++t) {
+        if (t >= n_tok) break;
+        float in[V];
+        input(t - (d.taps - 1 - j), in);
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[t][e] = fmaf(w[e], in[e], acc[t][e]);
+      }
     }
   }
 #pragma unroll
@@ -233,6 +269,11 @@ struct ChunkParams {
   const int* q_lens;
   const int* seq_lens;
   __nv_bfloat16* y;           // [tokens, inner]
+  // segments: seg_state [seq][n_seg][H][N][P4] (0: the state a sequence starts from, k > 0: what segment k - 1 adds to it),
+  // seg_decay [seq][n_seg][H] (decay of the state over segment k)
+  float* seg_state;
+  float* seg_decay;
+  int n_seg, seg_chunks;      // segments of the longest portion, blocks per segment
   SsmDims d;
   int n16;                    // N rounded up to 16
   int aligned;                // rows can be copied 16 bytes at a time
@@ -241,75 +282,237 @@ struct ChunkParams {
 constexpr int kChunk = 64;
 constexpr int kSlice = 32;            // channels of P per CTA
 constexpr int kLdX = kSlice + 8;
+constexpr float kLog2e = 1.4426950408889634f;
 
-// NI: state row tiles (16 rows) per warp; 4 warps cover N <= 64 NI.
-template <int NI>
-__global__ void __launch_bounds__(128) ssd_chunk_kernel(const ChunkParams p) {
-  extern __shared__ __align__(16) uint8_t ssd_smem[];
-  const SsmDims& d = p.d;
-  const int seq = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * kSlice;
-  const int len = p.q_lens[seq];
-  if (len <= 0) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, t4 = lane & 3;
-  const int ldn = p.n16 + 8;
-  const int tile_n = kChunk * ldn, tile_x = kChunk * kLdX;
-  __nv_bfloat16* sC = reinterpret_cast<__nv_bfloat16*>(ssd_smem);       // [2][64][ldn]
-  __nv_bfloat16* sB = sC + 2 * tile_n;                                   // [2][64][ldn]
-  __nv_bfloat16* sX = sB + 2 * tile_n;                                   // [2][64][kLdX]
-  __nv_bfloat16* sSh = sX + 2 * tile_x;                                  // [n16][kLdX]
-  __nv_bfloat16* sSl = sSh + p.n16 * kLdX;                               // [n16][kLdX]
-  float* sDt = reinterpret_cast<float*>(sSl + p.n16 * kLdX);             // [2][64]
-  float* sCum = sDt + 2 * kChunk;                                        // [4 warps][64]
-  float* sW = sCum + 4 * kChunk;                                         // [4 warps][64]
-
-  const long long q0 = p.q_start[seq];
-  const int start = p.seq_lens[seq] - len;
-  const long long slot = p.slots[seq];
-  const int g = h / (d.H / d.G);
-  const int cx = h * d.P + p0, cb = d.inner + g * d.N, cc = d.inner + (d.G + g) * d.N;
-  const int pw = min(kSlice, d.P - p0);
-  const float a = -expf(p.a_log[h]), skip = p.dskip[h];
-  const int n_chunks = (len + kChunk - 1) / kChunk;
-
-  auto load_rows = [&](__nv_bfloat16* dst, int ld, int width, int valid_w, int c0, int t0) {
-    if (p.aligned) {
-      const int per = width / 8;
-      for (int i = threadIdx.x; i < kChunk * per; i += 128) {
-        const int r = i / per, c = (i - r * per) * 8;
-        const bool ok = t0 + r < len && c < valid_w;
-        const __nv_bfloat16* src = p.act + (q0 + (ok ? t0 + r : 0)) * d.conv + c0 + (ok ? c : 0);
-        ms_cp16(ms_addr(dst + r * ld + c), src, ok);
+// Rows t0 .. t0 + 63 of `act`, `width` columns from c0 (multiple of 8, zero filled beyond valid_w and beyond the portion).
+__device__ __forceinline__ void ssd_load_rows(const ChunkParams& p, __nv_bfloat16* dst, int ld, int width, int valid_w, int c0,
+                                              long long q0, int t0, int len) {
+  if (p.aligned) {
+    const int per = width / 8, dr = 128 / per, dc = 128 - dr * per;
+    int r = threadIdx.x / per, c = threadIdx.x - r * per;
+    for (; r < kChunk; r += dr, c += dc) {
+      if (c >= per) {
+        c -= per;
+        if (++r >= kChunk) break;
       }
-    } else {
-      for (int i = threadIdx.x; i < kChunk * width; i += 128) {
-        const int r = i / width, c = i - r * width;
-        const bool ok = t0 + r < len && c < valid_w;
-        dst[r * ld + c] = ok ? p.act[(q0 + t0 + r) * d.conv + c0 + c] : __float2bfloat16(0.f);
-      }
+      const bool ok = t0 + r < len && c * 8 < valid_w;
+      const __nv_bfloat16* src = p.act + (q0 + (ok ? t0 + r : 0)) * p.d.conv + c0 + (ok ? c * 8 : 0);
+      ms_cp16(ms_addr(dst + r * ld + c * 8), src, ok);
     }
-  };
-  auto load_chunk = [&](int ch, int buf) {
-    const int t0 = ch * kChunk;
-    load_rows(sC + buf * tile_n, ldn, p.n16, d.N, cc, t0);
-    load_rows(sB + buf * tile_n, ldn, p.n16, d.N, cb, t0);
-    load_rows(sX + buf * tile_x, kLdX, kSlice, pw, cx, t0);
-    if (threadIdx.x < kChunk)
-      sDt[buf * kChunk + threadIdx.x] = t0 + static_cast<int>(threadIdx.x) < len ? p.dt[(q0 + t0 + threadIdx.x) * d.H + h] : 0.f;
-    ms_commit();
-  };
+  } else {
+    for (int i = threadIdx.x; i < kChunk * width; i += 128) {
+      const int r = i / width, c = i - r * width;
+      const bool ok = t0 + r < len && c < valid_w;
+      dst[r * ld + c] = ok ? p.act[(q0 + t0 + r) * p.d.conv + c0 + c] : __float2bfloat16(0.f);
+    }
+  }
+}
 
-  // this warp's rows of the state, accumulator layout
-  float S[NI][4][4];
-  float* st = p.state + ((slot * d.H + h) * d.N) * static_cast<long long>(d.P4) + p0;
+// One warp's copy of the block's running log2 decays and of the weights with which its tokens enter the state; returns the
+// log2 decay over the block.
+__device__ __forceinline__ float ssd_decays(const float* dts, float a2, float* cum, float* wgt, int lane) {
+  const float d0 = dts[2 * lane], d1 = dts[2 * lane + 1];
+  float run = a2 * d0 + a2 * d1;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float up = __shfl_up_sync(0xffffffffu, run, o);
+    if (lane >= o) run += up;
+  }
+  const float total = __shfl_sync(0xffffffffu, run, 31);
+  const float c1 = run, c0 = run - a2 * d1;
+  __syncwarp();
+  *reinterpret_cast<float2*>(cum + 2 * lane) = make_float2(c0, c1);
+  *reinterpret_cast<float2*>(wgt + 2 * lane) = make_float2(exp2f(total - c0) * d0, exp2f(total - c1) * d1);
+  __syncwarp();
+  return total;
+}
+
+// S (rows of this warp) <- keep * S + sum_j wgt_j B_j x_j^T
+template <int NI>
+__device__ __forceinline__ void ssd_update(float (&S)[NI][4][4], float keep, const float* wgt, uint32_t aB, uint32_t aX, int ldn,
+                                           int n16, int warp, int lane) {
 #pragma unroll
   for (int i = 0; i < NI; ++i)
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int n = (warp + 4 * i) * 16 + g4 + ((e & 2) ? 8 : 0), c = nt * 8 + 2 * t4 + (e & 1);
-        S[i][nt][e] = (start > 0 && n < d.N && c < pw) ? st[static_cast<long long>(n) * d.P4 + c] : 0.f;
+      for (int e = 0; e < 4; ++e) S[i][nt][e] *= keep;
+#pragma unroll
+  for (int kk = 0; kk < 4; ++kk) {
+    uint32_t fx[2][4];
+#pragma unroll
+    for (int np = 0; np < 2; ++np) ms_ldsm4_t(ms_b_nn_at(aX, kLdX, kk * 16, np * 16, lane), fx[np]);
+    const int j = kk * 16 + 2 * (lane & 3);
+    const float2 wa = *reinterpret_cast<const float2*>(wgt + j), wb = *reinterpret_cast<const float2*>(wgt + j + 8);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int n0 = (warp + 4 * i) * 16;
+      if (n0 >= n16) continue;
+      uint32_t fb[4], fh[4], fl[4];
+      ms_ldsm4_t(ms_a_t_at(aB, ldn, kk * 16, n0, lane), fb);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float lo = __uint_as_float(fb[q] << 16), hi = __uint_as_float(fb[q] & 0xffff0000u);
+        ms_split(lo * (q & 2 ? wb.x : wa.x), hi * (q & 2 ? wb.y : wa.y), fh[q], fl[q]);
       }
+#pragma unroll
+      for (int np = 0; np < 2; ++np) {
+        ms_mma(S[i][2 * np], fh, fx[np][0], fx[np][1]);
+        ms_mma(S[i][2 * np + 1], fh, fx[np][2], fx[np][3]);
+        ms_mma(S[i][2 * np], fl, fx[np][0], fx[np][1]);
+        ms_mma(S[i][2 * np + 1], fl, fx[np][2], fx[np][3]);
+      }
+    }
+  }
+}
+
+// Calls f(fragment pair, row n, channel c) for this thread's accumulator pairs (channels c, c + 1).
+template <int NI, typename F>
+__device__ __forceinline__ void ssd_each(float (&S)[NI][4][4], int n, int pw, int warp, int lane, F f) {
+#pragma unroll
+  for (int i = 0; i < NI; ++i)
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf) {
+        const int row = (warp + 4 * i) * 16 + (lane >> 2) + 8 * hf, c = nt * 8 + 2 * (lane & 3);
+        if (row < n && c < pw) f(S[i][nt][2 * hf], S[i][nt][2 * hf + 1], row, c);
+      }
+}
+
+// What every segment but the last adds to the state, with segment-parallel CTAs. grid (slices * n_seg, H, sequences).
+template <int NI>
+__global__ void __launch_bounds__(128) ssd_segment_kernel(const ChunkParams p) {
+  extern __shared__ __align__(16) uint8_t ssd_smem[];
+  const SsmDims& d = p.d;
+  const int slices = gridDim.x / p.n_seg;
+  const int seq = blockIdx.z, h = blockIdx.y, p0 = (blockIdx.x % slices) * kSlice, seg = blockIdx.x / slices;
+  const int len = p.q_lens[seq];
+  const int n_chunks = (len + kChunk - 1) / kChunk;
+  if ((seg + 1) * p.seg_chunks >= n_chunks) return;            // the last segment is summed by the main kernel
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int ldn = p.n16 + 8, tile_n = kChunk * ldn, tile_x = kChunk * kLdX;
+  __nv_bfloat16* sB = reinterpret_cast<__nv_bfloat16*>(ssd_smem);        // [2][64][ldn]
+  __nv_bfloat16* sX = sB + 2 * tile_n;                                   // [2][64][kLdX]
+  float* sDt = reinterpret_cast<float*>(sX + 2 * tile_x);                // [2][64]
+  float* cum = sDt + 2 * kChunk + warp * kChunk;                         // [4 warps][64]
+  float* wgt = sDt + 6 * kChunk + warp * kChunk;                         // [4 warps][64]
+  const long long q0 = p.q_start[seq];
+  const int start = p.seq_lens[seq] - len;
+  const int g = h / (d.H / d.G);
+  const int cx = h * d.P + p0, cb = d.inner + g * d.N, pw = min(kSlice, d.P - p0);
+  const float a2 = -expf(p.a_log[h]) * kLog2e;
+  const long long mat = static_cast<long long>(d.N) * d.P4;
+  auto slot_of = [&](int k) { return (static_cast<long long>(seq) * p.n_seg + k) * d.H + h; };
+  auto load_chunk = [&](int ch, int buf) {
+    const int t0 = ch * kChunk;
+    ssd_load_rows(p, sB + buf * tile_n, ldn, p.n16, d.N, cb, q0, t0, len);
+    ssd_load_rows(p, sX + buf * tile_x, kLdX, kSlice, pw, cx, q0, t0, len);
+    if (threadIdx.x < kChunk) sDt[buf * kChunk + threadIdx.x] = p.dt[(q0 + t0 + threadIdx.x) * d.H + h];
+    ms_commit();
+  };
+  float S[NI][4][4];
+#pragma unroll
+  for (int i = 0; i < NI; ++i)
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[i][nt][e] = 0.f;
+  const int c0 = seg * p.seg_chunks;
+  load_chunk(c0, 0);
+  if (seg == 0) {                                              // the starting state, before the main kernel overwrites it
+    const float* st = p.state + (static_cast<long long>(p.slots[seq]) * d.H + h) * mat + p0;
+    float* dst = p.seg_state + slot_of(0) * mat + p0;
+    ssd_each<NI>(S, d.N, pw, warp, lane, [&](float&, float&, int n, int c) {
+      const long long o = static_cast<long long>(n) * d.P4 + c;
+      *reinterpret_cast<float2*>(dst + o) = start > 0 ? *reinterpret_cast<const float2*>(st + o) : make_float2(0.f, 0.f);
+    });
+  }
+  float sum = 0.f;
+  for (int k = 0; k < p.seg_chunks; ++k) {
+    const int buf = k & 1;
+    ms_wait<0>();
+    __syncthreads();
+    if (k + 1 < p.seg_chunks) load_chunk(c0 + k + 1, buf ^ 1);
+    const float total = ssd_decays(sDt + buf * kChunk, a2, cum, wgt, lane);
+    sum += total;
+    ssd_update<NI>(S, exp2f(total), wgt, ms_addr(sB + buf * tile_n), ms_addr(sX + buf * tile_x), ldn, p.n16, warp, lane);
+  }
+  float* dst = p.seg_state + slot_of(seg + 1) * mat + p0;
+  ssd_each<NI>(S, d.N, pw, warp, lane, [&](float& v0, float& v1, int n, int c) {
+    *reinterpret_cast<float2*>(dst + static_cast<long long>(n) * d.P4 + c) = make_float2(v0, v1);
+  });
+  if (threadIdx.x == 0 && p0 == 0) p.seg_decay[slot_of(seg)] = exp2f(sum);
+}
+
+// NI: state row tiles (16 rows) per warp; 4 warps cover N <= 64 NI. Same grid as ssd_segment_kernel.
+template <int NI>
+__global__ void __launch_bounds__(128) ssd_chunk_kernel(const ChunkParams p) {
+  extern __shared__ __align__(16) uint8_t ssd_smem[];
+  const SsmDims& d = p.d;
+  const int slices = gridDim.x / p.n_seg;
+  const int seq = blockIdx.z, h = blockIdx.y, p0 = (blockIdx.x % slices) * kSlice, seg = blockIdx.x / slices;
+  const int len = p.q_lens[seq];
+  const int n_chunks = (len + kChunk - 1) / kChunk, ch0 = seg * p.seg_chunks, ch1 = min(n_chunks, ch0 + p.seg_chunks);
+  if (ch0 >= ch1) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, t4 = lane & 3;
+  const int ldn = p.n16 + 8, tile_n = kChunk * ldn, tile_x = kChunk * kLdX;
+  __nv_bfloat16* sC = reinterpret_cast<__nv_bfloat16*>(ssd_smem);        // [64][ldn]
+  __nv_bfloat16* sB = sC + tile_n;                                       // [64][ldn]
+  __nv_bfloat16* sX = sB + tile_n;                                       // [64][kLdX]
+  __nv_bfloat16* sSh = sX + tile_x;                                      // [n16][kLdX]
+  __nv_bfloat16* sSl = sSh + p.n16 * kLdX;                               // [n16][kLdX]
+  float* sDt = reinterpret_cast<float*>(sSl + p.n16 * kLdX);             // [64]
+  float* cum = sDt + kChunk + warp * kChunk;                             // [4 warps][64]
+  float* wgt = sDt + 5 * kChunk + warp * kChunk;                         // [4 warps][64]
+
+  const long long q0 = p.q_start[seq];
+  const int start = p.seq_lens[seq] - len;
+  const int g = h / (d.H / d.G);
+  const int cx = h * d.P + p0, cb = d.inner + g * d.N, cc = d.inner + (d.G + g) * d.N;
+  const int pw = min(kSlice, d.P - p0);
+  const float a2 = -expf(p.a_log[h]) * kLog2e, skip = p.dskip[h];
+  const long long mat = static_cast<long long>(d.N) * d.P4;
+  float* st = p.state + (static_cast<long long>(p.slots[seq]) * d.H + h) * mat + p0;
+
+  auto load_chunk = [&](int ch) {
+    const int t0 = ch * kChunk;
+    ssd_load_rows(p, sC, ldn, p.n16, d.N, cc, q0, t0, len);
+    ssd_load_rows(p, sB, ldn, p.n16, d.N, cb, q0, t0, len);
+    ssd_load_rows(p, sX, kLdX, kSlice, pw, cx, q0, t0, len);
+    if (threadIdx.x < kChunk)
+      sDt[threadIdx.x] = t0 + static_cast<int>(threadIdx.x) < len ? p.dt[(q0 + t0 + threadIdx.x) * d.H + h] : 0.f;
+    ms_commit();
+  };
+  load_chunk(ch0);
+
+  // this warp's rows of the state at the start of the segment, accumulator layout
+  float S[NI][4][4];
+#pragma unroll
+  for (int i = 0; i < NI; ++i)
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[i][nt][e] = 0.f;
+  if (n_chunks <= p.seg_chunks) {
+    if (start > 0)
+      ssd_each<NI>(S, d.N, pw, warp, lane, [&](float& v0, float& v1, int n, int c) {
+        const float2 v = *reinterpret_cast<const float2*>(st + static_cast<long long>(n) * d.P4 + c);
+        v0 = v.x;
+        v1 = v.y;
+      });
+  } else {
+    for (int k = 0; k <= seg; ++k) {
+      const long long o = (static_cast<long long>(seq) * p.n_seg + k) * d.H + h;
+      const float* src = p.seg_state + o * mat + p0;
+      const float keep = k > 0 ? p.seg_decay[o - d.H] : 0.f;
+      ssd_each<NI>(S, d.N, pw, warp, lane, [&](float& v0, float& v1, int n, int c) {
+        const float2 v = *reinterpret_cast<const float2*>(src + static_cast<long long>(n) * d.P4 + c);
+        v0 = fmaf(keep, v0, v.x);
+        v1 = fmaf(keep, v1, v.y);
+      });
+    }
+  }
   auto publish = [&]() {
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
@@ -328,36 +531,13 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const ChunkParams p) {
     }
   };
   publish();
-  load_chunk(0, 0);
-  float* cum = sCum + warp * kChunk;
-  float* wgt = sW + warp * kChunk;
-  const uint32_t aSh = ms_addr(sSh), aSl = ms_addr(sSl);
+  const uint32_t aC = ms_addr(sC), aB = ms_addr(sB), aX = ms_addr(sX), aSh = ms_addr(sSh), aSl = ms_addr(sSl);
+  const int r0 = warp * 16;
 
-  for (int ch = 0; ch < n_chunks; ++ch) {
-    const int buf = ch & 1;
+  for (int ch = ch0; ch < ch1; ++ch) {
     ms_wait<0>();
-    __syncthreads();                       // chunk data and the published state are visible; the other buffer is free
-    if (ch + 1 < n_chunks) load_chunk(ch + 1, buf ^ 1);
-    const float* dts = sDt + buf * kChunk;
-    // running sum of the log decays (every warp for itself)
-    const float d0 = dts[2 * lane], d1 = dts[2 * lane + 1];
-    float run = a * d0 + a * d1;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float up = __shfl_up_sync(0xffffffffu, run, o);
-      if (lane >= o) run += up;
-    }
-    const float total = __shfl_sync(0xffffffffu, run, 31);
-    const float c1 = run, c0 = run - a * d1;
-    __syncwarp();
-    cum[2 * lane] = c0;
-    cum[2 * lane + 1] = c1;
-    wgt[2 * lane] = __expf(total - c0) * d0;
-    wgt[2 * lane + 1] = __expf(total - c1) * d1;
-    __syncwarp();
-
-    const uint32_t aC = ms_addr(sC + buf * tile_n), aB = ms_addr(sB + buf * tile_n), aX = ms_addr(sX + buf * tile_x);
-    const int r0 = warp * 16;
+    __syncthreads();                       // the block's rows and the published state are visible
+    const float total = ssd_decays(sDt, a2, cum, wgt, lane);
     float s[8][4], yi[4][4], y[4][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i)
@@ -386,8 +566,8 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const ChunkParams p) {
         ms_ldsm4_t(ms_b_nn_at(aSh, kLdX, k, np * 16, lane), fh);
         ms_ldsm4_t(ms_b_nn_at(aSl, kLdX, k, np * 16, lane), fl);
         ms_mma(yi[2 * np], fa, fh[0], fh[1]);
-        ms_mma(yi[2 * np], fa, fl[0], fl[1]);
         ms_mma(yi[2 * np + 1], fa, fh[2], fh[3]);
+        ms_mma(yi[2 * np], fa, fl[0], fl[1]);
         ms_mma(yi[2 * np + 1], fa, fl[2], fl[3]);
       }
     }
@@ -397,12 +577,15 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const ChunkParams p) {
       if (kk > warp) break;
       float m[2][4];
 #pragma unroll
-      for (int q = 0; q < 2; ++q)
+      for (int q = 0; q < 2; ++q) {
+        const int j0 = kk * 16 + q * 8 + 2 * t4;
+        const float2 cj = *reinterpret_cast<const float2*>(cum + j0), dj = *reinterpret_cast<const float2*>(sDt + j0);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int j = kk * 16 + q * 8 + 2 * t4 + (e & 1), i = r0 + g4 + ((e & 2) ? 8 : 0);
-          m[q][e] = j <= i ? s[2 * kk + q][e] * __expf(ci[e >> 1] - cum[j]) * dts[j] : 0.f;
+          const bool seen = kk < warp || j0 + (e & 1) <= r0 + g4 + ((e & 2) ? 8 : 0);
+          m[q][e] = seen ? s[2 * kk + q][e] * exp2f(ci[e >> 1] - ((e & 1) ? cj.y : cj.x)) * ((e & 1) ? dj.y : dj.x) : 0.f;
         }
+      }
       uint32_t fh[4], fl[4];
       ms_split(m[0][0], m[0][1], fh[0], fl[0]);
       ms_split(m[0][2], m[0][3], fh[1], fl[1]);
@@ -413,13 +596,13 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const ChunkParams p) {
         uint32_t fx[4];
         ms_ldsm4_t(ms_b_nn_at(aX, kLdX, kk * 16, np * 16, lane), fx);
         ms_mma(y[2 * np], fh, fx[0], fx[1]);
-        ms_mma(y[2 * np], fl, fx[0], fx[1]);
         ms_mma(y[2 * np + 1], fh, fx[2], fx[3]);
+        ms_mma(y[2 * np], fl, fx[0], fx[1]);
         ms_mma(y[2 * np + 1], fl, fx[2], fx[3]);
       }
     }
     // y of this warp's 16 tokens
-    const float ei[2] = {__expf(ci[0]), __expf(ci[1])};
+    const float ei[2] = {exp2f(ci[0]), exp2f(ci[1])};
     const int t0 = ch * kChunk;
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt)
@@ -427,8 +610,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const ChunkParams p) {
       for (int hf = 0; hf < 2; ++hf) {
         const int i = r0 + g4 + 8 * hf, c = nt * 8 + 2 * t4;
         if (t0 + i >= len || c >= pw) continue;
-        const __nv_bfloat162 xv = *reinterpret_cast<const __nv_bfloat162*>(sX + buf * tile_x + i * kLdX + c);
-        const float2 xf = __bfloat1622float2(xv);
+        const float2 xf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + i * kLdX + c));
         const float v0 = fmaf(skip, xf.x, fmaf(ei[hf], yi[nt][2 * hf], y[nt][2 * hf]));
         const float v1 = fmaf(skip, xf.y, fmaf(ei[hf], yi[nt][2 * hf + 1], y[nt][2 * hf + 1]));
         __nv_bfloat16* dst = p.y + (q0 + t0 + i) * d.inner + cx + c;
@@ -439,53 +621,18 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const ChunkParams p) {
           if (c + 1 < pw) dst[1] = __float2bfloat16(v1);
         }
       }
-    // state
-    const float keep = __expf(total);
-#pragma unroll
-    for (int i = 0; i < NI; ++i)
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) S[i][nt][e] *= keep;
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
-      uint32_t fx[2][4];
-#pragma unroll
-      for (int np = 0; np < 2; ++np) ms_ldsm4_t(ms_b_nn_at(aX, kLdX, kk * 16, np * 16, lane), fx[np]);
-      const int j = kk * 16 + 2 * t4;
-      const float w[4] = {wgt[j], wgt[j + 1], wgt[j + 8], wgt[j + 9]};
-#pragma unroll
-      for (int i = 0; i < NI; ++i) {
-        const int n0 = (warp + 4 * i) * 16;
-        if (n0 >= p.n16) continue;
-        uint32_t fb[4], fh[4], fl[4];
-        ms_ldsm4_t(ms_a_t_at(aB, ldn, kk * 16, n0, lane), fb);
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          const float lo = __uint_as_float(fb[q] << 16), hi = __uint_as_float(fb[q] & 0xffff0000u);
-          ms_split(lo * w[(q & 2)], hi * w[(q & 2) + 1], fh[q], fl[q]);
-        }
-#pragma unroll
-        for (int np = 0; np < 2; ++np) {
-          ms_mma(S[i][2 * np], fh, fx[np][0], fx[np][1]);
-          ms_mma(S[i][2 * np], fl, fx[np][0], fx[np][1]);
-          ms_mma(S[i][2 * np + 1], fh, fx[np][2], fx[np][3]);
-          ms_mma(S[i][2 * np + 1], fl, fx[np][2], fx[np][3]);
-        }
-      }
+    if (ch + 1 < ch1 || ch1 == n_chunks)
+      ssd_update<NI>(S, exp2f(total), wgt, aB, aX, ldn, p.n16, warp, lane);
+    __syncthreads();                       // everyone has read this block's rows and the published state
+    if (ch + 1 < ch1) {
+      load_chunk(ch + 1);
+      publish();
     }
-    __syncthreads();                       // everyone has read the published state of this chunk
-    if (ch + 1 < n_chunks) publish();
   }
-#pragma unroll
-  for (int i = 0; i < NI; ++i)
-#pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int n = (warp + 4 * i) * 16 + g4 + ((e & 2) ? 8 : 0), c = nt * 8 + 2 * t4 + (e & 1);
-        if (n < d.N && c < pw) st[static_cast<long long>(n) * d.P4 + c] = S[i][nt][e];
-      }
+  if (ch1 == n_chunks)
+    ssd_each<NI>(S, d.N, pw, warp, lane, [&](float& v0, float& v1, int n, int c) {
+      *reinterpret_cast<float2*>(st + static_cast<long long>(n) * d.P4 + c) = make_float2(v0, v1);
+    });
 }
 
 // ------------------------------------------------------------------------------------------- gate, norm, ring
@@ -494,7 +641,7 @@ __global__ void ssm_gate_norm_kernel(const T* __restrict__ y, const T* __restric
                                      const float* __restrict__ w, float eps, int parts, T* __restrict__ out,
                                      T* __restrict__ ring, const int* __restrict__ slots, const int* __restrict__ seq_of,
                                      const int* __restrict__ pos, const int* __restrict__ seq_lens, SsmDims d) {
-  extern __shared__ float part_row[];
+  extern __shared__ __align__(16) float part_row[];
   const long long t = blockIdx.x;
   const int part = blockIdx.y, width = d.inner / parts, c0 = part * width;
   // the last taps - 1 inputs of the convolution stay with the sequence
@@ -523,6 +670,59 @@ __global__ void ssm_gate_norm_kernel(const T* __restrict__ y, const T* __restric
 #pragma unroll
     for (int e = 0; e < V; ++e) v[e] = part_row[k + e] * r * g[e];
     store_vec<V>(out + t * d.inner + c0 + k, v);
+  }
+}
+
+// The same with one warp per (token, part) and the part in registers: widths up to 256 IT, rows copied in 8-element vectors.
+template <typename T, int IT>
+__global__ void __launch_bounds__(256) ssm_gate_norm_warp_kernel(const T* __restrict__ y, const T* __restrict__ u, long long ldu,
+                                                                 const float* __restrict__ w, float eps, int parts,
+                                                                 T* __restrict__ out, T* __restrict__ ring,
+                                                                 const int* __restrict__ slots, const int* __restrict__ seq_of,
+                                                                 const int* __restrict__ pos, const int* __restrict__ seq_lens,
+                                                                 int n_tok, SsmDims d) {
+  const long long item = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  const long long t = item / parts;
+  if (t >= n_tok) return;
+  const int part = static_cast<int>(item - t * parts), width = d.inner / parts, c0 = part * width;
+  float v[IT][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < IT; ++i) {
+    const int k = (i * 32 + lane) * 8;
+    if (k < width) {
+      float z[8];
+      load_vec<8>(y + t * d.inner + c0 + k, v[i]);
+      load_vec<8>(u + t * ldu + c0 + k, z);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        v[i][e] *= silu_f(z[e]);
+        ss = fmaf(v[i][e], v[i][e], ss);
+      }
+    }
+  }
+  const float r = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(width) + eps);
+#pragma unroll
+  for (int i = 0; i < IT; ++i) {
+    const int k = (i * 32 + lane) * 8;
+    if (k < width) {
+      float g[8];
+      load_vec<8>(w + c0 + k, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[i][e] *= r * g[e];
+      store_vec<8>(out + t * d.inner + c0 + k, v[i]);
+    }
+  }
+  const int seq = seq_of[t], ps = pos[t];
+  if (seq_lens[seq] - ps < d.taps) {
+    T* dst = ring + (static_cast<long long>(slots[seq]) * d.taps + ps % d.taps) * d.conv;
+    const T* src = u + t * ldu + d.inner;
+    for (int c = (part * 32 + lane) * 8; c < d.conv; c += parts * 256) {
+      float x[8];
+      load_vec<8>(src + c, x);
+      store_vec<8>(dst + c, x);
+    }
   }
 }
 
@@ -557,6 +757,17 @@ static ScanParams<T> scan_params(const void* u, long long ldu, const float* conv
   p.a_log = a_log; p.dskip = dskip; p.ring = static_cast<const T*>(ring); p.state = state; p.slots = slots;
   p.q_start = q_start; p.q_lens = q_lens; p.seq_lens = seq_lens; p.y = static_cast<T*>(y); p.d = d;
   return p;
+}
+
+template <typename T, int IT>
+static int gate_norm_warp_launch(const void* y, const void* u, long long ldu, const float* w, float eps, int parts, void* out,
+                                 void* ring, const int* slots, const int* seq_of, const int* pos, const int* seq_lens, int n_tok,
+                                 const SsmDims& d, cudaStream_t st) {
+  const long long items = static_cast<long long>(n_tok) * parts;
+  ssm_gate_norm_warp_kernel<T, IT><<<static_cast<unsigned>((items + 7) / 8), 256, 0, st>>>(
+      static_cast<const T*>(y), static_cast<const T*>(u), ldu, w, eps, parts, static_cast<T*>(out), static_cast<T*>(ring),
+      slots, seq_of, pos, seq_lens, n_tok, d);
+  return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T, int V>
@@ -609,13 +820,15 @@ extern "C" int pm_ssm_scan(const void* u, int f32, long long ldu, const float* c
 // Whether pm_ssm_chunk covers a state of N rows.
 extern "C" int pm_ssm_chunk_supported(int N) { return N >= 1 && N <= 128; }
 
-// The same for longer portions of bf16 models: act [tokens, conv] bf16 and dt [tokens, H] fp32 are work buffers that the
-// first kernel fills, max_q is the longest of q_lens.
+// The same for longer portions of bf16 models: act [tokens, conv] bf16, dt [tokens, H], seg_state [n_seq][max_seg][H][N][P4]
+// and seg_decay [n_seq][max_seg][H] fp32 are work buffers, max_q is the longest of q_lens. A portion is cut into at most
+// max_seg segments that run in parallel (fewer when sequences and heads fill the machine by themselves).
 extern "C" int pm_ssm_chunk(const void* u, long long ldu, const float* conv_w, const float* conv_b, const float* dt_bias,
                             const float* a_log, const float* dskip, const void* ring, float* state, const int* slots,
                             const int* q_start, const int* q_lens, const int* seq_lens, int n_seq, int max_q, int H, int P,
-                            int N, int G, int taps, void* act, float* dt, void* y, cudaStream_t st) {
-  if (ssm_bad_dims(H, P, N, G, taps) || !pm_ssm_chunk_supported(N)) return -1;
+                            int N, int G, int taps, void* act, float* dt, float* seg_state, float* seg_decay,
+                            int max_seg, void* y, cudaStream_t st) {
+  if (ssm_bad_dims(H, P, N, G, taps) || !pm_ssm_chunk_supported(N) || max_seg < 1) return -1;
   if (n_seq < 1 || max_q < 1) return 0;
   const SsmDims d = make_dims(H, P, N, G, taps);
   if (ldu < d.inner + d.conv + H) return -2;
@@ -624,10 +837,11 @@ extern "C" int pm_ssm_chunk(const void* u, long long ldu, const float* conv_w, c
   c.ring = static_cast<const __nv_bfloat16*>(ring); c.slots = slots; c.q_start = q_start; c.q_lens = q_lens;
   c.seq_lens = seq_lens; c.act = static_cast<__nv_bfloat16*>(act); c.dt = dt; c.d = d;
   const int tiles = (max_q + kConvTokens - 1) / kConvTokens;
-  if (d.conv % 8 == 0 && d.inner % 8 == 0 && ldu % 8 == 0)
-    ssm_conv_kernel<8><<<dim3(tiles, n_seq, (d.conv / 8 + 127) / 128 + 1), 128, 0, st>>>(c);
-  else
-    ssm_conv_kernel<1><<<dim3(tiles, n_seq, (d.conv + 127) / 128 + 1), 128, 0, st>>>(c);
+  const int v = d.conv % 4 == 0 && d.inner % 4 == 0 && ldu % 4 == 0 ? 4 : 1;
+  const dim3 g_conv(tiles, n_seq, (d.conv / v + 127) / 128 + 1);
+  if (v == 4 && taps == 4) ssm_conv_kernel<4, 4><<<g_conv, 128, 0, st>>>(c);
+  else if (v == 4) ssm_conv_kernel<4, 0><<<g_conv, 128, 0, st>>>(c);
+  else ssm_conv_kernel<1, 0><<<g_conv, 128, 0, st>>>(c);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return static_cast<int>(e);
   ChunkParams p{};
@@ -635,15 +849,35 @@ extern "C" int pm_ssm_chunk(const void* u, long long ldu, const float* conv_w, c
   p.q_lens = q_lens; p.seq_lens = seq_lens; p.y = static_cast<__nv_bfloat16*>(y); p.d = d;
   p.n16 = (N + 15) / 16 * 16;
   p.aligned = d.conv % 8 == 0 && d.inner % 8 == 0 && N % 8 == 0 && P % 8 == 0;
-  const size_t smem = (2ull * 2 * kChunk * (p.n16 + 8) + 2ull * kChunk * kLdX + 2ull * p.n16 * kLdX) * 2 + 10ull * kChunk * 4;
+  // enough CTAs to keep three on every SM for a few rounds
+  const int slices = (P + kSlice - 1) / kSlice, n_chunks = (max_q + kChunk - 1) / kChunk;
+  const long long base = static_cast<long long>(slices) * H * n_seq;
+  long long want = (6ll * num_sms() + base - 1) / base;
+  if (want > max_seg) want = max_seg;
+  if (want > n_chunks) want = n_chunks;
+  p.seg_chunks = (n_chunks + static_cast<int>(want) - 1) / static_cast<int>(want);
+  p.n_seg = (n_chunks + p.seg_chunks - 1) / p.seg_chunks;
+  p.seg_state = seg_state;
+  p.seg_decay = seg_decay;
+  const size_t tile_n = static_cast<size_t>(kChunk) * (p.n16 + 8), tile_x = static_cast<size_t>(kChunk) * kLdX;
+  const size_t smem = (2 * tile_n + tile_x + 2 * static_cast<size_t>(p.n16) * kLdX) * 2 + 9 * kChunk * 4;
+  const size_t smem_seg = (2 * tile_n + 2 * tile_x) * 2 + 10 * kChunk * 4;
   static DeviceOnce once;
   if (once.pending()) {
-    e = cudaFuncSetAttribute(ssd_chunk_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(ssd_chunk_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+    e = cudaFuncSetAttribute(ssd_chunk_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(ssd_chunk_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(ssd_segment_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(ssd_segment_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
     if (e != cudaSuccess) return static_cast<int>(e);
     once.mark();
   }
-  const dim3 grid((P + kSlice - 1) / kSlice, H, n_seq);
+  const dim3 grid(slices * p.n_seg, H, n_seq);
+  if (p.n_seg > 1) {
+    if (p.n16 <= 64) ssd_segment_kernel<1><<<grid, 128, smem_seg, st>>>(p);
+    else ssd_segment_kernel<2><<<grid, 128, smem_seg, st>>>(p);
+    e = cudaGetLastError();
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
   if (p.n16 <= 64) ssd_chunk_kernel<1><<<grid, 128, smem, st>>>(p);
   else ssd_chunk_kernel<2><<<grid, 128, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
@@ -659,6 +893,13 @@ extern "C" int pm_ssm_gate_norm(const void* y, const void* u, int f32, long long
   const SsmDims d = make_dims(H, P, N, G, taps);
   const int width = d.inner / parts;
   if (static_cast<size_t>(width) * 4 > 200 * 1024) return -2;
+  if (!f32 && width % 8 == 0 && ldu % 8 == 0 && d.conv % 8 == 0 && width <= 1024) {
+    if (width <= 256)
+      return gate_norm_warp_launch<__nv_bfloat16, 1>(y, u, ldu, w, eps, parts, out, ring, slots, seq_of, pos, seq_lens, n_tok, d, st);
+    if (width <= 512)
+      return gate_norm_warp_launch<__nv_bfloat16, 2>(y, u, ldu, w, eps, parts, out, ring, slots, seq_of, pos, seq_lens, n_tok, d, st);
+    return gate_norm_warp_launch<__nv_bfloat16, 4>(y, u, ldu, w, eps, parts, out, ring, slots, seq_of, pos, seq_lens, n_tok, d, st);
+  }
   const bool vec = width % 4 == 0 && ldu % 4 == 0;
   if (f32)
     return vec ? gate_norm_launch<float, 4>(y, u, ldu, w, eps, parts, out, ring, slots, seq_of, pos, seq_lens, n_tok, d, st)

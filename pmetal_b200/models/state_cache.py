@@ -98,7 +98,7 @@ class StateCache(PagedBlocks):
 @dataclass
 class SeqGroup:
     """Some sequences of a step, as the kernels take them. ``q_start`` points into the step's token rows, ``c_start`` into
-    rows counted over the group alone."""
+    tokens counted over the group alone; ``tok_rows`` is the step's row of each of those tokens."""
     n: int
     n_tok: int
     max_q: int
@@ -109,6 +109,7 @@ class SeqGroup:
     q_lens: torch.Tensor
     c_start: torch.Tensor
     state_slots: Optional[torch.Tensor]
+    tok_rows: torch.Tensor
     host: List[Tuple[int, int, int, int]] = field(default_factory=list)     # (batch index, q_start, q_len, seq_len)
 
 
@@ -120,7 +121,7 @@ def split_groups(meta: BatchMeta, limit: int) -> Tuple[Optional[SeqGroup], Optio
             raise ValueError("a step without host metadata must bring one token per sequence")
         n = meta.q_lens.shape[0]
         return SeqGroup(n, n, 1, meta.max_kv, meta.block_table, meta.seq_lens, meta.q_start, meta.q_lens, meta.q_start,
-                        meta.state_slots), None
+                        meta.state_slots, meta.q_start), None
     _, _, seq_lens, q_start, q_lens, _ = meta.host
     sides = ([i for i, q in enumerate(q_lens) if q <= limit], [i for i, q in enumerate(q_lens) if q > limit])
     out = []
@@ -136,11 +137,13 @@ def split_groups(meta: BatchMeta, limit: int) -> Tuple[Optional[SeqGroup], Optio
         mq, mk = max(q_lens[i] for i in ix), max(seq_lens[i] for i in ix)
         if len(ix) == len(q_lens):
             out.append(SeqGroup(len(ix), c, mq, mk, meta.block_table, meta.seq_lens, meta.q_start, meta.q_lens,
-                                meta.q_start, meta.state_slots, host))
+                                meta.q_start, meta.state_slots,
+                                torch.arange(c, dtype=torch.int32, device=meta.q_lens.device), host))
             continue
         dev = meta.q_lens.device
+        rows = torch.tensor([q_start[i] + k for i in ix for k in range(q_lens[i])], dtype=torch.int32).to(dev, non_blocking=True)
         sel = torch.tensor(ix, dtype=torch.int64).to(dev, non_blocking=True)
         cs = torch.tensor(c_start, dtype=torch.int32).to(dev, non_blocking=True)
         out.append(SeqGroup(len(ix), c, mq, mk, meta.block_table[sel], meta.seq_lens[sel], meta.q_start[sel],
-                            meta.q_lens[sel], cs, meta.state_slots[sel] if meta.state_slots is not None else None, host))
+                            meta.q_lens[sel], cs, meta.state_slots[sel] if meta.state_slots is not None else None, rows, host))
     return out[0], out[1]

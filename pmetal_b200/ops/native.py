@@ -689,14 +689,17 @@ def attn_fwd(q, k, v, seq_start, scale: float, window: int = 0):
     return out, lse
 
 
-def attn_fwd_rect(q, k, v, seq_start, scale: float, shift: int):
+def attn_fwd_rect(q, k, v, seq_start, scale: float, shift: int, out=None):
     """Attention of Tq queries over Tk keys where key j is visible to query i iff seq_start[i] <= j <= i + shift
     (shift >= Tk - 1: every key). q [Tq, hq, 128], k/v [Tk, hkv, 128] (k/v may live in a peer GPU's memory: the
-    kernel's TMA loads read them in place). Returns (out bf16 [Tq, hq, 128], lse fp32 [hq, Tq])."""
+    kernel's TMA loads read them in place). Returns (out bf16 [Tq, hq, 128], lse fp32 [hq, Tq]); ``out`` may be given (any
+    token stride)."""
     T, hq, d = q.shape
     Tk, hkv = k.shape[0], k.shape[1]
     assert d == 128 and q.stride(1) == d and k.stride(1) == d and v.stride(1) == d
-    out = torch.empty(T, hq, d, dtype=q.dtype, device=q.device)
+    if out is None:
+        out = torch.empty(T, hq, d, dtype=q.dtype, device=q.device)
+    assert out.shape == q.shape and out.stride(1) == d
     lse = torch.empty(hq, T, dtype=torch.float32, device=q.device)
     _chk(lib().pm_attn_fwd_tc_rect(_p(q), c_ll(q.stride(0)), _p(k), c_ll(k.stride(0)), _p(v), c_ll(v.stride(0)), _p(out),
                                    c_ll(out.stride(0)), _p(lse), _p(seq_start), c_int(T), c_int(Tk), c_int(shift),
@@ -1247,11 +1250,15 @@ def ssm_chunk(u, conv_w, conv_b, dt_bias, a_log, dskip, ring, state, group, dims
     T = u.shape[0]
     act = torch.empty(T, H * P + 2 * G * N, dtype=torch.bfloat16, device=u.device)
     dt = torch.empty(T, H, dtype=torch.float32, device=u.device)
+    # segments in parallel: as many as the longest portion has blocks, no more than a few rounds of CTAs need
+    max_seg = max(1, min(-(-group.max_q // 64), -(-6 * sm_count() // max(-(-P // 32) * H * group.n, 1))))
+    seg = torch.empty(group.n * max_seg * H, N * (-(-P // 4) * 4) + 1, dtype=torch.float32, device=u.device)
+    seg_decay = seg.view(-1)[group.n * max_seg * H * N * (-(-P // 4) * 4):]
     _chk(lib().pm_ssm_chunk(_p(u), c_ll(u.stride(0)), _p(conv_w), _p(conv_b), _p(dt_bias), _p(a_log), _p(dskip), _p(ring),
                             _p(state), _p(group.state_slots), _p(group.q_start), _p(group.q_lens), _p(group.seq_lens),
                             c_int(group.n), c_int(group.max_q), c_int(H), c_int(P), c_int(N), c_int(G), c_int(taps),
-                            _p(act), _p(dt), _p(y), _stream()), "pm_ssm_chunk")
-    LAUNCHES += 1          # two kernels
+                            _p(act), _p(dt), _p(seg), _p(seg_decay), c_int(max_seg), _p(y), _stream()), "pm_ssm_chunk")
+    LAUNCHES += 1 + int(max_seg > 1)
 
 
 def ssm_gate_norm(y, u, w, eps: float, parts: int, ring, meta, dims):
@@ -1288,13 +1295,13 @@ def latent_attn(qd, wuk, wuv, pages, group, dims, scale: float, out) -> None:
         tile = 32 if H > 16 else 16
         ctas = group.n * -(-group.max_q * H // tile)
         n_blocks = -(-group.max_kv // 64)
-        n_split = max(1, min(sm_count() // max(ctas, 1), n_blocks, 64))
+        n_split = max(1, min(sm_count() // max(ctas, 1), -(-n_blocks // 2), 64))
     dev = qd.device
     q_lat = torch.empty(group.n_tok, H, W, dtype=qd.dtype, device=dev)
     po = torch.empty(n_split, group.n_tok * H, rank, dtype=torch.float32, device=dev)
     pml = torch.empty(n_split, group.n_tok * H, 2, dtype=torch.float32, device=dev)
     _chk(lib().pm_latent_attn(_p(qd), _is_f32(qd), c_ll(qd.stride(0)), _p(wuk), _p(wuv), _p(pages), _p(group.block_table),
-                              _p(group.seq_lens), _p(group.q_start), _p(group.c_start), _p(group.q_lens), c_int(group.n),
+                              _p(group.seq_lens), _p(group.c_start), _p(group.q_lens), _p(group.tok_rows), c_int(group.n),
                               c_int(group.block_table.shape[1]), c_int(group.n_tok), c_int(group.max_q), c_int(H), c_int(dn),
                               c_int(dr), c_int(dv), c_int(rank), c_int(W), c_int(n_split), c_float(scale), _p(q_lat), _p(po),
                               _p(pml), _p(out), c_ll(out.stride(0)), _stream()), "pm_latent_attn")
@@ -1311,12 +1318,21 @@ def latent_expand_attn(qd, wukv, pages, table_row, n_keys: int, dims, scale: flo
     _chk(lib().pm_latent_gather(_p(pages), _p(table_row), c_int(n_keys), c_int(W), c_int(rank), c_int(r8), _p(lat),
                                 _stream()), "pm_latent_gather")
     kv = gemm(lat, wukv)
-    q128 = torch.empty(n_q, H, 128, dtype=torch.bfloat16, device=dev)
-    k128 = torch.empty(n_keys, H, 128, dtype=torch.bfloat16, device=dev)
-    v128 = torch.empty(n_keys, H, 128, dtype=torch.bfloat16, device=dev)
+    # operands whose heads already have 128 channels in 16-byte aligned rows are read in place
+    heads = lambda t, c0: t[:, c0:c0 + H * 128].unflatten(1, (H, 128))      # noqa: E731
+    fits = lambda t: t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0      # noqa: E731
+    q128 = heads(qd, 0) if dn + dr == 128 else None
+    v128 = heads(kv, H * dn) if dv == 128 else None
+    o128 = heads(out, 0) if dv == 128 else None
+    q_in, v_in = q128 is not None and fits(q128), v128 is not None and fits(v128)
+    direct = o128 is not None and fits(o128)
+    buf = lambda n: torch.empty(n, H, 128, dtype=torch.bfloat16, device=dev)      # noqa: E731
+    q128, v128, k128 = q128 if q_in else buf(n_q), v128 if v_in else buf(n_keys), buf(n_keys)
     _chk(lib().pm_latent_assemble(_p(qd), c_ll(qd.stride(0)), c_int(n_q), _p(kv), c_ll(kv.stride(0)), c_int(n_keys),
                                   _p(pages), _p(table_row), c_int(W), c_int(rank), c_int(H), c_int(dn), c_int(dr),
-                                  c_int(dv), _p(q128), _p(k128), _p(v128), _stream()), "pm_latent_assemble")
-    o, _ = attn_fwd_rect(q128, k128, v128, zeros[:n_q], scale, n_keys - n_q)
-    _chk(lib().pm_latent_take(_p(o), c_int(n_q), c_int(H), c_int(dv), _p(out), c_ll(out.stride(0)), _stream()),
-         "pm_latent_take")
+                                  c_int(dv), _p(None if q_in else q128), _p(k128), _p(None if v_in else v128), _stream()),
+         "pm_latent_assemble")
+    o, _ = attn_fwd_rect(q128, k128, v128, zeros[:n_q], scale, n_keys - n_q, o128 if direct else None)
+    if not direct:
+        _chk(lib().pm_latent_take(_p(o), c_int(n_q), c_int(H), c_int(dv), _p(out), c_ll(out.stride(0)), _stream()),
+             "pm_latent_take")

@@ -256,6 +256,7 @@ def test_split_groups():
     meta = c.prepare([0, 1, 2, 3], [1, 40, 2, 17])
     s, l = split_groups(meta, 16)
     assert (s.n, s.n_tok, s.max_q, s.max_kv) == (2, 3, 2, 102) and s.q_start.tolist() == [0, 41] and s.c_start.tolist() == [0, 1]
+    assert s.tok_rows.tolist() == [0, 41, 42]
     assert s.seq_lens.tolist() == [1, 102] and s.state_slots.tolist() == [c.slot_of[0], c.slot_of[2]]
     assert (l.n, l.max_q) == (2, 40) and l.host == [(1, 1, 40, 40), (3, 43, 17, 17)]
     a, b = split_groups(meta, 64)
