@@ -9,8 +9,8 @@
 //   latent_prep_kernel      norm of the latent, rotation of k_r and of the queries' rotated part, cache append
 //   latent_absorb_kernel    [q_l | q_r | 0] rows of width W
 //   latent_attn_mma_kernel  bf16, split over key pages: 16 or 32 (token, head) rows share each 64-key page in shared
-//                           memory; S by mma.sync with keys and rows (or columns) cut over 16 warps, P V with the columns
-//                           cut over the warps
+//                           memory; S by mma.sync with keys and row quarters cut over the warps (query fragments stay in
+//                           registers), P V with the columns cut over the warps
 //   latent_attn_row_kernel  any type and size, one (token, head) row per CTA (fp32 models)
 //   latent_up_kernel        joins the splits and applies W_uv
 // Longer portions expand keys and values of the visible rows with one GEMM and run the flash-attention kernels of
@@ -83,15 +83,17 @@ __global__ void latent_prep_kernel(T* __restrict__ qd, long long ld, const float
   }
 }
 
-// grid (column tiles of 128 plus one, H, groups of kAbsTok tokens), 128 / V threads. The CTA computes 128 columns of q_l for
-// kAbsTok tokens of one head (compact token i is row rows[i] of qd); the last column tile copies the rotated part and zeroes
-// the rest.
+// grid (column tiles of 128 plus one, H, groups of kAbsTok tokens), 256 threads. The CTA computes 128 columns of q_l for
+// kAbsTok tokens of one head (compact token i is row rows[i] of qd): 128 / V threads side by side own the columns, the
+// groups of threads behind them cut the unrotated dimensions and meet in shared memory. The last column tile copies the
+// rotated part and zeroes the rest.
 constexpr int kAbsTok = 8;
 template <typename T, int V>
-__global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict__ qd, long long ld, const T* __restrict__ wuk,
+__global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict__ qd, long long ld, const T* __restrict__ wuk,
                                                             int H, int dn, int dr, int rank, int W, const int* __restrict__ rows,
                                                             int n, T* __restrict__ out) {
-  extern __shared__ __align__(16) float abs_q[];           // [kAbsTok][dn]
+  extern __shared__ __align__(16) float abs_q[];           // [dn][kAbsTok], then [groups][kAbsTok][128]
+  constexpr int kCols = 128 / V, kGroups = 256 / kCols;
   const int h = blockIdx.y, t0 = blockIdx.z * kAbsTok, n_tok = min(kAbsTok, n - t0);
   if (blockIdx.x == gridDim.x - 1) {
     const int tail = W - rank;
@@ -102,33 +104,46 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const T* __restrict_
     }
     return;
   }
-  for (int t = 0; t < kAbsTok; ++t) {
+  float* red = abs_q + dn * kAbsTok;
+  {
+    const int t = threadIdx.x >> 5;                        // one warp per token
     const T* q = qd + (t < n_tok ? rows[t0 + t] : 0) * ld + h * (dn + dr);
-    for (int j = threadIdx.x; j < dn; j += blockDim.x) abs_q[t * dn + j] = t < n_tok ? to_f(q[j]) : 0.f;
+    for (int j = threadIdx.x & 31; j < dn; j += 32) abs_q[j * kAbsTok + t] = t < n_tok ? to_f(q[j]) : 0.f;
   }
-  __syncthreads();
-  const int c = blockIdx.x * 128 + threadIdx.x * V;
-  if (c >= rank) return;
+  const int col = (threadIdx.x % kCols) * V, grp = threadIdx.x / kCols, c = blockIdx.x * 128 + col;
+  const int per = (dn + kGroups - 1) / kGroups, j0 = grp * per, j1 = min(dn, j0 + per);
   float acc[kAbsTok][V];
 #pragma unroll
   for (int t = 0; t < kAbsTok; ++t)
 #pragma unroll
     for (int e = 0; e < V; ++e) acc[t][e] = 0.f;
-  const T* w = wuk + static_cast<long long>(h) * dn * rank + c;
+  __syncthreads();
+  if (c < rank) {
+    const T* w = wuk + static_cast<long long>(h) * dn * rank + c;
 #pragma unroll 16
-  for (int j = 0; j < dn; ++j) {
-    float wv[V];
-    load_pair<V>(w + static_cast<long long>(j) * rank, wv);
+    for (int j = j0; j < j1; ++j) {
+      float wv[V], qa[kAbsTok];
+      load_pair<V>(w + static_cast<long long>(j) * rank, wv);
+      load_vec<kAbsTok>(abs_q + j * kAbsTok, qa);
 #pragma unroll
-    for (int t = 0; t < kAbsTok; ++t)
+      for (int t = 0; t < kAbsTok; ++t)
 #pragma unroll
-      for (int e = 0; e < V; ++e) acc[t][e] = fmaf(abs_q[t * dn + j], wv[e], acc[t][e]);
+        for (int e = 0; e < V; ++e) acc[t][e] = fmaf(qa[t], wv[e], acc[t][e]);
+    }
   }
 #pragma unroll
   for (int t = 0; t < kAbsTok; ++t)
-    if (t < n_tok)
 #pragma unroll
-      for (int e = 0; e < V; ++e) put(out + (static_cast<long long>(t0 + t) * H + h) * W + c + e, acc[t][e]);
+    for (int e = 0; e < V; ++e) red[(grp * kAbsTok + t) * 128 + col + e] = acc[t][e];
+  __syncthreads();
+  for (int i = threadIdx.x; i < n_tok * 128; i += 256) {
+    const int t = i >> 7, k = i & 127, cc = blockIdx.x * 128 + k;
+    if (cc >= rank) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int g = 0; g < kGroups; ++g) v += red[(g * kAbsTok + t) * 128 + k];
+    put(out + (static_cast<long long>(t0 + t) * H + h) * W + cc, v);
+  }
 }
 
 struct LatentParams {
@@ -201,19 +216,21 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const LatentParams
   }
 }
 
-// 16 warps. MT: 16-row tiles of (token, head) rows; NT: 8-column tiles of the latent per warp.
-constexpr int kMmaThreads = 512;
-template <int MT, int NT>
+// 8 warps. MT: 16-row tiles of (token, head) rows; KS: 16-column steps of a quarter of the row; NT: 8-column tiles of the
+// latent per warp. Warp w scores keys 32 (w % 2) .. + 31 of a page over column quarter w / 2, with the quarter's query
+// fragments in registers for all pages; the softmax adds the four partial scores; for P V warp w owns columns 8 (w + 8 j).
+constexpr int kMmaThreads = 256;
+constexpr int kLdS = kPage + 4, kLdP = kPage + 8;
+template <int MT, int KS, int NT>
 __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const LatentParams p) {
   extern __shared__ __align__(16) uint8_t lm_smem[];
   constexpr int RT = 16 * MT;
-  constexpr int kLdS = kPage + 4, kLdP = kPage + 8;
   const int ld = p.W + 8;
   __nv_bfloat16* sKV = reinterpret_cast<__nv_bfloat16*>(lm_smem);           // [2][64][ld]
-  __nv_bfloat16* sQ = sKV + 2 * kPage * ld;                                  // [RT][ld]
-  __nv_bfloat16* sP = sQ + RT * ld;                                          // [RT][kLdP]
-  float* sS = reinterpret_cast<float*>(sP + RT * kLdP);                      // [32][kLdS]
-  float* sCorr = sS + 32 * kLdS;                                             // [RT]
+  __nv_bfloat16* sQ = sKV + kPage * ld;                                      // [RT][ld], before the second page is loaded
+  __nv_bfloat16* sP = sKV + 2 * kPage * ld;                                  // [RT][kLdP]
+  float* sS = reinterpret_cast<float*>(sP + RT * kLdP);                      // [4][RT][kLdS]
+  float* sCorr = sS + 4 * RT * kLdS;                                         // [RT]
   const int seq = blockIdx.x / p.row_tiles, row0 = (blockIdx.x % p.row_tiles) * RT, split = blockIdx.y;
   const int len = p.q_lens[seq], n_rows = len * p.H;
   if (row0 >= n_rows) return;
@@ -241,8 +258,8 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     __nv_bfloat16* dst = sKV + buf * kPage * ld;
     const int valid = n_keys - b * kPage;
 #pragma unroll
-    for (int i = 0; i < kPage / 16; ++i) {
-      const int r = warp + 16 * i;
+    for (int i = 0; i < kPage / 8; ++i) {
+      const int r = warp + 8 * i;
       for (int c = lane; c < chunks; c += 32)
         ms_cp16(ms_addr(dst + r * ld + c * 8), src + static_cast<long long>(r) * p.W + c * 8, r < valid);
     }
@@ -251,14 +268,25 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
   {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + base_row * p.W;
 #pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const int r = warp + 16 * i;
+    for (int i = 0; i < RT / 8; ++i) {
+      const int r = warp + 8 * i;
       const bool ok = row0 + r < n_rows;
       for (int c = lane; c < chunks; c += 32)
         ms_cp16(ms_addr(sQ + r * ld + c * 8), q + static_cast<long long>(ok ? r : 0) * p.W + c * 8, ok);
     }
+    ms_commit();
   }
   load_page(b0, 0);
+  const int kg = warp & 1, slice = warp >> 1;
+  const int steps = p.W / 16, per_slice = (steps + 3) / 4, s0 = slice * per_slice, n_steps = max(0, min(per_slice, steps - s0));
+  uint32_t qf[MT][KS][4];
+  ms_wait<1>();
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < KS; ++k)
+    if (k < n_steps)
+#pragma unroll
+      for (int i = 0; i < MT; ++i) ms_ldsm4(ms_a_at(ms_addr(sQ), ld, i * 16, (s0 + k) * 16, lane), qf[i][k]);
   float acc[MT][NT][4];
 #pragma unroll
   for (int i = 0; i < MT; ++i)
@@ -266,17 +294,13 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
-  // softmax rows of this warp: MT consecutive rows
-  float m_run[MT], l_run[MT];
+  constexpr int kRows = RT / 8;                  // softmax rows of this warp
+  float m_run[kRows], l_run[kRows];
 #pragma unroll
-  for (int i = 0; i < MT; ++i) { m_run[i] = -CUDART_INF_F; l_run[i] = 0.f; }
-  const uint32_t aQ = ms_addr(sQ), aP = ms_addr(sP);
+  for (int i = 0; i < kRows; ++i) { m_run[i] = -CUDART_INF_F; l_run[i] = 0.f; }
+  const uint32_t aP = ms_addr(sP);
   const int n8 = (p.rank + 7) / 8;
-  // scores: warp w owns keys 8 (w % 8) .. + 7 of the page, and with w / 8 one of two row tiles (MT = 2) or one half of
-  // the columns, whose products the softmax adds (MT = 1)
-  const int kt = warp & 7, half = warp >> 3;
-  const int steps = p.W / 16, k0 = MT == 2 ? 0 : half * (steps / 2) * 16, k1 = MT == 2 || half == 1 ? p.W : (steps / 2) * 16;
-  const int q_row = MT == 2 ? half * 16 : 0;
+  __syncthreads();                               // the query tile may be overwritten
 
   for (int b = b0; b < b1; ++b) {
     const int buf = (b - b0) & 1;
@@ -288,50 +312,62 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     }
     __syncthreads();
     const uint32_t aK = ms_addr(sKV + buf * kPage * ld);
-    float s[2][4];
+    float s[MT][4][4];
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
+    for (int i = 0; i < MT; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[i][e] = 0.f;
-    const uint32_t k_at = aK + static_cast<uint32_t>(((kt * 8 + (lane & 7)) * ld + (lane >> 3) * 8) * 2);
-    int k = k0;
-#pragma unroll 2
-    for (; k + 32 <= k1; k += 32) {          // two steps with independent sums
-      uint32_t fb[4], fa0[4], fa1[4];
-      ms_ldsm4(k_at + k * 2, fb);
-      ms_ldsm4(ms_a_at(aQ, ld, q_row, k, lane), fa0);
-      ms_ldsm4(ms_a_at(aQ, ld, q_row, k + 16, lane), fa1);
-      ms_mma(s[0], fa0, fb[0], fb[1]);
-      ms_mma(s[1], fa1, fb[2], fb[3]);
-    }
-    if (k < k1) {
-      uint32_t fb0, fb1, fa[4];
-      ms_ldsm2(aK + static_cast<uint32_t>(((kt * 8 + (lane & 7)) * ld + k + ((lane >> 3) & 1) * 8) * 2), fb0, fb1);
-      ms_ldsm4(ms_a_at(aQ, ld, q_row, k, lane), fa);
-      ms_mma(s[0], fa, fb0, fb1);
-    }
+      for (int j = 0; j < 4; ++j)
 #pragma unroll
-    for (int hf = 0; hf < 2; ++hf)           // MT = 1: the two halves lie in rows 0 .. 15 and 16 .. 31
-      *reinterpret_cast<float2*>(sS + (half * 16 + g4 + 8 * hf) * kLdS + kt * 8 + 2 * t4) =
-          make_float2(s[0][2 * hf] + s[1][2 * hf], s[0][2 * hf + 1] + s[1][2 * hf + 1]);
+        for (int e = 0; e < 4; ++e) s[i][j][e] = 0.f;
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+      if (k < n_steps) {
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+          uint32_t fb[4];
+          ms_ldsm4(ms_b_nt_at(aK, ld, kg * 32 + np * 16, (s0 + k) * 16, lane), fb);
+#pragma unroll
+          for (int i = 0; i < MT; ++i) {
+            ms_mma(s[i][2 * np], qf[i][k], fb[0], fb[1]);
+            ms_mma(s[i][2 * np + 1], qf[i][k], fb[2], fb[3]);
+          }
+        }
+      }
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf)
+          *reinterpret_cast<float2*>(sS + (slice * RT + i * 16 + g4 + 8 * hf) * kLdS + kg * 32 + j * 8 + 2 * t4) =
+              make_float2(s[i][j][2 * hf], s[i][j][2 * hf + 1]);
     __syncthreads();
+    float x[kRows][2], mx[kRows];
 #pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const int r = warp * MT + i, lim = prior + (row0 + r) / p.H;           // last key this row sees
-      float2 v = *reinterpret_cast<const float2*>(sS + r * kLdS + 2 * lane);
-      if (MT == 1) {
-        const float2 w = *reinterpret_cast<const float2*>(sS + (16 + r) * kLdS + 2 * lane);
+    for (int i = 0; i < kRows; ++i) {
+      const int r = warp * kRows + i, lim = prior + (row0 + r) / p.H;        // last key this row sees
+      float2 v = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float2 w = *reinterpret_cast<const float2*>(sS + (q * RT + r) * kLdS + 2 * lane);
         v.x += w.x;
         v.y += w.y;
       }
       const int j = b * kPage + 2 * lane;
-      const float x0 = j <= lim ? v.x * p.scale_log2 : -CUDART_INF_F, x1 = j + 1 <= lim ? v.y * p.scale_log2 : -CUDART_INF_F;
-      float mx = fmaxf(x0, x1);
+      x[i][0] = j <= lim ? v.x * p.scale_log2 : -CUDART_INF_F;
+      x[i][1] = j + 1 <= lim ? v.y * p.scale_log2 : -CUDART_INF_F;
+      mx[i] = fmaxf(x[i][0], x[i][1]);
+    }
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float m_new = fmaxf(m_run[i], mx), m_use = m_new == -CUDART_INF_F ? 0.f : m_new;
-      const float corr = exp2f(m_run[i] - m_use), e0 = exp2f(x0 - m_use), e1 = exp2f(x1 - m_use);
-      l_run[i] = l_run[i] * corr + e0 + e1;  // this lane's keys; the lanes meet at the end
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int i = 0; i < kRows; ++i) mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], o));
+#pragma unroll
+    for (int i = 0; i < kRows; ++i) {
+      const int r = warp * kRows + i;
+      const float m_new = fmaxf(m_run[i], mx[i]), m_use = m_new == -CUDART_INF_F ? 0.f : m_new;
+      const float corr = exp2f(m_run[i] - m_use), e0 = exp2f(x[i][0] - m_use), e1 = exp2f(x[i][1] - m_use);
+      l_run[i] = l_run[i] * corr + e0 + e1;      // this lane's keys; the lanes meet at the end
       m_run[i] = m_new;
       *reinterpret_cast<uint32_t*>(sP + r * kLdP + 2 * lane) = pack_bf16(e0, e1);
       if (lane == 0) sCorr[r] = corr;
@@ -353,7 +389,7 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
       for (int i = 0; i < MT; ++i) ms_ldsm4(ms_a_at(aP, kLdP, i * 16, kk, lane), fp[i]);
 #pragma unroll
       for (int j = 0; j < NT; ++j) {
-        const int tile = warp + 16 * j;
+        const int tile = warp + 8 * j;
         if (tile < n8) {
           uint32_t fb0, fb1;
           ms_ldsm2_t(aK + static_cast<uint32_t>(((kk + (lane & 15)) * ld + tile * 8) * 2), fb0, fb1);
@@ -365,8 +401,8 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     __syncthreads();                  // the page buffer, scores and probabilities may be overwritten
   }
 #pragma unroll
-  for (int i = 0; i < MT; ++i) {
-    const int r = warp * MT + i;
+  for (int i = 0; i < kRows; ++i) {
+    const int r = warp * kRows + i;
     const float l = warp_sum(l_run[i]);
     if (lane == 0 && row0 + r < n_rows) {
       p.part_ml[(part_base + r) * 2] = m_run[i];
@@ -379,7 +415,7 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
-        const int r = i * 16 + g4 + 8 * hf, c = (warp + 16 * j) * 8 + 2 * t4;
+        const int r = i * 16 + g4 + 8 * hf, c = (warp + 8 * j) * 8 + 2 * t4;
         if (row0 + r >= n_rows || c >= p.rank) continue;
         float* dst = p.part_o + (part_base + r) * p.rank + c;
         if (p.rank % 2 == 0) {
@@ -425,13 +461,11 @@ __global__ void __launch_bounds__(256) latent_up_kernel(const float* __restrict_
     for (int e = 0; e < JV; ++e) v[e] = 0.f;
     if (t < n_tok) {
       const float* src = part_o + (static_cast<long long>(t0 + t) * H + h) * rank + c;
-#pragma unroll 4
-      for (int s = 0; s < n_split; ++s) {    // an empty split left its rows unwritten
+#pragma unroll 8
+      for (int s = 0; s < n_split; ++s) {    // an empty split left its rows unwritten: read those of the first one
         const float w = coef[t][s];
         float x[JV];
-#pragma unroll
-        for (int e = 0; e < JV; ++e) x[e] = 0.f;
-        if (w != 0.f) load_vec<JV>(src + s * part_rows * rank, x);
+        load_vec<JV>(src + (w != 0.f ? s : 0) * part_rows * rank, x);
 #pragma unroll
         for (int e = 0; e < JV; ++e) v[e] = fmaf(w, x[e], v[e]);
       }
@@ -558,23 +592,23 @@ __global__ void latent_take_kernel(const __nv_bfloat16* __restrict__ o128, int n
 
 static size_t latent_mma_smem(int mt, int W) {
   const size_t rt = 16 * mt, ld = W + 8;
-  return (2 * kPage * ld + rt * ld + rt * (kPage + 8)) * 2 + (32 * (kPage + 4) + rt) * 4;
+  return (2 * kPage * ld + rt * kLdP) * 2 + (4 * rt * kLdS + rt) * 4;
 }
 static int latent_mma_tiles(int H, int W) {      // 16-row tiles per CTA, 0: not covered
   if (H > 16 && latent_mma_smem(2, W) <= 220 * 1024) return 2;
   return latent_mma_smem(1, W) <= 220 * 1024 ? 1 : 0;
 }
 
-template <int MT, int NT>
+template <int MT, int KS, int NT>
 static int latent_mma_launch(const LatentParams& p, dim3 grid, size_t smem, cudaStream_t st) {
   static DeviceMax configured;
   if (smem > configured.get()) {
-    const cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    const cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, KS, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured.set(smem);
   }
-  latent_attn_mma_kernel<MT, NT><<<grid, kMmaThreads, smem, st>>>(p);
+  latent_attn_mma_kernel<MT, KS, NT><<<grid, kMmaThreads, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -583,8 +617,8 @@ static int latent_absorb_launch(const void* qd, long long ld, const void* wuk, i
                                 const int* rows, int n, int tiles, size_t smem, void* out, cudaStream_t st) {
   const dim3 grid((rank + 127) / 128 + 1, H, tiles);
   const T *q = static_cast<const T*>(qd), *w = static_cast<const T*>(wuk);
-  if (rank % 2 == 0) latent_absorb_kernel<T, 2><<<grid, 64, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out));
-  else latent_absorb_kernel<T, 1><<<grid, 128, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out));
+  if (rank % 2 == 0) latent_absorb_kernel<T, 2><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out));
+  else latent_absorb_kernel<T, 1><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out));
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -624,7 +658,7 @@ extern "C" int pm_latent_prep(void* qd, int f32, long long ld, const float* norm
 
 // Whether the tensor-core kernel covers H heads over rows of W columns with `rank` value columns.
 extern "C" int pm_latent_mma_supported(int H, int W, int rank) {
-  return W % 16 == 0 && rank <= 512 && latent_mma_tiles(H, W) > 0;
+  return W % 16 == 0 && W <= 640 && rank <= 512 && latent_mma_tiles(H, W) > 0;
 }
 
 // Attention of short portions in the latent space. qd as pm_latent_prep leaves it, wuk [H * dn, rank], wuv [H * dv, rank],
@@ -642,7 +676,7 @@ extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void*
   if (n_seq < 1 || max_q < 1 || n_tok < 1) return 0;
   const bool mma = !f32 && pm_latent_mma_supported(H, W, rank);
   if (!mma && n_split != 1) return -2;
-  const size_t sm_abs = static_cast<size_t>(kAbsTok) * dn * 4, sm_row = (static_cast<size_t>(W) + rank + kPage) * 4,
+  const size_t sm_abs = static_cast<size_t>(kAbsTok) * (dn + 512) * 4, sm_row = (static_cast<size_t>(W) + rank + kPage) * 4,
                sm_up = static_cast<size_t>(kUpTok) * rank * 4;
   if (sm_abs > 48 * 1024 || (!mma && sm_row > 48 * 1024) || sm_up > 46 * 1024) return -3;
   const int abs_tiles = (n_tok + kAbsTok - 1) / kAbsTok, up_tiles = (n_tok + kUpTok - 1) / kUpTok;
@@ -656,16 +690,18 @@ extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void*
   p.rows = static_cast<long long>(n_tok) * H;
   p.scale_log2 = scale * 1.4426950408889634f;
   if (mma) {
-    const int mt = latent_mma_tiles(H, W), rt = 16 * mt, nt = (rank + 127) / 128;
+    const int mt = latent_mma_tiles(H, W), rt = 16 * mt;
     p.row_tiles = (max_q * H + rt - 1) / rt;
     const dim3 grid(p.row_tiles * n_seq, n_split);
     const size_t smem = latent_mma_smem(mt, W);
+    // (steps per quarter, column tiles per warp): the smallest instance that holds both
+    const int size = W <= 128 && rank <= 128 ? 0 : (W <= 320 && rank <= 256 ? 1 : 2);
     if (mt == 1)
-      rc = nt <= 1 ? latent_mma_launch<1, 1>(p, grid, smem, st) : nt <= 2 ? latent_mma_launch<1, 2>(p, grid, smem, st)
-                                                                          : latent_mma_launch<1, 4>(p, grid, smem, st);
+      rc = size == 0 ? latent_mma_launch<1, 2, 2>(p, grid, smem, st) : size == 1 ? latent_mma_launch<1, 5, 4>(p, grid, smem, st)
+                                                                                 : latent_mma_launch<1, 10, 8>(p, grid, smem, st);
     else
-      rc = nt <= 1 ? latent_mma_launch<2, 1>(p, grid, smem, st) : nt <= 2 ? latent_mma_launch<2, 2>(p, grid, smem, st)
-                                                                          : latent_mma_launch<2, 4>(p, grid, smem, st);
+      rc = size == 0 ? latent_mma_launch<2, 2, 2>(p, grid, smem, st) : size == 1 ? latent_mma_launch<2, 5, 4>(p, grid, smem, st)
+                                                                                 : latent_mma_launch<2, 10, 8>(p, grid, smem, st);
     if (rc) return rc;
   } else {
     const dim3 grid(max_q * H, n_seq);

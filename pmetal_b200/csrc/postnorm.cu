@@ -151,12 +151,13 @@ static int postnorm_launch(const float* x, const void* y, long long ldy, const f
 template <typename T>
 static int glu_launch(const void* gu, long long ld, const float* bias, int n, int ff, float limit, float beta, float shift,
                       void* out, cudaStream_t st) {
-  const bool vec = ff % 4 == 0 && ld % 4 == 0;
-  const long long n_vec = static_cast<long long>(n) * (vec ? ff / 4 : ff);
+  const int v = ff % 8 == 0 && ld % 8 == 0 ? 8 : (ff % 4 == 0 && ld % 4 == 0 ? 4 : 1);
+  const long long n_vec = static_cast<long long>(n) * (ff / v);
   long long grid = (n_vec + 255) / 256;
   if (grid > num_sms() * 16) grid = num_sms() * 16;
   const T* src = static_cast<const T*>(gu);
-  if (vec) clamped_glu_kernel<T, 4><<<static_cast<int>(grid), 256, 0, st>>>(src, ld, bias, ff, limit, beta, shift, static_cast<T*>(out), n_vec);
+  if (v == 8) clamped_glu_kernel<T, 8><<<static_cast<int>(grid), 256, 0, st>>>(src, ld, bias, ff, limit, beta, shift, static_cast<T*>(out), n_vec);
+  else if (v == 4) clamped_glu_kernel<T, 4><<<static_cast<int>(grid), 256, 0, st>>>(src, ld, bias, ff, limit, beta, shift, static_cast<T*>(out), n_vec);
   else clamped_glu_kernel<T, 1><<<static_cast<int>(grid), 256, 0, st>>>(src, ld, bias, ff, limit, beta, shift, static_cast<T*>(out), n_vec);
   return static_cast<int>(cudaGetLastError());
 }

@@ -24,6 +24,7 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
+#include <type_traits>
 #include "elem.cuh"
 #include "host_util.cuh"
 #include "mma_sync.cuh"
@@ -99,6 +100,7 @@ __global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const ScanParams
   for (int t = 0; t < len; ++t) {
     const int pos = start + t;
     const T* row = p.u + static_cast<long long>(q0 + t) * p.ldu;
+    const int turn = pos % d.taps;
     __syncthreads();                          // the previous token's readers are done
     for (int i = threadIdx.x; i < p.pw + 2 * d.N; i += kScanThreads) {
       int c;
@@ -117,7 +119,7 @@ __global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const ScanParams
             const int j = j0 + k, back = d.taps - 1 - j, src = pos - back;
             const bool ok = j < d.taps && src >= 0;
             const T* at = t >= back ? row + d.inner + c - static_cast<long long>(back) * p.ldu
-                                    : p.ring + (slot * d.taps + (ok ? src % d.taps : 0)) * d.conv + c;
+                                    : p.ring + (slot * d.taps + (back > turn ? turn - back + d.taps : turn - back)) * d.conv + c;
             w[k] = ok ? p.conv_w[static_cast<long long>(j) * d.conv + c] : 0.f;
             in[k] = ok ? to_f(*at) : 0.f;
           }
@@ -222,11 +224,28 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const ConvParams p) {
     float w[TAPS > 0 ? TAPS : 1][V];
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) load_vec<V>(p.conv_w + static_cast<long long>(j) * d.conv + c, w[j]);
+    // all rows are requested before the first is used
+    using Raw = typename std::conditional<V == 4, uint2, __nv_bfloat16>::type;
+    Raw raw[kConvTokens + TAPS];
+    bool have[kConvTokens + TAPS];
+    const int turn = (start + t0 + d.taps) % d.taps;       // ring row of position start + t0
 #pragma unroll
     for (int r = 1 - TAPS; r < kConvTokens; ++r) {
-      if (r >= n_tok) break;
+      const int back = -r;                                 // only positions before this portion lie in the ring
+      const __nv_bfloat16* at = t0 + r >= 0 ? p.u + static_cast<long long>(q0 + t0 + r) * p.ldu + d.inner + c
+                                            : p.ring + (slot * d.taps + (back > turn ? turn - back + d.taps : turn - back)) * d.conv + c;
+      have[r + TAPS - 1] = r < n_tok && start + t0 + r >= 0;
+      if (have[r + TAPS - 1]) raw[r + TAPS - 1] = *reinterpret_cast<const Raw*>(at);
+    }
+#pragma unroll
+    for (int r = 1 - TAPS; r < kConvTokens; ++r) {
       float in[V];
-      input(r, in);
+      if (have[r + TAPS - 1]) {
+        load_vec<V>(reinterpret_cast<const __nv_bfloat16*>(&raw[r + TAPS - 1]), in);
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) in[e] = 0.f;
+      }
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) {
         const int t = r + TAPS - 1 - j;                    // row r is tap j of token t
