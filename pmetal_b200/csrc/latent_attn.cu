@@ -23,6 +23,7 @@
 #include "elem.cuh"
 #include "host_util.cuh"
 #include "mma_sync.cuh"
+#include "pdl.cuh"
 #include "pmetal_b200.h"
 
 namespace pm {
@@ -91,12 +92,17 @@ constexpr int kAbsTok = 8;
 template <typename T, int V>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict__ qd, long long ld, const T* __restrict__ wuk,
                                                             int H, int dn, int dr, int rank, int W, const int* __restrict__ rows,
-                                                            int n, T* __restrict__ out) {
+                                                            int n, T* __restrict__ out, const T* __restrict__ wuv,
+                                                            unsigned wuv_bytes) {
   extern __shared__ __align__(16) float abs_q[];           // [dn][kAbsTok], then [groups][kAbsTok][128]
   constexpr int kCols = 128 / V, kGroups = 256 / kCols;
   const int h = blockIdx.y, t0 = blockIdx.z * kAbsTok, n_tok = min(kAbsTok, n - t0);
   if (blockIdx.x == gridDim.x - 1) {
     const int tail = W - rank;
+    if (blockIdx.z == 0 && wuv_bytes) {                    // latent_up_kernel will want this head's value weights in L2
+      const char* v = reinterpret_cast<const char*>(wuv) + static_cast<size_t>(h) * wuv_bytes;
+      for (unsigned o = threadIdx.x * 4096u; o < wuv_bytes; o += blockDim.x * 4096u) l2_prefetch_bulk(v + o, min(4096u, wuv_bytes - o));
+    }
     for (int i = threadIdx.x; i < n_tok * tail; i += blockDim.x) {
       const int t = i / tail, j = i - t * tail;
       put(out + (static_cast<long long>(t0 + t) * H + h) * W + rank + j,
@@ -220,7 +226,7 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const LatentParams
 // latent per warp. Warp w scores keys 32 (w % 2) .. + 31 of a page over column quarter w / 2, with the quarter's query
 // fragments in registers for all pages; the softmax adds the four partial scores; for P V warp w owns columns 8 (w + 8 j).
 constexpr int kMmaThreads = 256;
-constexpr int kLdS = kPage + 4, kLdP = kPage + 8;
+constexpr int kLdS = kPage + 8, kLdP = kPage + 8;
 template <int MT, int KS, int NT>
 __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const LatentParams p) {
   extern __shared__ __align__(16) uint8_t lm_smem[];
@@ -474,31 +480,42 @@ __global__ void __launch_bounds__(256) latent_up_kernel(const float* __restrict_
   }
   __syncthreads();
   const int per = (dv + gridDim.z - 1) / gridDim.z, r1 = min(dv, (static_cast<int>(blockIdx.z) + 1) * per);
-  for (int r = blockIdx.z * per + warp; r < r1; r += 8) {
+  for (int r = blockIdx.z * per + warp; r < r1; r += 16) {         // rows r and r + 8
+    const bool two = r + 8 < r1;
     const T* w = wuv + (static_cast<long long>(h) * dv + r) * rank;
-    float acc[kUpTok];
+    const T* w2 = two ? w + 8ll * rank : w;
+    float acc[2][kUpTok];
 #pragma unroll
-    for (int t = 0; t < kUpTok; ++t) acc[t] = 0.f;
+    for (int t = 0; t < kUpTok; ++t) acc[0][t] = acc[1][t] = 0.f;
 #pragma unroll 2
     for (int c = lane * V; c < rank; c += 32 * V) {
-      float wv[V];
+      float wv[V], wv2[V];
       load_vec<V>(w + c, wv);
+      load_vec<V>(w2 + c, wv2);
 #pragma unroll
       for (int t = 0; t < kUpTok; ++t) {
         float x[V];
         load_vec<V>(up_o + t * rank + c, x);
 #pragma unroll
-        for (int e = 0; e < V; ++e) acc[t] = fmaf(wv[e], x[e], acc[t]);
+        for (int e = 0; e < V; ++e) {
+          acc[0][t] = fmaf(wv[e], x[e], acc[0][t]);
+          acc[1][t] = fmaf(wv2[e], x[e], acc[1][t]);
+        }
       }
     }
 #pragma unroll
-    for (int t = 0; t < kUpTok; ++t) acc[t] = warp_sum(acc[t]);
-    if (lane < n_tok) {
-      float v = acc[0];
+    for (int k = 0; k < 2; ++k)
 #pragma unroll
-      for (int t = 1; t < kUpTok; ++t)
-        if (lane == t) v = acc[t];
-      put(out + rows[t0 + lane] * ldo + h * dv + r, v);
+      for (int t = 0; t < kUpTok; ++t) acc[k][t] = warp_sum(acc[k][t]);
+    const int t = lane & (kUpTok - 1), k = lane / kUpTok;          // lane (k, t) writes row r + 8 k of token t
+    if (t < n_tok && (k == 0 || (k == 1 && two))) {
+      float v = 0.f;
+#pragma unroll
+      for (int kk = 0; kk < 2; ++kk)
+#pragma unroll
+        for (int tt = 0; tt < kUpTok; ++tt)
+          if (k == kk && t == tt) v = acc[kk][tt];
+      put(out + rows[t0 + t] * ldo + h * dv + r + 8 * k, v);
     }
   }
 }
@@ -614,11 +631,15 @@ static int latent_mma_launch(const LatentParams& p, dim3 grid, size_t smem, cuda
 
 template <typename T>
 static int latent_absorb_launch(const void* qd, long long ld, const void* wuk, int H, int dn, int dr, int rank, int W,
-                                const int* rows, int n, int tiles, size_t smem, void* out, cudaStream_t st) {
+                                const int* rows, int n, int tiles, size_t smem, void* out, const void* wuv, int dv,
+                                cudaStream_t st) {
   const dim3 grid((rank + 127) / 128 + 1, H, tiles);
-  const T *q = static_cast<const T*>(qd), *w = static_cast<const T*>(wuk);
-  if (rank % 2 == 0) latent_absorb_kernel<T, 2><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out));
-  else latent_absorb_kernel<T, 1><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out));
+  const T *q = static_cast<const T*>(qd), *w = static_cast<const T*>(wuk), *v = static_cast<const T*>(wuv);
+  // bulk prefetches take whole 16-byte pieces
+  const size_t head = static_cast<size_t>(dv) * rank * sizeof(T);
+  const unsigned bytes = head % 16 == 0 && !(reinterpret_cast<uintptr_t>(v) & 15) ? static_cast<unsigned>(head) : 0;
+  if (rank % 2 == 0) latent_absorb_kernel<T, 2><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out), v, bytes);
+  else latent_absorb_kernel<T, 1><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out), v, bytes);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -681,8 +702,8 @@ extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void*
   if (sm_abs > 48 * 1024 || (!mma && sm_row > 48 * 1024) || sm_up > 46 * 1024) return -3;
   const int abs_tiles = (n_tok + kAbsTok - 1) / kAbsTok, up_tiles = (n_tok + kUpTok - 1) / kUpTok;
   if (abs_tiles > 65535 || up_tiles > 65535) return -4;
-  int rc = f32 ? latent_absorb_launch<float>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, st)
-               : latent_absorb_launch<__nv_bfloat16>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, st);
+  int rc = f32 ? latent_absorb_launch<float>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, wuv, dv, st)
+               : latent_absorb_launch<__nv_bfloat16>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, wuv, dv, st);
   if (rc) return rc;
   LatentParams p{};
   p.q = q_lat; p.cache = cache; p.block_table = block_table; p.seq_lens = seq_lens; p.c_start = c_start; p.q_lens = q_lens;

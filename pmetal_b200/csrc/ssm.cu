@@ -71,7 +71,7 @@ constexpr int kScanThreads = 256;
 
 // E: state rows per thread (float4 each).
 template <typename T, int E>
-__global__ void __launch_bounds__(kScanThreads) ssm_scan_kernel(const ScanParams<T> p) {
+__global__ void __launch_bounds__(kScanThreads, E <= 8 ? 4 : 2) ssm_scan_kernel(const ScanParams<T> p) {
   extern __shared__ __align__(16) float scan_smem[];
   const SsmDims& d = p.d;
   const int seq = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * p.pw;
