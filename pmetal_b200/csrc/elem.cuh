@@ -92,12 +92,16 @@ __device__ __forceinline__ float block_sum(float v) {
 
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
+// The same through the fast exponential and division, for results that are rounded to bf16.
+__device__ __forceinline__ float sigmoid_fast(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+__device__ __forceinline__ float silu_fast(float v) { return v * sigmoid_fast(v); }
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
+template <bool kFast = false>
 __device__ __forceinline__ float clamped_glu(float g, float u, float limit, float beta, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return g * sigmoid_f(beta * g) * (u + shift);
+  return g * (kFast ? sigmoid_fast(beta * g) : sigmoid_f(beta * g)) * (u + shift);
 }
 
 }  // namespace pm

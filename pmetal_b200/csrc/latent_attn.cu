@@ -222,10 +222,11 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const LatentParams
   }
 }
 
-// 8 warps. MT: 16-row tiles of (token, head) rows; KS: 16-column steps of a quarter of the row; NT: 8-column tiles of the
-// latent per warp. Warp w scores keys 32 (w % 2) .. + 31 of a page over column quarter w / 2, with the quarter's query
-// fragments in registers for all pages; the softmax adds the four partial scores; for P V warp w owns columns 8 (w + 8 j).
-constexpr int kMmaThreads = 256;
+// 16 warps. MT: 16-row tiles of (token, head) rows; KS: 16-column steps of a quarter of the row; NT: 8-column tiles of the
+// latent per warp. For the scores a warp owns one row tile, one column quarter (its query fragments stay in registers for all
+// pages) and 32 (MT = 2) or 16 (MT = 1) keys of a page; the softmax adds the four partial scores of a key. For P V warp w
+// owns columns 8 (w + 16 j).
+constexpr int kMmaThreads = 512;
 constexpr int kLdS = kPage + 8, kLdP = kPage + 8;
 template <int MT, int KS, int NT>
 __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const LatentParams p) {
@@ -264,8 +265,8 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     __nv_bfloat16* dst = sKV + buf * kPage * ld;
     const int valid = n_keys - b * kPage;
 #pragma unroll
-    for (int i = 0; i < kPage / 8; ++i) {
-      const int r = warp + 8 * i;
+    for (int i = 0; i < kPage / 16; ++i) {
+      const int r = warp + 16 * i;
       for (int c = lane; c < chunks; c += 32)
         ms_cp16(ms_addr(dst + r * ld + c * 8), src + static_cast<long long>(r) * p.W + c * 8, r < valid);
     }
@@ -274,8 +275,8 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
   {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + base_row * p.W;
 #pragma unroll
-    for (int i = 0; i < RT / 8; ++i) {
-      const int r = warp + 8 * i;
+    for (int i = 0; i < MT; ++i) {
+      const int r = warp + 16 * i;
       const bool ok = row0 + r < n_rows;
       for (int c = lane; c < chunks; c += 32)
         ms_cp16(ms_addr(sQ + r * ld + c * 8), q + static_cast<long long>(ok ? r : 0) * p.W + c * 8, ok);
@@ -283,16 +284,15 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     ms_commit();
   }
   load_page(b0, 0);
-  const int kg = warp & 1, slice = warp >> 1;
+  constexpr int kGroups = 4 / MT, kTiles = 2 * MT;         // groups of keys and 8-key tiles per group
+  const int kg = warp & (kGroups - 1), slice = (warp / kGroups) & 3, row_tile = warp / (4 * kGroups);
   const int steps = p.W / 16, per_slice = (steps + 3) / 4, s0 = slice * per_slice, n_steps = max(0, min(per_slice, steps - s0));
-  uint32_t qf[MT][KS][4];
+  uint32_t qf[KS][4];
   ms_wait<1>();
   __syncthreads();
 #pragma unroll
   for (int k = 0; k < KS; ++k)
-    if (k < n_steps)
-#pragma unroll
-      for (int i = 0; i < MT; ++i) ms_ldsm4(ms_a_at(ms_addr(sQ), ld, i * 16, (s0 + k) * 16, lane), qf[i][k]);
+    if (k < n_steps) ms_ldsm4(ms_a_at(ms_addr(sQ), ld, row_tile * 16, (s0 + k) * 16, lane), qf[k]);
   float acc[MT][NT][4];
 #pragma unroll
   for (int i = 0; i < MT; ++i)
@@ -300,7 +300,7 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
-  constexpr int kRows = RT / 8;                  // softmax rows of this warp
+  constexpr int kRows = MT;                      // softmax rows of this warp
   float m_run[kRows], l_run[kRows];
 #pragma unroll
   for (int i = 0; i < kRows; ++i) { m_run[i] = -CUDART_INF_F; l_run[i] = 0.f; }
@@ -318,35 +318,28 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     }
     __syncthreads();
     const uint32_t aK = ms_addr(sKV + buf * kPage * ld);
-    float s[MT][4][4];
+    float s[kTiles][4];
 #pragma unroll
-    for (int i = 0; i < MT; ++i)
+    for (int j = 0; j < kTiles; ++j)
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[i][j][e] = 0.f;
+      for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
 #pragma unroll
     for (int k = 0; k < KS; ++k)
       if (k < n_steps) {
 #pragma unroll
-        for (int np = 0; np < 2; ++np) {
+        for (int np = 0; np < MT; ++np) {
           uint32_t fb[4];
-          ms_ldsm4(ms_b_nt_at(aK, ld, kg * 32 + np * 16, (s0 + k) * 16, lane), fb);
-#pragma unroll
-          for (int i = 0; i < MT; ++i) {
-            ms_mma(s[i][2 * np], qf[i][k], fb[0], fb[1]);
-            ms_mma(s[i][2 * np + 1], qf[i][k], fb[2], fb[3]);
-          }
+          ms_ldsm4(ms_b_nt_at(aK, ld, (kg * MT + np) * 16, (s0 + k) * 16, lane), fb);
+          ms_mma(s[2 * np], qf[k], fb[0], fb[1]);
+          ms_mma(s[2 * np + 1], qf[k], fb[2], fb[3]);
         }
       }
 #pragma unroll
-    for (int i = 0; i < MT; ++i)
+    for (int j = 0; j < kTiles; ++j)
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-#pragma unroll
-        for (int hf = 0; hf < 2; ++hf)
-          *reinterpret_cast<float2*>(sS + (slice * RT + i * 16 + g4 + 8 * hf) * kLdS + kg * 32 + j * 8 + 2 * t4) =
-              make_float2(s[i][j][2 * hf], s[i][j][2 * hf + 1]);
+      for (int hf = 0; hf < 2; ++hf)
+        *reinterpret_cast<float2*>(sS + (slice * RT + row_tile * 16 + g4 + 8 * hf) * kLdS + kg * MT * 16 + j * 8 + 2 * t4) =
+            make_float2(s[j][2 * hf], s[j][2 * hf + 1]);
     __syncthreads();
     float x[kRows][2], mx[kRows];
 #pragma unroll
@@ -395,7 +388,7 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
       for (int i = 0; i < MT; ++i) ms_ldsm4(ms_a_at(aP, kLdP, i * 16, kk, lane), fp[i]);
 #pragma unroll
       for (int j = 0; j < NT; ++j) {
-        const int tile = warp + 8 * j;
+        const int tile = warp + 16 * j;
         if (tile < n8) {
           uint32_t fb0, fb1;
           ms_ldsm2_t(aK + static_cast<uint32_t>(((kk + (lane & 15)) * ld + tile * 8) * 2), fb0, fb1);
@@ -421,7 +414,7 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
-        const int r = i * 16 + g4 + 8 * hf, c = (warp + 8 * j) * 8 + 2 * t4;
+        const int r = i * 16 + g4 + 8 * hf, c = (warp + 16 * j) * 8 + 2 * t4;
         if (row0 + r >= n_rows || c >= p.rank) continue;
         float* dst = p.part_o + (part_base + r) * p.rank + c;
         if (p.rank % 2 == 0) {
@@ -718,11 +711,11 @@ extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void*
     // (steps per quarter, column tiles per warp): the smallest instance that holds both
     const int size = W <= 128 && rank <= 128 ? 0 : (W <= 320 && rank <= 256 ? 1 : 2);
     if (mt == 1)
-      rc = size == 0 ? latent_mma_launch<1, 2, 2>(p, grid, smem, st) : size == 1 ? latent_mma_launch<1, 5, 4>(p, grid, smem, st)
-                                                                                 : latent_mma_launch<1, 10, 8>(p, grid, smem, st);
+      rc = size == 0 ? latent_mma_launch<1, 2, 1>(p, grid, smem, st) : size == 1 ? latent_mma_launch<1, 5, 2>(p, grid, smem, st)
+                                                                                 : latent_mma_launch<1, 10, 4>(p, grid, smem, st);
     else
-      rc = size == 0 ? latent_mma_launch<2, 2, 2>(p, grid, smem, st) : size == 1 ? latent_mma_launch<2, 5, 4>(p, grid, smem, st)
-                                                                                 : latent_mma_launch<2, 10, 8>(p, grid, smem, st);
+      rc = size == 0 ? latent_mma_launch<2, 2, 1>(p, grid, smem, st) : size == 1 ? latent_mma_launch<2, 5, 2>(p, grid, smem, st)
+                                                                                 : latent_mma_launch<2, 10, 4>(p, grid, smem, st);
     if (rc) return rc;
   } else {
     const dim3 grid(max_q * H, n_seq);

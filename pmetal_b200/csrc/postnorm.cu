@@ -97,7 +97,7 @@ __global__ void clamped_glu_kernel(const T* __restrict__ gu, long long ld, const
       for (int e = 0; e < V; ++e) { g[e] += a[e]; u[e] += c[e]; }
     }
 #pragma unroll
-    for (int e = 0; e < V; ++e) g[e] = clamped_glu(g[e], u[e], limit, beta, shift);
+    for (int e = 0; e < V; ++e) g[e] = clamped_glu<sizeof(T) == 2>(g[e], u[e], limit, beta, shift);
     store_vec<V>(out + t * ff + k, g);
   }
 }

@@ -272,7 +272,7 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const ConvParams p) {
   for (int t = 0; t < kConvTokens; ++t) {
     if (t >= n_tok) break;
 #pragma unroll
-    for (int e = 0; e < V; ++e) acc[t][e] = silu_f(acc[t][e]);
+    for (int e = 0; e < V; ++e) acc[t][e] = silu_fast(acc[t][e]);
     store_vec<V>(p.act + static_cast<long long>(q0 + t0 + t) * d.conv + c, acc[t]);
   }
 }
@@ -716,7 +716,7 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_warp_kernel(const T* __rest
       load_vec<8>(u + t * ldu + c0 + k, z);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
-        v[i][e] *= silu_f(z[e]);
+        v[i][e] *= sizeof(T) == 2 ? silu_fast(z[e]) : silu_f(z[e]);
         ss = fmaf(v[i][e], v[i][e], ss);
       }
     }
