@@ -187,7 +187,7 @@ def kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096
             case(tag + "clamped gated unit", lambda: nat.clamped_glu(gu, ff, 7.0, 1.702, 1.0, bgu), 3 * T * ff * 2)
             case(tag + "  | swiglu", lambda: nat.swiglu_fwd(gu), 3 * T * ff * 2)
         # attention | paged attention of the dense decoder at 16 / 8 heads of 128
-        c2 = StateCache([CacheSpec(page_width=row)], n_seq * (prior + new) // BLOCK + n_seq + 1, n_seq, torch.bfloat16, "cuda")
+        c2 = StateCache([CacheSpec(page_width=row + 8)], n_seq * (prior + new) // BLOCK + n_seq + 1, n_seq, torch.bfloat16, "cuda")
         meta, grp = _group(c2, n_seq, prior, new)
         c2.pages[0].normal_()
         dims = (H, dn, dr, dv, r, row)

@@ -1,5 +1,5 @@
 // Multi-head latent attention over a paged cache. Per token and layer the cache holds one row [c: R | k_r: D_r | 0 ..]
-// (W = R + D_r rounded up to 16 columns): the normed latent and one rotated key part shared by all heads. With per-head
+// (W = R + D_r rounded up to 16 columns, rows W + 8 apart): the normed latent and one rotated key part shared by all heads. With per-head
 // up-projections W_uk (D_n x R) and W_uv (D_v x R), head h scores  (q_n . W_uk c + q_r . k_r) * scale  and reads out
 // W_uv (sum_j p_j c_j).
 //
@@ -20,6 +20,7 @@
 #include <cuda_runtime.h>
 #include <math_constants.h>
 #include <stdint.h>
+#include "common.cuh"
 #include "elem.cuh"
 #include "host_util.cuh"
 #include "mma_sync.cuh"
@@ -29,6 +30,7 @@
 namespace pm {
 
 constexpr int kPage = 64;
+constexpr int kRowPad = 8;            // cache rows are W + 8 apart: a page copied as one block has conflict-free rows in shared memory
 
 // One element, or two neighbours at an even offset.
 template <int V>
@@ -69,7 +71,7 @@ __global__ void latent_prep_kernel(T* __restrict__ qd, long long ld, const float
   }
   if (!own) return;
   const T* d = row + H * (dn + dr);
-  T* dst = cache + slots[t] * W;
+  T* dst = cache + slots[t] * (W + kRowPad);
   float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) {
     const float v = to_f(d[i]);
@@ -154,7 +156,7 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict_
 
 struct LatentParams {
   const void* q;             // [compact tokens, H, W]
-  const void* cache;         // [pages, 64, W]
+  const void* cache;         // [pages, 64, W + 8]
   const int* block_table;
   const int* seq_lens;
   const int* c_start;        // first row of each sequence in the compact buffers (q, part_o, part_ml)
@@ -164,6 +166,7 @@ struct LatentParams {
   int max_blocks, H, W, rank, n_split, row_tiles;
   long long rows;            // compact tokens * H
   float scale_log2;          // scale * log2(e)
+  int* status;               // set when a bounded wait runs out
 };
 
 // One (token, head) row per CTA, all keys, any type. grid (rows of the longest portion, sequences).
@@ -185,11 +188,11 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const LatentParams
   for (int j0 = 0; j0 < n_keys; j0 += kPage) {
     const int n = min(kPage, n_keys - j0);
     const T* page = static_cast<const T*>(p.cache) +
-                    static_cast<long long>(p.block_table[static_cast<long long>(seq) * p.max_blocks + j0 / kPage]) * kPage * p.W;
+                    static_cast<long long>(p.block_table[static_cast<long long>(seq) * p.max_blocks + j0 / kPage]) * kPage * (p.W + kRowPad);
     __syncthreads();
     for (int k = warp; k < n; k += 4) {
       float v = 0.f;
-      for (int i = lane; i < p.W; i += 32) v = fmaf(sq[i], to_f(page[static_cast<long long>(k) * p.W + i]), v);
+      for (int i = lane; i < p.W; i += 32) v = fmaf(sq[i], to_f(page[static_cast<long long>(k) * (p.W + kRowPad) + i]), v);
       v = warp_sum(v);
       if (lane == 0) ss[k] = v;
     }
@@ -211,7 +214,7 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const LatentParams
     for (int i = threadIdx.x; i < p.rank; i += 128) {
       float o = so[i] * corr;
 #pragma unroll 4
-      for (int k = 0; k < n; ++k) o = fmaf(ss[k], to_f(page[static_cast<long long>(k) * p.W + i]), o);
+      for (int k = 0; k < n; ++k) o = fmaf(ss[k], to_f(page[static_cast<long long>(k) * (p.W + kRowPad) + i]), o);
       so[i] = o;
     }
   }
@@ -232,12 +235,14 @@ template <int MT, int KS, int NT>
 __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const LatentParams p) {
   extern __shared__ __align__(16) uint8_t lm_smem[];
   constexpr int RT = 16 * MT;
-  const int ld = p.W + 8;
+  const int ld = p.W + kRowPad;
   __nv_bfloat16* sKV = reinterpret_cast<__nv_bfloat16*>(lm_smem);           // [2][64][ld]
   __nv_bfloat16* sQ = sKV + kPage * ld;                                      // [RT][ld], before the second page is loaded
   __nv_bfloat16* sP = sKV + 2 * kPage * ld;                                  // [RT][kLdP]
   float* sS = reinterpret_cast<float*>(sP + RT * kLdP);                      // [4][RT][kLdS]
   float* sCorr = sS + 4 * RT * kLdS;                                         // [RT]
+  __shared__ uint64_t full[2];                                               // a page has arrived in its buffer
+  __shared__ int abort_flag;
   const int seq = blockIdx.x / p.row_tiles, row0 = (blockIdx.x % p.row_tiles) * RT, split = blockIdx.y;
   const int len = p.q_lens[seq], n_rows = len * p.H;
   if (row0 >= n_rows) return;
@@ -260,18 +265,27 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
   const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.cache);
   const int* bt = p.block_table + static_cast<long long>(seq) * p.max_blocks;
   const int chunks = p.W / 8;
+  // One bulk copy brings the rows of a page that a query of the tile sees; the others are zeroed: what lies there may belong
+  // to anyone.
   auto load_page = [&](int b, int buf) {
-    const __nv_bfloat16* src = cache + static_cast<long long>(bt[b]) * kPage * p.W;
     __nv_bfloat16* dst = sKV + buf * kPage * ld;
-    const int valid = n_keys - b * kPage;
-#pragma unroll
-    for (int i = 0; i < kPage / 16; ++i) {
-      const int r = warp + 16 * i;
-      for (int c = lane; c < chunks; c += 32)
-        ms_cp16(ms_addr(dst + r * ld + c * 8), src + static_cast<long long>(r) * p.W + c * 8, r < valid);
+    const int valid = min(kPage, n_keys - b * kPage);
+    if (threadIdx.x == 0) {
+      const uint32_t bytes = static_cast<uint32_t>(valid * ld) * 2;
+      mbar_expect_tx(&full[buf], bytes);
+      ms_bulk_copy(ms_addr(dst), cache + static_cast<long long>(bt[b]) * kPage * ld, bytes, &full[buf]);
     }
-    ms_commit();
+    for (int i = valid * ld / 8 + threadIdx.x; i < kPage * ld / 8; i += kMmaThreads)
+      reinterpret_cast<uint4*>(dst)[i] = make_uint4(0u, 0u, 0u, 0u);
   };
+  if (threadIdx.x == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    abort_flag = 0;
+    mbar_init_fence();
+  }
+  __syncthreads();
+  load_page(b0, 0);
   {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + base_row * p.W;
 #pragma unroll
@@ -283,12 +297,11 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     }
     ms_commit();
   }
-  load_page(b0, 0);
   constexpr int kGroups = 4 / MT, kTiles = 2 * MT;         // groups of keys and 8-key tiles per group
   const int kg = warp & (kGroups - 1), slice = (warp / kGroups) & 3, row_tile = warp / (4 * kGroups);
   const int steps = p.W / 16, per_slice = (steps + 3) / 4, s0 = slice * per_slice, n_steps = max(0, min(per_slice, steps - s0));
   uint32_t qf[KS][4];
-  ms_wait<1>();
+  ms_wait<0>();
   __syncthreads();
 #pragma unroll
   for (int k = 0; k < KS; ++k)
@@ -306,17 +319,15 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
   for (int i = 0; i < kRows; ++i) { m_run[i] = -CUDART_INF_F; l_run[i] = 0.f; }
   const uint32_t aP = ms_addr(sP);
   const int n8 = (p.rank + 7) / 8;
-  __syncthreads();                               // the query tile may be overwritten
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  __syncthreads();                               // the query tile may be overwritten by a bulk copy
 
   for (int b = b0; b < b1; ++b) {
     const int buf = (b - b0) & 1;
-    if (b + 1 < b1) {
-      load_page(b + 1, buf ^ 1);
-      ms_wait<1>();
-    } else {
-      ms_wait<0>();
-    }
+    if (b + 1 < b1) load_page(b + 1, buf ^ 1);
+    if (!mbar_wait(&full[buf], ((b - b0) >> 1) & 1, &abort_flag, p.status, kTimeoutProducer)) abort_flag = 1;
     __syncthreads();
+    if (abort_flag) break;                       // every thread sees the same value here
     const uint32_t aK = ms_addr(sKV + buf * kPage * ld);
     float s[kTiles][4];
 #pragma unroll
@@ -387,17 +398,29 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
 #pragma unroll
       for (int i = 0; i < MT; ++i) ms_ldsm4(ms_a_at(aP, kLdP, i * 16, kk, lane), fp[i]);
 #pragma unroll
-      for (int j = 0; j < NT; ++j) {
-        const int tile = warp + 16 * j;
+      for (int j = 0; j < NT; j += 2) {      // column tiles j and j + 1 in one load where both exist
+        const int tile = warp + 16 * j, next = NT > 1 && tile + 16 < n8 ? tile + 16 : tile;
         if (tile < n8) {
-          uint32_t fb0, fb1;
-          ms_ldsm2_t(aK + static_cast<uint32_t>(((kk + (lane & 15)) * ld + tile * 8) * 2), fb0, fb1);
+          uint32_t fb[4];
+          ms_ldsm4_t(aK + static_cast<uint32_t>(((kk + (lane & 15)) * ld + (lane < 16 ? tile : next) * 8) * 2), fb);
 #pragma unroll
-          for (int i = 0; i < MT; ++i) ms_mma(acc[i][j], fp[i], fb0, fb1);
+          for (int i = 0; i < MT; ++i) {
+            ms_mma(acc[i][j], fp[i], fb[0], fb[1]);
+            if (NT > 1 && next != tile) ms_mma(acc[i][j + (NT > 1 ? 1 : 0)], fp[i], fb[2], fb[3]);
+          }
         }
       }
     }
     __syncthreads();                  // the page buffer, scores and probabilities may be overwritten
+  }
+  if (abort_flag) {                   // abandoned wait: the copies in flight get one more limit to land before the CTA leaves
+    __syncthreads();
+    if (threadIdx.x == 0) {
+      const unsigned long long t0 = globaltimer_ns();
+      while (globaltimer_ns() - t0 < kWaitLimitNs) {}
+    }
+    __syncthreads();
+    return;
   }
 #pragma unroll
   for (int i = 0; i < kRows; ++i) {
@@ -520,7 +543,7 @@ __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, co
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < static_cast<long long>(n) * r8;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
     const int j = static_cast<int>(i / r8), c = static_cast<int>(i - static_cast<long long>(j) * r8);
-    const __nv_bfloat16* src = cache + (static_cast<long long>(table[j / kPage]) * kPage + j % kPage) * W;
+    const __nv_bfloat16* src = cache + (static_cast<long long>(table[j / kPage]) * kPage + j % kPage) * (W + kRowPad);
     lat[i] = c < rank ? src[c] : __float2bfloat16(0.f);
   }
 }
@@ -530,7 +553,7 @@ __global__ void latent_gather8_kernel(const __nv_bfloat16* __restrict__ cache, c
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < static_cast<long long>(n) * per;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
     const int j = static_cast<int>(i / per), c = static_cast<int>(i - static_cast<long long>(j) * per) * 8;
-    const __nv_bfloat16* src = cache + (static_cast<long long>(table[j / kPage]) * kPage + j % kPage) * W;
+    const __nv_bfloat16* src = cache + (static_cast<long long>(table[j / kPage]) * kPage + j % kPage) * (W + kRowPad);
     *reinterpret_cast<uint4*>(lat + static_cast<long long>(j) * rank + c) = *reinterpret_cast<const uint4*>(src + c);
   }
 }
@@ -560,7 +583,7 @@ __global__ void latent_assemble_kernel(const __nv_bfloat16* __restrict__ qd, lon
       na = nb = dn + dr;
     } else if (what == 1) {
       a = kv + t * ldkv + h * dn;
-      b = cache + (static_cast<long long>(table[t / kPage]) * kPage + t % kPage) * W + rank;
+      b = cache + (static_cast<long long>(table[t / kPage]) * kPage + t % kPage) * (W + kRowPad) + rank;
       na = dn;
       nb = dn + dr;
     } else {
@@ -653,7 +676,7 @@ static int latent_up_launch(const float* part_o, const float* part_ml, const voi
 using namespace pm;
 
 // qd [n, ld]: the queries' rotated parts are turned in place; with cache != null the down-projection behind the queries is
-// normed / rotated and written to row slots[t] of cache [.., W]. cs / sn [n, dr / 2].
+// normed / rotated and written to row slots[t] of cache [.., W + 8]. cs / sn [n, dr / 2].
 extern "C" int pm_latent_prep(void* qd, int f32, long long ld, const float* norm_w, float eps, const float* cs,
                               const float* sn, int n, int H, int dn, int dr, int rank, void* cache, int W,
                               const long long* slots, cudaStream_t st) {
@@ -676,7 +699,7 @@ extern "C" int pm_latent_mma_supported(int H, int W, int rank) {
 }
 
 // Attention of short portions in the latent space. qd as pm_latent_prep leaves it, wuk [H * dn, rank], wuv [H * dv, rank],
-// cache [pages, 64, W]. The n_tok tokens of the listed sequences are counted through: sequence i covers compact tokens
+// cache [pages, 64, W + 8]. The n_tok tokens of the listed sequences are counted through: sequence i covers compact tokens
 // c_start[i] .. of the work buffers q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32 and part_ml [n_split,
 // n_tok * H, 2] fp32, and compact token j is row tok_rows[j] of qd and out. out [.., ldo]: H * dv columns. max_q: longest of
 // q_lens. n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
@@ -684,7 +707,7 @@ extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void*
                               const int* block_table, const int* seq_lens, const int* c_start, const int* q_lens,
                               const int* tok_rows, int n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr,
                               int dv, int rank, int W, int n_split, float scale, void* q_lat, float* part_o, float* part_ml,
-                              void* out, long long ldo, cudaStream_t st) {
+                              void* out, long long ldo, int* status, cudaStream_t st) {
   if (H < 1 || rank < 1 || W < rank + dr || dv < 1 || n_split < 1 || n_split > 64 || ldo < static_cast<long long>(H) * dv)
     return -1;
   if (n_seq < 1 || max_q < 1 || n_tok < 1) return 0;
@@ -703,6 +726,7 @@ extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void*
   p.part_o = part_o; p.part_ml = part_ml; p.max_blocks = max_blocks; p.H = H; p.W = W; p.rank = rank; p.n_split = n_split;
   p.rows = static_cast<long long>(n_tok) * H;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.status = status;
   if (mma) {
     const int mt = latent_mma_tiles(H, W), rt = 16 * mt;
     p.row_tiles = (max_q * H + rt - 1) / rt;

@@ -21,6 +21,13 @@ __device__ __forceinline__ void ms_wait() {
   asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
+// Bulk copy global -> shared of this CTA (16-byte aligned addresses, a multiple of 16 bytes); arrival is counted on `bar`.
+__device__ __forceinline__ void ms_bulk_copy(uint32_t dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src),
+               "r"(bytes), "r"(ms_addr(bar))
+               : "memory");
+}
+
 __device__ __forceinline__ void ms_ldsm4(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])

@@ -204,20 +204,20 @@ int pm_grouped_gemm_skinny(const void* x, int ldx, int rows, const void* w, int 
 
 // ---------------------------------------------------------------- latent_attn.cu
 // qd [n, ld]: the queries' rotated parts are turned in place; with cache != null the down-projection behind the queries is
-// normed / rotated and written to row slots[t] of cache [.., W]. cs / sn [n, dr / 2].
+// normed / rotated and written to row slots[t] of cache [.., W + 8]. cs / sn [n, dr / 2].
 int pm_latent_prep(void* qd, int f32, long long ld, const float* norm_w, float eps, const float* cs, const float*
     sn, int n, int H, int dn, int dr, int rank, void* cache, int W, const long long* slots, cudaStream_t st);
 // Whether the tensor-core kernel covers H heads over rows of W columns with `rank` value columns.
 int pm_latent_mma_supported(int H, int W, int rank);
 // Attention of short portions in the latent space. qd as pm_latent_prep leaves it, wuk [H * dn, rank], wuv [H * dv, rank],
-// cache [pages, 64, W]. The n_tok tokens of the listed sequences are counted through: sequence i covers compact tokens
+// cache [pages, 64, W + 8]. The n_tok tokens of the listed sequences are counted through: sequence i covers compact tokens
 // c_start[i] .. of the work buffers q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32 and part_ml [n_split,
 // n_tok * H, 2] fp32, and compact token j is row tok_rows[j] of qd and out. out [.., ldo]: H * dv columns. max_q: longest of
 // q_lens. n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
 int pm_latent_attn(const void* qd, int f32, long long ld, const void* wuk, const void* wuv, const void* cache,
     const int* block_table, const int* seq_lens, const int* c_start, const int* q_lens, const int* tok_rows, int
     n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr, int dv, int rank, int W, int n_split, float
-    scale, void* q_lat, float* part_o, float* part_ml, void* out, long long ldo, cudaStream_t st);
+    scale, void* q_lat, float* part_o, float* part_ml, void* out, long long ldo, int* status, cudaStream_t st);
 // lat [n, r8] bf16 = latents of positions 0 .. n - 1 of the sequence whose block table row is `table` (zero padded).
 int pm_latent_gather(const void* cache, const int* table, int n, int W, int rank, int r8, void* lat, cudaStream_t
     st);

@@ -179,7 +179,7 @@ class LatentAttentionMixer(nn.Module):
         self.expand = dtype == torch.bfloat16 and dn + dr <= 128 and dv <= 128
 
     def cache_spec(self) -> CacheSpec:
-        return CacheSpec(page_width=self.row if self.own else 0)
+        return CacheSpec(page_width=self.row + 8 if self.own else 0)      # the kernels keep rows eight columns apart
 
     def named_weights(self):
         q, d, k, v = self.n_q, self.n_d, self.n_k, self.n_v

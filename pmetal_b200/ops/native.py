@@ -1304,7 +1304,7 @@ def latent_attn(qd, wuk, wuv, pages, group, dims, scale: float, out) -> None:
                               _p(group.seq_lens), _p(group.c_start), _p(group.q_lens), _p(group.tok_rows), c_int(group.n),
                               c_int(group.block_table.shape[1]), c_int(group.n_tok), c_int(group.max_q), c_int(H), c_int(dn),
                               c_int(dr), c_int(dv), c_int(rank), c_int(W), c_int(n_split), c_float(scale), _p(q_lat), _p(po),
-                              _p(pml), _p(out), c_ll(out.stride(0)), _stream()), "pm_latent_attn")
+                              _p(pml), _p(out), c_ll(out.stride(0)), _p(status_word(dev)), _stream()), "pm_latent_attn")
     LAUNCHES += 2          # three kernels
 
 

@@ -176,7 +176,7 @@ def test_registry_and_configuration():
     assert a.to_hf_dict() == cfg and a.to_hf_dict() is not cfg
     m = build_model(cfg, torch.float32, "cpu")
     assert isinstance(m, HybridDecoderLM)
-    assert [l.mixer.cache_spec().page_width for l in m.layers] == [48, 0, 0, 80, 0, 0]
+    assert [l.mixer.cache_spec().page_width for l in m.layers] == [56, 0, 0, 88, 0, 0]
     with pytest.raises(RuntimeError, match="CUDA"):
         m(torch.tensor([1, 2]))
 
