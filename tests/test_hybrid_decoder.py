@@ -712,3 +712,27 @@ def test_trace_replay(tmp_path, monkeypatch, capsys, dtype):
     tol = max(bound("mixed", t, getattr(torch, dtype)) for t in (x, y, z))
     assert err(load(0), ox[[0, 98]]) < tol and err(load(1), ox[[99]]) < tol
     assert err(load(3), torch.cat([oz[[69, 3]], oy[[29]]])) < tol
+
+
+@gpu
+def test_trace_replay_serves_the_dense_decoder_too():
+    """The replay takes any model on the paged caches: portions, captured single steps and recycled blocks of the key / value
+    cache against the model's own whole-sequence forward."""
+    from pmetal_b200.models.config import ModelArgs
+    from pmetal_b200.models.decoder import DecoderLM
+    from pmetal_b200.serve.trace import TraceReplay
+    cfg = ModelArgs(vocab_size=300, hidden_size=256, intermediate_size=320, num_hidden_layers=2, num_attention_heads=2,
+                    num_key_value_heads=1, head_dim=128)
+    m = DecoderLM(cfg).init_weights(0.05, 0).to("cuda").to(torch.bfloat16).eval()
+    for p in m.parameters():
+        p.requires_grad_(False)
+    r = TraceReplay(m, 192)
+    for seed in (1, 2):
+        x, y = tokens(100, 300, seed), tokens(40, 300, 10 + seed)
+        a = r.step([{"id": "x", "tokens": x[:70], "want": [0, 69]}], [])
+        b = r.step([{"id": "y", "tokens": y[:39], "want": []}, {"id": "x", "tokens": x[70:99], "want": [28]}], [])
+        assert r.step([{"id": "y", "tokens": y[39:], "want": []}], []) is None
+        c = r.step([{"id": "x", "tokens": x[99:], "want": [0]}], ["x", "y"])
+        want = m(torch.tensor(x, device="cuda")).double().cpu()
+        assert err(torch.cat([a, b, c]), want[[0, 69, 98, 99]]) < 0.08
+    assert r.gen.cache.num_free() == 3
