@@ -152,14 +152,14 @@ def main() -> None:
                          "times to stderr")
     ap.add_argument("--serve-hybrid", nargs="*", metavar="PRESET", default=None,
                     help="instead of the headline benchmark: prefill / decode throughput and kernel times of the hybrid "
-                         "decoder presets (default duvivik-1b duvivik-4b) beside the dense decoder of equal size")
+                         "decoder presets (default duvivik-1b duvivik-2b) beside the dense decoder of equal size")
     args = ap.parse_args()
     if args.serve_hybrid is not None:
         from pmetal_b200.bench.hybrid_serve import report
         sampler = ClockSampler(0)
         sampler.start()
         t0 = time.time()
-        res = report(args.serve_hybrid or ["duvivik-1b", "duvivik-4b"])
+        res = report(args.serve_hybrid or ["duvivik-1b", "duvivik-2b"])
         res["clocks"] = sampler.stop(t0, time.time())
         print(json.dumps(res))
         return

@@ -20,7 +20,7 @@ from .kernels import peaks
 DENSE = {
     "duvivik-1b": dict(hidden_size=2048, intermediate_size=6144, num_hidden_layers=12, num_attention_heads=16,
                        num_key_value_heads=8),
-    "duvivik-4b": dict(hidden_size=2560, intermediate_size=9728, num_hidden_layers=19, num_attention_heads=32,
+    "duvivik-2b": dict(hidden_size=2560, intermediate_size=9728, num_hidden_layers=19, num_attention_heads=32,
                        num_key_value_heads=8),
 }
 

@@ -112,7 +112,7 @@ def _ssm(heads, vdim, state, groups, conv=4, norm_groups=1):
 PRESETS: Dict[str, dict] = {
     "duvivik-tiny": _stack(64, 512, 96, _attn(4, 16, 8, 24, 40), _ssm(4, 24, 16, 2, norm_groups=2), "AmaM"),
     "duvivik-1b": _stack(2048, 65536, 6144, _attn(32, 64, 64, 128, 512), _ssm(64, 64, 128, 8, norm_groups=8), "Ammmammm" * 2),
-    "duvivik-4b": _stack(2560, 65536, 9728, _attn(32, 96, 32, 128, 512), _ssm(80, 64, 128, 8, norm_groups=8), "Ammmammm" * 4),
+    "duvivik-2b": _stack(2560, 65536, 9728, _attn(32, 96, 32, 128, 512), _ssm(80, 64, 128, 8, norm_groups=8), "Ammmammm" * 4),
 }
 
 
