@@ -254,6 +254,9 @@ class HybridDecoderLM(nn.Module):
                 put(rnd().normal_(0.0, std, generator=g))
         return self
 
+    def head_weight(self) -> torch.Tensor:
+        return self.head
+
     def num_parameters(self, trainable_only: bool = False) -> int:
         return 0 if trainable_only else sum(p.numel() for p in self.parameters())
 
@@ -267,15 +270,25 @@ class HybridDecoderLM(nn.Module):
                           device or p.device)
 
     @torch.no_grad()
-    def forward(self, input_ids: torch.Tensor) -> torch.Tensor:
-        """Logits of whole sequences [T] or [B, L] -> [.., vocab] on a cache of their own."""
-        seqs = input_ids[None] if input_ids.dim() == 1 else input_ids
-        B, L = seqs.shape
-        cache = self.new_cache(B * -(-L // BLOCK), max_seqs=B)
-        for i in range(B):
+    def forward_hidden(self, input_ids: torch.Tensor, positions=None, cu_seqlens: Optional[torch.Tensor] = None,
+                       seq_start=None) -> torch.Tensor:
+        """Final-normed hidden state of every token of whole documents, [T] (cut at ``cu_seqlens``) or [B, L], on a cache of
+        their own; positions count from 0 in each document, as the model has it."""
+        if input_ids.dim() == 2:
+            lens = [input_ids.shape[1]] * input_ids.shape[0]
+        else:
+            lens = cu_seqlens.diff().tolist() if cu_seqlens is not None else [input_ids.shape[0]]
+        lens = [n for n in lens if n > 0]
+        cache = self.new_cache(sum(-(-n // BLOCK) for n in lens), max_seqs=len(lens))
+        for i in range(len(lens)):
             cache.add_sequence(i)
-        out = self.forward_paged(seqs.reshape(-1), cache, cache.prepare(list(range(B)), [L] * B), all_logits=True)
-        return out.view(*input_ids.shape, -1)
+        return self.forward_paged(input_ids.reshape(-1), cache, cache.prepare(list(range(len(lens))), lens), all_logits=True,
+                                  return_hidden=True)
+
+    def forward(self, input_ids: torch.Tensor, positions=None, cu_seqlens=None, seq_start=None) -> torch.Tensor:
+        """Logits of every token, shaped like ``input_ids``."""
+        h = self.forward_hidden(input_ids, positions, cu_seqlens, seq_start)
+        return ops.project_f32(h, self.head, self.cfg.vocab_size).view(*input_ids.shape, -1)
 
     @torch.no_grad()
     def forward_paged(self, input_ids: torch.Tensor, cache: StateCache, meta, all_logits: bool = False,

@@ -260,6 +260,10 @@ class PagedKVCache(PagedBlocks):
             self.k_scale = [torch.ones(sshape, dtype=torch.float32, device=device) for _ in range(num_layers)]
             self.v_scale = [torch.ones(sshape, dtype=torch.float32, device=device) for _ in range(num_layers)]
 
+    def bytes_per_token(self) -> int:
+        k = self.k[0]
+        return 2 * self.num_layers * k.shape[2] * k.shape[3] * k.element_size()
+
     def _copy_block(self, dst: int, src: int) -> None:
         for l in range(self.num_layers):
             self.k[l][dst].copy_(self.k[l][src])

@@ -45,6 +45,7 @@ class StateCache(PagedBlocks):
                 self.slots[i] = {n: torch.zeros(max_seqs + 1, *shape, dtype=dt or dtype, device=device)
                                  for n, (shape, dt) in s.slots.items()}
         self.can_truncate = not self.slots
+        # without recurrent layers nothing is kept per sequence: every sequence names slot 0 and their number is not limited
         self.free_slots: List[int] = list(range(max_seqs - 1, -1, -1))
         self.slot_of: Dict[int, int] = {}
 
@@ -56,26 +57,35 @@ class StateCache(PagedBlocks):
         ts = list(self.pages.values()) + [t for d in self.slots.values() for t in d.values()]
         return sum(t.numel() * t.element_size() for t in ts)
 
+    def bytes_per_token(self) -> int:
+        return sum(t.shape[2] * t.element_size() for t in self.pages.values())
+
     # ------------------------------------------------------------------ sequences
     def can_admit(self) -> bool:
-        return bool(self.free_slots)
+        return not self.slots or bool(self.free_slots)
+
+    def _take_slot(self, seq_id: int) -> int:
+        slot = self.free_slots.pop() if self.slots else 0
+        self.slot_of[seq_id] = slot
+        return slot
 
     def add_sequence(self, seq_id: int) -> None:
-        if not self.free_slots:
+        if not self.can_admit():
             raise MemoryError(f"all {self.max_seqs} state slots are in use")
         super().add_sequence(seq_id)
-        self.slot_of[seq_id] = self.free_slots.pop()
+        self._take_slot(seq_id)
 
     def free_sequence(self, seq_id: int) -> None:
         super().free_sequence(seq_id)
-        self.free_slots.append(self.slot_of.pop(seq_id))
+        slot = self.slot_of.pop(seq_id)
+        if self.slots:
+            self.free_slots.append(slot)
 
     def fork(self, src_id: int, dst_id: int) -> None:
-        if not self.free_slots:
+        if not self.can_admit():
             raise MemoryError(f"all {self.max_seqs} state slots are in use")
         super().fork(src_id, dst_id)
-        a, b = self.slot_of[src_id], self.free_slots.pop()
-        self.slot_of[dst_id] = b
+        a, b = self.slot_of[src_id], self._take_slot(dst_id)
         for d in self.slots.values():
             for t in d.values():
                 t[b].copy_(t[a])

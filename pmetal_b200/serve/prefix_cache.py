@@ -9,19 +9,18 @@ from __future__ import annotations
 from collections import OrderedDict
 from typing import List, Optional, Sequence, Tuple
 
-from ..models.kv_cache import BLOCK, PagedKVCache
+from ..models.kv_cache import BLOCK, PagedBlocks
 
 
 class PrefixCache:
-    def __init__(self, cache: PagedKVCache, max_entries: int = 16, max_bytes: int = 2 << 30, min_tokens: int = BLOCK):
+    def __init__(self, cache: PagedBlocks, max_entries: int = 16, max_bytes: int = 2 << 30, min_tokens: int = BLOCK):
         self.cache, self.max_entries, self.max_bytes, self.min_tokens = cache, max_entries, max_bytes, min_tokens
         self.entries: "OrderedDict[int, Tuple[List[int], int]]" = OrderedDict()     # seq id -> (tokens, bytes)
         self.hits = self.misses = 0
         self._next = -1          # parked sequences use negative ids
 
     def _bytes_per_token(self) -> int:
-        k = self.cache.k[0]
-        return 2 * len(self.cache.k) * k.shape[2] * k.shape[3] * k.element_size()
+        return self.cache.bytes_per_token()
 
     def total_bytes(self) -> int:
         return sum(b for _, b in self.entries.values())

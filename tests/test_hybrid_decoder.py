@@ -245,7 +245,10 @@ def test_state_cache_bookkeeping():
     c.free_sequence(7)
     c.free_sequence(8)
     assert c.num_free() == 4 and sorted(c.free_slots) == [0, 1]
-    assert StateCache(specs[:1], 4, 2, torch.bfloat16, "cpu").can_truncate
+    c = StateCache(specs[:1], 4, 2, torch.bfloat16, "cpu")             # nothing per sequence: any number of them
+    for i in range(5):
+        c.add_sequence(i)
+    assert c.can_truncate and c.can_admit() and c.bytes_per_token() == 32 and set(c.slot_of.values()) == {0}
 
 
 def test_split_groups():
@@ -561,6 +564,9 @@ def test_model_whole_portions_and_decoding(name, dtype):
     toks = tokens(150, cfg["vocab"], 5)
     want, tol = oracle(name, toks), bound(name, toks, dtype)
     assert err(m(torch.tensor(toks, device="cuda")), want) < tol
+    docs = torch.tensor(toks[:70] + toks, device="cuda")                                  # two documents in one stream
+    got = m(docs, cu_seqlens=torch.tensor([0, 70, 220], device="cuda"))
+    assert err(got[:70], want[:70]) < tol and err(got[70:], want) < tol
     for sizes in ([150], [130, 1], [2], [1], [64, 1, 1, 63, 3], [5, 20, 70, 2, 1, 1]):
         gen = generator(m)
         got = feed(gen, gen.new_seq(), toks, sizes)
@@ -658,6 +664,25 @@ def test_greedy_generation_through_the_engine():
 
 
 @gpu
+def test_attention_only_stack_shares_prompt_prefixes():
+    """Without recurrent layers prompts may be parked and cut at block borders: a second request forks the cached pages."""
+    from pmetal_b200.models.sampling import SamplingParams
+    from pmetal_b200.serve.engine import ContinuousBatchEngine
+    cfg = config([(attn(2, 16, 8, 16, 32), 32, 1.0), (attn(3, 16, 8, 8, 32, kv_from=0), None, 0)], width=32, vocab=60)
+    sd = random_weights(cfg, 2)
+    m = build_model(cfg, torch.float32, "cuda")
+    m.load_hf_state_dict(sd)
+    e = ContinuousBatchEngine(m, max_slots=2, num_blocks=24)
+    p = tokens(150, 60, 9)
+    a = e.generate(p, SamplingParams.greedy(4))
+    b = e.generate(p[:140] + [1, 2, 3], SamplingParams.greedy(4))
+    ref = ContinuousBatchEngine(m, max_slots=2, num_blocks=24, prefix_cache=False)
+    assert e.stats.prefix_hits == 1 and b.cached_tokens == 128
+    assert a.output == ref.generate(p, SamplingParams.greedy(4)).output
+    assert b.output == ref.generate(p[:140] + [1, 2, 3], SamplingParams.greedy(4)).output
+
+
+@gpu
 def test_sampled_requests_and_background_thread():
     from pmetal_b200.models.sampling import SamplingParams
     from pmetal_b200.serve.engine import ContinuousBatchEngine
@@ -683,8 +708,32 @@ def test_command_line(tmp_path, capsys):
     assert out["generated_tokens"] == 5 and out["prompt_tokens"] == 5
     assert main(["infer", "-m", "random:duvivik-tiny", "-p", "hi", "--profile-layers", "--json"]) == 0
     assert len(json.loads(capsys.readouterr().out.strip().splitlines()[-1])["layers"]) == 4
+    data = tmp_path / "d.jsonl"
+    data.write_text('{"text": "some words"}\n{"text": "and a few more"}\n')
+    assert main(["eval", "-m", str(tmp_path), "-d", str(data)]) == 0
+    assert json.loads(capsys.readouterr().out.strip().splitlines()[-1])["perplexity"] > 1
     with pytest.raises(SystemExit, match="--lora"):
         main(["infer", "-m", str(tmp_path), "-p", "x", "-l", str(tmp_path)])
+
+
+@gpu
+def test_http_server():
+    from fastapi.testclient import TestClient
+
+    from pmetal_b200.data.tokenizer import ByteTokenizer
+    from pmetal_b200.serve.engine import ContinuousBatchEngine
+    from pmetal_b200.serve.server import ServerState, create_app
+    m, _, _ = load_pretrained("random:duvivik-tiny", torch.bfloat16, "cuda")
+    eng = ContinuousBatchEngine(m, max_slots=2, num_blocks=16)
+    eng.start()
+    try:
+        with TestClient(create_app(ServerState(eng, ByteTokenizer(), model_name="tiny"))) as c:
+            r = c.post("/v1/completions", json={"model": "tiny", "prompt": "hi there", "max_tokens": 5, "temperature": 0}).json()
+            assert r["usage"] == {"prompt_tokens": 8, "completion_tokens": 5, "total_tokens": 13}
+            e = c.post("/v1/embeddings", json={"model": "tiny", "input": ["a", "some text"]}).json()
+            assert len(e["data"]) == 2 and len(e["data"][0]["embedding"]) == m.cfg.hidden_size
+    finally:
+        eng.shutdown()
 
 
 @gpu
