@@ -16,7 +16,7 @@ import torch
 import torch.nn as nn
 
 from ..ops import functional as ops
-from .state_cache import CacheSpec, SeqGroup, split_groups
+from .state_cache import CacheSpec, split_groups
 
 # portions up to this many tokens take the decode kernels (state-space scan, attention in the latent space)
 SHORT = 16
