@@ -26,7 +26,9 @@ CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-ffp-contract=off", "-pthread"]   # 
 
 # sources (csrc/*.cu) that a product entry point can be built from alone, for a checkout where nothing is compiled yet
 COMPONENTS = {
-    "hybrid": ("attention_tc", "gemm_2sm", "gemm_tcgen05", "gemv", "latent_attn", "postnorm", "ssm"),
+    "duvivik": ("attention_tc", "gemm_2sm", "gemm_tcgen05", "gemv", "latent_attn", "postnorm", "ssd_chunk", "ssm"),
+    "resevik": ("gemm_2sm", "gemm_tcgen05", "gemv", "grouped_gemm", "linear_attn", "moe_experts", "moe_quant", "postnorm",
+                "ssd_chunk", "window_attn"),
     "decoder": ("attention", "attention_tc", "decode_mega", "elementwise", "gemm_2sm", "gemm_tcgen05", "gemv",
                 "grouped_gemm", "moe_quant"),
 }

@@ -1,0 +1,168 @@
+// Routed experts whose weight multiplies the expert's input: y = sum over a token's experts of down(silu(G w h) * (U w h)).
+// The (token, slot) pairs come sorted by expert (moe_quant.cu):
+//   expert_gather_kernel   rows w h in sorted order, or in a layout whose slabs start at multiples of `align` rows (zero rows
+//                          between them), for the grouped tensor-core GEMMs (grouped_gemm.cu)
+//   expert_rows_kernel     products of sorted rows with their experts' matrices on the CUDA cores, fp32 sums, any size and
+//                          type: fp32 models, and sizes that the GEMMs cannot copy in 16-byte pieces
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+#include "elem.cuh"
+#include "host_util.cuh"
+#include "pmetal_b200.h"
+
+namespace pm {
+
+// Largest e with off[e] <= row (off non-decreasing, row < off[E]).
+__device__ __forceinline__ int expert_at(const int* __restrict__ off, int E, int row) {
+  int lo = 0, hi = E;
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if (off[mid] <= row) lo = mid; else hi = mid;
+  }
+  return lo;
+}
+
+// One CTA per row of xs. Plain layout: row = sorted position. Padded layout (align > 0): every CTA derives the padded
+// offsets itself; CTA 0 writes them, and the rows write dest[pair] = padded row.
+template <typename T, int V>
+__global__ void __launch_bounds__(128) expert_gather_kernel(const T* __restrict__ h, long long ldh, const int* __restrict__ perm,
+                                                            const float* __restrict__ w, const int* __restrict__ off, int E,
+                                                            int k, int align, int width, T* __restrict__ xs,
+                                                            int* __restrict__ off_pad, int* __restrict__ dest) {
+  extern __shared__ int s_pad[];                  // [E + 1]
+  const int row = blockIdx.x;
+  int pos = row;
+  if (align > 0) {
+    const int lane = threadIdx.x & 31;
+    if (threadIdx.x < 32) {
+      int base = 0;
+      for (int e0 = 0; e0 < E; e0 += 32) {
+        const int e = e0 + lane;
+        int c = e < E ? (off[e + 1] - off[e] + align - 1) / align * align : 0;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const int up = __shfl_up_sync(0xffffffffu, c, o);
+          if (lane >= o) c += up;
+        }
+        if (e < E) s_pad[e + 1] = base + c;
+        base += __shfl_sync(0xffffffffu, c, 31);
+      }
+      if (lane == 0) s_pad[0] = 0;
+    }
+    __syncthreads();
+    if (row == 0)
+      for (int e = threadIdx.x; e <= E; e += blockDim.x) off_pad[e] = s_pad[e];
+    pos = -1;
+    if (row >= s_pad[E]) return;                  // past the last slab: never read
+    const int e = expert_at(s_pad, E, row);
+    const int in = row - s_pad[e];
+    if (in < off[e + 1] - off[e]) pos = off[e] + in;
+  }
+  const int pair = pos >= 0 ? perm[pos] : 0;
+  const float f = pos >= 0 ? w[pair] : 0.f;
+  if (align > 0 && pos >= 0 && threadIdx.x == 0) dest[pair] = row;
+  const T* src = h + static_cast<long long>(pair / k) * ldh;
+  T* dst = xs + static_cast<long long>(row) * width;
+  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+    float v[V];
+    if (pos >= 0) {
+      load_vec<V>(src + c, v);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] *= f;
+    } else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = 0.f;
+    }
+    store_vec<V>(dst + c, v);
+  }
+}
+
+constexpr int kRowTile = 8;
+
+// x [rows, K] sorted, W [E][M][K] -> out [rows, N]: M = N, or with `glu` M = 2 N (gate rows above up rows) and
+// out = silu(gate) * up. CTA: 8 rows; warp: one output channel at a time.
+template <typename T>
+__global__ void __launch_bounds__(256) expert_rows_kernel(const T* __restrict__ x, int rows, const T* __restrict__ W,
+                                                          const int* __restrict__ off, int E, int N, int K, int glu,
+                                                          T* __restrict__ out) {
+  const int r0 = blockIdx.y * kRowTile, n_rows = min(kRowTile, rows - r0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long mat = static_cast<long long>(glu ? 2 * N : N) * K;
+  for (int n = blockIdx.x * 8 + warp; n < N; n += gridDim.x * 8) {
+    for (int a = 0; a < n_rows;) {
+      const int e = expert_at(off, E, r0 + a);
+      const int b = max(a + 1, min(n_rows, off[e + 1] - r0));          // rows a .. b - 1 belong to expert e
+      const T* wg = W + e * mat + static_cast<long long>(n) * K;
+      const T* wu = wg + static_cast<long long>(N) * K;
+      float g[kRowTile], u[kRowTile];
+#pragma unroll
+      for (int i = 0; i < kRowTile; ++i) g[i] = u[i] = 0.f;
+      for (int c = lane; c < K; c += 32) {
+        const float fg = to_f(wg[c]), fu = glu ? to_f(wu[c]) : 0.f;
+#pragma unroll
+        for (int i = 0; i < kRowTile; ++i)
+          if (a + i < b) {
+            const float v = to_f(x[static_cast<long long>(r0 + a + i) * K + c]);
+            g[i] = fmaf(fg, v, g[i]);
+            u[i] = fmaf(fu, v, u[i]);
+          }
+      }
+#pragma unroll
+      for (int i = 0; i < kRowTile; ++i)
+        if (a + i < b) {
+          const float sg = warp_sum(g[i]), su = glu ? warp_sum(u[i]) : 0.f;
+          if (lane == 0) put(out + static_cast<long long>(r0 + a + i) * N + n, glu ? silu_f(sg) * su : sg);
+        }
+      a = b;
+    }
+  }
+}
+
+template <typename T>
+static int gather_launch(const void* h, long long ldh, const int* perm, const float* w, const int* off, int E, int k, int align,
+                         int rows, int width, void* xs, int* off_pad, int* dest, cudaStream_t st) {
+  const size_t smem = align > 0 ? sizeof(int) * (E + 1) : 0;
+  const T* src = static_cast<const T*>(h);
+  T* dst = static_cast<T*>(xs);
+  if (width % 8 == 0 && ldh % 8 == 0)
+    expert_gather_kernel<T, 8><<<rows, 128, smem, st>>>(src, ldh, perm, w, off, E, k, align, width, dst, off_pad, dest);
+  else
+    expert_gather_kernel<T, 1><<<rows, 128, smem, st>>>(src, ldh, perm, w, off, E, k, align, width, dst, off_pad, dest);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace pm
+
+using namespace pm;
+
+// xs [rows, width] = w[pair] * h[pair / k] for the pairs perm[0 .. n) sorted by expert (off [E + 1]). align 0: rows = n in
+// sorted order. align > 0: every expert's slab starts at a multiple of align (off_pad [E + 1]), dest [n] is the row of each
+// pair, rows between slabs are zero; rows must be at least n + (align - 1) per expert with pairs.
+extern "C" int pm_expert_gather(const void* h, int f32, long long ldh, const int* perm, const float* w, const int* off, int E,
+                                int k, int align, int rows, int width, void* xs, int* off_pad, int* dest, cudaStream_t st) {
+  if (E < 1 || E > 1024 || k < 1 || align < 0 || width < 1 || (align > 0 && (!off_pad || !dest))) return -1;
+  if (rows < 1) return 0;
+  return f32 ? gather_launch<float>(h, ldh, perm, w, off, E, k, align, rows, width, xs, off_pad, dest, st)
+             : gather_launch<__nv_bfloat16>(h, ldh, perm, w, off, E, k, align, rows, width, xs, off_pad, dest, st);
+}
+
+// x [rows, K] sorted by expert (off [E + 1], off[E] = rows), W [E][N or, glu 1, 2 N][K] -> out [rows, N] = x W_e^T, or with
+// glu silu(x G_e^T) * (x U_e^T) (gate rows above up rows).
+extern "C" int pm_expert_rows(const void* x, int f32, int rows, const void* W, const int* off, int E, int N, int K, int glu,
+                              void* out, cudaStream_t st) {
+  if (E < 1 || N < 1 || K < 1) return -1;
+  if (rows < 1) return 0;
+  const int tiles = (rows + kRowTile - 1) / kRowTile;
+  if (tiles > 65535) return -2;
+  const int want = (16 * num_sms() + tiles - 1) / tiles, cols = (N + 7) / 8;
+  const dim3 grid(want < cols ? (want < 1 ? 1 : want) : cols, tiles);
+  if (f32)
+    expert_rows_kernel<float><<<grid, 256, 0, st>>>(static_cast<const float*>(x), rows, static_cast<const float*>(W), off, E, N, K,
+                                                    glu, static_cast<float*>(out));
+  else
+    expert_rows_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(x), rows,
+                                                            static_cast<const __nv_bfloat16*>(W), off, E, N, K, glu,
+                                                            static_cast<__nv_bfloat16*>(out));
+  return static_cast<int>(cudaGetLastError());
+}

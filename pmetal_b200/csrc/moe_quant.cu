@@ -2,7 +2,8 @@
 //
 // MoE (reference: crates/pmetal-metal/src/kernels/metal/moe_routing.metal — moe_topk_selection,
 // moe_compute_indices, moe_compute_expert_offsets, moe_sort_indices; crates/pmetal-models/src/moe_routing.rs:52-108):
-//   moe_router_kernel   softmax over experts, top-k by repeated warp argmax, optional renormalisation of the k weights
+//   moe_router_kernel   softmax over experts (or the sigmoid of every logit), top-k by repeated warp argmax, optional
+//                       renormalisation of the k weights
 //   moe_count_kernel    tokens per expert
 //   moe_scan_kernel     exclusive prefix sum of the counts (one block)
 //   moe_sort_kernel     stable counting sort of the (token, slot) pairs by expert: perm[pos] = token*k + slot,
@@ -25,18 +26,20 @@ namespace pm {
 
 // ------------------------------------------------------------------------------------------------ MoE routing
 // One warp per token. E <= 1024 experts (NV = ceil(E / 32) per lane, kept in registers), k <= 16.
+// score 0: softmax over the experts, 1: sigmoid. Logit rows are ldl apart.
 template <int NV>
 __device__ __forceinline__ void moe_route_token_nv(const __nv_bfloat16* __restrict__ logits_bf16,
-                                                   const float* __restrict__ logits_f32, int t, int E, int k, int renorm,
-                                                   int* __restrict__ topk_idx, float* __restrict__ topk_w, int lane) {
+                                                   const float* __restrict__ logits_f32, int ldl, int score, int t, int E,
+                                                   int k, int renorm, int* __restrict__ topk_idx,
+                                                   float* __restrict__ topk_w, int lane) {
   float v[NV];
   float mx = -INFINITY;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int e = i * 32 + lane;
     float x = -INFINITY;
-    if (e < E) x = logits_f32 ? logits_f32[static_cast<long long>(t) * E + e]
-                              : __bfloat162float(logits_bf16[static_cast<long long>(t) * E + e]);
+    if (e < E) x = logits_f32 ? logits_f32[static_cast<long long>(t) * ldl + e]
+                              : __bfloat162float(logits_bf16[static_cast<long long>(t) * ldl + e]);
     v[i] = x;
     mx = fmaxf(mx, x);
   }
@@ -44,11 +47,12 @@ __device__ __forceinline__ void moe_route_token_nv(const __nv_bfloat16* __restri
   float z = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    v[i] = (i * 32 + lane < E) ? __expf(v[i] - mx) : -1.f;
+    if (score) v[i] = (i * 32 + lane < E) ? 1.f / (1.f + expf(-v[i])) : -1.f;
+    else v[i] = (i * 32 + lane < E) ? __expf(v[i] - mx) : -1.f;
     if (v[i] > 0.f) z += v[i];
   }
   for (int o = 16; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-  const float inv_z = 1.f / z;
+  const float inv_z = score ? 1.f : 1.f / z;
   float wsum = 0.f, my_w = 0.f;
   int my_idx = 0;
   for (int j = 0; j < k; ++j) {
@@ -64,6 +68,7 @@ __device__ __forceinline__ void moe_route_token_nv(const __nv_bfloat16* __restri
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
     }
+    if (bi >= E) { bi = j; bv = 0.f; }             // logits that are not numbers: any expert, no weight
     if ((bi & 31) == lane) {
 #pragma unroll
       for (int i = 0; i < NV; ++i)
@@ -80,20 +85,21 @@ __device__ __forceinline__ void moe_route_token_nv(const __nv_bfloat16* __restri
 }
 
 __device__ __forceinline__ void moe_route_token(const __nv_bfloat16* __restrict__ logits_bf16,
-                                                const float* __restrict__ logits_f32, int t, int E, int k, int renorm,
-                                                int* __restrict__ topk_idx, float* __restrict__ topk_w, int lane) {
-  if (E <= 64) moe_route_token_nv<2>(logits_bf16, logits_f32, t, E, k, renorm, topk_idx, topk_w, lane);
-  else if (E <= 128) moe_route_token_nv<4>(logits_bf16, logits_f32, t, E, k, renorm, topk_idx, topk_w, lane);
-  else if (E <= 256) moe_route_token_nv<8>(logits_bf16, logits_f32, t, E, k, renorm, topk_idx, topk_w, lane);
-  else moe_route_token_nv<32>(logits_bf16, logits_f32, t, E, k, renorm, topk_idx, topk_w, lane);
+                                                const float* __restrict__ logits_f32, int ldl, int score, int t, int E,
+                                                int k, int renorm, int* __restrict__ topk_idx, float* __restrict__ topk_w,
+                                                int lane) {
+  if (E <= 64) moe_route_token_nv<2>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
+  else if (E <= 128) moe_route_token_nv<4>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
+  else if (E <= 256) moe_route_token_nv<8>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
+  else moe_route_token_nv<32>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
 }
 
 __global__ void moe_router_kernel(const __nv_bfloat16* __restrict__ logits_bf16, const float* __restrict__ logits_f32,
-                                  int T, int E, int k, int renorm, int* __restrict__ topk_idx,
+                                  int ldl, int score, int T, int E, int k, int renorm, int* __restrict__ topk_idx,
                                   float* __restrict__ topk_w) {
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T) return;
-  moe_route_token(logits_bf16, logits_f32, t, E, k, renorm, topk_idx, topk_w, threadIdx.x & 31);
+  moe_route_token(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, threadIdx.x & 31);
 }
 
 // Few tokens (T * k <= 1024): routing, counting, offsets and the stable sort in one CTA, so that a decode step pays one
@@ -101,15 +107,16 @@ __global__ void moe_router_kernel(const __nv_bfloat16* __restrict__ logits_bf16,
 // and deterministic. offsets2 (optional) receives a second copy of the offsets (the expert-parallel exchange buffer).
 constexpr int kRouteSmallMax = 1024;
 __global__ void __launch_bounds__(1024) moe_route_small_kernel(const __nv_bfloat16* __restrict__ logits_bf16,
-                                                               const float* __restrict__ logits_f32, int T, int E, int k,
-                                                               int renorm, int* __restrict__ topk_idx,
+                                                               const float* __restrict__ logits_f32, int ldl, int score,
+                                                               int T, int E, int k, int renorm, int* __restrict__ topk_idx,
                                                                float* __restrict__ topk_w, int* __restrict__ counts,
                                                                int* __restrict__ offsets, int* __restrict__ offsets2,
                                                                int* __restrict__ perm, int* __restrict__ inv) {
   __shared__ int s_idx[kRouteSmallMax];
   __shared__ int s_off[1024 + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = T * k;
-  for (int t = warp; t < T; t += 32) moe_route_token(logits_bf16, logits_f32, t, E, k, renorm, topk_idx, topk_w, lane);
+  for (int t = warp; t < T; t += 32)
+    moe_route_token(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
   __syncthreads();
   for (int i = threadIdx.x; i < n; i += blockDim.x) s_idx[i] = topk_idx[i];
   __syncthreads();
@@ -155,7 +162,7 @@ __global__ void __launch_bounds__(1024) moe_route_local_kernel(const __nv_bfloat
   __shared__ int s_idx[kRouteLocalMax];
   __shared__ int s_off[1024 + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = T * k;
-  for (int t = warp; t < T; t += 32) moe_route_token(logits_bf16, logits_f32, t, E, k, renorm, topk_idx, topk_w, lane);
+  for (int t = warp; t < T; t += 32) moe_route_token(logits_bf16, logits_f32, E, 0, t, E, k, renorm, topk_idx, topk_w, lane);
   __syncthreads();
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
     const int x = topk_idx[i];
@@ -490,21 +497,22 @@ static inline int grid_cap(long long work, int per_block, int cap = 0) {
 
 using namespace pm;
 
-// offsets2: optional second destination for the [E + 1] offsets (may be null).
-extern "C" int pm_moe_route2(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx,
-                             float* topk_w, int* counts, int* offsets, int* offsets2, int* perm, int* inv,
+// Routing, counts, offsets and the expert-sorted order of T tokens. Logit rows (fp32 or bf16) are ldl apart; score 0 is the
+// softmax over the experts, 1 the sigmoid of every logit; renorm divides the k weights by their sum. offsets2: optional
+// second destination for the [E + 1] offsets (may be null).
+extern "C" int pm_moe_route3(const void* logits, int is_f32, int ldl, int score, int T, int E, int k, int renorm,
+                             int* topk_idx, float* topk_w, int* counts, int* offsets, int* offsets2, int* perm, int* inv,
                              cudaStream_t st) {
-  if (T <= 0 || E <= 0 || E > 1024 || k <= 0 || k > 16 || k > E) return -1;
+  if (T <= 0 || E <= 0 || E > 1024 || k <= 0 || k > 16 || k > E || ldl < E || score < 0 || score > 1) return -1;
   const long long n = static_cast<long long>(T) * k;
+  const __nv_bfloat16* lb = is_f32 ? nullptr : static_cast<const __nv_bfloat16*>(logits);
+  const float* lf = is_f32 ? static_cast<const float*>(logits) : nullptr;
   if (n <= kRouteSmallMax && E < 1024) {
-    moe_route_small_kernel<<<1, 1024, 0, st>>>(is_f32 ? nullptr : static_cast<const __nv_bfloat16*>(logits),
-                                               is_f32 ? static_cast<const float*>(logits) : nullptr, T, E, k, renorm,
-                                               topk_idx, topk_w, counts, offsets, offsets2, perm, inv);
+    moe_route_small_kernel<<<1, 1024, 0, st>>>(lb, lf, ldl, score, T, E, k, renorm, topk_idx, topk_w, counts, offsets,
+                                               offsets2, perm, inv);
     return static_cast<int>(cudaGetLastError());
   }
-  moe_router_kernel<<<(T + 7) / 8, 256, 0, st>>>(is_f32 ? nullptr : static_cast<const __nv_bfloat16*>(logits),
-                                                 is_f32 ? static_cast<const float*>(logits) : nullptr, T, E, k, renorm,
-                                                 topk_idx, topk_w);
+  moe_router_kernel<<<(T + 7) / 8, 256, 0, st>>>(lb, lf, ldl, score, T, E, k, renorm, topk_idx, topk_w);
   moe_count_kernel<<<E, 256, 0, st>>>(topk_idx, n, counts);
   moe_scan_kernel<<<1, 32, 0, st>>>(counts, E, offsets);
   moe_sort_kernel<<<E, 256, 0, st>>>(topk_idx, n, offsets, perm, inv);
@@ -513,6 +521,12 @@ extern "C" int pm_moe_route2(const void* logits, int is_f32, int T, int E, int k
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int pm_moe_route2(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx,
+                             float* topk_w, int* counts, int* offsets, int* offsets2, int* perm, int* inv,
+                             cudaStream_t st) {
+  return pm_moe_route3(logits, is_f32, E, 0, T, E, k, renorm, topk_idx, topk_w, counts, offsets, offsets2, perm, inv, st);
 }
 
 extern "C" int pm_moe_route(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx,

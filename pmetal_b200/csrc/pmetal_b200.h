@@ -229,6 +229,27 @@ int pm_latent_assemble(const void* qd, long long ldq, int n_q, const void* kv, l
 // out [n, ldo] (H * dv columns) = the first dv channels of every head of o128 [n, H, 128].
 int pm_latent_take(const void* o128, int n, int H, int dv, void* out, long long ldo, cudaStream_t st);
 
+// ---------------------------------------------------------------- linear_attn.cu
+// Token-by-token recurrence. u [tokens, ldu]; cs / sn fp32 [tokens, R / 2] (unused when R is 0); rot: 1 pairs (i, i + R / 2),
+// 2 pairs (2 i, 2 i + 1); act: 1 silu on q, k, v; decay fp32 [H]; state [slots][H][N][P4] fp32, read and written;
+// y [tokens, H P]. Sequence i covers tokens q_start[i] .. + q_lens[i] - 1 and ends at position seq_lens[i] - 1.
+int pm_linear_scan(const void* u, int f32, long long ldu, const float* cs, const float* sn, const float* decay,
+    float kscale, float* state, const int* slots, const int* q_start, const int* q_lens, const int* seq_lens, int
+    n_seq, int H, int N, int P, int R, int rot, int act, void* y, cudaStream_t st);
+// Whether pm_linear_chunk covers keys of N channels.
+int pm_linear_chunk_supported(int N);
+// The same for longer portions of bf16 models (act bf16 [n_tok, H P + 2 H N], twice the key and query columns when R > 0:
+// work buffer over all n_tok rows of the step; log2_decay fp32 [H]; seg_state [n_seq][max_seg][H][N][P4] and seg_decay
+// [n_seq][max_seg][H] fp32 work buffers; max_q: the longest of q_lens).
+int pm_linear_chunk(const void* u, long long ldu, const float* cs, const float* sn, const float* log2_decay, float
+    kscale, float* state, const int* slots, const int* q_start, const int* q_lens, const int* seq_lens, int n_seq,
+    int n_tok, int max_q, int H, int N, int P, int R, int rot, int act, void* act_buf, float* seg_state, float*
+    seg_decay, int max_seg, void* y, cudaStream_t st);
+// out [tokens, parts * width] = RMS norm over every part of y, times w (fp32 [parts * width] or null), times
+// sigmoid(gate) or, silu 1, silu(gate); gate rows are ldg apart.
+int pm_norm_gate(const void* y, const void* gate, int f32, long long ldg, const float* w, float eps, int parts, int
+    width, int silu, void* out, int n_tok, cudaStream_t st);
+
 // ---------------------------------------------------------------- mhc.cu
 // x [T, n, C] bf16; either phi [n C, n^2 + 2n] fp32 (dot products formed here) or raw [T, ld_raw] fp32 = x . phi computed by
 // the caller; bias [n^2 + 2n], alpha [3]; n in {2, 4, 8}, C % 8 == 0, iters <= 32.
@@ -248,6 +269,17 @@ int pm_mhc_amax_gain(const float* h_res, int T, int n, float* gains, cudaStream_
 int pm_mhc_expand(const void* x, int T, int n, int C, void* xs, cudaStream_t st);
 int pm_mhc_collapse(const void* xs, int T, int n, int C, void* x, cudaStream_t st);
 
+// ---------------------------------------------------------------- moe_experts.cu
+// xs [rows, width] = w[pair] * h[pair / k] for the pairs perm[0 .. n) sorted by expert (off [E + 1]). align 0: rows = n in
+// sorted order. align > 0: every expert's slab starts at a multiple of align (off_pad [E + 1]), dest [n] is the row of each
+// pair, rows between slabs are zero; rows must be at least n + (align - 1) per expert with pairs.
+int pm_expert_gather(const void* h, int f32, long long ldh, const int* perm, const float* w, const int* off, int E,
+    int k, int align, int rows, int width, void* xs, int* off_pad, int* dest, cudaStream_t st);
+// x [rows, K] sorted by expert (off [E + 1], off[E] = rows), W [E][N or, glu 1, 2 N][K] -> out [rows, N] = x W_e^T, or with
+// glu silu(x G_e^T) * (x U_e^T) (gate rows above up rows).
+int pm_expert_rows(const void* x, int f32, int rows, const void* W, const int* off, int E, int N, int K, int glu,
+    void* out, cudaStream_t st);
+
 // ---------------------------------------------------------------- moe_gemm.cu
 int pm_ep_prepare(const unsigned long long* offset_ptrs, const unsigned long long* pad_ptrs, int rank, int world,
     int e_loc, void* tiles, void* runs, int max_tiles, int max_runs, int* counts_out, double timeout_s, int*
@@ -262,7 +294,11 @@ int pm_moe_gemm(const void* a, int a_rows, int lda, const void* w, int ldw, int 
     copy_src_ptrs, void* tile_ready, double timeout_s, int* status, cudaStream_t st);
 
 // ---------------------------------------------------------------- moe_quant.cu
-// offsets2: optional second destination for the [E + 1] offsets (may be null).
+// Routing, counts, offsets and the expert-sorted order of T tokens. Logit rows (fp32 or bf16) are ldl apart; score 0 is the
+// softmax over the experts, 1 the sigmoid of every logit; renorm divides the k weights by their sum. offsets2: optional
+// second destination for the [E + 1] offsets (may be null).
+int pm_moe_route3(const void* logits, int is_f32, int ldl, int score, int T, int E, int k, int renorm, int*
+    topk_idx, float* topk_w, int* counts, int* offsets, int* offsets2, int* perm, int* inv, cudaStream_t st);
 int pm_moe_route2(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx, float* topk_w,
     int* counts, int* offsets, int* offsets2, int* perm, int* inv, cudaStream_t st);
 int pm_moe_route(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx, float* topk_w,
@@ -294,6 +330,12 @@ int pm_embed_scale(const long long* ids, const void* table, int f32, float scale
 int pm_post_layernorm(const float* x, const void* y, int f32, long long ldy, const float* bias, float alpha, const
     float* w, const float* b, float eps, int n, int width, const long long* rows, float* of, void* oc, cudaStream_t
     st);
+// v = x + y + sum_j z[inv[t * k + j]] + x0 for the n rows listed in `rows` (nullable: row i); of [n, width] fp32 (nullable, may
+// be x when rows is null) = v, oc [n, width] in the compute type = v / rms(v) * w. y [.., ldy], z [.., width] (compute type,
+// inv int32 per token and j < k) and x0 (fp32) are nullable.
+int pm_add_rmsnorm(const float* x, const void* y, int f32, long long ldy, const void* z, const int* inv, int k,
+    const float* x0, const float* w, float eps, int n, int width, const long long* rows, float* of, void* oc,
+    cudaStream_t st);
 // gu [n, ld]: gate columns [0, ff), up columns [ff, 2 ff); bias fp32 [2 ff] or null -> out [n, ff].
 int pm_clamped_glu(const void* gu, int f32, long long ld, const float* bias, int n, int ff, float limit, float
     beta, float shift, void* out, cudaStream_t st);
@@ -355,6 +397,20 @@ int pm_merge_fused(const void* const* models, const void* base, const float* wei
     const float* densities, int n_models, int in_bf16, int out_bf16, int consensus, int rescale, float lam,
     unsigned long long seed, void* out, long long n, cudaStream_t st);
 int pm_dot_norms(const void* a, const void* b, int bf16, long long n, float* out3, cudaStream_t st);
+
+// ---------------------------------------------------------------- window_attn.cu
+// u [n_tok, ldu]: q [H D], k [G D] and, own_v 1, v [G D] (else the values are the keys before rotation and norm). q_out
+// [n_tok, H, D8] and the cache rows pages[slot] get rotated (first R channels; pairs 1: (2 i, 2 i + 1), else (i, i + R / 2);
+// cs / sn fp32 [n_tok, R / 2]) and, normed 1, normalised vectors.
+int pm_window_prep(const void* u, int f32, long long ldu, const float* cs, const float* sn, int n_tok, int H, int
+    G, int D, int R, int pairs, int normed, float eps, int own_v, void* q_out, void* pages, const long long* slots,
+    cudaStream_t st);
+// Attention of the new tokens q_start[i] .. + q_lens[i] - 1 of n_seq sequences (rows of q [n_tok, H, D8] and out [.., ldo])
+// over their cached keys; sequence i has seq_lens[i] keys behind row i of block_table. few 1: decode tiles (a few rows per
+// sequence), which take n_split > 1 with work buffers po [n_split][n_tok][H][D8] and pml [n_split][n_tok][H][2].
+int pm_window_attn(const void* q, int f32, const void* pages, const int* block_table, const int* seq_lens, const
+    int* q_start, const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H, int G, int D, int
+    window, float scale, int few, int n_split, float* po, float* pml, void* out, long long ldo, cudaStream_t st);
 
 #ifdef __cplusplus
 }

@@ -1,7 +1,9 @@
-// Pieces of decoders whose residual stream is kept in fp32 and normalised after each sum:
+// Pieces of decoders whose residual stream is kept in fp32:
 //   * token embedding times a factor, written as the fp32 stream and as the compute-type copy the projections read
 //   * residual sum + layer norm:  x <- LN(alpha * x + y (+ bias)) * w + b, statistics in fp32 over the row held in
 //     shared memory (the variance is the mean of squared deviations, taken in a second pass)
+//   * residual sum of parallel sublayers + RMS norm of the next layer:  x <- x + y + (sum of a token's expert rows) + x0,
+//     h = x / rms(x) * w; every term but x is optional
 //   * clamped gated unit:  g = min(g, limit), u = clamp(u, -limit, limit), out = g * sigmoid(beta g) * (u + shift)
 //   * rotation table whose angles are formed and reduced in fp64, so that far positions keep fp32-accurate angles
 #include <cuda_bf16.h>
@@ -78,6 +80,69 @@ __global__ void post_layernorm_kernel(const float* x, const T* __restrict__ y, l
   }
 }
 
+struct AddRmsParams {
+  const float* x;
+  const void* y;               // [.., ldy] compute type
+  long long ldy;
+  const void* z;               // [.., width] compute type: rows inv[t * k] .. inv[t * k + k - 1] belong to token t
+  const int* inv;
+  int k;
+  const float* x0;
+  const float* w;
+  float eps;
+  int width;
+  const long long* rows;
+  float* of;
+  void* oc;
+};
+
+// One CTA per output row; `rows` (nullable) picks the input row. of may be x.
+template <typename T, int V>
+__global__ void add_rmsnorm_kernel(const AddRmsParams p) {
+  extern __shared__ __align__(16) float row_buf[];
+  const long long o = blockIdx.x, r = p.rows ? p.rows[o] : o;
+  const T* y = static_cast<const T*>(p.y);
+  const T* z = static_cast<const T*>(p.z);
+  float ss = 0.f;
+  for (int k = threadIdx.x * V; k < p.width; k += blockDim.x * V) {
+    float v[V], s[V];
+    load_vec<V>(p.x + r * p.width + k, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) s[e] = 0.f;
+    if (y) load_vec<V>(y + r * p.ldy + k, s);
+    if (z)
+      for (int j = 0; j < p.k; ++j) {
+        float c[V];
+        load_vec<V>(z + static_cast<long long>(p.inv[r * p.k + j]) * p.width + k, c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s[e] += c[e];
+      }
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] += s[e];
+    if (p.x0) {
+      float c[V];
+      load_vec<V>(p.x0 + r * p.width + k, c);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] += c[e];
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      row_buf[k + e] = v[e];
+      ss = fmaf(v[e], v[e], ss);
+    }
+    if (p.of) store_vec<V>(p.of + o * p.width + k, v);
+  }
+  const float scale = 1.f / sqrtf(block_sum(ss) / static_cast<float>(p.width) + p.eps);
+  T* oc = static_cast<T*>(p.oc);
+  for (int k = threadIdx.x * V; k < p.width; k += blockDim.x * V) {
+    float v[V], ww[V];
+    load_vec<V>(p.w + k, ww);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = row_buf[k + e] * scale * ww[e];
+    store_vec<V>(oc + o * p.width + k, v);
+  }
+}
+
 template <typename T, int V>
 __global__ void clamped_glu_kernel(const T* __restrict__ gu, long long ld, const float* __restrict__ bias, int ff,
                                    float limit, float beta, float shift, T* __restrict__ out, long long n_vec) {
@@ -148,6 +213,19 @@ static int postnorm_launch(const float* x, const void* y, long long ldy, const f
   return static_cast<int>(cudaGetLastError());
 }
 
+template <typename T, int V>
+static int add_rms_launch(const AddRmsParams& p, int n, cudaStream_t st) {
+  const size_t smem = static_cast<size_t>(p.width) * sizeof(float);
+  static DeviceMax configured;
+  if (smem > 40 * 1024 && smem > configured.get()) {
+    const cudaError_t e = cudaFuncSetAttribute(add_rmsnorm_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured.set(200 * 1024);
+  }
+  add_rmsnorm_kernel<T, V><<<n, row_threads(p.width, V), smem, st>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
 template <typename T>
 static int glu_launch(const void* gu, long long ld, const float* bias, int n, int ff, float limit, float beta, float shift,
                       void* out, cudaStream_t st) {
@@ -189,6 +267,20 @@ extern "C" int pm_post_layernorm(const float* x, const void* y, int f32, long lo
                : postnorm_launch<float, 1>(x, y, ldy, bias, alpha, w, b, eps, n, width, rows, of, oc, st);
   return vec ? postnorm_launch<__nv_bfloat16, 4>(x, y, ldy, bias, alpha, w, b, eps, n, width, rows, of, oc, st)
              : postnorm_launch<__nv_bfloat16, 1>(x, y, ldy, bias, alpha, w, b, eps, n, width, rows, of, oc, st);
+}
+
+// v = x + y + sum_j z[inv[t * k + j]] + x0 for the n rows listed in `rows` (nullable: row i); of [n, width] fp32 (nullable, may
+// be x when rows is null) = v, oc [n, width] in the compute type = v / rms(v) * w. y [.., ldy], z [.., width] (compute type,
+// inv int32 per token and j < k) and x0 (fp32) are nullable.
+extern "C" int pm_add_rmsnorm(const float* x, const void* y, int f32, long long ldy, const void* z, const int* inv, int k,
+                              const float* x0, const float* w, float eps, int n, int width, const long long* rows,
+                              float* of, void* oc, cudaStream_t st) {
+  if (n < 0 || width < 1 || static_cast<size_t>(width) * 4 > 200 * 1024 || (rows && of == x) || (z && (!inv || k < 1))) return -1;
+  if (n == 0) return 0;
+  const AddRmsParams p{x, y, ldy, z, inv, k, x0, w, eps, width, rows, of, oc};
+  const bool vec = width % 4 == 0 && ldy % 4 == 0;
+  if (f32) return vec ? add_rms_launch<float, 4>(p, n, st) : add_rms_launch<float, 1>(p, n, st);
+  return vec ? add_rms_launch<__nv_bfloat16, 4>(p, n, st) : add_rms_launch<__nv_bfloat16, 1>(p, n, st);
 }
 
 // gu [n, ld]: gate columns [0, ff), up columns [ff, 2 ff); bias fp32 [2 ff] or null -> out [n, ff].

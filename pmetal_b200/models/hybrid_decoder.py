@@ -1,9 +1,15 @@
-"""Config-driven serving decoder for stacks that mix attention and recurrent layers (Duvivik).
+"""Config-driven serving decoder for stacks that mix attention and recurrent layers (Duvivik, Resevik).
 
-Each layer has a token mixer (``mixers.MIXERS``) and optionally a feed-forward; both sublayers read the stream itself and
-the norm comes after the sum: x <- LN(alpha * x + sublayer(x)). The stream, norms, rotation angles, softmax and recurrent
-states are fp32; projections and their activations run in the model's type (bf16 on the sm_100a kernels, or fp32
-throughout with full-precision matrix products).
+Each layer has a token mixer (``mixers.MIXERS``) and optionally a feed-forward. The design (``DESIGNS``) says how they meet
+the stream:
+
+* ``post``: both sublayers read the stream itself and the norm comes after the sum, x <- LN(alpha * x + sublayer(x));
+* ``parallel``: both read one RMS norm of the stream, x <- x + mixer(h) + ff(h). A span of layers may run several times in a
+  row with the same weights, every run with a cache or state of its own; each pass but the first starts by adding the
+  embedding output to the stream. The sum, the re-added embedding and the next layer's norm are one kernel.
+
+The stream, norms, rotation angles, softmax, routers and recurrent states are fp32; projections and their activations run in
+the model's type (bf16 on the sm_100a kernels, or fp32 throughout with full-precision matrix products).
 
 ``forward_paged`` has the interface of ``DecoderLM.forward_paged``: the new tokens of several sequences in one batch, their
 cache a ``StateCache``, so the generator, the CUDA-graph decoder, the continuous-batching engine and the sampler serve it
@@ -15,7 +21,7 @@ import copy
 import json
 import os
 from dataclasses import dataclass, field
-from typing import Dict, List, Optional
+from typing import Dict, List, Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -23,11 +29,24 @@ import torch.nn as nn
 from ..ops import functional as ops
 from .kv_cache import BLOCK
 from .mixers import MIXERS, RotationFreqs, StepContext, frozen
+from .moe import WeightedInputExperts
 from .state_cache import StateCache
 
 GLU_BETA, GLU_SHIFT = 1.702, 1.0          # gate slope and the offset of the up half in the clamped gated unit
 
-ARCHITECTURES = {"duvivik"}
+
+
+@dataclass(frozen=True)
+class Design:
+    block: str                            # "post" or "parallel"
+    mixers: Tuple[str, ...]
+    feed_forward: str                     # kind of the layers' "mlp" entries
+
+
+DESIGNS: Dict[str, Design] = {
+    "duvivik": Design("post", ("mamba2", "latent_attention"), "dense"),
+    "resevik": Design("parallel", ("lightning", "retention", "attention"), "moe"),
+}
 
 
 @dataclass
@@ -39,6 +58,7 @@ class HybridArgs:
     residual_alpha: float = 1.0
     norm_eps: float = 1e-5
     model_type: str = "duvivik"
+    loop: Optional[Tuple[int, int, int]] = None      # (first layer, layer behind the last, passes)
     bos_token_id: Optional[int] = None
     eos_token_id: Optional[int] = None
     raw: dict = field(default_factory=dict, repr=False)
@@ -47,27 +67,49 @@ class HybridArgs:
     def num_hidden_layers(self) -> int:
         return len(self.layers)
 
+    @property
+    def design(self) -> Design:
+        return DESIGNS[self.model_type]
+
+    @property
+    def runs(self) -> List[Tuple[int, bool]]:
+        """Layers in the order of execution: (layer, whether a further pass of the loop starts with it)."""
+        n = len(self.layers)
+        a, b, times = self.loop or (0, 0, 0)
+        order = [(i, False) for i in range(a)]
+        for t in range(times):
+            order += [(i, t > 0 and i == a) for i in range(a, b)]
+        return order + [(i, False) for i in range(b, n)]
+
     @classmethod
     def from_dict(cls, d: dict) -> "HybridArgs":
         name = str(d.get("architecture", d.get("model_type", ""))).lower()
-        if name not in ARCHITECTURES:
+        if name not in DESIGNS:
             raise ValueError(f"unknown hybrid architecture {name!r}")
+        design = DESIGNS[name]
         layers = [dict(l, mlp=l.get("mlp")) for l in d["layers"]]
         for i, l in enumerate(layers):
-            kind = MIXERS.get(l["type"])
-            if kind is None:
-                raise ValueError(f"layer {i}: unknown mixer {l['type']!r} (known: {', '.join(sorted(MIXERS))})")
+            if l["type"] not in design.mixers:
+                raise ValueError(f"layer {i}: unknown mixer {l['type']!r} (known: {', '.join(design.mixers)})")
+            kind = MIXERS[l["type"]]
             missing = [k for k in kind.KEYS if k not in l["mixer"]]
             if missing:
                 raise ValueError(f"layer {i}: mixer entry lacks {', '.join(missing)}")
             kind.check(l["mixer"], i, layers)
             mlp = l["mlp"]
-            if mlp is not None and mlp.get("kind") != "dense":
+            if mlp is not None and mlp.get("kind") != design.feed_forward:
                 raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+            if mlp is not None and design.feed_forward == "moe":
+                WeightedInputExperts.check(mlp, i)
+        loop = d.get("loop")
+        if loop is not None:
+            loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+            if design.block != "parallel" or not 0 <= loop[0] < loop[1] <= len(layers) or loop[2] < 1:
+                raise ValueError(f"loop {loop} over {len(layers)} layers")
         eos = d.get("eos_token_id")
         return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
                    embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
-                   residual_alpha=float(d.get("postln_alpha", 1.0)), norm_eps=float(d["norm"]["eps"]), model_type=name,
+                   residual_alpha=float(d.get("postln_alpha", 1.0)), norm_eps=float(d["norm"]["eps"]), model_type=name, loop=loop,
                    bos_token_id=d.get("bos_token_id"), eos_token_id=eos[0] if isinstance(eos, list) else eos,
                    raw=copy.deepcopy(d))
 
@@ -99,6 +141,31 @@ def _stack(width: int, vocab: int, ff: int, attn: dict, ssm: dict, pattern: str,
             "norm": {"eps": 1e-5}, "layers": layers}
 
 
+def _parallel_stack(width: int, vocab: int, ff: int, experts: int, top: int, linear: dict, attn: dict, pattern: str,
+                    loop: Optional[Tuple[int, int, int]] = None) -> dict:
+    """Configuration dict: one letter per layer, L = lightning, R = retention, A = windowed attention, all with experts."""
+    h = linear["heads"]
+    kinds = {"L": ("lightning", dict(linear, decay=[1.0 - 2.0 ** (-1.0 - 9.0 * i / max(h - 1, 1)) for i in range(h)])),
+             "R": ("retention", dict(linear, decay=[1.0 - 2.0 ** (-5.0 - 5.0 * i / max(h - 1, 1)) for i in range(h)],
+                                     rot={"base": 10000.0, "dims": linear["dim"]})),
+             "A": ("attention", dict(attn))}
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    d = {"architecture": "Resevik", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5},
+         "layers": [{"type": kinds[c][0], "mixer": copy.deepcopy(kinds[c][1]), "mlp": copy.deepcopy(mlp)} for c in pattern]}
+    if loop:
+        d["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return d
+
+
+def _linear(heads, dim, vdim):
+    return {"heads": heads, "dim": dim, "vdim": vdim}
+
+
+def _window(heads, kv_heads, dim, size):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": size},
+            "rot": {"base": 10000.0, "dims": dim // 2}}
+
+
 def _attn(heads, dim, rot, vdim, rank):
     return {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "scale": (dim + rot) ** -0.5,
             "rot": {"base": 10000.0, "dims": rot}}
@@ -113,6 +180,9 @@ PRESETS: Dict[str, dict] = {
     "duvivik-tiny": _stack(64, 512, 96, _attn(4, 16, 8, 24, 40), _ssm(4, 24, 16, 2, norm_groups=2), "AmaM"),
     "duvivik-1b": _stack(2048, 65536, 6144, _attn(32, 64, 64, 128, 512), _ssm(64, 64, 128, 8, norm_groups=8), "Ammmammm" * 2),
     "duvivik-2b": _stack(2560, 65536, 9728, _attn(32, 96, 32, 128, 512), _ssm(80, 64, 128, 8, norm_groups=8), "Ammmammm" * 4),
+    "resevik-tiny": _parallel_stack(64, 512, 48, 6, 2, _linear(3, 16, 24), _window(4, 2, 20, 40), "LRAL", (0, 3, 2)),
+    # 16 layers, the middle eight twice: 24 layer runs
+    "resevik-2b": _parallel_stack(2048, 65536, 1024, 16, 2, _linear(16, 128, 128), _window(16, 8, 128, 1024), "LRAL" * 4, (4, 12, 2)),
 }
 
 
@@ -183,6 +253,29 @@ class HybridLayer(nn.Module):
         return xf, xc
 
 
+class ParallelLayer(nn.Module):
+    """One norm, read by the mixer and by the experts; the caller sums up (``HybridDecoderLM._parallel``)."""
+
+    def __init__(self, spec: dict, cfg: HybridArgs, index: int, dtype, device):
+        super().__init__()
+        self.cfg = cfg
+        self.mixer = MIXERS[spec["type"]](spec["mixer"], cfg, index, dtype, device)
+        self.mlp = WeightedInputExperts(spec["mlp"], cfg.hidden_size, dtype, device) if spec["mlp"] is not None else None
+        self.norm1_w = frozen(torch.zeros(cfg.hidden_size, device=device))
+
+    def named_weights(self):
+        yield "norm1", (self.cfg.hidden_size,), self.norm1_w.copy_, lambda: self.norm1_w
+        for pre, mod in (("mix.", self.mixer), ("mlp.", self.mlp)):
+            if mod is not None:
+                for name, *rest in mod.named_weights():
+                    yield (pre + name, *rest)
+
+    def forward(self, h, cache, ctx, run):
+        """(mixer output, expert rows, row of every (token, slot), experts per token)."""
+        y = self.mixer(h, cache, ctx, run)
+        return (y, *(self.mlp(h) if self.mlp is not None else (None, None, 1)))
+
+
 class HybridDecoderLM(nn.Module):
     graph_decode = True         # single-token steps can be captured (generation.GraphedDecoder)
     mixed_batches = True        # the scheduler puts prompt portions and decoded tokens into one step
@@ -194,9 +287,12 @@ class HybridDecoderLM(nn.Module):
             raise ValueError("the hybrid decoder runs in bf16 or fp32")
         self.cfg, self.dtype = cfg, dtype
         self.embed_tokens = frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
-        self.layers = nn.ModuleList([HybridLayer(s, cfg, i, dtype, device) for i, s in enumerate(cfg.layers)])
+        self.parallel = cfg.design.block == "parallel"
+        kind = ParallelLayer if self.parallel else HybridLayer
+        self.layers = nn.ModuleList([kind(s, cfg, i, dtype, device) for i, s in enumerate(cfg.layers)])
+        self.runs = cfg.runs
         self.norm_w = frozen(torch.zeros(cfg.hidden_size, device=device))
-        self.norm_b = frozen(torch.zeros(cfg.hidden_size, device=device))
+        self.norm_b = None if self.parallel else frozen(torch.zeros(cfg.hidden_size, device=device))
         self.head = frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
         self._freqs = RotationFreqs()
 
@@ -209,7 +305,8 @@ class HybridDecoderLM(nn.Module):
             for name, *rest in layer.named_weights():
                 yield (f"l{i}.{name}", *rest)
         yield "final.norm", (c.hidden_size,), self.norm_w.copy_, lambda: self.norm_w
-        yield "final.norm.b", (c.hidden_size,), self.norm_b.copy_, lambda: self.norm_b
+        if self.norm_b is not None:
+            yield "final.norm.b", (c.hidden_size,), self.norm_b.copy_, lambda: self.norm_b
         yield "head", (c.vocab_size, c.hidden_size), self.head.copy_, lambda: self.head
 
     @torch.no_grad()
@@ -240,7 +337,9 @@ class HybridDecoderLM(nn.Module):
         for name, shape, put, _ in self.named_weights():
             leaf = name.split(".", 1)[1] if name[0] == "l" and name[1].isdigit() else name
             rnd = lambda: torch.empty(shape, device=device or "cpu")      # noqa: E731
-            if leaf.endswith(".A_log"):
+            if leaf.endswith("mlp.router"):
+                put(rnd().normal_(0.0, 1.0, generator=g).div_(shape[1] ** 0.5))      # logits of order one: spread over the experts
+            elif leaf.endswith(".A_log"):
                 put(rnd().uniform_(1.0, 16.0, generator=g).log_())
             elif leaf.endswith(".dt_bias"):
                 put(rnd().uniform_(-4.6, -2.3, generator=g))
@@ -266,7 +365,7 @@ class HybridDecoderLM(nn.Module):
         if quant or window:
             raise ValueError("the latent / state cache has no quantised or windowed variant")
         p = self.embed_tokens
-        return StateCache([l.mixer.cache_spec() for l in self.layers], num_blocks, max_seqs, dtype or p.dtype,
+        return StateCache([self.layers[i].mixer.cache_spec() for i, _ in self.runs], num_blocks, max_seqs, dtype or p.dtype,
                           device or p.device)
 
     @torch.no_grad()
@@ -294,22 +393,49 @@ class HybridDecoderLM(nn.Module):
     def forward_paged(self, input_ids: torch.Tensor, cache: StateCache, meta, all_logits: bool = False,
                       return_hidden: bool = False, rows: Optional[torch.Tensor] = None, on_layer=None) -> torch.Tensor:
         """Logits (fp32) of the last new token of every sequence, of every new token (``all_logits``) or of the token rows
-        listed in ``rows`` (int64). ``on_layer(i, stream)`` sees the fp32 stream after every layer."""
+        listed in ``rows`` (int64). ``on_layer(i, stream)`` sees the fp32 stream after the i-th layer run."""
         from ..ops import native as nat
         if not self.embed_tokens.is_cuda or not nat.available():
             raise RuntimeError("the hybrid decoder runs on a CUDA device with the native kernel library "
                                f"({nat.load_error() or 'no CUDA device'})")
         cfg = self.cfg
         ctx = StepContext(meta, self._freqs)
+        if rows is None and not all_logits:
+            rows = (meta.q_start + meta.q_lens - 1).long()
         xf, xc = nat.embed_scale(input_ids, self.embed_tokens, cfg.embed_scale)
+        h = (self._parallel if self.parallel else self._post)(xf, xc, cache, ctx, rows, on_layer)
+        if h.shape[0] == 0:
+            return torch.empty(0, h.shape[1] if return_hidden else cfg.vocab_size, dtype=torch.float32, device=h.device)
+        return h if return_hidden else ops.project_f32(h, self.head, cfg.vocab_size)
+
+    def _post(self, xf, xc, cache, ctx, rows, on_layer) -> torch.Tensor:
+        from ..ops import native as nat
         for i, layer in enumerate(self.layers):
             xf, xc = layer(xf, xc, cache, ctx)
             if on_layer is not None:
                 on_layer(i, xf)
-        if rows is None and not all_logits:
-            rows = (meta.q_start + meta.q_lens - 1).long()
         if rows is not None and rows.shape[0] == 0:
-            return torch.empty(0, cfg.vocab_size, dtype=torch.float32, device=xf.device)
-        _, h = nat.post_layernorm(xf, None, self.norm_w, self.norm_b, cfg.norm_eps, rows=rows, want_stream=False,
-                                  dtype=self.dtype)
-        return h if return_hidden else ops.project_f32(h, self.head, cfg.vocab_size)
+            return xc[:0]
+        return nat.post_layernorm(xf, None, self.norm_w, self.norm_b, self.cfg.norm_eps, rows=rows, want_stream=False,
+                                  dtype=self.dtype)[1]
+
+    def _parallel(self, x0, _, cache, ctx, rows, on_layer) -> torch.Tensor:
+        from ..ops import native as nat
+        eps, dt = self.cfg.norm_eps, self.dtype
+        x = x0
+        _, h = nat.add_rmsnorm(x, self.layers[self.runs[0][0]].norm1_w, eps, dtype=dt, want_stream=False)
+        for n, (i, _) in enumerate(self.runs):
+            y, z, inv, k = self.layers[i](h, cache, ctx, n)
+            terms = dict(y=y, z=z, inv=inv, k=k)
+            last = n + 1 == len(self.runs)
+            if on_layer is not None:                       # the stream between the sum and what precedes the next layer
+                x, _ = nat.add_rmsnorm(x, self.norm_w, eps, dtype=dt, **terms)
+                on_layer(n, x)
+                terms = {}
+            if last:
+                if rows is not None and rows.shape[0] == 0:
+                    return h[:0]
+                return nat.add_rmsnorm(x, self.norm_w, eps, rows=rows, dtype=dt, want_stream=False, **terms)[1]
+            nxt, again = self.runs[n + 1]
+            x, h = nat.add_rmsnorm(x, self.layers[nxt].norm1_w, eps, x0=x0 if again else None, dtype=dt,
+                                   out=None if x is x0 or on_layer is not None else x, **terms)

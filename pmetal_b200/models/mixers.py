@@ -1,16 +1,21 @@
 """Token mixers of the config-driven serving decoder (``hybrid_decoder.py``).
 
-A mixer is built from its entry in the configuration, says what it keeps in the cache (``cache_spec``), reads its weights
-through ``take(name, shape)`` and runs on the new tokens of a step: ``forward(x, cache, ctx)`` with x [tokens, width] in
-the compute type returns [tokens, width]. ``MIXERS`` maps the configuration's ``type`` to the class; a new kind of mixer
-is one more entry.
+A mixer is built from its entry in the configuration, says what it keeps in the cache (``cache_spec``), lists its weights
+(``named_weights``) and runs on the new tokens of a step: ``forward(x, cache, ctx, run)`` with x [tokens, width] in the
+compute type returns [tokens, >= width]. ``run`` counts layer runs of the step (the layer's index in stacks without loops) and
+names what the mixer keeps in the cache for this run. ``MIXERS`` maps the configuration's ``type`` to the class; a new kind of
+mixer is one more entry.
 
 ``Mamba2Mixer``          selective state space with one decay per head (csrc/ssm.cu)
 ``LatentAttentionMixer`` multi-head latent attention on cached latents, its own or an earlier layer's (csrc/latent_attn.cu)
+``LinearAttentionMixer`` linear attention with a fixed decay per head; ``LightningMixer`` and ``RetentionMixer`` set its
+                         activation, rotation, norm and gate (csrc/linear_attn.cu)
+``WindowAttentionMixer`` grouped-query attention in a sliding window, keys as values (csrc/window_attn.cu)
 """
 from __future__ import annotations
 
-from typing import Callable, Dict, Optional
+import math
+from typing import Dict, Optional
 
 import torch
 import torch.nn as nn
@@ -73,9 +78,6 @@ class RotationFreqs:
         return self._t[key]
 
 
-Take = Callable[..., torch.Tensor]
-
-
 class Mamba2Mixer(nn.Module):
     """[z | x | B | C | dt] projection, causal convolution + silu on (x, B, C), recurrence, gate before a norm in
     ``norm_groups`` equal parts, output projection."""
@@ -122,9 +124,9 @@ class Mamba2Mixer(nn.Module):
         yield "norm", (self.inner,), self.norm_w.copy_, lambda: self.norm_w
         yield "o", (self.width, self.inner), lambda t: self.w_o[:self.width].copy_(t), lambda: self.w_o[:self.width]
 
-    def forward(self, x: torch.Tensor, cache, ctx: StepContext) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
         from ..ops import native as nat
-        store = cache.slots[self.index]
+        store = cache.slots[self.index if run is None else run]
         u = ops.project(x, self.w_in)
         y = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
         args = (u, self.conv_w, self.conv_b, self.dt_bias, self.a_log, self.dskip, store["conv"], store["state"])
@@ -201,10 +203,10 @@ class LatentAttentionMixer(nn.Module):
             self._ukv8 = torch.nn.functional.pad(self.w_ukv, (0, -r % 8)).contiguous()
         return self._ukv8
 
-    def forward(self, x: torch.Tensor, cache, ctx: StepContext) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
         from ..ops import native as nat
         H, dn, dr, dv, r, W = self.dims
-        pages = cache.pages[self.source]
+        pages = cache.pages[run if self.own and run is not None else self.source]
         qd = ops.project(x, self.w_q)
         cos, sin = ctx.rope(self.base, dr) if dr else (None, None)
         nat.latent_prep(qd, self.norm_w, self.eps, cos, sin, self.dims, pages if self.own else None, ctx.meta.slots)
@@ -220,4 +222,145 @@ class LatentAttentionMixer(nn.Module):
         return ops.project(o, self.w_o)
 
 
-MIXERS = {"mamba2": Mamba2Mixer, "latent_attention": LatentAttentionMixer}
+def check_rotation(m: dict, index: int) -> None:
+    if m["rot"]["dims"] % 2 or not 0 <= m["rot"]["dims"] <= m["dim"]:
+        raise ValueError(f"layer {index}: rot.dims must be even and at most dim")
+
+
+class LinearAttentionMixer(nn.Module):
+    """S <- decay S + k v^T, o = S^T q per head; the heads are RMS-normed (together or one by one), gated and projected."""
+
+    KEYS = ("heads", "dim", "vdim", "decay")
+    SILU = False               # activation of q, k and v
+    ROTATION = "none"          # layout of the rotated pairs of q and k
+    KEY_FACTOR = False         # k times dim^(-1/2)
+    HEAD_NORM = False          # every head by itself and without a weight, else all heads together with a weight
+    SILU_GATE = False          # silu gate, else sigmoid
+
+    @classmethod
+    def check(cls, m: dict, index: int, layers) -> None:
+        if len(m["decay"]) != m["heads"]:
+            raise ValueError(f"layer {index}: {len(m['decay'])} decays for {m['heads']} heads")
+        if not all(0.0 <= float(d) <= 1.0 for d in m["decay"]):
+            raise ValueError(f"layer {index}: decays must lie in [0, 1]")
+        if cls.ROTATION != "none":
+            check_rotation(m, index)
+
+    def __init__(self, m: dict, cfg, index: int, dtype, device):
+        super().__init__()
+        self.H, self.N, self.P = m["heads"], m["dim"], m["vdim"]
+        rot = m["rot"] if self.ROTATION != "none" else {"base": 1.0, "dims": 0}
+        self.base, self.R = float(rot["base"]), int(rot["dims"])
+        self.dims = (self.H, self.N, self.P, self.R, self.ROTATION if self.R else "none", self.SILU)
+        self.kscale = self.N ** -0.5 if self.KEY_FACTOR else 1.0
+        self.eps, self.index, self.width = cfg.norm_eps, index, cfg.hidden_size
+        self.inner, self.n_k = self.H * self.P, self.H * self.N
+        n_in = 2 * self.n_k + 2 * self.inner
+        kw = dict(device=device)
+        self.w_in = frozen(torch.zeros(-(-n_in // 8) * 8, self.width, dtype=dtype, **kw))      # q, k, v, gate
+        self.w_o = frozen(torch.zeros(-(-self.width // 8) * 8, self.inner, dtype=dtype, **kw))
+        self.norm_w = None if self.HEAD_NORM else frozen(torch.zeros(self.inner, **kw))
+        self.decay = frozen(torch.tensor([float(d) for d in m["decay"]], dtype=torch.float64).float().to(device or "cpu"))
+        # a decay below 2^-100 leaves nothing that fp32 sums would show
+        self.log2_decay = frozen(torch.tensor([max(math.log2(d), -100.0) if d > 0 else -100.0 for d in m["decay"]],
+                                              dtype=torch.float64).float().to(device or "cpu"))
+
+    def cache_spec(self) -> CacheSpec:
+        return CacheSpec(slots={"state": ((self.H, self.N, -(-self.P // 4) * 4), torch.float32)})
+
+    def named_weights(self):
+        at = 0
+        for name, n in (("q", self.n_k), ("k", self.n_k), ("v", self.inner), ("g", self.inner)):
+            yield (name, (n, self.width), lambda t, a=at, n=n: self.w_in[a:a + n].copy_(t), lambda a=at, n=n: self.w_in[a:a + n])
+            at += n
+        if self.norm_w is not None:
+            yield "norm", (self.inner,), self.norm_w.copy_, lambda: self.norm_w
+        yield "o", (self.width, self.inner), lambda t: self.w_o[:self.width].copy_(t), lambda: self.w_o[:self.width]
+
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
+        from ..ops import native as nat
+        state = cache.slots[self.index if run is None else run]["state"]
+        u = ops.project(x, self.w_in)
+        cos, sin = ctx.rope(self.base, self.R) if self.R else (None, None)
+        y = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
+        tensor_cores = x.dtype == torch.bfloat16 and nat.linear_chunk_supported(self.N)
+        short, long = ctx.groups(SHORT if tensor_cores else 1 << 30)
+        if short is not None:
+            nat.linear_scan(u, cos, sin, self.decay, self.kscale, state, short, self.dims, y)
+        if long is not None:
+            nat.linear_chunk(u, cos, sin, self.log2_decay, self.kscale, state, long, self.dims, y)
+        gate = u[:, 2 * self.n_k + self.inner:]
+        g = nat.norm_gate(y, gate, self.norm_w, self.eps, self.H if self.HEAD_NORM else 1, self.SILU_GATE)
+        return ops.project(g, self.w_o)
+
+
+class LightningMixer(LinearAttentionMixer):
+    SILU = True
+
+
+class RetentionMixer(LinearAttentionMixer):
+    KEYS = LinearAttentionMixer.KEYS + ("rot",)
+    ROTATION = "half"
+    KEY_FACTOR = HEAD_NORM = SILU_GATE = True
+
+
+class WindowAttentionMixer(nn.Module):
+    """Grouped-query softmax attention over a sliding window. Queries and keys are rotated, then divided by their root mean
+    square over the head; the values are the keys as projected."""
+
+    KEYS = ("heads", "kv_heads", "dim", "vdim", "rot", "mask", "scale")
+    ROTATION = "pairs"
+    UNIT_NORM = True
+    OWN_VALUES = False
+
+    @classmethod
+    def check(cls, m: dict, index: int, layers) -> None:
+        if m["heads"] % m["kv_heads"]:
+            raise ValueError(f"layer {index}: {m['heads']} heads do not divide into {m['kv_heads']} key/value heads")
+        if m["vdim"] != m["dim"]:
+            raise ValueError(f"layer {index}: vdim must equal dim where the values are the keys")
+        if m["dim"] > 1024:
+            raise ValueError(f"layer {index}: heads of more than 1024 channels")
+        if m["mask"].get("size", 0) < 1:
+            raise ValueError(f"layer {index}: mask.size must be at least 1")
+        check_rotation(m, index)
+
+    def __init__(self, m: dict, cfg, index: int, dtype, device):
+        super().__init__()
+        self.dims = (m["heads"], m["kv_heads"], m["dim"])
+        self.base, self.R = float(m["rot"]["base"]), int(m["rot"]["dims"])
+        self.scale, self.window, self.eps = float(m["scale"]), int(m["mask"]["size"]), cfg.norm_eps
+        self.index, self.width = index, cfg.hidden_size
+        self.n_q, self.n_k = m["heads"] * m["dim"], m["kv_heads"] * m["dim"]
+        kw = dict(dtype=dtype, device=device)
+        up8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        self.w_in = frozen(torch.zeros(up8(self.n_q + self.n_k), self.width, **kw))      # queries, keys
+        self.w_o = frozen(torch.zeros(up8(self.width), self.n_q, **kw))
+
+    def cache_spec(self) -> CacheSpec:
+        _, G, D = self.dims
+        return CacheSpec(page_width=2 * G * (-(-D // 8) * 8), window=self.window)
+
+    def named_weights(self):
+        q, k, w = self.n_q, self.n_k, self.width
+        yield "q", (q, w), lambda t: self.w_in[:q].copy_(t), lambda: self.w_in[:q]
+        yield "k", (k, w), lambda t: self.w_in[q:q + k].copy_(t), lambda: self.w_in[q:q + k]
+        yield "o", (w, q), lambda t: self.w_o[:w].copy_(t), lambda: self.w_o[:w]
+
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
+        from ..ops import native as nat
+        pages = cache.pages[self.index if run is None else run]
+        u = ops.project(x, self.w_in)
+        cos, sin = ctx.rope(self.base, self.R) if self.R else (None, None)
+        q = nat.window_prep(u, cos, sin, self.dims, (self.R, self.ROTATION), self.UNIT_NORM, self.eps, self.OWN_VALUES, pages,
+                            ctx.meta.slots)
+        o = torch.empty(x.shape[0], self.n_q, dtype=x.dtype, device=x.device)
+        short, long = ctx.groups(SHORT)
+        for group, few in ((short, True), (long, False)):
+            if group is not None:
+                nat.window_attn(q, pages, group, self.dims, self.window, self.scale, few, o)
+        return ops.project(o, self.w_o)
+
+
+MIXERS = {"mamba2": Mamba2Mixer, "latent_attention": LatentAttentionMixer, "lightning": LightningMixer,
+          "retention": RetentionMixer, "attention": WindowAttentionMixer}

@@ -35,6 +35,61 @@ def sort_by_expert(idx: torch.Tensor, num_experts: int):
     return order, counts, offsets
 
 
+class WeightedInputExperts(nn.Module):
+    """Routed experts for serving whose routing weight multiplies the expert's input: the sum over a token's experts of
+    down_e(silu(G_e w h) * (U_e w h)). Scores are the sigmoid (or softmax) of fp32 router logits, the chosen scores are the
+    weights.
+
+    ``forward`` returns (rows z, row of every (token, slot), experts per token): the caller adds a token's rows up together
+    with the residual. bf16 models run the grouped tensor-core GEMMs, with the token tile chosen from the number of rows per
+    expert; fp32 models and sizes that cannot be copied in 16-byte pieces a row kernel. No step waits for the host."""
+
+    SCORE, RENORM = "sigmoid", False
+    FEW = 128                  # rows per expert up to which the weights are streamed through the narrow-tile kernel
+
+    @classmethod
+    def check(cls, m: dict, index: int) -> None:
+        r = m["router"]
+        if not 1 <= r["top"] <= min(r["experts"], 16) or r["experts"] > 1024:
+            raise ValueError(f"layer {index}: top must lie between 1 and the number of experts (at most 16 of 1024)")
+
+    def __init__(self, m: dict, width: int, dtype, device):
+        super().__init__()
+        self.E, self.k, self.ff, self.width = m["router"]["experts"], m["router"]["top"], m["expert"]["ff"], width
+        new = lambda *s: nn.Parameter(torch.zeros(*s, dtype=dtype, device=device), requires_grad=False)      # noqa: E731
+        self.router = new(-(-self.E // 8) * 8, width)
+        self.gate_up = new(self.E, 2 * self.ff, width)
+        self.down = new(self.E, width, self.ff)
+
+    def named_weights(self):
+        f, w = self.ff, self.width
+        for e in range(self.E):
+            gu, dn = self.gate_up[e], self.down[e]
+            yield f"e{e}.gate", (f, w), gu[:f].copy_, lambda gu=gu: gu[:f]
+            yield f"e{e}.up", (f, w), gu[f:].copy_, lambda gu=gu: gu[f:]
+            yield f"e{e}.down", (w, f), dn.copy_, lambda dn=dn: dn
+        yield "router", (self.E, w), self.router[:self.E].copy_, lambda: self.router[:self.E]
+
+    def forward(self, h: torch.Tensor):
+        from ..ops import functional as ops
+        from ..ops import native as nat
+        r = nat.moe_route(ops.project_f32(h, self.router, self.E), self.k, self.RENORM, score=self.SCORE)
+        T, f, w = h.shape[0], self.ff, self.width
+        if h.dtype != torch.bfloat16 or f % 8 or w % 8:
+            xs, off, dest = nat.expert_gather(h, r, self.k)
+            return nat.expert_rows(nat.expert_rows(xs, self.gate_up, off, glu=True), self.down, off), dest, self.k
+        per = -(-T * self.k // self.E)                     # rows of an expert on average
+        if per <= self.FEW:
+            xs, off, dest = nat.expert_gather(h, r, self.k)
+            tile = min(T, 2 * per)
+            act = nat.grouped_gemm_skinny(xs, self.gate_up, off, swiglu=True, max_rows_per_expert=tile)
+            return nat.grouped_gemm_skinny(act, self.down, off, max_rows_per_expert=tile), dest, self.k
+        xs, off, dest = nat.expert_gather(h, r, self.k, align=128)
+        gu = nat.grouped_gemm(0, xs, self.gate_up, off, 2 * f, w)
+        act = nat.clamped_glu(gu, f, float("inf"), 1.0, 0.0)                        # silu(gate) * up
+        return nat.grouped_gemm(0, act, self.down, off, w, f), dest, self.k
+
+
 class SparseMoeBlock(nn.Module):
     def __init__(self, cfg: ModelArgs, dtype, device):
         super().__init__()

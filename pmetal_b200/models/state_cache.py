@@ -10,7 +10,10 @@ Two kinds of storage on one sequence table:
 
 The last block and the last slot lie outside the pools; padding rows of captured decode steps write there. A recurrent
 state has absorbed every token it saw, so a sequence with slots cannot be cut back (``can_truncate``); ``fork`` copies the
-slot and shares the pages.
+slot and shares the pages. When every layer with pages has a window, pages that lie wholly before the widest of them go back
+to the pool while the sequence lives.
+
+A layer that runs several times in a step (a looped stack) has a spec, pages and slots for every run.
 
 ``split_groups`` divides a step's sequences into short and long portions, which run on different kernels."""
 from __future__ import annotations
@@ -26,8 +29,9 @@ from .kv_cache import BLOCK, BatchMeta, PagedBlocks
 @dataclass
 class CacheSpec:
     """What one layer keeps per token (``page_width`` columns) and per sequence (``slots``: name -> (shape, dtype), a
-    dtype of None is the model's)."""
+    dtype of None is the model's). ``window`` > 0: no token looks back further than to the window - 1 tokens before it."""
     page_width: int = 0
+    window: int = 0
     slots: Dict[str, Tuple[Tuple[int, ...], Optional[torch.dtype]]] = field(default_factory=dict)
 
 
@@ -44,7 +48,9 @@ class StateCache(PagedBlocks):
             if s.slots:
                 self.slots[i] = {n: torch.zeros(max_seqs + 1, *shape, dtype=dt or dtype, device=device)
                                  for n, (shape, dt) in s.slots.items()}
-        self.can_truncate = not self.slots
+        windows = [s.window for s in specs if s.page_width]
+        self.window = max(windows) if windows and min(windows) > 0 else 0
+        self.can_truncate = not self.slots and self.window == 0
         # without recurrent layers nothing is kept per sequence: every sequence names slot 0 and their number is not limited
         self.free_slots: List[int] = list(range(max_seqs - 1, -1, -1))
         self.slot_of: Dict[int, int] = {}
@@ -92,7 +98,7 @@ class StateCache(PagedBlocks):
 
     def truncate(self, seq_id: int, new_len: int) -> None:
         if new_len not in (0, self.seqs[seq_id].length) and not self.can_truncate:
-            raise ValueError("a recurrent state cannot drop tokens it has absorbed")
+            raise ValueError("tokens that a recurrent state has absorbed or a window has left behind cannot be dropped")
         super().truncate(seq_id, new_len)
 
     # ------------------------------------------------------------------ batch metadata

@@ -653,7 +653,7 @@ def project(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 def project_f32(x: torch.Tensor, w: torch.Tensor, n: int) -> torch.Tensor:
     """First ``n`` columns of x w^T as fp32 (read-out)."""
     if x.dtype != torch.bfloat16 or w.shape[1] % 8 or x.stride(0) % 8 or not use_native(x):
-        return F.linear(x, w[:n]).float()
+        return F.linear(x.float(), w[:n].float())
     nat = _native()
     if gemv_fits(x.shape[0], x.shape[1]):
         return nat.gemv_ex(x, w, out_f32=True, n=n)

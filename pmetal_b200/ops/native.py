@@ -972,20 +972,23 @@ def count_tokens(counts, tokens, count_rows=None) -> None:
 
 
 # ------------------------------------------------------------------------------------------- MoE routing
-def moe_route(router_logits, k: int, renorm: bool = True, offsets_out=None):
-    """router_logits [T, E] (bf16 or fp32). Returns dict(topk_idx [T,k], topk_w [T,k], counts [E], offsets [E+1],
-    perm [T*k] (sorted position -> token*k+slot), inv [T*k] (token*k+slot -> sorted position))."""
+def moe_route(router_logits, k: int, renorm: bool = True, offsets_out=None, score: str = "softmax"):
+    """router_logits [T, E] (bf16 or fp32). The k experts with the largest scores (``softmax`` over the experts or the
+    ``sigmoid`` of every logit), weighted by their scores (``renorm``: divided by their sum). Returns dict(topk_idx [T,k],
+    topk_w [T,k], counts [E], offsets [E+1], perm [T*k] (sorted position -> token*k+slot), inv [T*k] (token*k+slot -> sorted
+    position))."""
     T, E = router_logits.shape
     dev = router_logits.device
-    x = router_logits.contiguous()
+    x = router_logits if router_logits.stride(1) == 1 else router_logits.contiguous()
     if x.dtype not in (torch.float32, torch.bfloat16):
         x = x.float()
     out = dict(topk_idx=torch.empty(T, k, dtype=torch.int32, device=dev), topk_w=torch.empty(T, k, dtype=torch.float32, device=dev),
                counts=torch.empty(E, dtype=torch.int32, device=dev), offsets=torch.empty(E + 1, dtype=torch.int32, device=dev),
                perm=torch.empty(T * k, dtype=torch.int32, device=dev), inv=torch.empty(T * k, dtype=torch.int32, device=dev))
-    _chk(lib().pm_moe_route2(_p(x), c_int(int(x.dtype == torch.float32)), c_int(T), c_int(E), c_int(k), c_int(int(renorm)),
+    _chk(lib().pm_moe_route3(_p(x), c_int(int(x.dtype == torch.float32)), c_int(x.stride(0)),
+                             c_int(("softmax", "sigmoid").index(score)), c_int(T), c_int(E), c_int(k), c_int(int(renorm)),
                              _p(out["topk_idx"]), _p(out["topk_w"]), _p(out["counts"]), _p(out["offsets"]),
-                             _p(offsets_out), _p(out["perm"]), _p(out["inv"]), _stream()), "pm_moe_route2")
+                             _p(offsets_out), _p(out["perm"]), _p(out["inv"]), _stream()), "pm_moe_route3")
     return out
 
 
@@ -1003,6 +1006,33 @@ def moe_combine(z, inv, w, k: int, residual=None):
     _chk(lib().pm_moe_combine2(_p(z.contiguous()), _p(inv), _p(w.contiguous()), c_int(k), _p(residual), _p(y), c_ll(T),
                                c_int(H), _stream()), "pm_moe_combine2")
     return y
+
+
+def expert_gather(h, route: dict, k: int, align: int = 0):
+    """Rows of ``h`` [T, H] times their routing weights, sorted by expert (``route`` of ``moe_route``). ``align`` > 0: every
+    expert's slab starts at a multiple of ``align`` rows. Returns (rows, row offsets [E + 1], row of every (token, slot))."""
+    n, E, H = route["perm"].numel(), route["counts"].numel(), h.shape[1]
+    off, dest = route["offsets"], route["inv"]
+    rows = n
+    if align:
+        rows = -(-(n + min(n, E) * (align - 1)) // align) * align      # only experts with rows pad their slab
+        off, dest = torch.empty_like(off), torch.empty_like(dest)
+    xs = torch.empty(rows, H, dtype=h.dtype, device=h.device)
+    _chk(lib().pm_expert_gather(_p(h), _is_f32(h), c_ll(h.stride(0)), _p(route["perm"]), _p(route["topk_w"]),
+                                _p(route["offsets"]), c_int(E), c_int(k), c_int(align), c_int(rows), c_int(H), _p(xs),
+                                _p(off if align else None), _p(dest if align else None), _stream()), "pm_expert_gather")
+    return xs, off, dest
+
+
+def expert_rows(x, w, off, glu: bool = False):
+    """Products of expert-sorted rows x [R, K] with w [E, N, K] on the CUDA cores (any size, fp32 or bf16); ``glu``: w is
+    [E, 2 N, K] (gate rows above up rows) and the result silu(gate) * up."""
+    E, M, K = w.shape
+    N = M // 2 if glu else M
+    out = torch.empty(x.shape[0], N, dtype=x.dtype, device=x.device)
+    _chk(lib().pm_expert_rows(_p(x), _is_f32(x), c_int(x.shape[0]), _p(w), _p(off), c_int(E), c_int(N), c_int(K),
+                              c_int(int(glu)), _p(out), _stream()), "pm_expert_rows")
+    return out
 
 
 # ------------------------------------------------------------------------------------------- GGUF / FP8
@@ -1209,6 +1239,24 @@ def post_layernorm(x, y, w, b, eps: float, alpha: float = 1.0, bias=None, rows=N
     return of, (of if single else oc)
 
 
+def add_rmsnorm(x, w, eps: float, y=None, z=None, inv=None, k: int = 1, x0=None, rows=None, dtype=None,
+                want_stream: bool = True, out=None):
+    """v = x + y + (the k rows z[inv] of every token) + x0 on the fp32 stream x [n, width] -> (v or None, v / rms(v) * w in
+    ``dtype``). y (any row stride) and z have the compute type; x0 is fp32; ``rows`` (int64) picks rows of x, y, z and x0.
+    ``out``: where v goes (may be x when there are no ``rows``)."""
+    n, width = (rows.shape[0] if rows is not None else x.shape[0]), x.shape[1]
+    ct = [t for t in (y, z) if t is not None]
+    dtype = dtype or (ct[0].dtype if ct else x.dtype)
+    if any(t.dtype != dtype or t.stride(1) != 1 for t in ct):
+        raise ValueError("summands must have the compute type and contiguous rows")
+    of = (out if out is not None else torch.empty(n, width, dtype=torch.float32, device=x.device)) if want_stream else None
+    oc = torch.empty(n, width, dtype=dtype, device=x.device)
+    _chk(lib().pm_add_rmsnorm(_p(x), _p(y), c_int(int(dtype == torch.float32)), c_ll(y.stride(0) if y is not None else 0), _p(z),
+                              _p(inv), c_int(k), _p(x0), _p(w), c_float(eps), c_int(n), c_int(width), _p(rows), _p(of), _p(oc),
+                              _stream()), "pm_add_rmsnorm")
+    return of, oc
+
+
 def clamped_glu(gu, ff: int, limit: float, beta: float, shift: float, bias=None):
     """gu [n, >= 2 ff] (gate columns, then up columns), bias fp32 [2 ff] or None -> [n, ff]."""
     out = torch.empty(gu.shape[0], ff, dtype=gu.dtype, device=gu.device)
@@ -1336,3 +1384,81 @@ def latent_expand_attn(qd, wukv, pages, table_row, n_keys: int, dims, scale: flo
     if not direct:
         _chk(lib().pm_latent_take(_p(o), c_int(n_q), c_int(H), c_int(dv), _p(out), c_ll(out.stride(0)), _stream()),
              "pm_latent_take")
+
+
+# ------------------------------------------------------------------------------------------- linear attention, fixed decays
+ROT_LAYOUTS = ("none", "half", "pairs")
+
+
+def linear_scan(u, cs, sn, decay, kscale: float, state, group, dims, y) -> None:
+    """Recurrence token by token for the sequences of ``group``; ``dims`` = (heads, key channels, value channels, rotated
+    channels, rotation layout, silu). Writes the rows of y [tokens, heads * value channels]; layouts in csrc/linear_attn.cu."""
+    H, N, P, R, rot, act = dims
+    _chk(lib().pm_linear_scan(_p(u), _is_f32(u), c_ll(u.stride(0)), _p(cs), _p(sn), _p(decay), c_float(kscale), _p(state),
+                              _p(group.state_slots), _p(group.q_start), _p(group.q_lens), _p(group.seq_lens), c_int(group.n),
+                              c_int(H), c_int(N), c_int(P), c_int(R), c_int(ROT_LAYOUTS.index(rot)), c_int(int(act)), _p(y),
+                              _stream()), "pm_linear_scan")
+
+
+def linear_chunk_supported(n_state: int) -> bool:
+    return n_state <= 256
+
+
+def linear_chunk(u, cs, sn, log2_decay, kscale: float, state, group, dims, y) -> None:
+    """As ``linear_scan`` for longer portions of bf16 models: the recurrence in blocks of 64 tokens on the tensor cores."""
+    global LAUNCHES
+    H, N, P, R, rot, act = dims
+    T, p4 = u.shape[0], -(-P // 4) * 4
+    buf = torch.empty(T, H * P + (4 if R else 2) * H * N, dtype=torch.bfloat16, device=u.device)
+    max_seg = max(1, min(-(-group.max_q // 64), -(-6 * sm_count() // max(-(-P // 32) * H * group.n, 1))))
+    seg = torch.empty(group.n * max_seg * H, N * p4 + 1, dtype=torch.float32, device=u.device)
+    seg_decay = seg.view(-1)[group.n * max_seg * H * N * p4:]
+    _chk(lib().pm_linear_chunk(_p(u), c_ll(u.stride(0)), _p(cs), _p(sn), _p(log2_decay), c_float(kscale), _p(state),
+                               _p(group.state_slots), _p(group.q_start), _p(group.q_lens), _p(group.seq_lens), c_int(group.n),
+                               c_int(T), c_int(group.max_q), c_int(H), c_int(N), c_int(P), c_int(R),
+                               c_int(ROT_LAYOUTS.index(rot)), c_int(int(act)), _p(buf), _p(seg), _p(seg_decay), c_int(max_seg),
+                               _p(y), _stream()), "pm_linear_chunk")
+    LAUNCHES += 1 + int(max_seg > 1)
+
+
+def norm_gate(y, gate, w, eps: float, parts: int, silu: bool):
+    """RMS norm over ``parts`` equal parts of y, times w (fp32, may be None), times silu or sigmoid of ``gate`` (rows of any
+    stride)."""
+    out = torch.empty_like(y)
+    _chk(lib().pm_norm_gate(_p(y), _p(gate), _is_f32(y), c_ll(gate.stride(0)), _p(w), c_float(eps), c_int(parts),
+                            c_int(y.shape[1] // parts), c_int(int(silu)), _p(out), c_int(y.shape[0]), _stream()), "pm_norm_gate")
+    return out
+
+
+# ------------------------------------------------------------------------------------------- windowed attention, any head size
+def window_prep(u, cs, sn, dims, rot, normed: bool, eps: float, own_v: bool, pages, slots):
+    """Rotated and normalised queries [tokens, heads, head size rounded up to 8]; keys and values of the tokens go to their
+    cache rows. ``dims`` = (query heads, key/value heads, head size), ``rot`` = (rotated channels, layout)."""
+    H, G, D = dims
+    q = torch.empty(u.shape[0], H, -(-D // 8) * 8, dtype=u.dtype, device=u.device)
+    _chk(lib().pm_window_prep(_p(u), _is_f32(u), c_ll(u.stride(0)), _p(cs), _p(sn), c_int(u.shape[0]), c_int(H), c_int(G), c_int(D),
+                              c_int(rot[0]), c_int(int(rot[1] == "pairs")), c_int(int(normed)), c_float(eps), c_int(int(own_v)),
+                              _p(q), _p(pages), _p(slots), _stream()), "pm_window_prep")
+    return q
+
+
+def window_attn(q, pages, group, dims, window: int, scale: float, few: bool, out) -> None:
+    """Attention of the sequences of ``group`` over their cached keys; rows of out [tokens, >= heads * head size]. ``few``:
+    tiles for a few rows per sequence, pages split over CTAs."""
+    global LAUNCHES
+    H, G, D = dims
+    T, D8, n_split, po, pml = q.shape[0], q.shape[2], 1, None, None
+    if few and q.dtype == torch.bfloat16 and D8 <= 256:
+        ctas = group.n * G * -(-group.max_q * (H // G) // 16)
+        n_blocks = -(-group.max_kv // 64)
+        if window > 0:
+            n_blocks = min(n_blocks, -(-(window + group.max_q) // 64) + 1)
+        n_split = max(1, min(2 * sm_count() // max(ctas, 1), n_blocks // 2, 32))
+        if n_split > 1:
+            po = torch.empty(n_split, T, H, D8, dtype=torch.float32, device=q.device)
+            pml = torch.empty(n_split, T, H, 2, dtype=torch.float32, device=q.device)
+    _chk(lib().pm_window_attn(_p(q), _is_f32(q), _p(pages), _p(group.block_table), _p(group.seq_lens), _p(group.q_start),
+                              _p(group.q_lens), c_int(group.n), c_int(group.block_table.shape[1]), c_int(T), c_int(group.max_q),
+                              c_int(H), c_int(G), c_int(D), c_int(window), c_float(scale), c_int(int(few)), c_int(n_split), _p(po),
+                              _p(pml), _p(out), c_ll(out.stride(0)), _stream()), "pm_window_attn")
+    LAUNCHES += int(n_split > 1)

@@ -114,7 +114,8 @@ class ContinuousBatchEngine:
         if opts.get("window"):
             prefix_cache = False      # a rotating cache recycles prompt blocks: there is no stable prefix to share
         if not self.gen.cache.can_truncate:
-            prefix_cache = False      # a recurrent state belongs to the whole prefix it has read, not to a part of it
+            # a recurrent state belongs to the whole prefix it has read, not to a part of it; a windowed cache recycles pages
+            prefix_cache = False
         if adapters is not None:
             self.gen.cuda_graphs = False      # the adapter of every row changes from step to step
             prefix_cache = False              # cached keys/values depend on the adapter that produced them

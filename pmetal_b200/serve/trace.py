@@ -61,11 +61,12 @@ def main(argv: Optional[List[str]] = None) -> int:
     from ..models.loader import load_pretrained
     from ..ops import native
     with open(os.path.join(a.model, "config.json"), "r", encoding="utf-8") as fh:
-        fam = family_of(json.load(fh))
+        config = json.load(fh)
+    fam = family_of(config)
     if fam not in PAGED_FAMILIES:
         print(f"error: {fam or 'unknown'} models are not served from the paged caches", file=sys.stderr)
         return 2
-    native.require("hybrid" if fam == "hybrid" else "decoder")
+    native.require(str(config.get("architecture", config.get("model_type"))).lower() if fam == "hybrid" else "decoder")
     if not native.available():
         print(f"error: no CUDA device or native library ({native.load_error()})", file=sys.stderr)
         return 2
