@@ -1,5 +1,8 @@
-"""Serving throughput of the hybrid decoder beside the dense fast decoder at equal size, and its kernels beside the like
-kernels of the existing models (``bench.py --serve-hybrid``). Random weights; device time by CUDA events."""
+"""Serving throughput of the hybrid decoder beside the closest other model at equal size, and its kernels beside the like
+kernels of the other models (``bench.py --serve-hybrid``). Random weights; device time by CUDA events.
+
+Duvivik presets stand beside the dense fast decoder; Resevik presets beside the Qwen3-MoE decoder with the same width, experts
+and attention heads and one layer per layer run (a looped stack has more runs than stored layers)."""
 from __future__ import annotations
 
 import statistics
@@ -25,10 +28,31 @@ DENSE = {
 }
 
 
+def like_kind(name: str) -> str:
+    return "moe" if hd.PRESETS[name]["architecture"] == "Resevik" else "dense"
+
+
 def build(name: str, kind: str):
     args = hd.HybridArgs.from_dict(hd.PRESETS[name])
     if kind == "hybrid":
         return hd.HybridDecoderLM(args, torch.bfloat16, "cuda").init_weights(0.02, 0, "cuda").eval()
+    if kind == "moe":
+        from ..parallel.ep import shard_experts
+        at = next(l["mixer"] for l in args.layers if l["type"] == "attention")
+        ex = next(l["mlp"] for l in args.layers if l["mlp"])
+        cfg = ModelArgs(vocab_size=args.vocab_size, hidden_size=args.hidden_size, num_hidden_layers=len(args.runs),
+                        num_attention_heads=at["heads"], num_key_value_heads=at["kv_heads"], head_dim=128,
+                        intermediate_size=ex["expert"]["ff"], moe_intermediate_size=ex["expert"]["ff"],
+                        num_experts=ex["router"]["experts"], num_experts_per_tok=ex["router"]["top"], tie_word_embeddings=False)
+        m = DecoderLM(cfg, torch.bfloat16, "cuda").init_weights_on_device().eval()
+        for p in m.parameters():
+            p.requires_grad_(False)
+        m.size = sum(p.numel() for p in m.parameters())
+        for layer in m.layers:
+            shard_experts(layer.mlp, None, max_tokens=4096)
+            layer.mlp.gate_up = torch.nn.Parameter(torch.empty(0, dtype=torch.bfloat16, device="cuda"), requires_grad=False)
+            layer.mlp.down = torch.nn.Parameter(torch.empty(0, dtype=torch.bfloat16, device="cuda"), requires_grad=False)
+        return m
     cfg = ModelArgs(vocab_size=args.vocab_size, head_dim=128, tie_word_embeddings=False, **DENSE[name])
     m = DecoderLM(cfg, torch.bfloat16, "cuda").init_weights_on_device().eval()
     for p in m.parameters():
@@ -122,6 +146,108 @@ def _group(cache, n_seq: int, prior: int, new: int):
             cache.reserve(i, prior)
     meta = cache.prepare(list(range(n_seq)), [new] * n_seq)
     return meta, (split_groups(meta, 1 << 30)[0] if isinstance(cache, StateCache) else None)
+
+
+def parallel_kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096) -> List[dict]:
+    """``kernel_cases`` for the parallel stacks (linear attention, windowed attention, experts with weighted inputs)."""
+    from ..models.moe import WeightedInputExperts
+    from ..parallel.ep import FusedExpertMoE
+    cfg = hd.HybridArgs.from_dict(hd.PRESETS[name])
+    W = cfg.hidden_size
+    first = lambda kind: next(l["mixer"] for l in cfg.layers if l["type"] == kind)      # noqa: E731
+    at, lin, ret = first("attention"), first("lightning"), first("retention")
+    ex = next(l["mlp"] for l in cfg.layers if l["mlp"])
+    E, k, ff = ex["router"]["experts"], ex["router"]["top"], ex["expert"]["ff"]
+    H, G, D, win = at["heads"], at["kv_heads"], at["dim"], at["mask"]["size"]
+    pk, out = peaks(), []
+
+    def case(label, fn, nbytes=0, flops=0):
+        us = graph_us(fn)
+        bound = max(nbytes / pk["hbm_gbs"] / 1e3, flops / pk["bf16_tflops"] / 1e6)
+        out.append({"kernel": label, "us": round(us, 2), "bound_us": round(bound, 2), "of_measured_peak": round(bound / us, 3)})
+
+    f = lambda *s: torch.randn(*s, device="cuda")      # noqa: E731
+    experts = WeightedInputExperts(ex, W, torch.bfloat16, "cuda")
+    with torch.no_grad():
+        for t in (experts.gate_up, experts.down):
+            t.normal_(0.0, 0.02)
+        experts.router.normal_(0.0, W ** -0.5)
+    for mode, n_seq, prior, new in (("decode", batch, ctx - 1, 1), ("prefill", 1, 0, prompt)):
+        T, blocks = n_seq * new, n_seq * (prior + new) // BLOCK + n_seq + 1
+        tag = f"{mode} T={T} "
+        # recurrences at the sizes of both linear layers | state-space recurrence of the same state
+        for label, m, rot in (("lightning", lin, 0), ("retention", ret, ret["rot"]["dims"])):
+            LH, N, P = m["heads"], m["dim"], m["vdim"]
+            c = StateCache([CacheSpec(slots={"state": ((LH, N, P), torch.float32)})], blocks, n_seq, torch.bfloat16, "cuda")
+            meta, grp = _group(c, n_seq, prior, new)
+            u, y = _bf(T, 2 * LH * (N + P)), torch.empty(T, LH * P, dtype=torch.bfloat16, device="cuda")
+            cs, sn = (f(T, rot // 2), f(T, rot // 2)) if rot else (None, None)
+            dec = torch.full((LH,), 0.99, device="cuda")
+            fn, d = (nat.linear_scan, dec) if mode == "decode" else (nat.linear_chunk, dec.log2())
+            dims = (LH, N, P, rot, "half" if rot else "none", not rot)
+            state_b = 2 * n_seq * LH * N * P * 4
+            blk = 2 * T * LH * (64 * (N + P) / 2 + 2 * N * P) if mode == "prefill" else 0
+            case(tag + label + " recurrence", lambda: fn(u, cs, sn, d, 1.0, c.slots[0]["state"], grp, dims, y),
+                 T * LH * (2 * N + 2 * P) * 2 + state_b, blk)
+        S = (LH, P, N, LH, 4)
+        inner, conv = LH * P, LH * P + 2 * LH * N
+        c = StateCache([CacheSpec(slots={"conv": ((4, conv), None), "state": ((LH, N, P), torch.float32)})], blocks, n_seq,
+                       torch.bfloat16, "cuda")
+        meta, grp = _group(c, n_seq, prior, new)
+        us = _bf(T, -(-(inner + conv + LH) // 8) * 8)
+        vec = (f(4, conv), f(conv), f(LH) - 3, f(LH), f(LH))
+        sfn = nat.ssm_scan if mode == "decode" else nat.ssm_chunk
+        case(tag + "  | ssm recurrence", lambda: sfn(us, *vec, c.slots[0]["conv"], c.slots[0]["state"], grp, S, y),
+             T * (conv + inner + LH) * 2 + state_b, blk)
+        nw = f(inner)
+        gate = u[:, 2 * LH * N + inner:]
+        case(tag + "norm of all heads + gate", lambda: nat.norm_gate(y, gate, nw, 1e-5, 1, False), 3 * T * inner * 2)
+        case(tag + "norm per head + gate", lambda: nat.norm_gate(y, gate, None, 1e-5, LH, True), 3 * T * inner * 2)
+        case(tag + "  | ssm gate + norm", lambda: nat.ssm_gate_norm(y, us, nw, 1e-5, 8, c.slots[0]["conv"], meta, S), 3 * T * inner * 2)
+        # residual sum with the experts' rows
+        x, yo, z, lw, h = f(T, W), _bf(T, W), _bf(T * k, W), f(W), _bf(T, W)
+        inv = torch.randperm(T * k, device="cuda").int()
+        case(tag + "sum of sublayers + rms norm", lambda: nat.add_rmsnorm(x, lw, 1e-5, y=yo, z=z, inv=inv, k=k, out=x),
+             T * W * (4 + 2 + 2 * k + 4 + 2))
+        rw = _bf(W)
+        case(tag + "  | residual sum + rms norm", lambda: nat.rmsnorm_fwd(h, rw, 1e-6, yo), 4 * T * W * 2)
+        # experts: routing, gather, both products (and the combination) | the same of the MoE decoder
+        eng = FusedExpertMoE(experts.gate_up.data, experts.down.data, E, k, T)
+        used = min(E, T * k)
+        nb, fl = used * 3 * ff * W * 2 + 2 * T * k * (W + ff) * 2, 2 * T * k * 3 * ff * W
+        case(tag + "router, routing and experts", lambda: experts(h), nb, fl)
+        case(tag + "  | router, routing and experts", lambda: eng.forward(h, torch.nn.functional.linear(h, experts.router[:E])), nb, fl)
+        del eng
+        # windowed attention | paged attention in the same window
+        c2 = StateCache([CacheSpec(page_width=2 * G * D)], blocks, n_seq, torch.bfloat16, "cuda")
+        meta, grp = _group(c2, n_seq, prior, new)
+        c2.pages[0].normal_()
+        ua, rd = _bf(T, (H + G) * D), at["rot"]["dims"]
+        cs, sn = f(T, rd // 2), f(T, rd // 2)
+        prep = lambda: nat.window_prep(ua, cs, sn, (H, G, D), (rd, "pairs"), True, 1e-5, False, c2.pages[0], meta.slots)      # noqa: E731
+        case(tag + "rotation + head norm + append", prep, T * (H + G) * D * 2 * 2 + T * G * D * 2)
+        c3 = PagedKVCache(1, G, 128, blocks, device="cuda")
+        meta3, _ = _group(c3, n_seq, prior, new)
+        c3.k[0].normal_()
+        c3.v[0].normal_()
+        qkv, cs3, sn3, w128 = _bf(T, (H + 2 * G) * 128), f(T, 64), f(T, 64), _bf(128)
+        case(tag + "  | rotation + head norm + append",
+             lambda: nat.qknorm_rope_cache(qkv, w128, w128, cs3, sn3, H, G, 1e-6, c3.k[0], c3.v[0], meta3.slots),
+             T * (2 * H + 4 * G) * 128 * 2)
+        q, o = prep(), torch.empty(T, H * D, dtype=torch.bfloat16, device="cuda")
+        if mode == "decode":
+            pairs, keys = n_seq * min(win, ctx), n_seq * min(win, ctx)
+        else:
+            pairs, keys = sum(min(i + 1, win) for i in range(new)), 0
+        case(tag + f"attention in a window of {win}",
+             lambda: nat.window_attn(q, c2.pages[0], grp, (H, G, D), win, 0.09, mode == "decode", o), keys * 2 * G * D * 2, pairs * H * 4 * D)
+        q3 = _bf(T, H, 128)
+        case(tag + "  | paged attention, same window", lambda: nat.paged_attn(q3, c3.k[0], c3.v[0], meta3, 0.09, win),
+             keys * 2 * G * 128 * 2, pairs * H * 4 * 128)
+        del c, c2, c3
+        torch.cuda.empty_cache()
+    nat.check_status()
+    return out
 
 
 def kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096) -> List[dict]:
@@ -218,17 +344,18 @@ def kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096
 
 
 def report(names: List[str], kernels: bool = True) -> dict:
-    """Throughput of every named preset beside the dense decoder of its size, and the kernel cases of the first."""
-    res = {"what": "hybrid decoder beside the dense decoder of equal size", "dtype": "bf16", "data": "synthetic",
+    """Throughput of every named preset beside the closest other model of its size, and the kernel cases of the first."""
+    res = {"what": "hybrid decoder beside the closest other model of equal size", "dtype": "bf16", "data": "synthetic",
            "device": torch.cuda.get_device_name(), "peaks": peaks(), "models": {}}
     for n in names:
         row = {}
-        for kind in ("hybrid", "dense"):
+        for kind in ("hybrid", like_kind(n)):
             m = build(n, kind)
-            row[kind] = {"parameters": sum(p.numel() for p in m.parameters()), **throughput(m)}
+            row[kind] = {"parameters": getattr(m, "size", None) or sum(p.numel() for p in m.parameters()), **throughput(m)}
             del m
             torch.cuda.empty_cache()
         res["models"][n] = row
     if kernels:
-        res["kernels"] = {names[0]: kernel_cases(names[0])}
+        cases = parallel_kernel_cases if like_kind(names[0]) == "moe" else kernel_cases
+        res["kernels"] = {names[0]: cases(names[0])}
     return res

@@ -567,10 +567,11 @@ def _infer_profile_layers(a, model, ids) -> int:
         torch.cuda.synchronize()
     for h in hooks:
         h.remove()
-    start = {i: m for i, k, m in marks if k == "start"}
-    table = []
-    for i, k, m in marks:
-        if k == "end":
+    start, table = {}, []
+    for i, k, m in marks:                                          # a layer of a looped stack has an entry for every run
+        if k == "start":
+            start[i] = m
+        else:
             ms = start[i].elapsed_time(m) if cuda else (m - start[i]) * 1e3
             table.append({"layer": i, "ms": round(ms, 4)})
     rep = {"tokens": len(ids), "total_ms": round(sum(r["ms"] for r in table), 4), "layers": table}
