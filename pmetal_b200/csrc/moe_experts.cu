@@ -2,11 +2,14 @@
 // The (token, slot) pairs come sorted by expert (moe_quant.cu):
 //   expert_gather_kernel   rows w h in sorted order, or in a layout whose slabs start at multiples of `align` rows (zero rows
 //                          between them), for the grouped tensor-core GEMMs (grouped_gemm.cu)
+//   expert_gemv_kernel     a few rows per expert (decode, bf16): every weight row is read once by one warp and multiplied with
+//                          all rows of its expert; fp32 sums, the routing weight applied to them, gated unit inside
 //   expert_rows_kernel     products of sorted rows with their experts' matrices on the CUDA cores, fp32 sums, any size and
 //                          type: fp32 models, and sizes that the GEMMs cannot copy in 16-byte pieces
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
+#include <type_traits>
 #include "elem.cuh"
 #include "host_util.cuh"
 #include "pmetal_b200.h"
@@ -78,6 +81,96 @@ __global__ void __launch_bounds__(128) expert_gather_kernel(const T* __restrict_
   }
 }
 
+struct ExpertGemvParams {
+  const __nv_bfloat16* x;      // GLU: token rows [.., ldx]; else sorted rows
+  long long ldx;
+  const __nv_bfloat16* W;      // [E][N or 2 N][K]
+  const int* perm;             // GLU: pair of every sorted position, its row is pair / k
+  const float* w;              // GLU: weight of every pair
+  const int* off;
+  __nv_bfloat16* out;          // [n, N] in sorted order
+  int n, E, k, N, K;
+};
+
+// grid (channel tiles, sorted positions): the position that begins an expert's slab works for the whole slab. A warp owns four
+// weight rows: two gate / up pairs (GLU) or four output channels.
+template <bool GLU>
+__global__ void __launch_bounds__(128) expert_gemv_kernel(const ExpertGemvParams p) {
+  const int pos0 = blockIdx.y, e = expert_at(p.off, p.E, pos0);
+  if (p.off[e] != pos0) return;
+  const int n_rows = p.off[e + 1] - pos0;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr int kPer = GLU ? 2 : 4;
+  const int c0 = (blockIdx.x * 4 + warp) * kPer;
+  if (c0 >= p.N) return;
+  const __nv_bfloat16* mat = p.W + static_cast<long long>(e) * (GLU ? 2 * p.N : p.N) * p.K;
+  const __nv_bfloat16* wr[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int c = min(c0 + (GLU ? i >> 1 : i), p.N - 1) + (GLU && (i & 1) ? p.N : 0);
+    wr[i] = mat + static_cast<long long>(c) * p.K;
+  }
+  auto pass = [&](auto rows_tag, int r0) {
+    constexpr int R = decltype(rows_tag)::value;
+    const __nv_bfloat16* xr[R];
+    float acc[4][R];
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int pos = pos0 + min(r0 + r, n_rows - 1);
+      xr[r] = p.x + static_cast<long long>(GLU ? p.perm[pos] / p.k : pos) * p.ldx;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i][r] = 0.f;
+    }
+#pragma unroll 2
+    for (int c = lane * 8; c < p.K; c += 256) {
+      uint4 raw[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) raw[i] = __ldg(reinterpret_cast<const uint4*>(wr[i] + c));
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        float xv[8];
+        load_vec<8>(xr[r] + c, xv);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const uint32_t q[4] = {raw[i].x, raw[i].y, raw[i].z, raw[i].w};
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            acc[i][r] = fmaf(__uint_as_float(q[j] << 16), xv[2 * j], acc[i][r]);
+            acc[i][r] = fmaf(__uint_as_float(q[j] & 0xffff0000u), xv[2 * j + 1], acc[i][r]);
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i][r] = warp_sum(acc[i][r]);
+      if (lane == 0 && r0 + r < n_rows) {
+        const int pos = pos0 + r0 + r;
+        __nv_bfloat16* dst = p.out + static_cast<long long>(pos) * p.N + c0;
+        const float f = GLU ? p.w[p.perm[pos]] : 1.f;
+#pragma unroll
+        for (int i = 0; i < kPer; ++i)
+          if (c0 + i < p.N)
+            dst[i] = __float2bfloat16(GLU ? silu_fast(acc[2 * i % 4][r] * f) * (acc[(2 * i + 1) % 4][r] * f) : acc[i][r]);
+      }
+    }
+  };
+  for (int r0 = 0; r0 < n_rows;) {
+    const int left = n_rows - r0;
+    if (left > 2) {
+      pass(std::integral_constant<int, 4>{}, r0);
+      r0 += 4;
+    } else if (left == 2) {
+      pass(std::integral_constant<int, 2>{}, r0);
+      r0 += 2;
+    } else {
+      pass(std::integral_constant<int, 1>{}, r0);
+      r0 += 1;
+    }
+  }
+}
+
 constexpr int kRowTile = 8;
 
 // x [rows, K] sorted, W [E][M][K] -> out [rows, N]: M = N, or with `glu` M = 2 N (gate rows above up rows) and
@@ -145,6 +238,20 @@ extern "C" int pm_expert_gather(const void* h, int f32, long long ldh, const int
   if (rows < 1) return 0;
   return f32 ? gather_launch<float>(h, ldh, perm, w, off, E, k, align, rows, width, xs, off_pad, dest, st)
              : gather_launch<__nv_bfloat16>(h, ldh, perm, w, off, E, k, align, rows, width, xs, off_pad, dest, st);
+}
+
+// Both bf16 products of a step with few rows per expert. glu 1: out [n, N] = silu(w G_e h) * (w U_e h) for the n sorted pairs
+// perm, h [.., ldx] token rows, w [n] weights by pair, W [E][2 N][K]. glu 0: out = x W_e^T for sorted rows x, W [E][N][K].
+// K, ldx and W in 16-byte pieces.
+extern "C" int pm_expert_gemv(const void* x, long long ldx, const void* W, const int* perm, const float* w, const int* off, int n,
+                              int E, int k, int N, int K, int glu, void* out, cudaStream_t st) {
+  if (E < 1 || k < 1 || N < 1 || K < 8 || K % 8 || ldx % 8 || n > 65535 || (glu && (!perm || !w))) return -1;
+  if (n < 1) return 0;
+  const ExpertGemvParams p{static_cast<const __nv_bfloat16*>(x), ldx, static_cast<const __nv_bfloat16*>(W), perm, w, off,
+                           static_cast<__nv_bfloat16*>(out), n, E, k, N, K};
+  if (glu) expert_gemv_kernel<true><<<dim3((N + 7) / 8, n), 128, 0, st>>>(p);
+  else expert_gemv_kernel<false><<<dim3((N + 15) / 16, n), 128, 0, st>>>(p);
+  return static_cast<int>(cudaGetLastError());
 }
 
 // x [rows, K] sorted by expert (off [E + 1], off[E] = rows), W [E][N or, glu 1, 2 N][K] -> out [rows, N] = x W_e^T, or with

@@ -103,8 +103,8 @@ __global__ void moe_router_kernel(const __nv_bfloat16* __restrict__ logits_bf16,
 }
 
 // Few tokens (T * k <= 1024): routing, counting, offsets and the stable sort in one CTA, so that a decode step pays one
-// launch instead of four. Thread e owns expert e and walks the (token, slot) list in order, which keeps the sort stable
-// and deterministic. offsets2 (optional) receives a second copy of the offsets (the expert-parallel exchange buffer).
+// launch instead of four. A warp owns an expert at a time and walks the (token, slot) list in order, which keeps the sort
+// stable and deterministic. offsets2 (optional) receives a second copy of the offsets (the expert-parallel exchange buffer).
 constexpr int kRouteSmallMax = 1024;
 __global__ void __launch_bounds__(1024) moe_route_small_kernel(const __nv_bfloat16* __restrict__ logits_bf16,
                                                                const float* __restrict__ logits_f32, int ldl, int score,
@@ -120,29 +120,47 @@ __global__ void __launch_bounds__(1024) moe_route_small_kernel(const __nv_bfloat
   __syncthreads();
   for (int i = threadIdx.x; i < n; i += blockDim.x) s_idx[i] = topk_idx[i];
   __syncthreads();
-  const int e = threadIdx.x;
-  int c = 0;
-  if (e < E)
-    for (int i = 0; i < n; ++i) c += (s_idx[i] == e);
-  if (e < E) s_off[e + 1] = c;
-  if (e == 0) s_off[0] = 0;
+  for (int e = warp; e < E; e += 32) {
+    int c = 0;
+    for (int i0 = 0; i0 < n; i0 += 32) c += __popc(__ballot_sync(0xffffffffu, i0 + lane < n && s_idx[i0 + lane] == e));
+    if (lane == 0) {
+      counts[e] = c;
+      s_off[e + 1] = c;
+    }
+  }
   __syncthreads();
-  if (threadIdx.x == 0)
-    for (int j = 1; j <= E; ++j) s_off[j] += s_off[j - 1];
+  if (warp == 0) {                                   // running sum of the counts
+    int base = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      int c = e0 + lane < E ? s_off[e0 + lane + 1] : 0;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, c, o);
+        if (lane >= o) c += up;
+      }
+      if (e0 + lane < E) s_off[e0 + lane + 1] = base + c;
+      base += __shfl_sync(0xffffffffu, c, 31);
+    }
+    if (lane == 0) s_off[0] = 0;
+  }
   __syncthreads();
-  if (e <= E) {
+  for (int e = threadIdx.x; e <= E; e += blockDim.x) {
     offsets[e] = s_off[e];
     if (offsets2) offsets2[e] = s_off[e];
   }
-  if (e < E) {
-    counts[e] = c;
+  for (int e = warp; e < E; e += 32) {
     int pos = s_off[e];
-    for (int i = 0; i < n; ++i)
-      if (s_idx[i] == e) {
-        perm[pos] = i;
-        inv[i] = pos;
-        ++pos;
+    if (s_off[e + 1] == pos) continue;
+    for (int i0 = 0; i0 < n; i0 += 32) {
+      const bool hit = i0 + lane < n && s_idx[i0 + lane] == e;
+      const unsigned bm = __ballot_sync(0xffffffffu, hit);
+      if (hit) {
+        const int at = pos + __popc(bm & ((1u << lane) - 1u));
+        perm[at] = i0 + lane;
+        inv[i0 + lane] = at;
       }
+      pos += __popc(bm);
+    }
   }
 }
 

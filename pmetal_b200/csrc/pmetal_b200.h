@@ -275,6 +275,11 @@ int pm_mhc_collapse(const void* xs, int T, int n, int C, void* x, cudaStream_t s
 // pair, rows between slabs are zero; rows must be at least n + (align - 1) per expert with pairs.
 int pm_expert_gather(const void* h, int f32, long long ldh, const int* perm, const float* w, const int* off, int E,
     int k, int align, int rows, int width, void* xs, int* off_pad, int* dest, cudaStream_t st);
+// Both bf16 products of a step with few rows per expert. glu 1: out [n, N] = silu(w G_e h) * (w U_e h) for the n sorted pairs
+// perm, h [.., ldx] token rows, w [n] weights by pair, W [E][2 N][K]. glu 0: out = x W_e^T for sorted rows x, W [E][N][K].
+// K, ldx and W in 16-byte pieces.
+int pm_expert_gemv(const void* x, long long ldx, const void* W, const int* perm, const float* w, const int* off,
+    int n, int E, int k, int N, int K, int glu, void* out, cudaStream_t st);
 // x [rows, K] sorted by expert (off [E + 1], off[E] = rows), W [E][N or, glu 1, 2 N][K] -> out [rows, N] = x W_e^T, or with
 // glu silu(x G_e^T) * (x U_e^T) (gate rows above up rows).
 int pm_expert_rows(const void* x, int f32, int rows, const void* W, const int* off, int E, int N, int K, int glu,

@@ -222,7 +222,9 @@ static int add_rms_launch(const AddRmsParams& p, int n, cudaStream_t st) {
     if (e != cudaSuccess) return static_cast<int>(e);
     configured.set(200 * 1024);
   }
-  add_rmsnorm_kernel<T, V><<<n, row_threads(p.width, V), smem, st>>>(p);
+  int threads = row_threads(p.width, V);
+  if (n < 2 * num_sms() && p.width >= 512 * V) threads = 512;       // few rows: one pass over each
+  add_rmsnorm_kernel<T, V><<<n, threads, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -79,6 +79,63 @@ __global__ void __launch_bounds__(256) window_prep_kernel(const WindowPrepParams
   }
 }
 
+// The same for heads in 8-channel pieces (bf16, D <= 256): a lane owns 8 channels of a head, gs lanes a head (gs: power of two).
+__global__ void __launch_bounds__(256) window_prep_vec_kernel(const WindowPrepParams<__nv_bfloat16> p, int gs) {
+  const int heads = p.H + p.G, lane = threadIdx.x & 31, per = 32 / gs;
+  const long long item = (blockIdx.x * 8ll + (threadIdx.x >> 5)) * per + lane / gs;
+  const long long t = item / heads;
+  const bool live = t < p.n_tok;
+  const int h = live ? static_cast<int>(item - t * heads) : 0, c = (lane % gs) * 8;
+  const bool key = h >= p.H, mine = live && c < p.D;
+  const __nv_bfloat16* src = p.u + (live ? t : 0) * p.ldu + static_cast<long long>(h) * p.D;
+  float v[8], raw[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) raw[e] = 0.f;
+  if (mine) load_vec<8>(src + c, raw);
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    v[e] = raw[e];
+    ss = fmaf(v[e], v[e], ss);
+  }
+  for (int o = gs / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float scale = p.normed ? 1.f / sqrtf(ss / static_cast<float>(p.D) + p.eps) : 1.f;
+  if (!mine) return;
+  const int half = p.R / 2;
+  const float* cs = p.cs + t * half;
+  const float* sn = p.sn + t * half;
+  if (c < p.R) {
+    if (p.pairs) {
+      float a[4], b[4];
+      load_vec<4>(cs + c / 2, a);
+      load_vec<4>(sn + c / 2, b);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        v[2 * i] = fmaf(raw[2 * i], a[i], -raw[2 * i + 1] * b[i]);
+        v[2 * i + 1] = fmaf(raw[2 * i + 1], a[i], raw[2 * i] * b[i]);
+      }
+    } else {
+      const bool second = c >= half;
+      float a[8], b[8], w[8];
+      load_vec<8>(src + (second ? c - half : c + half), w);
+      load_vec<8>(cs + (second ? c - half : c), a);
+      load_vec<8>(sn + (second ? c - half : c), b);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = fmaf(raw[e], a[e], second ? w[e] * b[e] : -w[e] * b[e]);
+    }
+  }
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] *= scale;
+  if (!key) {
+    store_vec<8>(p.q + (t * p.H + h) * p.D8 + c, v);
+    return;
+  }
+  __nv_bfloat16* row = p.pages + (p.slots[t] * p.G + (h - p.H)) * 2 * p.D8 + c;
+  store_vec<8>(row, v);
+  if (p.own_v) load_vec<8>(src + static_cast<long long>(p.G) * p.D + c, raw);
+  store_vec<8>(row + p.D8, raw);
+}
+
 template <typename T>
 struct WindowParams {
   const T* q;                // [tokens, H, D8]
@@ -315,21 +372,32 @@ __global__ void __launch_bounds__(128) window_mma_kernel(const WindowParams<__nv
   }
 }
 
-// Joins the splits: one warp per (token, head) of the sequences in q_start / q_lens. grid (tokens of the longest portion,
+// Joins the splits (at most 32): one warp per (token, head) of the sequences in q_start / q_lens. grid (tokens of the longest portion,
 // heads / 4, sequences).
 __global__ void __launch_bounds__(128) window_combine_kernel(const WindowParams<__nv_bfloat16> p) {
   const int seq = blockIdx.z, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (static_cast<int>(blockIdx.x) >= p.q_lens[seq] || h >= p.H) return;
   const long long t = p.q_start[seq] + blockIdx.x, step = static_cast<long long>(p.n_tok) * p.H, at = t * p.H + h;
-  float m = -CUDART_INF_F;
-  for (int s = 0; s < p.n_split; ++s) m = fmaxf(m, p.pml[(at + s * step) * 2]);
-  float l = 0.f;
-  for (int s = 0; s < p.n_split; ++s) l = fmaf(p.pml[(at + s * step) * 2 + 1], exp2f(p.pml[(at + s * step) * 2] - m), l);
-  const float inv = 1.f / l;
-  for (int c = lane; c < p.D; c += 32) {
-    float v = 0.f;
-    for (int s = 0; s < p.n_split; ++s) v = fmaf(p.po[(at + s * step) * p.D8 + c], exp2f(p.pml[(at + s * step) * 2] - m), v);
-    p.out[t * p.ldo + static_cast<long long>(h) * p.D + c] = __float2bfloat16(v * inv);
+  const float ms = lane < p.n_split ? p.pml[(at + lane * step) * 2] : -CUDART_INF_F;         // lane s: split s
+  const float ls = lane < p.n_split ? p.pml[(at + lane * step) * 2 + 1] : 0.f;
+  float m = ms;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+  float f = exp2f(ms - m);
+  f /= warp_sum(ls * f);
+  for (int c0 = 0; c0 < p.D; c0 += 128) {
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+    for (int s = 0; s < p.n_split; ++s) {
+      const float fs = __shfl_sync(0xffffffffu, f, s);
+      const float* src = p.po + (at + s * step) * p.D8 + c0 + lane;
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (c0 + lane + 32 * i < p.D) v[i] = fmaf(src[32 * i], fs, v[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (c0 + lane + 32 * i < p.D) p.out[t * p.ldo + static_cast<long long>(h) * p.D + c0 + lane + 32 * i] = __float2bfloat16(v[i]);
   }
 }
 
@@ -441,6 +509,16 @@ static int window_prep_launch(const void* u, long long ldu, const float* cs, con
   const WindowPrepParams<T> p{static_cast<const T*>(u), ldu, cs, sn, static_cast<T*>(q), static_cast<T*>(pages), slots, n_tok, H, G,
                               D, (D + 7) / 8 * 8, R, pairs, normed, own_v, eps};
   const long long items = static_cast<long long>(n_tok) * (H + G);
+  const int unit = pairs ? R : R / 2;
+  if constexpr (sizeof(T) == 2) {
+    if (D % 8 == 0 && D <= 256 && ldu % 8 == 0 && unit % 8 == 0 && reinterpret_cast<uintptr_t>(u) % 16 == 0) {
+      int gs = 1;
+      while (gs * 8 < D) gs *= 2;
+      const long long warps = (items + 32 / gs - 1) / (32 / gs);
+      window_prep_vec_kernel<<<static_cast<unsigned>((warps + 7) / 8), 256, 0, st>>>(p, gs);
+      return static_cast<int>(cudaGetLastError());
+    }
+  }
   window_prep_kernel<T><<<static_cast<unsigned>((items + 7) / 8), 256, 0, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
@@ -471,7 +549,7 @@ extern "C" int pm_window_attn(const void* q, int f32, const void* pages, const i
                               const int* q_start, const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H,
                               int G, int D, int window, float scale, int few, int n_split, float* po, float* pml, void* out,
                               long long ldo, cudaStream_t st) {
-  if (window_bad_dims(H, G, D) || window < 0 || n_split < 1 || (n_split > 1 && (!few || !po || !pml))) return -1;
+  if (window_bad_dims(H, G, D) || window < 0 || n_split < 1 || n_split > 32 || (n_split > 1 && (!few || !po || !pml))) return -1;
   if (n_seq < 1 || max_q < 1) return 0;
   if (static_cast<long long>(n_seq) * n_split > 65535) return -2;
   const int D8 = (D + 7) / 8 * 8;

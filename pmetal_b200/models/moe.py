@@ -41,10 +41,11 @@ class WeightedInputExperts(nn.Module):
     weights.
 
     ``forward`` returns (rows z, row of every (token, slot), experts per token): the caller adds a token's rows up together
-    with the residual. bf16 models run the grouped tensor-core GEMMs, with the token tile chosen from the number of rows per
-    expert; fp32 models and sizes that cannot be copied in 16-byte pieces a row kernel. No step waits for the host."""
+    with the residual. bf16 models run mat-vecs on a few rows, then the grouped tensor-core GEMMs, with the token tile chosen
+    from the number of rows per expert; fp32 models and sizes that cannot be copied in 16-byte pieces a row kernel. No step waits for the host."""
 
     SCORE, RENORM = "sigmoid", False
+    GEMV_ROWS, GEMV_PAIRS = 2, 128     # rows per expert and (token, slot) pairs up to which products are mat-vecs
     FEW = 128                  # rows per expert up to which the weights are streamed through the narrow-tile kernel
 
     @classmethod
@@ -79,6 +80,9 @@ class WeightedInputExperts(nn.Module):
             xs, off, dest = nat.expert_gather(h, r, self.k)
             return nat.expert_rows(nat.expert_rows(xs, self.gate_up, off, glu=True), self.down, off), dest, self.k
         per = -(-T * self.k // self.E)                     # rows of an expert on average
+        if per <= self.GEMV_ROWS and T * self.k <= self.GEMV_PAIRS:
+            act = nat.expert_gemv(h, self.gate_up, r, self.k, True)
+            return nat.expert_gemv(act, self.down, r, self.k, False), r["inv"], self.k
         if per <= self.FEW:
             xs, off, dest = nat.expert_gather(h, r, self.k)
             tile = min(T, 2 * per)

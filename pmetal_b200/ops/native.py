@@ -1024,6 +1024,18 @@ def expert_gather(h, route: dict, k: int, align: int = 0):
     return xs, off, dest
 
 
+def expert_gemv(x, w, route: dict, k: int, glu: bool):
+    """One product of a step with few rows per expert (bf16), in sorted order: ``glu`` with token rows x and w [E, 2 N, K] the
+    gated unit of the weighted inputs, else x (sorted rows) times w [E, N, K]."""
+    E, M, K = w.shape
+    N, n = (M // 2 if glu else M), route["perm"].numel()
+    out = torch.empty(n, N, dtype=x.dtype, device=x.device)
+    _chk(lib().pm_expert_gemv(_p(x), c_ll(x.stride(0)), _p(w), _p(route["perm"]), _p(route["topk_w"]), _p(route["offsets"]),
+                              c_int(n), c_int(E), c_int(k), c_int(N), c_int(K), c_int(int(glu)), _p(out), _stream()),
+         "pm_expert_gemv")
+    return out
+
+
 def expert_rows(x, w, off, glu: bool = False):
     """Products of expert-sorted rows x [R, K] with w [E, N, K] on the CUDA cores (any size, fp32 or bf16); ``glu``: w is
     [E, 2 N, K] (gate rows above up rows) and the result silu(gate) * up."""
