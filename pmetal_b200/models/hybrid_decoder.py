@@ -181,7 +181,8 @@ PRESETS: Dict[str, dict] = {
     "duvivik-1b": _stack(2048, 65536, 6144, _attn(32, 64, 64, 128, 512), _ssm(64, 64, 128, 8, norm_groups=8), "Ammmammm" * 2),
     "duvivik-2b": _stack(2560, 65536, 9728, _attn(32, 96, 32, 128, 512), _ssm(80, 64, 128, 8, norm_groups=8), "Ammmammm" * 4),
     "resevik-tiny": _parallel_stack(64, 512, 48, 6, 2, _linear(3, 16, 24), _window(4, 2, 20, 40), "LRAL", (0, 3, 2)),
-    # 16 layers, the middle eight twice: 24 layer runs
+    # 12 layers twice, and 16 layers with the middle eight twice: 24 layer runs each
+    "resevik-1b": _parallel_stack(1536, 65536, 768, 12, 2, _linear(12, 128, 96), _window(12, 4, 96, 512), "LRA" * 4, (0, 12, 2)),
     "resevik-2b": _parallel_stack(2048, 65536, 1024, 16, 2, _linear(16, 128, 128), _window(16, 8, 128, 1024), "LRAL" * 4, (4, 12, 2)),
 }
 

@@ -238,7 +238,7 @@ def test_engine_and_presets_build():
             e.submit(Request([1, 2, 3]))
         e._admit()
         assert len(e.slots) == 3
-    for p in ("resevik-tiny", "resevik-2b"):
+    for p in ("resevik-tiny", "resevik-1b", "resevik-2b"):
         HybridDecoderLM(HybridArgs.from_dict(PRESETS[p]), torch.bfloat16, "meta")
     a, args, d = load_pretrained("random:resevik-tiny", torch.float32)
     assert d is None and args.model_type == "resevik" and float(a.embed_tokens.abs().sum()) > 0
