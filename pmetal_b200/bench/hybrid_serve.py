@@ -224,7 +224,7 @@ def parallel_kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: i
         c2.pages[0].normal_()
         ua, rd = _bf(T, (H + G) * D), at["rot"]["dims"]
         cs, sn = f(T, rd // 2), f(T, rd // 2)
-        prep = lambda: nat.window_prep(ua, cs, sn, (H, G, D), (rd, "pairs"), True, 1e-5, False, c2.pages[0], meta.slots)      # noqa: E731
+        prep = lambda: nat.window_prep(ua, cs, sn, (H, G, 1, D, D), (rd, "pairs"), True, 1e-5, (H * D, H * D), c2.pages[0], meta.slots)      # noqa: E731
         case(tag + "rotation + head norm + append", prep, T * (H + G) * D * 2 * 2 + T * G * D * 2)
         c3 = PagedKVCache(1, G, 128, blocks, device="cuda")
         meta3, _ = _group(c3, n_seq, prior, new)
@@ -240,7 +240,7 @@ def parallel_kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: i
         else:
             pairs, keys = sum(min(i + 1, win) for i in range(new)), 0
         case(tag + f"attention in a window of {win}",
-             lambda: nat.window_attn(q, c2.pages[0], grp, (H, G, D), win, 0.09, mode == "decode", o), keys * 2 * G * D * 2, pairs * H * 4 * D)
+             lambda: nat.window_attn(q, c2.pages[0], grp, (H, G, 1, D, D), win, 0.09, mode == "decode", o), keys * 2 * G * D * 2, pairs * H * 4 * D)
         q3 = _bf(T, H, 128)
         case(tag + "  | paged attention, same window", lambda: nat.paged_attn(q3, c3.k[0], c3.v[0], meta3, 0.09, win),
              keys * 2 * G * 128 * 2, pairs * H * 4 * 128)

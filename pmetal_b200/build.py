@@ -29,6 +29,8 @@ COMPONENTS = {
     "duvivik": ("attention_tc", "gemm_2sm", "gemm_tcgen05", "gemv", "latent_attn", "postnorm", "ssd_chunk", "ssm"),
     "resevik": ("gemm_2sm", "gemm_tcgen05", "gemv", "grouped_gemm", "linear_attn", "moe_experts", "moe_quant", "postnorm",
                 "ssd_chunk", "window_attn"),
+    "vosezen": ("attention_tc", "gemm_2sm", "gemm_tcgen05", "gemv", "grouped_gemm", "latent_attn", "moe_experts", "moe_quant",
+                "postnorm", "window_attn"),
     "decoder": ("attention", "attention_tc", "decode_mega", "elementwise", "gemm_2sm", "gemm_tcgen05", "gemv",
                 "grouped_gemm", "moe_quant"),
 }

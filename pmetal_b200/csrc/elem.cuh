@@ -1,5 +1,5 @@
 // Element access shared by kernels that exist for fp32 and for bf16 activations: scalar and short-vector loads / stores
-// through fp32 registers, a block-wide sum, and the gated unit with clamped inputs.
+// through fp32 registers, a block-wide sum, activations, and the gated unit with clamped inputs.
 #pragma once
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -95,6 +95,7 @@ __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); 
 // The same through the fast exponential and division, for results that are rounded to bf16.
 __device__ __forceinline__ float sigmoid_fast(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
 __device__ __forceinline__ float silu_fast(float v) { return v * sigmoid_fast(v); }
+__device__ __forceinline__ float gelu_f(float v) { return 0.5f * v * erfcf(-0.70710678118654752f * v); }
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
 template <bool kFast = false>

@@ -55,7 +55,7 @@ struct GemvParams {
   int qblock;                    // elements per absmax block (multiple of 32)
   int fp4;
   const float* bias;             // [N_w] fp32 or null, added before the gate
-  int clamped;                   // gate of the SWIGLU variants: 0 silu(g) * u, 1 the clamped unit of elem.cuh
+  int clamped;                   // gate of the SWIGLU variants: 0 silu(g) * u, 1 the clamped unit of elem.cuh; others: 2 exact gelu
   float glu_limit, glu_beta, glu_shift;
   float* y_f32;                  // [M, ldy] instead of y
 };
@@ -71,6 +71,8 @@ __device__ __forceinline__ void gv_finish(const GemvParams& p, int m, int n, flo
     v2 *= p.alpha;
     if (p.bias) v2 += p.bias[n + p.N];
     v = p.clamped ? clamped_glu(v, v2, p.glu_limit, p.glu_beta, p.glu_shift) : gv_silu(v) * v2;
+  } else if (p.clamped == 2) {
+    v = gelu_f(v);
   }
   if (p.residual) v += __bfloat162float(p.residual[static_cast<long long>(m) * p.ldr + n]);
   if (p.y_f32) p.y_f32[static_cast<long long>(m) * p.ldy + n] = v;
@@ -580,7 +582,7 @@ using namespace pm;
 
 // As pm_gemv with the epilogue of models that have biases and clamped gated units: bias [N_w] fp32 (nullable) is added to
 // the scaled products; with swiglu and clamped != 0 the pair becomes min(g, limit) * sigmoid(beta min(g, limit)) *
-// (clamp(u, -limit, limit) + shift); out_f32 != 0: y is fp32.
+// (clamp(u, -limit, limit) + shift); without swiglu, clamped = 2 applies the exact gelu; out_f32 != 0: y is fp32.
 extern "C" int pm_gemv_ex(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps,
                           const void* residual, int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha,
                           const void* t, int ldt, const float* lora_b, int r, const int* seg_end, const float* bias,

@@ -13,6 +13,7 @@
 //
 // Same CTA layout as gemm_tcgen05.cu: warp 0 TMA producer, warp 1 MMA issuer (TMEM double-buffered), warps 2..5
 // epilogue; persistent over the tile list; every wait is bounded.
+#include "elem.cuh"
 #include "gemm_common.cuh"
 #include "pmetal_b200.h"
 
@@ -281,12 +282,12 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 // lane, token in the column). The MMA cost then scales with the token count, the slabs need no padding (a B tile may run
 // into the next expert's rows or past the buffer: those columns are never stored), and the kernel is a pure stream of the
 // weights of the experts that have rows.
-//   plain   Y[r, :] = X[r, :] W_e^T                           W stacked [E*N, K]
+//   plain   Y[r, :] = X[r, :] W_e^T                           W stacked [E*N, K]; with gelu the exact gelu of the products
 //   swiglu  Y[r, :] = silu(X[r, :] G_e^T) * (X[r, :] U_e^T)   W stacked [E*2N, K], rows [G_e (N rows); U_e (N rows)] per
 //           expert; the A tile is 64 rows of G_e on top of the same 64 rows of U_e, and the two halves meet in shared
 //           memory in the epilogue
 struct SkinnyParams {
-  int E, N, K, bn, swiglu;
+  int E, N, K, bn, swiglu, gelu;
   int stages, tmem_cols;
   const int* off;        // [E + 1] row offsets (no alignment)
   __nv_bfloat16* D;
@@ -429,7 +430,10 @@ grouped_gemm_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
               __nv_bfloat16* d = p.D + static_cast<size_t>(lo + t0 + c * 32) * p.ldd + n;
 #pragma unroll
               for (int j = 0; j < 32; ++j)
-                if (c * 32 + j < live) d[static_cast<size_t>(j) * p.ldd] = __float2bfloat16(__uint_as_float(r[j]) * p.alpha);
+                if (c * 32 + j < live) {
+                  const float v = __uint_as_float(r[j]) * p.alpha;
+                  d[static_cast<size_t>(j) * p.ldd] = __float2bfloat16(p.gelu ? gelu_f(v) : v);
+                }
             }
           }
         } else {
@@ -551,15 +555,16 @@ extern "C" int pm_grouped_gemm(int mode, const void* a, int lda, const void* b, 
 }
 
 // Few rows per expert (see the kernel): x [rows, K] expert-sorted with offsets off [E + 1] (any alignment), w stacked
-// [E * N, K] (swiglu 0) or [E * 2N, K] with gate rows above up rows per expert (swiglu 1); y [rows, N] bf16.
+// [E * N, K] (act 0; act 2: exact gelu of the products) or [E * 2N, K] with gate rows above up rows per expert (act 1); y [rows, N] bf16.
 // bn (32, 64, 128) is the token tile: experts with more rows take several passes over their weights.
 extern "C" int pm_grouped_gemm_skinny(const void* x, int ldx, int rows, const void* w, int ldw, void* y, int ldy,
-                                      const int* off, int E, int N, int K, int bn, int swiglu, float alpha, int* status,
+                                      const int* off, int E, int N, int K, int bn, int act, float alpha, int* status,
                                       cudaStream_t stream) {
+  const bool swiglu = act == 1;
   if (E < 1 || rows <= 0 || N <= 0 || K <= 0 || (K % 8) || (ldx % 8) || (ldw % 8)) return -1;
   if (bn != 32 && bn != 64 && bn != 128) return -2;
   SkinnyParams p{};
-  p.E = E; p.N = N; p.K = K; p.bn = bn; p.swiglu = swiglu ? 1 : 0;
+  p.E = E; p.N = N; p.K = K; p.bn = bn; p.swiglu = act == 1; p.gelu = act == 2;
   p.off = off; p.D = static_cast<__nv_bfloat16*>(y); p.ldd = ldy; p.alpha = alpha; p.status = status;
   const int stage_bytes = kBM * kBK * 2 + bn * kBK * 2;
   const int xch_bytes = swiglu ? 64 * (bn + 1) * 4 : 0;

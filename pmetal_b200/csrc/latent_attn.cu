@@ -6,8 +6,9 @@
 // Short portions (decode) move W_uk to the query side: q_l = W_uk^T q_n once per token and head, then every head attends
 // to the cached rows themselves (keys: all W columns, values: the first R), so a step streams the cache once for all
 // heads:
-//   latent_prep_kernel      norm of the latent, rotation of k_r and of the queries' rotated part, cache append
-//   latent_absorb_kernel    [q_l | q_r | 0] rows of width W
+//   latent_prep_kernel      norm of the latent, rotation of k_r and of the queries' rotated part (or norm of the latent that
+//                           the queries come from), cache append
+//   latent_absorb_kernel    [q_l | q_r | 0] rows of width W (q_r turned here where the queries come from a latent)
 //   latent_attn_mma_kernel  bf16, split over key pages: 16 or 32 (token, head) rows share each 64-key page in shared
 //                           memory; S by mma.sync with keys and row quarters cut over the warps (query fragments stay in
 //                           registers), P V with the columns cut over the warps
@@ -52,11 +53,13 @@ __device__ __forceinline__ void load_pair(const __nv_bfloat16* p, float (&v)[V])
   }
 }
 
-// One CTA per token. qd [tokens, ld]: H heads of [D_n | D_r], then (own != 0) the down-projection [R | D_r].
+// One CTA per token. qd [tokens, ld]: H heads of [D_n | D_r] or (lead > 0, H = 0) a query latent of `lead` channels, which is
+// normed in place; then (own != 0) the down-projection [R | D_r].
 template <typename T>
 __global__ void latent_prep_kernel(T* __restrict__ qd, long long ld, const float* __restrict__ norm_w, float eps,
                                    const float* __restrict__ cs, const float* __restrict__ sn, int H, int dn, int dr, int rank,
-                                   int own, T* __restrict__ cache, int W, const long long* __restrict__ slots) {
+                                   int own, T* __restrict__ cache, int W, const long long* __restrict__ slots, int lead,
+                                   const float* __restrict__ lead_w) {
   const long long t = blockIdx.x;
   T* row = qd + t * ld;
   const int half = dr / 2;
@@ -69,8 +72,17 @@ __global__ void latent_prep_kernel(T* __restrict__ qd, long long ld, const float
     put(p, a * c[j] - b * s[j]);
     put(p + 1, b * c[j] + a * s[j]);
   }
+  if (lead > 0) {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < lead; i += blockDim.x) {
+      const float v = to_f(row[i]);
+      ss = fmaf(v, v, ss);
+    }
+    const float r = 1.f / sqrtf(block_sum(ss) / static_cast<float>(lead) + eps);
+    for (int i = threadIdx.x; i < lead; i += blockDim.x) put(row + i, to_f(row[i]) * r * lead_w[i]);
+  }
   if (!own) return;
-  const T* d = row + H * (dn + dr);
+  const T* d = row + H * (dn + dr) + lead;
   T* dst = cache + slots[t] * (W + kRowPad);
   float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) {
@@ -95,7 +107,8 @@ template <typename T, int V>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict__ qd, long long ld, const T* __restrict__ wuk,
                                                             int H, int dn, int dr, int rank, int W, const int* __restrict__ rows,
                                                             int n, T* __restrict__ out, const T* __restrict__ wuv,
-                                                            unsigned wuv_bytes) {
+                                                            unsigned wuv_bytes, const float* __restrict__ cs,
+                                                            const float* __restrict__ sn) {
   extern __shared__ __align__(16) float abs_q[];           // [dn][kAbsTok], then [groups][kAbsTok][128]
   constexpr int kCols = 128 / V, kGroups = 256 / kCols;
   const int h = blockIdx.y, t0 = blockIdx.z * kAbsTok, n_tok = min(kAbsTok, n - t0);
@@ -107,8 +120,17 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict_
     }
     for (int i = threadIdx.x; i < n_tok * tail; i += blockDim.x) {
       const int t = i / tail, j = i - t * tail;
-      put(out + (static_cast<long long>(t0 + t) * H + h) * W + rank + j,
-          j < dr ? to_f(qd[rows[t0 + t] * ld + h * (dn + dr) + dn + j]) : 0.f);
+      float v = 0.f;
+      if (j < dr) {
+        const T* q = qd + rows[t0 + t] * ld + h * (dn + dr) + dn;
+        v = to_f(q[j]);
+        if (cs) {
+          const long long f = static_cast<long long>(rows[t0 + t]) * (dr / 2) + j / 2;
+          const float w = to_f(q[j ^ 1]);
+          v = fmaf(v, cs[f], j & 1 ? w * sn[f] : -w * sn[f]);
+        }
+      }
+      put(out + (static_cast<long long>(t0 + t) * H + h) * W + rank + j, v);
     }
     return;
   }
@@ -648,14 +670,14 @@ static int latent_mma_launch(const LatentParams& p, dim3 grid, size_t smem, cuda
 template <typename T>
 static int latent_absorb_launch(const void* qd, long long ld, const void* wuk, int H, int dn, int dr, int rank, int W,
                                 const int* rows, int n, int tiles, size_t smem, void* out, const void* wuv, int dv,
-                                cudaStream_t st) {
+                                const float* cs, const float* sn, cudaStream_t st) {
   const dim3 grid((rank + 127) / 128 + 1, H, tiles);
   const T *q = static_cast<const T*>(qd), *w = static_cast<const T*>(wuk), *v = static_cast<const T*>(wuv);
   // bulk prefetches take whole 16-byte pieces
   const size_t head = static_cast<size_t>(dv) * rank * sizeof(T);
   const unsigned bytes = head % 16 == 0 && !(reinterpret_cast<uintptr_t>(v) & 15) ? static_cast<unsigned>(head) : 0;
-  if (rank % 2 == 0) latent_absorb_kernel<T, 2><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out), v, bytes);
-  else latent_absorb_kernel<T, 1><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out), v, bytes);
+  if (rank % 2 == 0) latent_absorb_kernel<T, 2><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out), v, bytes, cs, sn);
+  else latent_absorb_kernel<T, 1><<<grid, 256, smem, st>>>(q, ld, w, H, dn, dr, rank, W, rows, n, static_cast<T*>(out), v, bytes, cs, sn);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -676,20 +698,21 @@ static int latent_up_launch(const float* part_o, const float* part_ml, const voi
 using namespace pm;
 
 // qd [n, ld]: the queries' rotated parts are turned in place; with cache != null the down-projection behind the queries is
-// normed / rotated and written to row slots[t] of cache [.., W + 8]. cs / sn [n, dr / 2].
+// normed / rotated and written to row slots[t] of cache [.., W + 8]. cs / sn [n, dr / 2]. lead > 0 (with H = 0): qd begins with
+// a query latent of that many channels, which is normed in place with the weight lead_w (fp32).
 extern "C" int pm_latent_prep(void* qd, int f32, long long ld, const float* norm_w, float eps, const float* cs,
                               const float* sn, int n, int H, int dn, int dr, int rank, void* cache, int W,
-                              const long long* slots, cudaStream_t st) {
-  if (n < 0 || H < 1 || dn < 0 || dr < 0 || (dr & 1) || rank < 1 || W < rank + dr) return -1;
-  if (ld < static_cast<long long>(H) * (dn + dr) + (cache ? rank + dr : 0)) return -2;
+                              const long long* slots, int lead, const float* lead_w, cudaStream_t st) {
+  if (n < 0 || H < 0 || lead < 0 || (H == 0) != (lead > 0) || (lead && !lead_w) || dn < 0 || dr < 0 || (dr & 1) || rank < 1 || W < rank + dr) return -1;
+  if (ld < static_cast<long long>(H) * (dn + dr) + lead + (cache ? rank + dr : 0)) return -2;
   if (n == 0) return 0;
   const int own = cache != nullptr;
   if (f32)
     latent_prep_kernel<float><<<n, 128, 0, st>>>(static_cast<float*>(qd), ld, norm_w, eps, cs, sn, H, dn, dr, rank, own,
-                                                 static_cast<float*>(cache), W, slots);
+                                                 static_cast<float*>(cache), W, slots, lead, lead_w);
   else
     latent_prep_kernel<__nv_bfloat16><<<n, 128, 0, st>>>(static_cast<__nv_bfloat16*>(qd), ld, norm_w, eps, cs, sn, H, dn, dr,
-                                                         rank, own, static_cast<__nv_bfloat16*>(cache), W, slots);
+                                                         rank, own, static_cast<__nv_bfloat16*>(cache), W, slots, lead, lead_w);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -702,12 +725,12 @@ extern "C" int pm_latent_mma_supported(int H, int W, int rank) {
 // cache [pages, 64, W + 8]. The n_tok tokens of the listed sequences are counted through: sequence i covers compact tokens
 // c_start[i] .. of the work buffers q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32 and part_ml [n_split,
 // n_tok * H, 2] fp32, and compact token j is row tok_rows[j] of qd and out. out [.., ldo]: H * dv columns. max_q: longest of
-// q_lens. n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
+// q_lens. cs / sn (nullable) [.., dr / 2]: the queries' rotated parts are still to be turned. n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
 extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void* wuk, const void* wuv, const void* cache,
                               const int* block_table, const int* seq_lens, const int* c_start, const int* q_lens,
                               const int* tok_rows, int n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr,
                               int dv, int rank, int W, int n_split, float scale, void* q_lat, float* part_o, float* part_ml,
-                              void* out, long long ldo, int* status, cudaStream_t st) {
+                              void* out, long long ldo, const float* cs, const float* sn, int* status, cudaStream_t st) {
   if (H < 1 || rank < 1 || W < rank + dr || dv < 1 || n_split < 1 || n_split > 64 || ldo < static_cast<long long>(H) * dv)
     return -1;
   if (n_seq < 1 || max_q < 1 || n_tok < 1) return 0;
@@ -718,8 +741,8 @@ extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void*
   if (sm_abs > 48 * 1024 || (!mma && sm_row > 48 * 1024) || sm_up > 46 * 1024) return -3;
   const int abs_tiles = (n_tok + kAbsTok - 1) / kAbsTok, up_tiles = (n_tok + kUpTok - 1) / kUpTok;
   if (abs_tiles > 65535 || up_tiles > 65535) return -4;
-  int rc = f32 ? latent_absorb_launch<float>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, wuv, dv, st)
-               : latent_absorb_launch<__nv_bfloat16>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, wuv, dv, st);
+  int rc = f32 ? latent_absorb_launch<float>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, wuv, dv, cs, sn, st)
+               : latent_absorb_launch<__nv_bfloat16>(qd, ld, wuk, H, dn, dr, rank, W, tok_rows, n_tok, abs_tiles, sm_abs, q_lat, wuv, dv, cs, sn, st);
   if (rc) return rc;
   LatentParams p{};
   p.q = q_lat; p.cache = cache; p.block_table = block_table; p.seq_lens = seq_lens; p.c_start = c_start; p.q_lens = q_lens;

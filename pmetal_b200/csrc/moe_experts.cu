@@ -1,9 +1,10 @@
-// Routed experts whose weight multiplies the expert's input: y = sum over a token's experts of down(silu(G w h) * (U w h)).
-// The (token, slot) pairs come sorted by expert (moe_quant.cu):
-//   expert_gather_kernel   rows w h in sorted order, or in a layout whose slabs start at multiples of `align` rows (zero rows
+// Routed experts, two forms: a gated unit whose routing weight multiplies the expert's input, y = sum over a token's experts of
+// down(silu(G w h) * (U w h)), and plain units y = sum of w down(gelu(U h)), whose weights the caller applies to the rows.
+// The (token, slot) pairs come sorted by expert (moe_quant.cu); pairs behind the last expert (offsets off[E] ..) are left alone:
+//   expert_gather_kernel   rows w h (or h) in sorted order, or in a layout whose slabs start at multiples of `align` rows (zero rows
 //                          between them), for the grouped tensor-core GEMMs (grouped_gemm.cu)
 //   expert_gemv_kernel     a few rows per expert (decode, bf16): every weight row is read once by one warp and multiplied with
-//                          all rows of its expert; fp32 sums, the routing weight applied to them, gated unit inside
+//                          all rows of its expert; fp32 sums, the routing weight applied to them, activation inside
 //   expert_rows_kernel     products of sorted rows with their experts' matrices on the CUDA cores, fp32 sums, any size and
 //                          type: fp32 models, and sizes that the GEMMs cannot copy in 16-byte pieces
 #include <cuda_bf16.h>
@@ -63,7 +64,7 @@ __global__ void __launch_bounds__(128) expert_gather_kernel(const T* __restrict_
     if (in < off[e + 1] - off[e]) pos = off[e] + in;
   }
   const int pair = pos >= 0 ? perm[pos] : 0;
-  const float f = pos >= 0 ? w[pair] : 0.f;
+  const float f = pos < 0 ? 0.f : w ? w[pair] : 1.f;
   if (align > 0 && pos >= 0 && threadIdx.x == 0) dest[pair] = row;
   const T* src = h + static_cast<long long>(pair / k) * ldh;
   T* dst = xs + static_cast<long long>(row) * width;
@@ -81,12 +82,14 @@ __global__ void __launch_bounds__(128) expert_gather_kernel(const T* __restrict_
   }
 }
 
+enum ExpertAct { kActNone = 0, kActSwiglu = 1, kActGelu = 2 };
+
 struct ExpertGemvParams {
-  const __nv_bfloat16* x;      // GLU: token rows [.., ldx]; else sorted rows
+  const __nv_bfloat16* x;      // kActNone: sorted rows; else token rows [.., ldx]
   long long ldx;
   const __nv_bfloat16* W;      // [E][N or 2 N][K]
-  const int* perm;             // GLU: pair of every sorted position, its row is pair / k
-  const float* w;              // GLU: weight of every pair
+  const int* perm;             // pair of every sorted position, its token row is pair / k
+  const float* w;              // kActSwiglu: weight of every pair
   const int* off;
   __nv_bfloat16* out;          // [n, N] in sorted order
   int n, E, k, N, K;
@@ -94,8 +97,9 @@ struct ExpertGemvParams {
 
 // grid (channel tiles, sorted positions): the position that begins an expert's slab works for the whole slab. A warp owns four
 // weight rows: two gate / up pairs (GLU) or four output channels.
-template <bool GLU>
+template <int ACT>
 __global__ void __launch_bounds__(128) expert_gemv_kernel(const ExpertGemvParams p) {
+  constexpr bool GLU = ACT == kActSwiglu;
   const int pos0 = blockIdx.y, e = expert_at(p.off, p.E, pos0);
   if (p.off[e] != pos0) return;
   const int n_rows = p.off[e + 1] - pos0;
@@ -117,7 +121,7 @@ __global__ void __launch_bounds__(128) expert_gemv_kernel(const ExpertGemvParams
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const int pos = pos0 + min(r0 + r, n_rows - 1);
-      xr[r] = p.x + static_cast<long long>(GLU ? p.perm[pos] / p.k : pos) * p.ldx;
+      xr[r] = p.x + static_cast<long long>(ACT != kActNone ? p.perm[pos] / p.k : pos) * p.ldx;
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[i][r] = 0.f;
     }
@@ -152,7 +156,8 @@ __global__ void __launch_bounds__(128) expert_gemv_kernel(const ExpertGemvParams
 #pragma unroll
         for (int i = 0; i < kPer; ++i)
           if (c0 + i < p.N)
-            dst[i] = __float2bfloat16(GLU ? silu_fast(acc[2 * i % 4][r] * f) * (acc[(2 * i + 1) % 4][r] * f) : acc[i][r]);
+            dst[i] = __float2bfloat16(GLU ? silu_fast(acc[2 * i % 4][r] * f) * (acc[(2 * i + 1) % 4][r] * f)
+                                          : ACT == kActGelu ? gelu_f(acc[i][r]) : acc[i][r]);
       }
     }
   };
@@ -173,13 +178,14 @@ __global__ void __launch_bounds__(128) expert_gemv_kernel(const ExpertGemvParams
 
 constexpr int kRowTile = 8;
 
-// x [rows, K] sorted, W [E][M][K] -> out [rows, N]: M = N, or with `glu` M = 2 N (gate rows above up rows) and
-// out = silu(gate) * up. CTA: 8 rows; warp: one output channel at a time.
+// x [rows, K] sorted, W [E][M][K] -> out [rows, N]: M = N (plain or gelu), or with kActSwiglu M = 2 N (gate rows above up rows)
+// and out = silu(gate) * up. CTA: 8 rows; warp: one output channel at a time.
 template <typename T>
 __global__ void __launch_bounds__(256) expert_rows_kernel(const T* __restrict__ x, int rows, const T* __restrict__ W,
-                                                          const int* __restrict__ off, int E, int N, int K, int glu,
+                                                          const int* __restrict__ off, int E, int N, int K, int act,
                                                           T* __restrict__ out) {
-  const int r0 = blockIdx.y * kRowTile, n_rows = min(kRowTile, rows - r0);
+  const int r0 = blockIdx.y * kRowTile, n_rows = min(kRowTile, min(rows, off[E]) - r0);
+  const bool glu = act == kActSwiglu;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long mat = static_cast<long long>(glu ? 2 * N : N) * K;
   for (int n = blockIdx.x * 8 + warp; n < N; n += gridDim.x * 8) {
@@ -205,7 +211,7 @@ __global__ void __launch_bounds__(256) expert_rows_kernel(const T* __restrict__ 
       for (int i = 0; i < kRowTile; ++i)
         if (a + i < b) {
           const float sg = warp_sum(g[i]), su = glu ? warp_sum(u[i]) : 0.f;
-          if (lane == 0) put(out + static_cast<long long>(r0 + a + i) * N + n, glu ? silu_f(sg) * su : sg);
+          if (lane == 0) put(out + static_cast<long long>(r0 + a + i) * N + n, glu ? silu_f(sg) * su : act == kActGelu ? gelu_f(sg) : sg);
         }
       a = b;
     }
@@ -229,7 +235,7 @@ static int gather_launch(const void* h, long long ldh, const int* perm, const fl
 
 using namespace pm;
 
-// xs [rows, width] = w[pair] * h[pair / k] for the pairs perm[0 .. n) sorted by expert (off [E + 1]). align 0: rows = n in
+// xs [rows, width] = w[pair] * h[pair / k] (w null: h) for the pairs perm[0 .. n) sorted by expert (off [E + 1]). align 0: rows = n in
 // sorted order. align > 0: every expert's slab starts at a multiple of align (off_pad [E + 1]), dest [n] is the row of each
 // pair, rows between slabs are zero; rows must be at least n + (align - 1) per expert with pairs.
 extern "C" int pm_expert_gather(const void* h, int f32, long long ldh, const int* perm, const float* w, const int* off, int E,
@@ -240,25 +246,26 @@ extern "C" int pm_expert_gather(const void* h, int f32, long long ldh, const int
              : gather_launch<__nv_bfloat16>(h, ldh, perm, w, off, E, k, align, rows, width, xs, off_pad, dest, st);
 }
 
-// Both bf16 products of a step with few rows per expert. glu 1: out [n, N] = silu(w G_e h) * (w U_e h) for the n sorted pairs
-// perm, h [.., ldx] token rows, w [n] weights by pair, W [E][2 N][K]. glu 0: out = x W_e^T for sorted rows x, W [E][N][K].
-// K, ldx and W in 16-byte pieces.
+// Both bf16 products of a step with few rows per expert. act 1: out [n, N] = silu(w G_e h) * (w U_e h) for the n sorted pairs
+// perm, h [.., ldx] token rows, w [n] weights by pair, W [E][2 N][K]. act 2: out = gelu(W_e h) for the same pairs, W [E][N][K].
+// act 0: out = x W_e^T for sorted rows x. K, ldx and W in 16-byte pieces.
 extern "C" int pm_expert_gemv(const void* x, long long ldx, const void* W, const int* perm, const float* w, const int* off, int n,
-                              int E, int k, int N, int K, int glu, void* out, cudaStream_t st) {
-  if (E < 1 || k < 1 || N < 1 || K < 8 || K % 8 || ldx % 8 || n > 65535 || (glu && (!perm || !w))) return -1;
+                              int E, int k, int N, int K, int act, void* out, cudaStream_t st) {
+  if (E < 1 || k < 1 || N < 1 || K < 8 || K % 8 || ldx % 8 || n > 65535 || act < 0 || act > 2 || (act && !perm) || (act == 1 && !w)) return -1;
   if (n < 1) return 0;
   const ExpertGemvParams p{static_cast<const __nv_bfloat16*>(x), ldx, static_cast<const __nv_bfloat16*>(W), perm, w, off,
                            static_cast<__nv_bfloat16*>(out), n, E, k, N, K};
-  if (glu) expert_gemv_kernel<true><<<dim3((N + 7) / 8, n), 128, 0, st>>>(p);
-  else expert_gemv_kernel<false><<<dim3((N + 15) / 16, n), 128, 0, st>>>(p);
+  if (act == kActSwiglu) expert_gemv_kernel<kActSwiglu><<<dim3((N + 7) / 8, n), 128, 0, st>>>(p);
+  else if (act == kActGelu) expert_gemv_kernel<kActGelu><<<dim3((N + 15) / 16, n), 128, 0, st>>>(p);
+  else expert_gemv_kernel<kActNone><<<dim3((N + 15) / 16, n), 128, 0, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 
-// x [rows, K] sorted by expert (off [E + 1], off[E] = rows), W [E][N or, glu 1, 2 N][K] -> out [rows, N] = x W_e^T, or with
-// glu silu(x G_e^T) * (x U_e^T) (gate rows above up rows).
-extern "C" int pm_expert_rows(const void* x, int f32, int rows, const void* W, const int* off, int E, int N, int K, int glu,
+// x [rows, K] sorted by expert (off [E + 1]; rows behind off[E] are skipped), W [E][N or, act 1, 2 N][K] -> out [rows, N] =
+// x W_e^T, act 1: silu(x G_e^T) * (x U_e^T) (gate rows above up rows), act 2: gelu(x W_e^T).
+extern "C" int pm_expert_rows(const void* x, int f32, int rows, const void* W, const int* off, int E, int N, int K, int act,
                               void* out, cudaStream_t st) {
-  if (E < 1 || N < 1 || K < 1) return -1;
+  if (E < 1 || N < 1 || K < 1 || act < 0 || act > 2) return -1;
   if (rows < 1) return 0;
   const int tiles = (rows + kRowTile - 1) / kRowTile;
   if (tiles > 65535) return -2;
@@ -266,10 +273,10 @@ extern "C" int pm_expert_rows(const void* x, int f32, int rows, const void* W, c
   const dim3 grid(want < cols ? (want < 1 ? 1 : want) : cols, tiles);
   if (f32)
     expert_rows_kernel<float><<<grid, 256, 0, st>>>(static_cast<const float*>(x), rows, static_cast<const float*>(W), off, E, N, K,
-                                                    glu, static_cast<float*>(out));
+                                                    act, static_cast<float*>(out));
   else
     expert_rows_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(x), rows,
-                                                            static_cast<const __nv_bfloat16*>(W), off, E, N, K, glu,
+                                                            static_cast<const __nv_bfloat16*>(W), off, E, N, K, act,
                                                             static_cast<__nv_bfloat16*>(out));
   return static_cast<int>(cudaGetLastError());
 }

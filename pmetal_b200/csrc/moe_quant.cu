@@ -3,7 +3,7 @@
 // MoE (reference: crates/pmetal-metal/src/kernels/metal/moe_routing.metal — moe_topk_selection,
 // moe_compute_indices, moe_compute_expert_offsets, moe_sort_indices; crates/pmetal-models/src/moe_routing.rs:52-108):
 //   moe_router_kernel   softmax over experts (or the sigmoid of every logit), top-k by repeated warp argmax, optional
-//                       renormalisation of the k weights
+//                       renormalisation of the k weights; the choice may go by corrected scores within the best groups
 //   moe_count_kernel    tokens per expert
 //   moe_scan_kernel     exclusive prefix sum of the counts (one block)
 //   moe_sort_kernel     stable counting sort of the (token, slot) pairs by expert: perm[pos] = token*k + slot,
@@ -25,6 +25,15 @@
 namespace pm {
 
 // ------------------------------------------------------------------------------------------------ MoE routing
+// How a choice differs from the largest scores: the experts form `groups` equal groups of neighbours, of which the `keep` with the
+// largest score + correction are open to it, and among their experts the largest sums win. Weights stay scores, times `factor`.
+struct RouteChoice {
+  const float* correction;      // [E], nullable
+  int groups, keep;             // groups 0: plain choice
+  float factor;
+};
+constexpr int kRouteGroups = 32;
+
 // One warp per token. E <= 1024 experts (NV = ceil(E / 32) per lane, kept in registers), k <= 16.
 // score 0: softmax over the experts, 1: sigmoid. Logit rows are ldl apart.
 template <int NV>
@@ -84,10 +93,100 @@ __device__ __forceinline__ void moe_route_token_nv(const __nv_bfloat16* __restri
   }
 }
 
+// The same with a RouteChoice (at most kRouteGroups groups).
+template <int NV>
+__device__ __forceinline__ void moe_choose_token_nv(const __nv_bfloat16* __restrict__ logits_bf16,
+                                                    const float* __restrict__ logits_f32, int ldl, int score, int t, int E,
+                                                    int k, int renorm, const RouteChoice ch, int* __restrict__ topk_idx,
+                                                    float* __restrict__ topk_w, int lane) {
+  float v[NV], c[NV];
+  float mx = -INFINITY;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int e = i * 32 + lane;
+    v[i] = -INFINITY;
+    if (e < E) v[i] = logits_f32 ? logits_f32[static_cast<long long>(t) * ldl + e]
+                                 : __bfloat162float(logits_bf16[static_cast<long long>(t) * ldl + e]);
+    mx = fmaxf(mx, v[i]);
+  }
+  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+  float z = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const bool in = i * 32 + lane < E;
+    v[i] = !in ? 0.f : score ? 1.f / (1.f + expf(-v[i])) : expf(v[i] - mx);
+    z += v[i];
+  }
+  for (int o = 16; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int e = i * 32 + lane;
+    if (!score) v[i] /= z;
+    c[i] = e < E ? v[i] + (ch.correction ? ch.correction[e] : 0.f) : -INFINITY;
+  }
+  if (ch.keep < ch.groups) {
+    const int per = E / ch.groups;
+    float mine = -INFINITY;                          // lane g: best sum of group g
+    for (int g = 0; g < ch.groups; ++g) {
+      float best = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int e = i * 32 + lane;
+        if (e >= g * per && e < (g + 1) * per) best = fmaxf(best, c[i]);
+      }
+      for (int o = 16; o > 0; o >>= 1) best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, o));
+      if (lane == g) mine = best;
+    }
+    int rank = 0;
+    for (int g = 0; g < ch.groups; ++g) {
+      const float other = __shfl_sync(0xffffffffu, mine, g);
+      rank += other > mine || (other == mine && g < lane);
+    }
+    const unsigned open = __ballot_sync(0xffffffffu, lane < ch.groups && rank < ch.keep);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = i * 32 + lane;
+      if (e >= E || !(open >> (e / per) & 1u)) c[i] = -INFINITY;
+    }
+  }
+  float wsum = 0.f, my_w = 0.f;
+  int my_idx = 0;
+  for (int j = 0; j < k; ++j) {
+    float bv = -INFINITY, bs = 0.f;
+    int bi = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (c[i] > bv) { bv = c[i]; bi = i * 32 + lane; bs = v[i]; }
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o), os = __shfl_xor_sync(0xffffffffu, bs, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; bs = os; }
+    }
+    if (bi >= E) { bi = j; bs = 0.f; }               // logits that are not numbers: any expert, no weight
+    if ((bi & 31) == lane) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (i == (bi >> 5)) c[i] = -INFINITY;
+    }
+    wsum += bs;
+    if (lane == j) { my_w = bs; my_idx = bi; }
+  }
+  if (lane < k) {
+    topk_idx[static_cast<long long>(t) * k + lane] = my_idx;
+    topk_w[static_cast<long long>(t) * k + lane] = (renorm ? my_w / wsum : my_w) * ch.factor;
+  }
+}
+
 __device__ __forceinline__ void moe_route_token(const __nv_bfloat16* __restrict__ logits_bf16,
                                                 const float* __restrict__ logits_f32, int ldl, int score, int t, int E,
-                                                int k, int renorm, int* __restrict__ topk_idx, float* __restrict__ topk_w,
-                                                int lane) {
+                                                int k, int renorm, const RouteChoice ch, int* __restrict__ topk_idx,
+                                                float* __restrict__ topk_w, int lane) {
+  if (ch.groups > 0) {
+    if (E <= 64) moe_choose_token_nv<2>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, ch, topk_idx, topk_w, lane);
+    else if (E <= 256) moe_choose_token_nv<8>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, ch, topk_idx, topk_w, lane);
+    else moe_choose_token_nv<32>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, ch, topk_idx, topk_w, lane);
+    return;
+  }
   if (E <= 64) moe_route_token_nv<2>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
   else if (E <= 128) moe_route_token_nv<4>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
   else if (E <= 256) moe_route_token_nv<8>(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
@@ -95,11 +194,11 @@ __device__ __forceinline__ void moe_route_token(const __nv_bfloat16* __restrict_
 }
 
 __global__ void moe_router_kernel(const __nv_bfloat16* __restrict__ logits_bf16, const float* __restrict__ logits_f32,
-                                  int ldl, int score, int T, int E, int k, int renorm, int* __restrict__ topk_idx,
-                                  float* __restrict__ topk_w) {
+                                  int ldl, int score, int T, int E, int k, int renorm, const RouteChoice ch,
+                                  int* __restrict__ topk_idx, float* __restrict__ topk_w) {
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T) return;
-  moe_route_token(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, threadIdx.x & 31);
+  moe_route_token(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, ch, topk_idx, topk_w, threadIdx.x & 31);
 }
 
 // Few tokens (T * k <= 1024): routing, counting, offsets and the stable sort in one CTA, so that a decode step pays one
@@ -108,15 +207,16 @@ __global__ void moe_router_kernel(const __nv_bfloat16* __restrict__ logits_bf16,
 constexpr int kRouteSmallMax = 1024;
 __global__ void __launch_bounds__(1024) moe_route_small_kernel(const __nv_bfloat16* __restrict__ logits_bf16,
                                                                const float* __restrict__ logits_f32, int ldl, int score,
-                                                               int T, int E, int k, int renorm, int* __restrict__ topk_idx,
-                                                               float* __restrict__ topk_w, int* __restrict__ counts,
+                                                               int T, int E, int k, int renorm, const RouteChoice ch,
+                                                               int* __restrict__ topk_idx, float* __restrict__ topk_w,
+                                                               int* __restrict__ counts,
                                                                int* __restrict__ offsets, int* __restrict__ offsets2,
                                                                int* __restrict__ perm, int* __restrict__ inv) {
   __shared__ int s_idx[kRouteSmallMax];
   __shared__ int s_off[1024 + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = T * k;
   for (int t = warp; t < T; t += 32)
-    moe_route_token(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, topk_idx, topk_w, lane);
+    moe_route_token(logits_bf16, logits_f32, ldl, score, t, E, k, renorm, ch, topk_idx, topk_w, lane);
   __syncthreads();
   for (int i = threadIdx.x; i < n; i += blockDim.x) s_idx[i] = topk_idx[i];
   __syncthreads();
@@ -180,7 +280,8 @@ __global__ void __launch_bounds__(1024) moe_route_local_kernel(const __nv_bfloat
   __shared__ int s_idx[kRouteLocalMax];
   __shared__ int s_off[1024 + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = T * k;
-  for (int t = warp; t < T; t += 32) moe_route_token(logits_bf16, logits_f32, E, 0, t, E, k, renorm, topk_idx, topk_w, lane);
+  for (int t = warp; t < T; t += 32)
+    moe_route_token(logits_bf16, logits_f32, E, 0, t, E, k, renorm, RouteChoice{}, topk_idx, topk_w, lane);
   __syncthreads();
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
     const int x = topk_idx[i];
@@ -516,21 +617,26 @@ static inline int grid_cap(long long work, int per_block, int cap = 0) {
 using namespace pm;
 
 // Routing, counts, offsets and the expert-sorted order of T tokens. Logit rows (fp32 or bf16) are ldl apart; score 0 is the
-// softmax over the experts, 1 the sigmoid of every logit; renorm divides the k weights by their sum. offsets2: optional
-// second destination for the [E + 1] offsets (may be null).
-extern "C" int pm_moe_route3(const void* logits, int is_f32, int ldl, int score, int T, int E, int k, int renorm,
+// softmax over the experts, 1 the sigmoid of every logit; renorm divides the k weights by their sum. groups > 0 (at most 32,
+// dividing E): the choice goes by score + correction (fp32 [E], nullable) among the experts of the `keep` groups of neighbours
+// with the largest such sum, and the weights are multiplied by factor. offsets2: optional second destination for the [E + 1]
+// offsets (may be null).
+extern "C" int pm_moe_route3(const void* logits, int is_f32, int ldl, int score, const float* correction, int groups, int keep,
+                             float factor, int T, int E, int k, int renorm,
                              int* topk_idx, float* topk_w, int* counts, int* offsets, int* offsets2, int* perm, int* inv,
                              cudaStream_t st) {
   if (T <= 0 || E <= 0 || E > 1024 || k <= 0 || k > 16 || k > E || ldl < E || score < 0 || score > 1) return -1;
+  if (groups < 0 || (groups > 0 && (groups > kRouteGroups || E % groups || keep < 1 || keep > groups || keep * (E / groups) < k))) return -1;
+  const RouteChoice ch{correction, groups, keep, factor};
   const long long n = static_cast<long long>(T) * k;
   const __nv_bfloat16* lb = is_f32 ? nullptr : static_cast<const __nv_bfloat16*>(logits);
   const float* lf = is_f32 ? static_cast<const float*>(logits) : nullptr;
   if (n <= kRouteSmallMax && E < 1024) {
-    moe_route_small_kernel<<<1, 1024, 0, st>>>(lb, lf, ldl, score, T, E, k, renorm, topk_idx, topk_w, counts, offsets,
+    moe_route_small_kernel<<<1, 1024, 0, st>>>(lb, lf, ldl, score, T, E, k, renorm, ch, topk_idx, topk_w, counts, offsets,
                                                offsets2, perm, inv);
     return static_cast<int>(cudaGetLastError());
   }
-  moe_router_kernel<<<(T + 7) / 8, 256, 0, st>>>(lb, lf, ldl, score, T, E, k, renorm, topk_idx, topk_w);
+  moe_router_kernel<<<(T + 7) / 8, 256, 0, st>>>(lb, lf, ldl, score, T, E, k, renorm, ch, topk_idx, topk_w);
   moe_count_kernel<<<E, 256, 0, st>>>(topk_idx, n, counts);
   moe_scan_kernel<<<1, 32, 0, st>>>(counts, E, offsets);
   moe_sort_kernel<<<E, 256, 0, st>>>(topk_idx, n, offsets, perm, inv);
@@ -544,7 +650,7 @@ extern "C" int pm_moe_route3(const void* logits, int is_f32, int ldl, int score,
 extern "C" int pm_moe_route2(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx,
                              float* topk_w, int* counts, int* offsets, int* offsets2, int* perm, int* inv,
                              cudaStream_t st) {
-  return pm_moe_route3(logits, is_f32, E, 0, T, E, k, renorm, topk_idx, topk_w, counts, offsets, offsets2, perm, inv, st);
+  return pm_moe_route3(logits, is_f32, E, 0, nullptr, 0, 0, 1.f, T, E, k, renorm, topk_idx, topk_w, counts, offsets, offsets2, perm, inv, st);
 }
 
 extern "C" int pm_moe_route(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx,

@@ -172,7 +172,7 @@ int pm_gemm_bf16(const void* A, int a_mn, int lda, int a_rows, const void* B, in
 // ---------------------------------------------------------------- gemv.cu
 // As pm_gemv with the epilogue of models that have biases and clamped gated units: bias [N_w] fp32 (nullable) is added to
 // the scaled products; with swiglu and clamped != 0 the pair becomes min(g, limit) * sigmoid(beta min(g, limit)) *
-// (clamp(u, -limit, limit) + shift); out_f32 != 0: y is fp32.
+// (clamp(u, -limit, limit) + shift); without swiglu, clamped = 2 applies the exact gelu; out_f32 != 0: y is fp32.
 int pm_gemv_ex(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps, const void* residual,
     int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha, const void* t, int ldt, const float*
     lora_b, int r, const int* seg_end, const float* bias, int clamped, float limit, float beta, float shift, int
@@ -197,27 +197,30 @@ int pm_gemv_q4(const void* x, int ldx, const void* qdata, const float* absmax, c
 int pm_grouped_gemm(int mode, const void* a, int lda, const void* b, int ldb, void* D, int ldd, const int* off, int
     E, int rows_cap, int N, int K, float alpha, int accumulate, int* status, cudaStream_t stream);
 // Few rows per expert (see the kernel): x [rows, K] expert-sorted with offsets off [E + 1] (any alignment), w stacked
-// [E * N, K] (swiglu 0) or [E * 2N, K] with gate rows above up rows per expert (swiglu 1); y [rows, N] bf16.
+// [E * N, K] (act 0; act 2: exact gelu of the products) or [E * 2N, K] with gate rows above up rows per expert (act 1); y [rows, N] bf16.
 // bn (32, 64, 128) is the token tile: experts with more rows take several passes over their weights.
 int pm_grouped_gemm_skinny(const void* x, int ldx, int rows, const void* w, int ldw, void* y, int ldy, const int*
-    off, int E, int N, int K, int bn, int swiglu, float alpha, int* status, cudaStream_t stream);
+    off, int E, int N, int K, int bn, int act, float alpha, int* status, cudaStream_t stream);
 
 // ---------------------------------------------------------------- latent_attn.cu
 // qd [n, ld]: the queries' rotated parts are turned in place; with cache != null the down-projection behind the queries is
-// normed / rotated and written to row slots[t] of cache [.., W + 8]. cs / sn [n, dr / 2].
+// normed / rotated and written to row slots[t] of cache [.., W + 8]. cs / sn [n, dr / 2]. lead > 0 (with H = 0): qd begins with
+// a query latent of that many channels, which is normed in place with the weight lead_w (fp32).
 int pm_latent_prep(void* qd, int f32, long long ld, const float* norm_w, float eps, const float* cs, const float*
-    sn, int n, int H, int dn, int dr, int rank, void* cache, int W, const long long* slots, cudaStream_t st);
+    sn, int n, int H, int dn, int dr, int rank, void* cache, int W, const long long* slots, int lead, const float*
+    lead_w, cudaStream_t st);
 // Whether the tensor-core kernel covers H heads over rows of W columns with `rank` value columns.
 int pm_latent_mma_supported(int H, int W, int rank);
 // Attention of short portions in the latent space. qd as pm_latent_prep leaves it, wuk [H * dn, rank], wuv [H * dv, rank],
 // cache [pages, 64, W + 8]. The n_tok tokens of the listed sequences are counted through: sequence i covers compact tokens
 // c_start[i] .. of the work buffers q_lat [n_tok, H, W], part_o [n_split, n_tok * H, rank] fp32 and part_ml [n_split,
 // n_tok * H, 2] fp32, and compact token j is row tok_rows[j] of qd and out. out [.., ldo]: H * dv columns. max_q: longest of
-// q_lens. n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
+// q_lens. cs / sn (nullable) [.., dr / 2]: the queries' rotated parts are still to be turned. n_split <= 64 (1 for fp32 and for sizes that the tensor-core kernel does not cover).
 int pm_latent_attn(const void* qd, int f32, long long ld, const void* wuk, const void* wuv, const void* cache,
     const int* block_table, const int* seq_lens, const int* c_start, const int* q_lens, const int* tok_rows, int
     n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr, int dv, int rank, int W, int n_split, float
-    scale, void* q_lat, float* part_o, float* part_ml, void* out, long long ldo, int* status, cudaStream_t st);
+    scale, void* q_lat, float* part_o, float* part_ml, void* out, long long ldo, const float* cs, const float* sn,
+    int* status, cudaStream_t st);
 // lat [n, r8] bf16 = latents of positions 0 .. n - 1 of the sequence whose block table row is `table` (zero padded).
 int pm_latent_gather(const void* cache, const int* table, int n, int W, int rank, int r8, void* lat, cudaStream_t
     st);
@@ -270,19 +273,19 @@ int pm_mhc_expand(const void* x, int T, int n, int C, void* xs, cudaStream_t st)
 int pm_mhc_collapse(const void* xs, int T, int n, int C, void* x, cudaStream_t st);
 
 // ---------------------------------------------------------------- moe_experts.cu
-// xs [rows, width] = w[pair] * h[pair / k] for the pairs perm[0 .. n) sorted by expert (off [E + 1]). align 0: rows = n in
+// xs [rows, width] = w[pair] * h[pair / k] (w null: h) for the pairs perm[0 .. n) sorted by expert (off [E + 1]). align 0: rows = n in
 // sorted order. align > 0: every expert's slab starts at a multiple of align (off_pad [E + 1]), dest [n] is the row of each
 // pair, rows between slabs are zero; rows must be at least n + (align - 1) per expert with pairs.
 int pm_expert_gather(const void* h, int f32, long long ldh, const int* perm, const float* w, const int* off, int E,
     int k, int align, int rows, int width, void* xs, int* off_pad, int* dest, cudaStream_t st);
-// Both bf16 products of a step with few rows per expert. glu 1: out [n, N] = silu(w G_e h) * (w U_e h) for the n sorted pairs
-// perm, h [.., ldx] token rows, w [n] weights by pair, W [E][2 N][K]. glu 0: out = x W_e^T for sorted rows x, W [E][N][K].
-// K, ldx and W in 16-byte pieces.
+// Both bf16 products of a step with few rows per expert. act 1: out [n, N] = silu(w G_e h) * (w U_e h) for the n sorted pairs
+// perm, h [.., ldx] token rows, w [n] weights by pair, W [E][2 N][K]. act 2: out = gelu(W_e h) for the same pairs, W [E][N][K].
+// act 0: out = x W_e^T for sorted rows x. K, ldx and W in 16-byte pieces.
 int pm_expert_gemv(const void* x, long long ldx, const void* W, const int* perm, const float* w, const int* off,
-    int n, int E, int k, int N, int K, int glu, void* out, cudaStream_t st);
-// x [rows, K] sorted by expert (off [E + 1], off[E] = rows), W [E][N or, glu 1, 2 N][K] -> out [rows, N] = x W_e^T, or with
-// glu silu(x G_e^T) * (x U_e^T) (gate rows above up rows).
-int pm_expert_rows(const void* x, int f32, int rows, const void* W, const int* off, int E, int N, int K, int glu,
+    int n, int E, int k, int N, int K, int act, void* out, cudaStream_t st);
+// x [rows, K] sorted by expert (off [E + 1]; rows behind off[E] are skipped), W [E][N or, act 1, 2 N][K] -> out [rows, N] =
+// x W_e^T, act 1: silu(x G_e^T) * (x U_e^T) (gate rows above up rows), act 2: gelu(x W_e^T).
+int pm_expert_rows(const void* x, int f32, int rows, const void* W, const int* off, int E, int N, int K, int act,
     void* out, cudaStream_t st);
 
 // ---------------------------------------------------------------- moe_gemm.cu
@@ -300,10 +303,13 @@ int pm_moe_gemm(const void* a, int a_rows, int lda, const void* w, int ldw, int 
 
 // ---------------------------------------------------------------- moe_quant.cu
 // Routing, counts, offsets and the expert-sorted order of T tokens. Logit rows (fp32 or bf16) are ldl apart; score 0 is the
-// softmax over the experts, 1 the sigmoid of every logit; renorm divides the k weights by their sum. offsets2: optional
-// second destination for the [E + 1] offsets (may be null).
-int pm_moe_route3(const void* logits, int is_f32, int ldl, int score, int T, int E, int k, int renorm, int*
-    topk_idx, float* topk_w, int* counts, int* offsets, int* offsets2, int* perm, int* inv, cudaStream_t st);
+// softmax over the experts, 1 the sigmoid of every logit; renorm divides the k weights by their sum. groups > 0 (at most 32,
+// dividing E): the choice goes by score + correction (fp32 [E], nullable) among the experts of the `keep` groups of neighbours
+// with the largest such sum, and the weights are multiplied by factor. offsets2: optional second destination for the [E + 1]
+// offsets (may be null).
+int pm_moe_route3(const void* logits, int is_f32, int ldl, int score, const float* correction, int groups, int
+    keep, float factor, int T, int E, int k, int renorm, int* topk_idx, float* topk_w, int* counts, int* offsets,
+    int* offsets2, int* perm, int* inv, cudaStream_t st);
 int pm_moe_route2(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx, float* topk_w,
     int* counts, int* offsets, int* offsets2, int* perm, int* inv, cudaStream_t st);
 int pm_moe_route(const void* logits, int is_f32, int T, int E, int k, int renorm, int* topk_idx, float* topk_w,
@@ -336,11 +342,18 @@ int pm_post_layernorm(const float* x, const void* y, int f32, long long ldy, con
     float* w, const float* b, float eps, int n, int width, const long long* rows, float* of, void* oc, cudaStream_t
     st);
 // v = x + y + sum_j z[inv[t * k + j]] + x0 for the n rows listed in `rows` (nullable: row i); of [n, width] fp32 (nullable, may
-// be x when rows is null) = v, oc [n, width] in the compute type = v / rms(v) * w. y [.., ldy], z [.., width] (compute type,
+// be x when rows is null) = v, oc [n, width] in the compute type = v / rms(v) * (w_base + w). y [.., ldy], z [.., width] (compute type,
 // inv int32 per token and j < k) and x0 (fp32) are nullable.
 int pm_add_rmsnorm(const float* x, const void* y, int f32, long long ldy, const void* z, const int* inv, int k,
-    const float* x0, const float* w, float eps, int n, int width, const long long* rows, float* of, void* oc,
-    cudaStream_t st);
+    const float* x0, const float* w, float w_base, float eps, int n, int width, const long long* rows, float* of,
+    void* oc, cudaStream_t st);
+// v = x + r / rms(r) * (w_base + w) with r = y + sum over j < k of wt[t, j] * (ids[t, j] < n_experts ? z[row[t, j]] : x[t]); of
+// [n, width] fp32 = v (may be x), oc the same in the compute type (nullable). y [.., ldy] is nullable, k may be 0.
+int pm_add_normed(const float* x, const void* y, int f32, long long ldy, const void* z, const int* row, const int*
+    ids, const float* wt, int k, int n_experts, const float* w, float w_base, float eps, int n, int width, float*
+    of, void* oc, cudaStream_t st);
+// out [n, ldo] = exact gelu of x [n, ldx] on the first `cols` columns; out may be x.
+int pm_gelu(const void* x, int f32, long long ldx, int n, int cols, void* out, long long ldo, cudaStream_t st);
 // gu [n, ld]: gate columns [0, ff), up columns [ff, 2 ff); bias fp32 [2 ff] or null -> out [n, ff].
 int pm_clamped_glu(const void* gu, int f32, long long ld, const float* bias, int n, int ff, float limit, float
     beta, float shift, void* out, cudaStream_t st);
@@ -404,18 +417,26 @@ int pm_merge_fused(const void* const* models, const void* base, const float* wei
 int pm_dot_norms(const void* a, const void* b, int bf16, long long n, float* out3, cudaStream_t st);
 
 // ---------------------------------------------------------------- window_attn.cu
-// u [n_tok, ldu]: q [H D], k [G D] and, own_v 1, v [G D] (else the values are the keys before rotation and norm). q_out
-// [n_tok, H, D8] and the cache rows pages[slot] get rotated (first R channels; pairs 1: (2 i, 2 i + 1), else (i, i + R / 2);
-// cs / sn fp32 [n_tok, R / 2]) and, normed 1, normalised vectors.
+// u [n_tok, ldu]: queries [H][M][D] from column 0 and, with pages, keys [G][M][D] from column k_at and values [G][DV] from
+// column v_at (k_at again: the values are the keys before rotation and norm). q_out [n_tok, H M, D8] and the cache rows
+// pages[slot] get rotated (first R channels; pairs 1: (2 i, 2 i + 1), else (i, i + R / 2); cs / sn fp32 [n_tok, R / 2]) and,
+// normed 1, normalised vectors times qw / kw (fp32 [D], nullable). temp_every > 0: queries at position p = pos[t] are multiplied
+// by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).
 int pm_window_prep(const void* u, int f32, long long ldu, const float* cs, const float* sn, int n_tok, int H, int
-    G, int D, int R, int pairs, int normed, float eps, int own_v, void* q_out, void* pages, const long long* slots,
+    G, int M, int D, int DV, int k_at, int v_at, int R, int pairs, int normed, float eps, const float* qw, const
+    float* kw, const int* pos, float temp_coef, int temp_every, void* q_out, void* pages, const long long* slots,
     cudaStream_t st);
-// Attention of the new tokens q_start[i] .. + q_lens[i] - 1 of n_seq sequences (rows of q [n_tok, H, D8] and out [.., ldo])
-// over their cached keys; sequence i has seq_lens[i] keys behind row i of block_table. few 1: decode tiles (a few rows per
-// sequence), which take n_split > 1 with work buffers po [n_split][n_tok][H][D8] and pml [n_split][n_tok][H][2].
+// Attention of the new tokens q_start[i] .. + q_lens[i] - 1 of n_seq sequences (rows of q [n_tok, H M, D8] and out [.., ldo])
+// over their cached keys; sequence i has seq_lens[i] keys behind row i of block_table. Scores times scale, capped when
+// softcap > 0; sink (fp32 [H], M = 1) adds exp(sink) to a head's softmax sum; gate [.., ldg] multiplies head h by the sigmoid of
+// column h. M = 2: the result of a head is a_1 - lambda[0] a_2 over its root mean square (eps inside), times keep; it takes o
+// [n_tok, H M, DV] in the compute type unless parts are given. few 1: decode tiles (a few rows per sequence), which take work
+// buffers po [n_split][n_tok][H M][DV8] and pml [n_split][n_tok][H M][2] (both or none; needed for n_split > 1).
 int pm_window_attn(const void* q, int f32, const void* pages, const int* block_table, const int* seq_lens, const
-    int* q_start, const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H, int G, int D, int
-    window, float scale, int few, int n_split, float* po, float* pml, void* out, long long ldo, cudaStream_t st);
+    int* q_start, const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H, int G, int M, int D,
+    int DV, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg, const
+    float* lambda, float keep, float eps, int few, int n_split, float* po, float* pml, void* o, void* out, long
+    long ldo, cudaStream_t st);
 
 #ifdef __cplusplus
 }

@@ -4,6 +4,9 @@
 //     shared memory (the variance is the mean of squared deviations, taken in a second pass)
 //   * residual sum of parallel sublayers + RMS norm of the next layer:  x <- x + y + (sum of a token's expert rows) + x0,
 //     h = x / rms(x) * w; every term but x is optional
+//   * norm of a sublayer's result ahead of the residual sum:  x <- x + r / rms(r) * w,  r = y + (weighted sum of a token's expert
+//     rows, where a choice may stand for x itself)
+//   * exact gelu of rows
 //   * clamped gated unit:  g = min(g, limit), u = clamp(u, -limit, limit), out = g * sigmoid(beta g) * (u + shift)
 //   * rotation table whose angles are formed and reduced in fp64, so that far positions keep fp32-accurate angles
 #include <cuda_bf16.h>
@@ -89,7 +92,7 @@ struct AddRmsParams {
   int k;
   const float* x0;
   const float* w;
-  float eps;
+  float w_base, eps;
   int width;
   const long long* rows;
   float* of;
@@ -138,8 +141,88 @@ __global__ void add_rmsnorm_kernel(const AddRmsParams p) {
     float v[V], ww[V];
     load_vec<V>(p.w + k, ww);
 #pragma unroll
-    for (int e = 0; e < V; ++e) v[e] = row_buf[k + e] * scale * ww[e];
+    for (int e = 0; e < V; ++e) v[e] = row_buf[k + e] * scale * (p.w_base + ww[e]);
     store_vec<V>(oc + o * p.width + k, v);
+  }
+}
+
+struct AddNormedParams {
+  const float* x;
+  const void* y;               // [.., ldy] compute type
+  long long ldy;
+  const void* z;               // [.., width] compute type: row[t * k + j] is the row of token t's choice j
+  const int* row;
+  const int* ids;              // the choices; from n_experts on they stand for x
+  const float* wt;             // their weights
+  int k, n_experts;
+  const float* w;
+  float w_base, eps;
+  int width;
+  float* of;
+  void* oc;
+};
+
+// One CTA per row. of may be x.
+template <typename T, int V>
+__global__ void add_normed_kernel(const AddNormedParams p) {
+  extern __shared__ __align__(16) float row_buf[];
+  const long long t = blockIdx.x;
+  const T* y = static_cast<const T*>(p.y);
+  const T* z = static_cast<const T*>(p.z);
+  const float* x = p.x + t * p.width;
+  float own = 0.f;             // weight of x itself
+  for (int j = 0; j < p.k; ++j)
+    if (p.ids[t * p.k + j] >= p.n_experts) own += p.wt[t * p.k + j];
+  float ss = 0.f;
+  for (int c = threadIdx.x * V; c < p.width; c += blockDim.x * V) {
+    float r[V], s[V];
+    load_vec<V>(x + c, r);
+#pragma unroll
+    for (int e = 0; e < V; ++e) r[e] *= own;
+    if (y) {
+      load_vec<V>(y + t * p.ldy + c, s);
+#pragma unroll
+      for (int e = 0; e < V; ++e) r[e] += s[e];
+    }
+    for (int j = 0; j < p.k; ++j) {
+      if (p.ids[t * p.k + j] >= p.n_experts) continue;
+      const float f = p.wt[t * p.k + j];
+      load_vec<V>(z + static_cast<long long>(p.row[t * p.k + j]) * p.width + c, s);
+#pragma unroll
+      for (int e = 0; e < V; ++e) r[e] = fmaf(f, s[e], r[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      row_buf[c + e] = r[e];
+      ss = fmaf(r[e], r[e], ss);
+    }
+  }
+  const float scale = 1.f / sqrtf(block_sum(ss) / static_cast<float>(p.width) + p.eps);
+  T* oc = static_cast<T*>(p.oc);
+  for (int c = threadIdx.x * V; c < p.width; c += blockDim.x * V) {
+    float v[V], ww[V];
+    load_vec<V>(x + c, v);
+    load_vec<V>(p.w + c, ww);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = fmaf(row_buf[c + e] * scale, p.w_base + ww[e], v[e]);
+    store_vec<V>(p.of + t * p.width + c, v);
+    if (oc) store_vec<V>(oc + t * p.width + c, v);
+  }
+}
+
+// May run in place (out = x, ldo = ldx).
+template <typename T, int V>
+__global__ void gelu_kernel(const T* x, long long ldx, int cols, T* out, long long ldo, long long n_vec) {
+  const int per_row = cols / V;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n_vec;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long t = i / per_row;
+    const int c = static_cast<int>(i - t * per_row) * V;
+    float v[V];
+    load_vec<V>(x + t * ldx + c, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = gelu_f(v[e]);
+    store_vec<V>(out + t * ldo + c, v);
   }
 }
 
@@ -228,6 +311,34 @@ static int add_rms_launch(const AddRmsParams& p, int n, cudaStream_t st) {
   return static_cast<int>(cudaGetLastError());
 }
 
+template <typename T, int V>
+static int add_normed_launch(const AddNormedParams& p, int n, cudaStream_t st) {
+  const size_t smem = static_cast<size_t>(p.width) * sizeof(float);
+  static DeviceMax configured;
+  if (smem > 40 * 1024 && smem > configured.get()) {
+    const cudaError_t e = cudaFuncSetAttribute(add_normed_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured.set(200 * 1024);
+  }
+  int threads = row_threads(p.width, V);
+  if (n < 2 * num_sms() && p.width >= 512 * V) threads = 512;       // few rows: one pass over each
+  add_normed_kernel<T, V><<<n, threads, smem, st>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+static int gelu_launch(const void* x, long long ldx, int n, int cols, void* out, long long ldo, cudaStream_t st) {
+  const int v = cols % 8 == 0 && ldx % 8 == 0 && ldo % 8 == 0 ? 8 : 1;
+  const long long n_vec = static_cast<long long>(n) * (cols / v);
+  long long grid = (n_vec + 255) / 256;
+  if (grid > num_sms() * 16) grid = num_sms() * 16;
+  const T* src = static_cast<const T*>(x);
+  T* dst = static_cast<T*>(out);
+  if (v == 8) gelu_kernel<T, 8><<<static_cast<int>(grid), 256, 0, st>>>(src, ldx, cols, dst, ldo, n_vec);
+  else gelu_kernel<T, 1><<<static_cast<int>(grid), 256, 0, st>>>(src, ldx, cols, dst, ldo, n_vec);
+  return static_cast<int>(cudaGetLastError());
+}
+
 template <typename T>
 static int glu_launch(const void* gu, long long ld, const float* bias, int n, int ff, float limit, float beta, float shift,
                       void* out, cudaStream_t st) {
@@ -272,17 +383,37 @@ extern "C" int pm_post_layernorm(const float* x, const void* y, int f32, long lo
 }
 
 // v = x + y + sum_j z[inv[t * k + j]] + x0 for the n rows listed in `rows` (nullable: row i); of [n, width] fp32 (nullable, may
-// be x when rows is null) = v, oc [n, width] in the compute type = v / rms(v) * w. y [.., ldy], z [.., width] (compute type,
+// be x when rows is null) = v, oc [n, width] in the compute type = v / rms(v) * (w_base + w). y [.., ldy], z [.., width] (compute type,
 // inv int32 per token and j < k) and x0 (fp32) are nullable.
 extern "C" int pm_add_rmsnorm(const float* x, const void* y, int f32, long long ldy, const void* z, const int* inv, int k,
-                              const float* x0, const float* w, float eps, int n, int width, const long long* rows,
+                              const float* x0, const float* w, float w_base, float eps, int n, int width, const long long* rows,
                               float* of, void* oc, cudaStream_t st) {
   if (n < 0 || width < 1 || static_cast<size_t>(width) * 4 > 200 * 1024 || (rows && of == x) || (z && (!inv || k < 1))) return -1;
   if (n == 0) return 0;
-  const AddRmsParams p{x, y, ldy, z, inv, k, x0, w, eps, width, rows, of, oc};
+  const AddRmsParams p{x, y, ldy, z, inv, k, x0, w, w_base, eps, width, rows, of, oc};
   const bool vec = width % 4 == 0 && ldy % 4 == 0;
   if (f32) return vec ? add_rms_launch<float, 4>(p, n, st) : add_rms_launch<float, 1>(p, n, st);
   return vec ? add_rms_launch<__nv_bfloat16, 4>(p, n, st) : add_rms_launch<__nv_bfloat16, 1>(p, n, st);
+}
+
+// v = x + r / rms(r) * (w_base + w) with r = y + sum over j < k of wt[t, j] * (ids[t, j] < n_experts ? z[row[t, j]] : x[t]); of
+// [n, width] fp32 = v (may be x), oc the same in the compute type (nullable). y [.., ldy] is nullable, k may be 0.
+extern "C" int pm_add_normed(const float* x, const void* y, int f32, long long ldy, const void* z, const int* row, const int* ids,
+                             const float* wt, int k, int n_experts, const float* w, float w_base, float eps, int n, int width,
+                             float* of, void* oc, cudaStream_t st) {
+  if (n < 0 || width < 1 || static_cast<size_t>(width) * 4 > 200 * 1024 || k < 0 || (k > 0 && (!z || !row || !ids || !wt)) || !of) return -1;
+  if (n == 0) return 0;
+  const AddNormedParams p{x, y, ldy, z, row, ids, wt, k, n_experts, w, w_base, eps, width, of, oc};
+  const bool vec = width % 4 == 0 && ldy % 4 == 0;
+  if (f32) return vec ? add_normed_launch<float, 4>(p, n, st) : add_normed_launch<float, 1>(p, n, st);
+  return vec ? add_normed_launch<__nv_bfloat16, 4>(p, n, st) : add_normed_launch<__nv_bfloat16, 1>(p, n, st);
+}
+
+// out [n, ldo] = exact gelu of x [n, ldx] on the first `cols` columns; out may be x.
+extern "C" int pm_gelu(const void* x, int f32, long long ldx, int n, int cols, void* out, long long ldo, cudaStream_t st) {
+  if (n < 0 || cols < 1 || ldx < cols || ldo < cols) return -1;
+  if (n == 0) return 0;
+  return f32 ? gelu_launch<float>(x, ldx, n, cols, out, ldo, st) : gelu_launch<__nv_bfloat16>(x, ldx, n, cols, out, ldo, st);
 }
 
 // gu [n, ld]: gate columns [0, ff), up columns [ff, 2 ff); bias fp32 [2 ff] or null -> out [n, ff].

@@ -1,12 +1,14 @@
-"""Config-driven serving decoder for stacks that mix attention and recurrent layers (Duvivik, Resevik).
+"""Config-driven serving decoder for stacks that mix kinds of attention and recurrent layers (Duvivik, Resevik, Vosezen).
 
-Each layer has a token mixer (``mixers.MIXERS``) and optionally a feed-forward. The design (``DESIGNS``) says how they meet
-the stream:
+Each layer has a token mixer (``mixers.MIXERS``) and optionally a feed-forward. The design (``DESIGNS``) says which mixers the
+configuration's layer types mean and how the sublayers meet the stream:
 
 * ``post``: both sublayers read the stream itself and the norm comes after the sum, x <- LN(alpha * x + sublayer(x));
 * ``parallel``: both read one RMS norm of the stream, x <- x + mixer(h) + ff(h). A span of layers may run several times in a
   row with the same weights, every run with a cache or state of its own; each pass but the first starts by adding the
-  embedding output to the stream. The sum, the re-added embedding and the next layer's norm are one kernel.
+  embedding output to the stream. The sum, the re-added embedding and the next layer's norm are one kernel;
+* ``branch``: both sublayers read the stream itself and only what they add is normed, x <- x + rms(sublayer(x)) (1 + w). The norm
+  and the sum (for experts also the weighted sum of a token's rows) are one kernel.
 
 The stream, norms, rotation angles, softmax, routers and recurrent states are fp32; projections and their activations run in
 the model's type (bf16 on the sm_100a kernels, or fp32 throughout with full-precision matrix products).
@@ -29,7 +31,7 @@ import torch.nn as nn
 from ..ops import functional as ops
 from .kv_cache import BLOCK
 from .mixers import MIXERS, RotationFreqs, StepContext, frozen
-from .moe import WeightedInputExperts
+from .moe import WeightedInputExperts, WeightedOutputExperts
 from .state_cache import StateCache
 
 GLU_BETA, GLU_SHIFT = 1.702, 1.0          # gate slope and the offset of the up half in the clamped gated unit
@@ -38,14 +40,20 @@ GLU_BETA, GLU_SHIFT = 1.702, 1.0          # gate slope and the offset of the up 
 
 @dataclass(frozen=True)
 class Design:
-    block: str                            # "post" or "parallel"
-    mixers: Tuple[str, ...]
+    block: str                            # "post", "parallel" or "branch"
+    mixers: Dict[str, str]                # "type" of a layer -> name in MIXERS
     feed_forward: str                     # kind of the layers' "mlp" entries
+    experts: Optional[type] = None        # class of the feed-forwards of kind "moe"
+    tied: bool = False                    # the embedding table is the output projection
+    norm_base: float = 0.0                # norms multiply with norm_base + weight ("branch")
 
 
 DESIGNS: Dict[str, Design] = {
-    "duvivik": Design("post", ("mamba2", "latent_attention"), "dense"),
-    "resevik": Design("parallel", ("lightning", "retention", "attention"), "moe"),
+    "duvivik": Design("post", {"mamba2": "mamba2", "latent_attention": "latent_attention"}, "dense"),
+    "resevik": Design("parallel", {"lightning": "lightning", "retention": "retention", "attention": "window_attention"}, "moe",
+                      WeightedInputExperts),
+    "vosezen": Design("branch", {"attention": "difference_attention", "latent_attention": "latent_attention",
+                                 "attention_2": "sink_attention"}, "moe", WeightedOutputExperts, tied=True, norm_base=1.0),
 }
 
 
@@ -91,7 +99,7 @@ class HybridArgs:
         for i, l in enumerate(layers):
             if l["type"] not in design.mixers:
                 raise ValueError(f"layer {i}: unknown mixer {l['type']!r} (known: {', '.join(design.mixers)})")
-            kind = MIXERS[l["type"]]
+            kind = MIXERS[design.mixers[l["type"]]]
             missing = [k for k in kind.KEYS if k not in l["mixer"]]
             if missing:
                 raise ValueError(f"layer {i}: mixer entry lacks {', '.join(missing)}")
@@ -99,8 +107,8 @@ class HybridArgs:
             mlp = l["mlp"]
             if mlp is not None and mlp.get("kind") != design.feed_forward:
                 raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
-            if mlp is not None and design.feed_forward == "moe":
-                WeightedInputExperts.check(mlp, i)
+            if mlp is not None and design.experts is not None:
+                design.experts.check(mlp, i)
         loop = d.get("loop")
         if loop is not None:
             loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
@@ -157,6 +165,30 @@ def _parallel_stack(width: int, vocab: int, ff: int, experts: int, top: int, lin
     return d
 
 
+def _branch_stack(width: int, vocab: int, ff: int, shared: int, experts: int, identity: int, top: int, groups: Tuple[int, int],
+                  latent: dict, diff: dict, sink: dict, pattern: str) -> dict:
+    """Configuration dict: one letter per layer, L = latent attention, S = attention with a sink, D = difference attention, d = the
+    same on the keys and values of the latest D; all with experts."""
+    kinds = {"L": ("latent_attention", latent), "S": ("attention_2", sink), "D": ("attention", diff), "d": ("attention", diff)}
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared},
+           "router": {"experts": experts, "identity": identity, "top": top, "scale": 2.0,
+                      "groups": dict(zip(("count", "keep"), groups))}}
+    layers, src = [], None
+    for i, c in enumerate(pattern):
+        m = copy.deepcopy(kinds[c][1])
+        if c == "D":
+            src = i
+        elif c == "d":
+            m["kv_from"] = src
+        layers.append({"type": kinds[c][0], "mixer": m, "mlp": copy.deepcopy(mlp)})
+    return {"architecture": "Vosezen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
+
+
+def _grouped(heads, kv_heads, dim, vdim, every, **more):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5,
+            "q_temp": {"coef": 0.2, "every": every}, **more}
+
+
 def _linear(heads, dim, vdim):
     return {"heads": heads, "dim": dim, "vdim": vdim}
 
@@ -169,6 +201,10 @@ def _window(heads, kv_heads, dim, size):
 def _attn(heads, dim, rot, vdim, rank):
     return {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "scale": (dim + rot) ** -0.5,
             "rot": {"base": 10000.0, "dims": rot}}
+
+
+def _q_latent(q_rank, *attn):
+    return dict(_attn(*attn), q_rank=q_rank)
 
 
 def _ssm(heads, vdim, state, groups, conv=4, norm_groups=1):
@@ -184,6 +220,12 @@ PRESETS: Dict[str, dict] = {
     # 12 layers twice, and 16 layers with the middle eight twice: 24 layer runs each
     "resevik-1b": _parallel_stack(1536, 65536, 768, 12, 2, _linear(12, 128, 96), _window(12, 4, 96, 512), "LRA" * 4, (0, 12, 2)),
     "resevik-2b": _parallel_stack(2048, 65536, 1024, 16, 2, _linear(16, 128, 128), _window(16, 8, 128, 1024), "LRAL" * 4, (4, 12, 2)),
+    "vosezen-tiny": _branch_stack(64, 512, 48, 56, 7, 1, 2, (4, 2), _q_latent(40, 4, 16, 8, 24, 32), _grouped(4, 2, 16, 24, 32, diff=0.2),
+                                  _grouped(6, 3, 24, 16, 48, softcap=30.0), "LSDLd"),
+    "vosezen-1b": _branch_stack(1536, 65536, 768, 1536, 12, 4, 2, (4, 2), _q_latent(768, 16, 64, 32, 96, 256),
+                                _grouped(12, 4, 64, 128, 1024, diff=0.3), _grouped(12, 4, 128, 128, 1024, softcap=50.0), "LSDLLSdL" * 2),
+    "vosezen-2b": _branch_stack(2048, 65536, 1024, 2048, 16, 4, 2, (4, 2), _q_latent(1024, 16, 96, 32, 128, 512),
+                                _grouped(16, 4, 64, 128, 1024, diff=0.3), _grouped(16, 4, 128, 128, 1024, softcap=50.0), "LSDLLSdL" * 3),
 }
 
 
@@ -223,7 +265,7 @@ class HybridLayer(nn.Module):
     def __init__(self, spec: dict, cfg: HybridArgs, index: int, dtype, device):
         super().__init__()
         self.cfg = cfg
-        self.mixer = MIXERS[spec["type"]](spec["mixer"], cfg, index, dtype, device)
+        self.mixer = MIXERS[cfg.design.mixers[spec["type"]]](spec["mixer"], cfg, index, dtype, device)
         self.mlp = ClampedMLP(spec["mlp"], cfg.hidden_size, dtype, device) if spec["mlp"] is not None else None
         vec = lambda: frozen(torch.zeros(cfg.hidden_size, device=device))      # noqa: E731
         self.norm1_w, self.norm1_b = vec(), vec()
@@ -260,8 +302,8 @@ class ParallelLayer(nn.Module):
     def __init__(self, spec: dict, cfg: HybridArgs, index: int, dtype, device):
         super().__init__()
         self.cfg = cfg
-        self.mixer = MIXERS[spec["type"]](spec["mixer"], cfg, index, dtype, device)
-        self.mlp = WeightedInputExperts(spec["mlp"], cfg.hidden_size, dtype, device) if spec["mlp"] is not None else None
+        self.mixer = MIXERS[cfg.design.mixers[spec["type"]]](spec["mixer"], cfg, index, dtype, device)
+        self.mlp = cfg.design.experts(spec["mlp"], cfg.hidden_size, dtype, device) if spec["mlp"] is not None else None
         self.norm1_w = frozen(torch.zeros(cfg.hidden_size, device=device))
 
     def named_weights(self):
@@ -277,6 +319,37 @@ class ParallelLayer(nn.Module):
         return (y, *(self.mlp(h) if self.mlp is not None else (None, None, 1)))
 
 
+class BranchLayer(nn.Module):
+    """Sublayers read the stream and add their normed results to it."""
+
+    def __init__(self, spec: dict, cfg: HybridArgs, index: int, dtype, device):
+        super().__init__()
+        self.cfg = cfg
+        self.mixer = MIXERS[cfg.design.mixers[spec["type"]]](spec["mixer"], cfg, index, dtype, device)
+        self.mlp = cfg.design.experts(spec["mlp"], cfg.hidden_size, dtype, device) if spec["mlp"] is not None else None
+        self.norm1_w = frozen(torch.zeros(cfg.hidden_size, device=device))
+        if self.mlp is not None:
+            self.norm2_w = frozen(torch.zeros(cfg.hidden_size, device=device))
+
+    def named_weights(self):
+        for name, p in [("norm1", self.norm1_w)] + ([("norm2", self.norm2_w)] if self.mlp is not None else []):
+            yield name, (self.cfg.hidden_size,), p.copy_, (lambda p=p: p)
+        for pre, mod in (("mix.", self.mixer), ("mlp.", self.mlp)):
+            if mod is not None:
+                for name, *rest in mod.named_weights():
+                    yield (pre + name, *rest)
+
+    def forward(self, xf, xc, cache, ctx):
+        """(fp32 stream, compute-type copy) -> the same after the layer."""
+        from ..ops import native as nat
+        cfg = self.cfg
+        kw = dict(w_base=cfg.design.norm_base)
+        xf, xc = nat.add_normed(xf, self.norm1_w, cfg.norm_eps, y=self.mixer(xc, cache, ctx), **kw)
+        if self.mlp is not None:
+            xf, xc = nat.add_normed(xf, self.norm2_w, cfg.norm_eps, **self.mlp(xc), **kw)
+        return xf, xc
+
+
 class HybridDecoderLM(nn.Module):
     graph_decode = True         # single-token steps can be captured (generation.GraphedDecoder)
     mixed_batches = True        # the scheduler puts prompt portions and decoded tokens into one step
@@ -288,13 +361,13 @@ class HybridDecoderLM(nn.Module):
             raise ValueError("the hybrid decoder runs in bf16 or fp32")
         self.cfg, self.dtype = cfg, dtype
         self.embed_tokens = frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
-        self.parallel = cfg.design.block == "parallel"
-        kind = ParallelLayer if self.parallel else HybridLayer
+        block = cfg.design.block
+        kind = {"post": HybridLayer, "parallel": ParallelLayer, "branch": BranchLayer}[block]
         self.layers = nn.ModuleList([kind(s, cfg, i, dtype, device) for i, s in enumerate(cfg.layers)])
         self.runs = cfg.runs
         self.norm_w = frozen(torch.zeros(cfg.hidden_size, device=device))
-        self.norm_b = None if self.parallel else frozen(torch.zeros(cfg.hidden_size, device=device))
-        self.head = frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
+        self.norm_b = frozen(torch.zeros(cfg.hidden_size, device=device)) if block == "post" else None
+        self.head = self.embed_tokens if cfg.design.tied else frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
         self._freqs = RotationFreqs()
 
     # ------------------------------------------------------------------ weights
@@ -308,7 +381,8 @@ class HybridDecoderLM(nn.Module):
         yield "final.norm", (c.hidden_size,), self.norm_w.copy_, lambda: self.norm_w
         if self.norm_b is not None:
             yield "final.norm.b", (c.hidden_size,), self.norm_b.copy_, lambda: self.norm_b
-        yield "head", (c.vocab_size, c.hidden_size), self.head.copy_, lambda: self.head
+        if not c.design.tied:
+            yield "head", (c.vocab_size, c.hidden_size), self.head.copy_, lambda: self.head
 
     @torch.no_grad()
     def load_hf_state_dict(self, sd: Dict[str, torch.Tensor], strict: bool = True) -> List[str]:
@@ -332,7 +406,7 @@ class HybridDecoderLM(nn.Module):
 
     @torch.no_grad()
     def init_weights(self, std: float = 0.02, seed: int = 0, device=None) -> "HybridDecoderLM":
-        """Random model: N(0, std) matrices, unit norms, decays and step sizes spread over their usual ranges. Drawn on
+        """Random model: N(0, std) matrices, unit norms, decays, step sizes and sinks spread over their usual ranges. Drawn on
         ``device`` (CPU unless given: the values then do not depend on the model's device)."""
         g = torch.Generator(device=device or "cpu").manual_seed(seed)
         for name, shape, put, _ in self.named_weights():
@@ -340,6 +414,14 @@ class HybridDecoderLM(nn.Module):
             rnd = lambda: torch.empty(shape, device=device or "cpu")      # noqa: E731
             if leaf.endswith("mlp.router"):
                 put(rnd().normal_(0.0, 1.0, generator=g).div_(shape[1] ** 0.5))      # logits of order one: spread over the experts
+            elif leaf.endswith("mlp.correction"):
+                put(rnd().normal_(0.0, 0.01, generator=g))
+            elif leaf.endswith("mix.sink"):
+                put(rnd().normal_(0.0, 1.0, generator=g))
+            elif leaf.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
+                put(rnd().normal_(0.0, 0.1, generator=g))
+            elif self.cfg.design.norm_base and leaf in ("norm1", "norm2", "final.norm"):
+                put(torch.full(shape, 1.0 - self.cfg.design.norm_base, device=device or "cpu"))
             elif leaf.endswith(".A_log"):
                 put(rnd().uniform_(1.0, 16.0, generator=g).log_())
             elif leaf.endswith(".dt_bias"):
@@ -404,12 +486,12 @@ class HybridDecoderLM(nn.Module):
         if rows is None and not all_logits:
             rows = (meta.q_start + meta.q_lens - 1).long()
         xf, xc = nat.embed_scale(input_ids, self.embed_tokens, cfg.embed_scale)
-        h = (self._parallel if self.parallel else self._post)(xf, xc, cache, ctx, rows, on_layer)
+        h = (self._parallel if cfg.design.block == "parallel" else self._serial)(xf, xc, cache, ctx, rows, on_layer)
         if h.shape[0] == 0:
             return torch.empty(0, h.shape[1] if return_hidden else cfg.vocab_size, dtype=torch.float32, device=h.device)
         return h if return_hidden else ops.project_f32(h, self.head, cfg.vocab_size)
 
-    def _post(self, xf, xc, cache, ctx, rows, on_layer) -> torch.Tensor:
+    def _serial(self, xf, xc, cache, ctx, rows, on_layer) -> torch.Tensor:
         from ..ops import native as nat
         for i, layer in enumerate(self.layers):
             xf, xc = layer(xf, xc, cache, ctx)
@@ -417,6 +499,9 @@ class HybridDecoderLM(nn.Module):
                 on_layer(i, xf)
         if rows is not None and rows.shape[0] == 0:
             return xc[:0]
+        if self.norm_b is None:
+            return nat.add_rmsnorm(xf, self.norm_w, self.cfg.norm_eps, rows=rows, want_stream=False, dtype=self.dtype,
+                                   w_base=self.cfg.design.norm_base)[1]
         return nat.post_layernorm(xf, None, self.norm_w, self.norm_b, self.cfg.norm_eps, rows=rows, want_stream=False,
                                   dtype=self.dtype)[1]
 

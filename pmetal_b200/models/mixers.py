@@ -3,14 +3,17 @@
 A mixer is built from its entry in the configuration, says what it keeps in the cache (``cache_spec``), lists its weights
 (``named_weights``) and runs on the new tokens of a step: ``forward(x, cache, ctx, run)`` with x [tokens, width] in the
 compute type returns [tokens, >= width]. ``run`` counts layer runs of the step (the layer's index in stacks without loops) and
-names what the mixer keeps in the cache for this run. ``MIXERS`` maps the configuration's ``type`` to the class; a new kind of
-mixer is one more entry.
+names what the mixer keeps in the cache for this run. ``MIXERS`` names the classes; a design (``hybrid_decoder.DESIGNS``) says
+which of them the ``type`` entries of its configuration mean. A new kind of mixer is one more entry.
 
 ``Mamba2Mixer``          selective state space with one decay per head (csrc/ssm.cu)
-``LatentAttentionMixer`` multi-head latent attention on cached latents, its own or an earlier layer's (csrc/latent_attn.cu)
+``LatentAttentionMixer`` multi-head latent attention on cached latents, its own or an earlier layer's; queries from the input
+                         or from a latent of their own (csrc/latent_attn.cu)
 ``LinearAttentionMixer`` linear attention with a fixed decay per head; ``LightningMixer`` and ``RetentionMixer`` set its
                          activation, rotation, norm and gate (csrc/linear_attn.cu)
-``WindowAttentionMixer`` grouped-query attention in a sliding window, keys as values (csrc/window_attn.cu)
+``GroupedAttentionMixer`` grouped-query attention of any key and value size (csrc/window_attn.cu): ``WindowAttentionMixer``
+                         (sliding window, keys as values), ``DifferenceAttentionMixer`` (difference of two maps) and
+                         ``SinkAttentionMixer`` (capped scores, a sink per head)
 """
 from __future__ import annotations
 
@@ -142,7 +145,7 @@ class Mamba2Mixer(nn.Module):
 
 class LatentAttentionMixer(nn.Module):
     """Causal attention whose cache is one latent and one rotated key part per token. ``kv_from`` makes the layer read an
-    earlier layer's rows with its own up-projections."""
+    earlier layer's rows with its own up-projections. ``q_rank``: the queries come from a normed latent of that size."""
 
     KEYS = ("heads", "dim", "rot_dim", "vdim", "kv_rank", "rot", "scale")
 
@@ -152,6 +155,8 @@ class LatentAttentionMixer(nn.Module):
             raise ValueError(f"layer {index}: rot_dim must be even")
         if m["rot"]["dims"] != m["rot_dim"]:
             raise ValueError(f"layer {index}: rot.dims must equal rot_dim")
+        if m.get("q_rank") is not None and m["q_rank"] < 1:
+            raise ValueError(f"layer {index}: q_rank must be at least 1")
         src = m.get("kv_from")
         if src is None:
             return
@@ -173,7 +178,11 @@ class LatentAttentionMixer(nn.Module):
         self.n_q, self.n_d, self.n_k, self.n_v = H * (dn + dr), (r + dr) if src is None else 0, H * dn, H * dv
         kw = dict(dtype=dtype, device=device)
         up8 = lambda n: -(-n // 8) * 8      # noqa: E731
-        self.w_q = frozen(torch.zeros(up8(self.n_q + self.n_d), self.width, **kw))       # queries, then the down-projection
+        self.q_rank = m.get("q_rank") or 0
+        self.n_in = self.q_rank or self.n_q
+        self.w_q = frozen(torch.zeros(up8(self.n_in + self.n_d), self.width, **kw))      # queries (or their latent), then the down-projection
+        self.w_uq = frozen(torch.zeros(up8(self.n_q), self.q_rank, **kw)) if self.q_rank else None
+        self.q_norm_w = frozen(torch.zeros(self.q_rank, device=device)) if self.q_rank else None
         self.w_ukv = frozen(torch.zeros(up8(self.n_k + self.n_v), r, **kw))              # keys of all heads, then values
         self.w_o = frozen(torch.zeros(up8(self.width), self.n_v, **kw))
         self.norm_w = frozen(torch.zeros(r, device=device)) if self.own else None
@@ -184,9 +193,12 @@ class LatentAttentionMixer(nn.Module):
         return CacheSpec(page_width=self.row + 8 if self.own else 0)      # the kernels keep rows eight columns apart
 
     def named_weights(self):
-        q, d, k, v = self.n_q, self.n_d, self.n_k, self.n_v
+        q, d, k, v, n_q = self.n_in, self.n_d, self.n_k, self.n_v, self.n_q
         r = self.dims[4]
-        yield "q", (q, self.width), lambda t: self.w_q[:q].copy_(t), lambda: self.w_q[:q]
+        yield "dq" if self.q_rank else "q", (q, self.width), lambda t: self.w_q[:q].copy_(t), lambda: self.w_q[:q]
+        if self.q_rank:
+            yield "dq.norm", (q,), self.q_norm_w.copy_, lambda: self.q_norm_w
+            yield "uq", (n_q, q), lambda t: self.w_uq[:n_q].copy_(t), lambda: self.w_uq[:n_q]
         if self.own:
             yield "dkv", (d, self.width), lambda t: self.w_q[q:q + d].copy_(t), lambda: self.w_q[q:q + d]
             yield "dkv.norm", (r,), self.norm_w.copy_, lambda: self.norm_w
@@ -208,12 +220,20 @@ class LatentAttentionMixer(nn.Module):
         H, dn, dr, dv, r, W = self.dims
         pages = cache.pages[run if self.own and run is not None else self.source]
         qd = ops.project(x, self.w_q)
-        cos, sin = ctx.rope(self.base, dr) if dr else (None, None)
-        nat.latent_prep(qd, self.norm_w, self.eps, cos, sin, self.dims, pages if self.own else None, ctx.meta.slots)
+        rope = ctx.rope(self.base, dr) if dr else (None, None)
+        nat.latent_prep(qd, self.norm_w, self.eps, *rope, self.dims, pages if self.own else None, ctx.meta.slots, self.q_rank,
+                        self.q_norm_w)
         o = torch.empty(x.shape[0], H * dv, dtype=x.dtype, device=x.device)
         short, long = ctx.groups(SHORT if self.expand else 1 << 30)
+        turn = (None, None)
+        if self.q_rank:
+            qd = ops.project(qd[:, :self.q_rank], self.w_uq)
+            if long is None:
+                turn = rope                                # on the way into the short portions' kernel
+            elif dr:
+                nat.latent_prep(qd, None, self.eps, *rope, self.dims, None, ctx.meta.slots)
         if short is not None:
-            nat.latent_attn(qd, self.w_ukv, self.w_ukv[self.n_k:], pages, short, self.dims, self.scale, o)
+            nat.latent_attn(qd, self.w_ukv, self.w_ukv[self.n_k:], pages, short, self.dims, self.scale, o, turn)
         if long is not None:
             w = self._expand_weight()
             for i, q0, n, n_keys in long.host:
@@ -304,63 +324,146 @@ class RetentionMixer(LinearAttentionMixer):
     KEY_FACTOR = HEAD_NORM = SILU_GATE = True
 
 
-class WindowAttentionMixer(nn.Module):
-    """Grouped-query softmax attention over a sliding window. Queries and keys are rotated, then divided by their root mean
-    square over the head; the values are the keys as projected."""
+class GroupedAttentionMixer(nn.Module):
+    """Grouped-query softmax attention on cached keys and values. The class says what the design fixes, the configuration entry
+    gives sizes and, where present, the rotation (``rot``), the window (``mask``), the query factor that grows with the position
+    (``q_temp``) and the cap of the scores (``softcap``). ``kv_from`` makes the layer read an earlier layer's keys and values with
+    its own queries."""
 
-    KEYS = ("heads", "kv_heads", "dim", "vdim", "rot", "mask", "scale")
-    ROTATION = "pairs"
-    UNIT_NORM = True
-    OWN_VALUES = False
+    KEYS = ("heads", "kv_heads", "dim", "vdim", "scale")
+    MAPS = 1                   # attention maps per head over the same values; with two their difference is taken
+    ROTATION = "none"          # layout of the rotated pairs of q and k
+    UNIT_NORM = True           # queries and keys divided by their root mean square over the head
+    NORM_WEIGHTS = True        # and multiplied with a weight
+    OWN_VALUES = True          # else the values are the keys as projected
+    SINK = False               # a learned score per head without a value
+    GATE = True                # sigmoid of a projection of the input, one number per head
 
     @classmethod
     def check(cls, m: dict, index: int, layers) -> None:
         if m["heads"] % m["kv_heads"]:
             raise ValueError(f"layer {index}: {m['heads']} heads do not divide into {m['kv_heads']} key/value heads")
-        if m["vdim"] != m["dim"]:
+        if not cls.OWN_VALUES and m["vdim"] != m["dim"]:
             raise ValueError(f"layer {index}: vdim must equal dim where the values are the keys")
-        if m["dim"] > 1024:
+        if max(m["dim"], m["vdim"]) > 1024:
             raise ValueError(f"layer {index}: heads of more than 1024 channels")
-        if m["mask"].get("size", 0) < 1:
+        if cls.ROTATION != "none":
+            check_rotation(m, index)
+        if m.get("mask") is not None and m["mask"].get("size", 0) < 1:
             raise ValueError(f"layer {index}: mask.size must be at least 1")
-        check_rotation(m, index)
+        temp = m.get("q_temp")
+        if temp is not None and (temp["every"] < 1 or temp["every"] != int(temp["every"])):
+            raise ValueError(f"layer {index}: q_temp.every must be a positive whole number")
+        if m.get("softcap") is not None and not m["softcap"] > 0:
+            raise ValueError(f"layer {index}: softcap must be positive")
+        src = m.get("kv_from")
+        if src is None:
+            return
+        if not 0 <= src < index or layers[src]["type"] != layers[index]["type"] or layers[src]["mixer"].get("kv_from") is not None:
+            raise ValueError(f"layer {index}: kv_from must name an earlier layer of the same kind with its own keys and values")
+        o = layers[src]["mixer"]
+        if any(o.get(k) != m.get(k) for k in ("heads", "kv_heads", "dim", "vdim", "rot", "mask")):
+            raise ValueError(f"layer {index}: head counts, sizes, rotation and window must equal layer {src}'s")
 
     def __init__(self, m: dict, cfg, index: int, dtype, device):
         super().__init__()
-        self.dims = (m["heads"], m["kv_heads"], m["dim"])
-        self.base, self.R = float(m["rot"]["base"]), int(m["rot"]["dims"])
-        self.scale, self.window, self.eps = float(m["scale"]), int(m["mask"]["size"]), cfg.norm_eps
-        self.index, self.width = index, cfg.hidden_size
-        self.n_q, self.n_k = m["heads"] * m["dim"], m["kv_heads"] * m["dim"]
-        kw = dict(dtype=dtype, device=device)
+        H, G, M, D, DV = self.dims = (m["heads"], m["kv_heads"], self.MAPS, m["dim"], m["vdim"])
+        rot = m["rot"] if self.ROTATION != "none" else {"base": 1.0, "dims": 0}
+        self.base, self.R = float(rot["base"]), int(rot["dims"])
+        self.scale, self.eps = float(m["scale"]), cfg.norm_eps
+        self.window = int(m["mask"]["size"]) if m.get("mask") is not None else 0
+        self.softcap = float(m["softcap"]) if m.get("softcap") is not None else 0.0
+        temp = m.get("q_temp")
+        self.temp = (float(temp["coef"]), int(temp["every"])) if temp is not None else None
+        src = m.get("kv_from")
+        self.own, self.source, self.index, self.width = src is None, index if src is None else src, index, cfg.hidden_size
+        parts = [("q", H * M * D)]
+        if self.own:
+            parts += [("k", G * M * D)] + ([("v", G * DV)] if self.OWN_VALUES else [])
+        if self.GATE:
+            parts.append(("g", H))
+        self.parts, self.at, n = parts, {}, 0
+        for name, rows in parts:
+            self.at[name] = n
+            n += rows
+        self.inner = H * DV
         up8 = lambda n: -(-n // 8) * 8      # noqa: E731
-        self.w_in = frozen(torch.zeros(up8(self.n_q + self.n_k), self.width, **kw))      # queries, keys
-        self.w_o = frozen(torch.zeros(up8(self.width), self.n_q, **kw))
+        vec = lambda n: frozen(torch.zeros(n, device=device))      # noqa: E731
+        self.w_in = frozen(torch.zeros(up8(n), self.width, dtype=dtype, device=device))
+        self.w_o = frozen(torch.zeros(up8(self.width), self.inner, dtype=dtype, device=device))
+        self.q_norm_w = vec(D) if self.NORM_WEIGHTS else None
+        self.k_norm_w = vec(D) if self.NORM_WEIGHTS and self.own else None
+        self.sink = vec(H) if self.SINK else None
+        self.diff = float(m["diff"]) if M > 1 else 0.0
+        if M > 1:
+            self.lq1, self.lk1, self.lq2, self.lk2 = (vec(D) for _ in range(4))
+            self.register_buffer("lam", torch.zeros(1, device=device), persistent=False)
 
     def cache_spec(self) -> CacheSpec:
-        _, G, D = self.dims
-        return CacheSpec(page_width=2 * G * (-(-D // 8) * 8), window=self.window)
+        _, G, M, D, DV = self.dims
+        pad8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        return CacheSpec(page_width=G * (M * pad8(D) + pad8(DV)), window=self.window) if self.own else CacheSpec()
+
+    @torch.no_grad()
+    def _put_lambda(self, dst: torch.Tensor, t: torch.Tensor) -> None:
+        dst.copy_(t)
+        self.lam.copy_((torch.exp((self.lq1 * self.lk1).sum()) - torch.exp((self.lq2 * self.lk2).sum()) + self.diff).view(1))
 
     def named_weights(self):
-        q, k, w = self.n_q, self.n_k, self.width
-        yield "q", (q, w), lambda t: self.w_in[:q].copy_(t), lambda: self.w_in[:q]
-        yield "k", (k, w), lambda t: self.w_in[q:q + k].copy_(t), lambda: self.w_in[q:q + k]
-        yield "o", (w, q), lambda t: self.w_o[:w].copy_(t), lambda: self.w_o[:w]
+        for name, n in self.parts:
+            a = self.at[name]
+            yield name, (n, self.width), lambda t, a=a, n=n: self.w_in[a:a + n].copy_(t), lambda a=a, n=n: self.w_in[a:a + n]
+        for name in ("q", "k"):
+            p = getattr(self, name + "_norm_w")
+            if p is not None:
+                yield name + ".norm", tuple(p.shape), p.copy_, lambda p=p: p
+        if self.sink is not None:
+            yield "sink", tuple(self.sink.shape), self.sink.copy_, lambda: self.sink
+        for name in ("lq1", "lk1", "lq2", "lk2") if self.dims[2] > 1 else ():
+            p = getattr(self, name)
+            yield name, tuple(p.shape), lambda t, p=p: self._put_lambda(p, t), lambda p=p: p
+        w = self.width
+        yield "o", (w, self.inner), lambda t: self.w_o[:w].copy_(t), lambda: self.w_o[:w]
 
     def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
         from ..ops import native as nat
-        pages = cache.pages[self.index if run is None else run]
+        pages = cache.pages[run if self.own and run is not None else self.source]
         u = ops.project(x, self.w_in)
         cos, sin = ctx.rope(self.base, self.R) if self.R else (None, None)
-        q = nat.window_prep(u, cos, sin, self.dims, (self.R, self.ROTATION), self.UNIT_NORM, self.eps, self.OWN_VALUES, pages,
-                            ctx.meta.slots)
-        o = torch.empty(x.shape[0], self.n_q, dtype=x.dtype, device=x.device)
+        k_at = self.at.get("k", 0)
+        q = nat.window_prep(u, cos, sin, self.dims, (self.R, self.ROTATION), self.UNIT_NORM, self.eps, (k_at, self.at.get("v", k_at)),
+                            pages if self.own else None, ctx.meta.slots, self.q_norm_w, self.k_norm_w, self.temp, ctx.meta.positions)
+        o = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
+        gate = u[:, self.at["g"]:] if self.GATE else None
+        diff = (self.lam, 1.0 - self.diff, self.eps) if self.dims[2] > 1 else None
         short, long = ctx.groups(SHORT)
         for group, few in ((short, True), (long, False)):
             if group is not None:
-                nat.window_attn(q, pages, group, self.dims, self.window, self.scale, few, o)
+                nat.window_attn(q, pages, group, self.dims, self.window, self.scale, few, o, self.softcap, self.sink, gate, diff)
         return ops.project(o, self.w_o)
 
 
+class WindowAttentionMixer(GroupedAttentionMixer):
+    """Sliding window. Queries and keys are rotated, then divided by their root mean square; the values are the keys as
+    projected."""
+
+    KEYS = GroupedAttentionMixer.KEYS + ("rot", "mask")
+    ROTATION = "pairs"
+    NORM_WEIGHTS = OWN_VALUES = GATE = False
+
+
+class DifferenceAttentionMixer(GroupedAttentionMixer):
+    """Two maps per head over the same values: a_1 - lambda a_2 with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, divided by
+    its root mean square over the head, times 1 - diff."""
+
+    KEYS = GroupedAttentionMixer.KEYS + ("diff",)
+    MAPS = 2
+
+
+class SinkAttentionMixer(GroupedAttentionMixer):
+    SINK = True
+
+
 MIXERS = {"mamba2": Mamba2Mixer, "latent_attention": LatentAttentionMixer, "lightning": LightningMixer,
-          "retention": RetentionMixer, "attention": WindowAttentionMixer}
+          "retention": RetentionMixer, "window_attention": WindowAttentionMixer, "difference_attention": DifferenceAttentionMixer,
+          "sink_attention": SinkAttentionMixer}

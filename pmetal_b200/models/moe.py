@@ -78,11 +78,11 @@ class WeightedInputExperts(nn.Module):
         T, f, w = h.shape[0], self.ff, self.width
         if h.dtype != torch.bfloat16 or f % 8 or w % 8:
             xs, off, dest = nat.expert_gather(h, r, self.k)
-            return nat.expert_rows(nat.expert_rows(xs, self.gate_up, off, glu=True), self.down, off), dest, self.k
+            return nat.expert_rows(nat.expert_rows(xs, self.gate_up, off, "swiglu"), self.down, off), dest, self.k
         per = -(-T * self.k // self.E)                     # rows of an expert on average
         if per <= self.GEMV_ROWS and T * self.k <= self.GEMV_PAIRS:
-            act = nat.expert_gemv(h, self.gate_up, r, self.k, True)
-            return nat.expert_gemv(act, self.down, r, self.k, False), r["inv"], self.k
+            act = nat.expert_gemv(h, self.gate_up, r, self.k, "swiglu")
+            return nat.expert_gemv(act, self.down, r, self.k, "none"), r["inv"], self.k
         if per <= self.FEW:
             xs, off, dest = nat.expert_gather(h, r, self.k)
             tile = min(T, 2 * per)
@@ -92,6 +92,92 @@ class WeightedInputExperts(nn.Module):
         gu = nat.grouped_gemm(0, xs, self.gate_up, off, 2 * f, w)
         act = nat.clamped_glu(gu, f, float("inf"), 1.0, 0.0)                        # silu(gate) * up
         return nat.grouped_gemm(0, act, self.down, off, w, f), dest, self.k
+
+
+class WeightedOutputExperts(nn.Module):
+    """Routed experts for serving without a gated unit, down_e(gelu(U_e h)), whose routing weight multiplies the expert's output,
+    beside a shared expert that every token uses. Scores are the softmax of fp32 router logits. The choice goes by score +
+    correction within the best groups of neighbours; the weights are the scores times a factor. The last ``identity`` router
+    outputs stand for h itself.
+
+    ``forward`` returns the summands of ``native.add_normed``, which adds a token's rows up, norms the sum and adds it to the
+    stream. The products take the paths of ``WeightedInputExperts``; pairs that chose an identity lie behind the experts' rows and
+    are not computed."""
+
+    GEMV_ROWS, GEMV_PAIRS, FEW = WeightedInputExperts.GEMV_ROWS, WeightedInputExperts.GEMV_PAIRS, WeightedInputExperts.FEW
+
+    @classmethod
+    def check(cls, m: dict, index: int) -> None:
+        r = m["router"]
+        n, groups = r["experts"] + r.get("identity", 0), r.get("groups") or {"count": 1, "keep": 1}
+        if r["experts"] < 1 or r.get("identity", 0) < 0 or not 1 <= r["top"] <= min(n, 16) or n > 1024:
+            raise ValueError(f"layer {index}: top must lie between 1 and the number of experts (at most 16 of 1024)")
+        if not 1 <= groups["keep"] <= groups["count"] <= 32 or n % groups["count"] or groups["keep"] * (n // groups["count"]) < r["top"]:
+            raise ValueError(f"layer {index}: {n} experts in {groups['count']} groups, of which {groups['keep']} are open to {r['top']} choices")
+
+    def __init__(self, m: dict, width: int, dtype, device):
+        super().__init__()
+        r = m["router"]
+        self.E, self.identity, self.k, self.ff, self.width = r["experts"], r.get("identity", 0), r["top"], m["expert"]["ff"], width
+        groups = r.get("groups") or {"count": 1, "keep": 1}
+        self.groups, self.keep, self.factor = groups["count"], groups["keep"], float(r.get("scale", 1.0))
+        self.shared_ff = m["shared"]["ff"] if m.get("shared") else 0
+        up8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        new = lambda *s: nn.Parameter(torch.zeros(*s, dtype=dtype, device=device), requires_grad=False)      # noqa: E731
+        self.router = new(up8(self.E + self.identity), width)
+        self.correction = nn.Parameter(torch.zeros(self.E + self.identity, device=device), requires_grad=False)
+        self.up, self.down = new(self.E, self.ff, width), new(self.E, width, self.ff)
+        if self.shared_ff:
+            self.shared_up, self.shared_down = new(up8(self.shared_ff), width), new(up8(width), self.shared_ff)
+
+    def named_weights(self):
+        f, w, n, s = self.ff, self.width, self.E + self.identity, self.shared_ff
+        for e in range(self.E):
+            up, dn = self.up[e], self.down[e]
+            yield f"e{e}.up", (f, w), up.copy_, lambda up=up: up
+            yield f"e{e}.down", (w, f), dn.copy_, lambda dn=dn: dn
+        yield "router", (n, w), self.router[:n].copy_, lambda: self.router[:n]
+        yield "correction", (n,), self.correction.copy_, lambda: self.correction
+        if s:
+            yield "shared.up", (s, w), self.shared_up[:s].copy_, lambda: self.shared_up[:s]
+            yield "shared.down", (w, s), self.shared_down[:w].copy_, lambda: self.shared_down[:w]
+
+    def _shared(self, h: torch.Tensor) -> torch.Tensor:
+        from ..ops import functional as ops
+        from ..ops import native as nat
+        if h.dtype == torch.bfloat16 and ops.gemv_fits(*h.shape) and h.stride(0) % 8 == 0:
+            a = nat.gemv_ex(h, self.shared_up, n=self.shared_ff, gelu=True)
+        else:
+            a = ops.project(h, self.shared_up)
+            a = nat.gelu(a, a)[:, :self.shared_ff]
+        return ops.project(a, self.shared_down)
+
+    def _routed(self, h: torch.Tensor, r: dict):
+        """(expert rows, row of every (token, slot))."""
+        from ..ops import native as nat
+        T, f, w, k = h.shape[0], self.ff, self.width, self.k
+        if h.dtype != torch.bfloat16 or f % 8 or w % 8:
+            xs, off, dest = nat.expert_gather(h, r, k, weighted=False)
+            return nat.expert_rows(nat.expert_rows(xs, self.up, off, "gelu"), self.down, off), dest
+        per = -(-T * k // self.E)                          # rows of an expert on average
+        if per <= self.GEMV_ROWS and T * k <= self.GEMV_PAIRS:
+            return nat.expert_gemv(nat.expert_gemv(h, self.up, r, k, "gelu"), self.down, r, k, "none"), r["inv"]
+        if per <= self.FEW:
+            xs, off, dest = nat.expert_gather(h, r, k, weighted=False)
+            tile = min(T, 2 * per)
+            act = nat.grouped_gemm_skinny(xs, self.up, off, max_rows_per_expert=tile, gelu=True)
+            return nat.grouped_gemm_skinny(act, self.down, off, max_rows_per_expert=tile), dest
+        xs, off, dest = nat.expert_gather(h, r, k, align=128, weighted=False)
+        act = nat.grouped_gemm(0, xs, self.up, off, f, w)
+        return nat.grouped_gemm(0, nat.gelu(act, act), self.down, off, w, f), dest
+
+    def forward(self, h: torch.Tensor) -> dict:
+        from ..ops import functional as ops
+        from ..ops import native as nat
+        r = nat.moe_route(ops.project_f32(h, self.router, self.E + self.identity), self.k, False,
+                          choice=(self.correction, self.groups, self.keep, self.factor))
+        z, row = self._routed(h, dict(r, counts=r["counts"][:self.E], offsets=r["offsets"][:self.E + 1]))
+        return dict(y=self._shared(h) if self.shared_ff else None, z=z, route=(r["topk_w"], r["topk_idx"], row, self.E), k=self.k)
 
 
 class SparseMoeBlock(nn.Module):

@@ -454,10 +454,10 @@ def grouped_gemm(mode: int, a: torch.Tensor, b: torch.Tensor, off: torch.Tensor,
 
 
 def grouped_gemm_skinny(x: torch.Tensor, w: torch.Tensor, off: torch.Tensor, swiglu: bool = False,
-                        max_rows_per_expert: int = 128) -> torch.Tensor:
+                        max_rows_per_expert: int = 128, gelu: bool = False) -> torch.Tensor:
     """Expert GEMM for steps that give each expert few rows (csrc/grouped_gemm.cu, swapped operands): ``x`` [R, K]
     expert-sorted with row offsets ``off`` (int32 [E + 1], no alignment), ``w`` [E, N, K], or [E, 2 N, K] with
-    ``swiglu`` (gate rows above up rows), in which case the result is silu(x G^T) * (x U^T). Returns [R, N] bf16; rows
+    ``swiglu`` (gate rows above up rows), in which case the result is silu(x G^T) * (x U^T); ``gelu``: exact gelu. Returns [R, N] bf16; rows
     that belong to no expert are left unwritten."""
     E = off.numel() - 1
     R, K = x.shape
@@ -468,7 +468,7 @@ def grouped_gemm_skinny(x: torch.Tensor, w: torch.Tensor, off: torch.Tensor, swi
     y = torch.empty(R, N, dtype=torch.bfloat16, device=x.device)
     lib().pm_grouped_gemm_skinny.restype = c_int
     rc = lib().pm_grouped_gemm_skinny(_p(x), c_int(x.stride(0)), c_int(R), _p(w), c_int(w.stride(1)), _p(y), c_int(N),
-                                      _p(off), c_int(E), c_int(N), c_int(K), c_int(bn), c_int(int(swiglu)),
+                                      _p(off), c_int(E), c_int(N), c_int(K), c_int(bn), c_int(1 if swiglu else 2 if gelu else 0),
                                       c_float(1.0), _p(status_word(x.device)), _stream())
     _chk(rc, "pm_grouped_gemm_skinny")
     return y
@@ -972,9 +972,11 @@ def count_tokens(counts, tokens, count_rows=None) -> None:
 
 
 # ------------------------------------------------------------------------------------------- MoE routing
-def moe_route(router_logits, k: int, renorm: bool = True, offsets_out=None, score: str = "softmax"):
+def moe_route(router_logits, k: int, renorm: bool = True, offsets_out=None, score: str = "softmax", choice=None):
     """router_logits [T, E] (bf16 or fp32). The k experts with the largest scores (``softmax`` over the experts or the
-    ``sigmoid`` of every logit), weighted by their scores (``renorm``: divided by their sum). Returns dict(topk_idx [T,k],
+    ``sigmoid`` of every logit), weighted by their scores (``renorm``: divided by their sum). ``choice`` = (correction fp32 [E],
+    groups, groups kept, factor): the choice goes by score + correction within the groups of neighbours that have the largest such
+    sums, and the weights (scores without the correction) are multiplied by the factor. Returns dict(topk_idx [T,k],
     topk_w [T,k], counts [E], offsets [E+1], perm [T*k] (sorted position -> token*k+slot), inv [T*k] (token*k+slot -> sorted
     position))."""
     T, E = router_logits.shape
@@ -985,8 +987,10 @@ def moe_route(router_logits, k: int, renorm: bool = True, offsets_out=None, scor
     out = dict(topk_idx=torch.empty(T, k, dtype=torch.int32, device=dev), topk_w=torch.empty(T, k, dtype=torch.float32, device=dev),
                counts=torch.empty(E, dtype=torch.int32, device=dev), offsets=torch.empty(E + 1, dtype=torch.int32, device=dev),
                perm=torch.empty(T * k, dtype=torch.int32, device=dev), inv=torch.empty(T * k, dtype=torch.int32, device=dev))
+    corr, groups, keep, factor = choice if choice is not None else (None, 0, 0, 1.0)
     _chk(lib().pm_moe_route3(_p(x), c_int(int(x.dtype == torch.float32)), c_int(x.stride(0)),
-                             c_int(("softmax", "sigmoid").index(score)), c_int(T), c_int(E), c_int(k), c_int(int(renorm)),
+                             c_int(("softmax", "sigmoid").index(score)), _p(corr), c_int(groups), c_int(keep), c_float(factor),
+                             c_int(T), c_int(E), c_int(k), c_int(int(renorm)),
                              _p(out["topk_idx"]), _p(out["topk_w"]), _p(out["counts"]), _p(out["offsets"]),
                              _p(offsets_out), _p(out["perm"]), _p(out["inv"]), _stream()), "pm_moe_route3")
     return out
@@ -1008,8 +1012,11 @@ def moe_combine(z, inv, w, k: int, residual=None):
     return y
 
 
-def expert_gather(h, route: dict, k: int, align: int = 0):
-    """Rows of ``h`` [T, H] times their routing weights, sorted by expert (``route`` of ``moe_route``). ``align`` > 0: every
+EXPERT_ACTS = ("none", "swiglu", "gelu")      # what the expert products do with their sums
+
+
+def expert_gather(h, route: dict, k: int, align: int = 0, weighted: bool = True):
+    """Rows of ``h`` [T, H], ``weighted`` times their routing weights, sorted by expert (``route`` of ``moe_route``). ``align`` > 0: every
     expert's slab starts at a multiple of ``align`` rows. Returns (rows, row offsets [E + 1], row of every (token, slot))."""
     n, E, H = route["perm"].numel(), route["counts"].numel(), h.shape[1]
     off, dest = route["offsets"], route["inv"]
@@ -1018,32 +1025,32 @@ def expert_gather(h, route: dict, k: int, align: int = 0):
         rows = -(-(n + min(n, E) * (align - 1)) // align) * align      # only experts with rows pad their slab
         off, dest = torch.empty_like(off), torch.empty_like(dest)
     xs = torch.empty(rows, H, dtype=h.dtype, device=h.device)
-    _chk(lib().pm_expert_gather(_p(h), _is_f32(h), c_ll(h.stride(0)), _p(route["perm"]), _p(route["topk_w"]),
-                                _p(route["offsets"]), c_int(E), c_int(k), c_int(align), c_int(rows), c_int(H), _p(xs),
+    _chk(lib().pm_expert_gather(_p(h), _is_f32(h), c_ll(h.stride(0)), _p(route["perm"]),
+                                _p(route["topk_w"] if weighted else None), _p(route["offsets"]), c_int(E), c_int(k), c_int(align), c_int(rows), c_int(H), _p(xs),
                                 _p(off if align else None), _p(dest if align else None), _stream()), "pm_expert_gather")
     return xs, off, dest
 
 
-def expert_gemv(x, w, route: dict, k: int, glu: bool):
-    """One product of a step with few rows per expert (bf16), in sorted order: ``glu`` with token rows x and w [E, 2 N, K] the
-    gated unit of the weighted inputs, else x (sorted rows) times w [E, N, K]."""
+def expert_gemv(x, w, route: dict, k: int, act: str):
+    """One product of a step with few rows per expert (bf16), in sorted order. ``swiglu``: token rows x and w [E, 2 N, K], the
+    gated unit of the weighted inputs; ``gelu``: token rows x and w [E, N, K]; ``none``: sorted rows x times w [E, N, K]."""
     E, M, K = w.shape
-    N, n = (M // 2 if glu else M), route["perm"].numel()
+    N, n = (M // 2 if act == "swiglu" else M), route["perm"].numel()
     out = torch.empty(n, N, dtype=x.dtype, device=x.device)
     _chk(lib().pm_expert_gemv(_p(x), c_ll(x.stride(0)), _p(w), _p(route["perm"]), _p(route["topk_w"]), _p(route["offsets"]),
-                              c_int(n), c_int(E), c_int(k), c_int(N), c_int(K), c_int(int(glu)), _p(out), _stream()),
+                              c_int(n), c_int(E), c_int(k), c_int(N), c_int(K), c_int(EXPERT_ACTS.index(act)), _p(out), _stream()),
          "pm_expert_gemv")
     return out
 
 
-def expert_rows(x, w, off, glu: bool = False):
-    """Products of expert-sorted rows x [R, K] with w [E, N, K] on the CUDA cores (any size, fp32 or bf16); ``glu``: w is
-    [E, 2 N, K] (gate rows above up rows) and the result silu(gate) * up."""
+def expert_rows(x, w, off, act: str = "none"):
+    """Products of expert-sorted rows x [R, K] with w [E, N, K] on the CUDA cores (any size, fp32 or bf16); ``swiglu``: w is
+    [E, 2 N, K] (gate rows above up rows) and the result silu(gate) * up. Rows behind off[E] are left unwritten."""
     E, M, K = w.shape
-    N = M // 2 if glu else M
+    N = M // 2 if act == "swiglu" else M
     out = torch.empty(x.shape[0], N, dtype=x.dtype, device=x.device)
     _chk(lib().pm_expert_rows(_p(x), _is_f32(x), c_int(x.shape[0]), _p(w), _p(off), c_int(E), c_int(N), c_int(K),
-                              c_int(int(glu)), _p(out), _stream()), "pm_expert_rows")
+                              c_int(EXPERT_ACTS.index(act)), _p(out), _stream()), "pm_expert_rows")
     return out
 
 
@@ -1133,16 +1140,17 @@ def gemv(x, w, norm_w=None, eps: float = 1e-6, residual=None, swiglu: bool = Fal
     return y
 
 
-def gemv_ex(x, w, bias=None, glu=None, out_f32: bool = False, n: Optional[int] = None):
+def gemv_ex(x, w, bias=None, glu=None, out_f32: bool = False, n: Optional[int] = None, gelu: bool = False):
     """x [M <= 16, K] bf16, w [>= n, K] bf16 -> [M, n]: products plus ``bias`` (fp32). ``glu`` = (limit, beta, shift): w
-    stacks gate rows above up rows and the result is the clamped gated unit, n = rows / 2. ``out_f32``: fp32 result."""
+    stacks gate rows above up rows and the result is the clamped gated unit, n = rows / 2. ``gelu``: exact gelu of the sums.
+    ``out_f32``: fp32 result."""
     M, K = x.shape
     N = n if n is not None else (w.shape[0] // 2 if glu else w.shape[0])
     y = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
     lim, beta, shift = glu if glu else (0.0, 0.0, 0.0)
     _chk(lib().pm_gemv_ex(_p(x), c_int(x.stride(0)), _p(w), c_int(w.stride(0)), _p(None), c_float(0.0), _p(None), c_int(0),
                           _p(y), c_int(N), c_int(M), c_int(N), c_int(K), c_int(1 if glu else 0), c_float(1.0), _p(None),
-                          c_int(0), _p(None), c_int(0), (c_int * 4)(*([0x7FFFFFFF] * 4)), _p(bias), c_int(1 if glu else 0),
+                          c_int(0), _p(None), c_int(0), (c_int * 4)(*([0x7FFFFFFF] * 4)), _p(bias), c_int(1 if glu else 2 if gelu else 0),
                           c_float(lim), c_float(beta), c_float(shift), c_int(int(out_f32)), _stream()), "pm_gemv_ex")
     return y
 
@@ -1252,9 +1260,9 @@ def post_layernorm(x, y, w, b, eps: float, alpha: float = 1.0, bias=None, rows=N
 
 
 def add_rmsnorm(x, w, eps: float, y=None, z=None, inv=None, k: int = 1, x0=None, rows=None, dtype=None,
-                want_stream: bool = True, out=None):
-    """v = x + y + (the k rows z[inv] of every token) + x0 on the fp32 stream x [n, width] -> (v or None, v / rms(v) * w in
-    ``dtype``). y (any row stride) and z have the compute type; x0 is fp32; ``rows`` (int64) picks rows of x, y, z and x0.
+                want_stream: bool = True, out=None, w_base: float = 0.0):
+    """v = x + y + (the k rows z[inv] of every token) + x0 on the fp32 stream x [n, width] -> (v or None, v / rms(v) *
+    (w_base + w) in ``dtype``). y (any row stride) and z have the compute type; x0 is fp32; ``rows`` (int64) picks rows of x, y, z and x0.
     ``out``: where v goes (may be x when there are no ``rows``)."""
     n, width = (rows.shape[0] if rows is not None else x.shape[0]), x.shape[1]
     ct = [t for t in (y, z) if t is not None]
@@ -1264,9 +1272,36 @@ def add_rmsnorm(x, w, eps: float, y=None, z=None, inv=None, k: int = 1, x0=None,
     of = (out if out is not None else torch.empty(n, width, dtype=torch.float32, device=x.device)) if want_stream else None
     oc = torch.empty(n, width, dtype=dtype, device=x.device)
     _chk(lib().pm_add_rmsnorm(_p(x), _p(y), c_int(int(dtype == torch.float32)), c_ll(y.stride(0) if y is not None else 0), _p(z),
-                              _p(inv), c_int(k), _p(x0), _p(w), c_float(eps), c_int(n), c_int(width), _p(rows), _p(of), _p(oc),
-                              _stream()), "pm_add_rmsnorm")
+                              _p(inv), c_int(k), _p(x0), _p(w), c_float(w_base), c_float(eps), c_int(n), c_int(width), _p(rows), _p(of),
+                              _p(oc), _stream()), "pm_add_rmsnorm")
     return of, oc
+
+
+def add_normed(x, w, eps: float, y=None, z=None, route=None, k: int = 1, w_base: float = 0.0, out=None, dtype=None):
+    """v = x + r / rms(r) * (w_base + w) with r = y + (the token's k routed rows, weighted) on the fp32 stream x [n, width] ->
+    (v, v in ``dtype``). ``z`` [rows, width] holds the experts' outputs, ``route`` = (weights fp32, chosen outputs, row of z of
+    every (token, slot), number of experts); a choice behind the experts stands for x itself. ``out``: where v goes (may be x)."""
+    n, width = x.shape
+    ct = [t for t in (y, z) if t is not None]
+    dtype = dtype or ct[0].dtype
+    if any(t.dtype != dtype or t.stride(1) != 1 for t in ct):
+        raise ValueError("summands must have the compute type and contiguous rows")
+    of = out if out is not None else torch.empty(n, width, dtype=torch.float32, device=x.device)
+    single = dtype == torch.float32
+    oc = None if single else torch.empty(n, width, dtype=dtype, device=x.device)
+    wt, ids, row, E = route if route is not None else (None, None, None, 0)
+    _chk(lib().pm_add_normed(_p(x), _p(y), c_int(int(single)), c_ll(y.stride(0) if y is not None else 0), _p(z), _p(row), _p(ids),
+                             _p(wt), c_int(k if route is not None else 0), c_int(E), _p(w), c_float(w_base), c_float(eps), c_int(n),
+                             c_int(width), _p(of), _p(oc), _stream()), "pm_add_normed")
+    return of, (of if single else oc)
+
+
+def gelu(x, out=None):
+    """Exact gelu of the rows of x [n, cols]; ``out`` may be x."""
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device) if out is None else out
+    _chk(lib().pm_gelu(_p(x), _is_f32(x), c_ll(x.stride(0)), c_int(x.shape[0]), c_int(x.shape[1]), _p(out), c_ll(out.stride(0)),
+                       _stream()), "pm_gelu")
+    return out
 
 
 def clamped_glu(gu, ff: int, limit: float, beta: float, shift: float, bias=None):
@@ -1333,21 +1368,23 @@ def ssm_gate_norm(y, u, w, eps: float, parts: int, ring, meta, dims):
 
 
 # ------------------------------------------------------------------------------------------- latent attention
-def latent_prep(qd, norm_w, eps: float, cos, sin, dims, pages, slots) -> None:
+def latent_prep(qd, norm_w, eps: float, cos, sin, dims, pages, slots, lead=0, lead_w=None) -> None:
     """Rotates the queries in place; with ``pages`` the latent and rotated key of every token go to its cache row. ``dims`` =
-    (heads, unrotated, rotated, value channels, rank, row width)."""
+    (heads, unrotated, rotated, value channels, rank, row width). ``lead`` > 0: qd holds a query latent of that many channels in
+    place of the queries, which is normed in place with the weight ``lead_w``."""
     H, dn, dr, _, rank, W = dims
     _chk(lib().pm_latent_prep(_p(qd), _is_f32(qd), c_ll(qd.stride(0)), _p(norm_w), c_float(eps), _p(cos), _p(sin),
-                              c_int(qd.shape[0]), c_int(H), c_int(dn), c_int(dr), c_int(rank), _p(pages), c_int(W),
-                              _p(slots), _stream()), "pm_latent_prep")
+                              c_int(qd.shape[0]), c_int(0 if lead else H), c_int(dn), c_int(dr), c_int(rank), _p(pages), c_int(W),
+                              _p(slots), c_int(lead), _p(lead_w), _stream()), "pm_latent_prep")
 
 
 def latent_mma_supported(H: int, W: int, rank: int) -> bool:
     return bool(lib().pm_latent_mma_supported(c_int(H), c_int(W), c_int(rank)))
 
 
-def latent_attn(qd, wuk, wuv, pages, group, dims, scale: float, out) -> None:
-    """Attention in the latent space for the sequences of ``group``: rows of out [tokens, >= heads * value channels]."""
+def latent_attn(qd, wuk, wuv, pages, group, dims, scale: float, out, rope=(None, None)) -> None:
+    """Attention in the latent space for the sequences of ``group``: rows of out [tokens, >= heads * value channels]. ``rope`` =
+    (cos, sin): the queries' rotated parts are turned on the way in."""
     global LAUNCHES
     H, dn, dr, dv, rank, W = dims
     n_split = 1
@@ -1364,7 +1401,8 @@ def latent_attn(qd, wuk, wuv, pages, group, dims, scale: float, out) -> None:
                               _p(group.seq_lens), _p(group.c_start), _p(group.q_lens), _p(group.tok_rows), c_int(group.n),
                               c_int(group.block_table.shape[1]), c_int(group.n_tok), c_int(group.max_q), c_int(H), c_int(dn),
                               c_int(dr), c_int(dv), c_int(rank), c_int(W), c_int(n_split), c_float(scale), _p(q_lat), _p(po),
-                              _p(pml), _p(out), c_ll(out.stride(0)), _p(status_word(dev)), _stream()), "pm_latent_attn")
+                              _p(pml), _p(out), c_ll(out.stride(0)), _p(rope[0]), _p(rope[1]), _p(status_word(dev)), _stream()),
+         "pm_latent_attn")
     LAUNCHES += 2          # three kernels
 
 
@@ -1442,35 +1480,48 @@ def norm_gate(y, gate, w, eps: float, parts: int, silu: bool):
     return out
 
 
-# ------------------------------------------------------------------------------------------- windowed attention, any head size
-def window_prep(u, cs, sn, dims, rot, normed: bool, eps: float, own_v: bool, pages, slots):
-    """Rotated and normalised queries [tokens, heads, head size rounded up to 8]; keys and values of the tokens go to their
-    cache rows. ``dims`` = (query heads, key/value heads, head size), ``rot`` = (rotated channels, layout)."""
-    H, G, D = dims
-    q = torch.empty(u.shape[0], H, -(-D // 8) * 8, dtype=u.dtype, device=u.device)
-    _chk(lib().pm_window_prep(_p(u), _is_f32(u), c_ll(u.stride(0)), _p(cs), _p(sn), c_int(u.shape[0]), c_int(H), c_int(G), c_int(D),
-                              c_int(rot[0]), c_int(int(rot[1] == "pairs")), c_int(int(normed)), c_float(eps), c_int(int(own_v)),
-                              _p(q), _p(pages), _p(slots), _stream()), "pm_window_prep")
+# ------------------------------------------------------------------------------------------- grouped attention, any head size
+def window_prep(u, cs, sn, dims, rot, normed: bool, eps: float, cols, pages, slots, qw=None, kw=None, temp=None, pos=None):
+    """Rotated and normalised queries [tokens, heads * maps, key size rounded up to 8]; with ``pages`` keys and values of the
+    tokens go to their cache rows. ``dims`` = (query heads, key/value heads, maps, key size, value size), ``rot`` = (rotated
+    channels, layout), ``cols`` = columns of u where keys and values begin (the same: the values are the keys as projected),
+    ``qw`` / ``kw`` the norms' weights (fp32), ``temp`` = (coefficient, interval) of the query factor at positions ``pos``."""
+    H, G, M, D, DV = dims
+    q = torch.empty(u.shape[0], H * M, -(-D // 8) * 8, dtype=u.dtype, device=u.device)
+    coef, every = temp if temp is not None else (0.0, 0)
+    _chk(lib().pm_window_prep(_p(u), _is_f32(u), c_ll(u.stride(0)), _p(cs), _p(sn), c_int(u.shape[0]), c_int(H), c_int(G), c_int(M),
+                              c_int(D), c_int(DV), c_int(cols[0]), c_int(cols[1]), c_int(rot[0]), c_int(int(rot[1] == "pairs")),
+                              c_int(int(normed)), c_float(eps), _p(qw), _p(kw), _p(pos), c_float(coef), c_int(every), _p(q),
+                              _p(pages), _p(slots), _stream()), "pm_window_prep")
     return q
 
 
-def window_attn(q, pages, group, dims, window: int, scale: float, few: bool, out) -> None:
-    """Attention of the sequences of ``group`` over their cached keys; rows of out [tokens, >= heads * head size]. ``few``:
-    tiles for a few rows per sequence, pages split over CTAs."""
+def window_attn(q, pages, group, dims, window: int, scale: float, few: bool, out, softcap: float = 0.0, sink=None, gate=None,
+                diff=None) -> None:
+    """Attention of the sequences of ``group`` over their cached keys; rows of out [tokens, >= heads * value size]. ``few``:
+    tiles for a few rows per sequence, pages split over CTAs. ``sink`` fp32 [heads], ``gate`` logits [tokens, heads] of any row
+    stride, ``diff`` = (lambda as an fp32 tensor, factor behind the norm, eps) where a head has two maps."""
     global LAUNCHES
-    H, G, D = dims
-    T, D8, n_split, po, pml = q.shape[0], q.shape[2], 1, None, None
-    if few and q.dtype == torch.bfloat16 and D8 <= 256:
-        ctas = group.n * G * -(-group.max_q * (H // G) // 16)
+    H, G, M, D, DV = dims
+    T, D8, DV8, n_split = q.shape[0], q.shape[2], -(-DV // 8) * 8, 1
+    po = pml = o = None
+    parts = few and q.dtype == torch.bfloat16 and max(D8, DV8) <= 256
+    if parts:
+        ctas = group.n * G * -(-group.max_q * (H // G) * M // 16)
         n_blocks = -(-group.max_kv // 64)
         if window > 0:
             n_blocks = min(n_blocks, -(-(window + group.max_q) // 64) + 1)
         n_split = max(1, min(2 * sm_count() // max(ctas, 1), n_blocks // 2, 32))
-        if n_split > 1:
-            po = torch.empty(n_split, T, H, D8, dtype=torch.float32, device=q.device)
-            pml = torch.empty(n_split, T, H, 2, dtype=torch.float32, device=q.device)
+        if n_split > 1 or M > 1:
+            po = torch.empty(n_split, T, H * M, DV8, dtype=torch.float32, device=q.device)
+            pml = torch.empty(n_split, T, H * M, 2, dtype=torch.float32, device=q.device)
+    if M > 1 and po is None:
+        o = torch.empty(T, H * M * DV, dtype=q.dtype, device=q.device)
+    lam, keep, eps = diff if diff is not None else (None, 1.0, 0.0)
     _chk(lib().pm_window_attn(_p(q), _is_f32(q), _p(pages), _p(group.block_table), _p(group.seq_lens), _p(group.q_start),
                               _p(group.q_lens), c_int(group.n), c_int(group.block_table.shape[1]), c_int(T), c_int(group.max_q),
-                              c_int(H), c_int(G), c_int(D), c_int(window), c_float(scale), c_int(int(few)), c_int(n_split), _p(po),
-                              _p(pml), _p(out), c_ll(out.stride(0)), _stream()), "pm_window_attn")
-    LAUNCHES += int(n_split > 1)
+                              c_int(H), c_int(G), c_int(M), c_int(D), c_int(DV), c_int(window), c_float(scale), c_float(softcap),
+                              _p(sink), _p(gate), c_ll(gate.stride(0) if gate is not None else 0), _p(lam), c_float(keep),
+                              c_float(eps), c_int(int(few)), c_int(n_split), _p(po), _p(pml), _p(o), _p(out), c_ll(out.stride(0)),
+                              _stream()), "pm_window_attn")
+    LAUNCHES += int(po is not None or o is not None)
