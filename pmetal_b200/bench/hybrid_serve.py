@@ -2,7 +2,9 @@
 kernels of the other models (``bench.py --serve-hybrid``). Random weights; device time by CUDA events.
 
 Duvivik presets stand beside the dense fast decoder; Resevik presets beside the Qwen3-MoE decoder with the same width, experts
-and attention heads and one layer per layer run (a looped stack has more runs than stored layers)."""
+and attention heads and one layer per layer run (a looped stack has more runs than stored layers); Vosezen presets beside the same
+with the layers' head counts of 128 channels and experts as wide as makes the stored weights equal (its experts have two matrices
+and a shared one, the other's have three)."""
 from __future__ import annotations
 
 import statistics
@@ -15,7 +17,7 @@ from ..models.config import ModelArgs
 from ..models.decoder import DecoderLM
 from ..models.generation import Generator
 from ..models.kv_cache import BLOCK, PagedKVCache
-from ..models.state_cache import CacheSpec, StateCache, split_groups
+from ..models.state_cache import CacheSpec, StateCache, attention_runs, split_groups
 from ..ops import native as nat
 from .kernels import peaks
 
@@ -29,7 +31,15 @@ DENSE = {
 
 
 def like_kind(name: str) -> str:
-    return "moe" if hd.PRESETS[name]["architecture"] == "Resevik" else "dense"
+    return "dense" if hd.PRESETS[name]["architecture"] == "Duvivik" else "moe"
+
+
+def like_expert_width(ex: dict) -> int:
+    """Width of gated experts with as many weights as those of ``ex`` (a multiple of 128)."""
+    if "shared" not in ex:
+        return ex["expert"]["ff"]
+    E = ex["router"]["experts"]
+    return round(2 * (E * ex["expert"]["ff"] + ex["shared"]["ff"]) / (3 * E * 128)) * 128
 
 
 def build(name: str, kind: str):
@@ -42,8 +52,9 @@ def build(name: str, kind: str):
         ex = next(l["mlp"] for l in args.layers if l["mlp"])
         cfg = ModelArgs(vocab_size=args.vocab_size, hidden_size=args.hidden_size, num_hidden_layers=len(args.runs),
                         num_attention_heads=at["heads"], num_key_value_heads=at["kv_heads"], head_dim=128,
-                        intermediate_size=ex["expert"]["ff"], moe_intermediate_size=ex["expert"]["ff"],
-                        num_experts=ex["router"]["experts"], num_experts_per_tok=ex["router"]["top"], tie_word_embeddings=False)
+                        intermediate_size=like_expert_width(ex), moe_intermediate_size=like_expert_width(ex),
+                        num_experts=ex["router"]["experts"], num_experts_per_tok=ex["router"]["top"],
+                        tie_word_embeddings=args.design.tied)
         m = DecoderLM(cfg, torch.bfloat16, "cuda").init_weights_on_device().eval()
         for p in m.parameters():
             p.requires_grad_(False)
@@ -250,6 +261,132 @@ def parallel_kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: i
     return out
 
 
+def branch_kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096) -> List[dict]:
+    """``kernel_cases`` for the stacks with normed branches (latent attention with latent queries, difference and sink attention,
+    experts with weighted outputs)."""
+    from ..models.moe import WeightedOutputExperts
+    from ..parallel.ep import FusedExpertMoE
+    cfg = hd.HybridArgs.from_dict(hd.PRESETS[name])
+    W = cfg.hidden_size
+    first = lambda kind: next(l["mixer"] for l in cfg.layers if l["type"] == kind)      # noqa: E731
+    at, df, sk = first("latent_attention"), first("attention"), first("attention_2")
+    ex = next(l["mlp"] for l in cfg.layers if l["mlp"])
+    E, I, k, ff, sf = ex["router"]["experts"], ex["router"]["identity"], ex["router"]["top"], ex["expert"]["ff"], ex["shared"]["ff"]
+    pk, out = peaks(), []
+
+    def case(label, fn, nbytes=0, flops=0):
+        us = graph_us(fn)
+        bound = max(nbytes / pk["hbm_gbs"] / 1e3, flops / pk["bf16_tflops"] / 1e6)
+        out.append({"kernel": label, "us": round(us, 2), "bound_us": round(bound, 2), "of_measured_peak": round(bound / us, 3)})
+
+    f = lambda *s: torch.randn(*s, device="cuda")      # noqa: E731
+    experts = WeightedOutputExperts(ex, W, torch.bfloat16, "cuda")
+    ffl = like_expert_width(ex)
+    gu, dn = _bf(E, 2 * ffl, W, scale=0.02), _bf(E, W, ffl, scale=0.02)
+    with torch.no_grad():
+        for t in (experts.up, experts.down, experts.shared_up, experts.shared_down):
+            t.normal_(0.0, 0.02)
+        experts.router.normal_(0.0, W ** -0.5)
+    for mode, n_seq, prior, new in (("decode", batch, ctx - 1, 1), ("prefill", 1, 0, prompt)):
+        T, blocks = n_seq * new, n_seq * (prior + new) // BLOCK + n_seq + 1
+        tag = f"{mode} T={T} "
+        few = mode == "decode"
+        pairs, keys = n_seq * (new * prior + new * (new + 1) // 2), n_seq * (prior + new)
+        # latent attention: the query latent's norm beside the append, both projections of the queries | rotation, append
+        H, dn_, dr, dv, r, qr = at["heads"], at["dim"], at["rot_dim"], at["vdim"], at["kv_rank"], at["q_rank"]
+        row = -(-(r + dr) // 16) * 16
+        dims = (H, dn_, dr, dv, r, row)
+        c = StateCache([CacheSpec(page_width=row + 8)], blocks, n_seq, torch.bfloat16, "cuda")
+        meta, grp = _group(c, n_seq, prior, new)
+        c.pages[0].normal_()
+        u, wukv, cs, sn = _bf(T, qr + r + dr), _bf(H * (dn_ + dv), r, scale=r ** -0.5), f(T, dr // 2), f(T, dr // 2)
+        f_w = f(max(r, qr))
+        qd, o, runs = _bf(T, H * (dn_ + dr)), torch.empty(T, H * dv, dtype=torch.bfloat16, device="cuda"), attention_runs(meta, grp)
+        case(tag + "latent norms + rotation + append",
+             lambda: nat.latent_prep(u, f_w[:r], 1e-5, cs, sn, dims, c.pages[0], meta.slots, qr, f_w[:qr]), T * 2 * (2 * qr + 2 * (r + dr)))if (f_w := f(max(r, qr))) is not None else None
+        u1 = _bf(T, H * (dn_ + dr) + r + dr)
+        case(tag + "  | latent norm + rotation + append", lambda: nat.latent_prep(u1, f_w[:r], 1e-5, cs, sn, dims, c.pages[0], meta.slots),
+             T * 2 * (2 * H * dr + 2 * (r + dr)))
+        if few:
+            nb = keys * row * 2 + wukv.numel() * 2
+            case(tag + f"latent attention with rotation, {ctx} keys",
+                 lambda: nat.latent_attn(qd, wukv, wukv[H * dn_:], c.pages[0], grp, dims, 0.1, o, (cs, sn)), nb)
+            case(tag + "  | latent attention", lambda: nat.latent_attn(qd, wukv, wukv[H * dn_:], c.pages[0], grp, dims, 0.1, o), nb)
+        else:
+            def latent():
+                nat.latent_prep(qd, None, 1e-5, cs, sn, dims, None, meta.slots)
+                nat.latent_expand_attn(qd, wukv, c.pages[0], runs[0], dims, 0.1, o)
+            fl = pairs * H * 2 * (dn_ + dr + dv) + 2 * T * wukv.numel()
+            case(tag + "rotation, latent attention, expanded", latent, 0, fl)
+            case(tag + "  | latent attention, expanded", lambda: nat.latent_expand_attn(qd, wukv, c.pages[0], runs[0], dims, 0.1, o), 0, fl)
+        del c
+        # difference and sink attention | paged attention with as many heads of 128
+        for label, m, M in (("difference", df, 2), ("sink", sk, 1)):
+            H, G, D, DV = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            dims = (H, G, M, D, DV)
+            c = StateCache([CacheSpec(page_width=G * (M * D + DV))], blocks, n_seq, torch.bfloat16, "cuda")
+            meta, grp = _group(c, n_seq, prior, new)
+            c.pages[0].normal_()
+            runs = attention_runs(meta, grp)
+            n_in = H * M * D + G * (M * D + DV) + H
+            ua, wn = _bf(T, -(-n_in // 8) * 8), f(D)
+            cols = (H * M * D, (H + G) * M * D)
+            wide = 0 if few else nat.window_wide(dims, torch.bfloat16, 0)
+            prep = lambda: nat.window_prep(ua, None, None, dims, (0, "none"), True, 1e-5, cols, c.pages[0], meta.slots, wn, wn, (0.3, 512),      # noqa: E731
+                                           meta.positions, wide)
+            case(tag + f"{label}: head norm + query factor + append", prep, 2 * T * (n_in - H) * 2)
+            q, o = prep(), torch.empty(T, H * DV, dtype=torch.bfloat16, device="cuda")
+            gate, lam, s = ua[:, n_in - H:], f(1), f(H)
+            kw = dict(gate=gate, diff=(lam, 0.7, 1e-5)) if M == 2 else dict(gate=gate, softcap=50.0, sink=s)
+            case(tag + f"{label} attention" + (f", {ctx} keys" if few else ""),
+                 lambda: (nat.window_expand_attn(q, c.pages[0], grp, runs, dims, 0.09, o, **kw) if wide else
+                          nat.window_attn(q, c.pages[0], grp, dims, 0, 0.09, few, o, **kw)),
+                 keys * 2 * G * (M * D + DV) if few else 0, pairs * H * M * 2 * (D + DV))
+            del c
+            c3 = PagedKVCache(1, G, 128, blocks, device="cuda")
+            meta3, _ = _group(c3, n_seq, prior, new)
+            c3.k[0].normal_()
+            c3.v[0].normal_()
+            qkv, cs3, sn3, w128 = _bf(T, (H + 2 * G) * 128), f(T, 64), f(T, 64), _bf(128)
+            case(tag + "  | head norm + rotation + append",
+                 lambda: nat.qknorm_rope_cache(qkv, w128, w128, cs3, sn3, H, G, 1e-6, c3.k[0], c3.v[0], meta3.slots),
+                 T * (2 * H + 4 * G) * 128 * 2)
+            q3 = _bf(T, H, 128)
+            case(tag + "  | paged attention", lambda: nat.paged_attn(q3, c3.k[0], c3.v[0], meta3, 0.09),
+                 keys * 2 * G * 256 if few else 0, pairs * H * 4 * 128)
+            del c3
+        # sums
+        x, y, zr, lw, h, rw = f(T, W), _bf(T, W), _bf(T * k, W), f(W), _bf(T, W), _bf(W)
+        inv = torch.randperm(T * k, device="cuda").int()
+        ids, wt = torch.randint(0, E + I, (T, k), device="cuda").int(), torch.rand(T, k, device="cuda")
+        case(tag + "norm of a branch + sum", lambda: nat.add_normed(x, lw, 1e-6, y=y, w_base=1.0, out=x), T * W * (4 + 2 + 4 + 2))
+        case(tag + "weighted rows + norm + sum", lambda: nat.add_normed(x, lw, 1e-6, y=y, z=zr, route=(wt, ids, inv, E), k=k, w_base=1.0, out=x),
+             T * W * (4 + 2 + 2 * k + 4 + 2))
+        case(tag + "  | residual sum + rms norm", lambda: nat.rmsnorm_fwd(h, rw, 1e-6, y), 4 * T * W * 2)
+        # experts
+        z, corr = f(T, E + I), f(E + I) * 0.01
+        gr = ex["router"]["groups"]
+        case(tag + "routing with grouped choice", lambda: nat.moe_route(z, k, False, choice=(corr, gr["count"], gr["keep"], 2.0)),
+             T * (E + I + 4 * k) * 4)
+        case(tag + "  | routing", lambda: nat.moe_route(z, k, True), T * (E + I + 4 * k) * 4)
+        eng = FusedExpertMoE(gu, dn, E, k, T)
+        live = E / (E + I)
+        used = min(E, round(T * k * live))
+        nb = used * 2 * ff * W * 2 + 2 * sf * W * 2 + 2 * T * (k + 1) * (W + ff) * 2
+        case(tag + "router, routing, experts, shared expert", lambda: experts(h), nb, 2 * T * (k * live * 2 * ff + 2 * sf) * W)
+        case(tag + "  | router, routing and experts", lambda: eng.forward(h, torch.nn.functional.linear(h, experts.router[:E])),
+             min(E, T * k) * 3 * ffl * W * 2 + 2 * T * k * (W + ffl) * 2, 2 * T * k * 3 * ffl * W)
+        del eng
+        if not few:
+            a = _bf(T * k, ff)
+            case(tag + "gelu", lambda: nat.gelu(a, a), 2 * a.numel() * 2)
+            b = _bf(T * k, 2 * ff)
+            case(tag + "  | swiglu", lambda: nat.swiglu_fwd(b), 3 * a.numel() * 2)
+        torch.cuda.empty_cache()
+    nat.check_status()
+    return out
+
+
 def kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096) -> List[dict]:
     """Every kernel of the hybrid layers at the sizes of preset ``name`` and, behind it, the like kernel of the other
     models: bytes and operations that the computation needs, device time, fraction of the slower of the two bounds."""
@@ -327,8 +464,8 @@ def kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096
             case(tag + f"latent attention, {ctx} keys", lambda: nat.latent_attn(qd, wukv, wukv[H * dn:], c2.pages[0], grp, dims, 0.1, o),
                  n_seq * ctx * row * 2 + wukv.numel() * 2, pairs * H * 2 * (2 * r + dr))
         else:
-            z = torch.zeros(T, dtype=torch.int32, device="cuda")
-            case(tag + "latent attention, expanded", lambda: nat.latent_expand_attn(qd, wukv, c2.pages[0], meta.block_table[0], T, dims, 0.1, o, z),
+            runs = attention_runs(meta, grp)
+            case(tag + "latent attention, expanded", lambda: nat.latent_expand_attn(qd, wukv, c2.pages[0], runs[0], dims, 0.1, o),
                  0, pairs * H * 2 * (dn + dr + dv) + 2 * T * wukv.numel())
         c3 = PagedKVCache(1, 8, 128, n_seq * (prior + new) // BLOCK + n_seq + 1, device="cuda")
         meta3, _ = _group(c3, n_seq, prior, new)
@@ -356,6 +493,7 @@ def report(names: List[str], kernels: bool = True) -> dict:
             torch.cuda.empty_cache()
         res["models"][n] = row
     if kernels:
-        cases = parallel_kernel_cases if like_kind(names[0]) == "moe" else kernel_cases
+        block = hd.HybridArgs.from_dict(hd.PRESETS[names[0]]).design.block
+        cases = {"post": kernel_cases, "parallel": parallel_kernel_cases, "branch": branch_kernel_cases}[block]
         res["kernels"] = {names[0]: cases(names[0])}
     return res

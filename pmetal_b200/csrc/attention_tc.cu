@@ -42,10 +42,12 @@ __device__ __forceinline__ float row_max(uint32_t taddr, int lo, int span) {
   return mx;
 }
 
-// p = exp2(s * a + b) for the 128 columns of this row, written as bf16 into the swizzled P tile; returns the row sum.
-template <bool kMask>
+// p = exp2(s * a + b) for the 128 columns of this row, written as bf16 into the swizzled P tile; returns the row sum. kCap:
+// p = exp2(b - c / (exp2(s * a) + 1)), a capped score in base 2 when c is twice the cap and b contains the cap
+// (tanh(x) = 1 - 2 / (exp(2 x) + 1)).
+template <bool kMask, bool kCap>
 __device__ __forceinline__ float exp_rows(uint32_t taddr, uint32_t tile_addr, int r, float a, float b, int lo,
-                                          int span) {
+                                          int span, float c2 = 0.f) {
   float rs = 0.f;
 #pragma unroll
   for (int c = 0; c < 4; ++c) {
@@ -55,8 +57,14 @@ __device__ __forceinline__ float exp_rows(uint32_t taddr, uint32_t tile_addr, in
     uint32_t pk[16];
 #pragma unroll
     for (int e = 0; e < 32; e += 2) {
-      float p0 = fast_exp2(fmaf(__uint_as_float(v[e]), a, b));
-      float p1 = fast_exp2(fmaf(__uint_as_float(v[e + 1]), a, b));
+      float p0, p1;
+      if (kCap) {
+        p0 = fast_exp2(fmaf(-c2, fast_rcp(fast_exp2(__uint_as_float(v[e]) * a) + 1.f), b));
+        p1 = fast_exp2(fmaf(-c2, fast_rcp(fast_exp2(__uint_as_float(v[e + 1]) * a) + 1.f), b));
+      } else {
+        p0 = fast_exp2(fmaf(__uint_as_float(v[e]), a, b));
+        p1 = fast_exp2(fmaf(__uint_as_float(v[e + 1]), a, b));
+      }
       if (kMask) {
         const bool any = span >= 0;
         p0 = (any && static_cast<unsigned>(c * 32 + e - lo) <= static_cast<unsigned>(span)) ? p0 : 0.f;
@@ -225,8 +233,8 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_const
         break;
       }
       // pass 2: p = exp2(s * scale - m), row sum, bf16 P into shared memory (128B-swizzled, two 64-key boxes)
-      const float rs = need_mask ? exp_rows<true>(tmem_base + b * 128 + lane_off, sP_addr, r, sl2, -m_use, lo, span)
-                                 : exp_rows<false>(tmem_base + b * 128 + lane_off, sP_addr, r, sl2, -m_use, 0, 0);
+      const float rs = need_mask ? exp_rows<true, false>(tmem_base + b * 128 + lane_off, sP_addr, r, sl2, -m_use, lo, span)
+                                 : exp_rows<false, false>(tmem_base + b * 128 + lane_off, sP_addr, r, sl2, -m_use, 0, 0);
       l_run = l_run * corr + rs;
       fence_async_smem();        // generic-proxy writes of P -> visible to the tensor-core (async) proxy
       tc_fence_before();         // this thread's TMEM reads of S are complete
@@ -355,6 +363,7 @@ __device__ __forceinline__ int fa_work(int k) {
   return k * g + ((k & 1) ? g - 1 - c : c);
 }
 
+template <bool kCap>
 __global__ void __launch_bounds__(kFaThreads2, 1)
 attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const FaParams p) {
@@ -488,7 +497,8 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int qd = warp & 3;
     const int r = qd * 32 + lane;
     const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
-    const float sl2 = p.scale * kFaLog2e;
+    const float cap2 = p.softcap * kFaLog2e;
+    const float sl2 = kCap ? 2.f * kFaLog2e * p.scale / p.softcap : p.scale * kFaLog2e;
     const uint32_t s_tmem = tmem_base + grp * 128 + lane_off;
     const uint32_t o_tmem = tmem_base + 256 + grp * 128 + lane_off;
     const uint32_t o_other = tmem_base + 256 + (grp ^ 1) * 128 + lane_off;
@@ -529,7 +539,9 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const int span = min(min(i + p.shift, p.Tk - 1) - j0, kFaTile - 1) - lo;
         // pass 1 over S_b: row maximum
         const float mx = need_mask ? row_max<true>(s_tmem, lo, span) : row_max<false>(s_tmem, 0, 0);
-        const float m_cand = fmaxf(m_run, mx * sl2);
+        // the cap is monotone: the capped maximum is the maximum of the capped scores
+        const float mc = !kCap ? mx * sl2 : mx == -INFINITY ? mx : fmaf(-2.f * cap2, fast_rcp(fast_exp2(mx * sl2) + 1.f), cap2);
+        const float m_cand = fmaxf(m_run, mc);
         // the previous tile's P·V must be complete: it read P_b and wrote O_b
         if (kk > 0 && !mbar_wait(&bar[kB2OFull + grp], (cnt - 1) & 1, abort_flag, p.status, kTimeoutEpilogue)) {
           ok = false;
@@ -554,8 +566,9 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         }
         const float m_use = (m_run == -INFINITY) ? 0.f : m_run;
         // pass 2 over S_b: p = exp2(s * scale - m), row sum, bf16 P into this group's shared-memory tile
-        const float rs = need_mask ? exp_rows<true>(s_tmem, sP_addr, r, sl2, -m_use, lo, span)
-                                   : exp_rows<false>(s_tmem, sP_addr, r, sl2, -m_use, 0, 0);
+        const float shift2 = kCap ? cap2 - m_use : -m_use;
+        const float rs = need_mask ? exp_rows<true, kCap>(s_tmem, sP_addr, r, sl2, shift2, lo, span, 2.f * cap2)
+                                   : exp_rows<false, kCap>(s_tmem, sP_addr, r, sl2, shift2, 0, 0, 2.f * cap2);
         l_run += rs;
         fence_async_smem();        // generic-proxy writes of P -> visible to the tensor-core (async) proxy
         tc_fence_before();         // TMEM reads / writes of this thread are ordered before the MMA that follows the arrive
@@ -579,11 +592,13 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const float m_o = n_other > 0 ? xo[r] : -INFINITY;
         const float l_o = n_other > 0 ? xo[128 + r] : 0.f;
         const float m_me = kk > 0 ? m_run : -INFINITY;
-        const float m = fmaxf(m_me, m_o);
+        const float s2 = p.sink ? p.sink[it.h] * kFaLog2e : -INFINITY;
+        const float m = fmaxf(fmaxf(m_me, m_o), s2);
         const float a_me = (m_me == -INFINITY) ? 0.f : fast_exp2(m_me - m);
         const float a_o = (m_o == -INFINITY) ? 0.f : fast_exp2(m_o - m);
-        const float l = l_run * a_me + l_o * a_o;
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        const float l = l_run * a_me + l_o * a_o + (p.sink ? fast_exp2(s2 - m) : 0.f);
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        if (p.gate) inv /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(ic) * p.ldg + it.h]));
         const float w_me = a_me * inv, w_o = a_o * inv;
         __nv_bfloat16* orow = p.out + static_cast<long long>(ic) * p.o_stride + static_cast<long long>(it.h) * 128;
 #pragma unroll
@@ -645,8 +660,9 @@ using namespace pm;
 // lse:[hq,T]. Key j is visible to query i iff seq_start[i] <= j <= i + shift.
 static int attn_fwd_tc_launch(int variant, const void* q, long long q_stride, const void* k, long long k_stride,
                               const void* v, long long v_stride, void* out, long long o_stride, float* lse,
-                              const int* seq_start, int T, int Tk, int shift, int hq, int hkv, float scale, int* status,
-                              cudaStream_t st) {
+                              const int* seq_start, int T, int Tk, int shift, int hq, int hkv, float scale, float softcap,
+                              const float* sink, const void* gate, long long ldg, int* status, cudaStream_t st) {
+  if (softcap < 0.f || (variant == 1 && (softcap > 0.f || sink || gate))) return -4;
   if (hq % hkv || T <= 0 || Tk <= 0) return -1;
   if ((q_stride | k_stride | v_stride | o_stride) % 8) return -2;
   CUtensorMap mq, mk, mv;
@@ -660,13 +676,16 @@ static int attn_fwd_tc_launch(int variant, const void* q, long long q_stride, co
   p.o_stride = o_stride; p.lse = lse; p.seq_start = seq_start;
   p.T = T; p.hq = hq; p.hkv = hkv; p.scale = scale; p.status = status;
   p.Tk = Tk; p.shift = shift;
+  p.softcap = softcap; p.sink = sink; p.gate = static_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
   const int smem = 6 * kFaTileBytes + 1024 + 256;
   const int smem2 = 7 * kFaTileBytes + 1024 + 256;
   static DeviceOnce once;
   if (once.pending()) {
     cudaError_t e = cudaFuncSetAttribute(attn_fwd_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
-    e = cudaFuncSetAttribute(attn_fwd_tc2_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
+    e = cudaFuncSetAttribute(attn_fwd_tc2_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    e = cudaFuncSetAttribute(attn_fwd_tc2_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
     if (e != cudaSuccess) return static_cast<int>(e);
     once.mark();
   }
@@ -675,7 +694,9 @@ static int attn_fwd_tc_launch(int variant, const void* q, long long q_stride, co
     attn_fwd_tc_kernel<<<grid, kFaThreads, smem, st>>>(mq, mk, mv, p);
   } else {
     const int items = static_cast<int>(grid.x) * hq;      // persistent: one CTA per SM walks the item list
-    attn_fwd_tc2_kernel<<<items < num_sms() ? items : num_sms(), kFaThreads2, smem2, st>>>(mq, mk, mv, p);
+    const int ctas = items < num_sms() ? items : num_sms();
+    if (softcap > 0.f) attn_fwd_tc2_kernel<true><<<ctas, kFaThreads2, smem2, st>>>(mq, mk, mv, p);
+    else attn_fwd_tc2_kernel<false><<<ctas, kFaThreads2, smem2, st>>>(mq, mk, mv, p);
   }
   return static_cast<int>(cudaGetLastError());
 }
@@ -685,7 +706,17 @@ extern "C" int pm_attn_fwd_tc_rect(const void* q, long long q_stride, const void
                                    int T, int Tk, int shift, int hq, int hkv, float scale, int* status,
                                    cudaStream_t st) {
   return attn_fwd_tc_launch(2, q, q_stride, k, k_stride, v, v_stride, out, o_stride, lse, seq_start, T, Tk, shift, hq,
-                            hkv, scale, status, st);
+                            hkv, scale, 0.f, nullptr, nullptr, 0, status, st);
+}
+
+// pm_attn_fwd_tc_rect with capped scores (softcap > 0: softcap tanh(score / softcap)), a sink per head (fp32 [hq], nullable:
+// exp(sink) joins the softmax sum) and an output gate (bf16 [T, ldg], nullable: head h times the sigmoid of column h).
+extern "C" int pm_attn_fwd_tc_ex(const void* q, long long q_stride, const void* k, long long k_stride, const void* v,
+                                 long long v_stride, void* out, long long o_stride, float* lse, const int* seq_start,
+                                 int T, int Tk, int shift, int hq, int hkv, float scale, float softcap, const float* sink,
+                                 const void* gate, long long ldg, int* status, cudaStream_t st) {
+  return attn_fwd_tc_launch(2, q, q_stride, k, k_stride, v, v_stride, out, o_stride, lse, seq_start, T, Tk, shift, hq,
+                            hkv, scale, softcap, sink, gate, ldg, status, st);
 }
 
 // Single-softmax-group variant of the same kernel (kept selectable for comparison measurements).
@@ -694,7 +725,7 @@ extern "C" int pm_attn_fwd_tc_rect_v1(const void* q, long long q_stride, const v
                                       const int* seq_start, int T, int Tk, int shift, int hq, int hkv, float scale,
                                       int* status, cudaStream_t st) {
   return attn_fwd_tc_launch(1, q, q_stride, k, k_stride, v, v_stride, out, o_stride, lse, seq_start, T, Tk, shift, hq,
-                            hkv, scale, status, st);
+                            hkv, scale, 0.f, nullptr, nullptr, 0, status, st);
 }
 
 extern "C" int pm_attn_fwd_tc(const void* q, long long q_stride, const void* k, long long k_stride, const void* v,

@@ -25,12 +25,25 @@ struct FaParams {
   // seq_start[i] <= j <= i + shift (and j < Tk). Tk = T, shift = 0 is ordinary causal attention; shift >= Tk - 1
   // makes every key visible (a block of ring attention that lies entirely in the past).
   int Tk, shift;
+  // forward kernel only: scores become softcap * tanh(score / softcap) when softcap > 0; sink [hq] (nullable) adds exp(sink_h) to
+  // the softmax sum of head h; gate [T, ldg] (nullable) multiplies head h of the output by the sigmoid of column h
+  float softcap;
+  const float* sink;
+  const __nv_bfloat16* gate;
+  long long ldg;
 };
 
 // 2^x on the SFU; -inf gives 0
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// 1 / x on the SFU; 1 / inf gives 0
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
 

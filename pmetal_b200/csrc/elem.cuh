@@ -96,6 +96,7 @@ __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); 
 __device__ __forceinline__ float sigmoid_fast(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
 __device__ __forceinline__ float silu_fast(float v) { return v * sigmoid_fast(v); }
 __device__ __forceinline__ float gelu_f(float v) { return 0.5f * v * erfcf(-0.70710678118654752f * v); }
+__device__ __forceinline__ float gelu_fast(float v) { return 0.5f * v * (1.f + erff(0.70710678118654752f * v)); }      // for bf16 results
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
 template <bool kFast = false>

@@ -72,7 +72,7 @@ __device__ __forceinline__ void gv_finish(const GemvParams& p, int m, int n, flo
     if (p.bias) v2 += p.bias[n + p.N];
     v = p.clamped ? clamped_glu(v, v2, p.glu_limit, p.glu_beta, p.glu_shift) : gv_silu(v) * v2;
   } else if (p.clamped == 2) {
-    v = gelu_f(v);
+    v = gelu_fast(v);
   }
   if (p.residual) v += __bfloat162float(p.residual[static_cast<long long>(m) * p.ldr + n]);
   if (p.y_f32) p.y_f32[static_cast<long long>(m) * p.ldy + n] = v;

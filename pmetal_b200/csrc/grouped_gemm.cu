@@ -32,6 +32,7 @@ struct GroupedParams {
   int accumulate;    // mode 2: add to D instead of overwriting
   float alpha;
   int* status;
+  int gelu;              // mode 0: exact gelu of the products
 };
 
 struct GroupTile {
@@ -228,21 +229,26 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         tmem_ld_wait();
         const int col0 = t.out_col + c * 32;
         if (!row_ok || col0 >= out_cols) continue;
+        if (p.gelu) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(gelu_fast(__uint_as_float(r[e]) * p.alpha));
+        }
+        const float alpha = p.gelu ? 1.f : p.alpha;
         if (p.mode < 2) {
           __nv_bfloat16* drow = static_cast<__nv_bfloat16*>(p.D) + static_cast<size_t>(row) * p.ldd + col0;
           if (col0 + 32 <= out_cols) {
 #pragma unroll
             for (int v = 0; v < 4; ++v) {
               uint4 o;
-              o.x = pack_bf16x2(__uint_as_float(r[v * 8]) * p.alpha, __uint_as_float(r[v * 8 + 1]) * p.alpha);
-              o.y = pack_bf16x2(__uint_as_float(r[v * 8 + 2]) * p.alpha, __uint_as_float(r[v * 8 + 3]) * p.alpha);
-              o.z = pack_bf16x2(__uint_as_float(r[v * 8 + 4]) * p.alpha, __uint_as_float(r[v * 8 + 5]) * p.alpha);
-              o.w = pack_bf16x2(__uint_as_float(r[v * 8 + 6]) * p.alpha, __uint_as_float(r[v * 8 + 7]) * p.alpha);
+              o.x = pack_bf16x2(__uint_as_float(r[v * 8]) * alpha, __uint_as_float(r[v * 8 + 1]) * alpha);
+              o.y = pack_bf16x2(__uint_as_float(r[v * 8 + 2]) * alpha, __uint_as_float(r[v * 8 + 3]) * alpha);
+              o.z = pack_bf16x2(__uint_as_float(r[v * 8 + 4]) * alpha, __uint_as_float(r[v * 8 + 5]) * alpha);
+              o.w = pack_bf16x2(__uint_as_float(r[v * 8 + 6]) * alpha, __uint_as_float(r[v * 8 + 7]) * alpha);
               *reinterpret_cast<uint4*>(drow + v * 8) = o;
             }
           } else {
             for (int e = 0; e < 32 && col0 + e < out_cols; ++e)
-              drow[e] = __float2bfloat16(__uint_as_float(r[e]) * p.alpha);
+              drow[e] = __float2bfloat16(__uint_as_float(r[e]) * alpha);
           }
         } else {
           float* drow = static_cast<float*>(p.D) + t.out_base + static_cast<size_t>(row) * p.ldd + col0;
@@ -432,7 +438,7 @@ grouped_gemm_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
               for (int j = 0; j < 32; ++j)
                 if (c * 32 + j < live) {
                   const float v = __uint_as_float(r[j]) * p.alpha;
-                  d[static_cast<size_t>(j) * p.ldd] = __float2bfloat16(p.gelu ? gelu_f(v) : v);
+                  d[static_cast<size_t>(j) * p.ldd] = __float2bfloat16(p.gelu ? gelu_fast(v) : v);
                 }
             }
           }
@@ -507,15 +513,16 @@ using namespace pm;
 
 // a, b: the two operands of the mode (see the table at the top); both bf16, row strides lda / ldb in elements.
 // off: int32 [E + 1] on the device, multiples of 128, off[E] <= rows_cap. D: bf16 [rows_cap, ldd] (modes 0, 1) or fp32
-// [E, N, ldd] (mode 2; experts without rows are left untouched, so clear D first unless accumulating).
+// [E, N, ldd] (mode 2; experts without rows are left untouched, so clear D first unless accumulating). gelu (mode 0): exact gelu of
+// the products.
 extern "C" int pm_grouped_gemm(int mode, const void* a, int lda, const void* b, int ldb, void* D, int ldd, const int* off,
-                               int E, int rows_cap, int N, int K, float alpha, int accumulate, int* status,
+                               int E, int rows_cap, int N, int K, float alpha, int accumulate, int gelu, int* status,
                                cudaStream_t stream) {
-  if (mode < 0 || mode > 2 || E < 1 || rows_cap <= 0 || (rows_cap % kBM) || N <= 0 || K <= 0) return -1;
+  if (mode < 0 || mode > 2 || (gelu && mode) || E < 1 || rows_cap <= 0 || (rows_cap % kBM) || N <= 0 || K <= 0) return -1;
   if ((N % 8) || (K % 8) || (ldd % 8 && mode < 2)) return -2;
   GroupedParams p{};
   p.mode = mode; p.E = E; p.rows_cap = rows_cap; p.N = N; p.K = K;
-  p.off = off; p.D = D; p.ldd = ldd; p.accumulate = accumulate; p.alpha = alpha; p.status = status;
+  p.off = off; p.D = D; p.ldd = ldd; p.accumulate = accumulate; p.gelu = gelu; p.alpha = alpha; p.status = status;
   const int out_cols = mode == 0 ? N : K;
   int bn = 256;
   while (bn > 64 && bn / 2 >= out_cols) bn /= 2;

@@ -55,7 +55,28 @@ __device__ __forceinline__ void load_pair(const __nv_bfloat16* p, float (&v)[V])
 
 // One CTA per token. qd [tokens, ld]: H heads of [D_n | D_r] or (lead > 0, H = 0) a query latent of `lead` channels, which is
 // normed in place; then (own != 0) the down-projection [R | D_r].
-template <typename T>
+// V: elements per access of the norms.
+template <typename T, int V>
+__device__ __forceinline__ void latent_norm_row(const T* src, T* dst, const float* __restrict__ w, int n, float eps) {
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
+    float v[V];
+    load_vec<V>(src + i, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
+  }
+  const float r = 1.f / sqrtf(block_sum(ss) / static_cast<float>(n) + eps);
+  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
+    float v[V], ww[V];
+    load_vec<V>(src + i, v);
+    load_vec<V>(w + i, ww);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] *= r * ww[e];
+    store_vec<V>(dst + i, v);
+  }
+}
+
+template <typename T, int V>
 __global__ void latent_prep_kernel(T* __restrict__ qd, long long ld, const float* __restrict__ norm_w, float eps,
                                    const float* __restrict__ cs, const float* __restrict__ sn, int H, int dn, int dr, int rank,
                                    int own, T* __restrict__ cache, int W, const long long* __restrict__ slots, int lead,
@@ -72,25 +93,11 @@ __global__ void latent_prep_kernel(T* __restrict__ qd, long long ld, const float
     put(p, a * c[j] - b * s[j]);
     put(p + 1, b * c[j] + a * s[j]);
   }
-  if (lead > 0) {
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < lead; i += blockDim.x) {
-      const float v = to_f(row[i]);
-      ss = fmaf(v, v, ss);
-    }
-    const float r = 1.f / sqrtf(block_sum(ss) / static_cast<float>(lead) + eps);
-    for (int i = threadIdx.x; i < lead; i += blockDim.x) put(row + i, to_f(row[i]) * r * lead_w[i]);
-  }
+  if (lead > 0) latent_norm_row<T, V>(row, row, lead_w, lead, eps);
   if (!own) return;
   const T* d = row + H * (dn + dr) + lead;
   T* dst = cache + slots[t] * (W + kRowPad);
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-    const float v = to_f(d[i]);
-    ss = fmaf(v, v, ss);
-  }
-  const float r = 1.f / sqrtf(block_sum(ss) / static_cast<float>(rank) + eps);
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) put(dst + i, to_f(d[i]) * r * norm_w[i]);
+  latent_norm_row<T, V>(d, dst, norm_w, rank, eps);
   for (int j = threadIdx.x; j < half; j += blockDim.x) {
     const float a = to_f(d[rank + 2 * j]), b = to_f(d[rank + 2 * j + 1]);
     put(dst + rank + 2 * j, a * c[j] - b * s[j]);
@@ -559,23 +566,23 @@ __global__ void __launch_bounds__(256) latent_up_kernel(const float* __restrict_
 }
 
 // ------------------------------------------------------------------------------------------- expanded keys and values
-// lat [n, R8] (R8 >= rank, zero padded) = latents of one sequence's first n positions, read through its block table row.
-__global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ table, int n, int W,
+// lat [n, R8] (R8 >= rank, zero padded) = latents of the n cache rows in `slots` (page * 64 + offset).
+__global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, const long long* __restrict__ slots, int n, int W,
                                      int rank, int r8, __nv_bfloat16* __restrict__ lat) {
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < static_cast<long long>(n) * r8;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
     const int j = static_cast<int>(i / r8), c = static_cast<int>(i - static_cast<long long>(j) * r8);
-    const __nv_bfloat16* src = cache + (static_cast<long long>(table[j / kPage]) * kPage + j % kPage) * (W + kRowPad);
+    const __nv_bfloat16* src = cache + slots[j] * (W + kRowPad);
     lat[i] = c < rank ? src[c] : __float2bfloat16(0.f);
   }
 }
-__global__ void latent_gather8_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ table, int n, int W,
+__global__ void latent_gather8_kernel(const __nv_bfloat16* __restrict__ cache, const long long* __restrict__ slots, int n, int W,
                                       int rank, __nv_bfloat16* __restrict__ lat) {
   const int per = rank / 8;
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < static_cast<long long>(n) * per;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
     const int j = static_cast<int>(i / per), c = static_cast<int>(i - static_cast<long long>(j) * per) * 8;
-    const __nv_bfloat16* src = cache + (static_cast<long long>(table[j / kPage]) * kPage + j % kPage) * (W + kRowPad);
+    const __nv_bfloat16* src = cache + slots[j] * (W + kRowPad);
     *reinterpret_cast<uint4*>(lat + static_cast<long long>(j) * rank + c) = *reinterpret_cast<const uint4*>(src + c);
   }
 }
@@ -585,7 +592,7 @@ __global__ void latent_gather8_kernel(const __nv_bfloat16* __restrict__ cache, c
 // A thread writes 8 channels. Operands without a destination are left out.
 __global__ void latent_assemble_kernel(const __nv_bfloat16* __restrict__ qd, long long ldq, int n_q,
                                        const __nv_bfloat16* __restrict__ kv, long long ldkv, int n,
-                                       const __nv_bfloat16* __restrict__ cache, const int* __restrict__ table, int W, int rank,
+                                       const __nv_bfloat16* __restrict__ cache, const long long* __restrict__ slots, int W, int rank,
                                        int H, int dn, int dr, int dv, __nv_bfloat16* __restrict__ q128,
                                        __nv_bfloat16* __restrict__ k128, __nv_bfloat16* __restrict__ v128) {
   const int what = blockIdx.y;
@@ -605,7 +612,7 @@ __global__ void latent_assemble_kernel(const __nv_bfloat16* __restrict__ qd, lon
       na = nb = dn + dr;
     } else if (what == 1) {
       a = kv + t * ldkv + h * dn;
-      b = cache + (static_cast<long long>(table[t / kPage]) * kPage + t % kPage) * (W + kRowPad) + rank;
+      b = cache + slots[t] * (W + kRowPad) + rank;
       na = dn;
       nb = dn + dr;
     } else {
@@ -707,12 +714,15 @@ extern "C" int pm_latent_prep(void* qd, int f32, long long ld, const float* norm
   if (ld < static_cast<long long>(H) * (dn + dr) + lead + (cache ? rank + dr : 0)) return -2;
   if (n == 0) return 0;
   const int own = cache != nullptr;
-  if (f32)
-    latent_prep_kernel<float><<<n, 128, 0, st>>>(static_cast<float*>(qd), ld, norm_w, eps, cs, sn, H, dn, dr, rank, own,
-                                                 static_cast<float*>(cache), W, slots, lead, lead_w);
-  else
-    latent_prep_kernel<__nv_bfloat16><<<n, 128, 0, st>>>(static_cast<__nv_bfloat16*>(qd), ld, norm_w, eps, cs, sn, H, dn, dr,
-                                                         rank, own, static_cast<__nv_bfloat16*>(cache), W, slots, lead, lead_w);
+  if (f32) {
+    latent_prep_kernel<float, 1><<<n, 128, 0, st>>>(static_cast<float*>(qd), ld, norm_w, eps, cs, sn, H, dn, dr, rank, own,
+                                                    static_cast<float*>(cache), W, slots, lead, lead_w);
+  } else {
+    const bool vec = ((H * (dn + dr)) | lead | (own ? rank : 0) | static_cast<int>(ld % 8)) % 8 == 0 && reinterpret_cast<uintptr_t>(qd) % 16 == 0;
+    const auto kernel = vec ? latent_prep_kernel<__nv_bfloat16, 8> : latent_prep_kernel<__nv_bfloat16, 1>;
+    kernel<<<n, 128, 0, st>>>(static_cast<__nv_bfloat16*>(qd), ld, norm_w, eps, cs, sn, H, dn, dr, rank, own,
+                              static_cast<__nv_bfloat16*>(cache), W, slots, lead, lead_w);
+  }
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -780,8 +790,8 @@ extern "C" int pm_latent_attn(const void* qd, int f32, long long ld, const void*
              : latent_up_launch<__nv_bfloat16>(part_o, part_ml, wuv, tok_rows, n_tok, H, dv, rank, n_split, g_up, sm_up, out, ldo, st);
 }
 
-// lat [n, r8] bf16 = latents of positions 0 .. n - 1 of the sequence whose block table row is `table` (zero padded).
-extern "C" int pm_latent_gather(const void* cache, const int* table, int n, int W, int rank, int r8, void* lat,
+// lat [n, r8] bf16 = latents of the n cache rows in `slots` (page * 64 + offset; zero padded).
+extern "C" int pm_latent_gather(const void* cache, const long long* slots, int n, int W, int rank, int r8, void* lat,
                                 cudaStream_t st) {
   if (n < 0 || rank < 1 || r8 < rank || W < rank) return -1;
   if (n == 0) return 0;
@@ -789,25 +799,25 @@ extern "C" int pm_latent_gather(const void* cache, const int* table, int n, int 
   long long grid = (static_cast<long long>(n) * (vec ? rank / 8 : r8) + 255) / 256;
   if (grid > num_sms() * 16) grid = num_sms() * 16;
   if (vec)
-    latent_gather8_kernel<<<static_cast<int>(grid), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(cache), table, n, W, rank,
+    latent_gather8_kernel<<<static_cast<int>(grid), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(cache), slots, n, W, rank,
                                                                   static_cast<__nv_bfloat16*>(lat));
   else
-    latent_gather_kernel<<<static_cast<int>(grid), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(cache), table, n, W, rank,
+    latent_gather_kernel<<<static_cast<int>(grid), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(cache), slots, n, W, rank,
                                                                  r8, static_cast<__nv_bfloat16*>(lat));
   return static_cast<int>(cudaGetLastError());
 }
 
-// Operands [.., H, 128] bf16 of the flash-attention kernels for n_q queries and n keys of one sequence; dn + dr <= 128,
+// Operands [.., H, 128] bf16 of the flash-attention kernels for n_q queries and the n keys in `slots`; dn + dr <= 128,
 // dv <= 128. qd: the first query row; kv [n, ldkv] = [keys: H * dn | values: H * dv].
 extern "C" int pm_latent_assemble(const void* qd, long long ldq, int n_q, const void* kv, long long ldkv, int n,
-                                  const void* cache, const int* table, int W, int rank, int H, int dn, int dr, int dv,
+                                  const void* cache, const long long* slots, int W, int rank, int H, int dn, int dr, int dv,
                                   void* q128, void* k128, void* v128, cudaStream_t st) {
   if (n_q < 1 || n < 1 || H < 1 || dn + dr > 128 || dv > 128 || W < rank + dr) return -1;
   long long grid = (static_cast<long long>(n > n_q ? n : n_q) * H * 16 + 255) / 256;
   if (grid > num_sms() * 16) grid = num_sms() * 16;
   latent_assemble_kernel<<<dim3(static_cast<int>(grid), 3), 256, 0, st>>>(
       static_cast<const __nv_bfloat16*>(qd), ldq, n_q, static_cast<const __nv_bfloat16*>(kv), ldkv, n,
-      static_cast<const __nv_bfloat16*>(cache), table, W, rank, H, dn, dr, dv, static_cast<__nv_bfloat16*>(q128),
+      static_cast<const __nv_bfloat16*>(cache), slots, W, rank, H, dn, dr, dv, static_cast<__nv_bfloat16*>(q128),
       static_cast<__nv_bfloat16*>(k128), static_cast<__nv_bfloat16*>(v128));
   return static_cast<int>(cudaGetLastError());
 }

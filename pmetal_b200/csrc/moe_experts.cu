@@ -1,6 +1,7 @@
 // Routed experts, two forms: a gated unit whose routing weight multiplies the expert's input, y = sum over a token's experts of
 // down(silu(G w h) * (U w h)), and plain units y = sum of w down(gelu(U h)), whose weights the caller applies to the rows.
 // The (token, slot) pairs come sorted by expert (moe_quant.cu); pairs behind the last expert (offsets off[E] ..) are left alone:
+//   router_logits_kernel   fp32 logits of a few experts for many tokens
 //   expert_gather_kernel   rows w h (or h) in sorted order, or in a layout whose slabs start at multiples of `align` rows (zero rows
 //                          between them), for the grouped tensor-core GEMMs (grouped_gemm.cu)
 //   expert_gemv_kernel     a few rows per expert (decode, bf16): every weight row is read once by one warp and multiplied with
@@ -13,9 +14,52 @@
 #include <type_traits>
 #include "elem.cuh"
 #include "host_util.cuh"
+#include "mma_sync.cuh"
 #include "pmetal_b200.h"
 
 namespace pm {
+
+// out [T, n] fp32 = h W^T for n <= 8 NT outputs: a CTA takes 16 tokens, its eight warps cut K into pieces of 32 in turn and meet in
+// shared memory. A lane loads 8 consecutive values of a row: the order of K inside a piece is the same for both operands, so it
+// need not be the one of the fragment layout.
+constexpr int kRouterWarps = 8;
+template <int NT>
+__global__ void __launch_bounds__(kRouterWarps * 32) router_logits_kernel(const __nv_bfloat16* __restrict__ h, long long ldh,
+                                                                          const __nv_bfloat16* __restrict__ W, int T, int n, int K,
+                                                                          float* __restrict__ out) {
+  __shared__ float part[kRouterWarps][16][8 * NT + 1];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, t4 = lane & 3, t0 = blockIdx.x * 16;
+  const __nv_bfloat16* a0 = h + static_cast<long long>(min(t0 + g4, T - 1)) * ldh + t4 * 8;
+  const __nv_bfloat16* a1 = h + static_cast<long long>(min(t0 + g4 + 8, T - 1)) * ldh + t4 * 8;
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+#pragma unroll 2
+  for (int k = warp * 32; k < K; k += kRouterWarps * 32) {
+    const uint4 x = *reinterpret_cast<const uint4*>(a0 + k), y = *reinterpret_cast<const uint4*>(a1 + k);
+    const uint32_t fa[4] = {x.x, y.x, x.y, y.y}, fb[4] = {x.z, y.z, x.w, y.w};
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const uint4 w = __ldg(reinterpret_cast<const uint4*>(W + static_cast<long long>(min(i * 8 + g4, n - 1)) * K + t4 * 8 + k));
+      ms_mma(acc[i], fa, w.x, w.y);
+      ms_mma(acc[i], fb, w.z, w.w);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) part[warp][g4 + 8 * (e >> 1)][i * 8 + 2 * t4 + (e & 1)] = acc[i][e];
+  __syncthreads();
+  for (int i = threadIdx.x; i < 16 * n; i += kRouterWarps * 32) {
+    const int r = i / n, c = i - r * n;
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < kRouterWarps; ++w) v += part[w][r][c];
+    if (t0 + r < T) out[static_cast<long long>(t0 + r) * n + c] = v;
+  }
+}
 
 // Largest e with off[e] <= row (off non-decreasing, row < off[E]).
 __device__ __forceinline__ int expert_at(const int* __restrict__ off, int E, int row) {
@@ -157,7 +201,7 @@ __global__ void __launch_bounds__(128) expert_gemv_kernel(const ExpertGemvParams
         for (int i = 0; i < kPer; ++i)
           if (c0 + i < p.N)
             dst[i] = __float2bfloat16(GLU ? silu_fast(acc[2 * i % 4][r] * f) * (acc[(2 * i + 1) % 4][r] * f)
-                                          : ACT == kActGelu ? gelu_f(acc[i][r]) : acc[i][r]);
+                                          : ACT == kActGelu ? gelu_fast(acc[i][r]) : acc[i][r]);
       }
     }
   };
@@ -234,6 +278,16 @@ static int gather_launch(const void* h, long long ldh, const int* perm, const fl
 }  // namespace pm
 
 using namespace pm;
+
+// out [T, n] fp32 = h [T, K] W^T (bf16, W [>= n, K]) for at most 64 outputs; K a multiple of 32, ldh of 8.
+extern "C" int pm_router_logits(const void* h, long long ldh, const void* W, int T, int n, int K, float* out, cudaStream_t st) {
+  if (n < 1 || n > 64 || K < 32 || K % 32 || ldh % 8 || ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(W)) & 15)) return -1;
+  if (T < 1) return 0;
+  const auto kernel = n <= 16 ? router_logits_kernel<2> : n <= 32 ? router_logits_kernel<4> : router_logits_kernel<8>;
+  kernel<<<(T + 15) / 16, kRouterWarps * 32, 0, st>>>(static_cast<const __nv_bfloat16*>(h), ldh, static_cast<const __nv_bfloat16*>(W),
+                                                      T, n, K, out);
+  return static_cast<int>(cudaGetLastError());
+}
 
 // xs [rows, width] = w[pair] * h[pair / k] (w null: h) for the pairs perm[0 .. n) sorted by expert (off [E + 1]). align 0: rows = n in
 // sorted order. align > 0: every expert's slab starts at a multiple of align (off_pad [E + 1]), dest [n] is the row of each

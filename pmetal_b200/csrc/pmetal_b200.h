@@ -58,6 +58,12 @@ const char* pm_paged_attn_static_strerror(int code);
 int pm_attn_fwd_tc_rect(const void* q, long long q_stride, const void* k, long long k_stride, const void* v, long
     long v_stride, void* out, long long o_stride, float* lse, const int* seq_start, int T, int Tk, int shift, int
     hq, int hkv, float scale, int* status, cudaStream_t st);
+// pm_attn_fwd_tc_rect with capped scores (softcap > 0: softcap tanh(score / softcap)), a sink per head (fp32 [hq], nullable:
+// exp(sink) joins the softmax sum) and an output gate (bf16 [T, ldg], nullable: head h times the sigmoid of column h).
+int pm_attn_fwd_tc_ex(const void* q, long long q_stride, const void* k, long long k_stride, const void* v, long
+    long v_stride, void* out, long long o_stride, float* lse, const int* seq_start, int T, int Tk, int shift, int
+    hq, int hkv, float scale, float softcap, const float* sink, const void* gate, long long ldg, int* status,
+    cudaStream_t st);
 // Single-softmax-group variant of the same kernel (kept selectable for comparison measurements).
 int pm_attn_fwd_tc_rect_v1(const void* q, long long q_stride, const void* k, long long k_stride, const void* v,
     long long v_stride, void* out, long long o_stride, float* lse, const int* seq_start, int T, int Tk, int shift,
@@ -193,9 +199,10 @@ int pm_gemv_q4(const void* x, int ldx, const void* qdata, const float* absmax, c
 // ---------------------------------------------------------------- grouped_gemm.cu
 // a, b: the two operands of the mode (see the table at the top); both bf16, row strides lda / ldb in elements.
 // off: int32 [E + 1] on the device, multiples of 128, off[E] <= rows_cap. D: bf16 [rows_cap, ldd] (modes 0, 1) or fp32
-// [E, N, ldd] (mode 2; experts without rows are left untouched, so clear D first unless accumulating).
+// [E, N, ldd] (mode 2; experts without rows are left untouched, so clear D first unless accumulating). gelu (mode 0): exact gelu of
+// the products.
 int pm_grouped_gemm(int mode, const void* a, int lda, const void* b, int ldb, void* D, int ldd, const int* off, int
-    E, int rows_cap, int N, int K, float alpha, int accumulate, int* status, cudaStream_t stream);
+    E, int rows_cap, int N, int K, float alpha, int accumulate, int gelu, int* status, cudaStream_t stream);
 // Few rows per expert (see the kernel): x [rows, K] expert-sorted with offsets off [E + 1] (any alignment), w stacked
 // [E * N, K] (act 0; act 2: exact gelu of the products) or [E * 2N, K] with gate rows above up rows per expert (act 1); y [rows, N] bf16.
 // bn (32, 64, 128) is the token tile: experts with more rows take several passes over their weights.
@@ -221,14 +228,14 @@ int pm_latent_attn(const void* qd, int f32, long long ld, const void* wuk, const
     n_seq, int max_blocks, int n_tok, int max_q, int H, int dn, int dr, int dv, int rank, int W, int n_split, float
     scale, void* q_lat, float* part_o, float* part_ml, void* out, long long ldo, const float* cs, const float* sn,
     int* status, cudaStream_t st);
-// lat [n, r8] bf16 = latents of positions 0 .. n - 1 of the sequence whose block table row is `table` (zero padded).
-int pm_latent_gather(const void* cache, const int* table, int n, int W, int rank, int r8, void* lat, cudaStream_t
-    st);
-// Operands [.., H, 128] bf16 of the flash-attention kernels for n_q queries and n keys of one sequence; dn + dr <= 128,
+// lat [n, r8] bf16 = latents of the n cache rows in `slots` (page * 64 + offset; zero padded).
+int pm_latent_gather(const void* cache, const long long* slots, int n, int W, int rank, int r8, void* lat,
+    cudaStream_t st);
+// Operands [.., H, 128] bf16 of the flash-attention kernels for n_q queries and the n keys in `slots`; dn + dr <= 128,
 // dv <= 128. qd: the first query row; kv [n, ldkv] = [keys: H * dn | values: H * dv].
 int pm_latent_assemble(const void* qd, long long ldq, int n_q, const void* kv, long long ldkv, int n, const void*
-    cache, const int* table, int W, int rank, int H, int dn, int dr, int dv, void* q128, void* k128, void* v128,
-    cudaStream_t st);
+    cache, const long long* slots, int W, int rank, int H, int dn, int dr, int dv, void* q128, void* k128, void*
+    v128, cudaStream_t st);
 // out [n, ldo] (H * dv columns) = the first dv channels of every head of o128 [n, H, 128].
 int pm_latent_take(const void* o128, int n, int H, int dv, void* out, long long ldo, cudaStream_t st);
 
@@ -273,6 +280,9 @@ int pm_mhc_expand(const void* x, int T, int n, int C, void* xs, cudaStream_t st)
 int pm_mhc_collapse(const void* xs, int T, int n, int C, void* x, cudaStream_t st);
 
 // ---------------------------------------------------------------- moe_experts.cu
+// out [T, n] fp32 = h [T, K] W^T (bf16, W [>= n, K]) for at most 64 outputs; K a multiple of 32, ldh of 8.
+int pm_router_logits(const void* h, long long ldh, const void* W, int T, int n, int K, float* out, cudaStream_t
+    st);
 // xs [rows, width] = w[pair] * h[pair / k] (w null: h) for the pairs perm[0 .. n) sorted by expert (off [E + 1]). align 0: rows = n in
 // sorted order. align > 0: every expert's slab starts at a multiple of align (off_pad [E + 1]), dest [n] is the row of each
 // pair, rows between slabs are zero; rows must be at least n + (align - 1) per expert with pairs.
@@ -418,15 +428,16 @@ int pm_dot_norms(const void* a, const void* b, int bf16, long long n, float* out
 
 // ---------------------------------------------------------------- window_attn.cu
 // u [n_tok, ldu]: queries [H][M][D] from column 0 and, with pages, keys [G][M][D] from column k_at and values [G][DV] from
-// column v_at (k_at again: the values are the keys before rotation and norm). q_out [n_tok, H M, D8] and the cache rows
+// column v_at (k_at again: the values are the keys before rotation and norm). q_out [n_tok, H M, D8] (wide > 0: rows of that many
+// channels, those of map i from i D8 on, zeros elsewhere) and the cache rows
 // pages[slot] get rotated (first R channels; pairs 1: (2 i, 2 i + 1), else (i, i + R / 2); cs / sn fp32 [n_tok, R / 2]) and,
 // normed 1, normalised vectors times qw / kw (fp32 [D], nullable). temp_every > 0: queries at position p = pos[t] are multiplied
 // by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).
 int pm_window_prep(const void* u, int f32, long long ldu, const float* cs, const float* sn, int n_tok, int H, int
-    G, int M, int D, int DV, int k_at, int v_at, int R, int pairs, int normed, float eps, const float* qw, const
-    float* kw, const int* pos, float temp_coef, int temp_every, void* q_out, void* pages, const long long* slots,
-    cudaStream_t st);
-// Attention of the new tokens q_start[i] .. + q_lens[i] - 1 of n_seq sequences (rows of q [n_tok, H M, D8] and out [.., ldo])
+    G, int M, int D, int DV, int wide, int k_at, int v_at, int R, int pairs, int normed, float eps, const float*
+    qw, const float* kw, const int* pos, float temp_coef, int temp_every, void* q_out, void* pages, const long
+    long* slots, cudaStream_t st);
+// Attention of the new tokens q_start[i] .. + q_lens[i] - 1 of n_seq sequences (rows of q as pm_window_prep leaves them and out [.., ldo])
 // over their cached keys; sequence i has seq_lens[i] keys behind row i of block_table. Scores times scale, capped when
 // softcap > 0; sink (fp32 [H], M = 1) adds exp(sink) to a head's softmax sum; gate [.., ldg] multiplies head h by the sigmoid of
 // column h. M = 2: the result of a head is a_1 - lambda[0] a_2 over its root mean square (eps inside), times keep; it takes o
@@ -434,9 +445,18 @@ int pm_window_prep(const void* u, int f32, long long ldu, const float* cs, const
 // buffers po [n_split][n_tok][H M][DV8] and pml [n_split][n_tok][H M][2] (both or none; needed for n_split > 1).
 int pm_window_attn(const void* q, int f32, const void* pages, const int* block_table, const int* seq_lens, const
     int* q_start, const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H, int G, int M, int D,
-    int DV, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg, const
-    float* lambda, float keep, float eps, int few, int n_split, float* po, float* pml, void* o, void* out, long
-    long ldo, cudaStream_t st);
+    int DV, int wide, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg,
+    const float* lambda, float keep, float eps, int few, int n_split, float* po, float* pml, void* o, void* out,
+    long long ldo, cudaStream_t st);
+// k128 / v128 [n, G, 128] bf16 = the cached keys (M maps of D8 channels side by side) and values (DV8) of the n cache rows in `slots`
+// (page * 64 + offset), zero padded. M D8 <= 128 and DV8 <= 128.
+int pm_window_expand(const void* pages, const long long* slots, int n, int G, int M, int D, int DV, void* k128,
+    void* v128, cudaStream_t st);
+// The last step of pm_window_attn by itself, for the tokens of n_seq sequences: o [n_tok, H M, OP] (bf16, DV channels per row) -> out
+// [.., ldo]: the difference of two maps with its norm (M = 2: lambda, keep, eps) and the heads' gates (nullable).
+int pm_window_finish(const void* o, int n_tok, int H, int M, int DV, int OP, const int* q_start, const int* q_lens,
+    int n_seq, int max_q, const float* lambda, float keep, float eps, const void* gate, long long ldg, void* out,
+    long long ldo, cudaStream_t st);
 
 #ifdef __cplusplus
 }

@@ -221,7 +221,7 @@ __global__ void gelu_kernel(const T* x, long long ldx, int cols, T* out, long lo
     float v[V];
     load_vec<V>(x + t * ldx + c, v);
 #pragma unroll
-    for (int e = 0; e < V; ++e) v[e] = gelu_f(v[e]);
+    for (int e = 0; e < V; ++e) v[e] = sizeof(T) == 2 ? gelu_fast(v[e]) : gelu_f(v[e]);
     store_vec<V>(out + t * ldo + c, v);
   }
 }

@@ -14,6 +14,8 @@
 //                       the pages; the parts are merged in shared memory and by window_finish_kernel. Pages outside every row's
 //                       window are not visited.
 //   window_row_kernel   any type and size, one (token, head, map) per CTA (fp32 models, heads beyond 256 channels)
+//   window_expand_kernel  keys (all maps side by side) and values of cached tokens in rows of 128 channels, for long portions on the
+//                       tcgen05 kernel of attention_tc.cu; queries then lie in rows of 128, at their map's channels
 //   window_finish_kernel  joins the parts of split pages; with two maps a_1 - lambda a_2, its RMS norm over the head and a
 //                       factor; one sigmoid gate per head
 #include <cuda_bf16.h>
@@ -36,13 +38,13 @@ struct WindowPrepParams {
   long long ldu;
   const float* cs;           // [tokens, R / 2]
   const float* sn;
-  T* q;                      // [tokens, H M, D8]
+  T* q;                      // [tokens, H M, QP], channels of map i from i QM on, zeros elsewhere
   T* pages;                  // [block][64][G][M D8 + DV8]; null: queries alone
   const long long* slots;    // page * 64 + offset of every token
   const float* qw;           // [D], nullable: weights of the norms
   const float* kw;
   const int* pos;            // position of every token (temp_every > 0)
-  int n_tok, H, G, M, D, D8, DV, DV8, k_at, v_at, R, pairs, normed, temp_every;
+  int n_tok, H, G, M, D, D8, DV, DV8, QP, QM, k_at, v_at, R, pairs, normed, temp_every;
   float eps, temp_coef;
 };
 
@@ -80,7 +82,10 @@ __global__ void __launch_bounds__(256) window_prep_kernel(const WindowPrepParams
     }
     scale /= sqrtf(warp_sum(ss) / static_cast<float>(p.D) + p.eps);
   }
-  T* dst = key ? p.pages + (p.slots[t] * p.G + hk / p.M) * kv + (hk % p.M) * p.D8 : p.q + (t * nq + h) * p.D8;
+  T* dst = key ? p.pages + (p.slots[t] * p.G + hk / p.M) * kv + (hk % p.M) * p.D8 : p.q + (t * nq + h) * p.QP + (h % p.M) * p.QM;
+  if (!key)
+    for (int c = lane; c < p.QP; c += 32)
+      if (c < h % p.M * p.QM || c >= h % p.M * p.QM + p.D8) put(p.q + (t * nq + h) * p.QP + c, 0.f);
   const float* w = key ? p.kw : p.qw;
   const int half = p.R / 2;
   const float* cs = p.cs + t * half;
@@ -168,12 +173,21 @@ __global__ void __launch_bounds__(256) window_prep_vec_kernel(const WindowPrepPa
   }
 #pragma unroll
   for (int e = 0; e < 8; ++e) v[e] *= scale;
-  store_vec<8>(key ? p.pages + (p.slots[t] * p.G + hk / p.M) * kv + (hk % p.M) * p.D8 + c : p.q + (t * nq + h) * p.D8 + c, v);
+  if (key) {
+    store_vec<8>(p.pages + (p.slots[t] * p.G + hk / p.M) * kv + (hk % p.M) * p.D8 + c, v);
+    return;
+  }
+  __nv_bfloat16* q = p.q + (t * nq + h) * p.QP;
+  const int at = h % p.M * p.QM;
+  store_vec<8>(q + at + c, v);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] = 0.f;
+  for (int z = c; z < p.QP - p.D; z += p.D) store_vec<8>(q + (z < at ? z : z + p.D), v);      // the lanes own D channels at a time
 }
 
 template <typename T>
 struct WindowParams {
-  const T* q;                // [tokens, H M, D8]
+  const T* q;                // [tokens, H M, QP], channels of map i from i QM on
   const T* pages;
   T* out;                    // [tokens, ldo], (head, map) n at column n DV
   long long ldo;
@@ -186,7 +200,7 @@ struct WindowParams {
   const float* sink;         // [H], nullable
   const T* gate;             // [tokens, ldg], nullable: logits of the heads' gates
   long long ldg;
-  int n_tok, max_blocks, H, G, rep, M, KM, D, D8, DV, DV8, window, n_split;      // KM: maps of a CTA, 1 or M
+  int n_tok, max_blocks, H, G, rep, M, KM, D, D8, DV, DV8, QP, QM, window, n_split;      // KM: maps of a CTA, 1 or M
   float scale, softcap;      // softcap 0: none
 };
 
@@ -229,7 +243,7 @@ __global__ void __launch_bounds__(128) window_mma_kernel(const WindowParams<__nv
     const int r = i / kw, c = i - r * kw, row = r0 + r, own = row % p.KM, at = c - own * kvec;
     const bool ok = r < n_rows && at >= 0 && at < kvec;                  // zeros at the channels of the other maps
     const __nv_bfloat16* src = p.q;
-    if (ok) src += ((static_cast<long long>(q0 + row / rpt) * p.H + g * p.rep + row % rpt / p.KM) * p.M + map0 + own) * p.D8 + at * 8;
+    if (ok) src += ((static_cast<long long>(q0 + row / rpt) * p.H + g * p.rep + row % rpt / p.KM) * p.M + map0 + own) * p.QP + (map0 + own) * p.QM + at * 8;
     ms_cp16(ms_addr(sQ + r * ldk + c * 8), src, ok);
   }
   const int* table = p.block_table + static_cast<long long>(seq) * p.max_blocks;
@@ -449,7 +463,7 @@ template <typename T>
 struct WindowFinishParams {
   const float* po;           // parts as in WindowParams, or
   const float* pml;
-  const T* o;                // [n_tok, H M, DV]
+  const T* o;                // [n_tok, H M, OP]
   T* out;                    // [tokens, ldo], head h at column h DV
   long long ldo;
   const int* q_start;
@@ -459,7 +473,7 @@ struct WindowFinishParams {
   long long ldg;
   const float* lambda;       // M = 2: one number
   float keep, eps;           // M = 2: factor behind the norm
-  int n_tok, H, M, DV, DV8, n_split;
+  int n_tok, H, M, DV, DV8, OP, n_split;
 };
 
 // One warp per (token, head) of the sequences in q_start / q_lens, NC * 32 channels. grid (tokens of the longest portion,
@@ -478,7 +492,7 @@ __global__ void __launch_bounds__(128) window_finish_kernel(const WindowFinishPa
     if (p.o) {
 #pragma unroll
       for (int i = 0; i < NC; ++i)
-        if (lane + 32 * i < p.DV) v[i] = fmaf(w, to_f(p.o[at * p.DV + lane + 32 * i]), v[i]);
+        if (lane + 32 * i < p.DV) v[i] = fmaf(w, to_f(p.o[at * p.OP + lane + 32 * i]), v[i]);
       continue;
     }
     const float ms = lane < p.n_split ? p.pml[(at + lane * step) * 2] : -CUDART_INF_F;       // lane s: split s
@@ -520,7 +534,7 @@ __global__ void __launch_bounds__(128) window_row_kernel(const WindowParams<T> p
   const long long t = p.q_start[seq] + i;
   const int pos = p.seq_lens[seq] - len + i;
   const int* table = p.block_table + static_cast<long long>(seq) * p.max_blocks;
-  const T* qr = p.q + (t * p.H * p.M + hm) * p.D8;
+  const T* qr = p.q + (t * p.H * p.M + hm) * p.QP + hm % p.M * p.QM;
   const int kv = p.M * p.D8 + p.DV8, k_at = hm % p.M * p.D8, v_at = p.M * p.D8;
   float q[NC], o[NC], m = -CUDART_INF_F, l = 0.f;
 #pragma unroll
@@ -578,6 +592,22 @@ __global__ void __launch_bounds__(128) window_row_kernel(const WindowParams<T> p
     if (warp == 0 && c * 32 + lane < p.DV)
       put(p.out + t * p.ldo + static_cast<long long>(hm) * p.DV + c * 32 + lane,
           (so[0][lane] + so[1][lane] + so[2][lane] + so[3][lane]) / ll * gate);
+  }
+}
+
+// k128 [n, G, 128] and v128 [n, G, 128] of the n cache rows in `slots`, zeros behind their channels. A thread writes 8 channels.
+__global__ void window_expand_kernel(const __nv_bfloat16* __restrict__ pages, const long long* __restrict__ slots, int n, int G, int keys,
+                                     int values, __nv_bfloat16* __restrict__ k128, __nv_bfloat16* __restrict__ v128) {
+  const long long total = static_cast<long long>(n) * G * 32;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long row = i >> 5;                        // (position, head)
+    const int c = static_cast<int>(i & 15) * 8, j = static_cast<int>(row / G), g = static_cast<int>(row - static_cast<long long>(j) * G);
+    const bool value = i & 16;
+    const __nv_bfloat16* src = pages + (slots[j] * G + g) * (keys + values);
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (c < (value ? values : keys)) v = *reinterpret_cast<const uint4*>(src + (value ? keys : 0) + c);
+    *reinterpret_cast<uint4*>((value ? v128 : k128) + row * 128 + c) = v;
   }
 }
 
@@ -666,11 +696,11 @@ static int window_prep_launch(WindowPrepParams<T> p, cudaStream_t st) {
 
 template <typename T>
 static WindowPrepParams<T> window_prep_params(const void* u, long long ldu, const float* cs, const float* sn, int n_tok, int H, int G, int M,
-                                              int D, int DV, int k_at, int v_at, int R, int pairs, int normed, float eps,
+                                              int D, int DV, int wide, int k_at, int v_at, int R, int pairs, int normed, float eps,
                                               const float* qw, const float* kw, const int* pos, float temp_coef, int temp_every,
                                               void* q, void* pages, const long long* slots) {
   return {static_cast<const T*>(u), ldu, cs, sn, static_cast<T*>(q), static_cast<T*>(pages), slots, qw, kw, pos, n_tok, H, G, M,
-          D, (D + 7) / 8 * 8, DV, (DV + 7) / 8 * 8, k_at, v_at, R, pairs, normed, temp_every, eps, temp_coef};
+          D, (D + 7) / 8 * 8, DV, (DV + 7) / 8 * 8, wide ? wide : (D + 7) / 8 * 8, wide ? (D + 7) / 8 * 8 : 0, k_at, v_at, R, pairs, normed, temp_every, eps, temp_coef};
 }
 
 template <typename T>
@@ -678,7 +708,7 @@ static int window_attn_launch(WindowParams<T> p, int n_seq, int max_q, int few, 
                               cudaStream_t st) {
   constexpr bool low = sizeof(T) == 2;
   WindowFinishParams<T> f{p.po, p.pml, nullptr, p.out, p.ldo, p.q_start, p.q_lens, p.sink, p.gate, p.ldg, lambda, keep, eps,
-                          p.n_tok, p.H, p.M, p.DV, p.DV8, p.n_split};
+                          p.n_tok, p.H, p.M, p.DV, p.DV8, p.DV, p.n_split};
   if (!p.po && p.M > 1) {                 // results of the maps, then their difference
     if (!o) return -3;
     f.o = static_cast<const T*>(o);
@@ -714,25 +744,27 @@ static bool window_bad_dims(int H, int G, int M, int D, int DV) {
 }
 
 // u [n_tok, ldu]: queries [H][M][D] from column 0 and, with pages, keys [G][M][D] from column k_at and values [G][DV] from
-// column v_at (k_at again: the values are the keys before rotation and norm). q_out [n_tok, H M, D8] and the cache rows
+// column v_at (k_at again: the values are the keys before rotation and norm). q_out [n_tok, H M, D8] (wide > 0: rows of that many
+// channels, those of map i from i D8 on, zeros elsewhere) and the cache rows
 // pages[slot] get rotated (first R channels; pairs 1: (2 i, 2 i + 1), else (i, i + R / 2); cs / sn fp32 [n_tok, R / 2]) and,
 // normed 1, normalised vectors times qw / kw (fp32 [D], nullable). temp_every > 0: queries at position p = pos[t] are multiplied
 // by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).
 extern "C" int pm_window_prep(const void* u, int f32, long long ldu, const float* cs, const float* sn, int n_tok, int H, int G, int M,
-                              int D, int DV, int k_at, int v_at, int R, int pairs, int normed, float eps, const float* qw,
+                              int D, int DV, int wide, int k_at, int v_at, int R, int pairs, int normed, float eps, const float* qw,
                               const float* kw, const int* pos, float temp_coef, int temp_every, void* q_out, void* pages,
                               const long long* slots, cudaStream_t st) {
-  if (window_bad_dims(H, G, M, D, DV) || R < 0 || R > D || R % 2 || temp_every < 0 || (temp_every && !pos)) return -1;
+  if (window_bad_dims(H, G, M, D, DV) || R < 0 || R > D || R % 2 || temp_every < 0 || (temp_every && !pos) ||
+      (wide && (wide % 8 || wide < M * ((D + 7) / 8 * 8)))) return -1;
   if (ldu < static_cast<long long>(H) * M * D || (pages && (k_at < 0 || v_at < 0 || ldu < k_at + static_cast<long long>(G) * M * D ||
                                                             ldu < v_at + static_cast<long long>(G) * DV))) return -2;
   if (n_tok < 1) return 0;
-  return f32 ? window_prep_launch(window_prep_params<float>(u, ldu, cs, sn, n_tok, H, G, M, D, DV, k_at, v_at, R, pairs, normed, eps, qw,
+  return f32 ? window_prep_launch(window_prep_params<float>(u, ldu, cs, sn, n_tok, H, G, M, D, DV, wide, k_at, v_at, R, pairs, normed, eps, qw,
                                                             kw, pos, temp_coef, temp_every, q_out, pages, slots), st)
-             : window_prep_launch(window_prep_params<__nv_bfloat16>(u, ldu, cs, sn, n_tok, H, G, M, D, DV, k_at, v_at, R, pairs, normed,
+             : window_prep_launch(window_prep_params<__nv_bfloat16>(u, ldu, cs, sn, n_tok, H, G, M, D, DV, wide, k_at, v_at, R, pairs, normed,
                                                                     eps, qw, kw, pos, temp_coef, temp_every, q_out, pages, slots), st);
 }
 
-// Attention of the new tokens q_start[i] .. + q_lens[i] - 1 of n_seq sequences (rows of q [n_tok, H M, D8] and out [.., ldo])
+// Attention of the new tokens q_start[i] .. + q_lens[i] - 1 of n_seq sequences (rows of q as pm_window_prep leaves them and out [.., ldo])
 // over their cached keys; sequence i has seq_lens[i] keys behind row i of block_table. Scores times scale, capped when
 // softcap > 0; sink (fp32 [H], M = 1) adds exp(sink) to a head's softmax sum; gate [.., ldg] multiplies head h by the sigmoid of
 // column h. M = 2: the result of a head is a_1 - lambda[0] a_2 over its root mean square (eps inside), times keep; it takes o
@@ -740,7 +772,7 @@ extern "C" int pm_window_prep(const void* u, int f32, long long ldu, const float
 // buffers po [n_split][n_tok][H M][DV8] and pml [n_split][n_tok][H M][2] (both or none; needed for n_split > 1).
 extern "C" int pm_window_attn(const void* q, int f32, const void* pages, const int* block_table, const int* seq_lens,
                               const int* q_start, const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H,
-                              int G, int M, int D, int DV, int window, float scale, float softcap, const float* sink, const void* gate,
+                              int G, int M, int D, int DV, int wide, int window, float scale, float softcap, const float* sink, const void* gate,
                               long long ldg, const float* lambda, float keep, float eps, int few, int n_split, float* po, float* pml,
                               void* o, void* out, long long ldo, cudaStream_t st) {
   if (window_bad_dims(H, G, M, D, DV) || window < 0 || n_split < 1 || n_split > 32 || (n_split > 1 && (!few || !po)) ||
@@ -752,11 +784,37 @@ extern "C" int pm_window_attn(const void* q, int f32, const void* pages, const i
   if (f32)
     return window_attn_launch<float>({static_cast<const float*>(q), static_cast<const float*>(pages), static_cast<float*>(out), ldo,
                                       block_table, seq_lens, q_start, q_lens, po, pml, sink, static_cast<const float*>(gate), ldg,
-                                      n_tok, max_blocks, H, G, H / G, M, 1, D, D8, DV, DV8, window, n_split, scale, softcap},
+                                      n_tok, max_blocks, H, G, H / G, M, 1, D, D8, DV, DV8, wide ? wide : D8, wide ? D8 : 0, window, n_split, scale, softcap},
                                      n_seq, max_q, few, o, lambda, keep, eps, st);
   return window_attn_launch<__nv_bfloat16>({static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(pages),
                                             static_cast<__nv_bfloat16*>(out), ldo, block_table, seq_lens, q_start, q_lens, po, pml,
                                             sink, static_cast<const __nv_bfloat16*>(gate), ldg, n_tok, max_blocks, H, G, H / G, M, 1,
-                                            D, D8, DV, DV8, window, n_split, scale, softcap},
+                                            D, D8, DV, DV8, wide ? wide : D8, wide ? D8 : 0, window, n_split, scale, softcap},
                                            n_seq, max_q, few, o, lambda, keep, eps, st);
+}
+
+// k128 / v128 [n, G, 128] bf16 = the cached keys (M maps of D8 channels side by side) and values (DV8) of the n cache rows in `slots`
+// (page * 64 + offset), zero padded. M D8 <= 128 and DV8 <= 128.
+extern "C" int pm_window_expand(const void* pages, const long long* slots, int n, int G, int M, int D, int DV, void* k128, void* v128,
+                                cudaStream_t st) {
+  const int keys = M * ((D + 7) / 8 * 8), values = (DV + 7) / 8 * 8;
+  if (n < 1 || window_bad_dims(G, G, M, D, DV) || keys > 128 || values > 128) return -1;
+  long long grid = (static_cast<long long>(n) * G * 32 + 255) / 256;
+  if (grid > num_sms() * 16) grid = num_sms() * 16;
+  window_expand_kernel<<<static_cast<int>(grid), 256, 0, st>>>(static_cast<const __nv_bfloat16*>(pages), slots, n, G, keys, values,
+                                                               static_cast<__nv_bfloat16*>(k128), static_cast<__nv_bfloat16*>(v128));
+  return static_cast<int>(cudaGetLastError());
+}
+
+// The last step of pm_window_attn by itself, for the tokens of n_seq sequences: o [n_tok, H M, OP] (bf16, DV channels per row) -> out
+// [.., ldo]: the difference of two maps with its norm (M = 2: lambda, keep, eps) and the heads' gates (nullable).
+extern "C" int pm_window_finish(const void* o, int n_tok, int H, int M, int DV, int OP, const int* q_start, const int* q_lens, int n_seq,
+                                int max_q, const float* lambda, float keep, float eps, const void* gate, long long ldg, void* out,
+                                long long ldo, cudaStream_t st) {
+  if (window_bad_dims(H, H, M, 1, DV) || OP < DV || (M > 1 && !lambda)) return -1;
+  if (n_seq < 1 || max_q < 1) return 0;
+  const WindowFinishParams<__nv_bfloat16> f{nullptr, nullptr, static_cast<const __nv_bfloat16*>(o), static_cast<__nv_bfloat16*>(out),
+                                            ldo, q_start, q_lens, nullptr, static_cast<const __nv_bfloat16*>(gate), ldg, lambda, keep,
+                                            eps, n_tok, H, M, DV, (DV + 7) / 8 * 8, OP, 1};
+  return window_finish_launch(f, n_seq, max_q, st);
 }

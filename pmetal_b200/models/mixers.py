@@ -24,7 +24,7 @@ import torch
 import torch.nn as nn
 
 from ..ops import functional as ops
-from .state_cache import CacheSpec, split_groups
+from .state_cache import CacheSpec, attention_runs, split_groups
 
 # portions up to this many tokens take the decode kernels (state-space scan, attention in the latent space)
 SHORT = 16
@@ -47,7 +47,7 @@ class StepContext:
         self.meta, self.freqs = meta, freqs
         self._rope: Dict[tuple, tuple] = {}
         self._groups: Dict[int, tuple] = {}
-        self._zeros: Optional[torch.Tensor] = None
+        self._runs: Dict[int, list] = {}
 
     def rope(self, base: float, dims: int):
         key = (base, dims)
@@ -61,10 +61,11 @@ class StepContext:
             self._groups[limit] = split_groups(self.meta, limit)
         return self._groups[limit]
 
-    def zeros(self, n: int) -> torch.Tensor:
-        if self._zeros is None or self._zeros.shape[0] < n:
-            self._zeros = torch.zeros(n, dtype=torch.int32, device=self.meta.positions.device)
-        return self._zeros
+    def runs(self, limit: int):
+        """The sequences with more than ``limit`` new tokens as launches of the flash-attention kernel."""
+        if limit not in self._runs:
+            self._runs[limit] = attention_runs(self.meta, self.groups(limit)[1])
+        return self._runs[limit]
 
 
 class RotationFreqs:
@@ -236,9 +237,8 @@ class LatentAttentionMixer(nn.Module):
             nat.latent_attn(qd, self.w_ukv, self.w_ukv[self.n_k:], pages, short, self.dims, self.scale, o, turn)
         if long is not None:
             w = self._expand_weight()
-            for i, q0, n, n_keys in long.host:
-                nat.latent_expand_attn(qd[q0:q0 + n], w, pages, ctx.meta.block_table[i], n_keys, self.dims, self.scale,
-                                       o[q0:q0 + n], ctx.zeros(n))
+            for r in ctx.runs(SHORT):
+                nat.latent_expand_attn(qd, w, pages, r, self.dims, self.scale, o)
         return ops.project(o, self.w_o)
 
 
@@ -431,15 +431,19 @@ class GroupedAttentionMixer(nn.Module):
         u = ops.project(x, self.w_in)
         cos, sin = ctx.rope(self.base, self.R) if self.R else (None, None)
         k_at = self.at.get("k", 0)
+        short, long = ctx.groups(SHORT)
+        wide = nat.window_wide(self.dims, x.dtype, self.window) if long is not None else 0
         q = nat.window_prep(u, cos, sin, self.dims, (self.R, self.ROTATION), self.UNIT_NORM, self.eps, (k_at, self.at.get("v", k_at)),
-                            pages if self.own else None, ctx.meta.slots, self.q_norm_w, self.k_norm_w, self.temp, ctx.meta.positions)
+                            pages if self.own else None, ctx.meta.slots, self.q_norm_w, self.k_norm_w, self.temp, ctx.meta.positions, wide)
         o = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
         gate = u[:, self.at["g"]:] if self.GATE else None
         diff = (self.lam, 1.0 - self.diff, self.eps) if self.dims[2] > 1 else None
-        short, long = ctx.groups(SHORT)
-        for group, few in ((short, True), (long, False)):
-            if group is not None:
-                nat.window_attn(q, pages, group, self.dims, self.window, self.scale, few, o, self.softcap, self.sink, gate, diff)
+        if short is not None:
+            nat.window_attn(q, pages, short, self.dims, self.window, self.scale, True, o, self.softcap, self.sink, gate, diff)
+        if long is not None and wide:
+            nat.window_expand_attn(q, pages, long, ctx.runs(SHORT), self.dims, self.scale, o, self.softcap, self.sink, gate, diff)
+        elif long is not None:
+            nat.window_attn(q, pages, long, self.dims, self.window, self.scale, False, o, self.softcap, self.sink, gate, diff)
         return ops.project(o, self.w_o)
 
 

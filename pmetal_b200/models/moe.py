@@ -74,7 +74,7 @@ class WeightedInputExperts(nn.Module):
     def forward(self, h: torch.Tensor):
         from ..ops import functional as ops
         from ..ops import native as nat
-        r = nat.moe_route(ops.project_f32(h, self.router, self.E), self.k, self.RENORM, score=self.SCORE)
+        r = nat.moe_route(ops.router_logits(h, self.router, self.E), self.k, self.RENORM, score=self.SCORE)
         T, f, w = h.shape[0], self.ff, self.width
         if h.dtype != torch.bfloat16 or f % 8 or w % 8:
             xs, off, dest = nat.expert_gather(h, r, self.k)
@@ -168,13 +168,12 @@ class WeightedOutputExperts(nn.Module):
             act = nat.grouped_gemm_skinny(xs, self.up, off, max_rows_per_expert=tile, gelu=True)
             return nat.grouped_gemm_skinny(act, self.down, off, max_rows_per_expert=tile), dest
         xs, off, dest = nat.expert_gather(h, r, k, align=128, weighted=False)
-        act = nat.grouped_gemm(0, xs, self.up, off, f, w)
-        return nat.grouped_gemm(0, nat.gelu(act, act), self.down, off, w, f), dest
+        return nat.grouped_gemm(0, nat.grouped_gemm(0, xs, self.up, off, f, w, gelu=True), self.down, off, w, f), dest
 
     def forward(self, h: torch.Tensor) -> dict:
         from ..ops import functional as ops
         from ..ops import native as nat
-        r = nat.moe_route(ops.project_f32(h, self.router, self.E + self.identity), self.k, False,
+        r = nat.moe_route(ops.router_logits(h, self.router, self.E + self.identity), self.k, False,
                           choice=(self.correction, self.groups, self.keep, self.factor))
         z, row = self._routed(h, dict(r, counts=r["counts"][:self.E], offsets=r["offsets"][:self.E + 1]))
         return dict(y=self._shared(h) if self.shared_ff else None, z=z, route=(r["topk_w"], r["topk_idx"], row, self.E), k=self.k)

@@ -15,7 +15,8 @@ to the pool while the sequence lives.
 
 A layer that runs several times in a step (a looped stack) has a spec, pages and slots for every run.
 
-``split_groups`` divides a step's sequences into short and long portions, which run on different kernels."""
+``split_groups`` divides a step's sequences into short and long portions, which run on different kernels; ``attention_runs`` joins
+long portions into launches of an attention kernel whose keys are rows of one buffer."""
 from __future__ import annotations
 
 from dataclasses import dataclass, field
@@ -163,3 +164,39 @@ def split_groups(meta: BatchMeta, limit: int) -> Tuple[Optional[SeqGroup], Optio
         out.append(SeqGroup(len(ix), c, mq, mk, meta.block_table[sel], meta.seq_lens[sel], meta.q_start[sel],
                             meta.q_lens[sel], cs, meta.state_slots[sel] if meta.state_slots is not None else None, rows, host))
     return out[0], out[1]
+
+
+@dataclass
+class AttnRun:
+    """Consecutive sequences of a step whose attention is one launch: query rows ``rows`` of the step, key rows gathered from the
+    cache rows ``slots``. Query i (from the first of ``rows`` on) sees key rows ``seq_start[i]`` .. i + ``shift``."""
+    rows: slice
+    n: int
+    slots: torch.Tensor
+    seq_start: torch.Tensor
+    shift: int
+
+
+def attention_runs(meta: BatchMeta, group: SeqGroup) -> List[AttnRun]:
+    """A run begins with any sequence and takes in the next ones as long as their rows follow and they have no earlier tokens: then
+    every query row lies ``shift`` before its own key row, the earlier tokens of the first sequence."""
+    runs: List[List[Tuple[int, int, int, int]]] = []
+    for s in group.host:
+        i, q0, n, total = s
+        if runs and total == n and q0 == runs[-1][-1][1] + runs[-1][-1][2]:
+            runs[-1].append(s)
+        else:
+            runs.append([s])
+    out, dev = [], meta.slots.device
+    for run in runs:
+        i, q0, n0, total = run[0]
+        prior, n = total - n0, sum(s[2] for s in run)
+        slots = meta.slots[q0:q0 + n]
+        if prior:
+            pages = meta.block_table[i, :-(-prior // BLOCK)].long()
+            old = (pages[:, None] * BLOCK + torch.arange(BLOCK, device=dev)).view(-1)[:prior]
+            slots = torch.cat([old, slots])
+        base = torch.tensor([0] + [s[1] - q0 + prior for s in run[1:]], dtype=torch.int32)
+        start = torch.repeat_interleave(base, torch.tensor([s[2] for s in run])).to(dev, non_blocking=True)
+        out.append(AttnRun(slice(q0, q0 + n), n, slots.contiguous(), start, prior))
+    return out

@@ -658,3 +658,11 @@ def project_f32(x: torch.Tensor, w: torch.Tensor, n: int) -> torch.Tensor:
     if gemv_fits(x.shape[0], x.shape[1]):
         return nat.gemv_ex(x, w, out_f32=True, n=n)
     return nat.gemm_f32(x, w)[:, :n]
+
+
+def router_logits(x: torch.Tensor, w: torch.Tensor, n: int) -> torch.Tensor:
+    """``project_f32`` for routers: a step of many tokens and few outputs has a kernel of its own."""
+    nat = _native()
+    if not gemv_fits(x.shape[0], x.shape[1]) and use_native(x) and nat.router_logits_supported(x, n):
+        return nat.router_logits(x, w, n)
+    return project_f32(x, w, n)

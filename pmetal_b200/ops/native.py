@@ -425,10 +425,10 @@ def lora_db(dy, t, seg_sizes, r: int, out: torch.Tensor) -> None:
 
 # ------------------------------------------------------------------------------------------- grouped (expert) GEMM
 def grouped_gemm(mode: int, a: torch.Tensor, b: torch.Tensor, off: torch.Tensor, n: int, k: int,
-                 out: Optional[torch.Tensor] = None, accumulate: bool = False, alpha: float = 1.0) -> torch.Tensor:
+                 out: Optional[torch.Tensor] = None, accumulate: bool = False, alpha: float = 1.0, gelu: bool = False) -> torch.Tensor:
     """Grouped GEMM over expert-sorted rows in the padded layout (``off`` int32 [E+1], multiples of 128; csrc/grouped_gemm.cu).
 
-    mode 0: a = X [R, K], b = W [E, N, K]      -> Y  [R, N] bf16
+    mode 0: a = X [R, K], b = W [E, N, K]      -> Y  [R, N] bf16 (``gelu``: its exact gelu)
     mode 1: a = dY [R, N], b = W [E, N, K]     -> dX [R, K] bf16
     mode 2: a = dY [R, N], b = X [R, K]        -> dW [E, N, K] fp32 (experts without rows keep ``out``'s contents)"""
     E = off.numel() - 1
@@ -448,7 +448,7 @@ def grouped_gemm(mode: int, a: torch.Tensor, b: torch.Tensor, off: torch.Tensor,
     lib().pm_grouped_gemm.restype = c_int
     rc = lib().pm_grouped_gemm(c_int(mode), _p(a), c_int(a.stride(0)), _p(b), c_int(ldb), _p(out), c_int(out.stride(-2)),
                                _p(off), c_int(E), c_int(R), c_int(n), c_int(k), c_float(alpha), c_int(int(accumulate)),
-                               _p(status_word(a.device)), _stream())
+                               c_int(int(gelu)), _p(status_word(a.device)), _stream())
     _chk(rc, "pm_grouped_gemm")
     return out
 
@@ -689,11 +689,12 @@ def attn_fwd(q, k, v, seq_start, scale: float, window: int = 0):
     return out, lse
 
 
-def attn_fwd_rect(q, k, v, seq_start, scale: float, shift: int, out=None):
+def attn_fwd_rect(q, k, v, seq_start, scale: float, shift: int, out=None, softcap: float = 0.0, sink=None, gate=None):
     """Attention of Tq queries over Tk keys where key j is visible to query i iff seq_start[i] <= j <= i + shift
     (shift >= Tk - 1: every key). q [Tq, hq, 128], k/v [Tk, hkv, 128] (k/v may live in a peer GPU's memory: the
     kernel's TMA loads read them in place). Returns (out bf16 [Tq, hq, 128], lse fp32 [hq, Tq]); ``out`` may be given (any
-    token stride)."""
+    token stride). ``softcap`` > 0 caps the scores, ``sink`` fp32 [hq] joins the softmax sums, ``gate`` [Tq, >= hq] (logits, any row
+    stride) multiplies the heads."""
     T, hq, d = q.shape
     Tk, hkv = k.shape[0], k.shape[1]
     assert d == 128 and q.stride(1) == d and k.stride(1) == d and v.stride(1) == d
@@ -701,10 +702,11 @@ def attn_fwd_rect(q, k, v, seq_start, scale: float, shift: int, out=None):
         out = torch.empty(T, hq, d, dtype=q.dtype, device=q.device)
     assert out.shape == q.shape and out.stride(1) == d
     lse = torch.empty(hq, T, dtype=torch.float32, device=q.device)
-    _chk(lib().pm_attn_fwd_tc_rect(_p(q), c_ll(q.stride(0)), _p(k), c_ll(k.stride(0)), _p(v), c_ll(v.stride(0)), _p(out),
-                                   c_ll(out.stride(0)), _p(lse), _p(seq_start), c_int(T), c_int(Tk), c_int(shift),
-                                   c_int(hq), c_int(hkv), c_float(scale), _p(status_word(q.device)), _stream()),
-         "pm_attn_fwd_tc_rect")
+    _chk(lib().pm_attn_fwd_tc_ex(_p(q), c_ll(q.stride(0)), _p(k), c_ll(k.stride(0)), _p(v), c_ll(v.stride(0)), _p(out),
+                                 c_ll(out.stride(0)), _p(lse), _p(seq_start), c_int(T), c_int(Tk), c_int(shift),
+                                 c_int(hq), c_int(hkv), c_float(scale), c_float(softcap), _p(sink), _p(gate),
+                                 c_ll(gate.stride(0) if gate is not None else 0), _p(status_word(q.device)), _stream()),
+         "pm_attn_fwd_tc_ex")
     return out, lse
 
 
@@ -1010,6 +1012,18 @@ def moe_combine(z, inv, w, k: int, residual=None):
     _chk(lib().pm_moe_combine2(_p(z.contiguous()), _p(inv), _p(w.contiguous()), c_int(k), _p(residual), _p(y), c_ll(T),
                                c_int(H), _stream()), "pm_moe_combine2")
     return y
+
+
+def router_logits_supported(h, n: int) -> bool:
+    return h.dtype == torch.bfloat16 and n <= 64 and h.shape[1] % 32 == 0 and h.stride(0) % 8 == 0 and h.stride(1) == 1
+
+
+def router_logits(h, w, n: int):
+    """fp32 [T, n] = h [T, K] w[:n]^T (bf16) for a few outputs."""
+    out = torch.empty(h.shape[0], n, dtype=torch.float32, device=h.device)
+    _chk(lib().pm_router_logits(_p(h), c_ll(h.stride(0)), _p(w), c_int(h.shape[0]), c_int(n), c_int(h.shape[1]), _p(out), _stream()),
+         "pm_router_logits")
+    return out
 
 
 EXPERT_ACTS = ("none", "swiglu", "gelu")      # what the expert products do with their sums
@@ -1406,14 +1420,14 @@ def latent_attn(qd, wuk, wuv, pages, group, dims, scale: float, out, rope=(None,
     LAUNCHES += 2          # three kernels
 
 
-def latent_expand_attn(qd, wukv, pages, table_row, n_keys: int, dims, scale: float, out, zeros) -> None:
-    """Attention of one sequence's new tokens (rows of qd / out) over its ``n_keys`` positions with keys and values expanded
-    from the latents: one GEMM, then the flash-attention kernel. ``zeros``: int32 zeros, at least as many as new tokens."""
+def latent_expand_attn(qd, wukv, pages, run, dims, scale: float, out) -> None:
+    """Attention of the tokens of ``run`` (models/state_cache.AttnRun; rows of qd / out) over their sequences' positions with keys
+    and values expanded from the latents: one GEMM, then the flash-attention kernel."""
     H, dn, dr, dv, rank, W = dims
-    n_q, dev = qd.shape[0], qd.device
+    qd, out, n_q, n_keys, dev = qd[run.rows], out[run.rows], run.n, run.slots.shape[0], qd.device
     r8 = wukv.shape[1]
     lat = torch.empty(n_keys, r8, dtype=torch.bfloat16, device=dev)
-    _chk(lib().pm_latent_gather(_p(pages), _p(table_row), c_int(n_keys), c_int(W), c_int(rank), c_int(r8), _p(lat),
+    _chk(lib().pm_latent_gather(_p(pages), _p(run.slots), c_int(n_keys), c_int(W), c_int(rank), c_int(r8), _p(lat),
                                 _stream()), "pm_latent_gather")
     kv = gemm(lat, wukv)
     # operands whose heads already have 128 channels in 16-byte aligned rows are read in place
@@ -1427,10 +1441,10 @@ def latent_expand_attn(qd, wukv, pages, table_row, n_keys: int, dims, scale: flo
     buf = lambda n: torch.empty(n, H, 128, dtype=torch.bfloat16, device=dev)      # noqa: E731
     q128, v128, k128 = q128 if q_in else buf(n_q), v128 if v_in else buf(n_keys), buf(n_keys)
     _chk(lib().pm_latent_assemble(_p(qd), c_ll(qd.stride(0)), c_int(n_q), _p(kv), c_ll(kv.stride(0)), c_int(n_keys),
-                                  _p(pages), _p(table_row), c_int(W), c_int(rank), c_int(H), c_int(dn), c_int(dr),
+                                  _p(pages), _p(run.slots), c_int(W), c_int(rank), c_int(H), c_int(dn), c_int(dr),
                                   c_int(dv), _p(None if q_in else q128), _p(k128), _p(None if v_in else v128), _stream()),
          "pm_latent_assemble")
-    o, _ = attn_fwd_rect(q128, k128, v128, zeros[:n_q], scale, n_keys - n_q, o128 if direct else None)
+    o, _ = attn_fwd_rect(q128, k128, v128, run.seq_start, scale, run.shift, o128 if direct else None)
     if not direct:
         _chk(lib().pm_latent_take(_p(o), c_int(n_q), c_int(H), c_int(dv), _p(out), c_ll(out.stride(0)), _stream()),
              "pm_latent_take")
@@ -1481,16 +1495,18 @@ def norm_gate(y, gate, w, eps: float, parts: int, silu: bool):
 
 
 # ------------------------------------------------------------------------------------------- grouped attention, any head size
-def window_prep(u, cs, sn, dims, rot, normed: bool, eps: float, cols, pages, slots, qw=None, kw=None, temp=None, pos=None):
-    """Rotated and normalised queries [tokens, heads * maps, key size rounded up to 8]; with ``pages`` keys and values of the
+def window_prep(u, cs, sn, dims, rot, normed: bool, eps: float, cols, pages, slots, qw=None, kw=None, temp=None, pos=None,
+                wide: int = 0):
+    """Rotated and normalised queries [tokens, heads * maps, key size rounded up to 8] (``wide`` > 0: in rows of that many channels,
+    a map's behind those of the maps before it, zeros elsewhere); with ``pages`` keys and values of the
     tokens go to their cache rows. ``dims`` = (query heads, key/value heads, maps, key size, value size), ``rot`` = (rotated
     channels, layout), ``cols`` = columns of u where keys and values begin (the same: the values are the keys as projected),
     ``qw`` / ``kw`` the norms' weights (fp32), ``temp`` = (coefficient, interval) of the query factor at positions ``pos``."""
     H, G, M, D, DV = dims
-    q = torch.empty(u.shape[0], H * M, -(-D // 8) * 8, dtype=u.dtype, device=u.device)
+    q = torch.empty(u.shape[0], H * M, wide or -(-D // 8) * 8, dtype=u.dtype, device=u.device)
     coef, every = temp if temp is not None else (0.0, 0)
     _chk(lib().pm_window_prep(_p(u), _is_f32(u), c_ll(u.stride(0)), _p(cs), _p(sn), c_int(u.shape[0]), c_int(H), c_int(G), c_int(M),
-                              c_int(D), c_int(DV), c_int(cols[0]), c_int(cols[1]), c_int(rot[0]), c_int(int(rot[1] == "pairs")),
+                              c_int(D), c_int(DV), c_int(wide), c_int(cols[0]), c_int(cols[1]), c_int(rot[0]), c_int(int(rot[1] == "pairs")),
                               c_int(int(normed)), c_float(eps), _p(qw), _p(kw), _p(pos), c_float(coef), c_int(every), _p(q),
                               _p(pages), _p(slots), _stream()), "pm_window_prep")
     return q
@@ -1503,7 +1519,8 @@ def window_attn(q, pages, group, dims, window: int, scale: float, few: bool, out
     stride, ``diff`` = (lambda as an fp32 tensor, factor behind the norm, eps) where a head has two maps."""
     global LAUNCHES
     H, G, M, D, DV = dims
-    T, D8, DV8, n_split = q.shape[0], q.shape[2], -(-DV // 8) * 8, 1
+    T, D8, DV8, n_split = q.shape[0], -(-D // 8) * 8, -(-DV // 8) * 8, 1
+    wide = q.shape[2] if q.shape[2] != D8 else 0
     po = pml = o = None
     parts = few and q.dtype == torch.bfloat16 and max(D8, DV8) <= 256
     if parts:
@@ -1520,8 +1537,40 @@ def window_attn(q, pages, group, dims, window: int, scale: float, few: bool, out
     lam, keep, eps = diff if diff is not None else (None, 1.0, 0.0)
     _chk(lib().pm_window_attn(_p(q), _is_f32(q), _p(pages), _p(group.block_table), _p(group.seq_lens), _p(group.q_start),
                               _p(group.q_lens), c_int(group.n), c_int(group.block_table.shape[1]), c_int(T), c_int(group.max_q),
-                              c_int(H), c_int(G), c_int(M), c_int(D), c_int(DV), c_int(window), c_float(scale), c_float(softcap),
+                              c_int(H), c_int(G), c_int(M), c_int(D), c_int(DV), c_int(wide), c_int(window), c_float(scale), c_float(softcap),
                               _p(sink), _p(gate), c_ll(gate.stride(0) if gate is not None else 0), _p(lam), c_float(keep),
                               c_float(eps), c_int(int(few)), c_int(n_split), _p(po), _p(pml), _p(o), _p(out), c_ll(out.stride(0)),
                               _stream()), "pm_window_attn")
     LAUNCHES += int(po is not None or o is not None)
+
+
+def window_wide(dims, dtype, window: int) -> int:
+    """Row width of the queries of steps whose long portions take ``window_expand_attn``; 0 where they cannot."""
+    _, _, M, D, DV = dims
+    fits = dtype == torch.bfloat16 and window == 0 and M * -(-D // 8) * 8 <= 128 and DV <= 128
+    return 128 if fits else 0
+
+
+def window_expand_attn(q, pages, group, runs, dims, scale: float, out, softcap: float = 0.0, sink=None, gate=None, diff=None) -> None:
+    """``window_attn`` for long portions without a window: keys and values of the sequences of ``group`` in rows of 128 channels,
+    then the flash-attention kernel (maps side by side in a key, queries with zeros at the other maps' channels). q as
+    ``window_prep`` leaves it with ``wide`` = 128; ``runs``: the group's sequences as ``AttnRun``s (models/state_cache.py)."""
+    H, G, M, D, DV = dims
+    T, dev = q.shape[0], q.device
+    direct = M == 1 and DV == 128 and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0
+    o = out[:, :H * 128].unflatten(1, (H, 128)) if direct else torch.empty(T, H * M, 128, dtype=q.dtype, device=dev)
+    for run in runs:
+        n_keys = run.slots.shape[0]
+        k128 = torch.empty(n_keys, G, 128, dtype=q.dtype, device=dev)
+        v128 = torch.empty_like(k128)
+        _chk(lib().pm_window_expand(_p(pages), _p(run.slots), c_int(n_keys), c_int(G), c_int(M), c_int(D), c_int(DV), _p(k128),
+                                    _p(v128), _stream()), "pm_window_expand")
+        attn_fwd_rect(q[run.rows], k128, v128, run.seq_start, scale, run.shift, o[run.rows], softcap, sink,
+                      gate[run.rows] if direct and gate is not None else None)
+    if direct:
+        return
+    lam, keep, eps = diff if diff is not None else (None, 1.0, 0.0)
+    _chk(lib().pm_window_finish(_p(o), c_int(T), c_int(H), c_int(M), c_int(DV), c_int(128), _p(group.q_start), _p(group.q_lens),
+                                c_int(group.n), c_int(group.max_q), _p(lam), c_float(keep), c_float(eps), _p(gate),
+                                c_ll(gate.stride(0) if gate is not None else 0), _p(out), c_ll(out.stride(0)), _stream()),
+         "pm_window_finish")

@@ -430,7 +430,64 @@ def test_routers_of_the_test_models_decide_clearly(monkeypatch):
     assert min(gaps) > 0.01, gaps
 
 
+def test_sequences_join_one_attention_launch():
+    """A launch takes in fresh prompts whose rows follow; earlier tokens of its first sequence shift the queries against the keys."""
+    from pmetal_b200.models.state_cache import CacheSpec, StateCache, attention_runs, split_groups
+    c = StateCache([CacheSpec(page_width=8)], 16, 8, torch.float32, "cpu")
+    for i in range(6):
+        c.add_sequence(i)
+    c.prepare([0], [70])
+    c.prepare([4], [5])
+    meta = c.prepare([0, 1, 2, 3, 4, 5], [30, 40, 1, 25, 20, 90])      # sequence 2 is a short portion, 4 has earlier tokens
+    runs = attention_runs(meta, split_groups(meta, 16)[1])
+    assert [(r.rows.start, r.rows.stop, r.n, r.shift) for r in runs] == [(0, 70, 70, 70), (71, 96, 25, 0), (96, 206, 110, 5)]
+    at = lambda i, p: c.seqs[i].blocks[p // BLOCK] * BLOCK + p % BLOCK      # noqa: E731
+    assert runs[0].slots.tolist() == [at(0, p) for p in range(100)] + [at(1, p) for p in range(40)]
+    assert runs[2].slots.tolist() == [at(4, p) for p in range(25)] + [at(5, p) for p in range(90)]
+    assert runs[0].seq_start.tolist() == [0] * 30 + [100] * 40 and runs[2].seq_start.tolist() == [0] * 20 + [25] * 90
+    for r in runs:                                            # the last key row a query sees is its own
+        rows = torch.arange(r.n) + r.shift
+        assert torch.equal(r.slots[rows], meta.slots[r.rows])
+
+
 # ------------------------------------------------------------------------------------------- kernels and modules
+@gpu
+@pytest.mark.parametrize("T,n,K", [(17, 1, 32), (64, 14, 192), (333, 33, 1024), (4100, 64, 96), (20, 20, 2048)])
+def test_router_logits(T, n, K):
+    from pmetal_b200.ops import functional as ops
+    from pmetal_b200.ops import native as nat
+    g = torch.Generator().manual_seed(T)
+    h, w = torch.randn(T, K + 8, generator=g).to(torch.bfloat16), torch.randn(-(-n // 8) * 8, K, generator=g).to(torch.bfloat16)
+    before = nat.LAUNCHES
+    got = ops.router_logits(h.cuda()[:, :K], w.cuda(), n)
+    assert nat.LAUNCHES == before + 1 and got.shape == (T, n) and got.dtype == torch.float32
+    want = h[:, :K].double() @ w[:n].double().t()
+    assert float((got.cpu().double() - want).abs().max()) < 1e-5 * K ** 0.5 * 4
+
+
+@gpu
+@pytest.mark.parametrize("cap", [0.0, 0.7, 30.0, 3000.0])
+def test_flash_attention_with_cap_sink_and_gate(cap):
+    """The tcgen05 kernel against the plain softmax: queries at an offset, documents, capped scores, a sink, output gates."""
+    from pmetal_b200.ops import native as nat
+    g = torch.Generator().manual_seed(int(cap))
+    H, G, T, prior = 4, 2, 300, 70
+    q, k, v = (torch.randn(n, h, 128, generator=g).to(torch.bfloat16) for n, h in ((T, H), (T + prior, G), (T + prior, G)))
+    sink_, gate = torch.randn(H, generator=g) * 2 + 2, torch.randn(T, H + 4, generator=g).to(torch.bfloat16)
+    start = torch.tensor([0] * 110 + [180] * 190, dtype=torch.int32)
+    o, lse = nat.attn_fwd_rect(q.cuda(), k.cuda(), v.cuda(), start.cuda(), 0.12, prior, softcap=cap, sink=sink_.cuda(), gate=gate.cuda()[:, 4:])
+    s = torch.einsum("ihd,jhd->hij", q.double(), k.double().repeat_interleave(H // G, 1)) * 0.12
+    s = cap * torch.tanh(s / cap) if cap else s
+    j, i = torch.arange(T + prior)[None], torch.arange(T)[:, None]
+    s = s.masked_fill((j > i + prior) | (j < start[:, None]), float("-inf"))
+    s = torch.cat([s, sink_.double()[:, None, None].expand(H, T, 1)], 2)
+    want = torch.einsum("hij,jhd->ihd", torch.softmax(s, -1)[:, :, :-1], v.double().repeat_interleave(H // G, 1))
+    want = want * torch.sigmoid(gate.double()[:, 4:])[:, :, None]
+    assert float((o.cpu().double() - want).abs().max()) < 0.02 * float(want.abs().max())
+    torch.testing.assert_close(lse.cpu().double(), torch.logsumexp(s, -1), atol=2e-3, rtol=1e-3)
+    nat.check_status()
+
+
 @gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("width", [48, 42, 1000, 2560])
