@@ -503,7 +503,7 @@ __global__ void __launch_bounds__(128) window_finish_kernel(const WindowFinishPa
     for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
     float f = exp2f(ms - m);
     f *= w / (warp_sum(ls * f) + exp2f(s2 - m));
-#pragma unroll 4
+#pragma unroll 8
     for (int s = 0; s < p.n_split; ++s) {
       const float fs = __shfl_sync(0xffffffffu, f, s);
       const float* src = p.po + (at + s * step) * p.DV8 + lane;
