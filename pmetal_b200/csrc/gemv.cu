@@ -58,6 +58,8 @@ struct GemvParams {
   int clamped;                   // gate of the SWIGLU variants: 0 silu(g) * u, 1 the clamped unit of elem.cuh; others: 2 exact gelu
   float glu_limit, glu_beta, glu_shift;
   float* y_f32;                  // [M, ldy] instead of y
+  float* tail;                   // nullable: columns from tail_from on go here as fp32, rows ld_tail apart
+  int tail_from, ld_tail;
 };
 
 __device__ __forceinline__ float gv_silu(float v) { return v / (1.f + __expf(-v)); }
@@ -75,7 +77,8 @@ __device__ __forceinline__ void gv_finish(const GemvParams& p, int m, int n, flo
     v = gelu_fast(v);
   }
   if (p.residual) v += __bfloat162float(p.residual[static_cast<long long>(m) * p.ldr + n]);
-  if (p.y_f32) p.y_f32[static_cast<long long>(m) * p.ldy + n] = v;
+  if (p.tail && n >= p.tail_from) p.tail[static_cast<long long>(m) * p.ld_tail + n - p.tail_from] = v;
+  else if (p.y_f32) p.y_f32[static_cast<long long>(m) * p.ldy + n] = v;
   else p.y[static_cast<long long>(m) * p.ldy + n] = __float2bfloat16(v);
 }
 
@@ -582,11 +585,13 @@ using namespace pm;
 
 // As pm_gemv with the epilogue of models that have biases and clamped gated units: bias [N_w] fp32 (nullable) is added to
 // the scaled products; with swiglu and clamped != 0 the pair becomes min(g, limit) * sigmoid(beta min(g, limit)) *
-// (clamp(u, -limit, limit) + shift); without swiglu, clamped = 2 applies the exact gelu; out_f32 != 0: y is fp32.
+// (clamp(u, -limit, limit) + shift); without swiglu, clamped = 2 applies the exact gelu; out_f32 != 0: y is fp32. tail (nullable):
+// output columns from tail_from on are stored there in fp32, rows ld_tail apart, and not in y.
 extern "C" int pm_gemv_ex(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps,
                           const void* residual, int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha,
                           const void* t, int ldt, const float* lora_b, int r, const int* seg_end, const float* bias,
-                          int clamped, float limit, float beta, float shift, int out_f32, cudaStream_t st) {
+                          int clamped, float limit, float beta, float shift, int out_f32, float* tail, int tail_from,
+                          int ld_tail, cudaStream_t st) {
   if (M < 1 || M > 16 || N < 1 || K < 8 || (K % 8) || (ldx % 8) || (ldw % 8)) return -1;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return -2;
   if (norm_w && (reinterpret_cast<uintptr_t>(norm_w) & 15)) return -2;
@@ -598,6 +603,7 @@ extern "C" int pm_gemv_ex(const void* x, int ldx, const void* w, int ldw, const 
   p.residual = static_cast<const __nv_bfloat16*>(residual); p.ldr = ldr;
   p.y = static_cast<__nv_bfloat16*>(y); p.ldy = ldy;
   if (out_f32) p.y_f32 = static_cast<float*>(y);
+  p.tail = tail; p.tail_from = tail_from; p.ld_tail = ld_tail;
   p.bias = bias; p.clamped = clamped; p.glu_limit = limit; p.glu_beta = beta; p.glu_shift = shift;
   p.M = M; p.N = N; p.K = K; p.swiglu = swiglu; p.alpha = alpha;
   p.t = static_cast<const __nv_bfloat16*>(t); p.ldt = ldt; p.lora_b = lora_b; p.r = r;
@@ -634,7 +640,7 @@ extern "C" int pm_gemv(const void* x, int ldx, const void* w, int ldw, const voi
                        int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha, const void* t, int ldt,
                        const float* lora_b, int r, const int* seg_end, cudaStream_t st) {
   return pm_gemv_ex(x, ldx, w, ldw, norm_w, eps, residual, ldr, y, ldy, M, N, K, swiglu, alpha, t, ldt, lora_b, r, seg_end,
-                    nullptr, 0, 0.f, 0.f, 0.f, 0, st);
+                    nullptr, 0, 0.f, 0.f, 0.f, 0, nullptr, 0, 0, st);
 }
 
 // 4-bit weights: qdata holds N_w * K / 2 bytes (two codes per byte, first element in the high nibble), absmax one fp32

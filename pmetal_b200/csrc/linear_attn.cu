@@ -226,16 +226,28 @@ __global__ void __launch_bounds__(256) linear_prep_kernel(const LinearPrepParams
 }
 
 // ------------------------------------------------------------------------------------------- norm and gate
-template <bool kSilu, bool kFast>
+enum : int { kGateSigmoid = 0, kGateSilu = 1, kGateNone = 2 };
+
+template <int kGate, bool kFast>
 __device__ __forceinline__ float gate_of(float g) {
-  if (kSilu) return kFast ? silu_fast(g) : silu_f(g);
+  if (kGate == kGateNone) return 1.f;
+  if (kGate == kGateSilu) return kFast ? silu_fast(g) : silu_f(g);
   return kFast ? sigmoid_fast(g) : sigmoid_f(g);
 }
 
+// What the norm kernels take beside y and the gate.
+struct NormGateExtra {
+  const float* w;          // nullable; [parts * width], shared: [width] for every part
+  const float* den;        // [tokens, parts], nullable: y is divided by it before the norm
+  int shared;
+  float scale;             // factor of the result
+  long long ldo;
+};
+
 // One warp per (token, part) with the part in registers: widths up to 256 IT, 8-element vectors.
-template <typename T, bool SILU, int IT>
+template <typename T, int GATE, int IT>
 __global__ void __launch_bounds__(256) norm_gate_warp_kernel(const T* __restrict__ y, const T* __restrict__ gate, long long ldg,
-                                                             const float* __restrict__ w, float eps, int parts, int width,
+                                                             const NormGateExtra x, float eps, int parts, int width,
                                                              T* __restrict__ out, int n_tok) {
   const long long item = blockIdx.x * 8ll + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -250,12 +262,14 @@ __global__ void __launch_bounds__(256) norm_gate_warp_kernel(const T* __restrict
     const int k = (i * 32 + lane) * 8;
     if (k < width) {
       load_vec<8>(y + row + c0 + k, v[i]);
-      load_vec<8>(gate + t * ldg + c0 + k, z[i]);
+      if (GATE != kGateNone) load_vec<8>(gate + t * ldg + c0 + k, z[i]);
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss = fmaf(v[i][e], v[i][e], ss);
     }
   }
-  const float r = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(width) + eps);
+  // y / den over its root mean square: y times r / den with the mean of squares over den^2
+  const float by = x.den ? 1.f / x.den[item] : 1.f;
+  const float r = x.scale * by / sqrtf(warp_sum(ss) * by * by / static_cast<float>(width) + eps);
 #pragma unroll
   for (int i = 0; i < IT; ++i) {
     const int k = (i * 32 + lane) * 8;
@@ -263,17 +277,17 @@ __global__ void __launch_bounds__(256) norm_gate_warp_kernel(const T* __restrict
       float g[8];
 #pragma unroll
       for (int e = 0; e < 8; ++e) g[e] = 1.f;
-      if (w) load_vec<8>(w + c0 + k, g);
+      if (x.w) load_vec<8>(x.w + (x.shared ? 0 : c0) + k, g);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) v[i][e] *= r * g[e] * gate_of<SILU, sizeof(T) == 2>(z[i][e]);
-      store_vec<8>(out + row + c0 + k, v[i]);
+      for (int e = 0; e < 8; ++e) v[i][e] *= r * g[e] * gate_of<GATE, sizeof(T) == 2>(z[i][e]);
+      store_vec<8>(out + t * x.ldo + c0 + k, v[i]);
     }
   }
 }
 
 // One CTA per (token, part), any width that shared memory holds.
-template <typename T, bool SILU, int V>
-__global__ void norm_gate_kernel(const T* __restrict__ y, const T* __restrict__ gate, long long ldg, const float* __restrict__ w,
+template <typename T, int GATE, int V>
+__global__ void norm_gate_kernel(const T* __restrict__ y, const T* __restrict__ gate, long long ldg, const NormGateExtra x,
                                  float eps, int width, T* __restrict__ out) {
   extern __shared__ __align__(16) float ng_row[];
   const long long t = blockIdx.x, row = t * gridDim.y * width;
@@ -288,16 +302,17 @@ __global__ void norm_gate_kernel(const T* __restrict__ y, const T* __restrict__ 
       ss = fmaf(v[e], v[e], ss);
     }
   }
-  const float r = 1.f / sqrtf(block_sum(ss) / static_cast<float>(width) + eps);
+  const float by = x.den ? 1.f / x.den[t * gridDim.y + blockIdx.y] : 1.f;
+  const float r = x.scale * by / sqrtf(block_sum(ss) * by * by / static_cast<float>(width) + eps);
   for (int k = threadIdx.x * V; k < width; k += blockDim.x * V) {
     float v[V], z[V], g[V];
-    load_vec<V>(gate + t * ldg + c0 + k, z);
+    if (GATE != kGateNone) load_vec<V>(gate + t * ldg + c0 + k, z);
 #pragma unroll
     for (int e = 0; e < V; ++e) g[e] = 1.f;
-    if (w) load_vec<V>(w + c0 + k, g);
+    if (x.w) load_vec<V>(x.w + (x.shared ? 0 : c0) + k, g);
 #pragma unroll
-    for (int e = 0; e < V; ++e) v[e] = ng_row[k + e] * r * g[e] * gate_of<SILU, sizeof(T) == 2>(z[e]);
-    store_vec<V>(out + row + c0 + k, v);
+    for (int e = 0; e < V; ++e) v[e] = ng_row[k + e] * r * g[e] * gate_of<GATE, sizeof(T) == 2>(z[e]);
+    store_vec<V>(out + t * x.ldo + c0 + k, v);
   }
 }
 
@@ -323,35 +338,36 @@ static int linear_scan_launch(LinearScanParams<T> p, int n_seq, cudaStream_t st)
   return static_cast<int>(cudaGetLastError());
 }
 
-template <typename T, bool SILU>
-static int norm_gate_launch(const void* y, const void* gate, long long ldg, const float* w, float eps, int parts, int width,
+template <typename T, int GATE>
+static int norm_gate_launch(const void* y, const void* gate, long long ldg, const NormGateExtra& x, float eps, int parts, int width,
                             void* out, int n_tok, cudaStream_t st) {
   const T* yy = static_cast<const T*>(y);
   const T* gg = static_cast<const T*>(gate);
   T* oo = static_cast<T*>(out);
-  const bool v8 = width % 8 == 0 && ldg % 8 == 0 && reinterpret_cast<uintptr_t>(gate) % (8 * sizeof(T)) == 0;
+  const bool v8 = width % 8 == 0 && ldg % 8 == 0 && x.ldo % 8 == 0 &&
+                  (reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) % (8 * sizeof(T)) == 0;
   // a warp per part pays when there are parts enough to fill the machine
   if (v8 && width <= 1024 && (width <= 256 || static_cast<long long>(n_tok) * parts >= 8ll * num_sms())) {
     const unsigned grid = static_cast<unsigned>((static_cast<long long>(n_tok) * parts + 7) / 8);
-    if (width <= 256) norm_gate_warp_kernel<T, SILU, 1><<<grid, 256, 0, st>>>(yy, gg, ldg, w, eps, parts, width, oo, n_tok);
-    else if (width <= 512) norm_gate_warp_kernel<T, SILU, 2><<<grid, 256, 0, st>>>(yy, gg, ldg, w, eps, parts, width, oo, n_tok);
-    else norm_gate_warp_kernel<T, SILU, 4><<<grid, 256, 0, st>>>(yy, gg, ldg, w, eps, parts, width, oo, n_tok);
+    if (width <= 256) norm_gate_warp_kernel<T, GATE, 1><<<grid, 256, 0, st>>>(yy, gg, ldg, x, eps, parts, width, oo, n_tok);
+    else if (width <= 512) norm_gate_warp_kernel<T, GATE, 2><<<grid, 256, 0, st>>>(yy, gg, ldg, x, eps, parts, width, oo, n_tok);
+    else norm_gate_warp_kernel<T, GATE, 4><<<grid, 256, 0, st>>>(yy, gg, ldg, x, eps, parts, width, oo, n_tok);
     return static_cast<int>(cudaGetLastError());
   }
   const size_t smem = static_cast<size_t>(width) * sizeof(float);
   static DeviceOnce once;
   if (once.pending()) {
-    cudaError_t e = cudaFuncSetAttribute(norm_gate_kernel<T, SILU, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(norm_gate_kernel<T, GATE, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(norm_gate_kernel<T, SILU, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      e = cudaFuncSetAttribute(norm_gate_kernel<T, GATE, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e != cudaSuccess) return static_cast<int>(e);
     once.mark();
   }
   const int v = v8 ? 8 : 1;
   int threads = (width / v + 31) / 32 * 32;
   threads = threads < 32 ? 32 : (threads > 512 ? 512 : threads);
-  if (v8) norm_gate_kernel<T, SILU, 8><<<dim3(n_tok, parts), threads, smem, st>>>(yy, gg, ldg, w, eps, width, oo);
-  else norm_gate_kernel<T, SILU, 1><<<dim3(n_tok, parts), threads, smem, st>>>(yy, gg, ldg, w, eps, width, oo);
+  if (v8) norm_gate_kernel<T, GATE, 8><<<dim3(n_tok, parts), threads, smem, st>>>(yy, gg, ldg, x, eps, width, oo);
+  else norm_gate_kernel<T, GATE, 1><<<dim3(n_tok, parts), threads, smem, st>>>(yy, gg, ldg, x, eps, width, oo);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -422,15 +438,24 @@ extern "C" int pm_linear_chunk(const void* u, long long ldu, const float* cs, co
   return ssd_chunk_launch(p, n_seq, max_q, max_seg, st);
 }
 
-// out [tokens, parts * width] = RMS norm over every part of y, times w (fp32 [parts * width] or null), times
-// sigmoid(gate) or, silu 1, silu(gate); gate rows are ldg apart.
+template <typename T>
+static int norm_gate_any(const void* y, const void* gate, long long ldg, const NormGateExtra& x, float eps, int parts, int width, int silu,
+                         void* out, int n_tok, cudaStream_t st) {
+  if (!gate) return norm_gate_launch<T, kGateNone>(y, nullptr, 0, x, eps, parts, width, out, n_tok, st);
+  return silu ? norm_gate_launch<T, kGateSilu>(y, gate, ldg, x, eps, parts, width, out, n_tok, st)
+              : norm_gate_launch<T, kGateSigmoid>(y, gate, ldg, x, eps, parts, width, out, n_tok, st);
+}
+
+// out [tokens, ldo] = RMS norm over every part of y [tokens, parts * width], times w (fp32 [parts * width], shared 1: [width] for every
+// part, or null), times sigmoid(gate) or, silu 1, silu(gate), times scale; gate rows are ldg apart (null: no gate). den (fp32
+// [tokens, parts], nullable): y is divided by it first.
 extern "C" int pm_norm_gate(const void* y, const void* gate, int f32, long long ldg, const float* w, float eps, int parts,
-                            int width, int silu, void* out, int n_tok, cudaStream_t st) {
-  if (parts < 1 || width < 1 || static_cast<size_t>(width) * 4 > 200 * 1024 || parts > 65535) return -1;
+                            int width, int silu, void* out, int n_tok, const float* den, int shared, float scale, long long ldo,
+                            cudaStream_t st) {
+  if (parts < 1 || width < 1 || static_cast<size_t>(width) * 4 > 200 * 1024 || parts > 65535 || ldo < static_cast<long long>(parts) * width)
+    return -1;
   if (n_tok < 1) return 0;
-  if (f32)
-    return silu ? norm_gate_launch<float, true>(y, gate, ldg, w, eps, parts, width, out, n_tok, st)
-                : norm_gate_launch<float, false>(y, gate, ldg, w, eps, parts, width, out, n_tok, st);
-  return silu ? norm_gate_launch<__nv_bfloat16, true>(y, gate, ldg, w, eps, parts, width, out, n_tok, st)
-              : norm_gate_launch<__nv_bfloat16, false>(y, gate, ldg, w, eps, parts, width, out, n_tok, st);
+  const NormGateExtra x{w, den, shared, scale, ldo};
+  return f32 ? norm_gate_any<float>(y, gate, ldg, x, eps, parts, width, silu, out, n_tok, st)
+             : norm_gate_any<__nv_bfloat16>(y, gate, ldg, x, eps, parts, width, silu, out, n_tok, st);
 }

@@ -142,6 +142,37 @@ int pm_f32_to_bf16(const float* in, void* out, long long n, cudaStream_t st);
 int pm_dequant_4bit(const void* data, const float* absmax, const void* absmax_q, float am_scale, float am_offset,
     void* out, long long n, int block_size, int fp4, cudaStream_t st);
 
+// ---------------------------------------------------------------- gated_linear.cu
+// Channel gates token by token. q / v: head 0's first column in row 0 of rows ldu apart, z fp32 rows of H N logits ldz apart, bias
+// and lower fp32 [H N]; state [slots][H][N][P4] fp32, read and written; y [tokens, H P]. Sequence i covers tokens q_start[i] ..
+// + q_lens[i] - 1 and ends at position seq_lens[i] - 1.
+int pm_channel_scan(const void* q, const void* v, int f32, long long ldu, const float* z, long long ldz, const
+    float* bias, const float* lower, float* state, const int* slots, const int* q_start, const int* q_lens, const
+    int* seq_lens, int n_seq, int H, int N, int P, void* y, cudaStream_t st);
+// Matrix memory token by token. q / k / v as above, z fp32 rows of H input gates and H forget gates, bias fp32 [2 H]; nstate
+// [slots][H][N] and mstate [slots][H][P4 / 4] fp32 beside the state; y [tokens, H P] without, den fp32 [tokens, H] with the
+// normaliser: the result is y / den.
+int pm_memory_scan(const void* q, const void* k, const void* v, int f32, long long ldu, const float* z, long long
+    ldz, const float* bias, float cap, float qscale, float den_eps, float* state, float* nstate, float* mstate,
+    const int* slots, const int* q_start, const int* q_lens, const int* seq_lens, int n_seq, int H, int N, int P,
+    void* y, float* den, cudaStream_t st);
+// pm_channel_scan for longer portions of bf16 models, N <= 256, n16 = N rounded up to 16. Work buffers over all rows of the step: act
+// bf16 [tokens, 4 H n16], score bf16 [tokens, H, 128]; block_decay fp32 [n_tok / 64 + n_seq + 1][H][n16]; seg_state
+// [n_seq][max_seg][H][N][P4] and seg_decay [n_seq][max_seg][H][N] fp32. c_start: first token of every sequence, counted over these
+// sequences alone; max_q: the longest of q_lens.
+int pm_channel_chunk(const void* q, const void* v, long long ldu, const float* z, long long ldz, const float* bias,
+    const float* lower, float* state, const int* slots, const int* q_start, const int* q_lens, const int* seq_lens,
+    const int* c_start, int n_seq, int max_q, int H, int N, int P, void* act, void* score, float* block_decay,
+    float* seg_state, float* seg_decay, int max_seg, void* y, cudaStream_t st);
+// pm_memory_scan for longer portions of bf16 models, N <= 256. u: rows ldu apart with the keys of head 0 at column k_at and the
+// queries at q_at; work buffers gates fp32 [3][tokens, H], seg_state [n_seq][max_seg][H][N][P4], seg_decay [n_seq][max_seg][H] and
+// seg_n [n_seq][max_seg][H][N] fp32.
+int pm_memory_chunk(const void* u, int q_at, int k_at, const void* v, long long ldu, const float* z, long long ldz,
+    const float* bias, float cap, float qscale, float den_eps, float* state, float* nstate, float* mstate, const
+    int* slots, const int* q_start, const int* q_lens, const int* seq_lens, int n_seq, int n_tok, int max_q, int H,
+    int N, int P, float* gates, float* seg_state, float* seg_decay, float* seg_n, int max_seg, void* y, float* den,
+    cudaStream_t st);
+
 // ---------------------------------------------------------------- gdn.cu
 // Returns 0, -1 for an unsupported head shape (supported: dk x dv in {64, 128} x {64, 128}), or a CUDA error code.
 int pm_gdn_scan(const float* q, const float* k, const float* v, const float* g, const float* beta, float* state,
@@ -178,11 +209,12 @@ int pm_gemm_bf16(const void* A, int a_mn, int lda, int a_rows, const void* B, in
 // ---------------------------------------------------------------- gemv.cu
 // As pm_gemv with the epilogue of models that have biases and clamped gated units: bias [N_w] fp32 (nullable) is added to
 // the scaled products; with swiglu and clamped != 0 the pair becomes min(g, limit) * sigmoid(beta min(g, limit)) *
-// (clamp(u, -limit, limit) + shift); without swiglu, clamped = 2 applies the exact gelu; out_f32 != 0: y is fp32.
+// (clamp(u, -limit, limit) + shift); without swiglu, clamped = 2 applies the exact gelu; out_f32 != 0: y is fp32. tail (nullable):
+// output columns from tail_from on are stored there in fp32, rows ld_tail apart, and not in y.
 int pm_gemv_ex(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps, const void* residual,
     int ldr, void* y, int ldy, int M, int N, int K, int swiglu, float alpha, const void* t, int ldt, const float*
     lora_b, int r, const int* seg_end, const float* bias, int clamped, float limit, float beta, float shift, int
-    out_f32, cudaStream_t st);
+    out_f32, float* tail, int tail_from, int ld_tail, cudaStream_t st);
 // Returns 0, a negative argument error, or a CUDA error code. K % 8 == 0, row strides % 8 == 0, M <= 16,
 // M * cols-per-warp <= 32.
 int pm_gemv(const void* x, int ldx, const void* w, int ldw, const void* norm_w, float eps, const void* residual,
@@ -255,10 +287,12 @@ int pm_linear_chunk(const void* u, long long ldu, const float* cs, const float* 
     kscale, float* state, const int* slots, const int* q_start, const int* q_lens, const int* seq_lens, int n_seq,
     int n_tok, int max_q, int H, int N, int P, int R, int rot, int act, void* act_buf, float* seg_state, float*
     seg_decay, int max_seg, void* y, cudaStream_t st);
-// out [tokens, parts * width] = RMS norm over every part of y, times w (fp32 [parts * width] or null), times
-// sigmoid(gate) or, silu 1, silu(gate); gate rows are ldg apart.
+// out [tokens, ldo] = RMS norm over every part of y [tokens, parts * width], times w (fp32 [parts * width], shared 1: [width] for every
+// part, or null), times sigmoid(gate) or, silu 1, silu(gate), times scale; gate rows are ldg apart (null: no gate). den (fp32
+// [tokens, parts], nullable): y is divided by it first.
 int pm_norm_gate(const void* y, const void* gate, int f32, long long ldg, const float* w, float eps, int parts, int
-    width, int silu, void* out, int n_tok, cudaStream_t st);
+    width, int silu, void* out, int n_tok, const float* den, int shared, float scale, long long ldo, cudaStream_t
+    st);
 
 // ---------------------------------------------------------------- mhc.cu
 // x [T, n, C] bf16; either phi [n C, n^2 + 2n] fp32 (dot products formed here) or raw [T, ld_raw] fp32 = x . phi computed by
@@ -380,6 +414,26 @@ int pm_spec_verify(const float* target, const float* draft, const int* tokens, i
     cudaStream_t st);
 int pm_count_tokens(int* counts, const int* count_rows, const int* tokens, int rows, int vocab, cudaStream_t st);
 
+// ---------------------------------------------------------------- sandwich.cu
+// xf [n, width] fp32 = table[id] + pairs[row] + pos_table[position], xc (nullable, rows ldc apart) the same in the tables' type; row =
+// (previous id * mul_prev + id * mul_cur) mod buckets, `buckets` itself for a sequence's first token. Sequence i brings the tokens
+// q_start[i] .. + q_lens[i] - 1; last[slots[i]] (int32) holds its latest token, read and written. Positions lie below max_pos.
+int pm_pair_embed(const long long* ids, const void* table, const void* pairs, const void* pos_table, int f32, const
+    int* pos, const int* seq_of, const int* q_start, const int* q_lens, const int* slots, int* last, long long
+    buckets, long long mul_prev, long long mul_cur, int n, int width, int max_pos, float* xf, void* xc, long long
+    ldc, cudaStream_t st);
+// v = x + r / rms(r) (base + wb), r = y + bias (y nullable: v = x), for the n rows listed in `rows` (nullable: row i); of [n, width]
+// fp32 (nullable, written when there is a y; may be x when rows is null) = v, oc (nullable, compute type, rows ldo apart) =
+// v / rms(v) (base + wn), without wn v itself. conv (nullable, [taps][width] fp32, with wn and without rows): row i is the only new
+// token of a sequence, at position pos[i] with the ring of slot slots[i]; oc = h + sum_j conv[j] h_(taps - 1 - j tokens earlier).
+int pm_branch_norm(const float* x, const void* y, int f32, long long ldy, const float* bias, const float* wb, const
+    float* wn, float base, float eps, const long long* rows, float* of, void* oc, long long ldo, const float* conv,
+    int taps, void* ring, const int* slots, const int* pos, int n, int width, cudaStream_t st);
+// out [tokens, width] = h + causal convolution of h with w [taps][width] fp32 along every sequence; h and out in the compute type,
+// two buffers. ring [slot][taps - 1][width] (compute type) holds the sequences' earlier inputs, read and written. taps <= 17.
+int pm_canon(const void* h, int f32, const float* w, int taps, void* ring, const int* slots, const int* q_start,
+    const int* q_lens, const int* seq_lens, int n_seq, int max_q, int width, void* out, cudaStream_t st);
+
 // ---------------------------------------------------------------- ssm.cu
 // Token-by-token recurrence with the convolution inside. u [tokens, ldu]; conv_w [taps][conv], conv_b, dt_bias, a_log,
 // dskip fp32; ring [slots][taps][conv] in u's type; state [slots][H][N][P4] fp32, read and written; y [tokens, H P].
@@ -442,12 +496,14 @@ int pm_window_prep(const void* u, int f32, long long ldu, const float* cs, const
 // softcap > 0; sink (fp32 [H], M = 1) adds exp(sink) to a head's softmax sum; gate [.., ldg] multiplies head h by the sigmoid of
 // column h. M = 2: the result of a head is a_1 - lambda[0] a_2 over its root mean square (eps inside), times keep; it takes o
 // [n_tok, H M, DV] in the compute type unless parts are given. few 1: decode tiles (a few rows per sequence), which take work
-// buffers po [n_split][n_tok][H M][DV8] and pml [n_split][n_tok][H M][2] (both or none; needed for n_split > 1).
+// buffers po [n_split][n_tok][H M][DV8] and pml [n_split][n_tok][H M][2] (both or none; needed for n_split > 1). chunked 1: a position
+// sees the keys of its own chunk of `window` positions. wbias (fp32 [H], nullable, M = 1, without sink): the weight of a key is the
+// sigmoid of its score + wbias, not divided by their sum. out_scale multiplies the result.
 int pm_window_attn(const void* q, int f32, const void* pages, const int* block_table, const int* seq_lens, const
     int* q_start, const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H, int G, int M, int D,
     int DV, int wide, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg,
     const float* lambda, float keep, float eps, int few, int n_split, float* po, float* pml, void* o, void* out,
-    long long ldo, cudaStream_t st);
+    long long ldo, int chunked, const float* wbias, float out_scale, cudaStream_t st);
 // k128 / v128 [n, G, 128] bf16 = the cached keys (M maps of D8 channels side by side) and values (DV8) of the n cache rows in `slots`
 // (page * 64 + offset), zero padded. M D8 <= 128 and DV8 <= 128.
 int pm_window_expand(const void* pages, const long long* slots, int n, int G, int M, int D, int DV, void* k128,

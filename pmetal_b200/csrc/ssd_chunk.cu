@@ -5,9 +5,11 @@
 //     S  <- exp(a_63) S + sum_j exp(a_63 - a_j) dt_j B_j x_j^T
 //
 // State-space layers (ssm.cu) have step sizes dt per token and B, C shared by groups of heads; linear attention
-// (linear_attn.cu) has keys and queries per head as B and C, values as x, steps of 1 and a fixed decay. x, B and C are bf16
-// activations (or, SPLIT, B and C the sums of two bf16 terms); every fp32 factor (decayed scores, state, decayed B) enters
-// the products as the sum of two bf16 terms, so the recurrence keeps about 16 bits in its operands and fp32 in its sums.
+// (linear_attn.cu) has keys and queries per head as B and C, values as x, steps of 1 and a fixed decay. The matrix memory
+// (gated_linear.cu) has decays and weights per token and a normaliser beside the state, kept in fp32; layers with a decay per
+// state row bring the scores within the blocks and B, C with the decays inside. x, B and C are bf16 activations (or, SPLIT, B and
+// C the sums of two bf16 terms); every fp32 factor (decayed scores, state, decayed B) enters the products as the sum of two bf16
+// terms, so the recurrence keeps about 16 bits in its operands and fp32 in its sums.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -21,12 +23,13 @@ namespace pm {
 constexpr int kChunk = 64;
 constexpr int kSlice = 32;            // channels of P per CTA
 constexpr int kLdX = kSlice + 8;
+constexpr int kLdA = kChunk + 8;
 constexpr float kLog2e = 1.4426950408889634f;
 
-// Rows t0 .. t0 + 63 of `act`, `width` columns from c0 (multiple of 8, zero filled beyond valid_w and beyond the portion).
-__device__ __forceinline__ void ssd_load_rows(const SsdParams& p, __nv_bfloat16* dst, int ld, int width, int valid_w, int c0,
-                                              long long q0, int t0, int len) {
-  if (p.aligned) {
+// Rows t0 .. t0 + 63 of `act` (lda apart), `width` columns from c0 (multiple of 8, zero filled beyond valid_w and beyond the portion).
+__device__ __forceinline__ void ssd_load_rows(const __nv_bfloat16* act, long long lda, bool aligned, __nv_bfloat16* dst, int ld,
+                                              int width, int valid_w, int c0, long long q0, int t0, int len) {
+  if (aligned) {
     const int per = width / 8, dr = 128 / per, dc = 128 - dr * per;
     int r = threadIdx.x / per, c = threadIdx.x - r * per;
     for (; r < kChunk; r += dr, c += dc) {
@@ -35,14 +38,14 @@ __device__ __forceinline__ void ssd_load_rows(const SsdParams& p, __nv_bfloat16*
         if (++r >= kChunk) break;
       }
       const bool ok = t0 + r < len && c * 8 < valid_w;
-      const __nv_bfloat16* src = p.act + (q0 + (ok ? t0 + r : 0)) * p.ld + c0 + (ok ? c * 8 : 0);
+      const __nv_bfloat16* src = act + (q0 + (ok ? t0 + r : 0)) * lda + c0 + (ok ? c * 8 : 0);
       ms_cp16(ms_addr(dst + r * ld + c * 8), src, ok);
     }
   } else {
     for (int i = threadIdx.x; i < kChunk * width; i += 128) {
       const int r = i / width, c = i - r * width;
       const bool ok = t0 + r < len && c < valid_w;
-      dst[r * ld + c] = ok ? p.act[(q0 + t0 + r) * p.ld + c0 + c] : __float2bfloat16(0.f);
+      dst[r * ld + c] = ok ? act[(q0 + t0 + r) * lda + c0 + c] : __float2bfloat16(0.f);
     }
   }
 }
@@ -53,17 +56,18 @@ __device__ __forceinline__ float ssd_rate(const SsdParams& p, int h) {
 }
 
 // One warp's copy of the block's running log2 decays and of the weights with which its tokens enter the state; returns the
-// log2 decay over the block.
-__device__ __forceinline__ float ssd_decays(const float* dts, float a2, float* cum, float* wgt, int lane) {
+// log2 decay over the block. A token's log2 decay is lds[.] or, where that is null, a2 times its step.
+__device__ __forceinline__ float ssd_decays(const float* dts, const float* lds, float a2, float* cum, float* wgt, int lane) {
   const float d0 = dts[2 * lane], d1 = dts[2 * lane + 1];
-  float run = a2 * d0 + a2 * d1;
+  const float l0 = lds ? lds[2 * lane] : a2 * d0, l1 = lds ? lds[2 * lane + 1] : a2 * d1;
+  float run = l0 + l1;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
     const float up = __shfl_up_sync(0xffffffffu, run, o);
     if (lane >= o) run += up;
   }
   const float total = __shfl_sync(0xffffffffu, run, 31);
-  const float c1 = run, c0 = run - a2 * d1;
+  const float c1 = run, c0 = run - l1;
   __syncwarp();
   *reinterpret_cast<float2*>(cum + 2 * lane) = make_float2(c0, c1);
   *reinterpret_cast<float2*>(wgt + 2 * lane) = make_float2(exp2f(total - c0) * d0, exp2f(total - c1) * d1);
@@ -71,23 +75,35 @@ __device__ __forceinline__ float ssd_decays(const float* dts, float a2, float* c
   return total;
 }
 
-// S (rows of this warp) <- keep * S + sum_j wgt_j B_j x_j^T; SPLIT: B = tile at aB + tile at aBl
-template <int NI, bool SPLIT>
-__device__ __forceinline__ void ssd_update(float (&S)[NI][4][4], float keep, const float* wgt, uint32_t aB, uint32_t aBl,
-                                           uint32_t aX, int ldn, int n16, int warp, int lane) {
+// S (rows of this warp) <- keep * S + sum_j wgt_j B_j x_j^T; SPLIT: B = tile at aB + tile at aBl. CHANNEL: keeps[row] in place of
+// keep, and B is taken as it is.
+template <int NI, bool SPLIT, bool CHANNEL>
+__device__ __forceinline__ void ssd_update(float (&S)[NI][4][4], float keep, const float* keeps, const float* wgt, uint32_t aB,
+                                           uint32_t aBl, uint32_t aX, int ldn, int n16, int warp, int lane) {
 #pragma unroll
-  for (int i = 0; i < NI; ++i)
+  for (int i = 0; i < NI; ++i) {
+    float k0 = keep, k1 = keep;
+    if (CHANNEL) {
+      const int row = (warp + 4 * i) * 16 + (lane >> 2);
+      k0 = row < n16 ? keeps[row] : 0.f;
+      k1 = row < n16 ? keeps[row + 8] : 0.f;
+    }
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) S[i][nt][e] *= keep;
+      for (int e = 0; e < 4; ++e) S[i][nt][e] *= e & 2 ? k1 : k0;
+  }
 #pragma unroll
   for (int kk = 0; kk < 4; ++kk) {
     uint32_t fx[2][4];
 #pragma unroll
     for (int np = 0; np < 2; ++np) ms_ldsm4_t(ms_b_nn_at(aX, kLdX, kk * 16, np * 16, lane), fx[np]);
     const int j = kk * 16 + 2 * (lane & 3);
-    const float2 wa = *reinterpret_cast<const float2*>(wgt + j), wb = *reinterpret_cast<const float2*>(wgt + j + 8);
+    float2 wa, wb;
+    if (!CHANNEL) {
+      wa = *reinterpret_cast<const float2*>(wgt + j);
+      wb = *reinterpret_cast<const float2*>(wgt + j + 8);
+    }
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
       const int n0 = (warp + 4 * i) * 16;
@@ -97,6 +113,11 @@ __device__ __forceinline__ void ssd_update(float (&S)[NI][4][4], float keep, con
       if (SPLIT) ms_ldsm4_t(ms_a_t_at(aBl, ldn, kk * 16, n0, lane), fbl);
 #pragma unroll
       for (int q = 0; q < 4; ++q) {
+        if (CHANNEL) {
+          fh[q] = fb[q];
+          fl[q] = fbl[q];
+          continue;
+        }
         float lo = __uint_as_float(fb[q] << 16), hi = __uint_as_float(fb[q] & 0xffff0000u);
         if (SPLIT) {
           lo += __uint_as_float(fbl[q] << 16);
@@ -129,9 +150,23 @@ __device__ __forceinline__ void ssd_each(float (&S)[NI][4][4], int n, int pw, in
       }
 }
 
+// n (rows threadIdx.x and threadIdx.x + 128) <- keep n + sum_j wgt_j B_j, in fp32.
+__device__ __forceinline__ void ssd_norm_add(float (&n)[2], float keep, const float* wgt, const __nv_bfloat16* B, int ldn, int N) {
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int row = threadIdx.x + 128 * i;
+    if (row >= N) continue;
+    float v = n[i] * keep;
+#pragma unroll 8
+    for (int j = 0; j < kChunk; ++j) v = fmaf(wgt[j], __bfloat162float(B[j * ldn + row]), v);
+    n[i] = v;
+  }
+}
+
 // What every segment but the last adds to the state, with segment-parallel CTAs. grid (slices * n_seg, H, sequences).
-template <int NI, bool SPLIT>
+template <int NI, bool SPLIT, int KIND>
 __global__ void __launch_bounds__(128) ssd_segment_kernel(const SsdParams p) {
+  constexpr bool MEMORY = KIND == kSsdMemory, CHANNEL = KIND == kSsdChannel;
   extern __shared__ __align__(16) uint8_t ssd_smem[];
   const SsdParams& d = p;
   const int slices = gridDim.x / p.n_seg;
@@ -147,19 +182,27 @@ __global__ void __launch_bounds__(128) ssd_segment_kernel(const SsdParams p) {
   float* sDt = reinterpret_cast<float*>(sX + 2 * tile_x);                // [2][64]
   float* cum = sDt + 2 * kChunk + warp * kChunk;                         // [4 warps][64]
   float* wgt = sDt + 6 * kChunk + warp * kChunk;                         // [4 warps][64]
+  float* sLd = sDt + 10 * kChunk;                                        // [2][64] (MEMORY) or the blocks' decays [2][n16] (CHANNEL)
   const long long q0 = p.q_start[seq];
   const int start = p.seq_lens[seq] - len;
   const int g = h / (d.H / d.G);
-  const int cx = h * d.P + p0, cb = d.b0 + g * d.N, pw = min(kSlice, d.P - p0);
-  const float a2 = ssd_rate(p, h);
+  const int cx = h * d.P + p0, cb = d.b0 + g * d.NB, pw = min(kSlice, d.P - p0);
+  const float a2 = KIND == kSsdPlain ? ssd_rate(p, h) : 0.f;
+  const bool norm = MEMORY && p0 == 0;                                   // this CTA keeps the head's normaliser
   const long long mat = static_cast<long long>(d.N) * d.P4;
   auto slot_of = [&](int k) { return (static_cast<long long>(seq) * p.n_seg + k) * d.H + h; };
   auto load_chunk = [&](int ch, int buf) {
     const int t0 = ch * kChunk;
-    ssd_load_rows(p, sB + buf * tile_n, ldn, p.n16, d.N, cb, q0, t0, len);
-    if (SPLIT) ssd_load_rows(p, sBl + buf * tile_n, ldn, p.n16, d.N, cb + d.lo, q0, t0, len);
-    ssd_load_rows(p, sX + buf * tile_x, kLdX, kSlice, pw, cx, q0, t0, len);
-    if (threadIdx.x < kChunk) sDt[buf * kChunk + threadIdx.x] = p.dt ? p.dt[(q0 + t0 + threadIdx.x) * d.H + h] : 1.f;
+    ssd_load_rows(p.act, p.ld, p.aligned, sB + buf * tile_n, ldn, p.n16, d.N, cb, q0, t0, len);
+    if (SPLIT) ssd_load_rows(p.act, p.ld, p.aligned, sBl + buf * tile_n, ldn, p.n16, d.N, cb + d.lo, q0, t0, len);
+    ssd_load_rows(p.x, p.ldx, p.aligned_x, sX + buf * tile_x, kLdX, kSlice, pw, cx, q0, t0, len);
+    if (CHANNEL) {
+      const long long block = p.c_start[seq] / kChunk + seq + ch;
+      for (int n = threadIdx.x; n < p.n16; n += 128) sLd[buf * p.n16 + n] = p.block_decay[(block * d.H + h) * d.NB + n];
+    } else if (threadIdx.x < kChunk) {
+      sDt[buf * kChunk + threadIdx.x] = p.dt ? p.dt[(q0 + t0 + threadIdx.x) * d.H + h] : 1.f;
+      if (MEMORY) sLd[buf * kChunk + threadIdx.x] = p.ldec[(q0 + t0 + threadIdx.x) * d.H + h];
+    }
     ms_commit();
   };
   float S[NI][4][4];
@@ -178,28 +221,48 @@ __global__ void __launch_bounds__(128) ssd_segment_kernel(const SsdParams p) {
       const long long o = static_cast<long long>(n) * d.P4 + c;
       *reinterpret_cast<float2*>(dst + o) = start > 0 ? *reinterpret_cast<const float2*>(st + o) : make_float2(0.f, 0.f);
     });
+    if (norm)
+      for (int n = threadIdx.x; n < d.N; n += 128)
+        p.seg_n[slot_of(0) * d.N + n] = start > 0 ? p.nstate[(static_cast<long long>(p.slots[seq]) * d.H + h) * d.N + n] : 0.f;
   }
-  float sum = 0.f;
+  float sum = 0.f, nacc[2] = {0.f, 0.f}, ndec[2] = {1.f, 1.f};       // CHANNEL: ndec, the decays of this thread's rows
   for (int k = 0; k < p.seg_chunks; ++k) {
     const int buf = k & 1;
     ms_wait<0>();
     __syncthreads();
     if (k + 1 < p.seg_chunks) load_chunk(c0 + k + 1, buf ^ 1);
-    const float total = ssd_decays(sDt + buf * kChunk, a2, cum, wgt, lane);
+    float total = 0.f;
+    if (!CHANNEL) total = ssd_decays(sDt + buf * kChunk, MEMORY ? sLd + buf * kChunk : nullptr, a2, cum, wgt, lane);
     sum += total;
-    ssd_update<NI, SPLIT>(S, exp2f(total), wgt, ms_addr(sB + buf * tile_n), ms_addr(sBl + buf * tile_n),
-                          ms_addr(sX + buf * tile_x), ldn, p.n16, warp, lane);
+    ssd_update<NI, SPLIT, CHANNEL>(S, exp2f(total), sLd + buf * p.n16, wgt, ms_addr(sB + buf * tile_n), ms_addr(sBl + buf * tile_n),
+                                   ms_addr(sX + buf * tile_x), ldn, p.n16, warp, lane);
+    if (norm) ssd_norm_add(nacc, exp2f(total), wgt, sB + buf * tile_n, ldn, d.N);
+    if (CHANNEL)
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        if (static_cast<int>(threadIdx.x) + 128 * i < d.N) ndec[i] *= sLd[buf * p.n16 + threadIdx.x + 128 * i];
   }
   float* dst = p.seg_state + slot_of(seg + 1) * mat + p0;
   ssd_each<NI>(S, d.N, pw, warp, lane, [&](float& v0, float& v1, int n, int c) {
     *reinterpret_cast<float2*>(dst + static_cast<long long>(n) * d.P4 + c) = make_float2(v0, v1);
   });
-  if (threadIdx.x == 0 && p0 == 0) p.seg_decay[slot_of(seg)] = exp2f(sum);
+  if (CHANNEL && p0 == 0) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (static_cast<int>(threadIdx.x) + 128 * i < d.N) p.seg_decay[slot_of(seg) * d.N + threadIdx.x + 128 * i] = ndec[i];
+  } else if (threadIdx.x == 0 && p0 == 0) {
+    p.seg_decay[slot_of(seg)] = exp2f(sum);
+  }
+  if (norm)
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (static_cast<int>(threadIdx.x) + 128 * i < d.N) p.seg_n[slot_of(seg + 1) * d.N + threadIdx.x + 128 * i] = nacc[i];
 }
 
 // NI: state row tiles (16 rows) per warp; 4 warps cover N <= 64 NI. Same grid as ssd_segment_kernel.
-template <int NI, bool SPLIT>
+template <int NI, bool SPLIT, int KIND>
 __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
+  constexpr bool MEMORY = KIND == kSsdMemory, CHANNEL = KIND == kSsdChannel;
   extern __shared__ __align__(16) uint8_t ssd_smem[];
   const SsdParams& d = p;
   const int slices = gridDim.x / p.n_seg;
@@ -216,30 +279,42 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
   __nv_bfloat16* sX = sB + (SPLIT ? 3 : 1) * tile_n;                     // [64][kLdX]
   __nv_bfloat16* sSh = sX + tile_x;                                      // [n16][kLdX]
   __nv_bfloat16* sSl = sSh + p.n16 * kLdX;                               // [n16][kLdX]
-  float* sDt = reinterpret_cast<float*>(sSl + p.n16 * kLdX);             // [64]
+  __nv_bfloat16* sA = sSl + p.n16 * kLdX;                                // [2][64][kLdA] (CHANNEL)
+  float* sDt = reinterpret_cast<float*>(sA + (CHANNEL ? 2 * kChunk * kLdA : 0));      // [64]
   float* cum = sDt + kChunk + warp * kChunk;                             // [4 warps][64]
   float* wgt = sDt + 5 * kChunk + warp * kChunk;                         // [4 warps][64]
+  float* sLd = sDt + 9 * kChunk;                                         // [64] (MEMORY) or the block's decays [n16] (CHANNEL)
+  float* sN = sLd + kChunk;                                              // [n16] (MEMORY)
 
   const long long q0 = p.q_start[seq];
   const int start = p.seq_lens[seq] - len;
   const int g = h / (d.H / d.G);
-  const int cx = h * d.P + p0, cb = d.b0 + g * d.N, cc = d.c0 + g * d.N;
+  const int cx = h * d.P + p0, cb = d.b0 + g * d.NB, cc = d.c0 + g * d.NB;
   const int pw = min(kSlice, d.P - p0);
-  const float a2 = ssd_rate(p, h), skip = p.dskip ? p.dskip[h] : 0.f;
+  const float a2 = KIND == kSsdPlain ? ssd_rate(p, h) : 0.f, skip = p.dskip ? p.dskip[h] : 0.f;
+  const bool norm = MEMORY && p0 == 0;                                   // this CTA keeps the head's normaliser
   const long long mat = static_cast<long long>(d.N) * d.P4;
   float* st = p.state + (static_cast<long long>(p.slots[seq]) * d.H + h) * mat + p0;
 
   auto load_chunk = [&](int ch) {
     const int t0 = ch * kChunk;
-    ssd_load_rows(p, sC, ldn, p.n16, d.N, cc, q0, t0, len);
-    ssd_load_rows(p, sB, ldn, p.n16, d.N, cb, q0, t0, len);
+    ssd_load_rows(p.act, p.ld, p.aligned, sC, ldn, p.n16, d.N, cc, q0, t0, len);
+    ssd_load_rows(p.act, p.ld, p.aligned, sB, ldn, p.n16, d.N, cb, q0, t0, len);
     if (SPLIT) {
-      ssd_load_rows(p, sCl, ldn, p.n16, d.N, cc + d.lo, q0, t0, len);
-      ssd_load_rows(p, sBl, ldn, p.n16, d.N, cb + d.lo, q0, t0, len);
+      ssd_load_rows(p.act, p.ld, p.aligned, sCl, ldn, p.n16, d.N, cc + d.lo, q0, t0, len);
+      ssd_load_rows(p.act, p.ld, p.aligned, sBl, ldn, p.n16, d.N, cb + d.lo, q0, t0, len);
     }
-    ssd_load_rows(p, sX, kLdX, kSlice, pw, cx, q0, t0, len);
-    if (threadIdx.x < kChunk)
-      sDt[threadIdx.x] = t0 + static_cast<int>(threadIdx.x) < len ? (p.dt ? p.dt[(q0 + t0 + threadIdx.x) * d.H + h] : 1.f) : 0.f;
+    ssd_load_rows(p.x, p.ldx, p.aligned_x, sX, kLdX, kSlice, pw, cx, q0, t0, len);
+    if (CHANNEL) {
+      ssd_load_rows(p.score, 2ll * kChunk * d.H, true, sA, kLdA, kChunk, kChunk, h * 2 * kChunk, q0, t0, len);
+      ssd_load_rows(p.score, 2ll * kChunk * d.H, true, sA + kChunk * kLdA, kLdA, kChunk, kChunk, (h * 2 + 1) * kChunk, q0, t0, len);
+      const long long block = p.c_start[seq] / kChunk + seq + ch;
+      for (int n = threadIdx.x; n < p.n16; n += 128) sLd[n] = p.block_decay[(block * d.H + h) * d.NB + n];
+    } else if (threadIdx.x < kChunk) {
+      const bool ok = t0 + static_cast<int>(threadIdx.x) < len;
+      sDt[threadIdx.x] = ok ? (p.dt ? p.dt[(q0 + t0 + threadIdx.x) * d.H + h] : 1.f) : 0.f;
+      if (MEMORY) sLd[threadIdx.x] = ok ? p.ldec[(q0 + t0 + threadIdx.x) * d.H + h] : 0.f;
+    }
     ms_commit();
   };
   load_chunk(ch0);
@@ -259,17 +334,31 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
         v0 = v.x;
         v1 = v.y;
       });
+    if (norm)
+      for (int n = threadIdx.x; n < p.n16; n += 128)
+        sN[n] = start > 0 && n < d.N ? p.nstate[(static_cast<long long>(p.slots[seq]) * d.H + h) * d.N + n] : 0.f;
   } else {
+    float nv[2] = {0.f, 0.f};
     for (int k = 0; k <= seg; ++k) {
       const long long o = (static_cast<long long>(seq) * p.n_seg + k) * d.H + h;
       const float* src = p.seg_state + o * mat + p0;
-      const float keep = k > 0 ? p.seg_decay[o - d.H] : 0.f;
+      const float keep = k > 0 && !CHANNEL ? p.seg_decay[o - d.H] : 0.f;
+      const float* keeps = p.seg_decay + (o - d.H) * d.N;              // CHANNEL, k > 0
       ssd_each<NI>(S, d.N, pw, warp, lane, [&](float& v0, float& v1, int n, int c) {
         const float2 v = *reinterpret_cast<const float2*>(src + static_cast<long long>(n) * d.P4 + c);
-        v0 = fmaf(keep, v0, v.x);
-        v1 = fmaf(keep, v1, v.y);
+        const float f = CHANNEL ? (k > 0 ? keeps[n] : 0.f) : keep;
+        v0 = fmaf(f, v0, v.x);
+        v1 = fmaf(f, v1, v.y);
       });
+      if (norm)
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+          if (static_cast<int>(threadIdx.x) + 128 * i < d.N) nv[i] = fmaf(keep, nv[i], p.seg_n[o * d.N + threadIdx.x + 128 * i]);
     }
+    if (norm)
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        if (static_cast<int>(threadIdx.x) + 128 * i < p.n16) sN[threadIdx.x + 128 * i] = nv[i];
   }
   auto publish = [&]() {
 #pragma unroll
@@ -296,8 +385,9 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
   for (int ch = ch0; ch < ch1; ++ch) {
     ms_wait<0>();
     __syncthreads();                       // the block's rows and the published state are visible
-    const float total = ssd_decays(sDt, a2, cum, wgt, lane);
-    float s[8][4], yi[4][4], y[4][4];
+    float total = 0.f;
+    if (!CHANNEL) total = ssd_decays(sDt, MEMORY ? sLd : nullptr, a2, cum, wgt, lane);
+    float s[8][4], yi[4][4], y[4][4], rows[2] = {0.f, 0.f};
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
@@ -313,7 +403,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
       if (SPLIT) ms_ldsm4(ms_a_at(aCl, ldn, r0, k, lane), fal);
 #pragma unroll
       for (int np = 0; np < 4; ++np) {
-        if (np <= warp) {
+        if (!CHANNEL && np <= warp) {
           uint32_t fb[4];
           ms_ldsm4(ms_b_nt_at(aB, ldn, np * 16, k, lane), fb);
           ms_mma(s[2 * np], fa, fb[0], fb[1]);
@@ -342,26 +432,38 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
         }
       }
     }
-    const float ci[2] = {cum[r0 + g4], cum[r0 + g4 + 8]};
+    float ci[2] = {0.f, 0.f};
+    if (!CHANNEL) {
+      ci[0] = cum[r0 + g4];
+      ci[1] = cum[r0 + g4 + 8];
+    }
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
       if (kk > warp) break;
+      uint32_t fh[4], fl[4];
+      if (CHANNEL) {
+        ms_ldsm4(ms_a_at(ms_addr(sA), kLdA, r0, kk * 16, lane), fh);
+        ms_ldsm4(ms_a_at(ms_addr(sA + kChunk * kLdA), kLdA, r0, kk * 16, lane), fl);
+      }
       float m[2][4];
 #pragma unroll
       for (int q = 0; q < 2; ++q) {
+        if (CHANNEL) break;
         const int j0 = kk * 16 + q * 8 + 2 * t4;
         const float2 cj = *reinterpret_cast<const float2*>(cum + j0), dj = *reinterpret_cast<const float2*>(sDt + j0);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const bool seen = kk < warp || j0 + (e & 1) <= r0 + g4 + ((e & 2) ? 8 : 0);
           m[q][e] = seen ? s[2 * kk + q][e] * exp2f(ci[e >> 1] - ((e & 1) ? cj.y : cj.x)) * ((e & 1) ? dj.y : dj.x) : 0.f;
+          if (MEMORY) rows[e >> 1] += m[q][e];
         }
       }
-      uint32_t fh[4], fl[4];
-      ms_split(m[0][0], m[0][1], fh[0], fl[0]);
-      ms_split(m[0][2], m[0][3], fh[1], fl[1]);
-      ms_split(m[1][0], m[1][1], fh[2], fl[2]);
-      ms_split(m[1][2], m[1][3], fh[3], fl[3]);
+      if (!CHANNEL) {
+        ms_split(m[0][0], m[0][1], fh[0], fl[0]);
+        ms_split(m[0][2], m[0][3], fh[1], fl[1]);
+        ms_split(m[1][0], m[1][1], fh[2], fl[2]);
+        ms_split(m[1][2], m[1][3], fh[3], fl[3]);
+      }
 #pragma unroll
       for (int np = 0; np < 2; ++np) {
         uint32_t fx[4];
@@ -375,6 +477,28 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
     // y of this warp's 16 tokens
     const float ei[2] = {exp2f(ci[0]), exp2f(ci[1])};
     const int t0 = ch * kChunk;
+    if (norm) {                            // n . c of the rows: the block's part from the scores, the rest from the normaliser at its start
+      float own = 0.f;
+      const int per = p.n16 / 2, from = (lane >> 4) * per;
+      for (int k = from; k < from + per; k += 8) {
+        float v[8];
+        load_vec<8>(sC + (r0 + (lane & 15)) * ldn + k, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) own = fmaf(v[e], sN[k + e], own);
+      }
+      own += __shfl_xor_sync(0xffffffffu, own, 16);
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf) {
+        rows[hf] += __shfl_xor_sync(0xffffffffu, rows[hf], 1);
+        rows[hf] += __shfl_xor_sync(0xffffffffu, rows[hf], 2);
+        const float nq = fmaf(ei[hf], __shfl_sync(0xffffffffu, own, g4 + 8 * hf), rows[hf]) * p.yscale;
+        const int i = r0 + g4 + 8 * hf;
+        if (t4 == 0 && t0 + i < len) {
+          const long long at = (q0 + t0 + i) * d.H + h;
+          p.den[at] = fmaxf(fabsf(nq), expf(-p.mrun[at])) + p.den_eps;
+        }
+      }
+    }
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
@@ -382,57 +506,92 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
         const int i = r0 + g4 + 8 * hf, c = nt * 8 + 2 * t4;
         if (t0 + i >= len || c >= pw) continue;
         const float2 xf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + i * kLdX + c));
-        const float v0 = fmaf(skip, xf.x, fmaf(ei[hf], yi[nt][2 * hf], y[nt][2 * hf]));
-        const float v1 = fmaf(skip, xf.y, fmaf(ei[hf], yi[nt][2 * hf + 1], y[nt][2 * hf + 1]));
+        float v0 = fmaf(skip, xf.x, fmaf(ei[hf], yi[nt][2 * hf], y[nt][2 * hf]));
+        float v1 = fmaf(skip, xf.y, fmaf(ei[hf], yi[nt][2 * hf + 1], y[nt][2 * hf + 1]));
+        if (MEMORY) {
+          v0 *= p.yscale;
+          v1 *= p.yscale;
+        }
         __nv_bfloat16* dst = p.y + (q0 + t0 + i) * (d.H * d.P) + cx + c;
-        if (p.aligned) {
+        if (d.P % 2 == 0) {
           *reinterpret_cast<uint32_t*>(dst) = pack_bf16(v0, v1);
         } else {
           dst[0] = __float2bfloat16(v0);
           if (c + 1 < pw) dst[1] = __float2bfloat16(v1);
         }
       }
-    if (ch + 1 < ch1 || ch1 == n_chunks)
-      ssd_update<NI, SPLIT>(S, exp2f(total), wgt, aB, aBl, aX, ldn, p.n16, warp, lane);
+    float nv[2] = {0.f, 0.f};
+    if (ch + 1 < ch1 || ch1 == n_chunks) {
+      ssd_update<NI, SPLIT, CHANNEL>(S, exp2f(total), sLd, wgt, aB, aBl, aX, ldn, p.n16, warp, lane);
+      if (norm) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+          if (static_cast<int>(threadIdx.x) + 128 * i < d.N) nv[i] = sN[threadIdx.x + 128 * i];
+        ssd_norm_add(nv, exp2f(total), wgt, sB, ldn, d.N);
+      }
+    }
     __syncthreads();                       // everyone has read this block's rows and the published state
+    if (norm && (ch + 1 < ch1 || ch1 == n_chunks))
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        if (static_cast<int>(threadIdx.x) + 128 * i < d.N) sN[threadIdx.x + 128 * i] = nv[i];
     if (ch + 1 < ch1) {
       load_chunk(ch + 1);
       publish();
     }
   }
-  if (ch1 == n_chunks)
+  if (ch1 == n_chunks) {
     ssd_each<NI>(S, d.N, pw, warp, lane, [&](float& v0, float& v1, int n, int c) {
       *reinterpret_cast<float2*>(st + static_cast<long long>(n) * d.P4 + c) = make_float2(v0, v1);
     });
+    if (norm)                              // every thread reads what it wrote
+      for (int n = threadIdx.x; n < d.N; n += 128) p.nstate[(static_cast<long long>(p.slots[seq]) * d.H + h) * d.N + n] = sN[n];
+  }
 }
 
-template <int NI, bool SPLIT>
+template <int NI, bool SPLIT, int KIND>
 static int ssd_launch_as(const SsdParams& p, dim3 grid, cudaStream_t st) {
   const size_t tile_n = static_cast<size_t>(kChunk) * (p.n16 + 8), tile_x = static_cast<size_t>(kChunk) * kLdX;
-  const size_t smem = ((SPLIT ? 4 : 2) * tile_n + tile_x + 2 * static_cast<size_t>(p.n16) * kLdX) * 2 + 9 * kChunk * 4;
-  const size_t smem_seg = ((SPLIT ? 4 : 2) * tile_n + 2 * tile_x) * 2 + 10 * kChunk * 4;
+  const size_t scores = KIND == kSsdChannel ? 2 * static_cast<size_t>(kChunk) * kLdA : 0;
+  const size_t more = KIND == kSsdPlain ? 0 : (KIND == kSsdMemory ? kChunk + p.n16 : p.n16), more_seg = KIND == kSsdPlain ? 0 : 2 * (KIND == kSsdMemory ? kChunk : p.n16);
+  const size_t smem = ((SPLIT ? 4 : 2) * tile_n + tile_x + 2 * static_cast<size_t>(p.n16) * kLdX + scores) * 2 + (9 * kChunk + more) * 4;
+  const size_t smem_seg = ((SPLIT ? 4 : 2) * tile_n + 2 * tile_x) * 2 + (10 * kChunk + more_seg) * 4;
+  if (smem > 224 * 1024 || smem_seg > 224 * 1024) return -4;
   static DeviceOnce once;
   if (once.pending()) {
-    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NI, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NI, SPLIT, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(ssd_segment_kernel<NI, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+      e = cudaFuncSetAttribute(ssd_segment_kernel<NI, SPLIT, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
     if (e != cudaSuccess) return static_cast<int>(e);
     once.mark();
   }
   if (p.n_seg > 1) {
-    ssd_segment_kernel<NI, SPLIT><<<grid, 128, smem_seg, st>>>(p);
+    ssd_segment_kernel<NI, SPLIT, KIND><<<grid, 128, smem_seg, st>>>(p);
     const cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  ssd_chunk_kernel<NI, SPLIT><<<grid, 128, smem, st>>>(p);
+  ssd_chunk_kernel<NI, SPLIT, KIND><<<grid, 128, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <bool SPLIT, int KIND>
+static int ssd_launch_any(const SsdParams& p, dim3 grid, cudaStream_t st) {
+  return p.n16 <= 64 ? ssd_launch_as<1, SPLIT, KIND>(p, grid, st)
+                     : (p.n16 <= 128 ? ssd_launch_as<2, SPLIT, KIND>(p, grid, st) : ssd_launch_as<4, SPLIT, KIND>(p, grid, st));
 }
 
 int ssd_chunk_launch(SsdParams p, int n_seq, int max_q, int max_seg, cudaStream_t st) {
   if (p.N < 1 || p.N > kSsdMaxState || max_seg < 1) return -1;
   if (n_seq < 1 || max_q < 1) return 0;
   p.n16 = (p.N + 15) / 16 * 16;
-  p.aligned = p.ld % 8 == 0 && p.b0 % 8 == 0 && p.c0 % 8 == 0 && p.lo % 8 == 0 && p.N % 8 == 0 && p.P % 8 == 0;
+  if (!p.x) {
+    p.x = p.act;
+    p.ldx = p.ld;
+  }
+  if (!p.NB) p.NB = p.N;
+  const auto whole = [](const void* a) { return reinterpret_cast<uintptr_t>(a) % 16 == 0; };
+  p.aligned = p.ld % 8 == 0 && p.b0 % 8 == 0 && p.c0 % 8 == 0 && p.lo % 8 == 0 && p.N % 8 == 0 && p.NB % 8 == 0 && whole(p.act);
+  p.aligned_x = p.ldx % 8 == 0 && p.P % 8 == 0 && whole(p.x);
   // enough CTAs to keep three on every SM for a few rounds
   const int slices = (p.P + kSlice - 1) / kSlice, n_chunks = (max_q + kChunk - 1) / kChunk;
   const long long base = static_cast<long long>(slices) * p.H * n_seq;
@@ -442,11 +601,9 @@ int ssd_chunk_launch(SsdParams p, int n_seq, int max_q, int max_seg, cudaStream_
   p.seg_chunks = (n_chunks + static_cast<int>(want) - 1) / static_cast<int>(want);
   p.n_seg = (n_chunks + p.seg_chunks - 1) / p.seg_chunks;
   const dim3 grid(slices * p.n_seg, p.H, n_seq);
-  if (p.lo > 0)
-    return p.n16 <= 64 ? ssd_launch_as<1, true>(p, grid, st)
-                       : (p.n16 <= 128 ? ssd_launch_as<2, true>(p, grid, st) : ssd_launch_as<4, true>(p, grid, st));
-  return p.n16 <= 64 ? ssd_launch_as<1, false>(p, grid, st)
-                     : (p.n16 <= 128 ? ssd_launch_as<2, false>(p, grid, st) : ssd_launch_as<4, false>(p, grid, st));
+  if (p.kind == kSsdMemory) return ssd_launch_any<false, kSsdMemory>(p, grid, st);
+  if (p.kind == kSsdChannel) return ssd_launch_any<true, kSsdChannel>(p, grid, st);
+  return p.lo > 0 ? ssd_launch_any<true, kSsdPlain>(p, grid, st) : ssd_launch_any<false, kSsdPlain>(p, grid, st);
 }
 
 }  // namespace pm

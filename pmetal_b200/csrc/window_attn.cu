@@ -1,6 +1,8 @@
 // Grouped-query attention over a paged cache for heads of any size: position i sees the keys j with 0 <= i - j < window (every
-// j <= i when window is 0). Key and value sizes may differ, a head may have several attention maps over the same values, scores
-// may be capped (cap tanh(s / cap)), and the softmax may have a sink per head (a score without a value). Per token and layer the
+// j <= i when window is 0) or, chunked, those of its own chunk (j <= i, the same j / window). Key and value sizes may differ, a head
+// may have several attention maps over the same values, scores may be capped (cap tanh(s / cap)), and the softmax may have a sink
+// per head (a score without a value). Instead of a softmax the weights may be sigmoids of score + a number per head, which nothing
+// is divided by. Per token and layer the
 // cache holds one row [head 0: k of map 0 | .. | v, head 1: ..] with D8 channels per key and DV8 per value (the sizes D and DV
 // rounded up to 8, zeros behind them).
 //
@@ -202,6 +204,9 @@ struct WindowParams {
   long long ldg;
   int n_tok, max_blocks, H, G, rep, M, KM, D, D8, DV, DV8, QP, QM, window, n_split;      // KM: maps of a CTA, 1 or M
   float scale, softcap;      // softcap 0: none
+  int chunked;               // window is the size of chunks counted from position 0
+  const float* wbias;        // [H], nullable: sigmoid weights, added to the scores
+  float out_scale;           // factor of the result
 };
 
 constexpr float kLog2e = 1.4426950408889634f;
@@ -213,7 +218,10 @@ __device__ __forceinline__ float window_tanh(float x) {
 }
 
 // First visible key of the query at position pos.
-__device__ __forceinline__ int window_first(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
+__device__ __forceinline__ int window_first(int pos, int window, int chunked) {
+  if (chunked) return pos - pos % window;
+  return window > 0 ? max(0, pos - window + 1) : 0;
+}
 
 // KK: 16-channel steps of a key row, 0: counted at run time. KD: 16-channel steps of the values. KEYW: warps that share 16 rows
 // and split the keys of a page (1 or 4).
@@ -234,7 +242,7 @@ __global__ void __launch_bounds__(128) window_mma_kernel(const WindowParams<__nv
   const int q0 = p.q_start[seq], base = p.seq_lens[seq] - len;           // position of the first new token
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int p_lo = base + r0 / rpt, p_hi = base + (r0 + n_rows - 1) / rpt;      // positions of the first and last row
-  const int b_all = window_first(p_lo, p.window) / kWinPage, n_all = p_hi / kWinPage + 1 - b_all;
+  const int b_all = window_first(p_lo, p.window, p.chunked) / kWinPage, n_all = p_hi / kWinPage + 1 - b_all;
   const int per = (n_all + p.n_split - 1) / p.n_split;
   const int b0 = b_all + split * per, b1 = min(b0 + per, b_all + n_all);
 
@@ -271,14 +279,21 @@ __global__ void __launch_bounds__(128) window_mma_kernel(const WindowParams<__nv
   for (int hf = 0; hf < 2; ++hf) {
     const int r = wr + g4 + 8 * hf;
     pos[hf] = r < n_rows ? base + (r0 + r) / rpt : -1;                 // rows that do not exist see nothing
-    first[hf] = window_first(pos[hf], p.window);
+    first[hf] = window_first(pos[hf], p.window, p.chunked);
   }
   float o[2 * KD][4], m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
 #pragma unroll
   for (int i = 0; i < 2 * KD; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
-  const bool capped = p.softcap > 0.f;
+  const bool capped = p.softcap > 0.f, plain = p.wbias != nullptr;       // plain: sigmoid weights, m stays 0
+  float wb2[2] = {0.f, 0.f};
+  if (plain) {
+    m[0] = m[1] = 0.f;
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf)
+      if (wr + g4 + 8 * hf < n_rows) wb2[hf] = p.wbias[g * p.rep + (r0 + wr + g4 + 8 * hf) % rpt / p.KM] * kLog2e;
+  }
   const float a2 = capped ? p.scale / p.softcap : p.scale * kLog2e, cap2 = p.softcap * kLog2e;
   const uint32_t aQ = ms_addr(sQ);
   const bool idle = wr >= n_rows;
@@ -309,9 +324,18 @@ __global__ void __launch_bounds__(128) window_mma_kernel(const WindowParams<__nv
         }
       }
       const int j0 = b * kWinPage + wk + 2 * t4;
-      const bool whole = b * kWinPage + kWinPage - 1 <= p_lo && b * kWinPage >= window_first(p_hi, p.window) && n_rows == kRows;
+      const bool whole = b * kWinPage + kWinPage - 1 <= p_lo && b * kWinPage >= window_first(p_hi, p.window, p.chunked) && n_rows == kRows;
       float mx[2] = {m[0], m[1]};
-      if (capped) {
+      if (plain) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int hf = e >> 1, j = j0 + n * 8 + (e & 1);
+            const float w = __fdividef(1.f, 1.f + exp2f(-fmaf(s[n][e], a2, wb2[hf])));
+            s[n][e] = !whole && (j > pos[hf] || j < first[hf]) ? 0.f : w;
+          }
+      } else if (capped) {
 #pragma unroll
         for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -322,28 +346,30 @@ __global__ void __launch_bounds__(128) window_mma_kernel(const WindowParams<__nv
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[n][e] *= a2;
       }
+      float keep[2], at[2] = {0.f, 0.f};
+      if (!plain) {
 #pragma unroll
-      for (int n = 0; n < NT; ++n)
+        for (int n = 0; n < NT; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int hf = e >> 1, j = j0 + n * 8 + (e & 1);
-          if (!whole && (j > pos[hf] || j < first[hf])) s[n][e] = -CUDART_INF_F;
-          mx[hf] = fmaxf(mx[hf], s[n][e]);
+          for (int e = 0; e < 4; ++e) {
+            const int hf = e >> 1, j = j0 + n * 8 + (e & 1);
+            if (!whole && (j > pos[hf] || j < first[hf])) s[n][e] = -CUDART_INF_F;
+            mx[hf] = fmaxf(mx[hf], s[n][e]);
+          }
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+          mx[hf] = fmaxf(mx[hf], __shfl_xor_sync(0xffffffffu, mx[hf], 1));
+          mx[hf] = fmaxf(mx[hf], __shfl_xor_sync(0xffffffffu, mx[hf], 2));
+          at[hf] = mx[hf] == -CUDART_INF_F ? 0.f : mx[hf];
+          keep[hf] = exp2f(m[hf] - at[hf]);
+          m[hf] = mx[hf];
+          l[hf] *= keep[hf];
         }
-      float keep[2], at[2];
 #pragma unroll
-      for (int hf = 0; hf < 2; ++hf) {
-        mx[hf] = fmaxf(mx[hf], __shfl_xor_sync(0xffffffffu, mx[hf], 1));
-        mx[hf] = fmaxf(mx[hf], __shfl_xor_sync(0xffffffffu, mx[hf], 2));
-        at[hf] = mx[hf] == -CUDART_INF_F ? 0.f : mx[hf];
-        keep[hf] = exp2f(m[hf] - at[hf]);
-        m[hf] = mx[hf];
-        l[hf] *= keep[hf];
-      }
-#pragma unroll
-      for (int i = 0; i < 2 * KD; ++i) {
-        o[i][0] *= keep[0]; o[i][1] *= keep[0];
-        o[i][2] *= keep[1]; o[i][3] *= keep[1];
+        for (int i = 0; i < 2 * KD; ++i) {
+          o[i][0] *= keep[0]; o[i][1] *= keep[0];
+          o[i][2] *= keep[1]; o[i][3] *= keep[1];
+        }
       }
 #pragma unroll
       for (int n = 0; n < NT / 2; ++n) {
@@ -352,7 +378,11 @@ __global__ void __launch_bounds__(128) window_mma_kernel(const WindowParams<__nv
         for (int q = 0; q < 2; ++q)
 #pragma unroll
           for (int hf = 0; hf < 2; ++hf) {
-            const float e0 = exp2f(s[2 * n + q][2 * hf] - at[hf]), e1 = exp2f(s[2 * n + q][2 * hf + 1] - at[hf]);
+            float e0 = s[2 * n + q][2 * hf], e1 = s[2 * n + q][2 * hf + 1];
+            if (!plain) {
+              e0 = exp2f(e0 - at[hf]);
+              e1 = exp2f(e1 - at[hf]);
+            }
             l[hf] += e0 + e1;
             fp[2 * q + hf] = pack_bf16(e0, e1);
           }
@@ -441,7 +471,8 @@ __global__ void __launch_bounds__(128) window_mma_kernel(const WindowParams<__nv
       f = exp2f(m[hf] - mm);
       ll = fmaf(ll, f, exp2f(s2 - mm));
     }
-    float inv = ll > 0.f ? f / ll : 0.f;
+    float inv = plain ? 1.f : (ll > 0.f ? f / ll : 0.f);
+    inv *= p.out_scale;
     if (p.gate) inv *= sigmoid_fast(to_f(p.gate[t * p.ldg + h]));
     __nv_bfloat16* dst = p.out + t * p.ldo + static_cast<long long>(hm) * p.DV;
     const bool even = (p.DV | static_cast<int>(p.ldo)) % 2 == 0;
@@ -474,6 +505,8 @@ struct WindowFinishParams {
   const float* lambda;       // M = 2: one number
   float keep, eps;           // M = 2: factor behind the norm
   int n_tok, H, M, DV, DV8, OP, n_split;
+  int plain;                 // parts are added up as they are
+  float out_scale;
 };
 
 // One warp per (token, head) of the sequences in q_start / q_lens, NC * 32 channels. grid (tokens of the longest portion,
@@ -501,8 +534,11 @@ __global__ void __launch_bounds__(128) window_finish_kernel(const WindowFinishPa
     float m = fmaxf(ms, s2);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-    float f = exp2f(ms - m);
-    f *= w / (warp_sum(ls * f) + exp2f(s2 - m));
+    float f = 1.f;
+    if (!p.plain) {
+      f = exp2f(ms - m);
+      f *= w / (warp_sum(ls * f) + exp2f(s2 - m));
+    }
 #pragma unroll 8
     for (int s = 0; s < p.n_split; ++s) {
       const float fs = __shfl_sync(0xffffffffu, f, s);
@@ -512,12 +548,12 @@ __global__ void __launch_bounds__(128) window_finish_kernel(const WindowFinishPa
         if (lane + 32 * i < p.DV) v[i] = fmaf(src[32 * i], fs, v[i]);
     }
   }
-  float f = 1.f;
+  float f = p.out_scale;
   if (p.M > 1) {
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NC; ++i) ss = fmaf(v[i], v[i], ss);
-    f = p.keep / sqrtf(warp_sum(ss) / static_cast<float>(p.DV) + p.eps);
+    f *= p.keep / sqrtf(warp_sum(ss) / static_cast<float>(p.DV) + p.eps);
   }
   if (p.gate) f *= sigmoid_f(to_f(p.gate[t * p.ldg + h]));
 #pragma unroll
@@ -536,13 +572,15 @@ __global__ void __launch_bounds__(128) window_row_kernel(const WindowParams<T> p
   const int* table = p.block_table + static_cast<long long>(seq) * p.max_blocks;
   const T* qr = p.q + (t * p.H * p.M + hm) * p.QP + hm % p.M * p.QM;
   const int kv = p.M * p.D8 + p.DV8, k_at = hm % p.M * p.D8, v_at = p.M * p.D8;
-  float q[NC], o[NC], m = -CUDART_INF_F, l = 0.f;
+  const bool plain = p.wbias != nullptr;
+  const float wb = plain ? p.wbias[h] : 0.f;
+  float q[NC], o[NC], m = plain ? 0.f : -CUDART_INF_F, l = 0.f;
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     q[c] = c * 32 + lane < p.D ? to_f(qr[c * 32 + lane]) * p.scale : 0.f;
     o[c] = 0.f;
   }
-  for (int j0 = window_first(pos, p.window) + warp * 4; j0 <= pos; j0 += 16) {
+  for (int j0 = window_first(pos, p.window, p.chunked) + warp * 4; j0 <= pos; j0 += 16) {
     float s[4];
     const T* row[4];
 #pragma unroll
@@ -559,8 +597,9 @@ __global__ void __launch_bounds__(128) window_row_kernel(const WindowParams<T> p
     for (int a = 0; a < 4; ++a) {
       s[a] = warp_sum(s[a]);
       if (p.softcap > 0.f) s[a] = p.softcap * tanhf(s[a] / p.softcap);
-      if (j0 + a > pos) s[a] = -CUDART_INF_F;
-      mx = fmaxf(mx, s[a]);
+      if (plain) s[a] = sigmoid_f(s[a] + wb);
+      if (j0 + a > pos) s[a] = plain ? 0.f : -CUDART_INF_F;
+      if (!plain) mx = fmaxf(mx, s[a]);
     }
     const float keep = expf(m - mx);
     m = mx;
@@ -569,7 +608,7 @@ __global__ void __launch_bounds__(128) window_row_kernel(const WindowParams<T> p
     for (int c = 0; c < NC; ++c) o[c] *= keep;
 #pragma unroll
     for (int a = 0; a < 4; ++a) {
-      const float w = expf(s[a] - m);
+      const float w = plain ? s[a] : expf(s[a] - m);
       l += w;
 #pragma unroll
       for (int c = 0; c < NC; ++c)
@@ -583,7 +622,8 @@ __global__ void __launch_bounds__(128) window_row_kernel(const WindowParams<T> p
   if (p.sink) mm = fmaxf(mm, p.sink[h]);
   float ll = p.sink ? expf(p.sink[h] - mm) : 0.f;
   for (int w = 0; w < 4; ++w) ll = fmaf(sl[w], expf(sm[w] - mm), ll);
-  const float f = expf(m - mm), gate = p.gate ? sigmoid_f(to_f(p.gate[t * p.ldg + h])) : 1.f;
+  if (plain) ll = 1.f;
+  const float f = expf(m - mm), gate = (p.gate ? sigmoid_f(to_f(p.gate[t * p.ldg + h])) : 1.f) * p.out_scale;
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     __syncthreads();
@@ -708,13 +748,14 @@ static int window_attn_launch(WindowParams<T> p, int n_seq, int max_q, int few, 
                               cudaStream_t st) {
   constexpr bool low = sizeof(T) == 2;
   WindowFinishParams<T> f{p.po, p.pml, nullptr, p.out, p.ldo, p.q_start, p.q_lens, p.sink, p.gate, p.ldg, lambda, keep, eps,
-                          p.n_tok, p.H, p.M, p.DV, p.DV8, p.DV, p.n_split};
+                          p.n_tok, p.H, p.M, p.DV, p.DV8, p.DV, p.n_split, p.wbias != nullptr, p.out_scale};
   if (!p.po && p.M > 1) {                 // results of the maps, then their difference
     if (!o) return -3;
     f.o = static_cast<const T*>(o);
     p.out = static_cast<T*>(o);
     p.ldo = static_cast<long long>(p.H) * p.M * p.DV;
     p.gate = nullptr;
+    p.out_scale = 1.f;
   }
   int rc;
   if constexpr (low) {
@@ -769,14 +810,16 @@ extern "C" int pm_window_prep(const void* u, int f32, long long ldu, const float
 // softcap > 0; sink (fp32 [H], M = 1) adds exp(sink) to a head's softmax sum; gate [.., ldg] multiplies head h by the sigmoid of
 // column h. M = 2: the result of a head is a_1 - lambda[0] a_2 over its root mean square (eps inside), times keep; it takes o
 // [n_tok, H M, DV] in the compute type unless parts are given. few 1: decode tiles (a few rows per sequence), which take work
-// buffers po [n_split][n_tok][H M][DV8] and pml [n_split][n_tok][H M][2] (both or none; needed for n_split > 1).
+// buffers po [n_split][n_tok][H M][DV8] and pml [n_split][n_tok][H M][2] (both or none; needed for n_split > 1). chunked 1: a position
+// sees the keys of its own chunk of `window` positions. wbias (fp32 [H], nullable, M = 1, without sink): the weight of a key is the
+// sigmoid of its score + wbias, not divided by their sum. out_scale multiplies the result.
 extern "C" int pm_window_attn(const void* q, int f32, const void* pages, const int* block_table, const int* seq_lens,
                               const int* q_start, const int* q_lens, int n_seq, int max_blocks, int n_tok, int max_q, int H,
                               int G, int M, int D, int DV, int wide, int window, float scale, float softcap, const float* sink, const void* gate,
                               long long ldg, const float* lambda, float keep, float eps, int few, int n_split, float* po, float* pml,
-                              void* o, void* out, long long ldo, cudaStream_t st) {
+                              void* o, void* out, long long ldo, int chunked, const float* wbias, float out_scale, cudaStream_t st) {
   if (window_bad_dims(H, G, M, D, DV) || window < 0 || n_split < 1 || n_split > 32 || (n_split > 1 && (!few || !po)) ||
-      (!po != !pml) || (M > 1 && (!lambda || sink)) || softcap < 0.f)
+      (!po != !pml) || (M > 1 && (!lambda || sink)) || softcap < 0.f || (chunked && window < 1) || (wbias && (M > 1 || sink || softcap > 0.f)))
     return -1;
   if (n_seq < 1 || max_q < 1) return 0;
   if (static_cast<long long>(n_seq) * n_split > 65535) return -2;
@@ -784,12 +827,13 @@ extern "C" int pm_window_attn(const void* q, int f32, const void* pages, const i
   if (f32)
     return window_attn_launch<float>({static_cast<const float*>(q), static_cast<const float*>(pages), static_cast<float*>(out), ldo,
                                       block_table, seq_lens, q_start, q_lens, po, pml, sink, static_cast<const float*>(gate), ldg,
-                                      n_tok, max_blocks, H, G, H / G, M, 1, D, D8, DV, DV8, wide ? wide : D8, wide ? D8 : 0, window, n_split, scale, softcap},
+                                      n_tok, max_blocks, H, G, H / G, M, 1, D, D8, DV, DV8, wide ? wide : D8, wide ? D8 : 0, window, n_split, scale, softcap, chunked, wbias, out_scale},
                                      n_seq, max_q, few, o, lambda, keep, eps, st);
   return window_attn_launch<__nv_bfloat16>({static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(pages),
                                             static_cast<__nv_bfloat16*>(out), ldo, block_table, seq_lens, q_start, q_lens, po, pml,
                                             sink, static_cast<const __nv_bfloat16*>(gate), ldg, n_tok, max_blocks, H, G, H / G, M, 1,
-                                            D, D8, DV, DV8, wide ? wide : D8, wide ? D8 : 0, window, n_split, scale, softcap},
+                                            D, D8, DV, DV8, wide ? wide : D8, wide ? D8 : 0, window, n_split, scale, softcap, chunked,
+                                            wbias, out_scale},
                                            n_seq, max_q, few, o, lambda, keep, eps, st);
 }
 
@@ -815,6 +859,6 @@ extern "C" int pm_window_finish(const void* o, int n_tok, int H, int M, int DV, 
   if (n_seq < 1 || max_q < 1) return 0;
   const WindowFinishParams<__nv_bfloat16> f{nullptr, nullptr, static_cast<const __nv_bfloat16*>(o), static_cast<__nv_bfloat16*>(out),
                                             ldo, q_start, q_lens, nullptr, static_cast<const __nv_bfloat16*>(gate), ldg, lambda, keep,
-                                            eps, n_tok, H, M, DV, (DV + 7) / 8 * 8, OP, 1};
+                                            eps, n_tok, H, M, DV, (DV + 7) / 8 * 8, OP, 1, 0, 1.f};
   return window_finish_launch(f, n_seq, max_q, st);
 }

@@ -3,7 +3,7 @@
 Mirrors the reference's dispatcher (crates/pmetal-models/src/dispatcher.rs:90-160: ``from_model_type`` then
 ``from_architectures``). The families with hand-written kernels (Qwen3, Qwen3-MoE, Llama, Qwen2, Mistral) resolve to
 ``models.decoder.DecoderLM``; the config-driven attention / recurrent stacks that run on the paged state cache (Duvivik,
-Resevik, Vosezen) to ``models.hybrid_decoder.HybridDecoderLM``; every other decoder resolves to the portable ``GenericDecoderLM``; other
+Resevik, Vosezen, Ravapel) to ``models.hybrid_decoder.HybridDecoderLM``; every other decoder resolves to the portable ``GenericDecoderLM``; other
 hybrids, encoders and encoder-decoders have their own classes."""
 from __future__ import annotations
 
@@ -16,7 +16,7 @@ GENERIC_DECODER = {"mixtral", "gemma", "gemma2", "gemma3", "gemma3_text", "phi",
                    "command_r", "command-r", "granite", "granitemoe", "granite_moe", "olmo2", "gpt_oss", "gptoss", "gpt-oss",
                    "llama4", "llama4_text", "deepseek", "deepseek2", "deepseek_v2", "deepseek_v3", "qwen3_next", "qwen3_5",
                    "qwen3.5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text"}
-HYBRID_DECODER = {"duvivik", "resevik", "vosezen"}
+HYBRID_DECODER = {"duvivik", "resevik", "vosezen", "ravapel"}
 PAGED_FAMILIES = ("fast", "hybrid")       # served from the paged caches by the generator and the batching engine
 OTHER = {"nemotron_h": "nemotron_h", "nemotronh": "nemotron_h", "nemotron-h": "nemotron_h", "bert": "bert", "roberta": "bert",
          "distilbert": "bert", "xlm-roberta": "bert", "xlm_roberta": "bert", "t5": "t5", "clip": "clip", "whisper": "whisper",

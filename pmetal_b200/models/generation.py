@@ -355,7 +355,7 @@ class Generator:
                     on_token(i, tok)
                 if tok in stop:
                     reasons[i] = "stop"
-                else:
+                elif not 0 < self.cache.max_length <= self.cache.length(seq_ids[i]):      # a further position exists
                     keep.append(j)
             if counts is not None:
                 counts[alive, ids] += 1
@@ -394,7 +394,7 @@ class Generator:
                 ids = sampler.sample(logits, counts)
                 tok = int(ids[0])
                 yield tok
-                if tok in stop:
+                if tok in stop or 0 < self.cache.max_length <= self.cache.length(sid):
                     break
                 if counts is not None:
                     counts[0, tok] += 1

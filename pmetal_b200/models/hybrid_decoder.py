@@ -1,4 +1,4 @@
-"""Config-driven serving decoder for stacks that mix kinds of attention and recurrent layers (Duvivik, Resevik, Vosezen).
+"""Config-driven serving decoder for stacks that mix kinds of attention and recurrent layers (Duvivik, Resevik, Vosezen, Ravapel).
 
 Each layer has a token mixer (``mixers.MIXERS``) and optionally a feed-forward. The design (``DESIGNS``) says which mixers the
 configuration's layer types mean and how the sublayers meet the stream:
@@ -8,7 +8,11 @@ configuration's layer types mean and how the sublayers meet the stream:
   row with the same weights, every run with a cache or state of its own; each pass but the first starts by adding the
   embedding output to the stream. The sum, the re-added embedding and the next layer's norm are one kernel;
 * ``branch``: both sublayers read the stream itself and only what they add is normed, x <- x + rms(sublayer(x)) (1 + w). The norm
-  and the sum (for experts also the weighted sum of a token's rows) are one kernel.
+  and the sum (for experts also the weighted sum of a token's rows) are one kernel;
+* ``sandwich``: a norm before and one after every sublayer, x <- x + rms(sublayer(rms(x) (1 + w))) (1 + w'); the mixer's input gets a
+  causal convolution over its own last values added. A span of layers may run several times; every pass starts with a projection of
+  the stream beside the embedding output. The embedding adds a row chosen by the pair of the previous and the current token and a row of
+  the position. Norm of the result, sum, norm of the next input and, in decode steps, the convolution are one kernel.
 
 The stream, norms, rotation angles, softmax, routers and recurrent states are fp32; projections and their activations run in
 the model's type (bf16 on the sm_100a kernels, or fp32 throughout with full-precision matrix products).
@@ -32,7 +36,7 @@ from ..ops import functional as ops
 from .kv_cache import BLOCK
 from .mixers import MIXERS, RotationFreqs, StepContext, frozen
 from .moe import WeightedInputExperts, WeightedOutputExperts
-from .state_cache import StateCache
+from .state_cache import CacheSpec, StateCache
 
 GLU_BETA, GLU_SHIFT = 1.702, 1.0          # gate slope and the offset of the up half in the clamped gated unit
 
@@ -40,12 +44,13 @@ GLU_BETA, GLU_SHIFT = 1.702, 1.0          # gate slope and the offset of the up 
 
 @dataclass(frozen=True)
 class Design:
-    block: str                            # "post", "parallel" or "branch"
+    block: str                            # "post", "parallel", "branch" or "sandwich"
     mixers: Dict[str, str]                # "type" of a layer -> name in MIXERS
     feed_forward: str                     # kind of the layers' "mlp" entries
     experts: Optional[type] = None        # class of the feed-forwards of kind "moe"
     tied: bool = False                    # the embedding table is the output projection
-    norm_base: float = 0.0                # norms multiply with norm_base + weight ("branch")
+    norm_base: float = 0.0                # norms multiply with norm_base + weight ("branch", "sandwich")
+    glu: Tuple[float, float] = (GLU_BETA, GLU_SHIFT)      # gate slope and offset of the up half of dense feed-forwards
 
 
 DESIGNS: Dict[str, Design] = {
@@ -54,6 +59,8 @@ DESIGNS: Dict[str, Design] = {
                       WeightedInputExperts),
     "vosezen": Design("branch", {"attention": "difference_attention", "latent_attention": "latent_attention",
                                  "attention_2": "sink_attention"}, "moe", WeightedOutputExperts, tied=True, norm_base=1.0),
+    "ravapel": Design("sandwich", {"hgrn2": "channel_gate", "parallel": "sigmoid_attention_and_memory"}, "dense", norm_base=1.0,
+                      glu=(1.0, 0.0)),
 }
 
 
@@ -67,6 +74,9 @@ class HybridArgs:
     norm_eps: float = 1e-5
     model_type: str = "duvivik"
     loop: Optional[Tuple[int, int, int]] = None      # (first layer, layer behind the last, passes)
+    pair: Optional[Tuple[int, int, int]] = None      # (buckets, factor of the previous id, factor of the id) of the pair embedding
+    taps: int = 0                                    # of the mixers' input convolution
+    max_positions: int = 0                           # rows of the position embedding; 0: sequences of any length
     bos_token_id: Optional[int] = None
     eos_token_id: Optional[int] = None
     raw: dict = field(default_factory=dict, repr=False)
@@ -81,12 +91,14 @@ class HybridArgs:
 
     @property
     def runs(self) -> List[Tuple[int, bool]]:
-        """Layers in the order of execution: (layer, whether a further pass of the loop starts with it)."""
+        """Layers in the order of execution: (layer, whether a further pass of the loop starts with it; in "sandwich" stacks, whether
+        any pass does)."""
         n = len(self.layers)
         a, b, times = self.loop or (0, 0, 0)
+        first = 0 if self.design.block == "sandwich" else 1
         order = [(i, False) for i in range(a)]
         for t in range(times):
-            order += [(i, t > 0 and i == a) for i in range(a, b)]
+            order += [(i, t >= first and i == a) for i in range(a, b)]
         return order + [(i, False) for i in range(b, n)]
 
     @classmethod
@@ -112,14 +124,25 @@ class HybridArgs:
         loop = d.get("loop")
         if loop is not None:
             loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
-            if design.block != "parallel" or not 0 <= loop[0] < loop[1] <= len(layers) or loop[2] < 1:
+            if design.block not in ("parallel", "sandwich") or not 0 <= loop[0] < loop[1] <= len(layers) or loop[2] < 1:
                 raise ValueError(f"loop {loop} over {len(layers)} layers")
         eos = d.get("eos_token_id")
+        more = {}
+        if design.block == "sandwich":
+            e = d["embedding"]["bigram"]
+            more = {"pair": (int(e["buckets"]), int(e["mul_prev"]), int(e["mul_cur"])), "taps": int(d["canon"]["taps"]),
+                    "max_positions": int(d["max_positions"])}
+            if more["pair"][0] < 1 or min(more["pair"]) < 0:
+                raise ValueError(f"pair embedding with {e}")
+            if not 1 <= more["taps"] <= 17:
+                raise ValueError(f"input convolution of {more['taps']} taps (1 to 17 are built)")
+            if more["max_positions"] < 1 or int(d["width"]) > 8192:
+                raise ValueError("max_positions must be positive, width at most 8192")
         return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
                    embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
                    residual_alpha=float(d.get("postln_alpha", 1.0)), norm_eps=float(d["norm"]["eps"]), model_type=name, loop=loop,
                    bos_token_id=d.get("bos_token_id"), eos_token_id=eos[0] if isinstance(eos, list) else eos,
-                   raw=copy.deepcopy(d))
+                   raw=copy.deepcopy(d), **more)
 
     @classmethod
     def from_pretrained(cls, model_dir: str) -> "HybridArgs":
@@ -184,6 +207,25 @@ def _branch_stack(width: int, vocab: int, ff: int, shared: int, experts: int, id
     return {"architecture": "Vosezen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
 
 
+def _sandwich_stack(width: int, vocab: int, ff: int, gate: dict, left: dict, right: dict, pattern: str, loop: Tuple[int, int, int],
+                    positions: int = 8192) -> dict:
+    """Configuration dict: one letter per layer, G = channel gates, P = attention and matrix memory side by side."""
+    kinds = {"G": ("hgrn2", gate), "P": ("parallel", {"left": left, "right": right, "left_scale": 1.0, "right_scale": 0.8})}
+    return {"architecture": "Ravapel", "vocab": vocab, "width": width, "max_positions": positions, "norm": {"eps": 1e-5},
+            "embedding": {"bigram": {"buckets": 2 * vocab + 1, "mul_prev": 31, "mul_cur": 5}}, "canon": {"taps": 3},
+            "loop": dict(zip(("start", "stop", "times"), loop)),
+            "layers": [{"type": kinds[c][0], "mixer": copy.deepcopy(kinds[c][1]), "mlp": {"kind": "dense", "ff": ff}} for c in pattern]}
+
+
+def _chunked(heads, kv_heads, dim, vdim, size, rot):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": size},
+            "rot": {"base": 10000.0, "dims": rot}}
+
+
+def _memory(heads, dim, vdim, cap=10.0):
+    return {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": cap}
+
+
 def _grouped(heads, kv_heads, dim, vdim, every, **more):
     return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5,
             "q_temp": {"coef": 0.2, "every": every}, **more}
@@ -226,15 +268,24 @@ PRESETS: Dict[str, dict] = {
                                 _grouped(12, 4, 64, 128, 1024, diff=0.3), _grouped(12, 4, 128, 128, 1024, softcap=50.0), "LSDLLSdL" * 2),
     "vosezen-2b": _branch_stack(2048, 65536, 1024, 2048, 16, 4, 2, (4, 2), _q_latent(1024, 16, 96, 32, 128, 512),
                                 _grouped(16, 4, 64, 128, 1024, diff=0.3), _grouped(16, 4, 128, 128, 1024, softcap=50.0), "LSDLLSdL" * 3),
+    "ravapel-tiny": _sandwich_stack(64, 512, 72, _linear(3, 16, 24), _chunked(4, 2, 20, 28, 40, 12), _memory(3, 24, 20), "GPPG", (1, 3, 2)),
+    # 12 layers with the middle six twice (18 layer runs), and 20 layers with eight twice (28 layer runs)
+    "ravapel-1b": _sandwich_stack(2048, 65536, 6144, _linear(16, 128, 128), _chunked(16, 4, 128, 128, 1024, 64), _memory(8, 128, 128),
+                                  "GGP" * 4, (3, 9, 2)),
+    "ravapel-2b": _sandwich_stack(2560, 65536, 8192, _linear(20, 128, 128), _chunked(20, 4, 128, 128, 1024, 64), _memory(10, 128, 128),
+                                  "GPGG" * 5, (4, 12, 2)),
 }
 
 
 class ClampedMLP(nn.Module):
-    """Gated feed-forward with clamped inputs and biases on all projections."""
+    """Gated feed-forward with biases on all projections: g sigmoid(beta g) (u + shift), g and u clamped where the entry has a
+    ``limit``. ``glu`` = (beta, shift)."""
 
-    def __init__(self, m: dict, width: int, dtype, device):
+    def __init__(self, m: dict, width: int, dtype, device, glu: Tuple[float, float] = (GLU_BETA, GLU_SHIFT)):
         super().__init__()
-        self.ff, self.limit, self.width = m["ff"], float(m["limit"]), width
+        limit = m.get("limit")
+        self.ff, self.width = m["ff"], width
+        self.glu = (float("inf") if limit is None else float(limit), *glu)
         up8 = lambda n: -(-n // 8) * 8      # noqa: E731
         self.w_gu = frozen(torch.zeros(up8(2 * self.ff), width, dtype=dtype, device=device))
         self.b_gu = frozen(torch.zeros(2 * self.ff, device=device))
@@ -253,7 +304,7 @@ class ClampedMLP(nn.Module):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         """Without the down-projection's bias, which the caller adds in fp32 with the residual."""
         from ..ops import native as nat
-        glu = (self.limit, GLU_BETA, GLU_SHIFT)
+        glu = self.glu
         if x.dtype == torch.bfloat16 and ops.gemv_fits(*x.shape) and x.stride(0) % 8 == 0:
             a = nat.gemv_ex(x, self.w_gu, self.b_gu, glu, n=self.ff)
         else:
@@ -266,7 +317,7 @@ class HybridLayer(nn.Module):
         super().__init__()
         self.cfg = cfg
         self.mixer = MIXERS[cfg.design.mixers[spec["type"]]](spec["mixer"], cfg, index, dtype, device)
-        self.mlp = ClampedMLP(spec["mlp"], cfg.hidden_size, dtype, device) if spec["mlp"] is not None else None
+        self.mlp = ClampedMLP(spec["mlp"], cfg.hidden_size, dtype, device, cfg.design.glu) if spec["mlp"] is not None else None
         vec = lambda: frozen(torch.zeros(cfg.hidden_size, device=device))      # noqa: E731
         self.norm1_w, self.norm1_b = vec(), vec()
         if self.mlp is not None:
@@ -350,6 +401,37 @@ class BranchLayer(nn.Module):
         return xf, xc
 
 
+class SandwichLayer(nn.Module):
+    """Norms before and after both sublayers and a convolution on the mixer's input; ``HybridDecoderLM._sandwich`` runs it."""
+
+    def __init__(self, spec: dict, cfg: HybridArgs, index: int, dtype, device):
+        super().__init__()
+        self.cfg = cfg
+        self.mixer = MIXERS[cfg.design.mixers[spec["type"]]](spec["mixer"], cfg, index, dtype, device)
+        self.mlp = ClampedMLP(spec["mlp"], cfg.hidden_size, dtype, device, cfg.design.glu) if spec["mlp"] is not None else None
+        vec = lambda: frozen(torch.zeros(cfg.hidden_size, device=device))      # noqa: E731
+        self.norm1_w, self.norm1b_w = vec(), vec()
+        if self.mlp is not None:
+            self.norm2_w, self.norm2b_w = vec(), vec()
+        self.conv_w = frozen(torch.zeros(cfg.taps, cfg.hidden_size, device=device))      # [taps][channel]
+
+    def cache_spec(self):
+        spec = self.mixer.cache_spec()
+        spec.slots["canon"] = ((self.cfg.taps - 1, self.cfg.hidden_size), None)
+        return spec
+
+    def named_weights(self):
+        names = ("norm1", "norm1b") + (("norm2", "norm2b") if self.mlp is not None else ())
+        for name in names:
+            p = getattr(self, name + "_w")
+            yield name, (self.cfg.hidden_size,), p.copy_, (lambda p=p: p)
+        yield "canon1", (self.cfg.hidden_size, self.cfg.taps), lambda t: self.conv_w.copy_(t.t()), lambda: self.conv_w.t()
+        for pre, mod in (("mix.", self.mixer), ("mlp.", self.mlp)):
+            if mod is not None:
+                for name, *rest in mod.named_weights():
+                    yield (pre + name, *rest)
+
+
 class HybridDecoderLM(nn.Module):
     graph_decode = True         # single-token steps can be captured (generation.GraphedDecoder)
     mixed_batches = True        # the scheduler puts prompt portions and decoded tokens into one step
@@ -362,9 +444,15 @@ class HybridDecoderLM(nn.Module):
         self.cfg, self.dtype = cfg, dtype
         self.embed_tokens = frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
         block = cfg.design.block
-        kind = {"post": HybridLayer, "parallel": ParallelLayer, "branch": BranchLayer}[block]
+        kind = {"post": HybridLayer, "parallel": ParallelLayer, "branch": BranchLayer, "sandwich": SandwichLayer}[block]
         self.layers = nn.ModuleList([kind(s, cfg, i, dtype, device) for i, s in enumerate(cfg.layers)])
         self.runs = cfg.runs
+        self.bigram = self.pos = self.loop_in = None
+        if block == "sandwich":
+            table = lambda n: frozen(torch.zeros(n, cfg.hidden_size, dtype=dtype, device=device))      # noqa: E731
+            self.bigram, self.pos = table(cfg.pair[0] + 1), table(cfg.max_positions)
+            if cfg.loop:
+                self.loop_in = frozen(torch.zeros(-(-cfg.hidden_size // 8) * 8, 2 * cfg.hidden_size, dtype=dtype, device=device))
         self.norm_w = frozen(torch.zeros(cfg.hidden_size, device=device))
         self.norm_b = frozen(torch.zeros(cfg.hidden_size, device=device)) if block == "post" else None
         self.head = self.embed_tokens if cfg.design.tied else frozen(torch.zeros(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
@@ -375,6 +463,13 @@ class HybridDecoderLM(nn.Module):
         """(checkpoint name, shape, setter, getter) of every tensor."""
         c = self.cfg
         yield "embed", (c.vocab_size, c.hidden_size), self.embed_tokens.copy_, lambda: self.embed_tokens
+        for name in ("bigram", "pos"):
+            p = getattr(self, name)
+            if p is not None:
+                yield name, tuple(p.shape), p.copy_, (lambda p=p: p)
+        if self.loop_in is not None:
+            w = c.hidden_size
+            yield "loop.in", (w, 2 * w), lambda t: self.loop_in[:w].copy_(t), lambda: self.loop_in[:w]
         for i, layer in enumerate(self.layers):
             for name, *rest in layer.named_weights():
                 yield (f"l{i}.{name}", *rest)
@@ -420,7 +515,13 @@ class HybridDecoderLM(nn.Module):
                 put(rnd().normal_(0.0, 1.0, generator=g))
             elif leaf.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
                 put(rnd().normal_(0.0, 0.1, generator=g))
-            elif self.cfg.design.norm_base and leaf in ("norm1", "norm2", "final.norm"):
+            elif leaf.endswith(".lower"):
+                put(rnd().uniform_(0.0, 0.9, generator=g))
+            elif leaf.endswith("mix.f.b") or leaf.endswith("right.f.b"):
+                put(rnd().uniform_(1.0, 6.0, generator=g))
+            elif leaf.endswith(".pb"):
+                put(torch.full(shape, -4.0, device=device or "cpu"))
+            elif self.cfg.design.norm_base and leaf in ("norm1", "norm2", "norm1b", "norm2b", "final.norm"):
                 put(torch.full(shape, 1.0 - self.cfg.design.norm_base, device=device or "cpu"))
             elif leaf.endswith(".A_log"):
                 put(rnd().uniform_(1.0, 16.0, generator=g).log_())
@@ -428,7 +529,7 @@ class HybridDecoderLM(nn.Module):
                 put(rnd().uniform_(-4.6, -2.3, generator=g))
             elif leaf.endswith(".D") or leaf.endswith("norm") or leaf in ("norm1", "norm2"):
                 put(torch.ones(shape, device=device or "cpu"))
-            elif leaf.endswith(".conv"):
+            elif leaf.endswith(".conv") or leaf == "canon1":
                 put(rnd().uniform_(-0.5, 0.5, generator=g))
             elif leaf.endswith(".b"):
                 put(torch.zeros(shape, device=device or "cpu"))
@@ -448,8 +549,12 @@ class HybridDecoderLM(nn.Module):
         if quant or window:
             raise ValueError("the latent / state cache has no quantised or windowed variant")
         p = self.embed_tokens
-        return StateCache([self.layers[i].mixer.cache_spec() for i, _ in self.runs], num_blocks, max_seqs, dtype or p.dtype,
-                          device or p.device)
+        if self.cfg.design.block == "sandwich":
+            specs = [self.layers[i].cache_spec() for i, _ in self.runs]
+            specs.append(CacheSpec(slots={"token": ((1,), torch.int32)}))      # behind the layer runs: the sequences' latest tokens
+        else:
+            specs = [self.layers[i].mixer.cache_spec() for i, _ in self.runs]
+        return StateCache(specs, num_blocks, max_seqs, dtype or p.dtype, device or p.device, max_length=self.cfg.max_positions)
 
     @torch.no_grad()
     def forward_hidden(self, input_ids: torch.Tensor, positions=None, cu_seqlens: Optional[torch.Tensor] = None,
@@ -485,8 +590,11 @@ class HybridDecoderLM(nn.Module):
         ctx = StepContext(meta, self._freqs)
         if rows is None and not all_logits:
             rows = (meta.q_start + meta.q_lens - 1).long()
-        xf, xc = nat.embed_scale(input_ids, self.embed_tokens, cfg.embed_scale)
-        h = (self._parallel if cfg.design.block == "parallel" else self._serial)(xf, xc, cache, ctx, rows, on_layer)
+        if cfg.design.block == "sandwich":
+            h = self._sandwich(input_ids, cache, ctx, rows, on_layer)
+        else:
+            xf, xc = nat.embed_scale(input_ids, self.embed_tokens, cfg.embed_scale)
+            h = (self._parallel if cfg.design.block == "parallel" else self._serial)(xf, xc, cache, ctx, rows, on_layer)
         if h.shape[0] == 0:
             return torch.empty(0, h.shape[1] if return_hidden else cfg.vocab_size, dtype=torch.float32, device=h.device)
         return h if return_hidden else ops.project_f32(h, self.head, cfg.vocab_size)
@@ -525,3 +633,43 @@ class HybridDecoderLM(nn.Module):
             nxt, again = self.runs[n + 1]
             x, h = nat.add_rmsnorm(x, self.layers[nxt].norm1_w, eps, x0=x0 if again else None, dtype=dt,
                                    out=None if x is x0 or on_layer is not None else x, **terms)
+
+    def _sandwich(self, ids, cache, ctx, rows, on_layer) -> torch.Tensor:
+        from ..ops import native as nat
+        cfg, dt, meta = self.cfg, self.dtype, ctx.meta
+        W, kw = cfg.hidden_size, {"base": cfg.design.norm_base, "dtype": self.dtype}
+        # [stream | embedding output] in the compute type, as the projection at the start of a pass reads it
+        cat = torch.empty(ids.shape[0], 2 * W, dtype=dt, device=ids.device) if self.loop_in is not None else None
+        x = nat.pair_embed(ids, self.embed_tokens, self.bigram, self.pos, meta, cache.slots[len(self.runs)]["token"], cfg.pair,
+                           cat[:, W:] if cat is not None else None)
+        single = meta.max_q == 1
+
+        def enter(n, x, **last):
+            """(stream, input of layer run n's mixer) behind the sublayer result in ``last``."""
+            i, starts = self.runs[n]
+            layer, ring = self.layers[i], cache.slots[n]["canon"]
+            if starts:
+                x, _ = nat.branch_norm(x, cfg.norm_eps, oc=cat[:, :W], out=x, **last, **kw)
+                if on_layer is not None and n:
+                    on_layer(n - 1, x.clone())
+                x, last = ops.project_f32(cat, self.loop_in, W).contiguous(), {}
+            conv = (layer.conv_w, ring, meta.state_slots, meta.positions) if single else None
+            x, h = nat.branch_norm(x, cfg.norm_eps, wn=layer.norm1_w, conv=conv, out=x, **last, **kw)
+            if on_layer is not None and n and not starts:
+                on_layer(n - 1, x.clone())
+            return x, (h if single else nat.canon(h, layer.conv_w, ring, meta))
+
+        x, h = enter(0, x)
+        for n, (i, _) in enumerate(self.runs):
+            layer = self.layers[i]
+            last = {"y": layer.mixer(h, cache, ctx, n), "wb": layer.norm1b_w}
+            if layer.mlp is not None:
+                x, h = nat.branch_norm(x, cfg.norm_eps, wn=layer.norm2_w, out=x, **last, **kw)
+                last = {"y": layer.mlp(h), "bias": layer.mlp.b_down, "wb": layer.norm2b_w}
+            if n + 1 < len(self.runs):
+                x, h = enter(n + 1, x, **last)
+        if on_layer is not None:
+            on_layer(len(self.runs) - 1, nat.branch_norm(x, cfg.norm_eps, **last, **kw)[0])
+        if rows is not None and rows.shape[0] == 0:
+            return h[:0]
+        return nat.branch_norm(x, cfg.norm_eps, wn=self.norm_w, rows=rows, want_stream=False, **last, **kw)[1]

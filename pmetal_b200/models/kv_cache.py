@@ -97,6 +97,7 @@ class PagedBlocks:
     window = 0
     sink = 0
     can_truncate = True                   # a sequence may drop its latest tokens (no state that has already absorbed them)
+    max_length = 0                        # most positions of a sequence (models with a table of positions); 0: any number
     scratch_block: Optional[int] = None   # block outside the pool that padding rows of a captured step may write to
 
     def __init__(self, num_blocks: int, device):
@@ -155,6 +156,8 @@ class PagedBlocks:
         st = self.seqs[seq_id]
         slots: List[int] = []
         pos, end = st.length, st.length + n
+        if 0 < self.max_length < end:
+            raise ValueError(f"sequence of {end} tokens: the model has {self.max_length} positions")
         while pos < end:
             bi = pos // BLOCK
             if bi == len(st.blocks):

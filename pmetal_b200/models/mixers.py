@@ -12,13 +12,16 @@ which of them the ``type`` entries of its configuration mean. A new kind of mixe
 ``LinearAttentionMixer`` linear attention with a fixed decay per head; ``LightningMixer`` and ``RetentionMixer`` set its
                          activation, rotation, norm and gate (csrc/linear_attn.cu)
 ``GroupedAttentionMixer`` grouped-query attention of any key and value size (csrc/window_attn.cu): ``WindowAttentionMixer``
-                         (sliding window, keys as values), ``DifferenceAttentionMixer`` (difference of two maps) and
-                         ``SinkAttentionMixer`` (capped scores, a sink per head)
+                         (sliding window, keys as values), ``DifferenceAttentionMixer`` (difference of two maps),
+                         ``SinkAttentionMixer`` (capped scores, a sink per head) and ``SigmoidAttentionMixer`` (chunks, sigmoid weights)
+``ChannelGateMixer``     linear attention with a forget gate per channel that also says what is written (csrc/gated_linear.cu)
+``MatrixMemoryMixer``    matrix memory with exponential input gates and a normaliser (csrc/gated_linear.cu)
+``ParallelMixer``        two mixers on one input: one input and one output projection around both
 """
 from __future__ import annotations
 
 import math
-from typing import Dict, Optional
+from typing import Callable, Dict, Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -324,11 +327,39 @@ class RetentionMixer(LinearAttentionMixer):
     KEY_FACTOR = HEAD_NORM = SILU_GATE = True
 
 
-class GroupedAttentionMixer(nn.Module):
-    """Grouped-query softmax attention on cached keys and values. The class says what the design fixes, the configuration entry
-    gives sizes and, where present, the rotation (``rot``), the window (``mask``), the query factor that grows with the position
-    (``q_temp``) and the cap of the scores (``softcap``). ``kv_from`` makes the layer read an earlier layer's keys and values with
-    its own queries."""
+Place = Callable[[], Tuple[torch.Tensor, torch.Tensor]]
+
+
+class StackedMixer(nn.Module):
+    """A mixer between one stacked input projection and one output projection, which may be parts of larger ones: ``place`` gives
+    the rows and columns that are this mixer's (``ParallelMixer``), else it owns both. ``n_in`` rows enter as activations (padded to 8),
+    ``n_gate`` further ones as fp32 logits; ``inner`` columns leave."""
+
+    n_in = n_gate = inner = 0
+
+    def _own_projections(self, width: int, dtype, device, place: Optional[Place]) -> None:
+        up8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        self.width, self.n_pad = width, up8(self.n_in)
+        self.place = place
+        if place is None:
+            self.w_in = frozen(torch.zeros(up8(self.n_pad + self.n_gate) if self.n_gate else self.n_pad, width, dtype=dtype, device=device))
+            self.w_o = frozen(torch.zeros(up8(width), self.inner, dtype=dtype, device=device))
+
+    def _rows(self, at: int, n: int):
+        """(setter, getter) of ``n`` rows of the input projection."""
+        part = lambda: (self.place()[0] if self.place else self.w_in)[at:at + n]      # noqa: E731
+        return (lambda t: part().copy_(t)), part
+
+    def _output(self):
+        part = lambda: (self.place()[1] if self.place else self.w_o)[:self.width, :self.inner]      # noqa: E731
+        return "o", (self.width, self.inner), (lambda t: part().copy_(t)), part
+
+
+class GroupedAttentionMixer(StackedMixer):
+    """Grouped-query attention on cached keys and values. The class says what the design fixes, the configuration entry
+    gives sizes and, where present, the rotation (``rot``), the window or the size of the chunks (``mask``), the query factor that grows
+    with the position (``q_temp``) and the cap of the scores (``softcap``). ``kv_from`` makes the layer read an earlier layer's keys and
+    values with its own queries."""
 
     KEYS = ("heads", "kv_heads", "dim", "vdim", "scale")
     MAPS = 1                   # attention maps per head over the same values; with two their difference is taken
@@ -338,6 +369,8 @@ class GroupedAttentionMixer(nn.Module):
     OWN_VALUES = True          # else the values are the keys as projected
     SINK = False               # a learned score per head without a value
     GATE = True                # sigmoid of a projection of the input, one number per head
+    CHUNKED = False            # a position sees its own chunk of ``mask.size`` positions, else a window of that size
+    SIGMOID = False            # sigmoid of score + a number per head in place of the softmax
 
     @classmethod
     def check(cls, m: dict, index: int, layers) -> None:
@@ -365,7 +398,7 @@ class GroupedAttentionMixer(nn.Module):
         if any(o.get(k) != m.get(k) for k in ("heads", "kv_heads", "dim", "vdim", "rot", "mask")):
             raise ValueError(f"layer {index}: head counts, sizes, rotation and window must equal layer {src}'s")
 
-    def __init__(self, m: dict, cfg, index: int, dtype, device):
+    def __init__(self, m: dict, cfg, index: int, dtype, device, place: Optional[Place] = None):
         super().__init__()
         H, G, M, D, DV = self.dims = (m["heads"], m["kv_heads"], self.MAPS, m["dim"], m["vdim"])
         rot = m["rot"] if self.ROTATION != "none" else {"base": 1.0, "dims": 0}
@@ -376,7 +409,7 @@ class GroupedAttentionMixer(nn.Module):
         temp = m.get("q_temp")
         self.temp = (float(temp["coef"]), int(temp["every"])) if temp is not None else None
         src = m.get("kv_from")
-        self.own, self.source, self.index, self.width = src is None, index if src is None else src, index, cfg.hidden_size
+        self.own, self.source, self.index = src is None, index if src is None else src, index
         parts = [("q", H * M * D)]
         if self.own:
             parts += [("k", G * M * D)] + ([("v", G * DV)] if self.OWN_VALUES else [])
@@ -386,11 +419,10 @@ class GroupedAttentionMixer(nn.Module):
         for name, rows in parts:
             self.at[name] = n
             n += rows
-        self.inner = H * DV
-        up8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        self.n_in, self.inner = n, H * DV
+        self._own_projections(cfg.hidden_size, dtype, device, place)
         vec = lambda n: frozen(torch.zeros(n, device=device))      # noqa: E731
-        self.w_in = frozen(torch.zeros(up8(n), self.width, dtype=dtype, device=device))
-        self.w_o = frozen(torch.zeros(up8(self.width), self.inner, dtype=dtype, device=device))
+        self.wbias = vec(H) if self.SIGMOID else None
         self.q_norm_w = vec(D) if self.NORM_WEIGHTS else None
         self.k_norm_w = vec(D) if self.NORM_WEIGHTS and self.own else None
         self.sink = vec(H) if self.SINK else None
@@ -411,40 +443,44 @@ class GroupedAttentionMixer(nn.Module):
 
     def named_weights(self):
         for name, n in self.parts:
-            a = self.at[name]
-            yield name, (n, self.width), lambda t, a=a, n=n: self.w_in[a:a + n].copy_(t), lambda a=a, n=n: self.w_in[a:a + n]
+            yield (name, (n, self.width), *self._rows(self.at[name], n))
         for name in ("q", "k"):
             p = getattr(self, name + "_norm_w")
             if p is not None:
                 yield name + ".norm", tuple(p.shape), p.copy_, lambda p=p: p
         if self.sink is not None:
             yield "sink", tuple(self.sink.shape), self.sink.copy_, lambda: self.sink
+        if self.wbias is not None:
+            yield "pb", tuple(self.wbias.shape), self.wbias.copy_, lambda: self.wbias
         for name in ("lq1", "lk1", "lq2", "lk2") if self.dims[2] > 1 else ():
             p = getattr(self, name)
             yield name, tuple(p.shape), lambda t, p=p: self._put_lambda(p, t), lambda p=p: p
-        w = self.width
-        yield "o", (w, self.inner), lambda t: self.w_o[:w].copy_(t), lambda: self.w_o[:w]
+        yield self._output()
 
     def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
+        o = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
+        self.mix(ops.project(x, self.w_in), None, cache, ctx, run, o)
+        return ops.project(o, self.w_o)
+
+    def mix(self, u: torch.Tensor, z, cache, ctx: StepContext, run: Optional[int], o: torch.Tensor, scale: float = 1.0) -> None:
+        """Between the projections: rows u (any stride) -> ``scale`` times the heads' results in the rows of o (any stride)."""
         from ..ops import native as nat
         pages = cache.pages[run if self.own and run is not None else self.source]
-        u = ops.project(x, self.w_in)
         cos, sin = ctx.rope(self.base, self.R) if self.R else (None, None)
         k_at = self.at.get("k", 0)
         short, long = ctx.groups(SHORT)
-        wide = nat.window_wide(self.dims, x.dtype, self.window) if long is not None else 0
+        wide = nat.window_wide(self.dims, u.dtype, self.window) if long is not None and not self.SIGMOID else 0
         q = nat.window_prep(u, cos, sin, self.dims, (self.R, self.ROTATION), self.UNIT_NORM, self.eps, (k_at, self.at.get("v", k_at)),
                             pages if self.own else None, ctx.meta.slots, self.q_norm_w, self.k_norm_w, self.temp, ctx.meta.positions, wide)
-        o = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
         gate = u[:, self.at["g"]:] if self.GATE else None
         diff = (self.lam, 1.0 - self.diff, self.eps) if self.dims[2] > 1 else None
+        more = (self.softcap, self.sink, gate, diff)
         if short is not None:
-            nat.window_attn(q, pages, short, self.dims, self.window, self.scale, True, o, self.softcap, self.sink, gate, diff)
+            nat.window_attn(q, pages, short, self.dims, self.window, self.scale, True, o, *more, self.CHUNKED, self.wbias, scale)
         if long is not None and wide:
-            nat.window_expand_attn(q, pages, long, ctx.runs(SHORT), self.dims, self.scale, o, self.softcap, self.sink, gate, diff)
+            nat.window_expand_attn(q, pages, long, ctx.runs(SHORT), self.dims, self.scale, o, *more)
         elif long is not None:
-            nat.window_attn(q, pages, long, self.dims, self.window, self.scale, False, o, self.softcap, self.sink, gate, diff)
-        return ops.project(o, self.w_o)
+            nat.window_attn(q, pages, long, self.dims, self.window, self.scale, False, o, *more, self.CHUNKED, self.wbias, scale)
 
 
 class WindowAttentionMixer(GroupedAttentionMixer):
@@ -468,6 +504,188 @@ class SinkAttentionMixer(GroupedAttentionMixer):
     SINK = True
 
 
+class SigmoidAttentionMixer(GroupedAttentionMixer):
+    """Normed and rotated queries and keys, chunks counted from position 0, unnormalised sigmoid weights."""
+
+    KEYS = GroupedAttentionMixer.KEYS + ("rot", "mask")
+    ROTATION = "half"
+    GATE = False
+    CHUNKED = SIGMOID = True
+
+    @classmethod
+    def check(cls, m: dict, index: int, layers) -> None:
+        super().check(m, index, layers)
+        if m["mask"] is None:
+            raise ValueError(f"layer {index}: mask.size must be at least 1")
+        if any(m.get(k) is not None for k in ("kv_from", "softcap")):
+            raise ValueError(f"layer {index}: attention with sigmoid weights takes neither kv_from nor softcap")
+
+
+class ChannelGateMixer(StackedMixer):
+    """f = lower + (1 - lower) sigmoid(W_f x + b) per head and channel, S <- diag(f) S + (1 - f) v^T, o = S^T silu(W_q x) per head; every
+    head RMS-normed with one weight for all heads, and projected. Gates are formed in fp32 from fp32 sums."""
+
+    KEYS = ("heads", "dim", "vdim")
+
+    @classmethod
+    def check(cls, m: dict, index: int, layers) -> None:
+        if min(m["heads"], m["dim"], m["vdim"]) < 1 or m["dim"] > 2048:
+            raise ValueError(f"layer {index}: heads, dim and vdim must be positive, dim at most 2048")
+
+    def __init__(self, m: dict, cfg, index: int, dtype, device, place: Optional[Place] = None):
+        super().__init__()
+        self.dims = self.H, self.N, self.P = m["heads"], m["dim"], m["vdim"]
+        self.n_k, self.inner = self.H * self.N, self.H * self.P
+        self.v_at = -(-self.n_k // 8) * 8
+        self.n_in, self.n_gate = self.v_at + self.inner, self.n_k
+        self.eps, self.index = cfg.norm_eps, index
+        self._own_projections(cfg.hidden_size, dtype, device, place)
+        vec = lambda n: frozen(torch.zeros(n, device=device))      # noqa: E731
+        self.f_bias, self.lower, self.norm_w = vec(self.n_k), vec(self.n_k), vec(self.P)
+
+    def cache_spec(self) -> CacheSpec:
+        return CacheSpec(slots={"state": ((self.H, self.N, -(-self.P // 4) * 4), torch.float32)})
+
+    def named_weights(self):
+        for name, at, n in (("q", 0, self.n_k), ("f", self.n_pad, self.n_k), ("v", self.v_at, self.inner)):
+            yield (name, (n, self.width), *self._rows(at, n))
+        for name, p in (("f.b", self.f_bias), ("lower", self.lower), ("norm", self.norm_w)):
+            yield name, tuple(p.shape), p.copy_, (lambda p=p: p)
+        yield self._output()
+
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
+        o = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
+        u, z = ops.project_mixed(x, self.w_in, self.n_pad)
+        self.mix(u, z, cache, ctx, run, o)
+        return ops.project(o, self.w_o)
+
+    def mix(self, u: torch.Tensor, z: torch.Tensor, cache, ctx: StepContext, run: Optional[int], o: torch.Tensor, scale: float = 1.0) -> None:
+        """Between the projections: rows u and gate logits z (any stride) -> ``scale`` times the heads' results in the rows of o."""
+        from ..ops import native as nat
+        state = cache.slots[self.index if run is None else run]["state"]
+        y = torch.empty(u.shape[0], self.inner, dtype=u.dtype, device=u.device)
+        args = (u, u[:, self.v_at:], z, self.f_bias, self.lower, state)
+        tensor_cores = u.dtype == torch.bfloat16 and nat.linear_chunk_supported(self.N)
+        short, long = ctx.groups(SHORT if tensor_cores else 1 << 30)
+        if short is not None:
+            nat.channel_scan(*args, short, self.dims, y)
+        if long is not None:
+            nat.channel_chunk(*args, long, self.dims, y)
+        nat.norm_gate(y, None, self.norm_w, self.eps, self.H, False, scale=scale, out=o)
+
+
+class MatrixMemoryMixer(StackedMixer):
+    """S <- exp(f + m - m') S + exp(i - m') k v^T with i = cap tanh(. / cap), f = log sigmoid(cap tanh(. / cap)) of fp32 sums and the
+    running maximum m' = max(f + m, i); the read-out is divided by max(|n . q|, exp(-m')) + 1e-6, every head RMS-normed, times a weight
+    and the sigmoid of a gate."""
+
+    KEYS = ("heads", "dim", "vdim", "gate_cap")
+    DEN_EPS = 1e-6
+
+    @classmethod
+    def check(cls, m: dict, index: int, layers) -> None:
+        if min(m["heads"], m["dim"], m["vdim"]) < 1 or m["dim"] > 2048:
+            raise ValueError(f"layer {index}: heads, dim and vdim must be positive, dim at most 2048")
+        if not m["gate_cap"] > 0:
+            raise ValueError(f"layer {index}: gate_cap must be positive")
+
+    def __init__(self, m: dict, cfg, index: int, dtype, device, place: Optional[Place] = None):
+        super().__init__()
+        self.dims = self.H, self.N, self.P = m["heads"], m["dim"], m["vdim"]
+        up8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        self.n_k, self.inner = self.H * self.N, self.H * self.P
+        self.at = {"q": 0, "k": up8(self.n_k), "v": 2 * up8(self.n_k), "g": 2 * up8(self.n_k) + up8(self.inner)}
+        self.n_in, self.n_gate = self.at["g"] + self.inner, 2 * self.H
+        self.gates = (float(m["gate_cap"]), self.N ** -0.5, self.DEN_EPS)
+        self.eps, self.index = cfg.norm_eps, index
+        self._own_projections(cfg.hidden_size, dtype, device, place)
+        vec = lambda n: frozen(torch.zeros(n, device=device))      # noqa: E731
+        self.g_bias, self.norm_w = vec(2 * self.H), vec(self.inner)      # input gates, then forget gates
+
+    def cache_spec(self) -> CacheSpec:
+        p4 = -(-self.P // 4) * 4
+        f32 = torch.float32
+        return CacheSpec(slots={"state": ((self.H, self.N, p4), f32), "norm": ((self.H, self.N), f32), "max": ((self.H, p4 // 4), f32)})
+
+    def named_weights(self):
+        for name, n in (("q", self.n_k), ("k", self.n_k), ("v", self.inner), ("g", self.inner)):
+            yield (name, (n, self.width), *self._rows(self.at[name], n))
+        yield self._output()
+        yield "norm", (self.inner,), self.norm_w.copy_, lambda: self.norm_w
+        H = self.H
+        for i, name in enumerate(("i", "f")):
+            yield (name, (H, self.width), *self._rows(self.n_pad + i * H, H))
+            yield name + ".b", (H,), lambda t, i=i: self.g_bias[i * H:(i + 1) * H].copy_(t), lambda i=i: self.g_bias[i * H:(i + 1) * H]
+
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
+        o = torch.empty(x.shape[0], self.inner, dtype=x.dtype, device=x.device)
+        u, z = ops.project_mixed(x, self.w_in, self.n_pad)
+        self.mix(u, z, cache, ctx, run, o)
+        return ops.project(o, self.w_o)
+
+    def mix(self, u: torch.Tensor, z: torch.Tensor, cache, ctx: StepContext, run: Optional[int], o: torch.Tensor, scale: float = 1.0) -> None:
+        """Between the projections: rows u and gate logits z (any stride) -> ``scale`` times the heads' results in the rows of o."""
+        from ..ops import native as nat
+        store, at = cache.slots[self.index if run is None else run], self.at
+        y = torch.empty(u.shape[0], self.inner, dtype=u.dtype, device=u.device)
+        den = torch.empty(u.shape[0], self.H, dtype=torch.float32, device=u.device)
+        more = (u[:, at["v"]:], z, self.g_bias, self.gates, store)
+        tensor_cores = u.dtype == torch.bfloat16 and nat.linear_chunk_supported(self.N)
+        short, long = ctx.groups(SHORT if tensor_cores else 1 << 30)
+        if short is not None:
+            nat.memory_scan(u, u[:, at["k"]:], *more, short, self.dims, y, den)
+        if long is not None:
+            nat.memory_chunk(u, at["q"], at["k"], *more, long, self.dims, y, den)
+        nat.norm_gate(y, u[:, at["g"]:], self.norm_w, self.eps, self.H, False, den, scale, o)
+
+
+class ParallelMixer(nn.Module):
+    """left_scale * left(x) + right_scale * right(x). Both mixers' input projections are one product and so are the output projections:
+    the scales go to the heads' results, whose columns lie side by side."""
+
+    KEYS = ("left", "right", "left_scale", "right_scale")
+    LEFT, RIGHT = SigmoidAttentionMixer, MatrixMemoryMixer
+
+    @classmethod
+    def check(cls, m: dict, index: int, layers) -> None:
+        for side, kind in (("left", cls.LEFT), ("right", cls.RIGHT)):
+            missing = [k for k in kind.KEYS if k not in m[side]]
+            if missing:
+                raise ValueError(f"layer {index}: {side} mixer entry lacks {', '.join(missing)}")
+            kind.check(m[side], index, layers)
+
+    def __init__(self, m: dict, cfg, index: int, dtype, device):
+        super().__init__()
+        up8 = lambda n: -(-n // 8) * 8      # noqa: E731
+        self.left = self.LEFT(m["left"], cfg, index, dtype, device, lambda: (self.w_in[:self.cut], self.w_o[:, :self.c_cut]))
+        self.right = self.RIGHT(m["right"], cfg, index, dtype, device, lambda: (self.w_in[self.cut:], self.w_o[:, self.c_cut:]))
+        self.scales = (float(m["left_scale"]), float(m["right_scale"]))
+        self.cut, self.c_cut = self.left.n_pad, up8(self.left.inner)      # the left mixer has no gate rows
+        self.n_low, self.cols = self.cut + self.right.n_pad, self.c_cut + up8(self.right.inner)
+        self.ragged = self.cols != self.left.inner + self.right.inner
+        width = cfg.hidden_size
+        self.w_in = frozen(torch.zeros(up8(self.n_low + self.right.n_gate), width, dtype=dtype, device=device))
+        self.w_o = frozen(torch.zeros(up8(width), self.cols, dtype=dtype, device=device))
+
+    def cache_spec(self) -> CacheSpec:
+        a, b = self.left.cache_spec(), self.right.cache_spec()
+        return CacheSpec(page_width=a.page_width, window=a.window, slots={**a.slots, **b.slots})
+
+    def named_weights(self):
+        for pre, mod in (("left.", self.left), ("right.", self.right)):
+            for name, *rest in mod.named_weights():
+                yield (pre + name, *rest)
+
+    def forward(self, x: torch.Tensor, cache, ctx: StepContext, run: Optional[int] = None) -> torch.Tensor:
+        u, z = ops.project_mixed(x, self.w_in, self.n_low)
+        make = torch.zeros if self.ragged else torch.empty
+        o = make(x.shape[0], self.cols, dtype=x.dtype, device=x.device)
+        self.left.mix(u[:, :self.cut], None, cache, ctx, run, o, self.scales[0])
+        self.right.mix(u[:, self.cut:], z, cache, ctx, run, o[:, self.c_cut:], self.scales[1])
+        return ops.project(o, self.w_o)
+
+
 MIXERS = {"mamba2": Mamba2Mixer, "latent_attention": LatentAttentionMixer, "lightning": LightningMixer,
           "retention": RetentionMixer, "window_attention": WindowAttentionMixer, "difference_attention": DifferenceAttentionMixer,
-          "sink_attention": SinkAttentionMixer}
+          "sink_attention": SinkAttentionMixer, "sigmoid_attention": SigmoidAttentionMixer, "channel_gate": ChannelGateMixer,
+          "matrix_memory": MatrixMemoryMixer, "sigmoid_attention_and_memory": ParallelMixer}

@@ -13,7 +13,8 @@ state has absorbed every token it saw, so a sequence with slots cannot be cut ba
 slot and shares the pages. When every layer with pages has a window, pages that lie wholly before the widest of them go back
 to the pool while the sequence lives.
 
-A layer that runs several times in a step (a looped stack) has a spec, pages and slots for every run.
+A layer that runs several times in a step (a looped stack) has a spec, pages and slots for every run; a model may add a spec of its own
+behind them (the latest token of every sequence).
 
 ``split_groups`` divides a step's sequences into short and long portions, which run on different kernels; ``attention_runs`` joins
 long portions into launches of an attention kernel whose keys are rows of one buffer."""
@@ -37,8 +38,10 @@ class CacheSpec:
 
 
 class StateCache(PagedBlocks):
-    def __init__(self, specs: Sequence[CacheSpec], num_blocks: int, max_seqs: int, dtype=torch.bfloat16, device="cuda"):
+    def __init__(self, specs: Sequence[CacheSpec], num_blocks: int, max_seqs: int, dtype=torch.bfloat16, device="cuda",
+                 max_length: int = 0):
         super().__init__(num_blocks, device)
+        self.max_length = max_length
         self.max_seqs = max_seqs
         self.scratch_block, self.scratch_slot = num_blocks, max_seqs
         self.pages: Dict[int, torch.Tensor] = {}

@@ -1154,19 +1154,23 @@ def gemv(x, w, norm_w=None, eps: float = 1e-6, residual=None, swiglu: bool = Fal
     return y
 
 
-def gemv_ex(x, w, bias=None, glu=None, out_f32: bool = False, n: Optional[int] = None, gelu: bool = False):
+def gemv_ex(x, w, bias=None, glu=None, out_f32: bool = False, n: Optional[int] = None, gelu: bool = False,
+            f32_from: Optional[int] = None):
     """x [M <= 16, K] bf16, w [>= n, K] bf16 -> [M, n]: products plus ``bias`` (fp32). ``glu`` = (limit, beta, shift): w
     stacks gate rows above up rows and the result is the clamped gated unit, n = rows / 2. ``gelu``: exact gelu of the sums.
-    ``out_f32``: fp32 result."""
+    ``out_f32``: fp32 result. ``f32_from``: returns ([M, f32_from] bf16, the other columns in fp32)."""
     M, K = x.shape
     N = n if n is not None else (w.shape[0] // 2 if glu else w.shape[0])
-    y = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
+    cut = N if f32_from is None else f32_from
+    y = torch.empty(M, cut, dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
+    tail = None if f32_from is None else torch.empty(M, N - cut, dtype=torch.float32, device=x.device)
     lim, beta, shift = glu if glu else (0.0, 0.0, 0.0)
     _chk(lib().pm_gemv_ex(_p(x), c_int(x.stride(0)), _p(w), c_int(w.stride(0)), _p(None), c_float(0.0), _p(None), c_int(0),
-                          _p(y), c_int(N), c_int(M), c_int(N), c_int(K), c_int(1 if glu else 0), c_float(1.0), _p(None),
+                          _p(y), c_int(cut), c_int(M), c_int(N), c_int(K), c_int(1 if glu else 0), c_float(1.0), _p(None),
                           c_int(0), _p(None), c_int(0), (c_int * 4)(*([0x7FFFFFFF] * 4)), _p(bias), c_int(1 if glu else 2 if gelu else 0),
-                          c_float(lim), c_float(beta), c_float(shift), c_int(int(out_f32)), _stream()), "pm_gemv_ex")
-    return y
+                          c_float(lim), c_float(beta), c_float(shift), c_int(int(out_f32)), _p(tail), c_int(cut), c_int(N - cut),
+                          _stream()), "pm_gemv_ex")
+    return y if tail is None else (y, tail)
 
 
 def gemv_q4(x, q, norm_w=None, eps: float = 1e-6, residual=None, swiglu: bool = False, alpha: float = 1.0, t=None,
@@ -1485,12 +1489,127 @@ def linear_chunk(u, cs, sn, log2_decay, kscale: float, state, group, dims, y) ->
     LAUNCHES += 1 + int(max_seg > 1)
 
 
-def norm_gate(y, gate, w, eps: float, parts: int, silu: bool):
-    """RMS norm over ``parts`` equal parts of y, times w (fp32, may be None), times silu or sigmoid of ``gate`` (rows of any
-    stride)."""
-    out = torch.empty_like(y)
-    _chk(lib().pm_norm_gate(_p(y), _p(gate), _is_f32(y), c_ll(gate.stride(0)), _p(w), c_float(eps), c_int(parts),
-                            c_int(y.shape[1] // parts), c_int(int(silu)), _p(out), c_int(y.shape[0]), _stream()), "pm_norm_gate")
+def norm_gate(y, gate, w, eps: float, parts: int, silu: bool, den=None, scale: float = 1.0, out=None):
+    """RMS norm over ``parts`` equal parts of y, times w (fp32, for all parts or one for each, may be None), times silu or sigmoid of
+    ``gate`` (rows of any stride, may be None), times ``scale``. ``den`` (fp32 [tokens, parts]): y is divided by it first. ``out``: rows
+    of any stride."""
+    width = y.shape[1] // parts
+    out = torch.empty_like(y) if out is None else out
+    if w is not None and w.numel() not in (width, y.shape[1]):
+        raise ValueError(f"{w.numel()} weights for {parts} parts of {width}")
+    _chk(lib().pm_norm_gate(_p(y), _p(gate), _is_f32(y), c_ll(gate.stride(0) if gate is not None else 0), _p(w), c_float(eps),
+                            c_int(parts), c_int(width), c_int(int(silu)), _p(out), c_int(y.shape[0]), _p(den),
+                            c_int(int(w is not None and w.numel() == width)), c_float(scale), c_ll(out.stride(0)), _stream()),
+         "pm_norm_gate")
+    return out
+
+
+# ------------------------------------------------------------------------------------------- linear attention, gates per token
+def _segments(group, H: int, N: int, P: int, per: int, device):
+    """(largest number of segments, buffer of the segments' states, buffer of ``per`` floats per segment and head)."""
+    max_seg = max(1, min(-(-group.max_q // 64), -(-6 * sm_count() // max(-(-P // 32) * H * group.n, 1))))
+    rows = group.n * max_seg * H
+    buf = torch.empty(rows * (N * (-(-P // 4) * 4) + per), dtype=torch.float32, device=device)
+    return max_seg, buf, buf[rows * N * (-(-P // 4) * 4):]
+
+
+def channel_scan(q, v, z, bias, lower, state, group, dims, y) -> None:
+    """Recurrence with a forget gate per channel, token by token, for the sequences of ``group``; q, v: columns of a projection (the
+    same row stride), z fp32 logits of the gates, ``dims`` = (heads, key channels, value channels). Writes the rows of y."""
+    H, N, P = dims
+    _chk(lib().pm_channel_scan(_p(q), _p(v), _is_f32(q), c_ll(q.stride(0)), _p(z), c_ll(z.stride(0)), _p(bias), _p(lower), _p(state),
+                               _p(group.state_slots), _p(group.q_start), _p(group.q_lens), _p(group.seq_lens), c_int(group.n), c_int(H),
+                               c_int(N), c_int(P), _p(y), _stream()), "pm_channel_scan")
+
+
+def channel_chunk(q, v, z, bias, lower, state, group, dims, y) -> None:
+    """As ``channel_scan`` for longer portions of bf16 models: the recurrence in blocks of 64 tokens on the tensor cores."""
+    global LAUNCHES
+    H, N, P = dims
+    T, n16, dev = q.shape[0], -(-N // 16) * 16, q.device
+    act = torch.empty(T, 4 * H * n16, dtype=torch.bfloat16, device=dev)
+    score = torch.empty(T, H, 128, dtype=torch.bfloat16, device=dev)
+    decay = torch.empty(group.n_tok // 64 + group.n + 1, H, n16, dtype=torch.float32, device=dev)
+    max_seg, seg, seg_decay = _segments(group, H, N, P, N, dev)
+    _chk(lib().pm_channel_chunk(_p(q), _p(v), c_ll(q.stride(0)), _p(z), c_ll(z.stride(0)), _p(bias), _p(lower), _p(state),
+                                _p(group.state_slots), _p(group.q_start), _p(group.q_lens), _p(group.seq_lens), _p(group.c_start),
+                                c_int(group.n), c_int(group.max_q), c_int(H), c_int(N), c_int(P), _p(act), _p(score), _p(decay), _p(seg),
+                                _p(seg_decay), c_int(max_seg), _p(y), _stream()), "pm_channel_chunk")
+    LAUNCHES += 1 + int(max_seg > 1)
+
+
+def memory_scan(q, k, v, z, bias, gates, store, group, dims, y, den) -> None:
+    """Matrix memory token by token for the sequences of ``group``; q, k, v: columns of a projection (the same row stride), z fp32
+    logits of the input and forget gates, ``gates`` = (cap, factor of the queries, eps of the normaliser), ``store``: the layer's
+    slots. Writes the rows of y and of the normaliser ``den`` (fp32 [tokens, heads])."""
+    H, N, P = dims
+    cap, qscale, eps = gates
+    _chk(lib().pm_memory_scan(_p(q), _p(k), _p(v), _is_f32(q), c_ll(q.stride(0)), _p(z), c_ll(z.stride(0)), _p(bias), c_float(cap),
+                              c_float(qscale), c_float(eps), _p(store["state"]), _p(store["norm"]), _p(store["max"]), _p(group.state_slots),
+                              _p(group.q_start), _p(group.q_lens), _p(group.seq_lens), c_int(group.n), c_int(H), c_int(N), c_int(P), _p(y),
+                              _p(den), _stream()), "pm_memory_scan")
+
+
+def memory_chunk(u, q_at: int, k_at: int, v, z, bias, gates, store, group, dims, y, den) -> None:
+    """As ``memory_scan`` for longer portions of bf16 models; queries and keys are the columns from q_at and k_at of u, v has its rows."""
+    global LAUNCHES
+    H, N, P = dims
+    cap, qscale, eps = gates
+    T, dev = u.shape[0], u.device
+    work = torch.empty(3, T, H, dtype=torch.float32, device=dev)
+    max_seg, seg, more = _segments(group, H, N, P, N + 1, dev)
+    _chk(lib().pm_memory_chunk(_p(u), c_int(q_at), c_int(k_at), _p(v), c_ll(u.stride(0)), _p(z), c_ll(z.stride(0)), _p(bias), c_float(cap),
+                               c_float(qscale), c_float(eps), _p(store["state"]), _p(store["norm"]), _p(store["max"]),
+                               _p(group.state_slots), _p(group.q_start), _p(group.q_lens), _p(group.seq_lens), c_int(group.n), c_int(T),
+                               c_int(group.max_q), c_int(H), c_int(N), c_int(P), _p(work), _p(seg), _p(more),
+                               _p(more[group.n * max_seg * H:]), c_int(max_seg), _p(y), _p(den), _stream()), "pm_memory_chunk")
+    LAUNCHES += 1 + int(max_seg > 1)
+
+
+# ------------------------------------------------------------------------------------------- norms on both sides of a sublayer
+def pair_embed(ids, table, pairs, pos_table, meta, last, pair, cat=None):
+    """fp32 stream [n, width]: token vector + row of the pair with the previous token + row of the position. ``pair`` = (buckets, factor
+    of the previous id, factor of the id), ``last`` int32 [slots]: every sequence's latest token. ``cat`` (table's type, rows of any
+    stride): gets the same."""
+    n, width = ids.shape[0], table.shape[1]
+    xf = torch.empty(n, width, dtype=torch.float32, device=table.device)
+    _chk(lib().pm_pair_embed(_p(ids), _p(table), _p(pairs), _p(pos_table), _is_f32(table), _p(meta.positions), _p(meta.seq_of),
+                             _p(meta.q_start), _p(meta.q_lens), _p(meta.state_slots), _p(last), c_ll(pair[0]), c_ll(pair[1]), c_ll(pair[2]),
+                             c_int(n), c_int(width), c_int(pos_table.shape[0]), _p(xf), _p(cat),
+                             c_ll(cat.stride(0) if cat is not None else 0), _stream()), "pm_pair_embed")
+    return xf
+
+
+def branch_norm(x, eps: float, base: float, y=None, bias=None, wb=None, wn=None, rows=None, out=None, oc=None, dtype=None, conv=None,
+                want_stream: bool = True):
+    """v = x + r / rms(r) (base + wb), r = y + bias (without y: v = x) on the fp32 stream x [n, width] -> (v or None, v / rms(v)
+    (base + wn) in ``dtype``, v itself without wn). y has the compute type and any row stride, ``rows`` (int64) picks rows of x and y,
+    ``out``: where v goes (may be x when there are no ``rows``), ``oc``: where the second result goes (rows of any stride). ``conv`` =
+    (weights [taps, width], ring, slots, positions): every row is a sequence's only new token, and the result has the causal convolution
+    over the sequence's last inputs added."""
+    n, width = (rows.shape[0] if rows is not None else x.shape[0]), x.shape[1]
+    dtype = dtype or (y.dtype if y is not None else x.dtype)
+    if y is not None and (y.dtype != dtype or y.stride(1) != 1):
+        raise ValueError("y must have the compute type and contiguous rows")
+    of = None
+    if want_stream and y is not None:
+        of = out if out is not None else torch.empty(n, width, dtype=torch.float32, device=x.device)
+    oc = torch.empty(n, width, dtype=dtype, device=x.device) if oc is None else oc
+    w, ring, slots, pos = conv if conv is not None else (None, None, None, None)
+    _chk(lib().pm_branch_norm(_p(x), _p(y), c_int(int(dtype == torch.float32)), c_ll(y.stride(0) if y is not None else 0), _p(bias), _p(wb),
+                              _p(wn), c_float(base), c_float(eps), _p(rows), _p(of), _p(oc), c_ll(oc.stride(0)), _p(w),
+                              c_int(w.shape[0] if w is not None else 1), _p(ring), _p(slots), _p(pos), c_int(n), c_int(width), _stream()),
+         "pm_branch_norm")
+    return (of if y is not None else x), oc
+
+
+def canon(h, w, ring, meta):
+    """h [tokens, width] + its causal convolution with w (fp32 [taps, width]) along every sequence of the step; ``ring`` [slots, taps - 1,
+    width] keeps the sequences' last inputs."""
+    out = torch.empty_like(h)
+    _chk(lib().pm_canon(_p(h), _is_f32(h), _p(w), c_int(w.shape[0]), _p(ring), _p(meta.state_slots), _p(meta.q_start), _p(meta.q_lens),
+                        _p(meta.seq_lens), c_int(meta.q_lens.shape[0]), c_int(meta.max_q), c_int(h.shape[1]), _p(out), _stream()),
+         "pm_canon")
     return out
 
 
@@ -1513,10 +1632,12 @@ def window_prep(u, cs, sn, dims, rot, normed: bool, eps: float, cols, pages, slo
 
 
 def window_attn(q, pages, group, dims, window: int, scale: float, few: bool, out, softcap: float = 0.0, sink=None, gate=None,
-                diff=None) -> None:
+                diff=None, chunked: bool = False, wbias=None, out_scale: float = 1.0) -> None:
     """Attention of the sequences of ``group`` over their cached keys; rows of out [tokens, >= heads * value size]. ``few``:
     tiles for a few rows per sequence, pages split over CTAs. ``sink`` fp32 [heads], ``gate`` logits [tokens, heads] of any row
-    stride, ``diff`` = (lambda as an fp32 tensor, factor behind the norm, eps) where a head has two maps."""
+    stride, ``diff`` = (lambda as an fp32 tensor, factor behind the norm, eps) where a head has two maps. ``chunked``: a position sees
+    its own chunk of ``window`` positions. ``wbias`` fp32 [heads]: keys are weighted with the sigmoid of score + wbias. ``out_scale``
+    multiplies the result."""
     global LAUNCHES
     H, G, M, D, DV = dims
     T, D8, DV8, n_split = q.shape[0], -(-D // 8) * 8, -(-DV // 8) * 8, 1
@@ -1540,7 +1661,7 @@ def window_attn(q, pages, group, dims, window: int, scale: float, few: bool, out
                               c_int(H), c_int(G), c_int(M), c_int(D), c_int(DV), c_int(wide), c_int(window), c_float(scale), c_float(softcap),
                               _p(sink), _p(gate), c_ll(gate.stride(0) if gate is not None else 0), _p(lam), c_float(keep),
                               c_float(eps), c_int(int(few)), c_int(n_split), _p(po), _p(pml), _p(o), _p(out), c_ll(out.stride(0)),
-                              _stream()), "pm_window_attn")
+                              c_int(int(chunked)), _p(wbias), c_float(out_scale), _stream()), "pm_window_attn")
     LAUNCHES += int(po is not None or o is not None)
 
 

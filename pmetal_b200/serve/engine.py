@@ -171,6 +171,10 @@ class ContinuousBatchEngine:
     def _admit(self) -> None:
         while self.queue and len(self.slots) < self.max_slots and self.cache.can_admit():
             req = self.queue[0]
+            if 0 < self.cache.max_length < len(req.prompt):
+                self.queue.popleft()
+                self._finish(req, "error:too_long")
+                continue
             need = self._blocks_needed(req)
             reserved = sum(self._blocks_needed(s.req) - (self.cache.length(s.seq) // BLOCK) for s in self.slots)
             if self.cache.num_free() - reserved < need:
@@ -235,7 +239,7 @@ class ContinuousBatchEngine:
                 del req.logprobs[len(req.output):]
                 del req.top_entries[len(req.output):]
                 return self._retire(slot, "stop")
-        if len(req.output) >= req.params.max_tokens:
+        if len(req.output) >= req.params.max_tokens or 0 < self.cache.max_length <= self.cache.length(slot.seq):
             return self._retire(slot, "length")
         slot.last_token = tok
         return False
