@@ -1,12 +1,14 @@
 """Serving throughput of the hybrid decoder beside the closest other model at equal size, and its kernels beside the like
 kernels of the other models (``bench.py --serve-hybrid``). Random weights; device time by CUDA events.
 
-Duvivik presets stand beside the dense fast decoder; Resevik presets beside the Qwen3-MoE decoder with the same width, experts
+Duvivik and Ravapel presets stand beside the dense fast decoder (Ravapel's with one layer per layer run, its weights counted once per
+run: equal work per token); Resevik presets beside the Qwen3-MoE decoder with the same width, experts
 and attention heads and one layer per layer run (a looped stack has more runs than stored layers); Vosezen presets beside the same
 with the layers' head counts of 128 channels and experts as wide as makes the stored weights equal (its experts have two matrices
 and a shared one, the other's have three)."""
 from __future__ import annotations
 
+import math
 import statistics
 from typing import Callable, Dict, List
 
@@ -17,6 +19,7 @@ from ..models.config import ModelArgs
 from ..models.decoder import DecoderLM
 from ..models.generation import Generator
 from ..models.kv_cache import BLOCK, PagedKVCache
+from ..models.mixers import RotationFreqs, StepContext
 from ..models.state_cache import CacheSpec, StateCache, attention_runs, split_groups
 from ..ops import native as nat
 from .kernels import peaks
@@ -27,11 +30,23 @@ DENSE = {
                        num_key_value_heads=8),
     "duvivik-2b": dict(hidden_size=2560, intermediate_size=9728, num_hidden_layers=19, num_attention_heads=32,
                        num_key_value_heads=8),
+    "ravapel-1b": dict(hidden_size=2048, intermediate_size=7552, num_hidden_layers=18, num_attention_heads=16,
+                       num_key_value_heads=4),
+    "ravapel-2b": dict(hidden_size=2560, intermediate_size=9856, num_hidden_layers=28, num_attention_heads=20,
+                       num_key_value_heads=4),
 }
 
 
 def like_kind(name: str) -> str:
-    return "dense" if hd.PRESETS[name]["architecture"] == "Duvivik" else "moe"
+    return "dense" if hd.PRESETS[name]["architecture"] in ("Duvivik", "Ravapel") else "moe"
+
+
+def run_weights(args) -> int:
+    """Matrix entries that one token meets in the layers and passes (weights of looped layers once per run)."""
+    m = hd.HybridDecoderLM(args, torch.bfloat16, "meta")
+    sizes = [sum(math.prod(s) for _, s, *_ in l.named_weights() if len(s) == 2) for l in m.layers]
+    passes = sum(1 for _, again in m.runs if again) if m.loop_in is not None else 0
+    return sum(sizes[i] for i, _ in m.runs) + passes * 2 * args.hidden_size ** 2
 
 
 def like_expert_width(ex: dict) -> int:
@@ -387,6 +402,131 @@ def branch_kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int
     return out
 
 
+def sandwich_kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096) -> List[dict]:
+    """``kernel_cases`` for the stacks with norms on both sides of the sublayers (channel gates, attention with sigmoid weights in
+    chunks, matrix memory, input convolution)."""
+    cfg = hd.HybridArgs.from_dict(hd.PRESETS[name])
+    W = cfg.hidden_size
+    gt = next(l["mixer"] for l in cfg.layers if l["type"] == "hgrn2")
+    both = next(l["mixer"] for l in cfg.layers if l["type"] == "parallel")
+    at, me = both["left"], both["right"]
+    ff = next(l["mlp"]["ff"] for l in cfg.layers if l["mlp"])
+    pk, out = peaks(), []
+
+    def case(label, fn, nbytes=0, flops=0):
+        us = graph_us(fn)
+        bound = max(nbytes / pk["hbm_gbs"] / 1e3, flops / pk["bf16_tflops"] / 1e6)
+        out.append({"kernel": label, "us": round(us, 2), "bound_us": round(bound, 2), "of_measured_peak": round(bound / us, 3)})
+
+    f = lambda *s: torch.randn(*s, device="cuda")      # noqa: E731
+    for mode, n_seq, prior, new in (("decode", batch, ctx - 1, 1), ("prefill", 1, 0, prompt)):
+        T, blocks = n_seq * new, n_seq * (prior + new) // BLOCK + n_seq + 1
+        tag = f"{mode} T={T} "
+        few = mode == "decode"
+
+        def cache(slots=None, page=0):
+            c = StateCache([CacheSpec(page_width=page, slots=slots or {})], blocks, n_seq, torch.bfloat16, "cuda")
+            return (c, *_group(c, n_seq, prior, new))
+        # channel gates and matrix memory | the state-space recurrence with a state of the same size
+        for label, m in (("channel gates", gt), ("matrix memory", me)):
+            H, N, P = m["heads"], m["dim"], m["vdim"]
+            c, meta, grp = cache({"state": ((H, N, P), torch.float32), "norm": ((H, N), torch.float32), "max": ((H, P // 4), torch.float32)})
+            store = c.slots[0]
+            y, den = torch.empty(T, H * P, dtype=torch.bfloat16, device="cuda"), torch.rand(T, H, device="cuda") + 0.5
+            state_b = 2 * n_seq * H * N * P * 4
+            blk = 0 if few else 2 * T * H * (64 * (N + P) / 2 + 2 * N * P)
+            if label == "channel gates":
+                u, z, b, lo = _bf(T, H * (N + P)), f(T, H * N) + 3, f(H * N), torch.rand(H * N, device="cuda")
+                fn = nat.channel_scan if few else nat.channel_chunk
+                case(tag + label + " recurrence", lambda: fn(u, u[:, H * N:], z, b, lo, store["state"], grp, (H, N, P), y),
+                     T * H * ((N + 2 * P) * 2 + N * 4) + state_b, blk)
+                w = f(P)
+                case(tag + "norm per head", lambda: nat.norm_gate(y, None, w, 1e-5, H, False), 2 * T * H * P * 2)
+            else:
+                u, z, b, g = _bf(T, H * (2 * N + 2 * P)), f(T, 2 * H), f(2 * H) + 2, (10.0, N ** -0.5, 1e-6)
+                v = u[:, 2 * H * N:]
+                if few:
+                    case(tag + label + " recurrence", lambda: nat.memory_scan(u, u[:, H * N:], v, z, b, g, store, grp, (H, N, P), y, den),
+                         T * H * (2 * N + 2 * P) * 2 + state_b)
+                else:
+                    case(tag + label + " recurrence", lambda: nat.memory_chunk(u, 0, H * N, v, z, b, g, store, grp, (H, N, P), y, den),
+                         T * H * (2 * N + 2 * P) * 2 + state_b, blk)
+                w = f(H * P)
+                case(tag + "normaliser + norm per head + gate", lambda: nat.norm_gate(y, u[:, H * (2 * N + P):], w, 1e-5, H, False, den), 3 * T * H * P * 2)
+            S = (H, P, N, H, 4)
+            inner, conv = H * P, H * P + 2 * H * N
+            c2, meta, grp2 = cache({"conv": ((4, conv), None), "state": ((H, N, P), torch.float32)})
+            us = _bf(T, -(-(inner + conv + H) // 8) * 8)
+            vec = (f(4, conv), f(conv), f(H) - 3, f(H), f(H))
+            sfn = nat.ssm_scan if few else nat.ssm_chunk
+            case(tag + "  | ssm recurrence", lambda: sfn(us, *vec, c2.slots[0]["conv"], c2.slots[0]["state"], grp2, S, y),
+                 T * (conv + inner + H) * 2 + state_b, blk)
+            nw = f(inner)
+            case(tag + "  | ssm gate + norm", lambda: nat.ssm_gate_norm(y, us, nw, 1e-5, H, c2.slots[0]["conv"], meta, S), 3 * T * inner * 2)
+            del c, c2
+        # attention with sigmoid weights in chunks | with a softmax in a window that sees as many keys on average
+        H, G, D, DV, size = at["heads"], at["kv_heads"], at["dim"], at["vdim"], at["mask"]["size"]
+        dims = (H, G, 1, D, DV)
+        c, meta, grp = cache(page=G * (D + DV))
+        c.pages[0].normal_()
+        ua, rd, wn = _bf(T, H * D + G * (D + DV)), at["rot"]["dims"], f(D)
+        cs, sn = f(T, rd // 2), f(T, rd // 2)
+        prep = lambda: nat.window_prep(ua, cs, sn, dims, (rd, "half"), True, 1e-5, (H * D, H * D + G * D), c.pages[0], meta.slots, wn, wn,      # noqa: E731
+                                       wide=0 if few else nat.window_wide(dims, torch.bfloat16, size, True))
+        case(tag + "head norm + rotation + append", prep, 2 * T * (H * D + G * (D + DV)) * 2)
+        c3 = PagedKVCache(1, G, 128, blocks, device="cuda")
+        meta3, _ = _group(c3, n_seq, prior, new)
+        c3.k[0].normal_()
+        c3.v[0].normal_()
+        qkv, cs3, sn3, w128 = _bf(T, (H + 2 * G) * 128), f(T, 64), f(T, 64), _bf(128)
+        case(tag + "  | head norm + rotation + append",
+             lambda: nat.qknorm_rope_cache(qkv, w128, w128, cs3, sn3, H, G, 1e-6, c3.k[0], c3.v[0], meta3.slots), T * (2 * H + 4 * G) * 128 * 2)
+        q, o = prep(), torch.empty(T, H * DV, dtype=torch.bfloat16, device="cuda")
+        if few:
+            pairs = keys = n_seq * ((ctx - 1) % size + 1)
+        else:
+            pairs, keys = sum(i % size + 1 for i in range(new)), 0
+        mixer = hd.MIXERS["sigmoid_attention"](at, cfg, 0, torch.bfloat16, "cuda")
+        ctxt = StepContext(meta, RotationFreqs())
+        case(tag + f"sigmoid attention in chunks of {size}", lambda: mixer.attend(q, c.pages[0], ctxt, None, o, 1.0),
+             keys * G * (D + DV) * 2, pairs * H * 2 * (D + DV))
+        case(tag + "  | softmax attention in a window, as many keys",
+             lambda: nat.window_attn(q, c.pages[0], grp, dims, size if few else size // 2, 0.09, few, o), keys * G * (D + DV) * 2,
+             n_seq * min(size, ctx) * H * 2 * (D + DV) if few else sum(min(i + 1, size // 2) for i in range(new)) * H * 2 * (D + DV))
+        q3 = _bf(T, H, 128)
+        case(tag + "  | paged attention, the same window", lambda: nat.paged_attn(q3, c3.k[0], c3.v[0], meta3, 0.09, size if few else size // 2),
+             keys * G * 512, n_seq * min(size, ctx) * H * 512 if few else sum(min(i + 1, size // 2) for i in range(new)) * H * 512)
+        del c, c3
+        # sums and norms, convolution, embedding, feed-forward
+        x, yo, lw, bias, xb, rw = f(T, W), _bf(T, W), f(W), f(W), _bf(T, W), _bf(W)
+        c, meta, grp = cache({"canon": ((cfg.taps - 1, W), None), "token": ((1,), torch.int32)})
+        taps, ring = f(cfg.taps, W), c.slots[0]["canon"]
+        case(tag + "norm + sum + norm", lambda: nat.branch_norm(x, 1e-5, 1.0, y=yo, bias=bias, wb=lw, wn=lw, out=x), T * W * (4 + 2 + 4 + 2))
+        if few:
+            conv = (taps, ring, meta.state_slots, meta.positions)
+            case(tag + "norm + sum + norm + convolution", lambda: nat.branch_norm(x, 1e-5, 1.0, y=yo, bias=bias, wb=lw, wn=lw, out=x, conv=conv),
+                 T * W * (4 + 2 + 4 + 2 + 2 * cfg.taps) + cfg.taps * W * 4)
+        else:
+            case(tag + "input convolution", lambda: nat.canon(yo, taps, ring, meta), 2 * T * W * 2)
+        case(tag + "  | residual sum + rms norm", lambda: nat.rmsnorm_fwd(xb, rw, 1e-6, yo), 4 * T * W * 2)
+        ids, tab, pos = torch.randint(0, 30000, (T,), device="cuda"), _bf(30000, W), _bf(cfg.max_positions, W)
+        case(tag + "embedding of pairs and positions", lambda: nat.pair_embed(ids, tab, tab, pos, meta, c.slots[0]["token"], (29999, 31, 5)),
+             T * W * (3 * 2 + 4))
+        case(tag + "  | embedding", lambda: nat.embed_scale(ids, tab, 1.0), T * W * (2 + 4 + 2))
+        wgu, bgu = _bf(2 * ff, W, scale=W ** -0.5), f(2 * ff)
+        if few:
+            case(tag + "gate/up mat-vec with biases", lambda: nat.gemv_ex(xb, wgu, bgu, (float("inf"), 1.0, 0.0), n=ff), 2 * ff * W * 2)
+            case(tag + "  | gate/up mat-vec, swiglu", lambda: nat.gemv(xb, wgu, swiglu=True), 2 * ff * W * 2)
+        else:
+            gu = _bf(T, 2 * ff)
+            case(tag + "gated unit with biases", lambda: nat.clamped_glu(gu, ff, float("inf"), 1.0, 0.0, bgu), 3 * T * ff * 2)
+            case(tag + "  | swiglu", lambda: nat.swiglu_fwd(gu), 3 * T * ff * 2)
+        del c
+        torch.cuda.empty_cache()
+    nat.check_status()
+    return out
+
+
 def kernel_cases(name: str, batch: int = 16, ctx: int = 4096, prompt: int = 4096) -> List[dict]:
     """Every kernel of the hybrid layers at the sizes of preset ``name`` and, behind it, the like kernel of the other
     models: bytes and operations that the computation needs, device time, fraction of the slower of the two bounds."""
@@ -489,11 +629,14 @@ def report(names: List[str], kernels: bool = True) -> dict:
         for kind in ("hybrid", like_kind(n)):
             m = build(n, kind)
             row[kind] = {"parameters": getattr(m, "size", None) or sum(p.numel() for p in m.parameters()), **throughput(m)}
+            if kind == "hybrid" and m.loop_in is not None:
+                row[kind]["weights_per_token"] = run_weights(m.cfg)
             del m
             torch.cuda.empty_cache()
         res["models"][n] = row
     if kernels:
         block = hd.HybridArgs.from_dict(hd.PRESETS[names[0]]).design.block
-        cases = {"post": kernel_cases, "parallel": parallel_kernel_cases, "branch": branch_kernel_cases}[block]
+        cases = {"post": kernel_cases, "parallel": parallel_kernel_cases, "branch": branch_kernel_cases,
+                 "sandwich": sandwich_kernel_cases}[block]
         res["kernels"] = {names[0]: cases(names[0])}
     return res

@@ -42,10 +42,12 @@ __device__ __forceinline__ float row_max(uint32_t taddr, int lo, int span) {
   return mx;
 }
 
-// p = exp2(s * a + b) for the 128 columns of this row, written as bf16 into the swizzled P tile; returns the row sum. kCap:
+// p = exp2(s * a + b) for the 128 columns of this row, written as bf16 into the swizzled P tile; returns the row sum. Capped:
 // p = exp2(b - c / (exp2(s * a) + 1)), a capped score in base 2 when c is twice the cap and b contains the cap
-// (tanh(x) = 1 - 2 / (exp(2 x) + 1)).
-template <bool kMask, bool kCap>
+// (tanh(x) = 1 - 2 / (exp(2 x) + 1)). Sigmoid weights: p = 1 / (1 + exp2(s * a + b)).
+enum : int { kFaPlain = 0, kFaCapped = 1, kFaSigmoid = 2 };
+
+template <bool kMask, int kMode>
 __device__ __forceinline__ float exp_rows(uint32_t taddr, uint32_t tile_addr, int r, float a, float b, int lo,
                                           int span, float c2 = 0.f) {
   float rs = 0.f;
@@ -58,7 +60,10 @@ __device__ __forceinline__ float exp_rows(uint32_t taddr, uint32_t tile_addr, in
 #pragma unroll
     for (int e = 0; e < 32; e += 2) {
       float p0, p1;
-      if (kCap) {
+      if (kMode == kFaSigmoid) {
+        p0 = fast_rcp(1.f + fast_exp2(fmaf(__uint_as_float(v[e]), a, b)));
+        p1 = fast_rcp(1.f + fast_exp2(fmaf(__uint_as_float(v[e + 1]), a, b)));
+      } else if (kMode == kFaCapped) {
         p0 = fast_exp2(fmaf(-c2, fast_rcp(fast_exp2(__uint_as_float(v[e]) * a) + 1.f), b));
         p1 = fast_exp2(fmaf(-c2, fast_rcp(fast_exp2(__uint_as_float(v[e + 1]) * a) + 1.f), b));
       } else {
@@ -233,8 +238,8 @@ attn_fwd_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_const
         break;
       }
       // pass 2: p = exp2(s * scale - m), row sum, bf16 P into shared memory (128B-swizzled, two 64-key boxes)
-      const float rs = need_mask ? exp_rows<true, false>(tmem_base + b * 128 + lane_off, sP_addr, r, sl2, -m_use, lo, span)
-                                 : exp_rows<false, false>(tmem_base + b * 128 + lane_off, sP_addr, r, sl2, -m_use, 0, 0);
+      const float rs = need_mask ? exp_rows<true, kFaPlain>(tmem_base + b * 128 + lane_off, sP_addr, r, sl2, -m_use, lo, span)
+                                 : exp_rows<false, kFaPlain>(tmem_base + b * 128 + lane_off, sP_addr, r, sl2, -m_use, 0, 0);
       l_run = l_run * corr + rs;
       fence_async_smem();        // generic-proxy writes of P -> visible to the tensor-core (async) proxy
       tc_fence_before();         // this thread's TMEM reads of S are complete
@@ -363,7 +368,7 @@ __device__ __forceinline__ int fa_work(int k) {
   return k * g + ((k & 1) ? g - 1 - c : c);
 }
 
-template <bool kCap>
+template <int kMode>
 __global__ void __launch_bounds__(kFaThreads2, 1)
 attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const FaParams p) {
@@ -497,6 +502,7 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int qd = warp & 3;
     const int r = qd * 32 + lane;
     const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
+    constexpr bool kCap = kMode == kFaCapped;
     const float cap2 = p.softcap * kFaLog2e;
     const float sl2 = kCap ? 2.f * kFaLog2e * p.scale / p.softcap : p.scale * kFaLog2e;
     const uint32_t s_tmem = tmem_base + grp * 128 + lane_off;
@@ -537,10 +543,10 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         // valid key columns of this row inside the tile: [lo, lo + span]; span < 0 means none
         const int lo = max(st - j0, 0);
         const int span = min(min(i + p.shift, p.Tk - 1) - j0, kFaTile - 1) - lo;
-        // pass 1 over S_b: row maximum
-        const float mx = need_mask ? row_max<true>(s_tmem, lo, span) : row_max<false>(s_tmem, 0, 0);
+        // pass 1 over S_b: row maximum (sigmoid weights need none: m_run stays 0)
+        const float mx = kMode == kFaSigmoid ? 0.f : (need_mask ? row_max<true>(s_tmem, lo, span) : row_max<false>(s_tmem, 0, 0));
         // the cap is monotone: the capped maximum is the maximum of the capped scores
-        const float mc = !kCap ? mx * sl2 : mx == -INFINITY ? mx : fmaf(-2.f * cap2, fast_rcp(fast_exp2(mx * sl2) + 1.f), cap2);
+        const float mc = kMode == kFaSigmoid ? 0.f : !kCap ? mx * sl2 : mx == -INFINITY ? mx : fmaf(-2.f * cap2, fast_rcp(fast_exp2(mx * sl2) + 1.f), cap2);
         const float m_cand = fmaxf(m_run, mc);
         // the previous tile's P·V must be complete: it read P_b and wrote O_b
         if (kk > 0 && !mbar_wait(&bar[kB2OFull + grp], (cnt - 1) & 1, abort_flag, p.status, kTimeoutEpilogue)) {
@@ -549,7 +555,7 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         }
         const bool grow = (m_run != -INFINITY) && (m_cand > m_run + kFaRescaleGap);
         if (m_run == -INFINITY) m_run = m_cand;          // nothing accumulated for this row yet (its O row is exactly 0)
-        if (kk > 0 && __any_sync(0xffffffffu, grow)) {
+        if (kMode != kFaSigmoid && kk > 0 && __any_sync(0xffffffffu, grow)) {
           tc_fence_after();
           const float corr = grow ? fast_exp2(m_run - m_cand) : 1.f;
           if (grow) { m_run = m_cand; l_run *= corr; }
@@ -566,9 +572,10 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         }
         const float m_use = (m_run == -INFINITY) ? 0.f : m_run;
         // pass 2 over S_b: p = exp2(s * scale - m), row sum, bf16 P into this group's shared-memory tile
-        const float shift2 = kCap ? cap2 - m_use : -m_use;
-        const float rs = need_mask ? exp_rows<true, kCap>(s_tmem, sP_addr, r, sl2, shift2, lo, span, 2.f * cap2)
-                                   : exp_rows<false, kCap>(s_tmem, sP_addr, r, sl2, shift2, 0, 0, 2.f * cap2);
+        const float shift2 = kMode == kFaSigmoid ? -p.wbias[it.h] * kFaLog2e : (kCap ? cap2 - m_use : -m_use);
+        const float a2 = kMode == kFaSigmoid ? -sl2 : sl2;
+        const float rs = need_mask ? exp_rows<true, kMode>(s_tmem, sP_addr, r, a2, shift2, lo, span, 2.f * cap2)
+                                   : exp_rows<false, kMode>(s_tmem, sP_addr, r, a2, shift2, 0, 0, 2.f * cap2);
         l_run += rs;
         fence_async_smem();        // generic-proxy writes of P -> visible to the tensor-core (async) proxy
         tc_fence_before();         // TMEM reads / writes of this thread are ordered before the MMA that follows the arrive
@@ -597,7 +604,7 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const float a_me = (m_me == -INFINITY) ? 0.f : fast_exp2(m_me - m);
         const float a_o = (m_o == -INFINITY) ? 0.f : fast_exp2(m_o - m);
         const float l = l_run * a_me + l_o * a_o + (p.sink ? fast_exp2(s2 - m) : 0.f);
-        float inv = l > 0.f ? 1.f / l : 0.f;
+        float inv = kMode == kFaSigmoid ? p.out_scale : (l > 0.f ? 1.f / l : 0.f);
         if (p.gate) inv /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(ic) * p.ldg + it.h]));
         const float w_me = a_me * inv, w_o = a_o * inv;
         __nv_bfloat16* orow = p.out + static_cast<long long>(ic) * p.o_stride + static_cast<long long>(it.h) * 128;
@@ -625,7 +632,7 @@ attn_fwd_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             }
           }
         }
-        if (grp == 0 && i < p.T) p.lse[static_cast<long long>(it.h) * p.T + i] = (m + log2f(l)) / kFaLog2e;
+        if (kMode != kFaSigmoid && grp == 0 && i < p.T) p.lse[static_cast<long long>(it.h) * p.T + i] = (m + log2f(l)) / kFaLog2e;
       }
       // both O buffers and both exchange areas are free again
       tc_fence_before();
@@ -661,8 +668,9 @@ using namespace pm;
 static int attn_fwd_tc_launch(int variant, const void* q, long long q_stride, const void* k, long long k_stride,
                               const void* v, long long v_stride, void* out, long long o_stride, float* lse,
                               const int* seq_start, int T, int Tk, int shift, int hq, int hkv, float scale, float softcap,
-                              const float* sink, const void* gate, long long ldg, int* status, cudaStream_t st) {
-  if (softcap < 0.f || (variant == 1 && (softcap > 0.f || sink || gate))) return -4;
+                              const float* sink, const void* gate, long long ldg, int* status, cudaStream_t st,
+                              const float* wbias = nullptr, float out_scale = 1.f) {
+  if (softcap < 0.f || (variant == 1 && (softcap > 0.f || sink || gate)) || (wbias && (variant == 1 || softcap > 0.f || sink))) return -4;
   if (hq % hkv || T <= 0 || Tk <= 0) return -1;
   if ((q_stride | k_stride | v_stride | o_stride) % 8) return -2;
   CUtensorMap mq, mk, mv;
@@ -677,15 +685,18 @@ static int attn_fwd_tc_launch(int variant, const void* q, long long q_stride, co
   p.T = T; p.hq = hq; p.hkv = hkv; p.scale = scale; p.status = status;
   p.Tk = Tk; p.shift = shift;
   p.softcap = softcap; p.sink = sink; p.gate = static_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
+  p.wbias = wbias; p.out_scale = out_scale;
   const int smem = 6 * kFaTileBytes + 1024 + 256;
   const int smem2 = 7 * kFaTileBytes + 1024 + 256;
   static DeviceOnce once;
   if (once.pending()) {
     cudaError_t e = cudaFuncSetAttribute(attn_fwd_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
-    e = cudaFuncSetAttribute(attn_fwd_tc2_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
+    e = cudaFuncSetAttribute(attn_fwd_tc2_kernel<kFaPlain>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
     if (e != cudaSuccess) return static_cast<int>(e);
-    e = cudaFuncSetAttribute(attn_fwd_tc2_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
+    e = cudaFuncSetAttribute(attn_fwd_tc2_kernel<kFaCapped>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    e = cudaFuncSetAttribute(attn_fwd_tc2_kernel<kFaSigmoid>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2);
     if (e != cudaSuccess) return static_cast<int>(e);
     once.mark();
   }
@@ -695,8 +706,9 @@ static int attn_fwd_tc_launch(int variant, const void* q, long long q_stride, co
   } else {
     const int items = static_cast<int>(grid.x) * hq;      // persistent: one CTA per SM walks the item list
     const int ctas = items < num_sms() ? items : num_sms();
-    if (softcap > 0.f) attn_fwd_tc2_kernel<true><<<ctas, kFaThreads2, smem2, st>>>(mq, mk, mv, p);
-    else attn_fwd_tc2_kernel<false><<<ctas, kFaThreads2, smem2, st>>>(mq, mk, mv, p);
+    if (wbias) attn_fwd_tc2_kernel<kFaSigmoid><<<ctas, kFaThreads2, smem2, st>>>(mq, mk, mv, p);
+    else if (softcap > 0.f) attn_fwd_tc2_kernel<kFaCapped><<<ctas, kFaThreads2, smem2, st>>>(mq, mk, mv, p);
+    else attn_fwd_tc2_kernel<kFaPlain><<<ctas, kFaThreads2, smem2, st>>>(mq, mk, mv, p);
   }
   return static_cast<int>(cudaGetLastError());
 }
@@ -717,6 +729,16 @@ extern "C" int pm_attn_fwd_tc_ex(const void* q, long long q_stride, const void* 
                                  const void* gate, long long ldg, int* status, cudaStream_t st) {
   return attn_fwd_tc_launch(2, q, q_stride, k, k_stride, v, v_stride, out, o_stride, lse, seq_start, T, Tk, shift, hq,
                             hkv, scale, softcap, sink, gate, ldg, status, st);
+}
+
+// The same with sigmoid weights: key j counts for head h with the sigmoid of its score + wbias[h] (fp32 [hq]), the sum is not divided
+// by anything and multiplied with out_scale.
+extern "C" int pm_attn_fwd_tc_sigmoid(const void* q, long long q_stride, const void* k, long long k_stride, const void* v,
+                                      long long v_stride, void* out, long long o_stride, const int* seq_start, int T, int Tk, int shift,
+                                      int hq, int hkv, float scale, const float* wbias, float out_scale, int* status, cudaStream_t st) {
+  if (!wbias) return -4;
+  return attn_fwd_tc_launch(2, q, q_stride, k, k_stride, v, v_stride, out, o_stride, nullptr, seq_start, T, Tk, shift, hq, hkv, scale, 0.f,
+                            nullptr, nullptr, 0, status, st, wbias, out_scale);
 }
 
 // Single-softmax-group variant of the same kernel (kept selectable for comparison measurements).

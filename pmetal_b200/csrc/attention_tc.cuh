@@ -28,6 +28,8 @@ struct FaParams {
   // forward kernel only: scores become softcap * tanh(score / softcap) when softcap > 0; sink [hq] (nullable) adds exp(sink_h) to
   // the softmax sum of head h; gate [T, ldg] (nullable) multiplies head h of the output by the sigmoid of column h
   float softcap;
+  const float* wbias;         // [hq], sigmoid weights: added to the scores
+  float out_scale;            // sigmoid weights: factor of the result
   const float* sink;
   const __nv_bfloat16* gate;
   long long ldg;

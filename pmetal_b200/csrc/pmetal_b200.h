@@ -64,6 +64,11 @@ int pm_attn_fwd_tc_ex(const void* q, long long q_stride, const void* k, long lon
     long v_stride, void* out, long long o_stride, float* lse, const int* seq_start, int T, int Tk, int shift, int
     hq, int hkv, float scale, float softcap, const float* sink, const void* gate, long long ldg, int* status,
     cudaStream_t st);
+// The same with sigmoid weights: key j counts for head h with the sigmoid of its score + wbias[h] (fp32 [hq]), the sum is not divided
+// by anything and multiplied with out_scale.
+int pm_attn_fwd_tc_sigmoid(const void* q, long long q_stride, const void* k, long long k_stride, const void* v,
+    long long v_stride, void* out, long long o_stride, const int* seq_start, int T, int Tk, int shift, int hq, int
+    hkv, float scale, const float* wbias, float out_scale, int* status, cudaStream_t st);
 // Single-softmax-group variant of the same kernel (kept selectable for comparison measurements).
 int pm_attn_fwd_tc_rect_v1(const void* q, long long q_stride, const void* k, long long k_stride, const void* v,
     long long v_stride, void* out, long long o_stride, float* lse, const int* seq_start, int T, int Tk, int shift,

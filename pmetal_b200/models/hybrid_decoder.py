@@ -402,7 +402,8 @@ class BranchLayer(nn.Module):
 
 
 class SandwichLayer(nn.Module):
-    """Norms before and after both sublayers and a convolution on the mixer's input; ``HybridDecoderLM._sandwich`` runs it."""
+    """Norms before and after both sublayers and a convolution on the mixer's input; ``HybridDecoderLM._sandwich`` forms the first norm
+    and the convolution, and adds what the last sublayer returns."""
 
     def __init__(self, spec: dict, cfg: HybridArgs, index: int, dtype, device):
         super().__init__()
@@ -430,6 +431,17 @@ class SandwichLayer(nn.Module):
             if mod is not None:
                 for name, *rest in mod.named_weights():
                     yield (pre + name, *rest)
+
+    def forward(self, x, h, cache, ctx, run):
+        """(fp32 stream, mixer input) -> (stream, what is left to add to it: the last sublayer's result, its bias, the weight of the
+        norm behind it)."""
+        from ..ops import native as nat
+        cfg = self.cfg
+        last = {"y": self.mixer(h, cache, ctx, run), "wb": self.norm1b_w}
+        if self.mlp is not None:
+            x, h = nat.branch_norm(x, cfg.norm_eps, cfg.design.norm_base, wn=self.norm2_w, out=x, **last)
+            last = {"y": self.mlp(h), "bias": self.mlp.b_down, "wb": self.norm2b_w}
+        return x, last
 
 
 class HybridDecoderLM(nn.Module):
@@ -661,11 +673,7 @@ class HybridDecoderLM(nn.Module):
 
         x, h = enter(0, x)
         for n, (i, _) in enumerate(self.runs):
-            layer = self.layers[i]
-            last = {"y": layer.mixer(h, cache, ctx, n), "wb": layer.norm1b_w}
-            if layer.mlp is not None:
-                x, h = nat.branch_norm(x, cfg.norm_eps, wn=layer.norm2_w, out=x, **last, **kw)
-                last = {"y": layer.mlp(h), "bias": layer.mlp.b_down, "wb": layer.norm2b_w}
+            x, last = self.layers[i](x, h, cache, ctx, n)
             if n + 1 < len(self.runs):
                 x, h = enter(n + 1, x, **last)
         if on_layer is not None:

@@ -50,7 +50,7 @@ class StepContext:
         self.meta, self.freqs = meta, freqs
         self._rope: Dict[tuple, tuple] = {}
         self._groups: Dict[int, tuple] = {}
-        self._runs: Dict[int, list] = {}
+        self._runs: Dict[tuple, list] = {}
 
     def rope(self, base: float, dims: int):
         key = (base, dims)
@@ -64,11 +64,13 @@ class StepContext:
             self._groups[limit] = split_groups(self.meta, limit)
         return self._groups[limit]
 
-    def runs(self, limit: int):
-        """The sequences with more than ``limit`` new tokens as launches of the flash-attention kernel."""
-        if limit not in self._runs:
-            self._runs[limit] = attention_runs(self.meta, self.groups(limit)[1])
-        return self._runs[limit]
+    def runs(self, limit: int, chunk: int = 0):
+        """The sequences with more than ``limit`` new tokens as launches of the flash-attention kernel; ``chunk`` > 0: tokens see their
+        own chunk of that many positions."""
+        key = (limit, chunk)
+        if key not in self._runs:
+            self._runs[key] = attention_runs(self.meta, self.groups(limit)[1], chunk)
+        return self._runs[key]
 
 
 class RotationFreqs:
@@ -468,17 +470,22 @@ class GroupedAttentionMixer(StackedMixer):
         pages = cache.pages[run if self.own and run is not None else self.source]
         cos, sin = ctx.rope(self.base, self.R) if self.R else (None, None)
         k_at = self.at.get("k", 0)
-        short, long = ctx.groups(SHORT)
-        wide = nat.window_wide(self.dims, u.dtype, self.window) if long is not None and not self.SIGMOID else 0
+        wide = nat.window_wide(self.dims, u.dtype, self.window, self.CHUNKED) if ctx.groups(SHORT)[1] is not None else 0
         q = nat.window_prep(u, cos, sin, self.dims, (self.R, self.ROTATION), self.UNIT_NORM, self.eps, (k_at, self.at.get("v", k_at)),
                             pages if self.own else None, ctx.meta.slots, self.q_norm_w, self.k_norm_w, self.temp, ctx.meta.positions, wide)
-        gate = u[:, self.at["g"]:] if self.GATE else None
+        self.attend(q, pages, ctx, u[:, self.at["g"]:] if self.GATE else None, o, scale)
+
+    def attend(self, q: torch.Tensor, pages, ctx: StepContext, gate, o: torch.Tensor, scale: float) -> None:
+        """Attention of prepared queries over the cached rows, short and long portions."""
+        from ..ops import native as nat
+        short, long = ctx.groups(SHORT)
         diff = (self.lam, 1.0 - self.diff, self.eps) if self.dims[2] > 1 else None
         more = (self.softcap, self.sink, gate, diff)
         if short is not None:
             nat.window_attn(q, pages, short, self.dims, self.window, self.scale, True, o, *more, self.CHUNKED, self.wbias, scale)
-        if long is not None and wide:
-            nat.window_expand_attn(q, pages, long, ctx.runs(SHORT), self.dims, self.scale, o, *more)
+        if long is not None and nat.window_wide(self.dims, q.dtype, self.window, self.CHUNKED):
+            runs = ctx.runs(SHORT, self.window if self.CHUNKED else 0)
+            nat.window_expand_attn(q, pages, long, runs, self.dims, self.scale, o, *more, self.wbias, scale)
         elif long is not None:
             nat.window_attn(q, pages, long, self.dims, self.window, self.scale, False, o, *more, self.CHUNKED, self.wbias, scale)
 

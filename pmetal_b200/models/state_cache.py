@@ -180,9 +180,10 @@ class AttnRun:
     shift: int
 
 
-def attention_runs(meta: BatchMeta, group: SeqGroup) -> List[AttnRun]:
+def attention_runs(meta: BatchMeta, group: SeqGroup, chunk: int = 0) -> List[AttnRun]:
     """A run begins with any sequence and takes in the next ones as long as their rows follow and they have no earlier tokens: then
-    every query row lies ``shift`` before its own key row, the earlier tokens of the first sequence."""
+    every query row lies ``shift`` before its own key row, the earlier tokens of the first sequence (``chunk`` > 0: those of its
+    chunk, as every query then sees the keys of its own chunk of positions alone)."""
     runs: List[List[Tuple[int, int, int, int]]] = []
     for s in group.host:
         i, q0, n, total = s
@@ -193,13 +194,20 @@ def attention_runs(meta: BatchMeta, group: SeqGroup) -> List[AttnRun]:
     out, dev = [], meta.slots.device
     for run in runs:
         i, q0, n0, total = run[0]
-        prior, n = total - n0, sum(s[2] for s in run)
+        first, n = total - n0, sum(s[2] for s in run)
+        key0 = first - first % chunk if chunk else 0          # position of the first key row
+        prior = first - key0
         slots = meta.slots[q0:q0 + n]
         if prior:
-            pages = meta.block_table[i, :-(-prior // BLOCK)].long()
-            old = (pages[:, None] * BLOCK + torch.arange(BLOCK, device=dev)).view(-1)[:prior]
+            b0 = key0 // BLOCK
+            pages = meta.block_table[i, b0:-(-first // BLOCK)].long()
+            old = (pages[:, None] * BLOCK + torch.arange(BLOCK, device=dev)).view(-1)[key0 - b0 * BLOCK:first - b0 * BLOCK]
             slots = torch.cat([old, slots])
         base = torch.tensor([0] + [s[1] - q0 + prior for s in run[1:]], dtype=torch.int32)
-        start = torch.repeat_interleave(base, torch.tensor([s[2] for s in run])).to(dev, non_blocking=True)
-        out.append(AttnRun(slice(q0, q0 + n), n, slots.contiguous(), start, prior))
+        start = torch.repeat_interleave(base, torch.tensor([s[2] for s in run]))
+        if chunk:
+            pos = torch.cat([torch.arange(t - m, t, dtype=torch.int32) for _, _, m, t in run])
+            at = torch.where(torch.arange(n) < n0, key0, 0)
+            start = start + (pos - pos % chunk - at).to(torch.int32)
+        out.append(AttnRun(slice(q0, q0 + n), n, slots.contiguous(), start.to(dev, non_blocking=True), prior))
     return out

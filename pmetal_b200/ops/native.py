@@ -710,6 +710,22 @@ def attn_fwd_rect(q, k, v, seq_start, scale: float, shift: int, out=None, softca
     return out, lse
 
 
+def attn_fwd_sigmoid(q, k, v, seq_start, scale: float, shift: int, wbias, out_scale: float = 1.0, out=None):
+    """``attn_fwd_rect`` with sigmoid weights in place of the softmax: a visible key counts with the sigmoid of its score + wbias (fp32
+    [hq]); the sum times ``out_scale``."""
+    T, hq, d = q.shape
+    Tk, hkv = k.shape[0], k.shape[1]
+    assert d == 128 and q.stride(1) == d and k.stride(1) == d and v.stride(1) == d
+    if out is None:
+        out = torch.empty(T, hq, d, dtype=q.dtype, device=q.device)
+    assert out.shape == q.shape and out.stride(1) == d
+    _chk(lib().pm_attn_fwd_tc_sigmoid(_p(q), c_ll(q.stride(0)), _p(k), c_ll(k.stride(0)), _p(v), c_ll(v.stride(0)), _p(out),
+                                      c_ll(out.stride(0)), _p(seq_start), c_int(T), c_int(Tk), c_int(shift), c_int(hq), c_int(hkv),
+                                      c_float(scale), _p(wbias), c_float(out_scale), _p(status_word(q.device)), _stream()),
+         "pm_attn_fwd_tc_sigmoid")
+    return out
+
+
 def attn_bwd(dout, q, k, v, o, lse, seq_start, scale: float, window: int = 0, dv_out=None):
     T, hq, d = q.shape
     hkv = k.shape[1]
@@ -1665,15 +1681,16 @@ def window_attn(q, pages, group, dims, window: int, scale: float, few: bool, out
     LAUNCHES += int(po is not None or o is not None)
 
 
-def window_wide(dims, dtype, window: int) -> int:
+def window_wide(dims, dtype, window: int, chunked: bool = False) -> int:
     """Row width of the queries of steps whose long portions take ``window_expand_attn``; 0 where they cannot."""
     _, _, M, D, DV = dims
-    fits = dtype == torch.bfloat16 and window == 0 and M * -(-D // 8) * 8 <= 128 and DV <= 128
+    fits = dtype == torch.bfloat16 and (window == 0 or chunked) and M * -(-D // 8) * 8 <= 128 and DV <= 128
     return 128 if fits else 0
 
 
-def window_expand_attn(q, pages, group, runs, dims, scale: float, out, softcap: float = 0.0, sink=None, gate=None, diff=None) -> None:
-    """``window_attn`` for long portions without a window: keys and values of the sequences of ``group`` in rows of 128 channels,
+def window_expand_attn(q, pages, group, runs, dims, scale: float, out, softcap: float = 0.0, sink=None, gate=None, diff=None,
+                       wbias=None, out_scale: float = 1.0) -> None:
+    """``window_attn`` for long portions without a window or in chunks (which the runs contain): keys and values of the sequences of ``group`` in rows of 128 channels,
     then the flash-attention kernel (maps side by side in a key, queries with zeros at the other maps' channels). q as
     ``window_prep`` leaves it with ``wide`` = 128; ``runs``: the group's sequences as ``AttnRun``s (models/state_cache.py)."""
     H, G, M, D, DV = dims
@@ -1686,6 +1703,9 @@ def window_expand_attn(q, pages, group, runs, dims, scale: float, out, softcap: 
         v128 = torch.empty_like(k128)
         _chk(lib().pm_window_expand(_p(pages), _p(run.slots), c_int(n_keys), c_int(G), c_int(M), c_int(D), c_int(DV), _p(k128),
                                     _p(v128), _stream()), "pm_window_expand")
+        if wbias is not None:
+            attn_fwd_sigmoid(q[run.rows], k128, v128, run.seq_start, scale, run.shift, wbias, out_scale, o[run.rows])
+            continue
         attn_fwd_rect(q[run.rows], k128, v128, run.seq_start, scale, run.shift, o[run.rows], softcap, sink,
                       gate[run.rows] if direct and gate is not None else None)
     if direct:

@@ -3,26 +3,32 @@ shares no code with the package: the tests compare the product path with it. ``p
 the parsed configuration; sequences are [T, width] with positions 0 .. T - 1.
 
 ``low`` marks every value that a bf16 model may hold in bf16 (projection inputs and outputs, what the input convolution leaves
-behind, normed queries and keys, cached rows, the heads' results, the gated units). It is the identity; inside ``rounding()`` it
-rounds to bf16, which shows how much of a difference such rounding alone explains."""
+behind, normed queries and keys, cached rows, attention weights as factors of the values, the heads' results, the gated units). It
+is the identity; inside ``rounding()`` it rounds to bf16, and inside ``rounding(seed)`` it moves every value by as much at random,
+which shows how much of a difference such rounding alone explains."""
 import contextlib
 
 import torch
 
-_ROUND = [False]
+_ROUND = [None]
 
 
 def low(x):
-    return x.to(torch.bfloat16).to(x.dtype) if _ROUND[0] else x
+    how = _ROUND[0]
+    if how is None:
+        return x
+    if how is True:
+        return x.to(torch.bfloat16).to(x.dtype)
+    return x * (1 + (2 * torch.rand(x.shape, generator=how, dtype=x.dtype) - 1) * 2.0 ** -9)
 
 
 @contextlib.contextmanager
-def rounding():
-    _ROUND[0] = True
+def rounding(seed=None):
+    _ROUND[0] = True if seed is None else torch.Generator().manual_seed(seed)
     try:
         yield
     finally:
-        _ROUND[0] = False
+        _ROUND[0] = None
 
 
 def linear(x, w, b=None):
@@ -110,7 +116,7 @@ def visible(T, chunk):
 def sigmoid_attend(q, k, v, scale, bias, seen):
     """One head: every visible key counts with the sigmoid of its score; nothing is divided by the sum of the weights."""
     w = 1 / (1 + torch.exp(-((q @ k.t()) * scale + bias)))
-    return torch.where(seen, w, torch.zeros_like(w)) @ v
+    return low(torch.where(seen, w, torch.zeros_like(w))) @ v
 
 
 def sigmoid_attention(h, p, pre, m, eps):
