@@ -276,80 +276,134 @@ struct ChannelBlockParams {
   int H, N, n16;
 };
 
-constexpr int kBlockTokens = 64, kBlockThreads = 256;
+constexpr int kBlockTokens = 64, kBlockThreads = 256, kBlockCols = 128;
 
-// grid (blocks of the longest portion, H, sequences)
+// 2^x, small results flushed to zero
+__device__ __forceinline__ float pow2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// channel_gate through the fast exponential and division, for sums of bf16 terms, and log2 f (no less than kMinLog2): close to one by
+// the series of log(1 - g).
+__device__ __forceinline__ float channel_gate_fast(float z, float lower, float& g) {
+  const float e = __expf(-fabsf(z)), big = __fdividef(1.f, 1.f + e), small = e * big;
+  const float f = fmaf(1.f - lower, z >= 0.f ? big : small, lower);
+  g = (1.f - lower) * (z >= 0.f ? small : big);
+  const float near = -g * kLog2e * fmaf(g, fmaf(g, fmaf(g, fmaf(g, fmaf(g, 1.f / 6.f, 0.2f), 0.25f), 1.f / 3.f), 0.5f), 1.f);
+  return fmaxf(g < 0.0625f ? near : __log2f(f), kMinLog2);
+}
+
+// Four consecutive elements from element n of a row; those from `end` on are zero.
+template <bool VEC, typename T>
+__device__ __forceinline__ void load_four(const T* row, int n, int end, float (&v)[4]) {
+  if (VEC) {
+    load_vec<4>(row + n, v);
+  } else {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = n + e < end ? to_f(row[n + e]) : 0.f;
+  }
+}
+
+// grid (blocks of the longest portion, H, sequences). A warp forms the operands of 8 tokens, 4 channels per lane and pass. VEC: heads
+// are whole 16-byte pieces of all rows.
+template <bool VEC>
 __global__ void __launch_bounds__(kBlockThreads) channel_block_kernel(const ChannelBlockParams p) {
   extern __shared__ __align__(16) uint8_t cb_smem[];
   const int seq = blockIdx.z, h = blockIdx.y, t0 = blockIdx.x * kBlockTokens, len = p.q_lens[seq] - t0;
   if (len <= 0) return;
-  const int n16 = p.n16, ldc = n16 + 8, ldn = n16 + 8, pairs = n16 / 2;
+  const int n16 = p.n16, ldc = n16 + 8, ldq = n16 + 8, ldk = 4 * n16 + 16;              // ldk: bytes
   float* sc = reinterpret_cast<float*>(cb_smem);                                        // [64][ldc] running sums of log2 f
-  __nv_bfloat16* sKh = reinterpret_cast<__nv_bfloat16*>(sc + kBlockTokens * ldc);       // [64][ldn]
-  __nv_bfloat16* sKl = sKh + kBlockTokens * ldn;
-  __nv_bfloat16* sQ = sKl + kBlockTokens * ldn;
+  float* sT = sc + kBlockTokens * ldc;                                                  // [8][128] their growth over 8 tokens
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(sT + 8 * kBlockCols);            // [64][ldq]
+  uint8_t* sK = reinterpret_cast<uint8_t*>(sQ + kBlockTokens * ldq);                    // [64][ldk]: keys, their second terms
   const long long row0 = p.q_start[seq] + t0;
-  const int col0 = h * p.N, tid = threadIdx.x;
-  for (int i = tid; i < kBlockTokens * n16; i += kBlockThreads) {
-    const int j = i / n16, n = i - j * n16;
-    float l = 0.f;
-    if (j < len && n < p.N) {
-      float f, g;
-      channel_gate(p.z[(row0 + j) * p.ldz + col0 + n] + p.bias[col0 + n], p.lower[col0 + n], f, g);
-      l = log2_gate(f, g);
+  const int col0 = h * p.N, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, HN = p.H * n16;
+  for (int n0 = 0; n0 < n16; n0 += kBlockCols) {
+    const int n = n0 + lane * 4;
+    const bool live = n < p.N;
+    float bias[4] = {}, lower[4] = {}, c[8][4], g[8][4], run[4] = {};
+    if (live) {
+      load_four<VEC>(p.bias + col0, n, p.N, bias);
+      load_four<VEC>(p.lower + col0, n, p.N, lower);
     }
-    sc[j * ldc + n] = l;
-  }
-  __syncthreads();
-  const long long block = p.c_start[seq] / kBlockTokens + seq + blockIdx.x;
-  for (int n = tid; n < n16; n += kBlockThreads) {
-    float c = 0.f;
-#pragma unroll 16
-    for (int j = 0; j < kBlockTokens; ++j) {
-      c += sc[j * ldc + n];
-      sc[j * ldc + n] = c;
-    }
-    p.block_decay[(block * p.H + h) * n16 + n] = exp2f(c);
-  }
-  __syncthreads();
-  const int HN = p.H * n16;
-  for (int i = tid; i < kBlockTokens * pairs; i += kBlockThreads) {
-    const int j = i / pairs, n = (i - j * pairs) * 2;
-    float q[2] = {0.f, 0.f}, g[2] = {0.f, 0.f};
-    if (j < len)
 #pragma unroll
-      for (int e = 0; e < 2; ++e)
-        if (n + e < p.N) {
-          float f;
-          channel_gate(p.z[(row0 + j) * p.ldz + col0 + n + e] + p.bias[col0 + n + e], p.lower[col0 + n + e], f, g[e]);
-          q[e] = silu_f(__bfloat162float(p.q[(row0 + j) * p.ldu + col0 + n + e]));
-        }
-    const uint32_t qb = pack_bf16(q[0], q[1]);
-    q[0] = __uint_as_float(qb << 16);
-    q[1] = __uint_as_float(qb & 0xffff0000u);
-    const float2 c = *reinterpret_cast<const float2*>(sc + j * ldc + n);
-    const float2 mid = *reinterpret_cast<const float2*>(sc + ((j & ~7) + 3) * ldc + n);
-    const float2 end = *reinterpret_cast<const float2*>(sc + (kBlockTokens - 1) * ldc + n);
-    uint32_t hi, lo;
-    ms_split(g[0] * exp2f(mid.x - c.x), g[1] * exp2f(mid.y - c.y), hi, lo);
-    *reinterpret_cast<uint32_t*>(sKh + j * ldn + n) = hi;
-    *reinterpret_cast<uint32_t*>(sKl + j * ldn + n) = lo;
-    *reinterpret_cast<uint32_t*>(sQ + j * ldn + n) = qb;
-    if (j >= len) continue;
-    __nv_bfloat16* dst = p.act + (row0 + j) * 4 * HN + h * n16 + n;
-    ms_split(q[0] * exp2f(c.x), q[1] * exp2f(c.y), hi, lo);
-    *reinterpret_cast<uint32_t*>(dst) = hi;
-    *reinterpret_cast<uint32_t*>(dst + HN) = lo;
-    ms_split(g[0] * exp2f(end.x - c.x), g[1] * exp2f(end.y - c.y), hi, lo);
-    *reinterpret_cast<uint32_t*>(dst + 2 * HN) = hi;
-    *reinterpret_cast<uint32_t*>(dst + 3 * HN) = lo;
+    for (int r = 0; r < 8; ++r) {
+      const int j = warp * 8 + r;
+      float z[4];
+      const bool ok = live && j < len;
+      if (ok) load_four<VEC>(p.z + (row0 + j) * p.ldz + col0, n, p.N, z);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        g[r][e] = 0.f;
+        if (ok && (VEC || n + e < p.N)) run[e] += channel_gate_fast(z[e] + bias[e], lower[e], g[r][e]);
+        c[r][e] = run[e];
+      }
+    }
+    *reinterpret_cast<float4*>(sT + warp * kBlockCols + lane * 4) = make_float4(run[0], run[1], run[2], run[3]);
+    __syncthreads();
+    float before[4] = {}, total[4] = {};
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+      const float4 t = *reinterpret_cast<const float4*>(sT + w * kBlockCols + lane * 4);
+      const float v[4] = {t.x, t.y, t.z, t.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (w < warp) before[e] += v[e];
+        total[e] += v[e];
+      }
+    }
+    __syncthreads();                                         // sT may be written again
+    if (n >= n16) continue;
+    if (warp == 0) {
+      const long long block = p.c_start[seq] / kBlockTokens + seq + blockIdx.x;
+      *reinterpret_cast<float4*>(p.block_decay + (block * p.H + h) * n16 + n) = make_float4(pow2(total[0]), pow2(total[1]), pow2(total[2]), pow2(total[3]));
+    }
+    const float mid[4] = {c[3][0], c[3][1], c[3][2], c[3][3]};
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const int j = warp * 8 + r;
+      float q[4] = {}, v[4];
+      if (live && j < len) load_four<VEC>(p.q + (row0 + j) * p.ldu + col0, n, p.N, q);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) q[e] = silu_fast(q[e]);
+      const uint2 qb = make_uint2(pack_bf16(q[0], q[1]), pack_bf16(q[2], q[3]));
+      q[0] = __uint_as_float(qb.x << 16); q[1] = __uint_as_float(qb.x & 0xffff0000u);
+      q[2] = __uint_as_float(qb.y << 16); q[3] = __uint_as_float(qb.y & 0xffff0000u);
+      uint2 hi, lo;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = g[r][e] * pow2(mid[e] - c[r][e]);
+      ms_split(v[0], v[1], hi.x, lo.x);
+      ms_split(v[2], v[3], hi.y, lo.y);
+      *reinterpret_cast<uint2*>(sQ + j * ldq + n) = qb;
+      *reinterpret_cast<uint2*>(sK + j * ldk + n * 2) = hi;
+      *reinterpret_cast<uint2*>(sK + j * ldk + (n16 + n) * 2) = lo;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) c[r][e] += before[e];
+      *reinterpret_cast<float4*>(sc + j * ldc + n) = make_float4(c[r][0], c[r][1], c[r][2], c[r][3]);
+      if (j >= len) continue;
+      __nv_bfloat16* dst = p.act + (row0 + j) * 4 * HN + h * n16 + n;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = q[e] * pow2(c[r][e]);
+      ms_split(v[0], v[1], hi.x, lo.x);
+      ms_split(v[2], v[3], hi.y, lo.y);
+      *reinterpret_cast<uint2*>(dst) = hi;
+      *reinterpret_cast<uint2*>(dst + HN) = lo;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = g[r][e] * pow2(total[e] - c[r][e]);
+      ms_split(v[0], v[1], hi.x, lo.x);
+      ms_split(v[2], v[3], hi.y, lo.y);
+      *reinterpret_cast<uint2*>(dst + 2 * HN) = hi;
+      *reinterpret_cast<uint2*>(dst + 3 * HN) = lo;
+    }
   }
   __syncthreads();
 
   // scores: a warp owns 16 queries and every second tile of 8 keys
-  const int warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3, I = warp & 3, par = warp >> 2, r0 = I * 16;
+  const int g4 = lane >> 2, t4 = lane & 3, I = warp & 3, par = warp >> 2, r0 = I * 16;
   if (r0 >= len) return;
-  const uint32_t aKh = ms_addr(sKh), aKl = ms_addr(sKl);
+  const uint32_t aK = ms_addr(sK);
   float s[4][4];
 #pragma unroll
   for (int i = 0; i < 4; ++i)
@@ -361,7 +415,7 @@ __global__ void __launch_bounds__(kBlockThreads) channel_block_kernel(const Chan
 #pragma unroll
     for (int a = 0; a < 4; ++a) {
       const int row = r0 + g4 + 8 * (a & 1), n = k0 + 2 * t4 + 8 * (a >> 1);
-      const uint32_t qb = *reinterpret_cast<const uint32_t*>(sQ + row * ldn + n);
+      const uint32_t qb = *reinterpret_cast<const uint32_t*>(sQ + row * ldq + n);
       q[2 * a] = __uint_as_float(qb << 16);
       q[2 * a + 1] = __uint_as_float(qb & 0xffff0000u);
       const float2 v = *reinterpret_cast<const float2*>(sc + row * ldc + n);
@@ -376,7 +430,7 @@ __global__ void __launch_bounds__(kBlockThreads) channel_block_kernel(const Chan
       ci[2 * a + 1] = v.y;
     }
 #pragma unroll
-    for (int a = 0; a < 8; ++a) qd[a] = q[a] * exp2f(c[a] - ci[(a >> 2) * 2 + (a & 1)]);
+    for (int a = 0; a < 8; ++a) qd[a] = q[a] * pow2(c[a] - ci[(a >> 2) * 2 + (a & 1)]);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int J = 2 * i + par;
@@ -391,22 +445,21 @@ __global__ void __launch_bounds__(kBlockThreads) channel_block_kernel(const Chan
       if (i < I) {
         float f[4];
 #pragma unroll
-        for (int a = 0; a < 4; ++a) f[a] = exp2f(ci[a] - mid[a]);
+        for (int a = 0; a < 4; ++a) f[a] = pow2(ci[a] - mid[a]);
 #pragma unroll
         for (int a = 0; a < 8; ++a) v[a] = qd[a] * f[(a >> 2) * 2 + (a & 1)];
       } else {
 #pragma unroll
-        for (int a = 0; a < 8; ++a) v[a] = q[a] * exp2f(c[a] - mid[(a >> 2) * 2 + (a & 1)]);
+        for (int a = 0; a < 8; ++a) v[a] = q[a] * pow2(c[a] - mid[(a >> 2) * 2 + (a & 1)]);
       }
-      uint32_t fh[4], fl[4], b0, b1;
+      uint32_t fh[4], fl[4], kb[4];
 #pragma unroll
       for (int a = 0; a < 4; ++a) ms_split(v[2 * a], v[2 * a + 1], fh[a], fl[a]);
-      const uint32_t at = static_cast<uint32_t>(((8 * J + (lane & 7)) * ldn + k0 + ((lane >> 3) & 1) * 8) * 2);
-      ms_ldsm2(aKh + at, b0, b1);
-      ms_mma(s[i], fh, b0, b1);
-      ms_mma(s[i], fl, b0, b1);
-      ms_ldsm2(aKl + at, b0, b1);
-      ms_mma(s[i], fh, b0, b1);
+      // lanes 0 - 15: the keys' halves of 16 channels, 16 - 31: those of the second terms
+      ms_ldsm4(aK + static_cast<uint32_t>((8 * J + (lane & 7)) * ldk + (k0 + ((lane >> 3) & 1) * 8 + (lane >> 4) * n16) * 2), kb);
+      ms_mma(s[i], fh, kb[0], kb[1]);
+      ms_mma(s[i], fl, kb[0], kb[1]);
+      ms_mma(s[i], fh, kb[2], kb[3]);
     }
   }
 #pragma unroll
@@ -504,14 +557,17 @@ extern "C" int pm_channel_chunk(const void* q, const void* v, long long ldu, con
   const int n16 = (N + 15) / 16 * 16;
   const ChannelBlockParams b{static_cast<const __nv_bfloat16*>(q), ldu, z, ldz, bias, lower, q_start, q_lens, c_start,
                              static_cast<__nv_bfloat16*>(act), static_cast<__nv_bfloat16*>(score), block_decay, H, N, n16};
-  const size_t smem = static_cast<size_t>(kBlockTokens) * (n16 + 8) * (4 + 3 * 2);
-  static DeviceMax configured;
-  if (smem > configured.get()) {
-    const cudaError_t e = cudaFuncSetAttribute(channel_block_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+  const size_t smem = static_cast<size_t>(kBlockTokens) * ((n16 + 8) * (4 + 2) + 4 * n16 + 16) + 8 * kBlockCols * sizeof(float);
+  const bool vec = N % 4 == 0 && ldu % 4 == 0 && ldz % 4 == 0 && reinterpret_cast<uintptr_t>(q) % 8 == 0 &&
+                   (reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(lower)) % 16 == 0;
+  const auto kernel = vec ? channel_block_kernel<true> : channel_block_kernel<false>;
+  static DeviceMax configured[2];
+  if (smem > configured[vec].get()) {
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
-    configured.set(smem);
+    configured[vec].set(smem);
   }
-  channel_block_kernel<<<dim3((max_q + kBlockTokens - 1) / kBlockTokens, H, n_seq), kBlockThreads, smem, st>>>(b);
+  kernel<<<dim3((max_q + kBlockTokens - 1) / kBlockTokens, H, n_seq), kBlockThreads, smem, st>>>(b);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return static_cast<int>(e);
   SsdParams p{};

@@ -21,17 +21,19 @@
 namespace pm {
 
 constexpr int kChunk = 64;
-constexpr int kSlice = 32;            // channels of P per CTA
+constexpr int kSlice = 32;            // channels of P per group of four warps
 constexpr int kLdX = kSlice + 8;
 constexpr int kLdA = kChunk + 8;
 constexpr float kLog2e = 1.4426950408889634f;
 
-// Rows t0 .. t0 + 63 of `act` (lda apart), `width` columns from c0 (multiple of 8, zero filled beyond valid_w and beyond the portion).
-__device__ __forceinline__ void ssd_load_rows(const __nv_bfloat16* act, long long lda, bool aligned, __nv_bfloat16* dst, int ld,
+// Rows t0 .. t0 + 63 of `act` (lda apart), `width` columns from c0 (multiple of 8, zero filled beyond valid_w and beyond the portion), by
+// NT threads, of which this is number tid.
+template <int NT>
+__device__ __forceinline__ void ssd_load_rows(int tid, const __nv_bfloat16* act, long long lda, bool aligned, __nv_bfloat16* dst, int ld,
                                               int width, int valid_w, int c0, long long q0, int t0, int len) {
   if (aligned) {
-    const int per = width / 8, dr = 128 / per, dc = 128 - dr * per;
-    int r = threadIdx.x / per, c = threadIdx.x - r * per;
+    const int per = width / 8, dr = NT / per, dc = NT - dr * per;
+    int r = tid / per, c = tid - r * per;
     for (; r < kChunk; r += dr, c += dc) {
       if (c >= per) {
         c -= per;
@@ -42,7 +44,7 @@ __device__ __forceinline__ void ssd_load_rows(const __nv_bfloat16* act, long lon
       ms_cp16(ms_addr(dst + r * ld + c * 8), src, ok);
     }
   } else {
-    for (int i = threadIdx.x; i < kChunk * width; i += 128) {
+    for (int i = tid; i < kChunk * width; i += NT) {
       const int r = i / width, c = i - r * width;
       const bool ok = t0 + r < len && c < valid_w;
       dst[r * ld + c] = ok ? act[(q0 + t0 + r) * lda + c0 + c] : __float2bfloat16(0.f);
@@ -163,42 +165,44 @@ __device__ __forceinline__ void ssd_norm_add(float (&n)[2], float keep, const fl
   }
 }
 
-// What every segment but the last adds to the state, with segment-parallel CTAs. grid (slices * n_seg, H, sequences).
-template <int NI, bool SPLIT, int KIND>
-__global__ void __launch_bounds__(128) ssd_segment_kernel(const SsdParams p) {
+// What every segment but the last adds to the state, with segment-parallel CTAs. A CTA has WG groups of four warps, each with a slice
+// of P, on the same B. grid (slices / WG * n_seg, H, sequences).
+template <int NI, bool SPLIT, int KIND, int WG>
+__global__ void __launch_bounds__(128 * WG) ssd_segment_kernel(const SsdParams p) {
+  constexpr int NT = 128 * WG;
   constexpr bool MEMORY = KIND == kSsdMemory, CHANNEL = KIND == kSsdChannel;
   extern __shared__ __align__(16) uint8_t ssd_smem[];
   const SsdParams& d = p;
-  const int slices = gridDim.x / p.n_seg;
-  const int seq = blockIdx.z, h = blockIdx.y, p0 = (blockIdx.x % slices) * kSlice, seg = blockIdx.x / slices;
+  const int slices = gridDim.x / p.n_seg, grp = threadIdx.x >> 7, gt = threadIdx.x & 127;
+  const int seq = blockIdx.z, h = blockIdx.y, p0 = (blockIdx.x % slices * WG + grp) * kSlice, seg = blockIdx.x / slices;
   const int len = p.q_lens[seq];
   const int n_chunks = (len + kChunk - 1) / kChunk;
   if ((seg + 1) * p.seg_chunks >= n_chunks) return;            // the last segment is summed by the main kernel
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = gt >> 5, lane = threadIdx.x & 31;
   const int ldn = p.n16 + 8, tile_n = kChunk * ldn, tile_x = kChunk * kLdX;
   __nv_bfloat16* sB = reinterpret_cast<__nv_bfloat16*>(ssd_smem);        // [2][64][ldn]
   __nv_bfloat16* sBl = sB + 2 * tile_n;                                  // [2][64][ldn] (SPLIT)
-  __nv_bfloat16* sX = sB + (SPLIT ? 4 : 2) * tile_n;                     // [2][64][kLdX]
-  float* sDt = reinterpret_cast<float*>(sX + 2 * tile_x);                // [2][64]
-  float* cum = sDt + 2 * kChunk + warp * kChunk;                         // [4 warps][64]
-  float* wgt = sDt + 6 * kChunk + warp * kChunk;                         // [4 warps][64]
-  float* sLd = sDt + 10 * kChunk;                                        // [2][64] (MEMORY) or the blocks' decays [2][n16] (CHANNEL)
+  __nv_bfloat16* sX = sB + (SPLIT ? 4 : 2) * tile_n + grp * 2 * tile_x;  // [WG][2][64][kLdX]
+  float* sDt = reinterpret_cast<float*>(sB + (SPLIT ? 4 : 2) * tile_n + WG * 2 * tile_x);      // [2][64]
+  float* cum = sDt + 2 * kChunk + (threadIdx.x >> 5) * kChunk;           // [4 WG warps][64]
+  float* wgt = cum + 4 * WG * kChunk;                                    // [4 WG warps][64]
+  float* sLd = sDt + (2 + 8 * WG) * kChunk;                              // [2][64] (MEMORY) or the blocks' decays [2][n16] (CHANNEL)
   const long long q0 = p.q_start[seq];
   const int start = p.seq_lens[seq] - len;
   const int g = h / (d.H / d.G);
-  const int cx = h * d.P + p0, cb = d.b0 + g * d.NB, pw = min(kSlice, d.P - p0);
+  const int cx = h * d.P + p0, cb = d.b0 + g * d.NB, pw = max(0, min(kSlice, d.P - p0));
   const float a2 = KIND == kSsdPlain ? ssd_rate(p, h) : 0.f;
   const bool norm = MEMORY && p0 == 0;                                   // this CTA keeps the head's normaliser
   const long long mat = static_cast<long long>(d.N) * d.P4;
   auto slot_of = [&](int k) { return (static_cast<long long>(seq) * p.n_seg + k) * d.H + h; };
   auto load_chunk = [&](int ch, int buf) {
     const int t0 = ch * kChunk;
-    ssd_load_rows(p.act, p.ld, p.aligned, sB + buf * tile_n, ldn, p.n16, d.N, cb, q0, t0, len);
-    if (SPLIT) ssd_load_rows(p.act, p.ld, p.aligned, sBl + buf * tile_n, ldn, p.n16, d.N, cb + d.lo, q0, t0, len);
-    ssd_load_rows(p.x, p.ldx, p.aligned_x, sX + buf * tile_x, kLdX, kSlice, pw, cx, q0, t0, len);
+    ssd_load_rows<NT>(threadIdx.x, p.act, p.ld, p.aligned, sB + buf * tile_n, ldn, p.n16, d.N, cb, q0, t0, len);
+    if (SPLIT) ssd_load_rows<NT>(threadIdx.x, p.act, p.ld, p.aligned, sBl + buf * tile_n, ldn, p.n16, d.N, cb + d.lo, q0, t0, len);
+    ssd_load_rows<128>(gt, p.x, p.ldx, p.aligned_x, sX + buf * tile_x, kLdX, kSlice, pw, cx, q0, t0, len);
     if (CHANNEL) {
       const long long block = p.c_start[seq] / kChunk + seq + ch;
-      for (int n = threadIdx.x; n < p.n16; n += 128) sLd[buf * p.n16 + n] = p.block_decay[(block * d.H + h) * d.NB + n];
+      for (int n = threadIdx.x; n < p.n16; n += NT) sLd[buf * p.n16 + n] = p.block_decay[(block * d.H + h) * d.NB + n];
     } else if (threadIdx.x < kChunk) {
       sDt[buf * kChunk + threadIdx.x] = p.dt ? p.dt[(q0 + t0 + threadIdx.x) * d.H + h] : 1.f;
       if (MEMORY) sLd[buf * kChunk + threadIdx.x] = p.ldec[(q0 + t0 + threadIdx.x) * d.H + h];
@@ -259,57 +263,55 @@ __global__ void __launch_bounds__(128) ssd_segment_kernel(const SsdParams p) {
       if (static_cast<int>(threadIdx.x) + 128 * i < d.N) p.seg_n[slot_of(seg + 1) * d.N + threadIdx.x + 128 * i] = nacc[i];
 }
 
-// NI: state row tiles (16 rows) per warp; 4 warps cover N <= 64 NI. Same grid as ssd_segment_kernel.
-template <int NI, bool SPLIT, int KIND>
-__global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
+// NI: state row tiles (16 rows) per warp; 4 warps cover N <= 64 NI. Same grid as ssd_segment_kernel. The next block's C, scores and x are
+// copied while the state is updated, its B (which the scores need unless they come from the caller) behind that.
+template <int NI, bool SPLIT, int KIND, int WG>
+__global__ void __launch_bounds__(128 * WG) ssd_chunk_kernel(const SsdParams p) {
+  constexpr int NT = 128 * WG;
   constexpr bool MEMORY = KIND == kSsdMemory, CHANNEL = KIND == kSsdChannel;
   extern __shared__ __align__(16) uint8_t ssd_smem[];
   const SsdParams& d = p;
-  const int slices = gridDim.x / p.n_seg;
-  const int seq = blockIdx.z, h = blockIdx.y, p0 = (blockIdx.x % slices) * kSlice, seg = blockIdx.x / slices;
+  const int slices = gridDim.x / p.n_seg, grp = threadIdx.x >> 7, gt = threadIdx.x & 127;
+  const int seq = blockIdx.z, h = blockIdx.y, p0 = (blockIdx.x % slices * WG + grp) * kSlice, seg = blockIdx.x / slices;
   const int len = p.q_lens[seq];
   const int n_chunks = (len + kChunk - 1) / kChunk, ch0 = seg * p.seg_chunks, ch1 = min(n_chunks, ch0 + p.seg_chunks);
   if (ch0 >= ch1) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, t4 = lane & 3;
+  const int warp = gt >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, t4 = lane & 3;
   const int ldn = p.n16 + 8, tile_n = kChunk * ldn, tile_x = kChunk * kLdX;
   __nv_bfloat16* sC = reinterpret_cast<__nv_bfloat16*>(ssd_smem);        // [64][ldn]
   __nv_bfloat16* sB = sC + tile_n;                                       // [64][ldn]
   __nv_bfloat16* sCl = sB + tile_n;                                      // [64][ldn] (SPLIT)
   __nv_bfloat16* sBl = sCl + tile_n;                                     // [64][ldn] (SPLIT)
-  __nv_bfloat16* sX = sB + (SPLIT ? 3 : 1) * tile_n;                     // [64][kLdX]
-  __nv_bfloat16* sSh = sX + tile_x;                                      // [n16][kLdX]
+  const int own = 2 * tile_x + 2 * p.n16 * kLdX;                         // what a group keeps by itself
+  __nv_bfloat16* sX = sB + (SPLIT ? 3 : 1) * tile_n + grp * own;         // [2][64][kLdX]
+  __nv_bfloat16* sSh = sX + 2 * tile_x;                                  // [n16][kLdX]
   __nv_bfloat16* sSl = sSh + p.n16 * kLdX;                               // [n16][kLdX]
-  __nv_bfloat16* sA = sSl + p.n16 * kLdX;                                // [2][64][kLdA] (CHANNEL)
+  __nv_bfloat16* sA = sB + (SPLIT ? 3 : 1) * tile_n + WG * own;          // [2][64][kLdA] (CHANNEL)
   float* sDt = reinterpret_cast<float*>(sA + (CHANNEL ? 2 * kChunk * kLdA : 0));      // [64]
-  float* cum = sDt + kChunk + warp * kChunk;                             // [4 warps][64]
-  float* wgt = sDt + 5 * kChunk + warp * kChunk;                         // [4 warps][64]
-  float* sLd = sDt + 9 * kChunk;                                         // [64] (MEMORY) or the block's decays [n16] (CHANNEL)
+  float* cum = sDt + kChunk + (threadIdx.x >> 5) * kChunk;               // [4 WG warps][64]
+  float* wgt = cum + 4 * WG * kChunk;                                    // [4 WG warps][64]
+  float* sLd = sDt + (1 + 8 * WG) * kChunk;                              // [64] (MEMORY) or the block's decays [n16] (CHANNEL)
   float* sN = sLd + kChunk;                                              // [n16] (MEMORY)
 
   const long long q0 = p.q_start[seq];
   const int start = p.seq_lens[seq] - len;
   const int g = h / (d.H / d.G);
   const int cx = h * d.P + p0, cb = d.b0 + g * d.NB, cc = d.c0 + g * d.NB;
-  const int pw = min(kSlice, d.P - p0);
+  const int pw = max(0, min(kSlice, d.P - p0));
   const float a2 = KIND == kSsdPlain ? ssd_rate(p, h) : 0.f, skip = p.dskip ? p.dskip[h] : 0.f;
   const bool norm = MEMORY && p0 == 0;                                   // this CTA keeps the head's normaliser
   const long long mat = static_cast<long long>(d.N) * d.P4;
   float* st = p.state + (static_cast<long long>(p.slots[seq]) * d.H + h) * mat + p0;
 
-  auto load_chunk = [&](int ch) {
+  auto load_c = [&](int ch) {               // C, scores, x (the buffer of the block's parity), steps and decays of the tokens
     const int t0 = ch * kChunk;
-    ssd_load_rows(p.act, p.ld, p.aligned, sC, ldn, p.n16, d.N, cc, q0, t0, len);
-    ssd_load_rows(p.act, p.ld, p.aligned, sB, ldn, p.n16, d.N, cb, q0, t0, len);
-    if (SPLIT) {
-      ssd_load_rows(p.act, p.ld, p.aligned, sCl, ldn, p.n16, d.N, cc + d.lo, q0, t0, len);
-      ssd_load_rows(p.act, p.ld, p.aligned, sBl, ldn, p.n16, d.N, cb + d.lo, q0, t0, len);
-    }
-    ssd_load_rows(p.x, p.ldx, p.aligned_x, sX, kLdX, kSlice, pw, cx, q0, t0, len);
+    ssd_load_rows<NT>(threadIdx.x, p.act, p.ld, p.aligned, sC, ldn, p.n16, d.N, cc, q0, t0, len);
+    if (SPLIT) ssd_load_rows<NT>(threadIdx.x, p.act, p.ld, p.aligned, sCl, ldn, p.n16, d.N, cc + d.lo, q0, t0, len);
+    ssd_load_rows<128>(gt, p.x, p.ldx, p.aligned_x, sX + (ch & 1) * tile_x, kLdX, kSlice, pw, cx, q0, t0, len);
     if (CHANNEL) {
-      ssd_load_rows(p.score, 2ll * kChunk * d.H, true, sA, kLdA, kChunk, kChunk, h * 2 * kChunk, q0, t0, len);
-      ssd_load_rows(p.score, 2ll * kChunk * d.H, true, sA + kChunk * kLdA, kLdA, kChunk, kChunk, (h * 2 + 1) * kChunk, q0, t0, len);
-      const long long block = p.c_start[seq] / kChunk + seq + ch;
-      for (int n = threadIdx.x; n < p.n16; n += 128) sLd[n] = p.block_decay[(block * d.H + h) * d.NB + n];
+      ssd_load_rows<NT>(threadIdx.x, p.score, 2ll * kChunk * d.H, true, sA, kLdA, kChunk, kChunk, h * 2 * kChunk, q0, t0, len);
+      ssd_load_rows<NT>(threadIdx.x, p.score, 2ll * kChunk * d.H, true, sA + kChunk * kLdA, kLdA, kChunk, kChunk, (h * 2 + 1) * kChunk, q0,
+                        t0, len);
     } else if (threadIdx.x < kChunk) {
       const bool ok = t0 + static_cast<int>(threadIdx.x) < len;
       sDt[threadIdx.x] = ok ? (p.dt ? p.dt[(q0 + t0 + threadIdx.x) * d.H + h] : 1.f) : 0.f;
@@ -317,7 +319,18 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
     }
     ms_commit();
   };
-  load_chunk(ch0);
+  auto load_b = [&](int ch) {
+    const int t0 = ch * kChunk;
+    ssd_load_rows<NT>(threadIdx.x, p.act, p.ld, p.aligned, sB, ldn, p.n16, d.N, cb, q0, t0, len);
+    if (SPLIT) ssd_load_rows<NT>(threadIdx.x, p.act, p.ld, p.aligned, sBl, ldn, p.n16, d.N, cb + d.lo, q0, t0, len);
+    if (CHANNEL) {
+      const long long block = p.c_start[seq] / kChunk + seq + ch;
+      for (int n = threadIdx.x; n < p.n16; n += NT) sLd[n] = p.block_decay[(block * d.H + h) * d.NB + n];
+    }
+    ms_commit();
+  };
+  load_c(ch0);
+  load_b(ch0);
 
   // this warp's rows of the state at the start of the segment, accumulator layout
   float S[NI][4][4];
@@ -378,13 +391,16 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
     }
   };
   publish();
-  const uint32_t aC = ms_addr(sC), aB = ms_addr(sB), aX = ms_addr(sX), aSh = ms_addr(sSh), aSl = ms_addr(sSl);
+  const uint32_t aC = ms_addr(sC), aB = ms_addr(sB), aSh = ms_addr(sSh), aSl = ms_addr(sSl);
   const uint32_t aCl = ms_addr(sCl), aBl = ms_addr(sBl);
   const int r0 = warp * 16;
 
   for (int ch = ch0; ch < ch1; ++ch) {
-    ms_wait<0>();
-    __syncthreads();                       // the block's rows and the published state are visible
+    if (CHANNEL) ms_wait<1>();
+    else ms_wait<0>();
+    __syncthreads();                       // the block's rows (CHANNEL: without B) and the published state are visible
+    const __nv_bfloat16* sXb = sX + (ch & 1) * tile_x;
+    const uint32_t aX = ms_addr(sXb);
     float total = 0.f;
     if (!CHANNEL) total = ssd_decays(sDt, MEMORY ? sLd : nullptr, a2, cum, wgt, lane);
     float s[8][4], yi[4][4], y[4][4], rows[2] = {0.f, 0.f};
@@ -478,20 +494,20 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
     const float ei[2] = {exp2f(ci[0]), exp2f(ci[1])};
     const int t0 = ch * kChunk;
     if (norm) {                            // n . c of the rows: the block's part from the scores, the rest from the normaliser at its start
-      float own = 0.f;
+      float at_start = 0.f;
       const int per = p.n16 / 2, from = (lane >> 4) * per;
       for (int k = from; k < from + per; k += 8) {
         float v[8];
         load_vec<8>(sC + (r0 + (lane & 15)) * ldn + k, v);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) own = fmaf(v[e], sN[k + e], own);
+        for (int e = 0; e < 8; ++e) at_start = fmaf(v[e], sN[k + e], at_start);
       }
-      own += __shfl_xor_sync(0xffffffffu, own, 16);
+      at_start += __shfl_xor_sync(0xffffffffu, at_start, 16);
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
         rows[hf] += __shfl_xor_sync(0xffffffffu, rows[hf], 1);
         rows[hf] += __shfl_xor_sync(0xffffffffu, rows[hf], 2);
-        const float nq = fmaf(ei[hf], __shfl_sync(0xffffffffu, own, g4 + 8 * hf), rows[hf]) * p.yscale;
+        const float nq = fmaf(ei[hf], __shfl_sync(0xffffffffu, at_start, g4 + 8 * hf), rows[hf]) * p.yscale;
         const int i = r0 + g4 + 8 * hf;
         if (t4 == 0 && t0 + i < len) {
           const long long at = (q0 + t0 + i) * d.H + h;
@@ -505,7 +521,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
       for (int hf = 0; hf < 2; ++hf) {
         const int i = r0 + g4 + 8 * hf, c = nt * 8 + 2 * t4;
         if (t0 + i >= len || c >= pw) continue;
-        const float2 xf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + i * kLdX + c));
+        const float2 xf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sXb + i * kLdX + c));
         float v0 = fmaf(skip, xf.x, fmaf(ei[hf], yi[nt][2 * hf], y[nt][2 * hf]));
         float v1 = fmaf(skip, xf.y, fmaf(ei[hf], yi[nt][2 * hf + 1], y[nt][2 * hf + 1]));
         if (MEMORY) {
@@ -520,6 +536,9 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
           if (c + 1 < pw) dst[1] = __float2bfloat16(v1);
         }
       }
+    if (CHANNEL) ms_wait<0>();
+    __syncthreads();                       // C, scores and steps have been read; CHANNEL: B is visible
+    if (ch + 1 < ch1) load_c(ch + 1);
     float nv[2] = {0.f, 0.f};
     if (ch + 1 < ch1 || ch1 == n_chunks) {
       ssd_update<NI, SPLIT, CHANNEL>(S, exp2f(total), sLd, wgt, aB, aBl, aX, ldn, p.n16, warp, lane);
@@ -530,13 +549,13 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
         ssd_norm_add(nv, exp2f(total), wgt, sB, ldn, d.N);
       }
     }
-    __syncthreads();                       // everyone has read this block's rows and the published state
+    __syncthreads();                       // everyone has read B and the published state
     if (norm && (ch + 1 < ch1 || ch1 == n_chunks))
 #pragma unroll
       for (int i = 0; i < 2; ++i)
         if (static_cast<int>(threadIdx.x) + 128 * i < d.N) sN[threadIdx.x + 128 * i] = nv[i];
     if (ch + 1 < ch1) {
-      load_chunk(ch + 1);
+      load_b(ch + 1);
       publish();
     }
   }
@@ -549,35 +568,69 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const SsdParams p) {
   }
 }
 
-template <int NI, bool SPLIT, int KIND>
-static int ssd_launch_as(const SsdParams& p, dim3 grid, cudaStream_t st) {
+static size_t ssd_bytes(const SsdParams& p, bool split, int kind, int wg) {
   const size_t tile_n = static_cast<size_t>(kChunk) * (p.n16 + 8), tile_x = static_cast<size_t>(kChunk) * kLdX;
-  const size_t scores = KIND == kSsdChannel ? 2 * static_cast<size_t>(kChunk) * kLdA : 0;
-  const size_t more = KIND == kSsdPlain ? 0 : (KIND == kSsdMemory ? kChunk + p.n16 : p.n16), more_seg = KIND == kSsdPlain ? 0 : 2 * (KIND == kSsdMemory ? kChunk : p.n16);
-  const size_t smem = ((SPLIT ? 4 : 2) * tile_n + tile_x + 2 * static_cast<size_t>(p.n16) * kLdX + scores) * 2 + (9 * kChunk + more) * 4;
-  const size_t smem_seg = ((SPLIT ? 4 : 2) * tile_n + 2 * tile_x) * 2 + (10 * kChunk + more_seg) * 4;
-  if (smem > 224 * 1024 || smem_seg > 224 * 1024) return -4;
+  const size_t scores = kind == kSsdChannel ? 2 * static_cast<size_t>(kChunk) * kLdA : 0;
+  const size_t more = kind == kSsdPlain ? 0 : (kind == kSsdMemory ? kChunk + p.n16 : p.n16);
+  return ((split ? 4 : 2) * tile_n + wg * (2 * tile_x + 2 * static_cast<size_t>(p.n16) * kLdX) + scores) * 2 + ((1 + 8 * wg) * kChunk + more) * 4;
+}
+static size_t ssd_bytes_segment(const SsdParams& p, bool split, int kind, int wg) {
+  const size_t tile_n = static_cast<size_t>(kChunk) * (p.n16 + 8), tile_x = static_cast<size_t>(kChunk) * kLdX;
+  const size_t more = kind == kSsdPlain ? 0 : 2 * (kind == kSsdMemory ? kChunk : p.n16);
+  return ((split ? 4 : 2) * tile_n + wg * 2 * tile_x) * 2 + ((2 + 8 * wg) * kChunk + more) * 4;
+}
+constexpr size_t kSsdSmem = 224 * 1024;
+
+template <int NI, bool SPLIT, int KIND, int WG>
+static int ssd_launch_as(const SsdParams& p, dim3 grid, cudaStream_t st) {
+  const size_t smem = ssd_bytes(p, SPLIT, KIND, WG), smem_seg = ssd_bytes_segment(p, SPLIT, KIND, WG);
+  if (smem > kSsdSmem || smem_seg > kSsdSmem) return -4;
   static DeviceOnce once;
   if (once.pending()) {
-    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NI, SPLIT, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NI, SPLIT, KIND, WG>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSsdSmem);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(ssd_segment_kernel<NI, SPLIT, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+      e = cudaFuncSetAttribute(ssd_segment_kernel<NI, SPLIT, KIND, WG>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSsdSmem);
     if (e != cudaSuccess) return static_cast<int>(e);
     once.mark();
   }
   if (p.n_seg > 1) {
-    ssd_segment_kernel<NI, SPLIT, KIND><<<grid, 128, smem_seg, st>>>(p);
+    ssd_segment_kernel<NI, SPLIT, KIND, WG><<<grid, 128 * WG, smem_seg, st>>>(p);
     const cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  ssd_chunk_kernel<NI, SPLIT, KIND><<<grid, 128, smem, st>>>(p);
+  ssd_chunk_kernel<NI, SPLIT, KIND, WG><<<grid, 128 * WG, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <bool SPLIT, int KIND>
-static int ssd_launch_any(const SsdParams& p, dim3 grid, cudaStream_t st) {
-  return p.n16 <= 64 ? ssd_launch_as<1, SPLIT, KIND>(p, grid, st)
-                     : (p.n16 <= 128 ? ssd_launch_as<2, SPLIT, KIND>(p, grid, st) : ssd_launch_as<4, SPLIT, KIND>(p, grid, st));
+static int ssd_launch_any(SsdParams p, int n_seq, int n_chunks, int max_seg, cudaStream_t st) {
+  // groups of warps on the same B and C: as many as there are slices, while registers and shared memory last
+  const int slices = (p.P + kSlice - 1) / kSlice;
+  int wg = 1;
+  if (KIND != kSsdPlain) {
+    wg = slices >= 3 ? 4 : slices;
+    if (p.n16 > 128 && wg > 2) wg = 2;
+    while (wg > 1 && ssd_bytes(p, SPLIT, KIND, wg) > kSsdSmem) wg /= 2;
+  }
+  // enough CTAs to keep three single groups on every SM for a few rounds, or one of several for a round
+  const int ctas = (slices + wg - 1) / wg;
+  const long long base = static_cast<long long>(ctas) * p.H * n_seq, rounds = wg == 1 ? 6 : (wg == 2 ? 2 : 1);
+  long long want = wg == 1 ? (rounds * num_sms() + base - 1) / base : rounds * num_sms() / base;
+  if (want < 1) want = 1;
+  if (want > max_seg) want = max_seg;
+  if (want > n_chunks) want = n_chunks;
+  p.seg_chunks = (n_chunks + static_cast<int>(want) - 1) / static_cast<int>(want);
+  p.n_seg = (n_chunks + p.seg_chunks - 1) / p.seg_chunks;
+  const dim3 grid(ctas * p.n_seg, p.H, n_seq);
+  if constexpr (KIND != kSsdPlain) {
+    if (wg == 4)
+      return p.n16 <= 64 ? ssd_launch_as<1, SPLIT, KIND, 4>(p, grid, st) : ssd_launch_as<2, SPLIT, KIND, 4>(p, grid, st);
+    if (wg == 2)
+      return p.n16 <= 64 ? ssd_launch_as<1, SPLIT, KIND, 2>(p, grid, st)
+                         : (p.n16 <= 128 ? ssd_launch_as<2, SPLIT, KIND, 2>(p, grid, st) : ssd_launch_as<4, SPLIT, KIND, 2>(p, grid, st));
+  }
+  return p.n16 <= 64 ? ssd_launch_as<1, SPLIT, KIND, 1>(p, grid, st)
+                     : (p.n16 <= 128 ? ssd_launch_as<2, SPLIT, KIND, 1>(p, grid, st) : ssd_launch_as<4, SPLIT, KIND, 1>(p, grid, st));
 }
 
 int ssd_chunk_launch(SsdParams p, int n_seq, int max_q, int max_seg, cudaStream_t st) {
@@ -592,18 +645,11 @@ int ssd_chunk_launch(SsdParams p, int n_seq, int max_q, int max_seg, cudaStream_
   const auto whole = [](const void* a) { return reinterpret_cast<uintptr_t>(a) % 16 == 0; };
   p.aligned = p.ld % 8 == 0 && p.b0 % 8 == 0 && p.c0 % 8 == 0 && p.lo % 8 == 0 && p.N % 8 == 0 && p.NB % 8 == 0 && whole(p.act);
   p.aligned_x = p.ldx % 8 == 0 && p.P % 8 == 0 && whole(p.x);
-  // enough CTAs to keep three on every SM for a few rounds
-  const int slices = (p.P + kSlice - 1) / kSlice, n_chunks = (max_q + kChunk - 1) / kChunk;
-  const long long base = static_cast<long long>(slices) * p.H * n_seq;
-  long long want = (6ll * num_sms() + base - 1) / base;
-  if (want > max_seg) want = max_seg;
-  if (want > n_chunks) want = n_chunks;
-  p.seg_chunks = (n_chunks + static_cast<int>(want) - 1) / static_cast<int>(want);
-  p.n_seg = (n_chunks + p.seg_chunks - 1) / p.seg_chunks;
-  const dim3 grid(slices * p.n_seg, p.H, n_seq);
-  if (p.kind == kSsdMemory) return ssd_launch_any<false, kSsdMemory>(p, grid, st);
-  if (p.kind == kSsdChannel) return ssd_launch_any<true, kSsdChannel>(p, grid, st);
-  return p.lo > 0 ? ssd_launch_any<true, kSsdPlain>(p, grid, st) : ssd_launch_any<false, kSsdPlain>(p, grid, st);
+  const int n_chunks = (max_q + kChunk - 1) / kChunk;
+  if (p.kind == kSsdMemory) return ssd_launch_any<false, kSsdMemory>(p, n_seq, n_chunks, max_seg, st);
+  if (p.kind == kSsdChannel) return ssd_launch_any<true, kSsdChannel>(p, n_seq, n_chunks, max_seg, st);
+  return p.lo > 0 ? ssd_launch_any<true, kSsdPlain>(p, n_seq, n_chunks, max_seg, st)
+                  : ssd_launch_any<false, kSsdPlain>(p, n_seq, n_chunks, max_seg, st);
 }
 
 }  // namespace pm
