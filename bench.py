@@ -153,7 +153,7 @@ def main() -> None:
     ap.add_argument("--serve-hybrid", nargs="*", metavar="PRESET", default=None,
                     help="instead of the headline benchmark: prefill / decode throughput and kernel times of the hybrid "
                          "decoder presets (default duvivik-1b duvivik-2b; also resevik-1b, resevik-2b, vosezen-1b, "
-                         "vosezen-2b) beside the closest other model of equal size")
+                         "vosezen-2b, ravapel-1b, ravapel-2b) beside the closest other model of equal size")
     args = ap.parse_args()
     if args.serve_hybrid is not None:
         from pmetal_b200.bench.hybrid_serve import report

@@ -31,7 +31,7 @@ COMPONENTS = {
                 "ssd_chunk", "window_attn"),
     "vosezen": ("attention_tc", "gemm_2sm", "gemm_tcgen05", "gemv", "grouped_gemm", "latent_attn", "moe_experts", "moe_quant",
                 "postnorm", "window_attn"),
-    "ravapel": ("attention_tc", "gated_linear", "gemm_2sm", "gemm_tcgen05", "gemv", "linear_attn", "moe_experts", "postnorm", "sandwich", "ssd_chunk",
+    "ravapel": ("attention_tc", "gated_linear", "gemm_2sm", "gemm_tcgen05", "gemv", "linear_attn", "postnorm", "sandwich", "ssd_chunk",
                 "window_attn"),
     "decoder": ("attention", "attention_tc", "decode_mega", "elementwise", "gemm_2sm", "gemm_tcgen05", "gemv",
                 "grouped_gemm", "moe_quant"),

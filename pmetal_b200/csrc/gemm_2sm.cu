@@ -262,8 +262,9 @@ extern "C" int pm_gemm_bf16_2sm(const void* A, int a_mn, int lda, int a_rows, co
                                 int b_rows, const void* A2, int a2_mn, int lda2, int a2_k, const void* B2, int b2_mn,
                                 int ldb2, int b2_rows, void* D, int out_mode, int ldd, const void* R, int ldr, int M,
                                 int N, int K, int K2, int n_store, float alpha, int splits, int seg_mode,
-                                const int* seg_end, int seg_r, int max_ctas, int* status,
-                                cudaStream_t stream) {
+                                const int* seg_end, int seg_r, int max_ctas, float* tail, int tail_from, int ld_tail,
+                                int* status, cudaStream_t stream) {
+  if (tail && (out_mode != 0 || R || tail_from % 8 || (reinterpret_cast<uintptr_t>(tail) & 15))) return -20;
   if (splits < 1 || (splits > 1 && (out_mode < 2 || out_mode > 3))) return -12;   // split-K needs the atomic modes
   if (M <= 0 || N <= 0 || K <= 0) return -13;
   if (out_mode == 0 && ((ldd % 8) || (reinterpret_cast<uintptr_t>(D) & 15))) return -14;
@@ -279,6 +280,7 @@ extern "C" int pm_gemm_bf16_2sm(const void* A, int a_mn, int lda, int a_rows, co
   p.seg_mode = seg_mode; p.seg_r = seg_r;
   for (int i = 0; i < 4; ++i) p.seg_end[i] = (seg_mode && seg_end) ? seg_end[i] : 0x7fffffff;
   p.status = status;
+  p.tail = tail; p.tail_from = tail_from; p.ld_tail = ld_tail;
   p.kps = 2;
   p.commit_both = 0;
   p.fwd_full = 0;

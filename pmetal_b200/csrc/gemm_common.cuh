@@ -37,6 +37,8 @@ struct GemmParams {
   int* status;
   float* ws;             // out_mode 6: [tiles][splits][128][bn] fp32 partial tiles
   unsigned* ws_cnt;      // out_mode 6: [tiles][4] arrival counters, zero between launches
+  float* tail;           // out_mode 0 / 6, nullable: columns from tail_from (a multiple of 8) on go here in fp32, rows ld_tail apart
+  int tail_from, ld_tail;
 };
 
 __device__ __forceinline__ int seg_of(const GemmParams& p, int x) {
@@ -56,6 +58,21 @@ __device__ __forceinline__ void epilogue_store_chunk(const GemmParams& p, const 
 #pragma unroll
       for (int v = 0; v < 4; ++v) {
         const int col = col0 + v * 8;
+        if (p.tail && col >= p.tail_from) {
+          float* trow = p.tail + static_cast<size_t>(row) * p.ld_tail + col - p.tail_from;
+          if (col + 8 <= p.n_store && p.ld_tail % 4 == 0) {
+#pragma unroll
+            for (int e = 0; e < 8; e += 4)
+              *reinterpret_cast<float4*>(trow + e) =
+                  make_float4(__uint_as_float(r[v * 8 + e]) * p.alpha, __uint_as_float(r[v * 8 + e + 1]) * p.alpha,
+                              __uint_as_float(r[v * 8 + e + 2]) * p.alpha, __uint_as_float(r[v * 8 + e + 3]) * p.alpha);
+          } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+              if (col + e < p.n_store) trow[e] = __uint_as_float(r[v * 8 + e]) * p.alpha;
+          }
+          continue;
+        }
         if (col + 8 <= p.n_store) {
           float f[8];
 #pragma unroll
@@ -85,9 +102,16 @@ __device__ __forceinline__ void epilogue_store_chunk(const GemmParams& p, const 
       }
     } else if (p.out_mode == 1) {
       float* drow = static_cast<float*>(p.D) + static_cast<size_t>(row) * p.ldd;
+      if (col0 + 32 <= p.n_store && p.ldd % 4 == 0 && (reinterpret_cast<uintptr_t>(p.D) & 15) == 0) {
 #pragma unroll
-      for (int e = 0; e < 32; ++e)
-        if (col0 + e < p.n_store) drow[col0 + e] = __uint_as_float(r[e]) * p.alpha;
+        for (int e = 0; e < 32; e += 4)
+          *reinterpret_cast<float4*>(drow + col0 + e) = make_float4(__uint_as_float(r[e]) * p.alpha, __uint_as_float(r[e + 1]) * p.alpha,
+                                                                    __uint_as_float(r[e + 2]) * p.alpha, __uint_as_float(r[e + 3]) * p.alpha);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 32; ++e)
+          if (col0 + e < p.n_store) drow[col0 + e] = __uint_as_float(r[e]) * p.alpha;
+      }
     } else if (p.out_mode == 2) {
       float* drow = static_cast<float*>(p.D) + static_cast<size_t>(row) * p.ldd;
 #pragma unroll

@@ -256,12 +256,14 @@ using namespace pm;
 
 // Returns 0 on success, negative on argument / descriptor errors, or the CUDA error code.
 //   a_rows/b_rows: extent of the operand along M / N as seen by the tensor map (rows beyond it read as zero).
+//   tail (nullable, bf16 output without R): columns from tail_from (a multiple of 8) on go there in fp32, rows ld_tail apart.
 extern "C" int pm_gemm_bf16(const void* A, int a_mn, int lda, int a_rows, const void* B, int b_mn, int ldb, int b_rows,
                             const void* A2, int a2_mn, int lda2, int a2_k, const void* B2, int b2_mn, int ldb2,
                             int b2_rows, void* D, int out_mode, int ldd, const void* R, int ldr, int M, int N, int K,
                             int K2, int n_store, float alpha, int bn, int splits, int seg_mode, const int* seg_end,
                             int seg_r, int max_ctas, float* ws, long long ws_floats, unsigned* ws_cnt,
-                            long long ws_cnt_len, int* status, cudaStream_t stream) {
+                            long long ws_cnt_len, float* tail, int tail_from, int ld_tail, int* status, cudaStream_t stream) {
+  if (tail && ((out_mode != 0 && out_mode != 6) || R || tail_from % 8 || (reinterpret_cast<uintptr_t>(tail) & 15))) return -20;
   if (bn != 32 && bn != 64 && bn != 128 && bn != 256) return -10;
   if ((b_mn || (K2 > 0 && b2_mn)) && (bn % 64)) return -11;
   // split-K needs the atomic modes, or mode 6 with its workspace (every split must own at least one K block)
@@ -290,6 +292,7 @@ extern "C" int pm_gemm_bf16(const void* A, int a_mn, int lda, int a_rows, const 
   for (int i = 0; i < 4; ++i) p.seg_end[i] = (seg_mode && seg_end) ? seg_end[i] : 0x7fffffff;
   p.status = status;
   p.ws = ws; p.ws_cnt = ws_cnt;
+  p.tail = tail; p.tail_from = tail_from; p.ld_tail = ld_tail;
   const int stage_bytes = kBM * kBK * 2 + bn * kBK * 2;
   int stages = (227 * 1024 - 2048) / stage_bytes;
   if (stages > kMaxStages) stages = kMaxStages;

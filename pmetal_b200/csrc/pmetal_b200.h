@@ -188,7 +188,8 @@ int pm_gdn_scan(const float* q, const float* k, const float* v, const float* g, 
 int pm_gemm_bf16_2sm(const void* A, int a_mn, int lda, int a_rows, const void* B, int b_mn, int ldb, int b_rows,
     const void* A2, int a2_mn, int lda2, int a2_k, const void* B2, int b2_mn, int ldb2, int b2_rows, void* D, int
     out_mode, int ldd, const void* R, int ldr, int M, int N, int K, int K2, int n_store, float alpha, int splits,
-    int seg_mode, const int* seg_end, int seg_r, int max_ctas, int* status, cudaStream_t stream);
+    int seg_mode, const int* seg_end, int seg_r, int max_ctas, float* tail, int tail_from, int ld_tail, int*
+    status, cudaStream_t stream);
 
 // ---------------------------------------------------------------- gemm_q4_2sm.cu
 // A [M, K] bf16 (K-major). codes: packed weight [w_rows, w_cols / 2] bytes, first element of a pair in the high nibble;
@@ -205,11 +206,12 @@ int pm_gemm_q4_2sm(const void* A, int lda, int a_rows, const void* codes, const 
 // ---------------------------------------------------------------- gemm_tcgen05.cu
 // Returns 0 on success, negative on argument / descriptor errors, or the CUDA error code.
 //   a_rows/b_rows: extent of the operand along M / N as seen by the tensor map (rows beyond it read as zero).
+//   tail (nullable, bf16 output without R): columns from tail_from (a multiple of 8) on go there in fp32, rows ld_tail apart.
 int pm_gemm_bf16(const void* A, int a_mn, int lda, int a_rows, const void* B, int b_mn, int ldb, int b_rows, const
     void* A2, int a2_mn, int lda2, int a2_k, const void* B2, int b2_mn, int ldb2, int b2_rows, void* D, int
     out_mode, int ldd, const void* R, int ldr, int M, int N, int K, int K2, int n_store, float alpha, int bn, int
     splits, int seg_mode, const int* seg_end, int seg_r, int max_ctas, float* ws, long long ws_floats, unsigned*
-    ws_cnt, long long ws_cnt_len, int* status, cudaStream_t stream);
+    ws_cnt, long long ws_cnt_len, float* tail, int tail_from, int ld_tail, int* status, cudaStream_t stream);
 
 // ---------------------------------------------------------------- gemv.cu
 // As pm_gemv with the epilogue of models that have biases and clamped gated units: bias [N_w] fp32 (nullable) is added to

@@ -662,12 +662,12 @@ def project_f32(x: torch.Tensor, w: torch.Tensor, n: int) -> torch.Tensor:
 
 def project_mixed(x: torch.Tensor, w: torch.Tensor, n_low: int):
     """(x w[:n_low]^T in x's type, x w[n_low:]^T in fp32): activations and the logits of gates from one stacked weight."""
-    if x.dtype != torch.bfloat16 or w.shape[1] % 8 or n_low % 8 or x.stride(0) % 8 or not use_native(x):
+    if x.dtype != torch.bfloat16 or w.shape[1] % 8 or w.shape[0] % 8 or n_low % 8 or x.stride(0) % 8 or not use_native(x):
         return F.linear(x, w[:n_low]), F.linear(x.float(), w[n_low:].float())
     nat = _native()
     if gemv_fits(x.shape[0], x.shape[1]):
         return nat.gemv_ex(x, w, f32_from=n_low)
-    return nat.gemm(x, w[:n_low]), router_logits(x, w[n_low:], w.shape[0] - n_low)
+    return nat.gemm_mixed(x, w, n_low)
 
 
 def router_logits(x: torch.Tensor, w: torch.Tensor, n: int) -> torch.Tensor:

@@ -173,8 +173,8 @@ def _seg_ends(seg_sizes: Sequence[int]):
 
 def raw_gemm(A, a_mn, lda, a_rows, B, b_mn, ldb, b_rows, D, out_mode, ldd, M, N, K, *, A2=None, a2_mn=0, lda2=0,
              a2_k=0, B2=None, b2_mn=0, ldb2=0, b2_rows=0, K2=0, R=None, ldr=0, n_store=0, alpha=1.0, bn=128, splits=1,
-             seg_mode=0, seg_sizes=(), seg_r=0, max_ctas=0) -> None:
-    """One GEMM launch. 256-wide tiles on at least 256 rows go to the CTA-pair (cta_group::2) kernel."""
+             seg_mode=0, seg_sizes=(), seg_r=0, max_ctas=0, tail=None, tail_from=0) -> None:
+    """One GEMM launch; ``tail`` (fp32) takes the columns from ``tail_from`` on. 256-wide tiles on at least 256 rows go to the CTA-pair (cta_group::2) kernel."""
     segs = _seg_ends(seg_sizes) if seg_mode else None
     if USE_2SM and bn == 256 and M >= 256 and (seg_mode != 2 or all(s % 256 == 0 for s in seg_sizes[:-1])):
         rc = lib().pm_gemm_bf16_2sm(_p(A), c_int(a_mn), c_int(lda), c_int(a_rows), _p(B), c_int(b_mn), c_int(ldb),
@@ -182,7 +182,8 @@ def raw_gemm(A, a_mn, lda, a_rows, B, b_mn, ldb, b_rows, D, out_mode, ldd, M, N,
                                     c_int(b2_mn), c_int(ldb2), c_int(b2_rows), _p(D), c_int(out_mode), c_int(ldd),
                                     _p(R), c_int(ldr), c_int(M), c_int(N), c_int(K), c_int(K2), c_int(n_store),
                                     c_float(alpha), c_int(splits), c_int(seg_mode), segs, c_int(seg_r),
-                                    c_int(max_ctas), _p(status_word(D.device)), _stream())
+                                    c_int(max_ctas), _p(tail), c_int(tail_from), c_int(tail.stride(0) if tail is not None else 0),
+                                    _p(status_word(D.device)), _stream())
         _chk(rc, "pm_gemm_bf16_2sm")
         return
     ws = cnt = None
@@ -205,7 +206,8 @@ def raw_gemm(A, a_mn, lda, a_rows, B, b_mn, ldb, b_rows, D, out_mode, ldd, M, N,
                             c_int(M), c_int(N), c_int(K), c_int(K2), c_int(n_store), c_float(alpha), c_int(bn),
                             c_int(splits), c_int(seg_mode), segs, c_int(seg_r), c_int(max_ctas), _p(ws),
                             ctypes.c_longlong(ws.numel() if ws is not None else 0), _p(cnt),
-                            ctypes.c_longlong(cnt.numel() if cnt is not None else 0), _p(status_word(D.device)), _stream())
+                            ctypes.c_longlong(cnt.numel() if cnt is not None else 0), _p(tail), c_int(tail_from),
+                            c_int(tail.stride(0) if tail is not None else 0), _p(status_word(D.device)), _stream())
     _chk(rc, "pm_gemm_bf16")
 
 
@@ -476,14 +478,27 @@ def grouped_gemm_skinny(x: torch.Tensor, w: torch.Tensor, off: torch.Tensor, swi
 
 # ------------------------------------------------------------------------------------------- hyper-connections
 def gemm_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """[M, K] x [N, K]^T -> [M, N padded to a multiple of 32] fp32 (extra columns are zero)."""
+    """[M, K] x [N, K]^T -> [M, N padded to the tile's width] fp32 (extra columns are zero)."""
     M, K = x.shape
     N = w.shape[0]
-    bn = 32 if N <= 32 else (64 if N <= 64 else 128)
+    if M <= 128:                            # a single row block: narrow tiles spread the columns over the machine
+        bn = _pick_bn(N, (), M)
+    else:
+        bn = 32 if N <= 32 else 64 if N <= 64 else 256 if M >= 256 and N % 256 == 0 else 128
     Np = -(-N // bn) * bn
-    out = torch.zeros(M, Np, dtype=torch.float32, device=x.device)
+    out = torch.empty(M, Np, dtype=torch.float32, device=x.device)
     raw_gemm(x, 0, x.stride(0), M, w, 0, w.stride(0), N, out, 1, Np, M, Np, K, bn=bn)
     return out
+
+
+def gemm_mixed(x: torch.Tensor, w: torch.Tensor, n_low: int):
+    """[M, K] x [N, K]^T -> ([M, n_low] bf16, [M, N - n_low] fp32); n_low a multiple of 8."""
+    M, K = x.shape
+    N = w.shape[0]
+    out = torch.empty(M, n_low, dtype=torch.bfloat16, device=x.device)
+    tail = torch.empty(M, N - n_low, dtype=torch.float32, device=x.device)
+    raw_gemm(x, 0, x.stride(0), M, w, 0, w.stride(0), N, out, 0, n_low, M, N, K, bn=_pick_bn(N, (), M), tail=tail, tail_from=n_low)
+    return out, tail
 
 
 def mhc_mappings(x, raw, bias, alpha, iters: int):
