@@ -22,6 +22,7 @@ from ..models.kv_cache import BLOCK, PagedKVCache
 from ..models.mixers import RotationFreqs, StepContext
 from ..models.state_cache import CacheSpec, StateCache, attention_runs, split_groups
 from ..ops import native as nat
+from ..utils.graphs import capture
 from .kernels import peaks
 
 # dense models of the fast path with about the same width, depth of weights and parameter count
@@ -146,7 +147,7 @@ def graph_us(fn: Callable[[], None], iters: int = 15) -> float:
     torch.cuda.current_stream().wait_stream(side)
     torch.cuda.synchronize()
     g = torch.cuda.CUDAGraph()
-    with torch.cuda.graph(g):
+    with capture(g):
         fn()
     ts = []
     for _ in range(iters + 3):

@@ -15,6 +15,7 @@ from typing import Callable, Iterator, List, Optional, Sequence
 
 import torch
 
+from ..utils.graphs import capture
 from .kv_cache import BLOCK, BatchMeta, PagedKVCache
 from .sampling import Sampler, SamplingParams
 
@@ -123,7 +124,7 @@ class GraphedDecoder:
         torch.cuda.current_stream().wait_stream(side)
         torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
+        with capture(g):
             st["logits"] = self.model.forward_paged(st["tokens"], self.cache, st["meta"])
         st["graph"] = g
         self.graphs[key] = st

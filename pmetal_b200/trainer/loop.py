@@ -134,8 +134,9 @@ class TrainingLoop:
         torch.cuda.synchronize()
         self._graph = torch.cuda.CUDAGraph()
         from ..ops import native
+        from ..utils.graphs import capture
         n0 = native.LAUNCHES
-        with torch.cuda.graph(self._graph):
+        with capture(self._graph):
             loss = self.micro_step(self._g_in)
             gn = self.optimizer_step()
         self.launches_per_graph = native.LAUNCHES - n0

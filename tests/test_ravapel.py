@@ -784,6 +784,32 @@ def test_long_decoding_in_a_batch(dtype, graphs):
         assert worst(torch.stack([g[j] for g in got]), oracle("mixed", r)[-170:], limits("mixed", r, dtype)[-170:]) < 1
 
 
+@gpu
+def test_captures_survive_discarded_graphs():
+    """A graph that becomes garbage (in a reference cycle) while another one is captured is freed behind the capture."""
+    import gc
+    from pmetal_b200.utils.graphs import capture
+
+    class Owner:
+        pass
+
+    x = torch.ones(4, device="cuda")
+    torch.cuda.synchronize()
+    old = Owner()
+    old.graph, old.self = torch.cuda.CUDAGraph(), old
+    with capture(old.graph):
+        x + 1
+    new = torch.cuda.CUDAGraph()
+    with capture(new):
+        del old
+        [[] for _ in range(200000)]                          # enough objects for several automatic collections
+        y = x * 3
+    assert gc.isenabled()
+    new.replay()
+    gc.collect()
+    assert y.tolist() == [3.0] * 4
+
+
 def _greedy(name, prompt, n):
     seq = list(prompt)
     for _ in range(n):
